@@ -117,6 +117,8 @@ def test_random_cases_against_the_compiled_reference(pkg):
         ref = binding.load_ref()
     except Exception as e:                                           # noqa: BLE001
         pytest.skip(f"compiled reference not available: {e}")
+    if ref is None:
+        pytest.skip("compiled reference not built here")
     rng = np.random.default_rng(5)
     for case in range(150):
         alpha = [bytes([c]) for c in rng.choice(np.arange(97, 123), size=int(rng.integers(2, 6)), replace=False)]
