@@ -2,7 +2,12 @@
 host/*.c with gcc -std=c11, linked into one shared library that exports the cmlb200 C-ABI
 and the C-ML-compatible host API -- exactly the functions and variables the two public headers
 declare (a linker version script generated from include/*.h hides everything else).
-Incremental (mtime based). No GPU is needed to build."""
+Incremental (mtime based). No GPU is needed to build.
+
+The programs under programs/ become executables in lib/. cml_generate links the library's objects; trace_run
+links only what a model folder needs, so that a fresh checkout compiles a few files.
+
+  build.py [-v] [--program NAME]"""
 import os
 import re
 import shutil
@@ -76,25 +81,56 @@ def _version_script() -> Path:
     return path
 
 
-def build(verbose: bool = False) -> Path:
+# Sources of the programs besides their own; None: everything the library holds.
+PROGRAMS = {
+    "trace_run": ["host/cml_json.c", "host/cml_safetensors.c", "host/cml_lm.c", "host/cml_lm_layered.c", "host/cml_paged.c", "host/cml_serving.c",
+                  "host/cml_sampling.c", "host/cml_tensor.c", "host/cml_tokenizer.c", "csrc/shim.cu", "csrc/argmax.cu",
+                  "csrc/lm_rows.cu", "csrc/attention_rows.cu", "csrc/gemv_bf16.cu", "csrc/gemm_bf16.cu", "csrc/llm_ops_f32.cu", "csrc/paged_attention.cu"],
+    "cml_generate": None,
+}
+LINK_LIBS = ["-lcudart_static", "-ldl", "-lpthread", "-lrt", "-lm"]
+
+
+def _library_sources():
+    return sorted((PKG / "csrc").glob("*.cu")) + sorted((PKG / "csrc").glob("*.c")) + sorted((PKG / "host").glob("*.c"))
+
+
+def _compile_all(srcs, verbose):
     OBJ.mkdir(parents=True, exist_ok=True)
-    srcs = sorted((PKG / "csrc").glob("*.cu")) + sorted((PKG / "csrc").glob("*.c")) + sorted((PKG / "host").glob("*.c"))
     with ThreadPoolExecutor(max_workers=min(8, len(srcs))) as ex:
         results = list(ex.map(lambda s: _compile(s, verbose), srcs))
-    objs = [o for o, _ in results]
-    if verbose:
-        for _, log in results:
-            if log:
-                print(log)
+    for _, log in results:
+        if verbose and log:
+            print(log)
+    return [o for o, _ in results]
+
+
+def _link(cmd):
+    r = subprocess.run(cmd, capture_output=True, text=True)
+    if r.returncode != 0:
+        raise RuntimeError(f"link failed: {' '.join(cmd)}\n{r.stdout}\n{r.stderr}")
+
+
+def build(verbose: bool = False) -> Path:
+    objs = _compile_all(_library_sources(), verbose)
     vs = _version_script()
     if _stale(LIB, objs + [vs]):
-        cmd = [_nvcc(), "-shared", "-o", str(LIB)] + [str(o) for o in objs] + ["-Xlinker", "-Bsymbolic", "-Xlinker", f"--version-script={vs}",
-                                                                             "-lcudart_static", "-ldl", "-lpthread", "-lrt", "-lm"]
-        r = subprocess.run(cmd, capture_output=True, text=True)
-        if r.returncode != 0:
-            raise RuntimeError(f"link failed: {' '.join(cmd)}\n{r.stdout}\n{r.stderr}")
+        _link([_nvcc(), "-shared", "-o", str(LIB)] + [str(o) for o in objs] + ["-Xlinker", "-Bsymbolic", "-Xlinker", f"--version-script={vs}"] + LINK_LIBS)
     return LIB
 
 
+def build_program(name: str, verbose: bool = False) -> Path:
+    srcs = PROGRAMS[name]
+    objs = _compile_all([PKG / "programs" / f"{name}.c"] + (_library_sources() if srcs is None else [PKG / s for s in srcs]), verbose)
+    out = PKG / "lib" / name
+    if _stale(out, objs):
+        _link([_nvcc(), "-o", str(out)] + [str(o) for o in objs] + LINK_LIBS)
+    return out
+
+
 if __name__ == "__main__":
-    print(build(verbose="-v" in sys.argv))
+    v = "-v" in sys.argv
+    if "--program" in sys.argv:
+        print(build_program(sys.argv[sys.argv.index("--program") + 1], v))
+    else:
+        print(build(v))

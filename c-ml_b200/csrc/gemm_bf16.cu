@@ -1,0 +1,300 @@
+// Prompt-sized product of dense bf16 weights on the 5th-generation tensor cores:
+//   Y[M][N] = X[M][K] W[N][K]^T, bf16 operands, fp32 accumulation in tensor memory.
+//
+// Persistent: one CTA per SM walks output tiles of 128 rows of x (the MMA "M" side, one per lane of
+// tensor memory) by BN weight rows (the "N" side). BN is 256, 128 or 64, picked by how the tiles fill
+// the SMs. Roles:
+//   warp 0     one lane issues TMA tensor loads of both operands (64-wide K slabs, 128-byte swizzle)
+//              into a ring of stages that runs on across tiles
+//   warp 1     owns tensor memory; one lane issues tcgen05.mma (128 x BN x 16)
+//   warps 2-5  epilogue: tcgen05.ld, through a per-warp transpose buffer to row-contiguous stores
+// Two accumulators alternate in tensor memory, so the epilogue of a tile overlaps the next tile's MMAs.
+// Output forms: fp32; or the gated activation of weights stored as pairs of 16-row groups (16 gate
+// rows, 16 up rows, ...): both halves of a pair sit in one lane's columns, and bf16 act(gate) * up is
+// all that leaves the SM. Rows and columns past the edges arrive as zeros and are not stored.
+// No cluster multicast. Every mbarrier wait is bounded; on expiry the CTA raises a status word
+// (cmlb200_gemm_dense_status), waits for its copies in flight, frees its tensor memory and returns.
+#include <cuda.h>
+#include "lm_util.cuh"
+
+namespace {
+
+constexpr int BM = 128, BK = 64;
+constexpr int EPI_WARPS = 4;
+constexpr int GEMM_THREADS = 64 + EPI_WARPS * 32;
+constexpr int A_BYTES = BM * BK * 2;
+constexpr uint32_t SPIN_LIMIT = 1u << 22;
+
+template <int BN> struct Tile {
+    static constexpr int B_BYTES = BN * BK * 2;
+    static constexpr int STAGE = A_BYTES + B_BYTES;
+    static constexpr int STAGES = BN == 256 ? 4 : (BN == 128 ? 6 : 8);
+    static constexpr int epi_off = STAGES * STAGE;                    // EPI_WARPS x [32][33] fp32
+    static constexpr int bar_off = epi_off + EPI_WARPS * 32 * 33 * 4;
+    static constexpr int nbars = 2 * STAGES + 4;
+    static constexpr int total = bar_off + 8 * nbars + 32;
+};
+
+__device__ int g_dense_status = 0;
+
+__device__ __forceinline__ uint32_t smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
+__device__ __forceinline__ void mbar_init(uint32_t bar, uint32_t count) { asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(bar), "r"(count)); }
+__device__ __forceinline__ void mbar_arrive(uint32_t bar) { asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(bar) : "memory"); }
+__device__ __forceinline__ void mbar_expect_tx(uint32_t bar, uint32_t bytes) {
+    asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(bar), "r"(bytes) : "memory");
+}
+__device__ __forceinline__ bool mbar_try(uint32_t bar, uint32_t parity) {
+    uint32_t ok;
+    asm volatile("{\n .reg .pred p;\n mbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2;\n selp.u32 %0, 1, 0, p;\n}\n"
+                 : "=r"(ok) : "r"(bar), "r"(parity) : "memory");
+    return ok != 0;
+}
+__device__ __forceinline__ bool mbar_wait(uint32_t bar, uint32_t parity, volatile int* abort_flag, int code) {
+    for (uint32_t it = 0; it < SPIN_LIMIT; ++it) {
+        if (mbar_try(bar, parity)) return true;
+        if (it > 1024) {
+            if (*abort_flag) return false;
+            __nanosleep(32);
+        }
+    }
+    *abort_flag = code;
+    atomicCAS(&g_dense_status, 0, code);
+    return false;
+}
+__device__ __forceinline__ void tma_load_2d(uint32_t dst, const CUtensorMap* map, int x, int y, uint32_t bar) {
+    asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];"
+                 ::"r"(dst), "l"(map), "r"(x), "r"(y), "r"(bar) : "memory");
+}
+// K-major operand, 128-byte swizzle: groups of 8 rows 1024 bytes apart
+__device__ __forceinline__ uint64_t make_desc(uint32_t saddr) {
+    return (uint64_t)((saddr & 0x3FFFF) >> 4) | ((uint64_t)1 << 16) | ((uint64_t)(1024 >> 4) << 32) | ((uint64_t)1 << 46) | ((uint64_t)2 << 61);
+}
+__device__ __forceinline__ void umma(uint32_t tmem_d, uint64_t adesc, uint64_t bdesc, uint32_t idesc, uint32_t accum) {
+    asm volatile("{\n .reg .pred p;\n setp.ne.b32 p, %4, 0;\n tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n}\n"
+                 ::"r"(tmem_d), "l"(adesc), "l"(bdesc), "r"(idesc), "r"(accum) : "memory");
+}
+__device__ __forceinline__ void umma_commit(uint32_t bar) {
+    asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(bar) : "memory");
+}
+__device__ __forceinline__ void tmem_ld32(uint32_t taddr, uint32_t (&r)[32]) {
+    asm volatile(
+        "tcgen05.ld.sync.aligned.32x32b.x32.b32 "
+        "{%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,"
+        "%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31}, [%32];"
+        : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]),
+          "=r"(r[8]), "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15]),
+          "=r"(r[16]), "=r"(r[17]), "=r"(r[18]), "=r"(r[19]), "=r"(r[20]), "=r"(r[21]), "=r"(r[22]), "=r"(r[23]),
+          "=r"(r[24]), "=r"(r[25]), "=r"(r[26]), "=r"(r[27]), "=r"(r[28]), "=r"(r[29]), "=r"(r[30]), "=r"(r[31])
+        : "r"(taddr));
+    asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+}
+
+// Tile number -> (row tile, column tile): groups of 8 row tiles share a sweep over the columns, so that
+// the CTAs working at one time read few distinct slabs.
+__device__ __forceinline__ void tile_at(int i, int tm, int tn, int& m, int& n) {
+    const int per = 8 * tn, gq = i / per, in = i - gq * per, rows = min(8, tm - gq * 8);
+    m = gq * 8 + in % rows;
+    n = in / rows;
+}
+
+template <int BN>
+__global__ void __launch_bounds__(GEMM_THREADS, 1)
+gemm_bf16_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constant__ CUtensorMap wmap, int M, int N, int K, int glu, int act,
+                 void* __restrict__ y, int ldy, int n_out) {
+    using C = Tile<BN>;
+    constexpr int ST = C::STAGES;
+    extern __shared__ uint8_t smem_raw[];
+    uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
+    const uint32_t sbase = smem_u32(smem), bars = sbase + C::bar_off;
+    auto full = [&](int s) { return bars + 8 * s; };
+    auto empty = [&](int s) { return bars + 8 * (ST + s); };
+    auto acc_full = [&](int b) { return bars + 8 * (2 * ST + b); };
+    auto acc_empty = [&](int b) { return bars + 8 * (2 * ST + 2 + b); };
+    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(smem + C::bar_off + 8 * C::nbars);
+    volatile int* abort_flag = reinterpret_cast<volatile int*>(smem + C::bar_off + 8 * C::nbars + 8);
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int tm = (M + BM - 1) / BM, tn = (N + BN - 1) / BN, tiles = tm * tn, nkb = (K + BK - 1) / BK;
+
+    if (threadIdx.x == 0) {
+        for (int s = 0; s < ST; s++) { mbar_init(full(s), 1); mbar_init(empty(s), 1); }
+        for (int b = 0; b < 2; b++) { mbar_init(acc_full(b), 1); mbar_init(acc_empty(b), EPI_WARPS); }
+        *abort_flag = 0;
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    if (warp == 1) {
+        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(tmem_slot)), "r"((uint32_t)(2 * BN)) : "memory");
+        asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
+    }
+    asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+    __syncthreads();
+    asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+    const uint32_t tmem_base = *tmem_slot;
+    dep_wait();
+    dep_trigger();
+
+    if (warp == 0) {
+        if (lane == 0) {
+            int it = 0;
+            bool ok = true;
+            for (int tile = blockIdx.x; tile < tiles && ok; tile += gridDim.x) {
+                int mi, ni;
+                tile_at(tile, tm, tn, mi, ni);
+                for (int k = 0; k < nkb; k++, it++) {
+                    const int s = it % ST;
+                    ok = mbar_wait(empty(s), ((it / ST) & 1) ^ 1, abort_flag, 1);
+                    if (!ok) break;
+                    mbar_expect_tx(full(s), (uint32_t)C::STAGE);
+                    tma_load_2d(sbase + s * C::STAGE, &xmap, k * BK, mi * BM, full(s));
+                    tma_load_2d(sbase + s * C::STAGE + A_BYTES, &wmap, k * BK, ni * BN, full(s));
+                }
+            }
+            for (int i = max(0, it - ST); i < it; i++) mbar_wait(full(i % ST), (i / ST) & 1, abort_flag, 2);      // no copy outlives the CTA
+        }
+    } else if (warp == 1) {
+        if (lane == 0) {
+            const uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(BN >> 3) << 17) | ((uint32_t)(BM >> 4) << 24);
+            int it = 0, done = 0;
+            bool ok = true;
+            for (int tile = blockIdx.x; tile < tiles && ok; tile += gridDim.x, done++) {
+                const int b = done & 1;
+                ok = mbar_wait(acc_empty(b), ((done >> 1) & 1) ^ 1, abort_flag, 3);
+                if (!ok) break;
+                asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+                for (int k = 0; k < nkb; k++, it++) {
+                    const int s = it % ST;
+                    ok = mbar_wait(full(s), (it / ST) & 1, abort_flag, 4);
+                    if (!ok) break;
+                    asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+                    const uint64_t ad = make_desc(sbase + s * C::STAGE), bd = make_desc(sbase + s * C::STAGE + A_BYTES);
+#pragma unroll
+                    for (int kk = 0; kk < BK / 16; kk++)
+                        umma(tmem_base + (uint32_t)(b * BN), ad + (uint64_t)(2 * kk), bd + (uint64_t)(2 * kk), idesc, (k | kk) ? 1u : 0u);
+                    umma_commit(empty(s));
+                }
+                umma_commit(acc_full(b));
+            }
+        }
+    } else {
+        const int q = warp & 3;                         // the quarter of tensor memory's lanes this warp may read
+        float* buf = reinterpret_cast<float*>(smem + C::epi_off) + (warp - 2) * 32 * 33;
+        int done = 0;
+        for (int tile = blockIdx.x; tile < tiles; tile += gridDim.x, done++) {
+            int mi, ni;
+            tile_at(tile, tm, tn, mi, ni);
+            const int b = done & 1, m0 = mi * BM + q * 32, n0 = ni * BN;
+            const bool ok = __all_sync(0xffffffffu, mbar_wait(acc_full(b), (done >> 1) & 1, abort_flag, 5));
+            if (!ok) break;
+            asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+            for (int c0 = 0; c0 < BN; c0 += 32) {
+                uint32_t v[32];
+                tmem_ld32(tmem_base + ((uint32_t)(q * 32) << 16) + (uint32_t)(b * BN + c0), v);
+                if (c0 + 32 == BN) {                    // this warp has read the whole accumulator
+                    asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+                    if (lane == 0) mbar_arrive(acc_empty(b));
+                }
+                if (m0 >= M || n0 + c0 >= N) continue;
+                __syncwarp();
+                if (glu) {
+#pragma unroll
+                    for (int j = 0; j < 16; j++) buf[lane * 33 + j] = glu_act(act, __uint_as_float(v[j]), __uint_as_float(v[16 + j]));
+                    __syncwarp();
+                    const int col = (n0 + c0) / 2 + (lane & 15);
+#pragma unroll 4
+                    for (int j = 0; j < 32; j += 2) {
+                        const int rr = j + (lane >> 4);
+                        if (m0 + rr < M && col < n_out)
+                            static_cast<__nv_bfloat16*>(y)[(size_t)(m0 + rr) * ldy + col] = __float2bfloat16_rn(buf[rr * 33 + (lane & 15)]);
+                    }
+                } else {
+#pragma unroll
+                    for (int j = 0; j < 32; j++) buf[lane * 33 + j] = __uint_as_float(v[j]);
+                    __syncwarp();
+                    const int col = n0 + c0 + lane;
+#pragma unroll 8
+                    for (int j = 0; j < 32; j++)
+                        if (m0 + j < M && col < n_out) static_cast<float*>(y)[(size_t)(m0 + j) * ldy + col] = buf[j * 33 + lane];
+                }
+            }
+        }
+    }
+    asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+    __syncthreads();
+    if (warp == 1) {
+        asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+        asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem_base), "r"((uint32_t)(2 * BN)) : "memory");
+    }
+}
+
+typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*, const cuuint32_t*,
+                                  const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
+
+int make_map(CUtensorMap* map, const void* base, int rows, int cols, int ld, int box_rows) {
+    static EncodeTiledFn fn = nullptr;
+    if (!fn) {
+        void* p = nullptr;
+        cudaDriverEntryPointQueryResult q;
+        CMLB_CUDA(cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &p, cudaEnableDefault, &q));
+        CMLB_REQUIRE(p && q == cudaDriverEntryPointSuccess, "cuTensorMapEncodeTiled is not available in this driver");
+        fn = reinterpret_cast<EncodeTiledFn>(p);
+    }
+    const cuuint64_t dims[2] = {(cuuint64_t)cols, (cuuint64_t)rows}, strides[1] = {(cuuint64_t)ld * 2};
+    const cuuint32_t box[2] = {BK, (cuuint32_t)box_rows}, one[2] = {1, 1};
+    const CUresult r = fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, one, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                          CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+    CMLB_REQUIRE(r == CUDA_SUCCESS, "cuTensorMapEncodeTiled failed with %d for [%d, %d], stride %d", (int)r, rows, cols, ld);
+    return CMLB200_OK;
+}
+
+template <int BN>
+int launch_gemm(const cmlb200_dense* W, const uint16_t* x, int ldx, int M, int glu, int act, void* y, int ldy, int n_out, cudaStream_t st) {
+    CUtensorMap xmap, wmap;
+    int rc = make_map(&xmap, x, M, W->cols, ldx, BM);
+    if (!rc) rc = make_map(&wmap, W->w, W->rows, W->cols, W->ld, BN);
+    if (rc) return rc;
+    const int tiles = ((M + BM - 1) / BM) * ((W->rows + BN - 1) / BN);
+    const size_t smem = Tile<BN>::total + 1024;
+    static_assert(Tile<BN>::total + 1024 <= 227 * 1024, "the stages do not fit shared memory");
+    static size_t attr[kMaxDevices] = {};
+    CMLB_CUDA(cmlb_ensure_smem(gemm_bf16_kernel<BN>, smem, attr));
+    CMLB_CUDA(launch_chain(gemm_bf16_kernel<BN>, dim3(tiles < cmlb_num_sms() ? tiles : cmlb_num_sms()), dim3(GEMM_THREADS), smem, 1, st, xmap, wmap, M,
+                           W->rows, W->cols, glu, act, y, ldy, n_out));
+    return CMLB200_OK;
+}
+
+int gemm_entry(const cmlb200_dense* W, const uint16_t* x, int ldx, int M, int glu, int act, void* y, int ldy, int n_out, const char* who, void* stream) {
+    CMLB_REQUIRE(W && W->w && x && y && M > 0, "%s: bad argument", who);
+    CMLB_REQUIRE(W->dtype == CMLB200_DT_BF16 && W->rows > 0 && W->cols > 0 && W->ld % 8 == 0 && W->ld >= W->cols, "%s: bad weight [%d, %d], stride %d", who, W->rows, W->cols, W->ld);
+    CMLB_REQUIRE(ldx % 8 == 0 && ldx >= W->cols && (((uintptr_t)x | (uintptr_t)W->w) & 15) == 0, "%s: x stride %d / alignment", who, ldx);
+    // The widest tile moves the fewest bytes per flop; narrower ones spread a small product over more
+    // SMs. Cost of a form: waves of tiles times its width, with the narrow forms' extra operand traffic.
+    const int gm = (M + BM - 1) / BM, sms = cmlb_num_sms();
+    auto waves = [&](int bn) { return (double)((gm * ((W->rows + bn - 1) / bn) + sms - 1) / sms); };
+    const double c256 = waves(256) * 256, c128 = waves(128) * 128 * 1.15, c64 = waves(64) * 64 * 1.6;
+    cudaStream_t st = as_stream(stream);
+    if (c256 <= c128 && c256 <= c64) return launch_gemm<256>(W, x, ldx, M, glu, act, y, ldy, n_out, st);
+    if (c128 <= c64) return launch_gemm<128>(W, x, ldx, M, glu, act, y, ldy, n_out, st);
+    return launch_gemm<64>(W, x, ldx, M, glu, act, y, ldy, n_out, st);
+}
+
+}  // namespace
+
+extern "C" int cmlb200_gemm_dense(const cmlb200_dense* W, const uint16_t* d_x, int ldx, int M, float* d_y, int ldy, void* stream) {
+    CMLB_REQUIRE(W && ldy >= W->rows, "cmlb200_gemm_dense: output stride %d", ldy);
+    return gemm_entry(W, d_x, ldx, M, 0, 0, d_y, ldy, W->rows, "cmlb200_gemm_dense", stream);
+}
+
+extern "C" int cmlb200_gemm_dense_glu(const cmlb200_dense* W, const uint16_t* d_x, int ldx, int M, int ff, int act, uint16_t* d_f, int ldf, void* stream) {
+    CMLB_REQUIRE(W && ff > 0 && W->rows == 2 * ((ff + 15) & ~15) && ldf >= ff, "cmlb200_gemm_dense_glu: weight rows do not fit %d outputs", ff);
+    return gemm_entry(W, d_x, ldx, M, 1, act, d_f, ldf, ff, "cmlb200_gemm_dense_glu", stream);
+}
+
+extern "C" int cmlb200_gemm_dense_status(int* status, int reset) {
+    CMLB_REQUIRE(status, "cmlb200_gemm_dense_status: NULL argument");
+    CMLB_CUDA(cudaDeviceSynchronize());
+    CMLB_CUDA(cudaMemcpyFromSymbol(status, g_dense_status, sizeof(int)));
+    if (reset) {
+        const int zero = 0;
+        CMLB_CUDA(cudaMemcpyToSymbol(g_dense_status, &zero, sizeof(int)));
+    }
+    return CMLB200_OK;
+}

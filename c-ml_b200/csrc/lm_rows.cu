@@ -1,0 +1,227 @@
+// Row-wise kernels of the layered models: embedding with a sinusoidal position vector, the fused
+// "norm a sublayer's output, add it to the residual, norm the sum for the next sublayer" step, the
+// query/key norm with query temperature and paged cache append, and the gated activation of the
+// 32-bit path. The residual and every norm are fp32; the operand handed to the next matrix product
+// is bf16 or fp32.
+#include "lm_util.cuh"
+
+namespace {
+
+// x[r] = table[token[r]] (+ the position vector: entry 2i = sin(p f_i), entry 2i + 1 = cos(p f_i),
+// f_i = freq[i], angle and sine in fp32). freq == NULL: no position vector.
+template <typename T>
+__global__ void __launch_bounds__(256)
+embed_rows_kernel(const T* __restrict__ table, const int* __restrict__ tokens, const int* __restrict__ pos, const float* __restrict__ freq,
+                  int width, int vocab, float* __restrict__ x) {
+    dep_wait();
+    dep_trigger();
+    const int r = blockIdx.x;
+    int t = tokens[r];
+    if (t < 0 || t >= vocab) t = 0;
+    const float p = (float)pos[r];
+    const T* src = table + (size_t)t * width;
+    float* dst = x + (size_t)r * width;
+    for (int i = blockIdx.y * 256 + threadIdx.x; 2 * i < width; i += gridDim.y * 256) {
+        float s = 0.f, c = 0.f;
+        if (freq) sincosf(p * freq[i], &s, &c);
+        dst[2 * i] = widen(src[2 * i]) + s;
+        if (2 * i + 1 < width) dst[2 * i + 1] = widen(src[2 * i + 1]) + c;
+    }
+}
+
+// One CTA per output row. y == NULL: out = norm(x[idx]) * w_next. Otherwise x += norm(y) * w_post
+// (w_post == NULL: x += y) and, when w_next is given, out = norm(x) * w_next. The row stays in shared
+// memory between the passes. Columns dim .. ldo of `out` are left alone.
+template <typename TO, bool VEC>
+__global__ void __launch_bounds__(256)
+residual_norm_kernel(float* __restrict__ x, const float* __restrict__ y, int ldy, const float* __restrict__ w_post,
+                     const float* __restrict__ w_next, float eps, int dim, const int* __restrict__ idx, TO* __restrict__ out, int ldo) {
+    extern __shared__ __align__(16) float row[];
+    __shared__ float red[32];
+    dep_wait();
+    dep_trigger();
+    const int r = blockIdx.x;
+    float* xr = x + (size_t)(idx ? idx[r] : r) * dim;
+    float ss = 0.f;
+    if (y) {
+        const float* yr = y + (size_t)r * ldy;
+        if (VEC) {
+            for (int i = threadIdx.x * 4; i < dim; i += 1024) {
+                const float4 v = *reinterpret_cast<const float4*>(yr + i);
+                *reinterpret_cast<float4*>(row + i) = v;
+                ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
+            }
+        } else {
+            for (int i = threadIdx.x; i < dim; i += 256) { const float v = yr[i]; row[i] = v; ss = fmaf(v, v, ss); }
+        }
+        const float inv = w_post ? 1.0f / sqrtf(block_sum(ss, red) / (float)dim + eps) : 1.0f;
+        ss = 0.f;
+        if (VEC) {                                      // a thread meets the same columns in every pass
+            for (int i = threadIdx.x * 4; i < dim; i += 1024) {
+                const float4 a = *reinterpret_cast<const float4*>(xr + i), v = *reinterpret_cast<const float4*>(row + i);
+                const float4 w = w_post ? *reinterpret_cast<const float4*>(w_post + i) : make_float4(1.f, 1.f, 1.f, 1.f);
+                const float4 o = make_float4(a.x + v.x * inv * w.x, a.y + v.y * inv * w.y, a.z + v.z * inv * w.z, a.w + v.w * inv * w.w);
+                *reinterpret_cast<float4*>(xr + i) = o;
+                *reinterpret_cast<float4*>(row + i) = o;
+                ss = fmaf(o.x, o.x, fmaf(o.y, o.y, fmaf(o.z, o.z, fmaf(o.w, o.w, ss))));
+            }
+        } else {
+            for (int i = threadIdx.x; i < dim; i += 256) {
+                const float o = xr[i] + row[i] * inv * (w_post ? w_post[i] : 1.0f);
+                xr[i] = o;
+                row[i] = o;
+                ss = fmaf(o, o, ss);
+            }
+        }
+    } else if (VEC) {
+        for (int i = threadIdx.x * 4; i < dim; i += 1024) {
+            const float4 v = *reinterpret_cast<const float4*>(xr + i);
+            *reinterpret_cast<float4*>(row + i) = v;
+            ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
+        }
+    } else {
+        for (int i = threadIdx.x; i < dim; i += 256) { const float v = xr[i]; row[i] = v; ss = fmaf(v, v, ss); }
+    }
+    if (!w_next) return;
+    const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)dim + eps);
+    TO* o = out + (size_t)r * ldo;
+    if (VEC) {
+        for (int i = threadIdx.x * 4; i < dim; i += 1024) {
+            const float4 v = *reinterpret_cast<const float4*>(row + i), w = *reinterpret_cast<const float4*>(w_next + i);
+            const float a = v.x * inv * w.x, b = v.y * inv * w.y, c = v.z * inv * w.z, d = v.w * inv * w.w;
+            if (sizeof(TO) == 2) {
+                const __nv_bfloat162 lo = __floats2bfloat162_rn(a, b), hi = __floats2bfloat162_rn(c, d);
+                *reinterpret_cast<uint2*>(o + i) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+            } else {
+                *reinterpret_cast<float4*>(o + i) = make_float4(a, b, c, d);
+            }
+        }
+    } else {
+        for (int i = threadIdx.x; i < dim; i += 256) o[i] = narrow<TO>(row[i] * inv * w_next[i]);
+    }
+}
+
+// One CTA per row of stacked projections [q | k | v | ..]: q is normed over all of its heads at once,
+// multiplied by the temperature of its position and left in place (fp32); k is normed the same way and
+// goes with v into the row's cache slot, each head padded with zeros to its stride in the pool.
+template <typename KV>
+__global__ void __launch_bounds__(256)
+qk_norm_append_kernel(float* __restrict__ qkv, int ld, const int* __restrict__ row_pos, const int* __restrict__ row_slot,
+                      const cmlb200_attn a, KV* __restrict__ kpool, KV* __restrict__ vpool) {
+    __shared__ float red[32];
+    dep_wait();
+    dep_trigger();
+    const int r = blockIdx.x, qw = a.heads * a.dim, kw = a.kv_heads * a.dim;
+    float* row = qkv + (size_t)r * ld;
+    const int p = row_pos[r];
+    float sq = 0.f, sk = 0.f;
+    for (int i = threadIdx.x; i < qw; i += 256) { const float v = row[i]; sq = fmaf(v, v, sq); }
+    for (int i = threadIdx.x; i < kw; i += 256) { const float v = row[qw + i]; sk = fmaf(v, v, sk); }
+    const float iq = a.q_norm ? 1.0f / sqrtf(block_sum(sq, red) / (float)qw + a.eps) : 1.0f;
+    const float ik = a.k_norm ? 1.0f / sqrtf(block_sum(sk, red) / (float)kw + a.eps) : 1.0f;
+    const float temp = a.temp_every > 0.f ? 1.0f + a.temp_coef * logf(floorf((float)(p + 1) / a.temp_every) + 1.0f) : 1.0f;
+    for (int i = threadIdx.x; i < qw; i += 256) row[i] = row[i] * iq * (a.q_norm ? a.q_norm[i] : 1.0f) * temp;
+    const size_t slot = (size_t)a.block_table[(size_t)row_slot[r] * a.table_ld + p / a.block_size] * a.block_size + p % a.block_size;
+    KV* kd = kpool + slot * a.kv_heads * a.dim_ld;
+    for (int i = threadIdx.x; i < a.kv_heads * a.dim_ld; i += 256) {
+        const int g = i / a.dim_ld, d = i - g * a.dim_ld, c = g * a.dim + d;
+        kd[i] = narrow<KV>(d < a.dim ? row[qw + c] * ik * (a.k_norm ? a.k_norm[c] : 1.0f) : 0.f);
+    }
+    KV* vd = vpool + slot * a.kv_heads * a.vdim_ld;
+    for (int i = threadIdx.x; i < a.kv_heads * a.vdim_ld; i += 256) {
+        const int g = i / a.vdim_ld, d = i - g * a.vdim_ld;
+        vd[i] = narrow<KV>(d < a.vdim ? row[qw + kw + g * a.vdim + d] : 0.f);
+    }
+}
+
+// f[r][c] = act(gate) * up of rows whose columns come in pairs of 16-wide groups (16 gate, 16 up, ..)
+__global__ void __launch_bounds__(256)
+glu_rows_f32_kernel(const float* __restrict__ gu, int ld, int ff, int act, float* __restrict__ f, int ldf) {
+    dep_wait();
+    dep_trigger();
+    const float* g = gu + (size_t)blockIdx.x * ld;
+    for (int c = blockIdx.y * 256 + threadIdx.x; c < ff; c += gridDim.y * 256) {
+        const int b = (c >> 4) * 32 + (c & 15);
+        f[(size_t)blockIdx.x * ldf + c] = glu_act(act, g[b], g[b + 16]);
+    }
+}
+
+// The next step of a decode loop that stays on the device: token = the one just picked, position + 1.
+__global__ void advance_tokens_kernel(const int* __restrict__ picked, int rows, int* __restrict__ tokens, int* __restrict__ pos, int* __restrict__ hist,
+                                      int* __restrict__ step) {
+    dep_wait();
+    dep_trigger();
+    const int s = *step;
+    for (int i = threadIdx.x; i < rows; i += blockDim.x) {
+        tokens[i] = picked[i];
+        pos[i] += 1;
+        hist[(size_t)s * rows + i] = picked[i];
+    }
+    __syncthreads();
+    if (threadIdx.x == 0) *step = s + 1;
+}
+
+}  // namespace
+
+extern "C" int cmlb200_embed_rows(const void* d_table, int dtype, const int* d_tokens, const int* d_pos, const float* d_freq, int rows, int width,
+                                  int vocab, float* d_x, void* stream) {
+    CMLB_REQUIRE(d_table && d_tokens && d_pos && d_x && rows > 0 && width > 0 && vocab > 0, "cmlb200_embed_rows: bad argument");
+    CMLB_REQUIRE(dtype == CMLB200_DT_F32 || dtype == CMLB200_DT_BF16, "cmlb200_embed_rows: dtype %d", dtype);
+    const dim3 grid(rows, rows < 64 ? (width + 2047) / 2048 : 1);
+    cudaStream_t st = as_stream(stream);
+    if (dtype == CMLB200_DT_BF16)
+        CMLB_CUDA(launch_chain(embed_rows_kernel<__nv_bfloat16>, grid, dim3(256), 0, 1, st, (const __nv_bfloat16*)d_table, d_tokens, d_pos, d_freq, width, vocab, d_x));
+    else
+        CMLB_CUDA(launch_chain(embed_rows_kernel<float>, grid, dim3(256), 0, 1, st, (const float*)d_table, d_tokens, d_pos, d_freq, width, vocab, d_x));
+    return CMLB200_OK;
+}
+
+extern "C" int cmlb200_residual_norm(float* d_x, const float* d_y, int ldy, const float* d_w_post, const float* d_w_next, float eps, int rows,
+                                     int dim, const int* d_row_idx, void* d_out, int out_dtype, int ldo, void* stream) {
+    CMLB_REQUIRE(d_x && rows > 0 && dim > 0 && (d_y || d_w_next), "cmlb200_residual_norm: bad argument");
+    CMLB_REQUIRE(!d_w_next || (d_out && ldo >= dim), "cmlb200_residual_norm: no output for the normed rows");
+    CMLB_REQUIRE(!(d_y && d_row_idx) && (!d_y || ldy >= dim), "cmlb200_residual_norm: a row list goes with the norm-only form");
+    CMLB_REQUIRE(out_dtype == CMLB200_DT_F32 || out_dtype == CMLB200_DT_BF16, "cmlb200_residual_norm: dtype %d", out_dtype);
+    const size_t smem = (size_t)((dim + 3) / 4) * 16;
+    CMLB_REQUIRE(smem <= 200 * 1024, "cmlb200_residual_norm: rows of %d elements do not fit shared memory", dim);
+    const bool vec = dim % 4 == 0 && (!d_y || ldy % 4 == 0) && (!d_w_next || ldo % 4 == 0) &&
+                     (((uintptr_t)d_x | (uintptr_t)d_y | (uintptr_t)d_w_post | (uintptr_t)d_w_next | (uintptr_t)d_out) & 15) == 0;
+    cudaStream_t st = as_stream(stream);
+    static size_t attr[4][kMaxDevices] = {};
+#define RN_LAUNCH(TO, V, slot)                                                                                                      \
+    do {                                                                                                                            \
+        auto kern = residual_norm_kernel<TO, V>;                                                                                    \
+        CMLB_CUDA(cmlb_ensure_smem(kern, smem, attr[slot]));                                                                        \
+        CMLB_CUDA(launch_chain(kern, dim3(rows), dim3(256), smem, 1, st, d_x, d_y, ldy, d_w_post, d_w_next, eps, dim, d_row_idx, (TO*)d_out, ldo)); \
+    } while (0)
+    if (out_dtype == CMLB200_DT_BF16) { if (vec) RN_LAUNCH(__nv_bfloat16, true, 0); else RN_LAUNCH(__nv_bfloat16, false, 1); }
+    else { if (vec) RN_LAUNCH(float, true, 2); else RN_LAUNCH(float, false, 3); }
+#undef RN_LAUNCH
+    return CMLB200_OK;
+}
+
+extern "C" int cmlb200_qk_norm_append(const cmlb200_attn* a, float* d_qkv, int ld, const int* d_row_pos, const int* d_row_slot, int rows,
+                                      void* stream) {
+    CMLB_REQUIRE(a && d_qkv && d_row_pos && d_row_slot && rows > 0, "cmlb200_qk_norm_append: bad argument");
+    const int rc = cmlb200_attn_check_(a, "cmlb200_qk_norm_append");
+    if (rc) return rc;
+    CMLB_REQUIRE(ld >= a->heads * a->dim + a->kv_heads * (a->dim + a->vdim), "cmlb200_qk_norm_append: row stride %d", ld);
+    cudaStream_t st = as_stream(stream);
+    if (a->cache_dtype == CMLB200_DT_F32)
+        CMLB_CUDA(launch_chain(qk_norm_append_kernel<float>, dim3(rows), dim3(256), 0, 1, st, d_qkv, ld, d_row_pos, d_row_slot, *a, (float*)a->k_pool, (float*)a->v_pool));
+    else
+        CMLB_CUDA(launch_chain(qk_norm_append_kernel<__half>, dim3(rows), dim3(256), 0, 1, st, d_qkv, ld, d_row_pos, d_row_slot, *a, (__half*)a->k_pool, (__half*)a->v_pool));
+    return CMLB200_OK;
+}
+
+extern "C" int cmlb200_glu_rows_f32(const float* d_gu, int ld, int rows, int ff, int act, float* d_f, int ldf, void* stream) {
+    CMLB_REQUIRE(d_gu && d_f && rows > 0 && ff > 0 && ldf >= ff && ld >= 2 * ((ff + 15) & ~15), "cmlb200_glu_rows_f32: bad argument");
+    CMLB_CUDA(launch_chain(glu_rows_f32_kernel, dim3(rows, (ff + 1023) / 1024), dim3(256), 0, 1, as_stream(stream), d_gu, ld, ff, act, d_f, ldf));
+    return CMLB200_OK;
+}
+
+extern "C" int cmlb200_advance_tokens(const int* d_picked, int rows, int* d_tokens, int* d_pos, int* d_hist, int* d_step, void* stream) {
+    CMLB_REQUIRE(d_picked && d_tokens && d_pos && d_hist && d_step && rows > 0, "cmlb200_advance_tokens: bad argument");
+    CMLB_CUDA(launch_chain(advance_tokens_kernel, dim3(1), dim3(128), 0, 1, as_stream(stream), d_picked, rows, d_tokens, d_pos, d_hist, d_step));
+    return CMLB200_OK;
+}

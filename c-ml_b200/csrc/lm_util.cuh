@@ -1,0 +1,71 @@
+// Shared pieces of the layered-model kernels: programmatic dependent launches, reductions and the
+// element conversions of the two number formats those models run in.
+#pragma once
+#include "common.cuh"
+
+namespace {
+
+// Every kernel of a step is launched so that it may become resident while its predecessor drains;
+// each one waits here before it touches anything an earlier kernel of the stream wrote.
+__device__ __forceinline__ void dep_wait() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
+__device__ __forceinline__ void dep_trigger() { asm volatile("griddepcontrol.launch_dependents;" ::: "memory"); }
+
+// cluster > 1: the grid's x dimension is cut into clusters of that many CTAs.
+template <typename Kern, typename... Args>
+cudaError_t launch_chain(Kern kern, dim3 grid, dim3 block, size_t smem, int cluster, cudaStream_t st, Args... args) {
+    cudaLaunchAttribute attr[2];
+    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[0].val.programmaticStreamSerializationAllowed = 1;
+    attr[1].id = cudaLaunchAttributeClusterDimension;
+    attr[1].val.clusterDim.x = (unsigned)cluster;
+    attr[1].val.clusterDim.y = 1;
+    attr[1].val.clusterDim.z = 1;
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = grid;
+    cfg.blockDim = block;
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = st;
+    cfg.attrs = attr;
+    cfg.numAttrs = cluster > 1 ? 2 : 1;
+    return cudaLaunchKernelEx(&cfg, kern, args...);
+}
+
+__device__ __forceinline__ float lane_sum(float v) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+    return v;
+}
+__device__ __forceinline__ float lane_max(float v) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, o));
+    return v;
+}
+// Sum over the block of up to 32 warps; `red` holds 32 floats and may be reused after the next barrier.
+__device__ __forceinline__ float block_sum(float v, float* red) {
+    v = lane_sum(v);
+    __syncthreads();
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+    __syncthreads();
+    float t = 0.f;
+    for (int k = 0; k < (int)(blockDim.x >> 5); k++) t += red[k];
+    return t;
+}
+
+__device__ __forceinline__ float widen(float v) { return v; }
+__device__ __forceinline__ float widen(__nv_bfloat16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ float widen(__half v) { return __half2float(v); }
+template <typename T> __device__ __forceinline__ T narrow(float v);
+template <> __device__ __forceinline__ float narrow<float>(float v) { return v; }
+template <> __device__ __forceinline__ __nv_bfloat16 narrow<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
+// fp16 is only used for cached keys and values; anything beyond its range is held at its end
+template <> __device__ __forceinline__ __half narrow<__half>(float v) { return __float2half_rn(fminf(fmaxf(v, -65504.f), 65504.f)); }
+
+// tanh form of gelu: 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))
+__device__ __forceinline__ float gelu_tanh(float z) {
+    return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+}
+__device__ __forceinline__ float silu(float z) { return z / (1.0f + expf(-z)); }
+__device__ __forceinline__ float glu_act(int act, float g, float u) { return (act == CMLB200_ACT_GELU_TANH ? gelu_tanh(g) : silu(g)) * u; }
+
+}  // namespace
+extern "C" int cmlb200_attn_check_(const cmlb200_attn* a, const char* who);

@@ -7,7 +7,12 @@
  * one host pool; the same pool exists once on the device ([blocks][16][kv_heads * head_dim] per K and
  * V, allocated at the first forward call), and a forward call first uploads the tokens appended
  * since the previous one (whole slot ranges per block), then launches cmlb200_paged_gqa_f32 with
- * the sequence's block table. Tokens must be written through cml_paged_cache_append. */
+ * the sequence's block table. Tokens must be written through cml_paged_cache_append.
+ *
+ * cml_paged_kv_cache_create_device makes a cache of bookkeeping alone, for models whose kernels write and
+ * read device pools of their own through the block tables (cml_lm.c): blocks are taken with
+ * cml_paged_cache_extend and those that every layer's window has passed go back with
+ * cml_paged_cache_release_before. */
 #include <math.h>
 #include <pthread.h>
 #include <stdlib.h>
@@ -83,6 +88,31 @@ CMLPagedKVCache* cml_paged_kv_cache_create(int max_blocks, int max_sequences, in
     return c;
 }
 
+CMLPagedKVCache* cml_paged_kv_cache_create_device(int max_blocks, int max_sequences, int block_size) {
+    if (max_blocks <= 0 || max_sequences <= 0 || block_size <= 0) {
+        LOG_ERROR("cml_paged_kv_cache_create_device: invalid parameters (max_blocks=%d, max_sequences=%d, block_size=%d)", max_blocks, max_sequences, block_size);
+        return NULL;
+    }
+    CMLPagedKVCache* c = (CMLPagedKVCache*)calloc(1, sizeof *c);
+    if (!c) return NULL;
+    c->max_blocks = c->num_blocks = c->free_count = max_blocks;
+    c->max_sequences = max_sequences;
+    c->block_size = block_size;
+    c->blocks = (CMLPageBlock*)calloc((size_t)max_blocks, sizeof(CMLPageBlock));
+    c->free_list = (int*)malloc((size_t)max_blocks * sizeof(int));
+    c->sequences = (CMLBlockTable*)calloc((size_t)max_sequences, sizeof(CMLBlockTable));
+    if (!c->blocks || !c->free_list || !c->sequences) {
+        LOG_ERROR("cml_paged_kv_cache_create_device: allocation failed");
+        free(c->blocks); free(c->free_list); free(c->sequences); free(c);
+        return NULL;
+    }
+    for (int i = 0; i < max_blocks; i++) {
+        c->blocks[i].block_id = i;
+        c->free_list[i] = max_blocks - 1 - i;              /* block 0 is handed out first */
+    }
+    return c;
+}
+
 void cml_paged_kv_cache_free(CMLPagedKVCache* cache) {
     if (!cache) return;
     pthread_mutex_lock(&g_paged_mu);
@@ -111,9 +141,11 @@ int cml_paged_cache_alloc_block(CMLPagedKVCache* cache) {
     CMLPageBlock* b = &cache->blocks[id];
     b->in_use = true;
     b->num_tokens = 0;
-    memset(b->key_data, 0, block_floats(cache) * sizeof(float));
-    memset(b->value_data, 0, block_floats(cache) * sizeof(float));
-    PagedDev* p = pd_find(cache);
+    if (b->key_data) {
+        memset(b->key_data, 0, block_floats(cache) * sizeof(float));
+        memset(b->value_data, 0, block_floats(cache) * sizeof(float));
+    }
+    PagedDev* p = b->key_data ? pd_find(cache) : NULL;
     if (p) p->dev_tokens[id] = 0;                          /* nothing of the new owner's tokens is on the device yet */
     cache->total_allocated++;
     return id;
@@ -149,11 +181,51 @@ void cml_paged_cache_free_sequence(CMLPagedKVCache* cache, int seq_id) {
     if (seq_id < 0 || seq_id >= cache->max_sequences) { LOG_ERROR("cml_paged_cache_free_sequence: invalid seq_id %d", seq_id); return; }
     CMLBlockTable* bt = &cache->sequences[seq_id];
     if (!bt->block_ids) { LOG_WARNING("cml_paged_cache_free_sequence: sequence %d not initialised", seq_id); return; }
-    for (int i = 0; i < bt->num_blocks; i++) cml_paged_cache_free_block(cache, bt->block_ids[i]);
+    for (int i = 0; i < bt->num_blocks; i++)
+        if (bt->block_ids[i] >= 0) cml_paged_cache_free_block(cache, bt->block_ids[i]);       /* -1: released before */
     free(bt->block_ids);
     bt->block_ids = NULL;
     bt->num_blocks = bt->capacity = bt->seq_len = 0;
     cache->num_sequences--;
+}
+
+static CMLBlockTable* live_sequence(CMLPagedKVCache* cache, int seq_id) {
+    return cache && seq_id >= 0 && seq_id < cache->max_sequences && cache->sequences[seq_id].block_ids ? &cache->sequences[seq_id] : NULL;
+}
+
+int cml_paged_cache_blocks_for(CMLPagedKVCache* cache, int seq_id, int num_tokens) {
+    const CMLBlockTable* bt = live_sequence(cache, seq_id);
+    if (!bt || num_tokens < 0 || num_tokens > 0x7fffffff - bt->seq_len - cache->block_size) return -1;
+    return (bt->seq_len + num_tokens + cache->block_size - 1) / cache->block_size - bt->num_blocks;
+}
+
+int cml_paged_cache_extend(CMLPagedKVCache* cache, int seq_id, int num_tokens) {
+    CMLBlockTable* bt = live_sequence(cache, seq_id);
+    const int need = cml_paged_cache_blocks_for(cache, seq_id, num_tokens);
+    if (!bt || need < 0) { LOG_ERROR("cml_paged_cache_extend: sequence %d cannot take %d tokens", seq_id, num_tokens); return -1; }
+    if (need > cache->free_count) { LOG_ERROR("cml_paged_cache_extend: %d blocks needed, %d free", need, cache->free_count); return -1; }
+    if (bt->num_blocks + need > bt->capacity) {
+        int cap = bt->capacity;
+        while (cap < bt->num_blocks + need) cap *= 2;
+        int* ids = (int*)realloc(bt->block_ids, (size_t)cap * sizeof(int));
+        if (!ids) { LOG_ERROR("cml_paged_cache_extend: block table realloc failed"); return -1; }
+        bt->block_ids = ids;
+        bt->capacity = cap;
+    }
+    for (int i = 0; i < need; i++) bt->block_ids[bt->num_blocks++] = cml_paged_cache_alloc_block(cache);
+    bt->seq_len += num_tokens;
+    return 0;
+}
+
+void cml_paged_cache_release_before(CMLPagedKVCache* cache, int seq_id, int position) {
+    CMLBlockTable* bt = live_sequence(cache, seq_id);
+    if (!bt) return;
+    int last = position / cache->block_size - 1;           /* the last block that ends at or before `position` */
+    if (last >= bt->num_blocks) last = bt->num_blocks - 1;
+    for (int i = last; i >= 0 && bt->block_ids[i] >= 0; i--) {
+        cml_paged_cache_free_block(cache, bt->block_ids[i]);
+        bt->block_ids[i] = -1;
+    }
 }
 
 int cml_paged_cache_append(CMLPagedKVCache* cache, int seq_id, const float* key, const float* value) {
@@ -161,6 +233,7 @@ int cml_paged_cache_append(CMLPagedKVCache* cache, int seq_id, const float* key,
     if (seq_id < 0 || seq_id >= cache->max_sequences) { LOG_ERROR("cml_paged_cache_append: invalid seq_id %d", seq_id); return -1; }
     CMLBlockTable* bt = &cache->sequences[seq_id];
     if (!bt->block_ids) { LOG_ERROR("cml_paged_cache_append: sequence %d not initialised", seq_id); return -1; }
+    if (!cache->blocks[0].key_data) { LOG_ERROR("cml_paged_cache_append: the cache holds no host data"); return -1; }
     if (bt->num_blocks == 0 || cache->blocks[bt->block_ids[bt->num_blocks - 1]].num_tokens >= cache->block_size) {
         const int nb = cml_paged_cache_alloc_block(cache);
         if (nb < 0) { LOG_ERROR("cml_paged_cache_append: failed to allocate new block for seq %d", seq_id); return -1; }

@@ -399,6 +399,78 @@ int cmlb200_ipc_get_handle(void* d_ptr, void* handle64);
 int cmlb200_ipc_open(const void* handle64, void** d_ptr);
 int cmlb200_ipc_close(void* d_ptr);
 
+/* ---- layered language models: dense weights, paged rows ------------------------------------------
+ * The operations of models whose layers are described by a configuration file (cml_lm.h). A step's rows
+ * belong to several sequences; row r has a position and a sequence slot, and finds its cached keys
+ * through that slot's row of a block table. Replaces nothing in C-ML. */
+#define CMLB200_DT_F32 0
+#define CMLB200_DT_BF16 1
+#define CMLB200_DT_F16 2
+#define CMLB200_ACT_SILU 0
+#define CMLB200_ACT_GELU_TANH 1
+
+/* A dense [rows, cols] weight (rows = out features), row stride `ld` elements. Allocated with rows rounded
+ * up to 16 and ld a multiple of 64, the padding zero. dtype CMLB200_DT_F32 or CMLB200_DT_BF16. */
+typedef struct cmlb200_dense {
+    int dtype;
+    int rows, cols, ld;
+    void* w;
+} cmlb200_dense;
+
+/* An attention layer over a paged cache, as the kernels below see it. Projection rows hold
+ * [q (heads*dim) | k (kv_heads*dim) | v (kv_heads*vdim) | ..] in fp32. */
+typedef struct cmlb200_attn {
+    int heads, kv_heads, dim, vdim;
+    int dim_ld, vdim_ld;        /* elements per head in the pools, multiples of 16, zeros behind dim / vdim */
+    float scale;                /* score = q.k * scale - slopes[h] * (i - j) */
+    int window;                 /* row at position i sees i - window + 1 .. i; <= 0: everything before it */
+    const float* slopes;        /* device, one per query head; NULL: no distance bias */
+    int sink;                   /* 1: the softmax denominator starts at exp(0) */
+    const float *q_norm, *k_norm; /* device, RMS norm weights over the whole q / k projection; NULL: none */
+    float eps;
+    float temp_coef, temp_every;  /* q *= 1 + coef ln(floor((i + 1) / every) + 1); every <= 0: none */
+    int gate_col;               /* column of the first of `heads` gate logits in a projection row; -1: none */
+    int cache_dtype;            /* CMLB200_DT_F32 or CMLB200_DT_F16 */
+    void *k_pool, *v_pool;      /* [blocks][block_size][kv_heads][dim_ld] and [..][vdim_ld] */
+    int block_size;             /* a power of two >= 16 */
+    const int* block_table;     /* device, [slots][table_ld] block ids */
+    int table_ld;
+} cmlb200_attn;
+
+/* x[r] = table[token[r]] (+ a sinusoidal vector of position pos[r]: sin, cos of pos * freq[i] in entries
+ * 2i, 2i + 1; d_freq NULL: none). fp32 rows of `width`. */
+int cmlb200_embed_rows(const void* d_table, int dtype, const int* d_tokens, const int* d_pos, const float* d_freq, int rows, int width,
+                       int vocab, float* d_x, void* stream);
+/* x += rms_norm(y) * w_post (w_post NULL: x += y; y NULL: x unchanged), then out = rms_norm(x) * w_next when
+ * w_next is given. Without y, d_row_idx (optional) picks the rows of x. out: fp32 or bf16, stride ldo. */
+int cmlb200_residual_norm(float* d_x, const float* d_y, int ldy, const float* d_w_post, const float* d_w_next, float eps, int rows, int dim,
+                          const int* d_row_idx, void* d_out, int out_dtype, int ldo, void* stream);
+/* Norms q (in place) and k of projection rows, applies the query temperature, appends k and v to the cache. */
+int cmlb200_qk_norm_append(const cmlb200_attn* a, float* d_qkv, int ld, const int* d_row_pos, const int* d_row_slot, int rows, void* stream);
+/* Attention of prompt portions whose q is normed and whose k, v are appended already: tiles of up to 64
+ * consecutive rows of one sequence, d_tiles[i] = {first row, rows, slot, position of the first row}. */
+int cmlb200_attention_tiles(const cmlb200_attn* a, const float* d_qkv, int ld, const int* d_tiles, int tiles, uint16_t* d_out_bf16, int out_ld,
+                            void* stream);
+/* Decoded tokens, at most one row per sequence: norms, temperature, append, attention and gate from the raw
+ * projection rows in one launch. max_keys bounds the cached keys of any row (it picks the launch shape). */
+int cmlb200_attention_one(const cmlb200_attn* a, const float* d_qkv, int ld, const int* d_row_pos, const int* d_row_slot, int rows, int max_keys,
+                          uint16_t* d_out_bf16, int out_ld, void* stream);
+/* The 32-bit form for any rows (after cmlb200_qk_norm_append), fp32 cache and output. */
+int cmlb200_attention_rows_f32(const cmlb200_attn* a, const float* d_qkv, int ld, const int* d_row_pos, const int* d_row_slot, int rows,
+                               float* d_out, int out_ld, void* stream);
+/* y[M, rows] = x[M, cols] . W^T. _gemv_: bf16, M <= 32, x readable up to W->ld columns. _gemm_: bf16 on tcgen05,
+ * any M. _linear_: fp32. The _glu forms take a weight of `ff` gate and `ff` up rows interleaved in groups of
+ * 16 (padded with zero rows) and write bf16 act(gate) * up. */
+int cmlb200_gemv_dense(const cmlb200_dense* W, const uint16_t* d_x, int ldx, int M, float* d_y, int ldy, void* stream);
+int cmlb200_gemv_dense_glu(const cmlb200_dense* W, const uint16_t* d_x, int ldx, int M, int ff, int act, uint16_t* d_f, int ldf, void* stream);
+int cmlb200_gemm_dense(const cmlb200_dense* W, const uint16_t* d_x, int ldx, int M, float* d_y, int ldy, void* stream);
+int cmlb200_gemm_dense_glu(const cmlb200_dense* W, const uint16_t* d_x, int ldx, int M, int ff, int act, uint16_t* d_f, int ldf, void* stream);
+int cmlb200_gemm_dense_status(int* status, int reset);
+int cmlb200_linear_dense_f32(const cmlb200_dense* W, const float* d_x, int ldx, int M, float* d_y, int ldy, void* stream);
+int cmlb200_glu_rows_f32(const float* d_gu, int ld, int rows, int ff, int act, float* d_f, int ldf, void* stream);
+/* tokens[i] = picked[i], pos[i] += 1, hist[step * rows + i] = picked[i], step += 1 */
+int cmlb200_advance_tokens(const int* d_picked, int rows, int* d_tokens, int* d_pos, int* d_hist, int* d_step, void* stream);
+
 #ifdef __cplusplus
 }
 #endif
