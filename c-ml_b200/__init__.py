@@ -163,6 +163,11 @@ class GenerationConfig(C.Structure):
                 ("eos_token_id", C.c_int), ("do_sample", C.c_bool)]
 
 
+class GenerationResult(C.Structure):
+    _fields_ = [("token_ids", C.POINTER(C.c_int)), ("num_tokens", C.c_int), ("text", C.c_char_p), ("total_time_ms", C.c_float),
+                ("tokens_per_second", C.c_float)]
+
+
 class NF4Tensor(C.Structure):
     _fields_ = [("packed_data", C.POINTER(Tensor)), ("scales", C.POINTER(C.c_float)), ("num_scales", C.c_int),
                 ("block_size", C.c_int), ("original_numel", C.c_size_t), ("original_shape", C.POINTER(C.c_int)),
@@ -421,6 +426,110 @@ _sig("cml_cleanup", ci)
 _sig("tensor_manual_seed", None, C.c_uint64)
 _sig("tensor_get_seed", C.c_uint64)
 REFERENCE_QUIRKS, KV_FP32, ALL_LOGITS_FP32 = 1, 2, 4
+
+
+# ---- layered models (include/cml_lm.h and the kernels behind it) ---------------------------------
+DT_F32, DT_BF16, DT_F16 = 0, 1, 2
+ACT_SILU, ACT_GELU_TANH = 0, 1
+DTYPE_FLOAT32, DTYPE_BFLOAT16 = 0, 6
+
+
+class Dense(C.Structure):
+    """cmlb200_dense."""
+    _fields_ = [("dtype", ci), ("rows", ci), ("cols", ci), ("ld", ci), ("w", vp)]
+
+
+class Attn(C.Structure):
+    """cmlb200_attn."""
+    _fields_ = [("heads", ci), ("kv_heads", ci), ("dim", ci), ("vdim", ci), ("dim_ld", ci), ("vdim_ld", ci), ("scale", C.c_float),
+                ("window", ci), ("slopes", vp), ("sink", ci), ("q_norm", vp), ("k_norm", vp), ("eps", C.c_float), ("temp_coef", C.c_float),
+                ("temp_every", C.c_float), ("gate_col", ci), ("cache_dtype", ci), ("k_pool", vp), ("v_pool", vp), ("block_size", ci),
+                ("block_table", vp), ("table_ld", ci)]
+
+
+class LMOptions(C.Structure):
+    _fields_ = [("dtype", ci), ("max_tokens", ci), ("max_sequences", ci), ("max_step_rows", ci)]
+
+
+class LMEntry(C.Structure):
+    _fields_ = [("seq", ci), ("tokens", vp), ("num_tokens", ci), ("want", vp), ("num_want", ci)]
+
+
+_sig("cmlb200_embed_rows", ci, vp, ci, vp, vp, vp, ci, ci, ci, vp, vp)
+_sig("cmlb200_residual_norm", ci, vp, vp, ci, vp, vp, C.c_float, ci, ci, vp, vp, ci, ci, vp)
+_sig("cmlb200_qk_norm_append", ci, C.POINTER(Attn), vp, ci, vp, vp, ci, vp)
+_sig("cmlb200_attention_tiles", ci, C.POINTER(Attn), vp, ci, vp, ci, vp, ci, vp)
+_sig("cmlb200_attention_one", ci, C.POINTER(Attn), vp, ci, vp, vp, ci, ci, vp, ci, vp)
+_sig("cmlb200_attention_rows_f32", ci, C.POINTER(Attn), vp, ci, vp, vp, ci, vp, ci, vp)
+for _n in ("cmlb200_gemv_dense", "cmlb200_gemm_dense", "cmlb200_linear_dense_f32"):
+    _sig(_n, ci, C.POINTER(Dense), vp, ci, ci, vp, ci, vp)
+for _n in ("cmlb200_gemv_dense_glu", "cmlb200_gemm_dense_glu"):
+    _sig(_n, ci, C.POINTER(Dense), vp, ci, ci, ci, ci, vp, ci, vp)
+_sig("cmlb200_gemm_dense_status", ci, C.POINTER(ci), ci)
+_sig("cmlb200_glu_rows_f32", ci, vp, ci, ci, ci, ci, vp, ci, vp)
+_sig("cml_lm_default_options", LMOptions)
+_sig("cml_lm_known", ci, C.c_char_p)
+_sig("cml_lm_load", vp, C.c_char_p, C.POINTER(LMOptions))
+_sig("cml_lm_free", None, vp)
+_sig("cml_lm_architecture", C.c_char_p, vp)
+for _n in ("cml_lm_vocab_size", "cml_lm_sequence_open", "cml_lm_block_size", "cml_lm_blocks_total", "cml_lm_blocks_free"):
+    _sig(_n, ci, vp)
+_sig("cml_lm_sequence_close", ci, vp, ci)
+_sig("cml_lm_sequence_length", ci, vp, ci)
+_sig("cml_lm_step", ci, vp, C.POINTER(LMEntry), ci, vp)
+_sig("cml_lm_step_greedy", ci, vp, C.POINTER(LMEntry), ci, vp)
+_sig("cml_lm_decode_greedy", ci, vp, vp, vp, ci, ci, vp, C.POINTER(C.c_float))
+_sig("cml_serving_run_lm", ci, vp, vp, C.POINTER(GenerationConfig), ci, vp, vp)
+_sig("cml_lm_generate", C.POINTER(GenerationResult), vp, vp, ci, C.POINTER(GenerationConfig))
+_sig("cml_paged_kv_cache_create_device", C.POINTER(PagedKVCache), ci, ci, ci)
+_sig("cml_paged_cache_blocks_for", ci, C.POINTER(PagedKVCache), ci, ci)
+_sig("cml_paged_cache_extend", ci, C.POINTER(PagedKVCache), ci, ci)
+_sig("cml_paged_cache_release_before", None, C.POINTER(PagedKVCache), ci, ci)
+
+
+class LanguageModel:
+    """A model loaded through cml_lm_load, with numpy arrays in and out."""
+
+    def __init__(self, path, dtype=DTYPE_BFLOAT16, max_tokens=2048, max_sequences=8, max_step_rows=0):
+        self.h = lib.cml_lm_load(str(path).encode(), C.byref(LMOptions(dtype, max_tokens, max_sequences, max_step_rows)))
+        if not self.h:
+            raise CmlB200Error(f"cml_lm_load({path}) failed")
+        self.vocab = lib.cml_lm_vocab_size(self.h)
+
+    def close(self):
+        if self.h:
+            lib.cml_lm_free(self.h)
+            self.h = None
+
+    def open(self):
+        s = lib.cml_lm_sequence_open(self.h)
+        if s < 0:
+            raise CmlB200Error("no free sequence")
+        return s
+
+    def end(self, seq):
+        check(lib.cml_lm_sequence_close(self.h, seq), "cml_lm_sequence_close")
+
+    def step(self, entries, greedy=False):
+        """entries: (seq, tokens, wanted places or None for all). One list item of logits [n, vocab] (or picks [n]) per entry."""
+        import numpy as np
+        keep, arr = [], (LMEntry * len(entries))()
+        for i, (seq, tokens, want) in enumerate(entries):
+            t = np.ascontiguousarray(tokens, np.int32)
+            w = np.arange(len(t), dtype=np.int32) if want is None else np.ascontiguousarray(want, np.int32)
+            keep += [t, w]
+            arr[i] = LMEntry(seq, np_ptr(t), len(t), np_ptr(w), len(w))
+        counts = [arr[i].num_want for i in range(len(entries))]
+        out = np.zeros(max(1, sum(counts)), np.int32) if greedy else np.zeros((max(1, sum(counts)), self.vocab), np.float32)
+        check((lib.cml_lm_step_greedy if greedy else lib.cml_lm_step)(self.h, arr, len(entries), np_ptr(out)), "cml_lm_step")
+        return np.split(out[:sum(counts)], np.cumsum(counts)[:-1])
+
+    def decode_greedy(self, seqs, first, steps):
+        import numpy as np
+        s, f, ms = np.ascontiguousarray(seqs, np.int32), np.ascontiguousarray(first, np.int32), C.c_float(0)
+        out = np.zeros((steps, len(s)), np.int32)
+        check(lib.cml_lm_decode_greedy(self.h, np_ptr(s), np_ptr(f), len(s), steps, np_ptr(out), C.byref(ms)), "cml_lm_decode_greedy")
+        return out, ms.value
 
 
 def tensor_to_numpy(tp, free=True):

@@ -230,3 +230,76 @@ def write_random_llama_gguf(path, rng, cfg, qtype=2, weight_std=0.02, alias_laye
             f.write(raw)
             f.write(b"\0" * ((-len(raw)) % 32))
     return len(head) + off
+
+
+# ---- layered models: a folder with config.json and model.safetensors --------------------------------
+def bf16_round(a):
+    """fp32 values rounded to the nearest bf16 (ties to even), as fp32."""
+    u = np.ascontiguousarray(a, np.float32).view(np.uint32).astype(np.uint64)
+    return (((u + 0x7FFF + ((u >> 16) & 1)) >> 16).astype(np.uint32) << 16).view(np.float32)
+
+
+def layered_layer(heads, kv_heads, dim, vdim, window, ff, scale=None, coef=0.2, every=50, weights_of=None):
+    layer = {"type": "attention", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale or dim ** -0.5,
+                                            "mask": {"size": window}, "q_temp": {"coef": coef, "every": every}},
+             "mlp": {"kind": "dense", "ff": ff} if ff else None}
+    if weights_of is not None:
+        layer["weights_of"] = weights_of
+    return layer
+
+
+def layered_config(vocab, width, layers, eps=1e-5):
+    return {"architecture": "Rarolorn", "vocab": vocab, "width": width, "norm": {"eps": eps}, "layers": layers}
+
+
+def layered_shapes(cfg):
+    """Tensor name -> shape of every tensor a configuration asks for."""
+    W, out = cfg["width"], {"embed": (cfg["vocab"], cfg["width"])}
+    for i, layer in enumerate(cfg["layers"]):
+        if layer.get("weights_of") is not None:
+            continue
+        m, p = layer["mixer"], f"l{i}."
+        q, k, v = m["heads"] * m["dim"], m["kv_heads"] * m["dim"], m["kv_heads"] * m["vdim"]
+        out.update({p + "norm1": (W,), p + "norm1b": (W,), p + "mix.q": (q, W), p + "mix.k": (k, W), p + "mix.v": (v, W), p + "mix.q.norm": (q,),
+                    p + "mix.k.norm": (k,), p + "mix.g": (m["heads"], W), p + "mix.o": (W, m["heads"] * m["vdim"])})
+        if layer["mlp"] is not None:
+            f = layer["mlp"]["ff"]
+            out.update({p + "norm2": (W,), p + "norm2b": (W,), p + "mlp.gate": (f, W), p + "mlp.up": (f, W), p + "mlp.down": (W, f)})
+    out.update({"final.norm": (W,), "head": (cfg["vocab"], W)})
+    return out
+
+
+def layered_weights(rng, cfg):
+    """Random bf16-exact fp32 weights: products of unit inputs have unit size, norms lie around 1."""
+    w = {}
+    for name, shape in layered_shapes(cfg).items():
+        a = rng.standard_normal(shape, dtype=np.float32)
+        w[name] = bf16_round(1.0 + 0.2 * a if len(shape) == 1 else (a if name == "embed" else a / np.sqrt(shape[1])))
+    return w
+
+
+def write_layered(folder, cfg, weights, alias_layers=False):
+    """Writes config.json and model.safetensors (bf16). `weights`: name -> fp32 array, or a function (name, shape)
+    giving one. alias_layers: every layer's tensors point at the bytes of the first layer with that tensor and shape."""
+    import json
+    from pathlib import Path
+    folder = Path(folder)
+    folder.mkdir(parents=True, exist_ok=True)
+    (folder / "config.json").write_text(json.dumps(cfg))
+    header, stored, placed, off = {}, [], {}, 0
+    for name, shape in layered_shapes(cfg).items():
+        n = 2 * int(np.prod(shape))
+        key = (name.split(".", 1)[1] if name[0] == "l" and name[1].isdigit() else name, shape)
+        at = placed.get(key) if alias_layers else None
+        if at is None:
+            at = placed[key] = off
+            stored.append((name, shape))
+            off += n
+        header[name] = {"dtype": "BF16", "shape": list(shape), "data_offsets": [at, at + n]}
+    text = json.dumps(header).encode()
+    text += b" " * ((-len(text)) % 8)
+    with open(folder / "model.safetensors", "wb") as f:
+        f.write(len(text).to_bytes(8, "little") + text)
+        for name, shape in stored:
+            a = weights(name, shape) if callable(weights) else weights[name]
+            f.write((bf16_round(a).view(np.uint32) >> 16).astype(np.uint16).tobytes())

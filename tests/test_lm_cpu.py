@@ -1,0 +1,183 @@
+"""Layered models without a device: the restatement's mechanisms against hand-worked cases, the registry and
+the file readers' refusals, the block bookkeeping of the paged cache."""
+import json
+import subprocess
+from pathlib import Path
+
+import numpy as np
+import pytest
+
+import lm_oracle as lo
+import lm_util
+
+ROOT = Path(__file__).resolve().parents[1]
+
+
+# ---- the restatement ----------------------------------------------------------------------------------
+def test_sinusoid_entries():
+    s = lo.sinusoid([0, 3], 6)
+    assert np.allclose(s[0], [0, 1, 0, 1, 0, 1])
+    f = [1.0, 10000 ** (-2 / 6), 10000 ** (-4 / 6)]
+    assert np.allclose(s[1], [np.sin(3 * f[0]), np.cos(3 * f[0]), np.sin(3 * f[1]), np.cos(3 * f[1]), np.sin(3 * f[2]), np.cos(3 * f[2])])
+
+
+def test_window_edge_and_bias():
+    assert lo.window_mask([5], range(8), 3)[0].tolist() == [False] * 3 + [True] * 3 + [False] * 2
+    assert lo.window_mask([0, 1], [0, 1], 1).tolist() == [[True, False], [False, True]]
+    assert np.allclose(lo.alibi_slopes(4), [2.0 ** -2, 2.0 ** -4, 2.0 ** -6, 2.0 ** -8])
+    assert np.allclose(lo.distance_bias(np.zeros((1, 3)), [2], [0, 1, 2], 0.5), [[-1.0, -0.5, 0.0]])
+
+
+def test_sink_takes_its_share():
+    p = lo.softmax_with_sink(np.array([[0.0, 0.0, 5.0]]), np.array([[True, True, False]]))
+    assert np.allclose(p, [[1 / 3, 1 / 3, 0]])
+    p = lo.softmax_with_sink(np.array([[-800.0, 800.0]]), np.array([[True, True]]))
+    assert np.allclose(p, [[0, 1]])
+
+
+def test_query_temperature_steps():
+    t = lo.query_temperature([0, 8, 9, 18, 19], 0.5, 10)
+    assert np.allclose(t, 1 + 0.5 * np.log([1, 1, 2, 2, 3]))
+
+
+def test_norm_and_activation():
+    x = np.array([[3.0, -4.0]])
+    assert np.allclose(lo.rms_norm(x, np.array([1.0, 2.0]), 0.5), x / np.sqrt(13.0) * [1, 2])
+    assert np.allclose(lo.gelu_tanh(np.array([0.0, 1.0, -1.0])), [0.0, 0.841192, -0.158808], atol=1e-6)
+
+
+@pytest.mark.parametrize("name", ["mixed", "odd", "wide", "plain"])
+def test_portions_change_nothing(synth, tmp_path, name):
+    cfg, w, _ = lm_util.build(synth, tmp_path, name)
+    m = lo.Model(cfg, w)
+    tokens = np.random.default_rng(3).integers(0, cfg["vocab"], 60)
+    whole = m.forward(tokens)
+    state = m.new_state()
+    parts = [m.forward(tokens[a:b], state) for a, b in lm_util.cut(60, [2, 17, 1, 5])]
+    assert np.allclose(np.concatenate(parts), whole, atol=1e-9)
+
+
+def test_shared_weights_keep_their_own_cache(synth, tmp_path):
+    cfg, w, _ = lm_util.build(synth, tmp_path, "mixed")
+    m = lo.Model(cfg, w)
+    st = m.new_state()
+    m.forward([1, 2, 3], st)
+    assert not np.allclose(st["caches"][0]["k"], st["caches"][2]["k"]) and not any(n.startswith("l2.") for n in w)
+
+
+# ---- registry and readers ------------------------------------------------------------------------------
+def test_registry_knows_its_classes(pkg):
+    assert pkg.lib.cml_lm_known(b"Rarolorn") == 1 and pkg.lib.cml_lm_known(b"llama") == 1
+    assert pkg.lib.cml_lm_known(b"nothing") == 0 and pkg.lib.cml_lm_known(None) == 0
+    o = pkg.lib.cml_lm_default_options()
+    assert (o.dtype, o.max_tokens, o.max_sequences, o.max_step_rows) == (pkg.DTYPE_BFLOAT16, 8192, 8, 0)
+
+
+def _load(pkg, folder, **kw):
+    o = pkg.LMOptions(kw.get("dtype", pkg.DTYPE_BFLOAT16), kw.get("max_tokens", 64), kw.get("max_sequences", 1), 0)
+    return pkg.lib.cml_lm_load(str(folder).encode(), o)
+
+
+def test_load_refusals(pkg, synth, tmp_path):
+    """Everything here is refused while reading config.json, before a device is needed."""
+    cfg, w, folder = lm_util.build(synth, tmp_path, "plain")
+
+    def with_config(change):
+        c = json.loads(json.dumps(cfg))
+        change(c)
+        (folder / "config.json").write_text(json.dumps(c))
+        assert not _load(pkg, folder)
+
+    with_config(lambda c: c.pop("architecture"))
+    with_config(lambda c: c.update(architecture="Other"))
+    with_config(lambda c: c.pop("width"))
+    with_config(lambda c: c.pop("norm"))
+    with_config(lambda c: c.update(layers=[]))
+    with_config(lambda c: c["layers"][0].update(type="recurrent"))
+    with_config(lambda c: c["layers"][0]["mixer"].pop("scale"))
+    with_config(lambda c: c["layers"][0]["mixer"].update(kv_heads=3))
+    with_config(lambda c: c["layers"][0]["mixer"]["mask"].update(size=0))
+    with_config(lambda c: c["layers"][0]["mixer"]["q_temp"].pop("every"))
+    with_config(lambda c: c["layers"][0]["mlp"].update(kind="sparse"))
+    with_config(lambda c: c["layers"][1].update(weights_of=0))          # another shape
+    with_config(lambda c: c["layers"][1].update(weights_of=7))
+    for text in ("", "{", '{"architecture": "Rarolorn",}', '{"architecture": "Rarolorn"} x', "[" * 100, '{"a": "\\ud800"}', '{"a": 1e999}'):
+        (folder / "config.json").write_text(text)
+        assert not _load(pkg, folder)
+    (folder / "config.json").unlink()
+    assert not _load(pkg, folder) and not _load(pkg, tmp_path / "absent")
+    (folder / "config.json").write_text(json.dumps(cfg))
+    assert not _load(pkg, folder, dtype=pkg.DTYPE_BFLOAT16 + 1) and not _load(pkg, folder, max_tokens=0) and not _load(pkg, folder, max_sequences=0)
+
+
+def test_tensor_file_refusals(pkg, synth, tmp_path):
+    cfg, w, folder = lm_util.build(synth, tmp_path, "plain")
+    path = folder / "model.safetensors"
+    raw = path.read_bytes()
+    n = int.from_bytes(raw[:8], "little")
+    head = json.loads(raw[8:8 + n])
+
+    def with_header(change):
+        h = json.loads(json.dumps(head))
+        change(h)
+        t = json.dumps(h).encode()
+        path.write_bytes(len(t).to_bytes(8, "little") + t + raw[8 + n:])
+        assert not _load(pkg, folder)
+
+    with_header(lambda h: h.pop("embed"))
+    with_header(lambda h: h["embed"].update(dtype="U8"))
+    with_header(lambda h: h["embed"].update(shape=[64, 63]))
+    with_header(lambda h: h["embed"].update(data_offsets=[0, 1 << 40]))
+    with_header(lambda h: h["embed"].update(data_offsets=[8, 4]))
+    for bad in (b"", raw[:4], (1 << 60).to_bytes(8, "little") + raw[8:], raw[:8 + n // 2]):
+        path.write_bytes(bad)
+        assert not _load(pkg, folder)
+
+
+def test_null_arguments(pkg):
+    lib = pkg.lib
+    lib.cml_lm_free(None)
+    assert not lib.cml_lm_load(None, None) and lib.cml_lm_sequence_open(None) == -1 and lib.cml_lm_sequence_close(None, 0) == -1
+    assert lib.cml_lm_step(None, None, 0, None) == -1 and lib.cml_lm_step_greedy(None, None, 0, None) == -1
+    assert lib.cml_serving_run_lm(None, None, None, 0, None, None) == -1 and not lib.cml_lm_generate(None, None, 0, None)
+
+
+# ---- blocks ----------------------------------------------------------------------------------------------
+def test_blocks_are_taken_released_and_used_again(pkg):
+    lib = pkg.lib
+    c = lib.cml_paged_kv_cache_create_device(6, 3, 16)
+    a, b = lib.cml_paged_cache_init_sequence(c), lib.cml_paged_cache_init_sequence(c)
+    assert lib.cml_paged_cache_blocks_for(c, a, 16) == 1 and lib.cml_paged_cache_blocks_for(c, a, 17) == 2
+    assert lib.cml_paged_cache_extend(c, a, 40) == 0 and c.contents.free_count == 3
+    assert lib.cml_paged_cache_blocks_for(c, a, 8) == 0 and lib.cml_paged_cache_blocks_for(c, a, 9) == 1
+    assert lib.cml_paged_cache_extend(c, b, 49) == -1 and c.contents.free_count == 3 and c.contents.sequences[b].seq_len == 0
+    assert lib.cml_paged_cache_extend(c, b, 48) == 0 and c.contents.free_count == 0
+    first = [c.contents.sequences[a].block_ids[i] for i in range(3)]
+    lib.cml_paged_cache_release_before(c, a, 31)                       # block 1 still holds position 31
+    assert c.contents.free_count == 1 and [c.contents.sequences[a].block_ids[i] for i in range(3)] == [-1] + first[1:]
+    lib.cml_paged_cache_release_before(c, a, 32)
+    lib.cml_paged_cache_release_before(c, a, -5)
+    assert c.contents.free_count == 2
+    assert lib.cml_paged_cache_extend(c, b, 17) == 0
+    assert {c.contents.sequences[b].block_ids[i] for i in (3, 4)} == set(first[:2])
+    lib.cml_paged_cache_free_sequence(c, a)
+    lib.cml_paged_cache_free_sequence(c, b)
+    assert c.contents.free_count == 6
+    one = np.zeros(4, np.float32)
+    s = lib.cml_paged_cache_init_sequence(c)
+    assert lib.cml_paged_cache_append(c, s, pkg.np_ptr(one), pkg.np_ptr(one)) == -1          # no host data
+    lib.cml_paged_kv_cache_free(c)
+    assert not lib.cml_paged_kv_cache_create_device(0, 1, 16)
+
+
+# ---- programs --------------------------------------------------------------------------------------------
+@pytest.mark.parametrize("name", ["trace_run", "cml_generate"])
+def test_programs_build_and_refuse_bad_arguments(name):
+    run = lambda *a: subprocess.run([str(ROOT / "bin" / name), *a], capture_output=True, text=True, timeout=600)
+    r = run()
+    assert r.returncode == 2 and "usage" in r.stderr
+    r = run("--nonsense", "1")
+    assert r.returncode == 2 and "unknown option" in r.stderr
+    args = ["--model", "/nonexistent"] + (["--out", "/tmp", "--max-tokens", "64"] if name == "trace_run" else ["--tokens", "1,2"])
+    r = run(*args)
+    assert r.returncode == 2 and "cannot load" in r.stderr
