@@ -385,6 +385,8 @@ def main():
     ap.add_argument("--profile-m", type=int, default=1, help="rows of x of the --profile run")
     ap.add_argument("--profile-batch", type=int, default=1, help="batch size of --profile llama")
     ap.add_argument("--only-gemm", action="store_true", help="run the NF4 prefill-GEMM leg alone")
+    ap.add_argument("--layered", nargs="?", const="all", default=None, choices=["all", "kernels", "models"],
+                    help="instead of the default workload: the layered models beside LLaMA at equal layer sizes, and their kernels")
     ap.add_argument("--cpu-leg", default=None, choices=["gemv", "llama"], help=argparse.SUPPRESS)
     ap.add_argument("--calls", type=int, default=3, help=argparse.SUPPRESS)
     ap.add_argument("--llama-steps", type=int, default=4, help=argparse.SUPPRESS)
@@ -418,6 +420,9 @@ def main():
             except ImportError:
                 pass
     peaks = measured_peaks()
+    if args.layered:
+        import bench_layered
+        return bench_layered.run(pkg, synth, torch, peaks, ClockSampler(local), args.layered == "kernels", args.layered == "models")
     stream = torch.cuda.Stream(device=dev)
     sp = stream.cuda_stream
 
