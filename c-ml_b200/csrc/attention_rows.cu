@@ -42,17 +42,23 @@ __device__ __forceinline__ uint32_t pack_h2(float lo, float hi) {
     const __half2 v = __floats2half2_rn(lo, hi);
     return *reinterpret_cast<const uint32_t*>(&v);
 }
+__device__ __forceinline__ float ex2(float v) {
+    float r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(v));
+    return r;
+}
 __device__ __forceinline__ float sigmoidf(float z) { return 1.0f / (1.0f + expf(-z)); }
 
 constexpr int QT = 64, KT = 64, TILE_THREADS = 128;
 
 // grid = (tiles, heads). tiles[i] = {first row, rows (1..64), sequence slot, position of the first row}.
-template <int DV>
+// DV: room for value columns. DK: 0, or the padded key size, and then DV is the padded value size.
+template <int DV, int DK>
 __global__ void __launch_bounds__(TILE_THREADS)
 attention_tiles_kernel(const cmlb200_attn a, const float* __restrict__ qkv, int ld, const int4* __restrict__ tiles, __nv_bfloat16* __restrict__ out,
                        int out_ld) {
     extern __shared__ __align__(16) __half sm[];
-    const int dk = a.dim_ld, dv = a.vdim_ld, LK = dk + 8, LV = dv + 8;
+    const int dk = DK ? DK : a.dim_ld, dv = DK ? DV : a.vdim_ld, LK = dk + 8, LV = dv + 8;
     __half* Qs = sm;
     __half* Ks = Qs + QT * LK;                         // two stages each
     __half* Vs = Ks + 2 * KT * LK;
@@ -85,9 +91,10 @@ attention_tiles_kernel(const cmlb200_attn a, const float* __restrict__ qkv, int 
     load(0);
     {
         const float qs = a.scale * kLog2e;
-        for (int i = threadIdx.x; i < QT * dk; i += TILE_THREADS) {
-            const int r = i / dk, d = i - r * dk;
-            Qs[r * LK + d] = (r < n && d < a.dim) ? narrow<__half>(qkv[(size_t)(tl.x + r) * ld + h * a.dim + d] * qs) : __float2half_rn(0.f);
+        for (int r = warp; r < QT; r += TILE_THREADS / 32) {
+            const float* src = qkv + (size_t)(tl.x + min(r, n - 1)) * ld + h * a.dim;
+#pragma unroll 4
+            for (int d = lane; d < dk; d += 32) Qs[r * LK + d] = d < a.dim ? narrow<__half>(src[d] * qs) : __float2half_rn(0.f);
         }
     }
     const float slope = a.slopes ? a.slopes[h] * kLog2e : 0.f;
@@ -98,6 +105,11 @@ attention_tiles_kernel(const cmlb200_attn a, const float* __restrict__ qkv, int 
 #pragma unroll
     for (int i = 0; i < DV / 8; i++) { o[i][0] = 0.f; o[i][1] = 0.f; o[i][2] = 0.f; o[i][3] = 0.f; }
     float m0 = a.sink ? 0.f : -INFINITY, m1 = m0, l0 = 0.f, l1 = 0.f;
+    // score of key kt + c from position q: dot - slope (q - kt - c). The part that depends on the column alone
+    // is what the accumulators start from; the rest is one constant per row and tile.
+    float bias[KT / 8][2];
+#pragma unroll
+    for (int i = 0; i < KT / 8; i++) { bias[i][0] = slope * (float)(i * 8 + 2 * t); bias[i][1] = slope * (float)(i * 8 + 2 * t + 1); }
     const uint32_t q_base = smem_addr(Qs + (warp * 16 + (lane & 15)) * LK + (lane >> 4) * 8);
 
     for (int it = 0; it < ntiles; it++) {
@@ -114,8 +126,9 @@ attention_tiles_kernel(const cmlb200_attn a, const float* __restrict__ qkv, int 
         if (active) {
             float s[KT / 8][4];
 #pragma unroll
-            for (int i = 0; i < KT / 8; i++) { s[i][0] = 0.f; s[i][1] = 0.f; s[i][2] = 0.f; s[i][3] = 0.f; }
+            for (int i = 0; i < KT / 8; i++) { s[i][0] = bias[i][0]; s[i][1] = bias[i][1]; s[i][2] = bias[i][0]; s[i][3] = bias[i][1]; }
             const uint32_t k_base = smem_addr(Ks + (st * KT + (lane & 7) + ((lane >> 4) & 1) * 8) * LK + ((lane >> 3) & 1) * 8);
+#pragma unroll (DK ? DK / 16 : 1)
             for (int kk = 0; kk < dk; kk += 16) {
                 uint32_t qa[4];
                 ldsm4(q_base + kk * 2, qa);
@@ -127,30 +140,41 @@ attention_tiles_kernel(const cmlb200_attn a, const float* __restrict__ qkv, int 
                     mma_f16(s[2 * j + 1], qa, b[2], b[3]);
                 }
             }
-            float mx0 = m0, mx1 = m1;
+            // unless every row of the warp sees every key of the tile
+            if (!(kt + KT - 1 <= w_first && (window > w_last - kt)) || w_last - w_first < 15) {
+#pragma unroll
+                for (int i = 0; i < KT / 8; i++) {
+#pragma unroll
+                    for (int e = 0; e < 2; e++) {
+                        const int key = kt + i * 8 + 2 * t + e, d0 = q0 - key, d1 = q1 - key;
+                        if (d0 < 0 || d0 >= window) s[i][e] = -INFINITY;
+                        if (d1 < 0 || d1 >= window) s[i][2 + e] = -INFINITY;
+                    }
+                }
+            }
+            float mx0 = -INFINITY, mx1 = -INFINITY;
 #pragma unroll
             for (int i = 0; i < KT / 8; i++) {
-#pragma unroll
-                for (int e = 0; e < 2; e++) {
-                    const int key = kt + i * 8 + 2 * t + e, d0 = q0 - key, d1 = q1 - key;
-                    s[i][e] = (d0 >= 0 && d0 < window) ? s[i][e] - slope * (float)d0 : -INFINITY;
-                    s[i][2 + e] = (d1 >= 0 && d1 < window) ? s[i][2 + e] - slope * (float)d1 : -INFINITY;
-                    mx0 = fmaxf(mx0, s[i][e]);
-                    mx1 = fmaxf(mx1, s[i][2 + e]);
-                }
+                mx0 = fmaxf(mx0, fmaxf(s[i][0], s[i][1]));
+                mx1 = fmaxf(mx1, fmaxf(s[i][2], s[i][3]));
             }
             mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 1)); mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 2));
             mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 1)); mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 2));
+            const float f0 = slope * (float)(kt - q0), f1 = slope * (float)(kt - q1);
+            mx0 = fmaxf(m0, mx0 + f0);
+            mx1 = fmaxf(m1, mx1 + f1);
             const float u0 = mx0 == -INFINITY ? 0.f : mx0, u1 = mx1 == -INFINITY ? 0.f : mx1;      // a row that has seen nothing yet
-            const float c0 = exp2f(m0 - u0), c1 = exp2f(m1 - u1);
+            const float c0 = ex2(m0 - u0), c1 = ex2(m1 - u1), g0 = u0 - f0, g1 = u1 - f1;
             m0 = mx0; m1 = mx1;
             l0 *= c0; l1 *= c1;
+            if (__any_sync(0xffffffffu, c0 != 1.f || c1 != 1.f)) {
 #pragma unroll
-            for (int i = 0; i < DV / 8; i++) { o[i][0] *= c0; o[i][1] *= c0; o[i][2] *= c1; o[i][3] *= c1; }
+                for (int i = 0; i < DV / 8; i++) { o[i][0] *= c0; o[i][1] *= c0; o[i][2] *= c1; o[i][3] *= c1; }
+            }
             uint32_t pa[KT / 16][4];
 #pragma unroll
             for (int i = 0; i < KT / 8; i++) {
-                const float e0 = exp2f(s[i][0] - u0), e1 = exp2f(s[i][1] - u0), e2 = exp2f(s[i][2] - u1), e3 = exp2f(s[i][3] - u1);
+                const float e0 = ex2(s[i][0] - g0), e1 = ex2(s[i][1] - g0), e2 = ex2(s[i][2] - g1), e3 = ex2(s[i][3] - g1);
                 l0 += e0 + e1;
                 l1 += e2 + e3;
                 pa[i >> 1][(i & 1) * 2] = pack_h2(e0, e1);
@@ -222,7 +246,7 @@ attention_one_kernel(const cmlb200_attn a, const float* __restrict__ qkv, int ld
     float* c_m = w_l + ONE_WARPS * RM;                 // [RM] this CTA's
     float* c_l = c_m + RM;
     float* w_acc = c_l + RM;                           // [ONE_WARPS][RM][dv]; the CTA's sums end up in warp 0's part
-    __shared__ float red[32];
+    __shared__ float2 red[ONE_WARPS];
     dep_wait();
     dep_trigger();
     const int splits = gridDim.x, rank = blockIdx.x, kh = blockIdx.y / passes, pass = blockIdx.y % passes, r = blockIdx.z;
@@ -233,11 +257,12 @@ attention_one_kernel(const cmlb200_attn a, const float* __restrict__ qkv, int ld
     const int shift = __ffs(a.block_size) - 1;
     const int* table = a.block_table + (size_t)row_slot[r] * a.table_ld;
 
-    float sq = 0.f, sk = 0.f;
-    if (a.q_norm) for (int i = threadIdx.x; i < qw; i += ONE_THREADS) { const float v = row[i]; sq = fmaf(v, v, sq); }
-    if (a.k_norm) for (int i = threadIdx.x; i < kw; i += ONE_THREADS) { const float v = row[qw + i]; sk = fmaf(v, v, sk); }
-    const float iq = a.q_norm ? 1.0f / sqrtf(block_sum(sq, red) / (float)qw + a.eps) : 1.0f;
-    const float ik = a.k_norm ? 1.0f / sqrtf(block_sum(sk, red) / (float)kw + a.eps) : 1.0f;
+    float iq = 1.0f, ik = 1.0f;
+    if (a.q_norm || a.k_norm) {
+        const float2 ss = block_sum2(a.q_norm ? square_share(row, qw) : 0.f, a.k_norm && rank == 0 ? square_share(row + qw, kw) : 0.f, red);
+        if (a.q_norm) iq = 1.0f / sqrtf(ss.x / (float)qw + a.eps);
+        if (a.k_norm) ik = 1.0f / sqrtf(ss.y / (float)kw + a.eps);      // used where the row's own key is made: rank 0
+    }
     const float temp = a.temp_every > 0.f ? 1.0f + a.temp_coef * logf(floorf((float)(p + 1) / a.temp_every) + 1.0f) : 1.0f;
     const float qs = a.scale * kLog2e;
     for (int i = threadIdx.x; i < RM * dk; i += ONE_THREADS) {
@@ -278,6 +303,20 @@ attention_one_kernel(const cmlb200_attn a, const float* __restrict__ qkv, int ld
     const int kstride = a.kv_heads * dk, vstride = a.kv_heads * dv;
     const int vcol = lane * 2 * VP;
     const bool has_v = vcol < dv;
+    constexpr int PRE = VP == 4 ? 8 : 16;
+    auto load_values = [&](uint32_t (&u)[PRE][VP], int slot, int k0) {
+#pragma unroll
+        for (int k = 0; k < PRE; k++) {
+            const int ks = __shfl_sync(0xffffffffu, slot, k0 + k);       // lanes past the last key hold its slot
+#pragma unroll
+            for (int e = 0; e < VP; e++) u[k][e] = 0u;
+            if (!has_v) continue;
+            const __half* src = vp + (size_t)ks * vstride + vcol;
+            if (VP == 4) { const uint4 w = *reinterpret_cast<const uint4*>(src); u[k][0] = w.x; u[k][1 % VP] = w.y; u[k][2 % VP] = w.z; u[k][3 % VP] = w.w; }
+            else if (VP == 2) { const uint2 w = *reinterpret_cast<const uint2*>(src); u[k][0] = w.x; u[k][1 % VP] = w.y; }
+            else u[k][0] = *reinterpret_cast<const uint32_t*>(src);
+        }
+    };
     // cached keys k_lo .. p - 1, 32 per warp and step; a lane scores one key
     for (int kt = k_lo + (rank * ONE_WARPS + warp) * 32; kt < p; kt += splits * ONE_WARPS * 32) {
         const int key = kt + lane, count = min(32, p - kt);
@@ -286,12 +325,15 @@ attention_one_kernel(const cmlb200_attn a, const float* __restrict__ qkv, int ld
         float s[RM];
 #pragma unroll
         for (int j = 0; j < RM; j++) s[j] = 0.f;
+        // the value rows do not depend on the scores: the first PRE of them are requested ahead of the keys
+        uint32_t u[PRE][VP];
+        load_values(u, slot, 0);
         const uint4* kr = reinterpret_cast<const uint4*>(kp + (size_t)slot * kstride);
-#pragma unroll 4
+#pragma unroll 8
         for (int c = 0; c < (dk >> 3); c++) {
-            const uint4 u = kr[c];
-            const float2 k01 = __half22float2(*reinterpret_cast<const __half2*>(&u.x)), k23 = __half22float2(*reinterpret_cast<const __half2*>(&u.y));
-            const float2 k45 = __half22float2(*reinterpret_cast<const __half2*>(&u.z)), k67 = __half22float2(*reinterpret_cast<const __half2*>(&u.w));
+            const uint4 w = kr[c];
+            const float2 k01 = __half22float2(*reinterpret_cast<const __half2*>(&w.x)), k23 = __half22float2(*reinterpret_cast<const __half2*>(&w.y));
+            const float2 k45 = __half22float2(*reinterpret_cast<const __half2*>(&w.z)), k67 = __half22float2(*reinterpret_cast<const __half2*>(&w.w));
 #pragma unroll
             for (int j = 0; j < RM; j++) {
                 const float4 x = *reinterpret_cast<const float4*>(q_s + j * dk + c * 8), y = *reinterpret_cast<const float4*>(q_s + j * dk + c * 8 + 4);
@@ -310,27 +352,19 @@ attention_one_kernel(const cmlb200_attn a, const float* __restrict__ qkv, int ld
 #pragma unroll
             for (int e = 0; e < 2 * VP; e++) acc[j][e] *= c;
         }
-#pragma unroll 8
-        for (int k = 0; k < 32; k++) {
-            if (k >= count) break;
-            const int ks = __shfl_sync(0xffffffffu, slot, k);
-            uint32_t u[VP];
+        for (int k0 = 0; k0 < count; k0 += PRE) {
+            if (k0) load_values(u, slot, k0);
 #pragma unroll
-            for (int e = 0; e < VP; e++) u[e] = 0u;
-            if (has_v) {
-                const __half* src = vp + (size_t)ks * vstride + vcol;
-                if (VP == 4) { const uint4 w = *reinterpret_cast<const uint4*>(src); u[0] = w.x; u[1 % VP] = w.y; u[2 % VP] = w.z; u[3 % VP] = w.w; }
-                else if (VP == 2) { const uint2 w = *reinterpret_cast<const uint2*>(src); u[0] = w.x; u[1 % VP] = w.y; }
-                else u[0] = *reinterpret_cast<const uint32_t*>(src);
-            }
+            for (int k = 0; k < PRE; k++) {            // weights past the last key are zero
 #pragma unroll
-            for (int j = 0; j < RM; j++) {
-                const float w = __shfl_sync(0xffffffffu, s[j], k);
+                for (int j = 0; j < RM; j++) {
+                    const float w = __shfl_sync(0xffffffffu, s[j], k0 + k);
 #pragma unroll
-                for (int e = 0; e < VP; e++) {
-                    const float2 v = __half22float2(*reinterpret_cast<const __half2*>(&u[e]));
-                    acc[j][2 * e] = fmaf(w, v.x, acc[j][2 * e]);
-                    acc[j][2 * e + 1] = fmaf(w, v.y, acc[j][2 * e + 1]);
+                    for (int e = 0; e < VP; e++) {
+                        const float2 v = __half22float2(*reinterpret_cast<const __half2*>(&u[k][e]));
+                        acc[j][2 * e] = fmaf(w, v.x, acc[j][2 * e]);
+                        acc[j][2 * e + 1] = fmaf(w, v.y, acc[j][2 * e + 1]);
+                    }
                 }
             }
         }
@@ -512,16 +546,18 @@ extern "C" int cmlb200_attention_tiles(const cmlb200_attn* a, const float* d_qkv
     CMLB_REQUIRE(smem <= 227 * 1024, "cmlb200_attention_tiles: head sizes %d / %d do not fit shared memory", a->dim, a->vdim);
     cudaStream_t st = as_stream(stream);
     const dim3 grid(tiles, a->heads);
-    static size_t attr[3][kMaxDevices] = {};
-#define AT_LAUNCH(DV, slot)                                                                                                     \
+    static size_t attr[5][kMaxDevices] = {};
+#define AT_LAUNCH(DV, DK, slot)                                                                                                   \
     do {                                                                                                                        \
-        auto kern = attention_tiles_kernel<DV>;                                                                                 \
+        auto kern = attention_tiles_kernel<DV, DK>;                                                                               \
         CMLB_CUDA(cmlb_ensure_smem(kern, smem, attr[slot]));                                                                    \
         CMLB_CUDA(launch_chain(kern, grid, dim3(TILE_THREADS), smem, 1, st, *a, d_qkv, ld, (const int4*)d_tiles, (__nv_bfloat16*)d_out_bf16, out_ld)); \
     } while (0)
-    if (a->vdim_ld <= 64) AT_LAUNCH(64, 0);
-    else if (a->vdim_ld <= 128) AT_LAUNCH(128, 1);
-    else AT_LAUNCH(256, 2);
+    if (a->vdim_ld == 64 && a->dim_ld == 64) AT_LAUNCH(64, 64, 3);
+    else if (a->vdim_ld == 128 && a->dim_ld == 128) AT_LAUNCH(128, 128, 4);
+    else if (a->vdim_ld <= 64) AT_LAUNCH(64, 0, 0);
+    else if (a->vdim_ld <= 128) AT_LAUNCH(128, 0, 1);
+    else AT_LAUNCH(256, 0, 2);
 #undef AT_LAUNCH
     return CMLB200_OK;
 }
@@ -532,7 +568,8 @@ extern "C" int cmlb200_attention_one(const cmlb200_attn* a, const float* d_qkv, 
     const int rc = cmlb200_attn_check_(a, "cmlb200_attention_one");
     if (rc) return rc;
     CMLB_REQUIRE(a->cache_dtype == CMLB200_DT_F16 && a->vdim_ld <= 256 && rows <= 65535, "cmlb200_attention_one: fp16 cache and value heads up to 256");
-    const int group = a->heads / a->kv_heads, rm = group == 1 ? 1 : (group <= 4 ? 4 : 8), passes = (group + rm - 1) / rm;
+    // few rows: fewer heads per CTA, so that more CTAs share the work (the keys are read again from L2)
+    const int group = a->heads / a->kv_heads, rm = group == 1 ? 1 : (group <= 4 || rows * a->kv_heads * 8 < cmlb_num_sms() ? 4 : 8), passes = (group + rm - 1) / rm;
     CMLB_REQUIRE((long long)a->kv_heads * passes <= 65535, "cmlb200_attention_one: too many heads");
     const int keys = (a->window > 0 && a->window < max_keys) ? a->window : max_keys;
     const long long base = (long long)rows * a->kv_heads * passes;

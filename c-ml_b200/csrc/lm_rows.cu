@@ -33,7 +33,7 @@ embed_rows_kernel(const T* __restrict__ table, const int* __restrict__ tokens, c
 // (w_post == NULL: x += y) and, when w_next is given, out = norm(x) * w_next. The row stays in shared
 // memory between the passes. Columns dim .. ldo of `out` are left alone.
 template <typename TO, bool VEC>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(1024)
 residual_norm_kernel(float* __restrict__ x, const float* __restrict__ y, int ldy, const float* __restrict__ w_post,
                      const float* __restrict__ w_next, float eps, int dim, const int* __restrict__ idx, TO* __restrict__ out, int ldo) {
     extern __shared__ __align__(16) float row[];
@@ -46,18 +46,18 @@ residual_norm_kernel(float* __restrict__ x, const float* __restrict__ y, int ldy
     if (y) {
         const float* yr = y + (size_t)r * ldy;
         if (VEC) {
-            for (int i = threadIdx.x * 4; i < dim; i += 1024) {
+            for (int i = threadIdx.x * 4; i < dim; i += blockDim.x * 4) {
                 const float4 v = *reinterpret_cast<const float4*>(yr + i);
                 *reinterpret_cast<float4*>(row + i) = v;
                 ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
             }
         } else {
-            for (int i = threadIdx.x; i < dim; i += 256) { const float v = yr[i]; row[i] = v; ss = fmaf(v, v, ss); }
+            for (int i = threadIdx.x; i < dim; i += blockDim.x) { const float v = yr[i]; row[i] = v; ss = fmaf(v, v, ss); }
         }
         const float inv = w_post ? 1.0f / sqrtf(block_sum(ss, red) / (float)dim + eps) : 1.0f;
         ss = 0.f;
         if (VEC) {                                      // a thread meets the same columns in every pass
-            for (int i = threadIdx.x * 4; i < dim; i += 1024) {
+            for (int i = threadIdx.x * 4; i < dim; i += blockDim.x * 4) {
                 const float4 a = *reinterpret_cast<const float4*>(xr + i), v = *reinterpret_cast<const float4*>(row + i);
                 const float4 w = w_post ? *reinterpret_cast<const float4*>(w_post + i) : make_float4(1.f, 1.f, 1.f, 1.f);
                 const float4 o = make_float4(a.x + v.x * inv * w.x, a.y + v.y * inv * w.y, a.z + v.z * inv * w.z, a.w + v.w * inv * w.w);
@@ -66,7 +66,7 @@ residual_norm_kernel(float* __restrict__ x, const float* __restrict__ y, int ldy
                 ss = fmaf(o.x, o.x, fmaf(o.y, o.y, fmaf(o.z, o.z, fmaf(o.w, o.w, ss))));
             }
         } else {
-            for (int i = threadIdx.x; i < dim; i += 256) {
+            for (int i = threadIdx.x; i < dim; i += blockDim.x) {
                 const float o = xr[i] + row[i] * inv * (w_post ? w_post[i] : 1.0f);
                 xr[i] = o;
                 row[i] = o;
@@ -74,19 +74,19 @@ residual_norm_kernel(float* __restrict__ x, const float* __restrict__ y, int ldy
             }
         }
     } else if (VEC) {
-        for (int i = threadIdx.x * 4; i < dim; i += 1024) {
+        for (int i = threadIdx.x * 4; i < dim; i += blockDim.x * 4) {
             const float4 v = *reinterpret_cast<const float4*>(xr + i);
             *reinterpret_cast<float4*>(row + i) = v;
             ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
         }
     } else {
-        for (int i = threadIdx.x; i < dim; i += 256) { const float v = xr[i]; row[i] = v; ss = fmaf(v, v, ss); }
+        for (int i = threadIdx.x; i < dim; i += blockDim.x) { const float v = xr[i]; row[i] = v; ss = fmaf(v, v, ss); }
     }
     if (!w_next) return;
     const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)dim + eps);
     TO* o = out + (size_t)r * ldo;
     if (VEC) {
-        for (int i = threadIdx.x * 4; i < dim; i += 1024) {
+        for (int i = threadIdx.x * 4; i < dim; i += blockDim.x * 4) {
             const float4 v = *reinterpret_cast<const float4*>(row + i), w = *reinterpret_cast<const float4*>(w_next + i);
             const float a = v.x * inv * w.x, b = v.y * inv * w.y, c = v.z * inv * w.z, d = v.w * inv * w.w;
             if (sizeof(TO) == 2) {
@@ -97,7 +97,7 @@ residual_norm_kernel(float* __restrict__ x, const float* __restrict__ y, int ldy
             }
         }
     } else {
-        for (int i = threadIdx.x; i < dim; i += 256) o[i] = narrow<TO>(row[i] * inv * w_next[i]);
+        for (int i = threadIdx.x; i < dim; i += blockDim.x) o[i] = narrow<TO>(row[i] * inv * w_next[i]);
     }
 }
 
@@ -105,29 +105,63 @@ residual_norm_kernel(float* __restrict__ x, const float* __restrict__ y, int ldy
 // multiplied by the temperature of its position and left in place (fp32); k is normed the same way and
 // goes with v into the row's cache slot, each head padded with zeros to its stride in the pool.
 template <typename KV>
+__device__ __forceinline__ void store4(KV* dst, float4 v) {
+    if (sizeof(KV) == 4) *reinterpret_cast<float4*>(dst) = v;
+    else {
+        const KV h[4] = {narrow<KV>(v.x), narrow<KV>(v.y), narrow<KV>(v.z), narrow<KV>(v.w)};
+        *reinterpret_cast<uint2*>(dst) = *reinterpret_cast<const uint2*>(h);
+    }
+}
+
+// VEC: dim and vdim are multiples of 4 and so is the row stride: four elements at a time, none of which
+// straddles a head.
+template <typename KV, bool VEC>
 __global__ void __launch_bounds__(256)
 qk_norm_append_kernel(float* __restrict__ qkv, int ld, const int* __restrict__ row_pos, const int* __restrict__ row_slot,
                       const cmlb200_attn a, KV* __restrict__ kpool, KV* __restrict__ vpool) {
-    __shared__ float red[32];
+    __shared__ float2 red[32];
     dep_wait();
     dep_trigger();
     const int r = blockIdx.x, qw = a.heads * a.dim, kw = a.kv_heads * a.dim;
     float* row = qkv + (size_t)r * ld;
     const int p = row_pos[r];
-    float sq = 0.f, sk = 0.f;
-    for (int i = threadIdx.x; i < qw; i += 256) { const float v = row[i]; sq = fmaf(v, v, sq); }
-    for (int i = threadIdx.x; i < kw; i += 256) { const float v = row[qw + i]; sk = fmaf(v, v, sk); }
-    const float iq = a.q_norm ? 1.0f / sqrtf(block_sum(sq, red) / (float)qw + a.eps) : 1.0f;
-    const float ik = a.k_norm ? 1.0f / sqrtf(block_sum(sk, red) / (float)kw + a.eps) : 1.0f;
-    const float temp = a.temp_every > 0.f ? 1.0f + a.temp_coef * logf(floorf((float)(p + 1) / a.temp_every) + 1.0f) : 1.0f;
-    for (int i = threadIdx.x; i < qw; i += 256) row[i] = row[i] * iq * (a.q_norm ? a.q_norm[i] : 1.0f) * temp;
     const size_t slot = (size_t)a.block_table[(size_t)row_slot[r] * a.table_ld + p / a.block_size] * a.block_size + p % a.block_size;
+    const float2 ss = block_sum2(square_share(row, qw), square_share(row + qw, kw), red);
+    const float temp = a.temp_every > 0.f ? 1.0f + a.temp_coef * logf(floorf((float)(p + 1) / a.temp_every) + 1.0f) : 1.0f;
+    const float iq = a.q_norm ? 1.0f / sqrtf(ss.x / (float)qw + a.eps) : 1.0f, ik = a.k_norm ? 1.0f / sqrtf(ss.y / (float)kw + a.eps) : 1.0f;
     KV* kd = kpool + slot * a.kv_heads * a.dim_ld;
+    KV* vd = vpool + slot * a.kv_heads * a.vdim_ld;
+    if (VEC) {
+#pragma unroll 4
+        for (int i = threadIdx.x * 4; i < qw; i += 1024) {
+            float4 v = *reinterpret_cast<const float4*>(row + i);
+            const float4 w = a.q_norm ? *reinterpret_cast<const float4*>(a.q_norm + i) : make_float4(1.f, 1.f, 1.f, 1.f);
+            v.x = v.x * iq * w.x * temp; v.y = v.y * iq * w.y * temp; v.z = v.z * iq * w.z * temp; v.w = v.w * iq * w.w * temp;
+            *reinterpret_cast<float4*>(row + i) = v;
+        }
+#pragma unroll 4
+        for (int i = threadIdx.x * 4; i < a.kv_heads * a.dim_ld; i += 1024) {
+            const int g = i / a.dim_ld, d = i - g * a.dim_ld, c = g * a.dim + d;
+            float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (d < a.dim) {
+                v = *reinterpret_cast<const float4*>(row + qw + c);
+                const float4 w = a.k_norm ? *reinterpret_cast<const float4*>(a.k_norm + c) : make_float4(1.f, 1.f, 1.f, 1.f);
+                v.x *= ik * w.x; v.y *= ik * w.y; v.z *= ik * w.z; v.w *= ik * w.w;
+            }
+            store4(kd + i, v);
+        }
+#pragma unroll 4
+        for (int i = threadIdx.x * 4; i < a.kv_heads * a.vdim_ld; i += 1024) {
+            const int g = i / a.vdim_ld, d = i - g * a.vdim_ld;
+            store4(vd + i, d < a.vdim ? *reinterpret_cast<const float4*>(row + qw + kw + g * a.vdim + d) : make_float4(0.f, 0.f, 0.f, 0.f));
+        }
+        return;
+    }
+    for (int i = threadIdx.x; i < qw; i += 256) row[i] = row[i] * iq * (a.q_norm ? a.q_norm[i] : 1.0f) * temp;
     for (int i = threadIdx.x; i < a.kv_heads * a.dim_ld; i += 256) {
         const int g = i / a.dim_ld, d = i - g * a.dim_ld, c = g * a.dim + d;
         kd[i] = narrow<KV>(d < a.dim ? row[qw + c] * ik * (a.k_norm ? a.k_norm[c] : 1.0f) : 0.f);
     }
-    KV* vd = vpool + slot * a.kv_heads * a.vdim_ld;
     for (int i = threadIdx.x; i < a.kv_heads * a.vdim_ld; i += 256) {
         const int g = i / a.vdim_ld, d = i - g * a.vdim_ld;
         vd[i] = narrow<KV>(d < a.vdim ? row[qw + kw + g * a.vdim + d] : 0.f);
@@ -167,7 +201,7 @@ extern "C" int cmlb200_embed_rows(const void* d_table, int dtype, const int* d_t
                                   int vocab, float* d_x, void* stream) {
     CMLB_REQUIRE(d_table && d_tokens && d_pos && d_x && rows > 0 && width > 0 && vocab > 0, "cmlb200_embed_rows: bad argument");
     CMLB_REQUIRE(dtype == CMLB200_DT_F32 || dtype == CMLB200_DT_BF16, "cmlb200_embed_rows: dtype %d", dtype);
-    const dim3 grid(rows, rows < 64 ? (width + 2047) / 2048 : 1);
+    const dim3 grid(rows, rows < 64 ? (width + 511) / 512 : 1);
     cudaStream_t st = as_stream(stream);
     if (dtype == CMLB200_DT_BF16)
         CMLB_CUDA(launch_chain(embed_rows_kernel<__nv_bfloat16>, grid, dim3(256), 0, 1, st, (const __nv_bfloat16*)d_table, d_tokens, d_pos, d_freq, width, vocab, d_x));
@@ -186,13 +220,16 @@ extern "C" int cmlb200_residual_norm(float* d_x, const float* d_y, int ldy, cons
     CMLB_REQUIRE(smem <= 200 * 1024, "cmlb200_residual_norm: rows of %d elements do not fit shared memory", dim);
     const bool vec = dim % 4 == 0 && (!d_y || ldy % 4 == 0) && (!d_w_next || ldo % 4 == 0) &&
                      (((uintptr_t)d_x | (uintptr_t)d_y | (uintptr_t)d_w_post | (uintptr_t)d_w_next | (uintptr_t)d_out) & 15) == 0;
+    // few rows: enough threads that each meets its row once; many rows: small CTAs, several to an SM
+    int threads = 256;
+    if (rows <= 2 * cmlb_num_sms()) while (threads < 1024 && threads * 4 < dim) threads *= 2;
     cudaStream_t st = as_stream(stream);
     static size_t attr[4][kMaxDevices] = {};
 #define RN_LAUNCH(TO, V, slot)                                                                                                      \
     do {                                                                                                                            \
         auto kern = residual_norm_kernel<TO, V>;                                                                                    \
         CMLB_CUDA(cmlb_ensure_smem(kern, smem, attr[slot]));                                                                        \
-        CMLB_CUDA(launch_chain(kern, dim3(rows), dim3(256), smem, 1, st, d_x, d_y, ldy, d_w_post, d_w_next, eps, dim, d_row_idx, (TO*)d_out, ldo)); \
+        CMLB_CUDA(launch_chain(kern, dim3(rows), dim3(threads), smem, 1, st, d_x, d_y, ldy, d_w_post, d_w_next, eps, dim, d_row_idx, (TO*)d_out, ldo)); \
     } while (0)
     if (out_dtype == CMLB200_DT_BF16) { if (vec) RN_LAUNCH(__nv_bfloat16, true, 0); else RN_LAUNCH(__nv_bfloat16, false, 1); }
     else { if (vec) RN_LAUNCH(float, true, 2); else RN_LAUNCH(float, false, 3); }
@@ -207,10 +244,11 @@ extern "C" int cmlb200_qk_norm_append(const cmlb200_attn* a, float* d_qkv, int l
     if (rc) return rc;
     CMLB_REQUIRE(ld >= a->heads * a->dim + a->kv_heads * (a->dim + a->vdim), "cmlb200_qk_norm_append: row stride %d", ld);
     cudaStream_t st = as_stream(stream);
-    if (a->cache_dtype == CMLB200_DT_F32)
-        CMLB_CUDA(launch_chain(qk_norm_append_kernel<float>, dim3(rows), dim3(256), 0, 1, st, d_qkv, ld, d_row_pos, d_row_slot, *a, (float*)a->k_pool, (float*)a->v_pool));
-    else
-        CMLB_CUDA(launch_chain(qk_norm_append_kernel<__half>, dim3(rows), dim3(256), 0, 1, st, d_qkv, ld, d_row_pos, d_row_slot, *a, (__half*)a->k_pool, (__half*)a->v_pool));
+    const bool vec = a->dim % 4 == 0 && a->vdim % 4 == 0 && ld % 4 == 0 && (((uintptr_t)d_qkv | (uintptr_t)a->q_norm | (uintptr_t)a->k_norm) & 15) == 0;
+#define QK_LAUNCH(KV, V) CMLB_CUDA(launch_chain(qk_norm_append_kernel<KV, V>, dim3(rows), dim3(256), 0, 1, st, d_qkv, ld, d_row_pos, d_row_slot, *a, (KV*)a->k_pool, (KV*)a->v_pool))
+    if (a->cache_dtype == CMLB200_DT_F32) { if (vec) QK_LAUNCH(float, true); else QK_LAUNCH(float, false); }
+    else { if (vec) QK_LAUNCH(__half, true); else QK_LAUNCH(__half, false); }
+#undef QK_LAUNCH
     return CMLB200_OK;
 }
 

@@ -51,6 +51,33 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
     return t;
 }
 
+// Two sums at once.
+__device__ __forceinline__ float2 block_sum2(float a, float b, float2* red) {
+    a = lane_sum(a);
+    b = lane_sum(b);
+    __syncthreads();
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = make_float2(a, b);
+    __syncthreads();
+    float2 t = make_float2(0.f, 0.f);
+    for (int k = 0; k < (int)(blockDim.x >> 5); k++) { t.x += red[k].x; t.y += red[k].y; }
+    return t;
+}
+// This thread's share of the sum of squares of n floats; 16-byte loads where p allows them.
+__device__ __forceinline__ float square_share(const float* p, int n) {
+    float s = 0.f;
+    if ((((uintptr_t)p | (unsigned)(n * 4)) & 15) == 0) {
+#pragma unroll 4
+        for (int i = threadIdx.x; i < (n >> 2); i += blockDim.x) {
+            const float4 v = reinterpret_cast<const float4*>(p)[i];
+            s = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, s))));
+        }
+    } else {
+#pragma unroll 4
+        for (int i = threadIdx.x; i < n; i += blockDim.x) { const float v = p[i]; s = fmaf(v, v, s); }
+    }
+    return s;
+}
+
 __device__ __forceinline__ float widen(float v) { return v; }
 __device__ __forceinline__ float widen(__nv_bfloat16 v) { return __bfloat162float(v); }
 __device__ __forceinline__ float widen(__half v) { return __half2float(v); }
