@@ -233,12 +233,6 @@ def write_random_llama_gguf(path, rng, cfg, qtype=2, weight_std=0.02, alias_laye
 
 
 # ---- layered models: a folder with config.json and model.safetensors --------------------------------
-def bf16_round(a):
-    """fp32 values rounded to the nearest bf16 (ties to even), as fp32."""
-    u = np.ascontiguousarray(a, np.float32).view(np.uint32).astype(np.uint64)
-    return (((u + 0x7FFF + ((u >> 16) & 1)) >> 16).astype(np.uint32) << 16).view(np.float32)
-
-
 def layered_layer(heads, kv_heads, dim, vdim, window, ff, scale=None, coef=0.2, every=50, weights_of=None):
     layer = {"type": "attention", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale or dim ** -0.5,
                                             "mask": {"size": window}, "q_temp": {"coef": coef, "every": every}},
@@ -274,7 +268,7 @@ def layered_weights(rng, cfg):
     w = {}
     for name, shape in layered_shapes(cfg).items():
         a = rng.standard_normal(shape, dtype=np.float32)
-        w[name] = bf16_round(1.0 + 0.2 * a if len(shape) == 1 else (a if name == "embed" else a / np.sqrt(shape[1])))
+        w[name] = bf16_round(1.0 + 0.2 * a if len(shape) == 1 else (a if name == "embed" else a / np.sqrt(shape[1])))[1]
     return w
 
 
@@ -302,4 +296,4 @@ def write_layered(folder, cfg, weights, alias_layers=False):
         f.write(len(text).to_bytes(8, "little") + text)
         for name, shape in stored:
             a = weights(name, shape) if callable(weights) else weights[name]
-            f.write((bf16_round(a).view(np.uint32) >> 16).astype(np.uint16).tobytes())
+            f.write(bf16_round(a)[0].tobytes())

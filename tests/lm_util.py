@@ -21,12 +21,10 @@ def variants(synth):
     }
 
 
-def build(synth, tmp_path, name, seed=0, **tweak):
+def build(synth, tmp_path, name, seed=0):
     cfg = variants(synth)[name]
     rng = np.random.default_rng(seed + sum(map(ord, name)))
     w = synth.layered_weights(rng, cfg)
-    for k, f in tweak.items():
-        w[k] = synth.bf16_round(f(w[k]))
     folder = tmp_path / f"{name}_{seed}"
     synth.write_layered(folder, cfg, w)
     return cfg, w, folder

@@ -114,7 +114,7 @@ SHAPES = [(16, 64), (75, 75), (200, 144), (1000, 33), (130, 1111), (2064, 520)]
 def test_decode_product(pkg, synth, torch_dev, N, K, M):
     import torch
     r = RNG(N + K + M)
-    w, x = synth.bf16_round(r.standard_normal((N, K))), synth.bf16_round(r.standard_normal((M, K)))
+    w, x = synth.bf16_round(r.standard_normal((N, K)))[1], synth.bf16_round(r.standard_normal((M, K)))[1]
     t, W = dense(pkg, torch_dev, w, pkg.DT_BF16)
     xd = operand(torch_dev, x)
     y = torch.full((M + 1, N + 5), 7.0, device=torch_dev)
@@ -130,7 +130,7 @@ def test_decode_product(pkg, synth, torch_dev, N, K, M):
 def test_prompt_product(pkg, synth, torch_dev, N, K, M):
     import torch
     r = RNG(N + K + M)
-    w, x = synth.bf16_round(r.standard_normal((N, K))), synth.bf16_round(r.standard_normal((M, K)))
+    w, x = synth.bf16_round(r.standard_normal((N, K)))[1], synth.bf16_round(r.standard_normal((M, K)))[1]
     t, W = dense(pkg, torch_dev, w, pkg.DT_BF16)
     xd = operand(torch_dev, x)
     y = torch.full((M + 1, N + 5), 7.0, device=torch_dev)
@@ -165,8 +165,8 @@ def test_prompt_product_many_tiles_per_cta(pkg, torch_dev, M, N, K):
 def test_gated_products(pkg, synth, torch_dev, ff, K, M, act):
     import torch
     r = RNG(ff + K + M)
-    g, u = (synth.bf16_round(r.standard_normal((ff, K)) / K ** 0.5) for _ in range(2))
-    x = synth.bf16_round(r.standard_normal((M, K)))
+    g, u = (synth.bf16_round(r.standard_normal((ff, K)) / K ** 0.5)[1] for _ in range(2))
+    x = synth.bf16_round(r.standard_normal((M, K)))[1]
     rows = (ff + 15) // 16 * 32
     w = np.zeros((rows, K), np.float32)
     c = np.arange(ff) // 16 * 32 + np.arange(ff) % 16
