@@ -430,7 +430,7 @@ REFERENCE_QUIRKS, KV_FP32, ALL_LOGITS_FP32 = 1, 2, 4
 
 # ---- layered models (include/cml_lm.h and the kernels behind it) ---------------------------------
 DT_F32, DT_BF16, DT_F16 = 0, 1, 2
-ACT_SILU, ACT_GELU_TANH = 0, 1
+ACT_SILU, ACT_GELU_TANH, ACT_CLAMPED = 0, 1, 2
 DTYPE_FLOAT32, DTYPE_BFLOAT16 = 0, 6
 
 
@@ -444,7 +444,20 @@ class Attn(C.Structure):
     _fields_ = [("heads", ci), ("kv_heads", ci), ("dim", ci), ("vdim", ci), ("dim_ld", ci), ("vdim_ld", ci), ("scale", C.c_float),
                 ("window", ci), ("slopes", vp), ("sink", ci), ("q_norm", vp), ("k_norm", vp), ("eps", C.c_float), ("temp_coef", C.c_float),
                 ("temp_every", C.c_float), ("gate_col", ci), ("cache_dtype", ci), ("k_pool", vp), ("v_pool", vp), ("block_size", ci),
-                ("block_table", vp), ("table_ld", ci)]
+                ("block_table", vp), ("table_ld", ci), ("gate_wide", ci)]
+
+
+class Latent(C.Structure):
+    """cmlb200_latent."""
+    _fields_ = [("heads", ci), ("dim", ci), ("rot_dim", ci), ("vdim", ci), ("rank", ci), ("ld", ci), ("ld_rank", ci), ("scale", C.c_float), ("window", ci),
+                ("c_norm", vp), ("eps", C.c_float), ("freq", vp), ("rot_mul", C.c_float), ("kv_col", ci), ("gate_col", ci), ("cache_dtype", ci), ("pool", vp),
+                ("block_size", ci), ("block_table", vp), ("table_ld", ci)]
+
+
+class Moe(C.Structure):
+    """cmlb200_moe."""
+    _fields_ = [("experts", ci), ("top", ci)] + [(n, vp) for n in ("ids", "weight", "pos", "src", "expert", "start", "count", "active", "num_active", "tiles",
+                                                                     "num_tiles")]
 
 
 class LMOptions(C.Structure):
@@ -467,6 +480,26 @@ for _n in ("cmlb200_gemv_dense_glu", "cmlb200_gemm_dense_glu"):
     _sig(_n, ci, C.POINTER(Dense), vp, ci, ci, ci, ci, vp, ci, vp)
 _sig("cmlb200_gemm_dense_status", ci, C.POINTER(ci), ci)
 _sig("cmlb200_glu_rows_f32", ci, vp, ci, ci, ci, ci, vp, ci, vp)
+_LAT, _MOE, _DENSE, _cf = C.POINTER(Latent), C.POINTER(Moe), C.POINTER(Dense), C.c_float
+_sig("cmlb200_residual_add", ci, vp, vp, ci, _MOE, vp, _cf, ci, ci, vp, ci, ci, vp)
+_sig("cmlb200_poly_norm", ci, vp, ci, ci, ci, vp, _cf, vp, ci, ci, vp)
+_sig("cmlb200_latent_append", ci, _LAT, vp, ci, vp, vp, ci, vp)
+for _n in ("cmlb200_latent_query", "cmlb200_latent_query_f32"):
+    _sig(_n, ci, _LAT, vp, vp, ci, vp, vp, ci, vp, vp)
+_sig("cmlb200_attention_latent", ci, _LAT, vp, vp, vp, ci, ci, vp, ci, vp, vp)
+for _n in ("cmlb200_latent_output", "cmlb200_latent_output_f32"):
+    _sig(_n, ci, _LAT, vp, vp, vp, ci, ci, vp, ci, vp)
+_sig("cmlb200_latent_gather", ci, _LAT, vp, ci, vp, C.POINTER(Attn), vp)
+_sig("cmlb200_latent_expand", ci, _LAT, _DENSE, vp, ci, C.POINTER(Attn), vp)
+_sig("cmlb200_moe_positions", C.c_long, ci, ci, ci, ci)
+_sig("cmlb200_moe_route", ci, _MOE, vp, ci, ci, ci, vp)
+_sig("cmlb200_moe_gather", ci, _MOE, vp, ci, ci, ci, vp, ci, vp)
+_sig("cmlb200_moe_gemv", ci, _MOE, _DENSE, vp, ci, ci, ci, ci, vp, ci, vp)
+_sig("cmlb200_moe_gemv_glu", ci, _MOE, _DENSE, vp, ci, ci, ci, ci, ci, _cf, vp, ci, vp)
+_sig("cmlb200_moe_gemm", ci, _MOE, _DENSE, vp, ci, ci, ci, vp, ci, vp)
+_sig("cmlb200_moe_gemm_glu", ci, _MOE, _DENSE, vp, ci, ci, ci, ci, _cf, vp, ci, vp)
+_sig("cmlb200_moe_linear_f32", ci, _MOE, _DENSE, vp, ci, ci, ci, ci, vp, ci, vp)
+_sig("cmlb200_moe_glu_rows_f32", ci, vp, ci, ci, ci, ci, _cf, vp, ci, vp)
 _sig("cml_lm_default_options", LMOptions)
 _sig("cml_lm_known", ci, C.c_char_p)
 _sig("cml_lm_load", vp, C.c_char_p, C.POINTER(LMOptions))

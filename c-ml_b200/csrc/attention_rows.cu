@@ -15,40 +15,14 @@
 //
 // Scores are kept in units of log2 in the first two kernels (the scale carries log2 e). A sink starts
 // the running maximum at 0, so its weight exp(0 - m) joins the denominator exactly once.
-#include <cuda_fp16.h>
 #include "lm_util.cuh"
 
 namespace {
 
-constexpr float kLog2e = 1.4426950408889634f;
-
-__device__ __forceinline__ uint32_t smem_addr(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
-__device__ __forceinline__ void cp16(uint32_t dst, const void* src) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
-}
-__device__ __forceinline__ void mma_f16(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.f16.f16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ void ldsm4(uint32_t addr, uint32_t (&r)[4]) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
-}
-__device__ __forceinline__ void ldsm4_t(uint32_t addr, uint32_t (&r)[4]) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
-}
 __device__ __forceinline__ uint32_t pack_h2(float lo, float hi) {
     const __half2 v = __floats2half2_rn(lo, hi);
     return *reinterpret_cast<const uint32_t*>(&v);
 }
-__device__ __forceinline__ float ex2(float v) {
-    float r;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(v));
-    return r;
-}
-__device__ __forceinline__ float sigmoidf(float z) { return 1.0f / (1.0f + expf(-z)); }
-
 constexpr int QT = 64, KT = 64, TILE_THREADS = 128;
 
 // grid = (tiles, heads). tiles[i] = {first row, rows (1..64), sequence slot, position of the first row}.
@@ -200,7 +174,7 @@ attention_tiles_kernel(const cmlb200_attn a, const float* __restrict__ qkv, int 
     l1 += __shfl_xor_sync(0xffffffffu, l1, 1); l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
     if (a.sink) { l0 += exp2f(-m0); l1 += exp2f(-m1); }
     float i0 = l0 > 0.f ? 1.0f / l0 : 0.f, i1 = l1 > 0.f ? 1.0f / l1 : 0.f;
-    if (a.gate_col >= 0) {
+    if (a.gate_col >= 0 && !a.gate_wide) {
         if (r0 < n) i0 *= sigmoidf(qkv[(size_t)(tl.x + r0) * ld + a.gate_col + h]);
         if (r1 < n) i1 *= sigmoidf(qkv[(size_t)(tl.x + r1) * ld + a.gate_col + h]);
     }
@@ -208,6 +182,12 @@ attention_tiles_kernel(const cmlb200_attn a, const float* __restrict__ qkv, int 
 #pragma unroll
     for (int i = 0; i < DV / 8; i++) {
         const int d = i * 8 + 2 * t;
+        if (a.gate_wide && d < a.vdim) {
+            const float* g0 = qkv + (size_t)(tl.x + r0) * ld + a.gate_col + h * a.vdim + d;
+            const float* g1 = g0 + (size_t)8 * ld;
+            if (r0 < n) { o[i][0] *= sigmoidf(g0[0]); if (d + 1 < a.vdim) o[i][1] *= sigmoidf(g0[1]); }
+            if (r1 < n) { o[i][2] *= sigmoidf(g1[0]); if (d + 1 < a.vdim) o[i][3] *= sigmoidf(g1[1]); }
+        }
         __nv_bfloat16* a0 = out + (size_t)(tl.x + r0) * out_ld + h * a.vdim + d;
         __nv_bfloat16* a1 = out + (size_t)(tl.x + r1) * out_ld + h * a.vdim + d;
         if (pairs) {
@@ -529,6 +509,7 @@ extern "C" int cmlb200_attn_check_(const cmlb200_attn* a, const char* who) {
     CMLB_REQUIRE(a->dim > 0 && a->vdim > 0 && a->dim_ld >= a->dim && a->vdim_ld >= a->vdim && a->dim_ld % 16 == 0 && a->vdim_ld % 16 == 0,
                  "%s: head sizes %d (stride %d) / %d (stride %d)", who, a->dim, a->dim_ld, a->vdim, a->vdim_ld);
     CMLB_REQUIRE(a->cache_dtype == CMLB200_DT_F32 || a->cache_dtype == CMLB200_DT_F16, "%s: cache dtype %d", who, a->cache_dtype);
+    CMLB_REQUIRE(!a->gate_wide || a->gate_col >= 0, "%s: gate_wide without a gate column", who);
     CMLB_REQUIRE(a->k_pool && a->v_pool && a->block_table && a->table_ld > 0, "%s: no cache", who);
     CMLB_REQUIRE(a->block_size > 0 && (a->block_size & (a->block_size - 1)) == 0 && a->block_size % 16 == 0, "%s: block size %d must be a power of two >= 16", who, a->block_size);
     CMLB_REQUIRE((((uintptr_t)a->k_pool | (uintptr_t)a->v_pool) & 15) == 0, "%s: pools must be 16-byte aligned", who);
@@ -546,7 +527,7 @@ extern "C" int cmlb200_attention_tiles(const cmlb200_attn* a, const float* d_qkv
     CMLB_REQUIRE(smem <= 227 * 1024, "cmlb200_attention_tiles: head sizes %d / %d do not fit shared memory", a->dim, a->vdim);
     cudaStream_t st = as_stream(stream);
     const dim3 grid(tiles, a->heads);
-    static size_t attr[5][kMaxDevices] = {};
+    static size_t attr[6][kMaxDevices] = {};
 #define AT_LAUNCH(DV, DK, slot)                                                                                                   \
     do {                                                                                                                        \
         auto kern = attention_tiles_kernel<DV, DK>;                                                                               \
@@ -555,6 +536,7 @@ extern "C" int cmlb200_attention_tiles(const cmlb200_attn* a, const float* d_qkv
     } while (0)
     if (a->vdim_ld == 64 && a->dim_ld == 64) AT_LAUNCH(64, 64, 3);
     else if (a->vdim_ld == 128 && a->dim_ld == 128) AT_LAUNCH(128, 128, 4);
+    else if (a->vdim_ld == 128 && a->dim_ld == 192) AT_LAUNCH(128, 192, 5);
     else if (a->vdim_ld <= 64) AT_LAUNCH(64, 0, 0);
     else if (a->vdim_ld <= 128) AT_LAUNCH(128, 0, 1);
     else AT_LAUNCH(256, 0, 2);
@@ -568,6 +550,7 @@ extern "C" int cmlb200_attention_one(const cmlb200_attn* a, const float* d_qkv, 
     const int rc = cmlb200_attn_check_(a, "cmlb200_attention_one");
     if (rc) return rc;
     CMLB_REQUIRE(a->cache_dtype == CMLB200_DT_F16 && a->vdim_ld <= 256 && rows <= 65535, "cmlb200_attention_one: fp16 cache and value heads up to 256");
+    CMLB_REQUIRE(!a->gate_wide, "cmlb200_attention_one: one gate per head");
     // few rows: fewer heads per CTA, so that more CTAs share the work (the keys are read again from L2)
     const int group = a->heads / a->kv_heads, rm = group == 1 ? 1 : (group <= 4 || rows * a->kv_heads * 8 < cmlb_num_sms() ? 4 : 8), passes = (group + rm - 1) / rm;
     CMLB_REQUIRE((long long)a->kv_heads * passes <= 65535, "cmlb200_attention_one: too many heads");
@@ -607,6 +590,7 @@ extern "C" int cmlb200_attention_rows_f32(const cmlb200_attn* a, const float* d_
     const int rc = cmlb200_attn_check_(a, "cmlb200_attention_rows_f32");
     if (rc) return rc;
     CMLB_REQUIRE(a->cache_dtype == CMLB200_DT_F32 && a->heads <= 65535, "cmlb200_attention_rows_f32: fp32 cache");
+    CMLB_REQUIRE(!a->gate_wide, "cmlb200_attention_rows_f32: one gate per head");
     const size_t smem = sizeof(float) * ((size_t)a->dim + a->vdim);
     CMLB_REQUIRE(smem <= 40 * 1024, "cmlb200_attention_rows_f32: head sizes %d / %d", a->dim, a->vdim);
     CMLB_CUDA(launch_chain(attention_rows_f32_kernel, dim3(rows, a->heads), dim3(ROW_THREADS), smem, 1, as_stream(stream), *a, d_qkv, ld, d_row_pos,

@@ -15,26 +15,32 @@ namespace {
 
 constexpr int GV_WARPS = 8;
 
-__device__ __forceinline__ uint4 ld_stream(const __nv_bfloat16* p) {
-    uint4 v;
-    asm volatile("ld.global.nc.L1::no_allocate.L2::128B.v4.u32 {%0,%1,%2,%3}, [%4];" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "l"(p));
-    return v;
-}
-__device__ __forceinline__ void mma_bf16(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
-}
-
 // RT tiles of 16 weight rows per CTA, NB groups of 8 rows of x. GLU: tile 0 = 16 gate rows, tile 1 = the
 // 16 up rows that go with them; the output is bf16 act(gate) * up.
-template <int RT, int NB, bool GLU>
+// EXPERT: blockIdx.y counts the chosen experts; an expert's w_rows weight rows follow those of the one before it, its
+// rows of x are those that chose it (m.src, or the positions themselves), and y has a row per position.
+struct GemvExperts {
+    cmlb200_moe m;
+    int w_rows, gather;
+};
+template <int RT, int NB, bool GLU, bool EXPERT>
 __global__ void __launch_bounds__(GV_WARPS * 32)
 gemv_bf16_kernel(const __nv_bfloat16* __restrict__ W, int ldw, const __nv_bfloat16* __restrict__ x, int ldx, int M, int N, int K, int act,
-                 void* __restrict__ y, int ldy) {
+                 float limit, void* __restrict__ y, int ldy, const GemvExperts ex) {
     __shared__ float part[GV_WARPS][RT * 16][NB * 8 + 1];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, t = lane & 3;
     const int n0 = blockIdx.x * RT * 16;
     const int chunks = (K + 63) / 64;
+    int first = 0;
+    if (EXPERT) {                                       // which weights are needed is known only now
+        dep_wait();
+        dep_trigger();
+        if ((int)blockIdx.y >= *ex.m.num_active) return;
+        const int e = ex.m.active[blockIdx.y];
+        first = ex.m.start[e];
+        M = ex.m.count[e];
+        W += (size_t)e * ex.w_rows * ldw;
+    }
     const __nv_bfloat16* wrow[RT][2];
 #pragma unroll
     for (int i = 0; i < RT; i++) {
@@ -54,8 +60,10 @@ gemv_bf16_kernel(const __nv_bfloat16* __restrict__ W, int ldw, const __nv_bfloat
     };
 #pragma unroll
     for (int u = 0; u < RING; u++) fetch(u, warp + u * GV_WARPS);
-    dep_wait();
-    dep_trigger();
+    if (!EXPERT) {
+        dep_wait();
+        dep_trigger();
+    }
     float acc[RT][NB][4];
 #pragma unroll
     for (int i = 0; i < RT; i++)
@@ -63,13 +71,18 @@ gemv_bf16_kernel(const __nv_bfloat16* __restrict__ W, int ldw, const __nv_bfloat
         for (int b = 0; b < NB; b++) { acc[i][b][0] = 0.f; acc[i][b][1] = 0.f; acc[i][b][2] = 0.f; acc[i][b][3] = 0.f; }
     const __nv_bfloat16* xr[NB];
 #pragma unroll
-    for (int b = 0; b < NB; b++) xr[b] = x + (size_t)min(b * 8 + g, M - 1) * ldx + 8 * t;      // rows past M repeat the last, never stored
+    for (int b = 0; b < NB; b++) {                      // rows past M repeat the last, never stored
+        int r = min(b * 8 + g, M - 1);
+        if (EXPERT) r = ex.gather ? ex.m.src[first + r] : first + r;
+        xr[b] = x + (size_t)r * ldx + 8 * t;
+    }
     for (int c0 = warp; c0 < chunks; c0 += RING * GV_WARPS) {
 #pragma unroll
         for (int u = 0; u < RING; u++) {
             const int c = min(c0 + u * GV_WARPS, chunks - 1);         // past the end: zero weights
 #pragma unroll
             for (int b = 0; b < NB; b++) {
+                if (EXPERT && b * 8 >= M) continue;
                 const uint4 x0 = *reinterpret_cast<const uint4*>(xr[b] + (size_t)c * 64), x1 = *reinterpret_cast<const uint4*>(xr[b] + (size_t)c * 64 + 32);
 #pragma unroll
                 for (int i = 0; i < RT; i++) {
@@ -105,9 +118,9 @@ gemv_bf16_kernel(const __nv_bfloat16* __restrict__ W, int ldw, const __nv_bfloat
         }
         if (GLU) {
             const int c = blockIdx.x * 16 + n;
-            if (c < N) static_cast<__nv_bfloat16*>(y)[(size_t)m * ldy + c] = __float2bfloat16_rn(glu_act(act, s, s2));
+            if (c < N) static_cast<__nv_bfloat16*>(y)[(size_t)(first + m) * ldy + c] = __float2bfloat16_rn(glu_act(act, s, s2, limit));
         } else if (n0 + n < N) {
-            static_cast<float*>(y)[(size_t)m * ldy + n0 + n] = s;
+            static_cast<float*>(y)[(size_t)(first + m) * ldy + n0 + n] = s;
         }
     }
 }
@@ -117,11 +130,27 @@ int launch_gemv(const cmlb200_dense* W, const uint16_t* x, int ldx, int M, int a
     const dim3 grid((unsigned)((W->rows + RT * 16 - 1) / (RT * 16)));
     const __nv_bfloat16* w = static_cast<const __nv_bfloat16*>(W->w);
     const __nv_bfloat16* xb = reinterpret_cast<const __nv_bfloat16*>(x);
-#define GV_LAUNCH(NB) CMLB_CUDA(launch_chain(gemv_bf16_kernel<RT, NB, GLU>, grid, dim3(GV_WARPS * 32), 0, 1, st, w, W->ld, xb, ldx, M, n_out, W->cols, act, y, ldy))
+#define GV_LAUNCH(NB) CMLB_CUDA(launch_chain(gemv_bf16_kernel<RT, NB, GLU, false>, grid, dim3(GV_WARPS * 32), 0, 1, st, w, W->ld, xb, ldx, M, n_out, W->cols, act, 0.f, y, ldy, GemvExperts{}))
     if (M <= 8) GV_LAUNCH(1);
     else if (M <= 16) GV_LAUNCH(2);
     else GV_LAUNCH(4);
 #undef GV_LAUNCH
+    return CMLB200_OK;
+}
+
+template <int RT, bool GLU>
+int launch_gemv_experts(const cmlb200_moe* m, const cmlb200_dense* W, const uint16_t* x, int ldx, int gather, int rows, int act, float limit, void* y,
+                        int ldy, int n_out, cudaStream_t st) {
+    const int per = W->rows / m->experts, pairs = rows * m->top;
+    const dim3 grid((unsigned)((GLU ? (per + 31) / 32 : (n_out + 15) / 16)), (unsigned)(pairs < m->experts ? pairs : m->experts));
+    const __nv_bfloat16* w = static_cast<const __nv_bfloat16*>(W->w);
+    const __nv_bfloat16* xb = reinterpret_cast<const __nv_bfloat16*>(x);
+    const GemvExperts ex = {*m, per, gather};
+#define GE_LAUNCH(NB) CMLB_CUDA(launch_chain(gemv_bf16_kernel<RT, NB, GLU, true>, grid, dim3(GV_WARPS * 32), 0, 1, st, w, W->ld, xb, ldx, rows, n_out, W->cols, act, limit, y, ldy, ex))
+    if (rows <= 8) GE_LAUNCH(1);
+    else if (rows <= 16) GE_LAUNCH(2);
+    else GE_LAUNCH(4);
+#undef GE_LAUNCH
     return CMLB200_OK;
 }
 
@@ -147,4 +176,22 @@ extern "C" int cmlb200_gemv_dense_glu(const cmlb200_dense* W, const uint16_t* d_
     if (rc) return rc;
     CMLB_REQUIRE(ff > 0 && W->rows == 2 * ((ff + 15) & ~15) && ldf >= ff, "cmlb200_gemv_dense_glu: %d weight rows for %d outputs", W->rows, ff);
     return launch_gemv<2, true>(W, d_x, ldx, M, act, d_f, ldf, ff, as_stream(stream));
+}
+
+extern "C" int cmlb200_moe_gemv(const cmlb200_moe* m, const cmlb200_dense* W, const uint16_t* d_x, int ldx, int gather, int rows, int n_out, float* d_y,
+                                int ldy, void* stream) {
+    const int rc = check_gemv(W, d_x, ldx, rows, d_y, "cmlb200_moe_gemv");
+    if (rc) return rc;
+    CMLB_REQUIRE(m && m->experts > 0 && m->experts <= 65535 && W->rows % (16 * m->experts) == 0 && n_out > 0 && n_out <= W->rows / m->experts && ldy >= n_out,
+                 "cmlb200_moe_gemv: %d weight rows, %d outputs, stride %d", W->rows, n_out, ldy);
+    return launch_gemv_experts<1, false>(m, W, d_x, ldx, gather, rows, 0, 0.f, d_y, ldy, n_out, as_stream(stream));
+}
+
+extern "C" int cmlb200_moe_gemv_glu(const cmlb200_moe* m, const cmlb200_dense* W, const uint16_t* d_x, int ldx, int gather, int rows, int ff, int act,
+                                    float limit, uint16_t* d_f, int ldf, void* stream) {
+    const int rc = check_gemv(W, d_x, ldx, rows, d_f, "cmlb200_moe_gemv_glu");
+    if (rc) return rc;
+    CMLB_REQUIRE(m && m->experts > 0 && m->experts <= 65535 && ff > 0 && W->rows == m->experts * 2 * ((ff + 15) & ~15) && ldf >= ff,
+                 "cmlb200_moe_gemv_glu: %d weight rows for %d outputs", W->rows, ff);
+    return launch_gemv_experts<2, true>(m, W, d_x, ldx, gather, rows, act, limit, d_f, ldf, ff, as_stream(stream));
 }

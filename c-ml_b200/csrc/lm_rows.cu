@@ -30,29 +30,46 @@ embed_rows_kernel(const T* __restrict__ table, const int* __restrict__ tokens, c
 }
 
 // One CTA per output row. y == NULL: out = norm(x[idx]) * w_next. Otherwise x += norm(y) * w_post
-// (w_post == NULL: x += y) and, when w_next is given, out = norm(x) * w_next. The row stays in shared
-// memory between the passes. Columns dim .. ldo of `out` are left alone.
-template <typename TO, bool VEC>
+// (w_post == NULL: x += y) and, when w_next is given, out = norm(x) * w_next; raw: out = x. The row stays in
+// shared memory between the passes. Columns dim .. ldo of `out` are left alone. PARTS: row r of y is the sum of the rows
+// part_pos[r * parts + k] with weights part_w[r * parts + k].
+template <typename TO, bool VEC, bool PARTS>
 __global__ void __launch_bounds__(1024)
 residual_norm_kernel(float* __restrict__ x, const float* __restrict__ y, int ldy, const float* __restrict__ w_post,
-                     const float* __restrict__ w_next, float eps, int dim, const int* __restrict__ idx, TO* __restrict__ out, int ldo) {
+                     const float* __restrict__ w_next, float eps, int dim, const int* __restrict__ idx, TO* __restrict__ out, int ldo, int raw,
+                     int parts, const int* __restrict__ part_pos, const float* __restrict__ part_w) {
     extern __shared__ __align__(16) float row[];
     __shared__ float red[32];
     dep_wait();
     dep_trigger();
     const int r = blockIdx.x;
+    auto part_sum = [&](auto zero, int i) {
+        auto s = zero;
+#pragma unroll 4
+        for (int k = 0; k < parts; k++) {
+            const float w = part_w[r * parts + k];
+            const float* p = y + (size_t)part_pos[r * parts + k] * ldy + i;
+            if constexpr (sizeof(s) == 16) {
+                const float4 v = *reinterpret_cast<const float4*>(p);
+                s.x = fmaf(w, v.x, s.x); s.y = fmaf(w, v.y, s.y); s.z = fmaf(w, v.z, s.z); s.w = fmaf(w, v.w, s.w);
+            } else {
+                s = fmaf(w, *p, s);
+            }
+        }
+        return s;
+    };
     float* xr = x + (size_t)(idx ? idx[r] : r) * dim;
     float ss = 0.f;
     if (y) {
         const float* yr = y + (size_t)r * ldy;
         if (VEC) {
             for (int i = threadIdx.x * 4; i < dim; i += blockDim.x * 4) {
-                const float4 v = *reinterpret_cast<const float4*>(yr + i);
+                const float4 v = PARTS ? part_sum(make_float4(0.f, 0.f, 0.f, 0.f), i) : *reinterpret_cast<const float4*>(yr + i);
                 *reinterpret_cast<float4*>(row + i) = v;
                 ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
             }
         } else {
-            for (int i = threadIdx.x; i < dim; i += blockDim.x) { const float v = yr[i]; row[i] = v; ss = fmaf(v, v, ss); }
+            for (int i = threadIdx.x; i < dim; i += blockDim.x) { const float v = PARTS ? part_sum(0.f, i) : yr[i]; row[i] = v; ss = fmaf(v, v, ss); }
         }
         const float inv = w_post ? 1.0f / sqrtf(block_sum(ss, red) / (float)dim + eps) : 1.0f;
         ss = 0.f;
@@ -82,12 +99,12 @@ residual_norm_kernel(float* __restrict__ x, const float* __restrict__ y, int ldy
     } else {
         for (int i = threadIdx.x; i < dim; i += blockDim.x) { const float v = xr[i]; row[i] = v; ss = fmaf(v, v, ss); }
     }
-    if (!w_next) return;
-    const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)dim + eps);
+    if (!w_next && !raw) return;
+    const float inv = raw ? 1.0f : 1.0f / sqrtf(block_sum(ss, red) / (float)dim + eps);
     TO* o = out + (size_t)r * ldo;
     if (VEC) {
         for (int i = threadIdx.x * 4; i < dim; i += blockDim.x * 4) {
-            const float4 v = *reinterpret_cast<const float4*>(row + i), w = *reinterpret_cast<const float4*>(w_next + i);
+            const float4 v = *reinterpret_cast<const float4*>(row + i), w = raw ? make_float4(1.f, 1.f, 1.f, 1.f) : *reinterpret_cast<const float4*>(w_next + i);
             const float a = v.x * inv * w.x, b = v.y * inv * w.y, c = v.z * inv * w.z, d = v.w * inv * w.w;
             if (sizeof(TO) == 2) {
                 const __nv_bfloat162 lo = __floats2bfloat162_rn(a, b), hi = __floats2bfloat162_rn(c, d);
@@ -97,7 +114,51 @@ residual_norm_kernel(float* __restrict__ x, const float* __restrict__ y, int ldy
             }
         }
     } else {
-        for (int i = threadIdx.x; i < dim; i += blockDim.x) o[i] = narrow<TO>(row[i] * inv * w_next[i]);
+        for (int i = threadIdx.x; i < dim; i += blockDim.x) o[i] = narrow<TO>(raw ? row[i] : row[i] * inv * w_next[i]);
+    }
+}
+
+// f = a N(z) + b N(z^2) + c N(z^3) + e, N(v) = v / sqrt(mean(v^2) + eps) over the row. One CTA per row.
+template <typename TO, bool VEC>
+__global__ void __launch_bounds__(1024)
+poly_norm_kernel(const float* __restrict__ z, int ld, int ff, const float* __restrict__ coef, float eps, TO* __restrict__ f, int ldf) {
+    extern __shared__ __align__(16) float row[];
+    __shared__ float red[32];
+    __shared__ float2 red2[32];
+    const float a = coef[0], b = coef[1], c = coef[2], e = coef[3];
+    dep_wait();
+    dep_trigger();
+    const float* zr = z + (size_t)blockIdx.x * ld;
+    float s1 = 0.f, s2 = 0.f, s3 = 0.f;
+    auto add = [&](float v) {
+        const float q = v * v;
+        s1 += q;
+        s2 = fmaf(q, q, s2);
+        s3 = fmaf(q * q, q, s3);
+    };
+    if (VEC) {
+        for (int i = threadIdx.x * 4; i < ff; i += blockDim.x * 4) {
+            const float4 v = *reinterpret_cast<const float4*>(zr + i);
+            *reinterpret_cast<float4*>(row + i) = v;
+            add(v.x); add(v.y); add(v.z); add(v.w);
+        }
+    } else {
+        for (int i = threadIdx.x; i < ff; i += blockDim.x) { const float v = zr[i]; row[i] = v; add(v); }
+    }
+    const float2 t = block_sum2(s1, s2, red2);
+    const float n = (float)ff, u = block_sum(s3, red);
+    const float i1 = a / sqrtf(t.x / n + eps), i2 = b / sqrtf(t.y / n + eps), i3 = c / sqrtf(u / n + eps);
+    auto value = [&](float v) { return fmaf(v, fmaf(v, fmaf(v, i3, i2), i1), e); };
+    TO* o = f + (size_t)blockIdx.x * ldf;
+    if (VEC) {
+        for (int i = threadIdx.x * 4; i < ff; i += blockDim.x * 4) {
+            const float4 v = *reinterpret_cast<const float4*>(row + i);
+            const TO w[4] = {narrow<TO>(value(v.x)), narrow<TO>(value(v.y)), narrow<TO>(value(v.z)), narrow<TO>(value(v.w))};
+            if (sizeof(TO) == 2) *reinterpret_cast<uint2*>(o + i) = *reinterpret_cast<const uint2*>(w);
+            else *reinterpret_cast<float4*>(o + i) = *reinterpret_cast<const float4*>(w);
+        }
+    } else {
+        for (int i = threadIdx.x; i < ff; i += blockDim.x) o[i] = narrow<TO>(value(row[i]));
     }
 }
 
@@ -170,13 +231,13 @@ qk_norm_append_kernel(float* __restrict__ qkv, int ld, const int* __restrict__ r
 
 // f[r][c] = act(gate) * up of rows whose columns come in pairs of 16-wide groups (16 gate, 16 up, ..)
 __global__ void __launch_bounds__(256)
-glu_rows_f32_kernel(const float* __restrict__ gu, int ld, int ff, int act, float* __restrict__ f, int ldf) {
+glu_rows_f32_kernel(const float* __restrict__ gu, int ld, int ff, int act, float limit, float* __restrict__ f, int ldf) {
     dep_wait();
     dep_trigger();
     const float* g = gu + (size_t)blockIdx.x * ld;
     for (int c = blockIdx.y * 256 + threadIdx.x; c < ff; c += gridDim.y * 256) {
         const int b = (c >> 4) * 32 + (c & 15);
-        f[(size_t)blockIdx.x * ldf + c] = glu_act(act, g[b], g[b + 16]);
+        f[(size_t)blockIdx.x * ldf + c] = glu_act(act, g[b], g[b + 16], limit);
     }
 }
 
@@ -210,30 +271,65 @@ extern "C" int cmlb200_embed_rows(const void* d_table, int dtype, const int* d_t
     return CMLB200_OK;
 }
 
+static int launch_residual(float* d_x, const float* d_y, int ldy, const cmlb200_moe* parts, const float* d_w_post, const float* d_w_next, float eps,
+                           int rows, int dim, const int* d_row_idx, void* d_out, int out_dtype, int ldo, int raw, cudaStream_t st) {
+    CMLB_REQUIRE(out_dtype == CMLB200_DT_F32 || out_dtype == CMLB200_DT_BF16, "residual norm: dtype %d", out_dtype);
+    const size_t smem = (size_t)((dim + 3) / 4) * 16;
+    CMLB_REQUIRE(smem <= 200 * 1024, "residual norm: rows of %d elements do not fit shared memory", dim);
+    const bool vec = dim % 4 == 0 && (!d_y || ldy % 4 == 0) && ((!d_w_next && !raw) || ldo % 4 == 0) &&
+                     (((uintptr_t)d_x | (uintptr_t)d_y | (uintptr_t)d_w_post | (uintptr_t)d_w_next | (uintptr_t)d_out) & 15) == 0;
+    // few rows: enough threads that each meets its row once; many rows: small CTAs, several to an SM
+    int threads = 256;
+    if (rows <= 2 * cmlb_num_sms()) while (threads < 1024 && threads * 4 < dim) threads *= 2;
+    static size_t attr[8][kMaxDevices] = {};
+#define RN_LAUNCH(TO, V, P, slot)                                                                                                   \
+    do {                                                                                                                            \
+        auto kern = residual_norm_kernel<TO, V, P>;                                                                                 \
+        CMLB_CUDA(cmlb_ensure_smem(kern, smem, attr[slot]));                                                                        \
+        CMLB_CUDA(launch_chain(kern, dim3(rows), dim3(threads), smem, 1, st, d_x, d_y, ldy, d_w_post, d_w_next, eps, dim, d_row_idx, (TO*)d_out, ldo, raw, \
+                               parts ? parts->top : 0, (const int*)(parts ? parts->pos : nullptr), (const float*)(parts ? parts->weight : nullptr))); \
+    } while (0)
+#define RN_VEC(TO, P, slot) do { if (vec) RN_LAUNCH(TO, true, P, slot); else RN_LAUNCH(TO, false, P, slot + 1); } while (0)
+    if (out_dtype == CMLB200_DT_BF16) { if (parts) RN_VEC(__nv_bfloat16, true, 0); else RN_VEC(__nv_bfloat16, false, 2); }
+    else { if (parts) RN_VEC(float, true, 4); else RN_VEC(float, false, 6); }
+#undef RN_VEC
+#undef RN_LAUNCH
+    return CMLB200_OK;
+}
+
 extern "C" int cmlb200_residual_norm(float* d_x, const float* d_y, int ldy, const float* d_w_post, const float* d_w_next, float eps, int rows,
                                      int dim, const int* d_row_idx, void* d_out, int out_dtype, int ldo, void* stream) {
     CMLB_REQUIRE(d_x && rows > 0 && dim > 0 && (d_y || d_w_next), "cmlb200_residual_norm: bad argument");
     CMLB_REQUIRE(!d_w_next || (d_out && ldo >= dim), "cmlb200_residual_norm: no output for the normed rows");
     CMLB_REQUIRE(!(d_y && d_row_idx) && (!d_y || ldy >= dim), "cmlb200_residual_norm: a row list goes with the norm-only form");
-    CMLB_REQUIRE(out_dtype == CMLB200_DT_F32 || out_dtype == CMLB200_DT_BF16, "cmlb200_residual_norm: dtype %d", out_dtype);
-    const size_t smem = (size_t)((dim + 3) / 4) * 16;
-    CMLB_REQUIRE(smem <= 200 * 1024, "cmlb200_residual_norm: rows of %d elements do not fit shared memory", dim);
-    const bool vec = dim % 4 == 0 && (!d_y || ldy % 4 == 0) && (!d_w_next || ldo % 4 == 0) &&
-                     (((uintptr_t)d_x | (uintptr_t)d_y | (uintptr_t)d_w_post | (uintptr_t)d_w_next | (uintptr_t)d_out) & 15) == 0;
-    // few rows: enough threads that each meets its row once; many rows: small CTAs, several to an SM
+    return launch_residual(d_x, d_y, ldy, nullptr, d_w_post, d_w_next, eps, rows, dim, d_row_idx, d_out, out_dtype, ldo, 0, as_stream(stream));
+}
+
+extern "C" int cmlb200_residual_add(float* d_x, const float* d_y, int ldy, const cmlb200_moe* parts, const float* d_w_post, float eps, int rows, int dim,
+                                    void* d_out, int out_dtype, int ldo, void* stream) {
+    CMLB_REQUIRE(d_x && rows > 0 && dim > 0 && d_out && ldo >= dim && (!d_y || ldy >= dim), "cmlb200_residual_add: bad argument");
+    CMLB_REQUIRE(!parts || (d_y && parts->top > 0 && parts->pos && parts->weight), "cmlb200_residual_add: parts without rows");
+    return launch_residual(d_x, d_y, ldy, parts, d_w_post, nullptr, eps, rows, dim, nullptr, d_out, out_dtype, ldo, 1, as_stream(stream));
+}
+
+extern "C" int cmlb200_poly_norm(const float* d_z, int ld, int rows, int ff, const float* d_coef, float eps, void* d_f, int out_dtype, int ldf, void* stream) {
+    CMLB_REQUIRE(d_z && d_coef && d_f && rows > 0 && ff > 0 && ld >= ff && ldf >= ff, "cmlb200_poly_norm: bad argument");
+    CMLB_REQUIRE(out_dtype == CMLB200_DT_F32 || out_dtype == CMLB200_DT_BF16, "cmlb200_poly_norm: dtype %d", out_dtype);
+    const size_t smem = (size_t)((ff + 3) / 4) * 16;
+    CMLB_REQUIRE(smem <= 200 * 1024, "cmlb200_poly_norm: rows of %d elements do not fit shared memory", ff);
+    const bool vec = ff % 4 == 0 && ld % 4 == 0 && ldf % 4 == 0 && (((uintptr_t)d_z | (uintptr_t)d_f) & 15) == 0;
     int threads = 256;
-    if (rows <= 2 * cmlb_num_sms()) while (threads < 1024 && threads * 4 < dim) threads *= 2;
-    cudaStream_t st = as_stream(stream);
+    if (rows <= 2 * cmlb_num_sms()) while (threads < 1024 && threads * 4 < ff) threads *= 2;
     static size_t attr[4][kMaxDevices] = {};
-#define RN_LAUNCH(TO, V, slot)                                                                                                      \
+#define PN_LAUNCH(TO, V, slot)                                                                                                      \
     do {                                                                                                                            \
-        auto kern = residual_norm_kernel<TO, V>;                                                                                    \
+        auto kern = poly_norm_kernel<TO, V>;                                                                                        \
         CMLB_CUDA(cmlb_ensure_smem(kern, smem, attr[slot]));                                                                        \
-        CMLB_CUDA(launch_chain(kern, dim3(rows), dim3(threads), smem, 1, st, d_x, d_y, ldy, d_w_post, d_w_next, eps, dim, d_row_idx, (TO*)d_out, ldo)); \
+        CMLB_CUDA(launch_chain(kern, dim3(rows), dim3(threads), smem, 1, as_stream(stream), d_z, ld, ff, d_coef, eps, (TO*)d_f, ldf)); \
     } while (0)
-    if (out_dtype == CMLB200_DT_BF16) { if (vec) RN_LAUNCH(__nv_bfloat16, true, 0); else RN_LAUNCH(__nv_bfloat16, false, 1); }
-    else { if (vec) RN_LAUNCH(float, true, 2); else RN_LAUNCH(float, false, 3); }
-#undef RN_LAUNCH
+    if (out_dtype == CMLB200_DT_BF16) { if (vec) PN_LAUNCH(__nv_bfloat16, true, 0); else PN_LAUNCH(__nv_bfloat16, false, 1); }
+    else { if (vec) PN_LAUNCH(float, true, 2); else PN_LAUNCH(float, false, 3); }
+#undef PN_LAUNCH
     return CMLB200_OK;
 }
 
@@ -254,7 +350,13 @@ extern "C" int cmlb200_qk_norm_append(const cmlb200_attn* a, float* d_qkv, int l
 
 extern "C" int cmlb200_glu_rows_f32(const float* d_gu, int ld, int rows, int ff, int act, float* d_f, int ldf, void* stream) {
     CMLB_REQUIRE(d_gu && d_f && rows > 0 && ff > 0 && ldf >= ff && ld >= 2 * ((ff + 15) & ~15), "cmlb200_glu_rows_f32: bad argument");
-    CMLB_CUDA(launch_chain(glu_rows_f32_kernel, dim3(rows, (ff + 1023) / 1024), dim3(256), 0, 1, as_stream(stream), d_gu, ld, ff, act, d_f, ldf));
+    CMLB_CUDA(launch_chain(glu_rows_f32_kernel, dim3(rows, (ff + 1023) / 1024), dim3(256), 0, 1, as_stream(stream), d_gu, ld, ff, act, 0.f, d_f, ldf));
+    return CMLB200_OK;
+}
+
+extern "C" int cmlb200_moe_glu_rows_f32(const float* d_gu, int ld, int rows, int ff, int act, float limit, float* d_f, int ldf, void* stream) {
+    CMLB_REQUIRE(d_gu && d_f && rows > 0 && ff > 0 && ldf >= ff && ld >= 2 * ((ff + 15) & ~15), "cmlb200_moe_glu_rows_f32: bad argument");
+    CMLB_CUDA(launch_chain(glu_rows_f32_kernel, dim3(rows, (ff + 1023) / 1024), dim3(256), 0, 1, as_stream(stream), d_gu, ld, ff, act, limit, d_f, ldf));
     return CMLB200_OK;
 }
 

@@ -1,0 +1,173 @@
+// Experts: the router's choice and the plan that orders a step's (row, expert) pairs by expert, the copy of rows into
+// that order for the tensor-core product, and the product of the 32-bit path. See cmlb200_moe.
+#include "lm_util.cuh"
+
+namespace {
+
+constexpr int ROUTE_WARPS = 8, PLAN_THREADS = 1024;
+
+// One warp, one row: softmax over all experts, then `top` times the largest that is left (the lower index wins a tie).
+__device__ __forceinline__ void route_row(const cmlb200_moe& m, const float* __restrict__ logits, int r, float* z) {
+    const int lane = threadIdx.x & 31;
+    float mx = -INFINITY;
+    for (int e = lane; e < m.experts; e += 32) { const float v = logits[e]; z[e] = v; mx = fmaxf(mx, v); }
+    mx = lane_max(mx);
+    float sum = 0.f;
+    for (int e = lane; e < m.experts; e += 32) sum += expf(z[e] - mx);
+    sum = lane_sum(sum);
+    for (int k = 0; k < m.top; k++) {
+        float best = -INFINITY;
+        int at = 0x7fffffff;
+        for (int e = lane; e < m.experts; e += 32)
+            if (z[e] > best || at == 0x7fffffff) { best = z[e]; at = e; }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            const float v = __shfl_xor_sync(0xffffffffu, best, o);
+            const int i = __shfl_xor_sync(0xffffffffu, at, o);
+            if (v > best || (v == best && i < at)) { best = v; at = i; }
+        }
+        at = min(at, m.experts - 1);
+        __syncwarp();
+        if (lane == (at & 31)) {
+            m.ids[r * m.top + k] = at;
+            m.weight[r * m.top + k] = expf(best - mx) / sum;
+            z[at] = -INFINITY;
+        }
+        __syncwarp();
+    }
+}
+
+__global__ void __launch_bounds__(ROUTE_WARPS * 32)
+route_rows_kernel(const cmlb200_moe m, const float* __restrict__ logits, int ld, int rows) {
+    extern __shared__ float z[];
+    dep_wait();
+    dep_trigger();
+    const int warp = threadIdx.x >> 5, r = blockIdx.x * ROUTE_WARPS + warp;
+    if (r < rows) route_row(m, logits + (size_t)r * ld, r, z + warp * m.experts);
+}
+
+// One CTA. logits given (up to 32 rows): routes the rows first. Then counts, first positions (multiples of `align`), the
+// lists of chosen experts and of row tiles, and a position for every pair.
+__global__ void __launch_bounds__(PLAN_THREADS)
+plan_kernel(const cmlb200_moe m, const float* __restrict__ logits, int ld, int rows, int align) {
+    extern __shared__ float z[];
+    int* count = reinterpret_cast<int*>(z);                             // [experts], then the next free position
+    dep_wait();
+    dep_trigger();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, pairs = rows * m.top;
+    if (logits) {
+        if (warp < rows) route_row(m, logits + (size_t)warp * ld, warp, z + warp * m.experts);
+        __syncthreads();                                                // also orders the choices' global writes for this block
+    }
+    for (int e = threadIdx.x; e < m.experts; e += PLAN_THREADS) count[e] = 0;
+    __syncthreads();
+    for (int p = threadIdx.x; p < pairs; p += PLAN_THREADS) atomicAdd(&count[m.ids[p]], 1);
+    __syncthreads();
+    if (warp == 0) {
+        int pos = 0, act = 0, til = 0;                                  // positions, chosen experts, tiles so far
+        for (int e0 = 0; e0 < m.experts; e0 += 32) {
+            const int e = e0 + lane, c = e < m.experts ? count[e] : 0;
+            int a = (c + align - 1) / align * align, b = c > 0, t = (c + 127) / 128;
+            const int a0 = a, b0 = b, t0 = t;
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) {
+                const int x = __shfl_up_sync(0xffffffffu, a, o), y = __shfl_up_sync(0xffffffffu, b, o), w = __shfl_up_sync(0xffffffffu, t, o);
+                if (lane >= o) { a += x; b += y; t += w; }
+            }
+            if (e < m.experts) {
+                const int first = pos + a - a0;
+                m.start[e] = first;
+                m.count[e] = c;
+                if (b0) m.active[act + b - 1] = e;
+                if (m.tiles)
+                    for (int i = 0; i < t0; i++) reinterpret_cast<int4*>(m.tiles)[til + t - t0 + i] = make_int4(first + i * 128, e, min(128, c - i * 128), 0);
+                count[e] = first;
+            }
+            pos += __shfl_sync(0xffffffffu, a, 31);
+            act += __shfl_sync(0xffffffffu, b, 31);
+            til += __shfl_sync(0xffffffffu, t, 31);
+        }
+        if (lane == 0) { *m.num_active = act; *m.num_tiles = til; }
+    }
+    __syncthreads();
+    for (int p = threadIdx.x; p < pairs; p += PLAN_THREADS) {
+        const int e = m.ids[p], at = atomicAdd(&count[e], 1);
+        m.pos[p] = at;
+        m.src[at] = p / m.top;
+        m.expert[at] = e;
+    }
+}
+
+// xp[pos[pair]] = x[row of the pair], 16 bytes at a time
+__global__ void __launch_bounds__(256)
+gather_rows_kernel(const cmlb200_moe m, const uint4* __restrict__ x, int ldx, int width, uint4* __restrict__ xp, int ldxp) {
+    dep_wait();
+    dep_trigger();
+    const uint4* s = x + (size_t)blockIdx.x * ldx;
+    for (int i = threadIdx.x; i < width; i += 256) {
+        const uint4 v = s[i];
+        for (int k = 0; k < m.top; k++) xp[(size_t)m.pos[blockIdx.x * m.top + k] * ldxp + i] = v;
+    }
+}
+
+// 32-bit product: a warp per output value. grid = (columns / 8, rows * top); blockIdx.y counts pairs.
+__global__ void __launch_bounds__(256)
+moe_linear_f32_kernel(const cmlb200_moe m, const float* __restrict__ W, int ldw, int w_rows, int K, const float* __restrict__ x, int ldx, int gather,
+                      int n_out, float* __restrict__ y, int ldy) {
+    dep_wait();
+    dep_trigger();
+    const int p = m.pos[blockIdx.y], n = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (n >= n_out) return;
+    const float* w = W + ((size_t)m.expert[p] * w_rows + n) * ldw;
+    const float* xr = x + (size_t)(gather ? (int)blockIdx.y / m.top : p) * ldx;
+    float s = 0.f;
+    for (int k = lane; k < K; k += 32) s = fmaf(w[k], xr[k], s);
+    s = lane_sum(s);
+    if (lane == 0) y[(size_t)p * ldy + n] = s;
+}
+
+}  // namespace
+
+extern "C" long cmlb200_moe_positions(int rows, int top, int experts, int align) {
+    const long pairs = (long)rows * top, used = pairs < experts ? pairs : experts;
+    return pairs + used * (align - 1);
+}
+
+extern "C" int cmlb200_moe_route(const cmlb200_moe* m, const float* d_logits, int ld, int rows, int align, void* stream) {
+    CMLB_REQUIRE(m && d_logits && rows > 0 && align > 0 && m->experts > 0 && m->top > 0 && m->top <= m->experts && ld >= m->experts, "cmlb200_moe_route: bad argument");
+    CMLB_REQUIRE(m->ids && m->weight && m->pos && m->src && m->expert && m->start && m->count && m->active && m->num_active && m->num_tiles, "cmlb200_moe_route: a plan without arrays");
+    CMLB_REQUIRE(m->experts <= 1536 && (long)rows * m->top < (1l << 30), "cmlb200_moe_route: %d experts", m->experts);
+    cudaStream_t st = as_stream(stream);
+    static size_t attr[kMaxDevices] = {};
+    const bool fused = rows <= 32;
+    const size_t row = (size_t)m->experts * 4;
+    if (!fused) CMLB_CUDA(launch_chain(route_rows_kernel, dim3((rows + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(ROUTE_WARPS * 32), ROUTE_WARPS * row, 1, st, *m, d_logits, ld, rows));
+    const size_t smem = fused ? (size_t)rows * row : row;
+    CMLB_CUDA(cmlb_ensure_smem(plan_kernel, smem, attr));
+    CMLB_CUDA(launch_chain(plan_kernel, dim3(1), dim3(PLAN_THREADS), smem, 1, st, *m, fused ? d_logits : (const float*)nullptr, ld, rows, align));
+    return CMLB200_OK;
+}
+
+extern "C" int cmlb200_moe_gather(const cmlb200_moe* m, const uint16_t* d_x, int ldx, int rows, int width, uint16_t* d_xp, int ldxp, void* stream) {
+    CMLB_REQUIRE(m && d_x && d_xp && rows > 0 && width > 0, "cmlb200_moe_gather: bad argument");
+    const int w8 = (width + 7) / 8;
+    CMLB_REQUIRE(ldx % 8 == 0 && ldxp % 8 == 0 && ldx >= w8 * 8 && ldxp >= w8 * 8 && (((uintptr_t)d_x | (uintptr_t)d_xp) & 15) == 0, "cmlb200_moe_gather: strides %d / %d", ldx, ldxp);
+    CMLB_CUDA(launch_chain(gather_rows_kernel, dim3(rows), dim3(256), 0, 1, as_stream(stream), *m, (const uint4*)d_x, ldx / 8, w8, (uint4*)d_xp, ldxp / 8));
+    return CMLB200_OK;
+}
+
+extern "C" int cmlb200_moe_linear_f32(const cmlb200_moe* m, const cmlb200_dense* W, const float* d_x, int ldx, int gather, int rows, int n_out, float* d_y,
+                                      int ldy, void* stream) {
+    CMLB_REQUIRE(m && W && W->w && d_x && d_y && rows > 0, "cmlb200_moe_linear_f32: bad argument");
+    CMLB_REQUIRE(W->dtype == CMLB200_DT_F32 && m->experts > 0 && W->rows % m->experts == 0 && n_out > 0 && n_out <= W->rows / m->experts && W->ld >= W->cols &&
+                 ldx >= W->cols && ldy >= n_out, "cmlb200_moe_linear_f32: weight [%d, %d], strides %d / %d", W->rows, W->cols, ldx, ldy);
+    const int pairs = rows * m->top;
+    for (int at = 0; at < pairs; at += 65535 / m->top * m->top) {       // whole rows per launch
+        const int n = pairs - at < 65535 / m->top * m->top ? pairs - at : 65535 / m->top * m->top;
+        cmlb200_moe part = *m;
+        part.pos = m->pos + at;
+        CMLB_CUDA(launch_chain(moe_linear_f32_kernel, dim3((n_out + 7) / 8, n), dim3(256), 0, 1, as_stream(stream), part, (const float*)W->w, W->ld,
+                               W->rows / m->experts, W->cols, gather ? d_x + (size_t)(at / m->top) * ldx : d_x, ldx, gather, n_out, d_y, ldy));
+    }
+    return CMLB200_OK;
+}

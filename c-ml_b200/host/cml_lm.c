@@ -45,6 +45,7 @@ struct CMLLanguageModel {
     StepGraph graphs[MAX_GRAPHS];
     unsigned clock;
     unsigned char* in_step;        /* per sequence: already in the entries being checked */
+    CMLLMPortion* portions;        /* of the step being run, one per sequence at most */
 };
 
 /* ---- registry ------------------------------------------------------------------------------------ */
@@ -87,7 +88,7 @@ static int make_buffers(CMLLanguageModel* lm) {
     DEV(cmlb200_malloc((void**)&lm->d_picked, HEAD_ROWS * sizeof(int)));
     DEV(cmlb200_host_alloc_pinned((void**)&lm->h_picked, HEAD_ROWS * sizeof(int)));
     DEV(cmlb200_malloc((void**)&lm->d_step, sizeof(int)));
-    return lm->cls->make_pools(lm->model, blocks, BLOCK);
+    return lm->cls->make_pools(lm->model, blocks, BLOCK, lm->opt.max_sequences, lm->table_ld);
 }
 
 CMLLanguageModel* cml_lm_load(const char* path, const CMLLMOptions* options) {
@@ -118,10 +119,11 @@ CMLLanguageModel* cml_lm_load(const char* path, const CMLLMOptions* options) {
         lm->cls = cls;
         lm->opt = o;
         lm->in_step = (unsigned char*)calloc((size_t)o.max_sequences, 1);
+        lm->portions = (CMLLMPortion*)calloc((size_t)o.max_sequences, sizeof *lm->portions);
         lm->model = cls->load(path, config, &o, &lm->info);
     }
     cml_json_free(config);
-    if (!lm || !lm->in_step || !lm->model || (cls->make_pools && make_buffers(lm))) {
+    if (!lm || !lm->in_step || !lm->portions || !lm->model || (cls->make_pools && make_buffers(lm))) {
         LOG_ERROR("%s: %s could not be loaded", who, path);
         cml_lm_free(lm);
         return NULL;
@@ -141,6 +143,7 @@ void cml_lm_free(CMLLanguageModel* lm) {
     cmlb200_host_free_pinned(lm->h_picked);
     if (lm->stream) cmlb200_stream_destroy(lm->stream);
     free(lm->in_step);
+    free(lm->portions);
     free(lm);
 }
 
@@ -238,33 +241,46 @@ static int round_keys(int keys) {
 static int upload_rows(CMLLanguageModel* lm, const CMLLMEntry* entries, int n, int rows, CMLLMBatch* b, const int** d_want) {
     const int stride = rows <= SMALL_ROWS ? SMALL_ROWS : (lm->opt.max_step_rows + 3) & ~3;
     int *tok = lm->h_meta, *pos = tok + stride, *slot = pos + stride, *want = slot + stride, *tiles = want + stride;
-    int one = 0, one_keys = 0, at = 0, w = 0, t = 0;
-    for (int i = 0; i < n; i++) one += entries[i].num_tokens == 1;
-    int next_one = 0;
-    at = one;
+    int one = 0, one_keys = 0, w = 0, t = 0, short_rows = 0, short_tiles = 0, portions = 0;
+    for (int i = 0; i < n; i++) {
+        const int k = entries[i].num_tokens;
+        one += k == 1;
+        if (k > 1 && k <= TILE_ROWS) { short_rows += k; short_tiles++; }
+    }
+    /* next row and, for portions, next tile of each of the three kinds */
+    int at_one = 0, at_short = one, at_long = one + short_rows, tile_short = 0;
+    t = short_tiles;
     for (int i = 0; i < n; i++) {
         const CMLLMEntry* e = &entries[i];
-        const int first = lm->cache->sequences[e->seq].seq_len - e->num_tokens, r0 = e->num_tokens == 1 ? next_one++ : at;
-        for (int k = 0; k < e->num_tokens; k++) {
+        const int len = e->num_tokens, first = lm->cache->sequences[e->seq].seq_len - len;
+        int* at = len == 1 ? &at_one : (len <= TILE_ROWS ? &at_short : &at_long);
+        int* tile = len <= TILE_ROWS ? &tile_short : &t;
+        const int r0 = *at;
+        *at += len;
+        for (int k = 0; k < len; k++) {
             tok[r0 + k] = e->tokens[k];
             pos[r0 + k] = first + k;
             slot[r0 + k] = e->seq;
         }
         for (int k = 0; k < e->num_want; k++) want[w++] = r0 + e->want[k];
-        if (e->num_tokens == 1) { if (first > one_keys) one_keys = first; continue; }
-        for (int k = 0; k < e->num_tokens; k += TILE_ROWS, t++) {
-            tiles[4 * t] = r0 + k;
-            tiles[4 * t + 1] = e->num_tokens - k < TILE_ROWS ? e->num_tokens - k : TILE_ROWS;
-            tiles[4 * t + 2] = e->seq;
-            tiles[4 * t + 3] = first + k;
+        if (len == 1) { if (first > one_keys) one_keys = first; continue; }
+        if (len > TILE_ROWS) { CMLLMPortion p = {r0, len, e->seq, first, t}; lm->portions[portions++] = p; }
+        for (int k = 0; k < len; k += TILE_ROWS, ++*tile) {
+            tiles[4 * *tile] = r0 + k;
+            tiles[4 * *tile + 1] = len - k < TILE_ROWS ? len - k : TILE_ROWS;
+            tiles[4 * *tile + 2] = e->seq;
+            tiles[4 * *tile + 3] = first + k;
         }
-        at += e->num_tokens;
     }
     DEV(cmlb200_memcpy_h2d(lm->d_meta, lm->h_meta, (4 * (size_t)stride + 4 * (size_t)t) * sizeof(int), lm->stream));
     memset(b, 0, sizeof *b);
     b->rows = rows;
     b->one_rows = one;
     b->tiles = t;
+    b->short_rows = short_rows;
+    b->short_tiles = short_tiles;
+    b->portions = lm->portions;
+    b->num_portions = portions;
     b->max_keys = round_keys(one_keys);
     b->d_tokens = lm->d_meta;
     b->d_pos = lm->d_meta + stride;

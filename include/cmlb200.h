@@ -408,6 +408,7 @@ int cmlb200_ipc_close(void* d_ptr);
 #define CMLB200_DT_F16 2
 #define CMLB200_ACT_SILU 0
 #define CMLB200_ACT_GELU_TANH 1
+#define CMLB200_ACT_CLAMPED 2     /* g = min(gate, limit), u = clamp(up, -limit, limit): g sigmoid(1.702 g) (u + 1) */
 
 /* A dense [rows, cols] weight (rows = out features), row stride `ld` elements. Allocated with rows rounded
  * up to 16 and ld a multiple of 64, the padding zero. dtype CMLB200_DT_F32 or CMLB200_DT_BF16. */
@@ -435,7 +436,44 @@ typedef struct cmlb200_attn {
     int block_size;             /* a power of two >= 16 */
     const int* block_table;     /* device, [slots][table_ld] block ids */
     int table_ld;
+    int gate_wide;              /* 1: heads * vdim gate logits, one for every element of the output (_tiles only) */
 } cmlb200_attn;
+
+/* Latent attention over a paged cache of one vector per token: a normed latent of `rank` values and a rotated key
+ * part of rot_dim values that all heads share. Per head the key is [Wuk c | rotated part], the value Wuv c.
+ * Projection rows hold heads * (dim + rot_dim) query columns (per head: unrotated, rotated), fp32. */
+typedef struct cmlb200_latent {
+    int heads, dim, rot_dim, vdim, rank;
+    int ld;                     /* elements per token in the pool: rank + rot_dim rounded up to 16, zeros behind them */
+    int ld_rank;                /* per-head stride of the weighted latents: rank rounded up to 64 */
+    float scale;
+    int window;                 /* as in cmlb200_attn */
+    const float* c_norm;        /* device, RMS norm weights of the latent */
+    float eps;
+    const float* freq;          /* device, rot_dim / 2: entry i turns with entry i + rot_dim / 2 by pos * freq[i] */
+    float rot_mul;              /* factor on sine and cosine */
+    int kv_col;                 /* column of the rank + rot_dim latent projections; -1: another layer fills the cache */
+    int gate_col;               /* column of heads * vdim gate logits; -1: none */
+    int cache_dtype;            /* CMLB200_DT_F32 or CMLB200_DT_F16 */
+    void* pool;                 /* [blocks][block_size][ld] */
+    int block_size;             /* a power of two >= 16 */
+    const int* block_table;
+    int table_ld;
+} cmlb200_latent;
+
+/* Where a step's (row, expert) pairs go: `top` pairs per row, ordered by expert, each expert's first position a
+ * multiple of the alignment. All arrays live on the device; cmlb200_moe_positions gives their extent. */
+typedef struct cmlb200_moe {
+    int experts, top;
+    int* ids;                   /* [rows * top] chosen experts */
+    float* weight;              /* [rows * top] their weights */
+    int* pos;                   /* [rows * top] position of a pair */
+    int* src;                   /* [positions] row of a position */
+    int* expert;                /* [positions] expert of a position */
+    int *start, *count;         /* [experts] */
+    int *active, *num_active;   /* [experts] experts that were chosen at all */
+    int *tiles, *num_tiles;     /* {first position, expert, rows, 0} per 128 positions of an expert */
+} cmlb200_moe;
 
 /* x[r] = table[token[r]] (+ a sinusoidal vector of position pos[r]: sin, cos of pos * freq[i] in entries
  * 2i, 2i + 1; d_freq NULL: none). fp32 rows of `width`. */
@@ -468,6 +506,55 @@ int cmlb200_gemm_dense_glu(const cmlb200_dense* W, const uint16_t* d_x, int ldx,
 int cmlb200_gemm_dense_status(int* status, int reset);
 int cmlb200_linear_dense_f32(const cmlb200_dense* W, const float* d_x, int ldx, int M, float* d_y, int ldy, void* stream);
 int cmlb200_glu_rows_f32(const float* d_gu, int ld, int rows, int ff, int act, float* d_f, int ldf, void* stream);
+/* x += rms_norm(y) * w_post, then out = x. parts (optional): y holds one row per pair, and row r of the norm's input is
+ * the weighted sum of the rows of its pairs. y NULL: out = x alone. */
+int cmlb200_residual_add(float* d_x, const float* d_y, int ldy, const cmlb200_moe* parts, const float* d_w_post, float eps, int rows, int dim,
+                         void* d_out, int out_dtype, int ldo, void* stream);
+/* f = a N(z) + b N(z^2) + c N(z^3) + e per element, N dividing a row by its root mean square; d_coef = {a, b, c, e}. */
+int cmlb200_poly_norm(const float* d_z, int ld, int rows, int ff, const float* d_coef, float eps, void* d_f, int out_dtype, int ldf, void* stream);
+
+/* Latent attention. _append: rotates the query columns in place and fills the cache (any rows). _query: the same for
+ * rows whose attention runs over the latents themselves, into fp16 rows [heads][ld] = [Wuk^T q | rotated q] times
+ * scale log2 e. Wuk^T is stored per head as [rank rounded up to 16][dim rounded up to 64]. */
+int cmlb200_latent_append(const cmlb200_latent* a, float* d_proj, int ld, const int* d_row_pos, const int* d_row_slot, int rows, void* stream);
+int cmlb200_latent_query(const cmlb200_latent* a, const uint16_t* d_wukt, const float* d_proj, int ld, const int* d_row_pos, const int* d_row_slot,
+                         int rows, uint16_t* d_q_f16, void* stream);
+/* Weighted latents bf16 [rows][heads][ld_rank] of such query rows. d_tiles NULL: row r is one token (position and slot
+ * from the row arrays); otherwise tiles as in cmlb200_attention_tiles, and `rows` is the row that d_q_f16 begins with. */
+int cmlb200_attention_latent(const cmlb200_latent* a, const uint16_t* d_q_f16, const int* d_row_pos, const int* d_row_slot, int rows, int max_keys,
+                             const int* d_tiles, int tiles, uint16_t* d_o_bf16, void* stream);
+/* out[row][head * vdim + v] = Wuv o, times the sigmoid of the gate. Wuv per head: [vdim rounded up to 16][ld_rank]. */
+int cmlb200_latent_output(const cmlb200_latent* a, const uint16_t* d_wuv, const uint16_t* d_o_bf16, const float* d_proj, int ld, int rows,
+                          uint16_t* d_out_bf16, int out_ld, void* stream);
+/* Long portions: the latents keys[i] = {slot, first key, keys, first scratch row} of up to 16 sequences become per-head
+ * keys and values. _gather: bf16 latents, the shared key part in every head's key row, and the scratch's block table
+ * (first key and first scratch row are multiples of the block size). _expand: both products on tcgen05, fp16; W holds the
+ * heads' Wuk rows and behind them their Wuv rows, each head's padded to 16. */
+int cmlb200_latent_gather(const cmlb200_latent* a, const int (*keys)[4], int n, uint16_t* d_c_bf16, const cmlb200_attn* scratch, void* stream);
+int cmlb200_latent_expand(const cmlb200_latent* a, const cmlb200_dense* W, const uint16_t* d_c_bf16, int rows, const cmlb200_attn* scratch, void* stream);
+/* 32-bit forms: _query_f32 writes [heads][rank + rot_dim] rows and fills an fp32 cache; cmlb200_attention_rows_f32 runs
+ * over it as one key/value head; _output_f32 as above. Weights [heads][rank][dim] and [heads][vdim][rank]. */
+int cmlb200_latent_query_f32(const cmlb200_latent* a, const float* d_wukt, const float* d_proj, int ld, const int* d_row_pos, const int* d_row_slot,
+                             int rows, float* d_q, void* stream);
+int cmlb200_latent_output_f32(const cmlb200_latent* a, const float* d_wuv, const float* d_o, const float* d_proj, int ld, int rows, float* d_out,
+                              int out_ld, void* stream);
+
+/* Experts. _route: softmax over all experts of fp32 router logits, the `top` largest scores (ties: lower index), and
+ * the plan. The products take a weight whose experts are stacked, each `rows / experts` rows (a multiple of 16);
+ * gather: x has one row per step row, otherwise one per position. y has one row per position. _gemv: up to 32 rows. */
+long cmlb200_moe_positions(int rows, int top, int experts, int align);
+int cmlb200_moe_route(const cmlb200_moe* m, const float* d_logits, int ld, int rows, int align, void* stream);
+int cmlb200_moe_gather(const cmlb200_moe* m, const uint16_t* d_x, int ldx, int rows, int width, uint16_t* d_xp, int ldxp, void* stream);
+int cmlb200_moe_gemv(const cmlb200_moe* m, const cmlb200_dense* W, const uint16_t* d_x, int ldx, int gather, int rows, int n_out, float* d_y, int ldy,
+                     void* stream);
+int cmlb200_moe_gemv_glu(const cmlb200_moe* m, const cmlb200_dense* W, const uint16_t* d_x, int ldx, int gather, int rows, int ff, int act, float limit,
+                         uint16_t* d_f, int ldf, void* stream);
+int cmlb200_moe_gemm(const cmlb200_moe* m, const cmlb200_dense* W, const uint16_t* d_x, int ldx, int rows, int n_out, float* d_y, int ldy, void* stream);
+int cmlb200_moe_gemm_glu(const cmlb200_moe* m, const cmlb200_dense* W, const uint16_t* d_x, int ldx, int rows, int ff, int act, float limit, uint16_t* d_f,
+                         int ldf, void* stream);
+int cmlb200_moe_linear_f32(const cmlb200_moe* m, const cmlb200_dense* W, const float* d_x, int ldx, int gather, int rows, int n_out, float* d_y, int ldy,
+                           void* stream);
+int cmlb200_moe_glu_rows_f32(const float* d_gu, int ld, int rows, int ff, int act, float limit, float* d_f, int ldf, void* stream);
 /* tokens[i] = picked[i], pos[i] += 1, hist[step * rows + i] = picked[i], step += 1 */
 int cmlb200_advance_tokens(const int* d_picked, int rows, int* d_tokens, int* d_pos, int* d_hist, int* d_step, void* stream);
 
