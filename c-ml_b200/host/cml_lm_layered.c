@@ -31,7 +31,7 @@
 #define SKINNY_ROWS 32
 #define MAX_LAYERS 4096
 #define EXPERT_ROWS 128            /* row tile of the experts' tensor-core product */
-#define EXPAND_KEYS 65536          /* keys the scratch cache of long portions holds at most */
+#define EXPAND_KEYS 65536          /* keys the scratch cache of long portions holds at most (CMLB200_EXPAND_KEYS: another number) */
 #define DEV(call) do { if (CML_DEV_FAIL((call), __func__)) return -1; } while (0)
 
 typedef struct MixerKind {
@@ -595,7 +595,10 @@ static int make_expansion(Layered* m, int blocks, int block_size, int slots, int
     if (!k || m->f32) return 0;
     m->slots = slots;
     m->table_ld = table_ld;
-    m->expand_keys = (long)blocks * block_size < EXPAND_KEYS ? blocks * block_size : EXPAND_KEYS;
+    const char* env = getenv("CMLB200_EXPAND_KEYS");
+    int keys = env && atoi(env) > 0 && atoi(env) < (1 << 28) ? round_up(atoi(env), block_size) : EXPAND_KEYS;
+    if ((long)blocks * block_size < keys) keys = blocks * block_size;
+    m->expand_keys = keys;
     const size_t n = (size_t)m->expand_keys;
     return zeroed(&m->expand_k, n * (size_t)k * 2) || zeroed(&m->expand_v, n * (size_t)v * 2) || zeroed(&m->expand_c, n * (size_t)c * 2) ||
            zeroed((void**)&m->expand_table, (size_t)slots * (size_t)table_ld * sizeof(int)) ? -1 : 0;

@@ -246,11 +246,56 @@ def layered_config(vocab, width, layers, eps=1e-5):
     return {"architecture": "Rarolorn", "vocab": vocab, "width": width, "norm": {"eps": eps}, "layers": layers}
 
 
+def latent_layer(heads, dim, rot_dim, vdim, rank, mlp, window=None, gated=False, base=10000.0, scaling=None, scale=None, kv_from=None):
+    """mlp: a dense layer's size, (experts, top, size, limit), or None. scaling: (factor, original, fast, slow)."""
+    rot = {"base": base, "dims": rot_dim}
+    if scaling:
+        rot["scaling"] = dict(zip(("factor", "original", "fast", "slow"), scaling))
+    mixer = {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": rank, "rot": rot, "scale": scale or (dim + rot_dim) ** -0.5}
+    if window:
+        mixer["mask"] = {"size": window}
+    if kv_from is not None:
+        mixer["kv_from"] = kv_from
+    if isinstance(mlp, tuple):
+        mlp = {"kind": "moe", "router": {"experts": mlp[0], "top": mlp[1]}, "expert": {"ff": mlp[2], "limit": mlp[3]}}
+    elif mlp:
+        mlp = {"kind": "dense", "ff": mlp}
+    return {"type": "latent_attention_2" if gated else "latent_attention", "mixer": mixer, "mlp": mlp or None}
+
+
+def latent_config(vocab, width, layers, eps=1e-5):
+    return {"architecture": "Situlorn", "vocab": vocab, "width": width, "norm": {"eps": eps}, "layers": layers}
+
+
+def latent_layer_shapes(layer, W, p):
+    m, f = layer["mixer"], layer["mlp"]
+    H, R = m["heads"], m["kv_rank"]
+    out = {p + "norm1": (W,), p + "mix.q": (H * (m["dim"] + m["rot_dim"]), W), p + "mix.uk": (H * m["dim"], R), p + "mix.uv": (H * m["vdim"], R),
+           p + "mix.o": (W, H * m["vdim"])}
+    if m.get("kv_from") is None:
+        out.update({p + "mix.dkv": (R + m["rot_dim"], W), p + "mix.dkv.norm": (R,)})
+    if layer["type"] == "latent_attention_2":
+        out[p + "mix.g"] = (H * m["vdim"], W)
+    if f:
+        out[p + "norm2"] = (W,)
+        if f["kind"] == "dense":
+            out.update({p + "mlp.up": (f["ff"], W), p + "mlp.down": (W, f["ff"]), p + "mlp.act": (4,)})
+        else:
+            n = f["expert"]["ff"]
+            out[p + "mlp.router"] = (f["router"]["experts"], W)
+            for e in range(f["router"]["experts"]):
+                out.update({p + f"mlp.e{e}.gate": (n, W), p + f"mlp.e{e}.up": (n, W), p + f"mlp.e{e}.down": (W, n)})
+    return out
+
+
 def layered_shapes(cfg):
     """Tensor name -> shape of every tensor a configuration asks for."""
     W, out = cfg["width"], {"embed": (cfg["vocab"], cfg["width"])}
     for i, layer in enumerate(cfg["layers"]):
         if layer.get("weights_of") is not None:
+            continue
+        if layer["type"].startswith("latent"):
+            out.update(latent_layer_shapes(layer, W, f"l{i}."))
             continue
         m, p = layer["mixer"], f"l{i}."
         q, k, v = m["heads"] * m["dim"], m["kv_heads"] * m["dim"], m["kv_heads"] * m["vdim"]
@@ -268,14 +313,18 @@ def layered_weights(rng, cfg):
     w = {}
     for name, shape in layered_shapes(cfg).items():
         a = rng.standard_normal(shape, dtype=np.float32)
+        if name.endswith("mlp.act"):
+            w[name] = bf16_round(0.6 * a)[1]
+            continue
         w[name] = bf16_round(1.0 + 0.2 * a if len(shape) == 1 else (a if name == "embed" else a / np.sqrt(shape[1])))[1]
     return w
 
 
 def write_layered(folder, cfg, weights, alias_layers=False):
     """Writes config.json and model.safetensors (bf16). `weights`: name -> fp32 array, or a function (name, shape)
-    giving one. alias_layers: every layer's tensors point at the bytes of the first layer with that tensor and shape."""
+    giving one. alias_layers: every layer's tensors (and every expert's) point at the bytes of the first one with that tensor and shape."""
     import json
+    import re
     from pathlib import Path
     folder = Path(folder)
     folder.mkdir(parents=True, exist_ok=True)
@@ -283,7 +332,7 @@ def write_layered(folder, cfg, weights, alias_layers=False):
     header, stored, placed, off = {}, [], {}, 0
     for name, shape in layered_shapes(cfg).items():
         n = 2 * int(np.prod(shape))
-        key = (name.split(".", 1)[1] if name[0] == "l" and name[1].isdigit() else name, shape)
+        key = (re.sub(r"\.e\d+\.", ".e.", name.split(".", 1)[1]) if name[0] == "l" and name[1].isdigit() else name, shape)
         at = placed.get(key) if alias_layers else None
         if at is None:
             at = placed[key] = off

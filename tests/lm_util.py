@@ -1,12 +1,13 @@
 """Small layered models for the tests, and running them on the device and in the plain restatement."""
 import numpy as np
 
+import latent_oracle
 import lm_oracle
 
 
 def variants(synth):
     """name -> configuration. Sizes are chosen so that no two of them coincide by accident."""
-    L = synth.layered_layer
+    L, A = synth.layered_layer, synth.latent_layer
     return {
         # grouped heads, two windows, a layer without feed-forward, shared weights with another layer between
         "mixed": synth.layered_config(211, 144, [L(6, 3, 24, 40, 19, 200, coef=0.4, every=7), L(4, 1, 32, 16, 70, None, coef=0.1, every=33),
@@ -17,14 +18,47 @@ def variants(synth):
         # many query heads on one key/value head, wide heads, a window longer than the prompts
         "wide": synth.layered_config(130, 192, [L(20, 2, 72, 136, 400, 96, coef=0.25, every=100), L(12, 1, 136, 72, 65, 320, weights_of=None)]),
         # a temperature that does nothing and one that does, value size equal to the key size
+        # latents: full and windowed layers, gates, frequency scaling, caches read by later layers with other head counts (one of
+        # them two layers on), experts with 2 of 5, all and one chosen, a layer without feed-forward
+        "latent": synth.latent_config(211, 144, [A(5, 24, 8, 40, 56, 200), A(3, 40, 24, 16, 72, (5, 2, 40, 0.8), 19, True, 3e4, (4.0, 64, 8.0, 1.0)),
+                                                 A(7, 16, 8, 8, 56, None, kv_from=0), A(2, 24, 16, 24, 40, (3, 3, 33, 1.1), 70, True, 500.0),
+                                                 A(4, 32, 8, 24, 56, (4, 1, 72, 2.0), kv_from=0, scale=0.3)], eps=1e-3),
+        # odd sizes everywhere, a window of one token, every layer with a window, one pair of rotated dimensions
+        "latent_odd": synth.latent_config(97, 75, [A(3, 13, 6, 7, 21, 51, 33), A(1, 5, 2, 9, 17, (7, 1, 17, 0.5), 1, True, 100.0),
+                                                   A(5, 11, 6, 3, 21, 51, 50, kv_from=0), A(3, 3, 10, 21, 33, (2, 1, 45, 3.0), 23, True, 1e3, (1.0, 32, 4.0, 0.5))],
+                                          eps=2e-2),
+        # many heads, wide latents
+        "latent_wide": synth.latent_config(130, 192, [A(20, 72, 64, 136, 300, 320, base=1e6), A(12, 104, 32, 72, 200, (40, 3, 48, 1.0), 90, True, 1e4, (8.0, 40, 16.0, 2.0))]),
+        # sizes with tiles of their own, more than 64 (token, head) pairs per token
+        "latent_full": synth.latent_config(64, 128, [A(4, 128, 64, 128, 512, 96, base=1e5), A(70, 8, 8, 8, 128, (9, 4, 24, 1.5), 40, True)]),
         "plain": synth.layered_config(64, 64, [L(2, 1, 32, 32, 16, 64, coef=0.0, every=1), L(2, 2, 32, 32, 17, 64, coef=1.0, every=1)], eps=1e-6),
     }
+
+
+def steady_routes(synth, rng, cfg, w):
+    """Makes the experts' choice independent of rounding: the routers read only the last columns of the residual, which
+    hold well separated levels in an order of each token's own and which no sublayer adds to."""
+    moe = [i for i, l in enumerate(cfg["layers"]) if (l["mlp"] or {}).get("kind") == "moe"]
+    if not moe:
+        return
+    n = max(cfg["layers"][i]["mlp"]["router"]["experts"] for i in moe)
+    level = (np.arange(n) - n / 2) * min(0.5, 4.0 / n)
+    w["embed"][:, -n:] = synth.bf16_round(np.stack([rng.permutation(level) for _ in range(cfg["vocab"])]))[1]
+    for name in w:
+        if name.endswith((".norm1", ".norm2")):
+            w[name][-n:] = 0.0
+            w[name] *= 0.5                             # rounding errors then grow little from layer to layer
+    for i in moe:
+        r = w[f"l{i}.mlp.router"]
+        r[:] = 0.0
+        r[np.arange(len(r)), cfg["width"] - n + rng.permutation(n)[:len(r)]] = 1.0
 
 
 def build(synth, tmp_path, name, seed=0):
     cfg = variants(synth)[name]
     rng = np.random.default_rng(seed + sum(map(ord, name)))
     w = synth.layered_weights(rng, cfg)
+    steady_routes(synth, rng, cfg, w)
     folder = tmp_path / f"{name}_{seed}"
     synth.write_layered(folder, cfg, w)
     return cfg, w, folder
@@ -41,8 +75,13 @@ def error(got, want):
 TOL = {6: 0.02, 0: 2e-5}            # by dtype of the device model: bfloat16, float32
 
 
+def model(cfg, w):
+    """The plain restatement of a configuration's design."""
+    return (latent_oracle if cfg["architecture"] == "Situlorn" else lm_oracle).Model(cfg, w)
+
+
 def reference(cfg, w, tokens):
-    return lm_oracle.Model(cfg, w).forward(tokens)
+    return model(cfg, w).forward(tokens)
 
 
 def cut(n, sizes):

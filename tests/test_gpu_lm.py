@@ -8,13 +8,13 @@ from pathlib import Path
 import numpy as np
 import pytest
 
-import lm_oracle as lo
 import lm_util
 from lm_util import TOL, cut, error
 
 pytestmark = pytest.mark.gpu
 ROOT = Path(__file__).resolve().parents[1]
-NAMES = ["mixed", "odd", "wide", "plain"]
+LATENT = ["latent", "latent_odd", "latent_wide", "latent_full"]
+NAMES = ["mixed", "odd", "wide", "plain"] + LATENT
 DTYPES = [6, 0]                      # bfloat16, float32
 
 
@@ -72,7 +72,7 @@ def test_first_tokens(synth, tmp_path, load, name, dtype):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("name", ["mixed", "odd"])
+@pytest.mark.parametrize("name", ["mixed", "odd", "latent", "latent_odd", "latent_wide"])
 def test_unequal_requests_in_one_batch_with_blocks_used_again(pkg, synth, tmp_path, load, name, dtype):
     """Random schedules over a pool that is too small for all requests together: requests come and go, pause,
     take portions beside single tokens, and sit on blocks and slots that others have used."""
@@ -109,8 +109,9 @@ def test_unequal_requests_in_one_batch_with_blocks_used_again(pkg, synth, tmp_pa
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-def test_batch_does_not_change_a_request(synth, tmp_path, load, dtype):
-    cfg, w, folder = lm_util.build(synth, tmp_path, "wide")
+@pytest.mark.parametrize("name", ["wide", "latent", "latent_wide"])
+def test_batch_does_not_change_a_request(synth, tmp_path, load, name, dtype):
+    cfg, w, folder = lm_util.build(synth, tmp_path, name)
     m = load(folder, dtype, max_sequences=8)
     t = [prompt(cfg, 60, seed=i) for i in range(8)]
     alone = []
@@ -128,10 +129,11 @@ def test_batch_does_not_change_a_request(synth, tmp_path, load, dtype):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-def test_long_decoding(pkg, synth, tmp_path, load, dtype):
+@pytest.mark.parametrize("name", ["mixed", "latent_odd"])
+def test_long_decoding(pkg, synth, tmp_path, load, name, dtype):
     """Hundreds of decoded tokens, over many blocks; windows let blocks go on the way, so the sequence outgrows what
     the pool could hold of it at once."""
-    cfg, w, folder = lm_util.build(synth, tmp_path, "mixed")
+    cfg, w, folder = lm_util.build(synth, tmp_path, name)
     t = prompt(cfg, 420)
     m = load(folder, dtype, max_tokens=128, max_sequences=2)
     s = m.open()
@@ -163,7 +165,7 @@ def test_shared_weights_and_a_missing_feed_forward(synth, tmp_path, load, dtype)
 # ---- greedy decoding, scheduler, generation ----------------------------------------------------------------
 def greedy_reference(cfg, w, tokens, steps):
     """(ids, margins): the restatement's own greedy continuation and the gap between its best two logits at each step."""
-    m = lo.Model(cfg, w)
+    m = lm_util.model(cfg, w)
     st = m.new_state()
     lg, out, gap = m.forward(tokens, st)[-1], [], []
     for _ in range(steps):
@@ -222,8 +224,9 @@ def serve(pkg, m, prompts, lengths, batch, gen=None):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-def test_scheduler_serves_more_requests_than_fit(pkg, synth, tmp_path, load, dtype):
-    cfg, w, folder = lm_util.build(synth, tmp_path, "wide")
+@pytest.mark.parametrize("name", ["wide", "latent"])
+def test_scheduler_serves_more_requests_than_fit(pkg, synth, tmp_path, load, name, dtype):
+    cfg, w, folder = lm_util.build(synth, tmp_path, name)
     m = load(folder, dtype, max_tokens=256, max_sequences=3, max_step_rows=48)       # prompts are cut, requests wait
     lens, new = [70, 3, 120, 33, 1, 64, 90], [9, 30, 12, 1, 25, 20, 7]
     prompts = [prompt(cfg, n, seed=n) for n in lens]
@@ -238,8 +241,9 @@ def test_scheduler_serves_more_requests_than_fit(pkg, synth, tmp_path, load, dty
     assert [len(g) for g in got] == [4, 0, 0, 5] and status[1] == status[2] == 4
 
 
-def test_generation_and_sampling(pkg, synth, tmp_path, load):
-    cfg, w, folder = lm_util.build(synth, tmp_path, "plain")
+@pytest.mark.parametrize("name", ["plain", "latent"])
+def test_generation_and_sampling(pkg, synth, tmp_path, load, name):
+    cfg, w, folder = lm_util.build(synth, tmp_path, name)
     m, lib = load(folder, 0), pkg.lib
     p = np.ascontiguousarray(prompt(cfg, 21), np.int32)
     want, gap = greedy_reference(cfg, w, p, 12)
@@ -284,8 +288,9 @@ def test_step_refusals_change_nothing(pkg, synth, tmp_path, load):
     assert error(np.concatenate(parts), lm_util.reference(cfg, w, t)) < TOL[0]
 
 
-def test_wanted_places_only_and_many_of_them(synth, tmp_path, load):
-    cfg, w, folder = lm_util.build(synth, tmp_path, "odd")
+@pytest.mark.parametrize("name", ["odd", "latent_odd"])
+def test_wanted_places_only_and_many_of_them(synth, tmp_path, load, name):
+    cfg, w, folder = lm_util.build(synth, tmp_path, name)
     m = load(folder, 6, max_tokens=1024)
     t = prompt(cfg, 600)
     want = lm_util.reference(cfg, w, t)
@@ -327,8 +332,9 @@ def test_llama_behind_the_same_interface(pkg, tmp_path, load):
     assert [len(g) for g in got] == [5, 8] and got[0][0] == int(want[6].argmax())
 
 
-def test_trace_run_replays(synth, tmp_path, torch_dev):
-    cfg, w, folder = lm_util.build(synth, tmp_path, "mixed")
+@pytest.mark.parametrize("name", ["mixed", "latent"])
+def test_trace_run_replays(synth, tmp_path, torch_dev, name):
+    cfg, w, folder = lm_util.build(synth, tmp_path, name)
     t = {"a": prompt(cfg, 90, 1), "b": prompt(cfg, 50, 2), "c": prompt(cfg, 30, 3)}
     want = {k: lm_util.reference(cfg, w, v) for k, v in t.items()}
     plan = [[("a", 40), ("b", 1)], [("b", 48), ("a", 1)], [("a", 2)], [("b", 1), ("a", 20)], [("c", 30), ("a", 27)]]
@@ -358,8 +364,9 @@ def test_trace_run_replays(synth, tmp_path, torch_dev):
                 assert error(got, np.array(mine)) < TOL[code]
 
 
-def test_cml_generate_program(pkg, synth, tmp_path, load):
-    cfg, w, folder = lm_util.build(synth, tmp_path, "plain")
+@pytest.mark.parametrize("name", ["plain", "latent_odd"])
+def test_cml_generate_program(pkg, synth, tmp_path, load, name):
+    cfg, w, folder = lm_util.build(synth, tmp_path, name)
     prompts = [prompt(cfg, 9, 1).tolist(), prompt(cfg, 30, 2).tolist()]
     args = sum((["--tokens", ",".join(map(str, p))] for p in prompts), [])
     r = subprocess.run([str(ROOT / "bin" / "cml_generate"), "--model", str(folder), "--dtype", "float32", "--max-new", "11", *args],

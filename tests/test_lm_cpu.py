@@ -7,6 +7,7 @@ from pathlib import Path
 import numpy as np
 import pytest
 
+import latent_oracle as la
 import lm_oracle as lo
 import lm_util
 
@@ -46,10 +47,10 @@ def test_norm_and_activation():
     assert np.allclose(lo.gelu_tanh(np.array([0.0, 1.0, -1.0])), [0.0, 0.841192, -0.158808], atol=1e-6)
 
 
-@pytest.mark.parametrize("name", ["mixed", "odd", "wide", "plain"])
+@pytest.mark.parametrize("name", ["mixed", "odd", "wide", "plain", "latent", "latent_odd", "latent_wide", "latent_full"])
 def test_portions_change_nothing(synth, tmp_path, name):
     cfg, w, _ = lm_util.build(synth, tmp_path, name)
-    m = lo.Model(cfg, w)
+    m = lm_util.model(cfg, w)
     tokens = np.random.default_rng(3).integers(0, cfg["vocab"], 60)
     whole = m.forward(tokens)
     state = m.new_state()
@@ -65,8 +66,92 @@ def test_shared_weights_keep_their_own_cache(synth, tmp_path):
     assert not np.allclose(st["caches"][0]["k"], st["caches"][2]["k"]) and not any(n.startswith("l2.") for n in w)
 
 
+def test_every_setting_shows_in_the_logits(synth, tmp_path):
+    """Configurations of the end-to-end tests are such that a setting read wrongly moves the logits."""
+    cfg, w, _ = lm_util.build(synth, tmp_path, "latent")
+    t = np.random.default_rng(3).integers(0, cfg["vocab"], 90)
+    want = lm_util.reference(cfg, w, t)
+
+    def moved(change, w2=None):
+        other = json.loads(json.dumps(cfg))
+        change(other["layers"])
+        assert lm_util.error(lm_util.reference(other, w2 or w, t), want) > 100 * lm_util.TOL[0]
+    moved(lambda l: l[1]["mixer"]["mask"].update(size=18))
+    moved(lambda l: l[3]["mixer"]["mask"].update(size=71))
+    moved(lambda l: l[0]["mixer"]["rot"].update(base=10100.0))
+    moved(lambda l: l[0]["mixer"].update(scale=0.18))
+    for k, v in (("factor", 3.0), ("original", 32), ("fast", 4.0), ("slow", 3.0)):
+        moved(lambda l: l[1]["mixer"]["rot"]["scaling"].update({k: v}))
+    moved(lambda l: l[1]["mixer"]["rot"].pop("scaling"))
+    moved(lambda l: l[1]["mlp"]["router"].update(top=1))
+    moved(lambda l: l[4]["mlp"]["expert"].update(limit=0.5))
+    moved(lambda l: l[1].update(type="latent_attention"))                # no gate
+    for name in ("l0.mlp.act", "l2.mix.uk", "l2.mix.uv", "l3.mix.g", "l0.mix.dkv.norm", "l4.mlp.e3.up", "final.norm"):
+        w2 = dict(w)
+        w2[name] = w[name][::-1]
+        moved(lambda l: None, w2)
+
+
+# ---- the latents' restatement -----------------------------------------------------------------------------
+def test_rotation_by_hand():
+    rot = {"dims": 4, "base": 100.0}
+    f, mul = la.frequencies(rot)
+    assert np.allclose(f, [1.0, 0.1]) and mul == 1.0
+    x = np.array([[1.0, 2.0, 3.0, 4.0]] * 2)
+    y = la.rotate(x, [0, 5], rot)
+    assert np.allclose(y[0], x[0])
+    c, s = np.cos([5.0, 0.5]), np.sin([5.0, 0.5])
+    assert np.allclose(y[1], [1 * c[0] - 3 * s[0], 2 * c[1] - 4 * s[1], 3 * c[0] + 1 * s[0], 4 * c[1] + 2 * s[1]])
+
+
+def test_frequency_scaling_by_hand():
+    # dims 8, base 10^4: f = 1, .1, .01, .001. Turns within 200 positions: 31.8, 3.18, 0.318, 0.0318
+    f, mul = la.frequencies({"dims": 8, "base": 10000.0, "scaling": {"factor": 5.0, "original": 200, "fast": 10.0, "slow": 0.1}})
+    at = lambda t: 8 * np.log(200 / (2 * np.pi * t)) / (2 * np.log(10000.0))
+    lo, hi = np.floor(at(10.0)), np.ceil(at(0.1))
+    assert (lo, hi) == (0, 3)
+    ramp = np.arange(4) / 3
+    plain = np.array([1, 0.1, 0.01, 0.001])
+    assert np.allclose(f, plain * (1 - ramp) + plain / 5 * ramp) and np.isclose(mul, 1 + 0.1 * np.log(5.0))
+    f, _ = la.frequencies({"dims": 8, "base": 10000.0, "scaling": {"factor": 5.0, "original": 2, "fast": 10.0, "slow": 9.0}})
+    assert np.allclose(f, plain / 5 * np.array([0, 1, 1, 1]) + plain * np.array([1, 0, 0, 0]))     # both ends below the first pair: a step
+
+
+def test_visibility_and_softmax():
+    assert la.visible([5], range(8), 3)[0].tolist() == [False] * 3 + [True] * 3 + [False] * 2
+    assert la.visible([5], range(8), None)[0].tolist() == [True] * 6 + [False] * 2
+    assert np.allclose(la.softmax(np.array([[0.0, np.log(3.0), 9.0]]), np.array([[True, True, False]])), [[0.25, 0.75, 0.0]])
+
+
+def test_poly_norm_by_hand():
+    z = np.array([[1.0, -2.0]])
+    n = lambda v: v / np.sqrt((v ** 2).mean() + 0.5)
+    assert np.allclose(la.poly_norm(z, [2.0, 3.0, 5.0, 7.0], 0.5), 2 * n(z) + 3 * n(z ** 2) + 5 * n(z ** 3) + 7)
+
+
+def test_routing_and_experts_by_hand():
+    ids, wt = la.route(np.array([[1.0, 0.0]]), np.array([[0.0, 9.0], [2.0, 0.0], [2.0, 0.0], [1.0, 0.0]]), 2)
+    e = np.exp([0.0, 2.0, 2.0, 1.0])
+    assert ids.tolist() == [[1, 2]] and np.allclose(wt, e[1] / e.sum())                  # not renormalised; a tie goes to the lower index
+    g, u = np.array([5.0, -5.0, 1.0]), np.array([3.0, -3.0, 0.5])
+    sg = lambda z: 1 / (1 + np.exp(-1.702 * z))
+    assert np.allclose(la.clamped_glu(g, u, 2.0), [2 * sg(2.0) * 3, -5 * sg(-5.0) * -1, sg(1.0) * 1.5])
+    w = {"router": np.array([[1.0], [2.0]]), **{f"e{i}.{n}": np.array([[float(i + 1)]]) for i in range(2) for n in ("gate", "up", "down")}}
+    out = la.experts(np.array([[1.0]]), w, {"router": {"experts": 2, "top": 1}, "expert": {"limit": 9.0}})
+    assert np.allclose(out, np.exp(2) / (np.exp(1) + np.exp(2)) * 2 * (2 * sg(2.0) * 3))
+
+
+def test_a_layer_reads_the_named_cache(synth, tmp_path):
+    cfg, w, _ = lm_util.build(synth, tmp_path, "latent")
+    m = lm_util.model(cfg, w)
+    st = m.new_state()
+    m.forward([1, 2, 3], st)
+    assert st["caches"][2] == {} and len(st["caches"][0]["c"]) == 3 and "l2.mix.dkv" not in w
+
+
 # ---- registry and readers ------------------------------------------------------------------------------
 def test_registry_knows_its_classes(pkg):
+    assert pkg.lib.cml_lm_known(b"Situlorn") == 1
     assert pkg.lib.cml_lm_known(b"Rarolorn") == 1 and pkg.lib.cml_lm_known(b"llama") == 1
     assert pkg.lib.cml_lm_known(b"nothing") == 0 and pkg.lib.cml_lm_known(None) == 0
     o = pkg.lib.cml_lm_default_options()
@@ -108,6 +193,38 @@ def test_load_refusals(pkg, synth, tmp_path):
     assert not _load(pkg, folder) and not _load(pkg, tmp_path / "absent")
     (folder / "config.json").write_text(json.dumps(cfg))
     assert not _load(pkg, folder, dtype=pkg.DTYPE_BFLOAT16 + 1) and not _load(pkg, folder, max_tokens=0) and not _load(pkg, folder, max_sequences=0)
+
+
+def test_latent_load_refusals(pkg, synth, tmp_path):
+    cfg, w, folder = lm_util.build(synth, tmp_path, "latent")
+    mixer = lambda c, i: c["layers"][i]["mixer"]
+
+    def with_config(change):
+        c = json.loads(json.dumps(cfg))
+        change(c)
+        (folder / "config.json").write_text(json.dumps(c))
+        assert not _load(pkg, folder)
+
+    for key in ("heads", "dim", "rot_dim", "vdim", "kv_rank", "scale", "rot"):
+        with_config(lambda c: mixer(c, 0).pop(key))
+    with_config(lambda c: c["layers"][0].update(type="attention"))                        # another design's mixer
+    with_config(lambda c: c["layers"][0].update(type="latent_attention_3"))
+    with_config(lambda c: mixer(c, 0)["rot"].update(dims=6))                                 # not rot_dim
+    with_config(lambda c: (mixer(c, 0)["rot"].update(dims=7), mixer(c, 0).update(rot_dim=7)))
+    with_config(lambda c: mixer(c, 0)["rot"].update(base=1.0))
+    with_config(lambda c: mixer(c, 1)["rot"]["scaling"].pop("slow"))
+    with_config(lambda c: mixer(c, 1)["rot"]["scaling"].update(factor=0))
+    with_config(lambda c: mixer(c, 1)["mask"].update(size=0))
+    with_config(lambda c: mixer(c, 0).update(kv_rank=513))
+    for j in (-1, 2, 3, 4, 9, 1, 0.5):                                                       # itself or later, unlike latents, not a layer
+        with_config(lambda c: mixer(c, 2).update(kv_from=j))
+    with_config(lambda c: mixer(c, 4).update(kv_from=2))                                     # has no latents of its own
+    with_config(lambda c: mixer(c, 2)["rot"].update(base=500.0))
+    with_config(lambda c: c["layers"][1]["mlp"]["router"].update(top=6))
+    with_config(lambda c: c["layers"][1]["mlp"]["router"].update(experts=0))
+    with_config(lambda c: c["layers"][1]["mlp"].pop("expert"))
+    with_config(lambda c: c["layers"][1]["mlp"].update(kind="dense"))
+    with_config(lambda c: c["layers"][0]["mlp"].update(ff=-1))
 
 
 def test_tensor_file_refusals(pkg, synth, tmp_path):
