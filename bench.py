@@ -387,6 +387,8 @@ def main():
     ap.add_argument("--only-gemm", action="store_true", help="run the NF4 prefill-GEMM leg alone")
     ap.add_argument("--layered", nargs="?", const="all", default=None, choices=["all", "kernels", "models"],
                     help="instead of the default workload: the layered models beside LLaMA at equal layer sizes, and their kernels")
+    ap.add_argument("--latent", nargs="?", const="all", default=None, choices=["all", "kernels", "models"],
+                    help="instead of the default workload: models with latent attention and experts beside the layered model of equal sizes, and their kernels")
     ap.add_argument("--cpu-leg", default=None, choices=["gemv", "llama"], help=argparse.SUPPRESS)
     ap.add_argument("--calls", type=int, default=3, help=argparse.SUPPRESS)
     ap.add_argument("--llama-steps", type=int, default=4, help=argparse.SUPPRESS)
@@ -423,6 +425,9 @@ def main():
     if args.layered:
         import bench_layered
         return bench_layered.run(pkg, synth, torch, peaks, ClockSampler(local), args.layered == "kernels", args.layered == "models")
+    if args.latent:
+        import bench_latent
+        return bench_latent.run(pkg, synth, torch, peaks, ClockSampler(local), args.latent == "kernels", args.latent == "models")
     stream = torch.cuda.Stream(device=dev)
     sp = stream.cuda_stream
 

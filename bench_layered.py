@@ -23,11 +23,17 @@ def model_sizes(c):
 
 
 def layered_leg(pkg, synth, torch, c, peaks):
-    rng = np.random.default_rng(5)
     layer = lambda: synth.layered_layer(c["heads"], c["kv_heads"], c["dim"], c["dim"], c["window"], c["ff"], coef=0.1, every=512)
     cfg = synth.layered_config(c["vocab"], c["width"], [layer() for _ in range(c["layers"])])
     total, body = model_sizes(c)
-    out = {"weight_bytes": 2 * total}
+    return model_leg(pkg, synth, torch, cfg, c, peaks, body, lambda B: total, lambda: 4 * c["layers"] * c["kv_heads"] * c["dim"])
+
+
+def model_leg(pkg, synth, torch, cfg, c, peaks, body, weights, cache_bytes):
+    """Prefill and decode of a configuration with random weights. body: multiplications per token of a prompt. weights(B): those a
+    decode step of B rows reads. cache_bytes(): read per row and cached token, all layers together (c["window"] of them)."""
+    rng = np.random.default_rng(5)
+    out = {"weight_bytes": 2 * weights(max(c["batches"]))}
     with tempfile.TemporaryDirectory() as tmp:
         gen = lambda name, shape: (1 + 0.1 * rng.standard_normal(shape, dtype=np.float32)) if len(shape) == 1 else \
             rng.standard_normal(shape, dtype=np.float32) * np.float32(1.0 if name == "embed" else shape[1] ** -0.5)
@@ -58,7 +64,7 @@ def layered_leg(pkg, synth, torch, c, peaks):
         for s in seqs:
             m.end(s)
         step = ms / NEW
-        nbytes = 2 * total + 2 * 2 * c["layers"] * B * c["window"] * c["kv_heads"] * c["dim"]
+        nbytes = 2 * weights(B) + B * c["window"] * cache_bytes()
         out[f"decode_b{B}"] = {"tok_s": B / (step * 1e-3), "ms_per_step": step, "gbs": nbytes / (step * 1e-3) / 1e9,
                                "frac_of_hbm": nbytes / (step * 1e-3) / 1e9 / peaks["hbm_gbs"]}
     m.close()
@@ -115,6 +121,7 @@ class Timer:
 
     def us(self, calls, sweeps):
         torch = self.torch
+        torch.cuda.synchronize()                       # the buffers were filled on another stream
         with torch.cuda.stream(self.stream):
             for f in calls:
                 f(self.stream.cuda_stream)
