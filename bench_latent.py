@@ -182,7 +182,7 @@ def attention(pkg, torch, T, add):
             tile = i32([0, rows, 0, ctx])
             pairs = rows * ctx + rows * (rows + 1) / 2
             add("attention_latent (portion)", f"H={H} rows={rows} ctx={ctx}",
-                T.us([lambda s: ck(lib.cmlb200_attention_latent(a, q.data_ptr(), None, None, 0, 0, tile.data_ptr(), 1, o.data_ptr(), s))], 10), 2.0 * ctx * (R + P), 2.0 * pairs * H * (2 * R + P))
+                T.us([lambda s: ck(lib.cmlb200_attention_latent(a, q.data_ptr(), None, None, 0, ctx + rows, tile.data_ptr(), 1, o.data_ptr(), s))], 10), 2.0 * ctx * (R + P), 2.0 * pairs * H * (2 * R + P))
             per, kp = (ctx + rows) // 16 + 1, []
             tab = torch.arange(per, device=dev, dtype=torch.int32).view(1, -1).contiguous()
             kk, vv = torch.randn(per * 16, H, D, device=dev).half(), torch.randn(per * 16, H, D, device=dev).half()

@@ -3,20 +3,22 @@
 // (cmlb200_latent_query), in units of log2. One kernel serves decoded tokens and short prompt portions:
 // the (token, head) pairs of a portion are the rows of the matrix products, 16, 32 or 64 to a CTA.
 //
-// A key tile of 32 tokens is fetched once through the block table (cp.async, three stages) and serves both products on
-// mma.sync m16n8k16: S = Q K^T with the warps splitting rows, keys and, for few rows, the key columns; O += P K with the
-// warps splitting the latent's columns. Scores pass through shared memory, where a few threads per row keep
-// the running maximum and sum in fp32. A cluster of up to 8 CTAs splits the keys and merges through distributed
-// shared memory, each CTA finishing a share of the values.
+// A key tile of 32 tokens is fetched once through the block table (cp.async, two or three stages) and serves both products
+// on mma.sync m16n8k16: S = Q K^T with the warps splitting rows, keys and, for few rows, the key columns; O += P K with
+// the warps splitting the latent's columns. Scores pass through shared memory, where a few threads per row keep
+// the running maximum and sum in fp32. A cluster of up to 16 CTAs splits the keys and merges through distributed
+// shared memory, each CTA finishing a share of the values. A tile is a chain of short dependent phases, so the narrow
+// form (16 rows) is sized for two CTAs to an SM.
 #include "lm_util.cuh"
 
 namespace {
 
-constexpr int LT_THREADS = 256, LT_WARPS = 8, LT_KEYS = 32, LT_STAGES = 3, LT_SLD = LT_KEYS + 4, LT_PLD = LT_KEYS + 8;
+constexpr int LT_THREADS = 256, LT_WARPS = 8, LT_KEYS = 32, LT_SPLITS = 16, LT_SLD = LT_KEYS + 4, LT_PLD = LT_KEYS + 8;
 
+__host__ __device__ constexpr int latent_stages(int rows) { return rows == 16 ? 2 : 3; }
 __host__ __device__ inline size_t latent_smem(int rows, int ld, int ldo) {
     const size_t lk = ld + 8;
-    const size_t tiles = 2 * lk * (rows + LT_STAGES * LT_KEYS), merge = 4 * (size_t)rows * ldo;
+    const size_t tiles = 2 * lk * (rows + latent_stages(rows) * LT_KEYS), merge = 4 * (size_t)rows * ldo;
     // operands, or the merged values in their place; scores (64 rows of partial sums), weights, per-row factors
     return (tiles > merge ? tiles : merge) + 4 * 64 * LT_SLD + 2 * (size_t)rows * LT_PLD + 3 * 4 * (size_t)rows;
 }
@@ -24,15 +26,15 @@ __host__ __device__ inline size_t latent_smem(int rows, int ld, int ldo) {
 // grid = (splits, ceil(tokens * heads / (16 MT)), items), clusters of `splits` CTAs along x. CU: 16-column groups of the
 // latent per warp.
 template <int MT, int CU>
-__global__ void __launch_bounds__(LT_THREADS)
+__global__ void __launch_bounds__(LT_THREADS, MT == 1 ? 2 : 1)
 attention_latent_kernel(const cmlb200_latent a, const __half* __restrict__ q, const int* __restrict__ row_pos, const int* __restrict__ row_slot,
                         const int4* __restrict__ tiles, int first, __nv_bfloat16* __restrict__ out) {
-    constexpr int MR = 16 * MT, KS = 4 / MT, TPR = LT_THREADS / MR, KPT = LT_KEYS / TPR;
+    constexpr int MR = 16 * MT, NS = latent_stages(MR), KS = 4 / MT, TPR = LT_THREADS / MR, KPT = LT_KEYS / TPR;
     extern __shared__ __align__(16) uint8_t sm[];
     const int LK = a.ld + 8, rank16 = (a.rank + 15) & ~15, LDO = rank16 + 4;
     __half* Qs = reinterpret_cast<__half*>(sm);
     __half* Ks = Qs + MR * LK;
-    const size_t tile_bytes = 2 * (size_t)LK * (MR + LT_STAGES * LT_KEYS), merge_bytes = 4 * (size_t)MR * LDO;
+    const size_t tile_bytes = 2 * (size_t)LK * (MR + NS * LT_KEYS), merge_bytes = 4 * (size_t)MR * LDO;
     float* Ss = reinterpret_cast<float*>(sm + (tile_bytes > merge_bytes ? tile_bytes : merge_bytes));   // [KS][MR][LT_SLD]
     __half* Ps = reinterpret_cast<__half*>(Ss + 64 * LT_SLD);
     float* corr = reinterpret_cast<float*>(Ps + MR * LT_PLD);           // factor on the sums so far, then 1 / sum
@@ -55,24 +57,29 @@ attention_latent_kernel(const cmlb200_latent a, const __half* __restrict__ q, co
     const __half* pool = static_cast<const __half*>(a.pool);
     const int kc = a.ld >> 3;
 
+    // a thread copies a part of one key per tile; where that key lies is looked up a tile ahead
+    auto slot_of = [&](int it) {
+        const int key = min(k_lo + it * LT_KEYS + (int)(threadIdx.x >> 3), p_last);        // past the end: the last key, masked below
+        return (table[key >> shift] << shift) + (key & (a.block_size - 1));
+    };
+    int next_slot = slot_of(rank);
     auto load = [&](int it, int stage) {
         if (it < ntiles) {
-            const int row = threadIdx.x >> 3, key = min(k_lo + it * LT_KEYS + row, p_last);       // past the end: the last key, masked below
-            const __half* src = pool + (((size_t)table[key >> shift] << shift) + (key & (a.block_size - 1))) * a.ld;
-            const uint32_t dst = smem_addr(Ks + (stage * LT_KEYS + row) * LK);
+            const __half* src = pool + (size_t)next_slot * a.ld;
+            const uint32_t dst = smem_addr(Ks + (stage * LT_KEYS + (threadIdx.x >> 3)) * LK);
+#pragma unroll 3
             for (int c = threadIdx.x & 7; c < kc; c += 8) cp16(dst + c * 16, src + c * 8);
+            next_slot = slot_of(it + splits);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     {
         const __half* src = q + ((size_t)tl.x * a.heads + m0) * a.ld;
-        for (int i = threadIdx.x; i < MR * kc; i += LT_THREADS) {
-            const int r = i / kc, c = i - r * kc;
-            cp16(smem_addr(Qs + r * LK + c * 8), src + (size_t)min(r, total - 1 - m0) * a.ld + c * 8);
-        }
+        for (int r = threadIdx.x >> 3; r < MR; r += LT_THREADS / 8)
+            for (int c = threadIdx.x & 7; c < kc; c += 8) cp16(smem_addr(Qs + r * LK + c * 8), src + (size_t)min(r, total - 1 - m0) * a.ld + c * 8);
     }
-    load(rank, 0);
-    load(rank + splits, 1);
+#pragma unroll
+    for (int i = 0; i < NS - 1; i++) load(rank + i * splits, i);
 
     float o[MT][CU][2][4];
 #pragma unroll
@@ -91,20 +98,34 @@ attention_latent_kernel(const cmlb200_latent a, const __half* __restrict__ q, co
 
     int stage = 0;
     for (int it = rank; it < ntiles; it += splits) {
-        asm volatile("cp.async.wait_group 1;" ::: "memory");
+        asm volatile("cp.async.wait_group %0;" ::"n"(NS - 2) : "memory");
         __syncthreads();                                                // this tile is there; the stage of the one before is free
-        load(it + 2 * splits, stage == 0 ? 2 : stage - 1);
+        load(it + (NS - 1) * splits, stage == 0 ? NS - 1 : stage - 1);
         {
-            float s[2][4] = {};
+            float s[2][4] = {}, s2[2][4] = {};
             const uint32_t k_base = smem_addr(Ks + (stage * LT_KEYS + w_k * 16 + (lane & 7) + ((lane >> 4) & 1) * 8) * LK + ((lane >> 3) & 1) * 8);
-#pragma unroll 4
-            for (int kk = w_s * 16; kk < a.ld; kk += KS * 16) {
-                uint32_t qa[4], b[4];
-                ldsm4(q_base + kk * 2, qa);
-                ldsm4(k_base + kk * 2, b);
-                mma_f16(s[0], qa, b[0], b[1]);
-                mma_f16(s[1], qa, b[2], b[3]);
+            // fragments of a step are requested before the products of the one ahead of it
+            uint32_t qa[2][4], kb[2][4];
+            auto fetch = [&](int kk, int e) {
+                ldsm4(q_base + kk * 2, qa[e]);
+                ldsm4(k_base + kk * 2, kb[e]);
+            };
+            constexpr int STEP = KS * 16;
+            if (w_s * 16 < a.ld) fetch(w_s * 16, 0);
+#pragma unroll 1
+            for (int kk = w_s * 16; kk < a.ld; kk += 2 * STEP) {
+                if (kk + STEP < a.ld) fetch(kk + STEP, 1);
+                mma_f16(s[0], qa[0], kb[0][0], kb[0][1]);
+                mma_f16(s[1], qa[0], kb[0][2], kb[0][3]);
+                if (kk + STEP >= a.ld) break;
+                if (kk + 2 * STEP < a.ld) fetch(kk + 2 * STEP, 0);
+                mma_f16(s2[0], qa[1], kb[1][0], kb[1][1]);
+                mma_f16(s2[1], qa[1], kb[1][2], kb[1][3]);
             }
+#pragma unroll
+            for (int j = 0; j < 2; j++)
+#pragma unroll
+                for (int e = 0; e < 4; e++) s[j][e] += s2[j][e];
             float* d = Ss + (w_s * MR + w_m * 16 + g) * LT_SLD + w_k * 16 + 2 * t;
 #pragma unroll
             for (int j = 0; j < 2; j++) {
@@ -155,24 +176,26 @@ attention_latent_kernel(const cmlb200_latent a, const __half* __restrict__ q, co
                 }
             }
             const uint32_t v_base = smem_addr(Ks + (stage * LT_KEYS + (lane & 15)) * LK + (lane >> 4) * 8);
+            constexpr int KK = LT_KEYS / 16;
+            uint32_t vb[2][4];
+            auto fetch = [&](int i) {                                   // product i: columns i / KK, keys i % KK
+                const int col = (i / KK * LT_WARPS + warp) * 16;
+                if (col < rank16) ldsm4_t(v_base + (i % KK * 16 * LK + col) * 2, vb[i & 1]);
+            };
+            fetch(0);
 #pragma unroll
-            for (int u = 0; u < CU; u++) {
-                const int col = (u * LT_WARPS + warp) * 16;
-                if (col < rank16) {
+            for (int i = 0; i < CU * KK; i++) {
+                if (i + 1 < CU * KK) fetch(i + 1);
+                if ((i / KK * LT_WARPS + warp) * 16 < rank16) {
 #pragma unroll
-                    for (int kk = 0; kk < LT_KEYS / 16; kk++) {
-                        uint32_t b[4];
-                        ldsm4_t(v_base + (kk * 16 * LK + col) * 2, b);
-#pragma unroll
-                        for (int i = 0; i < MT; i++) {
-                            mma_f16(o[i][u][0], pa[i][kk], b[0], b[1]);
-                            mma_f16(o[i][u][1], pa[i][kk], b[2], b[3]);
-                        }
+                    for (int r = 0; r < MT; r++) {
+                        mma_f16(o[r][i / KK][0], pa[r][i % KK], vb[i & 1][0], vb[i & 1][1]);
+                        mma_f16(o[r][i / KK][1], pa[r][i % KK], vb[i & 1][2], vb[i & 1][3]);
                     }
                 }
             }
         }
-        stage = stage == 2 ? 0 : stage + 1;
+        stage = stage == NS - 1 ? 0 : stage + 1;
     }
     asm volatile("cp.async.wait_group 0;" ::: "memory");
 #pragma unroll
@@ -224,9 +247,9 @@ attention_latent_kernel(const cmlb200_latent a, const __half* __restrict__ q, co
     const int live = min(MR, total - m0);
     for (int i = rank * LT_THREADS + threadIdx.x; i < live * a.rank; i += splits * LT_THREADS) {
         const int r = i / a.rank, d = i - r * a.rank;
-        float ms[8], ls[8], xs[8];
+        float ms[LT_SPLITS], ls[LT_SPLITS], xs[LT_SPLITS];
 #pragma unroll
-        for (int s = 0; s < 8; s++) {
+        for (int s = 0; s < LT_SPLITS; s++) {
             ms[s] = -INFINITY; ls[s] = 0.f; xs[s] = 0.f;
             if (s < splits) {
                 uint32_t am, al, ax;
@@ -240,9 +263,9 @@ attention_latent_kernel(const cmlb200_latent a, const __half* __restrict__ q, co
         }
         float mx = ms[0], x = 0.f, sum = 0.f;
 #pragma unroll
-        for (int s = 1; s < 8; s++) mx = fmaxf(mx, ms[s]);
+        for (int s = 1; s < LT_SPLITS; s++) mx = fmaxf(mx, ms[s]);
 #pragma unroll
-        for (int s = 0; s < 8; s++) {
+        for (int s = 0; s < LT_SPLITS; s++) {
             const float c = ms[s] == -INFINITY ? 0.f : exp2f(ms[s] - mx);
             x = fmaf(xs[s], c, x);
             sum = fmaf(ls[s], c, sum);
@@ -258,7 +281,7 @@ attention_latent_kernel(const cmlb200_latent a, const __half* __restrict__ q, co
 extern "C" int cmlb200_attention_latent(const cmlb200_latent* a, const uint16_t* d_q_f16, const int* d_row_pos, const int* d_row_slot, int rows, int max_keys,
                                         const int* d_tiles, int tiles, uint16_t* d_o_bf16, void* stream) {
     static const char* who = "cmlb200_attention_latent";
-    CMLB_REQUIRE(a && d_q_f16 && d_o_bf16 && (d_tiles ? tiles > 0 && rows >= 0 : d_row_pos && d_row_slot && rows > 0 && max_keys >= 0), "%s: bad argument", who);
+    CMLB_REQUIRE(a && d_q_f16 && d_o_bf16 && (d_tiles ? tiles > 0 && rows >= 0 : d_row_pos && d_row_slot && rows > 0) && max_keys >= 0, "%s: bad argument", who);
     CMLB_REQUIRE(a->heads > 0 && a->rank > 0 && a->ld >= a->rank && a->ld % 16 == 0 && a->ld_rank >= a->rank && a->ld_rank % 64 == 0 && a->rank <= 512,
                  "%s: rank %d (up to 512), strides %d / %d", who, a->rank, a->ld, a->ld_rank);
     CMLB_REQUIRE(a->pool && a->block_table && a->table_ld > 0 && a->cache_dtype == CMLB200_DT_F16, "%s: fp16 cache", who);
@@ -266,17 +289,25 @@ extern "C" int cmlb200_attention_latent(const cmlb200_latent* a, const uint16_t*
     CMLB_REQUIRE((((uintptr_t)d_q_f16 | (uintptr_t)a->pool | (uintptr_t)d_tiles) & 15) == 0 && ((uintptr_t)d_o_bf16 & 3) == 0, "%s: alignment", who);
     const int items = d_tiles ? tiles : rows, most = d_tiles ? 64 * a->heads : a->heads, sms = cmlb_num_sms();
     CMLB_REQUIRE(items <= 65535, "%s: %d rows", who, items);
-    const int keys = d_tiles ? LT_KEYS : ((a->window > 0 && a->window < max_keys + 1) ? a->window : max_keys + 1);
-    const int rank16 = (a->rank + 15) & ~15;
-    // rows per CTA: wide tiles read the keys fewest times; narrow ones spread few heads over more SMs
-    int mt = most > 32 ? 4 : (most > 16 ? 2 : 1);
+    const int keys = (a->window > 0 && a->window < max_keys + 1) ? a->window : max_keys + 1, rank16 = (a->rank + 15) & ~15;
     auto blocks = [&](int m) { return (long)items * ((most + 16 * m - 1) / (16 * m)); };
-    auto most_splits = [&]() { int s = 1; while (s < 8 && keys > s * LT_KEYS) s *= 2; return s; };
-    while (mt > 1 && (latent_smem(16 * mt, a->ld, rank16 + 4) > 227 * 1024 || (!d_tiles && blocks(mt) * most_splits() < sms))) mt /= 2;
-    int splits = 1;
-    while (splits < 8 && blocks(mt) * splits < sms && keys > splits * LT_KEYS) splits *= 2;
+    // rows per CTA and parts of the keys, by an estimate of the time in microseconds: wide tiles do more per key, narrow
+    // ones and more parts spread few heads over more SMs
+    int mt = 0, splits = 1;
+    double best = 0.0;
+    for (int m = 1; m <= 4; m *= 2) {
+        const size_t bytes = latent_smem(16 * m, a->ld, rank16 + 4);
+        if (bytes > 227 * 1024 || (m > 1 && most <= 8 * m)) continue;
+        const double tile = m == 1 ? 1.2 : (m == 2 ? 1.6 : 2.8);
+        const long room = (long)sms * (m == 1 && 2 * bytes + 2048 <= 228 * 1024 ? 2 : 1);
+        for (int s = 1; s <= (m == 1 ? LT_SPLITS : LT_SPLITS / 2) && (s == 1 || (s - 1) * LT_KEYS < keys); s *= 2) {
+            const long ctas = blocks(m) * s, waves = (ctas + room - 1) / room, tiles_each = ((keys + LT_KEYS - 1) / LT_KEYS + s - 1) / s;
+            const double t = (double)waves * (3.0 + tile * (double)tiles_each) + (s > 1 ? 1.0 : 0.0);
+            if (!mt || t < best) { mt = m; splits = s; best = t; }
+        }
+    }
+    CMLB_REQUIRE(mt > 0, "%s: rank %d and %d elements per token do not fit shared memory", who, a->rank, a->ld);
     const size_t smem = latent_smem(16 * mt, a->ld, rank16 + 4);
-    CMLB_REQUIRE(smem <= 227 * 1024, "%s: rank %d and %d elements per token do not fit shared memory", who, a->rank, a->ld);
     const long per = blocks(mt) / items;
     CMLB_REQUIRE(per <= 65535, "%s: %d heads", who, a->heads);
     const dim3 grid(splits, (unsigned)per, items);
@@ -286,6 +317,7 @@ extern "C" int cmlb200_attention_latent(const cmlb200_latent* a, const uint16_t*
     do {                                                                                                                         \
         auto kern = attention_latent_kernel<MT, CU>;                                                                             \
         CMLB_CUDA(cmlb_ensure_smem(kern, smem, attr[slot]));                                                                     \
+        if (splits > 8) CMLB_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeNonPortableClusterSizeAllowed, 1));                \
         CMLB_CUDA(launch_chain(kern, grid, dim3(LT_THREADS), smem, splits, st, *a, (const __half*)d_q_f16, d_row_pos, d_row_slot, (const int4*)d_tiles, d_tiles ? rows : 0, \
                                (__nv_bfloat16*)d_o_bf16));                                                                       \
     } while (0)

@@ -219,7 +219,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constant
                 __syncwarp();
                 if (out.form == OUT_GLU) {
 #pragma unroll
-                    for (int j = 0; j < 16; j++) buf[lane * 33 + j] = glu_act(out.act, __uint_as_float(v[j]), __uint_as_float(v[16 + j]), out.limit);
+                    for (int j = 0; j < 16; j++) buf[lane * 33 + j] = glu_act_fast(out.act, __uint_as_float(v[j]), __uint_as_float(v[16 + j]), out.limit);
                     __syncwarp();
                     const int col = (n0 + c0) / 2 + (lane & 15);
 #pragma unroll 4

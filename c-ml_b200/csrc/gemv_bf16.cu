@@ -118,7 +118,7 @@ gemv_bf16_kernel(const __nv_bfloat16* __restrict__ W, int ldw, const __nv_bfloat
         }
         if (GLU) {
             const int c = blockIdx.x * 16 + n;
-            if (c < N) static_cast<__nv_bfloat16*>(y)[(size_t)(first + m) * ldy + c] = __float2bfloat16_rn(glu_act(act, s, s2, limit));
+            if (c < N) static_cast<__nv_bfloat16*>(y)[(size_t)(first + m) * ldy + c] = __float2bfloat16_rn(glu_act_fast(act, s, s2, limit));
         } else if (n0 + n < N) {
             static_cast<float*>(y)[(size_t)(first + m) * ldy + n0 + n] = s;
         }

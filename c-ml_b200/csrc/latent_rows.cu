@@ -38,6 +38,7 @@ __device__ __forceinline__ void latent_row(const cmlb200_latent& a, const float*
     if (a.kv_col >= 0) {
         const size_t at = (size_t)a.block_table[(size_t)slot * a.table_ld + p / a.block_size] * a.block_size + p % a.block_size;
         KV* d = static_cast<KV*>(a.pool) + at * a.ld;
+#pragma unroll 4
         for (int i = threadIdx.x; i < a.rank; i += nt) d[i] = narrow<KV>(kv[i] * inv * a.c_norm[i]);
         for (int i = threadIdx.x; i < half; i += nt) {
             const float u = kv[a.rank + i], v = kv[a.rank + half + i];
@@ -47,6 +48,7 @@ __device__ __forceinline__ void latent_row(const cmlb200_latent& a, const float*
         for (int i = a.rank + a.rot_dim + threadIdx.x; i < a.ld; i += nt) d[i] = narrow<KV>(0.f);
     }
     const int hd = a.dim + a.rot_dim;
+#pragma unroll 4
     for (int j = threadIdx.x; j < a.heads * half; j += nt) {
         const int h = j / half, i = j - h * half;
         const float* s = row + h * hd + a.dim;
@@ -79,8 +81,8 @@ latent_append_kernel(const cmlb200_latent a, float* proj, int ld, const int* __r
 
 constexpr int LQ_WARPS = 4, LQ_THREADS = LQ_WARPS * 32, LQ_COLS = LQ_WARPS * 16, LQ_ROWS = 32;
 
-// grid = (rank / 64, heads + 1, rows / 32). Blocks y < heads: q16[row][y][n] = scale log2 e sum_d q[row][y][d] Wuk[y][d][n],
-// a warp per 16 outputs n, up to 32 rows. Blocks y == heads: latent_row of the same rows, shared out over x.
+// grid = (rank / 64, heads + extra, rows / 32). Blocks y < heads: q16[row][y][n] = scale log2 e sum_d q[row][y][d] Wuk[y][d][n],
+// a warp per 16 outputs n, up to 32 rows. The blocks behind them: latent_row of the same rows, one each.
 template <int NB>
 __global__ void __launch_bounds__(LQ_THREADS)
 latent_query_kernel(const cmlb200_latent a, const __nv_bfloat16* __restrict__ wukt, const float* __restrict__ proj, int ld, const int* __restrict__ row_pos,
@@ -89,14 +91,13 @@ latent_query_kernel(const cmlb200_latent a, const __nv_bfloat16* __restrict__ wu
     __shared__ float red[32];
     const int r0 = blockIdx.z * LQ_ROWS, n = min(LQ_ROWS, rows - r0), hd = a.dim + a.rot_dim;
     const float mul = a.scale * kLog2e;
-    if ((int)blockIdx.y == a.heads) {
+    if ((int)blockIdx.y >= a.heads) {
         dep_wait();
         dep_trigger();
-        for (int r = r0 + blockIdx.x; r < r0 + n; r += gridDim.x) {
-            const QueryOut<__half> q = {q16 + (size_t)r * a.heads * a.ld, a.ld, a.rank, a.ld - a.rank, mul};
-            latent_row<__half, __half>(a, proj + (size_t)r * ld, row_pos[r], row_slot[r], q, reinterpret_cast<float*>(sm), red);
-            __syncthreads();
-        }
+        const int r = r0 + (blockIdx.y - a.heads) * gridDim.x + blockIdx.x;
+        if (r >= r0 + n) return;
+        const QueryOut<__half> q = {q16 + (size_t)r * a.heads * a.ld, a.ld, a.rank, a.ld - a.rank, mul};
+        latent_row<__half, __half>(a, proj + (size_t)r * ld, row_pos[r], row_slot[r], q, reinterpret_cast<float*>(sm), red);
         return;
     }
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, t = lane & 3, h = blockIdx.y;
@@ -119,9 +120,9 @@ latent_query_kernel(const cmlb200_latent a, const __nv_bfloat16* __restrict__ wu
     fetch(1, 64);
     dep_wait();
     dep_trigger();
-    for (int i = threadIdx.x; i < NB * 8 * dp; i += LQ_THREADS) {
-        const int m = i / dp, d = i - m * dp;
-        xs[m * lx + d] = __float2bfloat16_rn(m < n && d < a.dim ? proj[(size_t)(r0 + m) * ld + h * hd + d] : 0.f);
+    for (int d = threadIdx.x; d < dp; d += LQ_THREADS) {
+#pragma unroll
+        for (int m = 0; m < NB * 8; m++) xs[m * lx + d] = __float2bfloat16_rn(m < n && d < a.dim ? proj[(size_t)(r0 + m) * ld + h * hd + d] : 0.f);
     }
     __syncthreads();
     float acc[NB][4];
@@ -235,29 +236,55 @@ struct GatherList {
     int4 k[16];                                         // {slot, first key, keys, first scratch row}
 };
 
-// grid = (blocks of keys, sequences), a warp per key: the latent as bf16 (zeros up to ld_rank), the shared key part into
-// every head's key row behind its `dim` columns, and this block's entry of the scratch's block table.
+// grid = (blocks of keys, sequences, parts): the latent as bf16 (zeros up to ld_rank), the shared key part into every
+// head's key row behind its `dim` columns (heads shared out over the parts), and the block's entry of the scratch's block
+// table. VEC: 8 elements at a time.
+template <bool VEC>
 __global__ void __launch_bounds__(256)
 latent_gather_kernel(const cmlb200_latent a, const GatherList list, __nv_bfloat16* __restrict__ c, __half* __restrict__ keys, int dim_ld,
                      int* __restrict__ table, int table_ld) {
     dep_wait();
     dep_trigger();
     const int4 it = list.k[blockIdx.y];
-    const int bs = a.block_size, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, b = blockIdx.x;
+    const int bs = a.block_size, b = blockIdx.x;
     if (b * bs >= it.z) return;
     const int blk = it.y / bs + b;
     if (threadIdx.x == 0) table[(size_t)it.x * table_ld + blk] = it.w / bs + b;
     const size_t from = (size_t)a.block_table[(size_t)it.x * a.table_ld + blk] * bs;
-    for (int i = warp; i < bs && b * bs + i < it.z; i += 8) {
-        const __half* s = static_cast<const __half*>(a.pool) + (from + i) * a.ld;
-        const size_t row = (size_t)it.w + b * bs + i;
-        for (int d = lane; d < a.ld_rank; d += 32) c[row * a.ld_rank + d] = __float2bfloat16_rn(d < a.rank ? __half2float(s[d]) : 0.f);
-        const int tail = dim_ld - a.dim;
-        __half* k = keys + row * a.heads * dim_ld + a.dim;
-        for (int j = lane; j < a.heads * tail; j += 32) {
-            const int h = j / tail, d = j - h * tail;
-            k[(size_t)h * dim_ld + d] = d < a.rot_dim ? s[a.rank + d] : __float2half_rn(0.f);
+    const int n = min(bs, it.z - b * bs), tail = dim_ld - a.dim, h0 = blockIdx.z, hs = gridDim.z;
+    const size_t row0 = (size_t)it.w + b * bs;
+    const __half* pool = static_cast<const __half*>(a.pool) + from * a.ld;
+    if (VEC) {
+        const int c8 = a.ld_rank >> 3, t8 = tail >> 3;
+        for (int j = blockIdx.z * 256 + threadIdx.x; j < n * c8; j += 256 * hs) {
+            const int i = j / c8, d = (j - i * c8) * 8;
+            uint4 v = make_uint4(0u, 0u, 0u, 0u);
+            if (d < a.rank) {
+                const uint4 w = *reinterpret_cast<const uint4*>(pool + (size_t)i * a.ld + d);
+                const __half2* x = reinterpret_cast<const __half2*>(&w);
+                __nv_bfloat162* y = reinterpret_cast<__nv_bfloat162*>(&v);
+#pragma unroll
+                for (int e = 0; e < 4; e++) { const float2 f = __half22float2(x[e]); y[e] = __floats2bfloat162_rn(f.x, f.y); }
+            }
+            *reinterpret_cast<uint4*>(c + (row0 + i) * a.ld_rank + d) = v;
         }
+        for (int j = threadIdx.x; j < n * t8; j += 256) {
+            const int i = j / t8, d = (j - i * t8) * 8;
+            const uint4 v = d < a.rot_dim ? *reinterpret_cast<const uint4*>(pool + (size_t)i * a.ld + a.rank + d) : make_uint4(0u, 0u, 0u, 0u);
+            __half* k = keys + (row0 + i) * a.heads * dim_ld + a.dim + d;
+            for (int h = h0; h < a.heads; h += hs) *reinterpret_cast<uint4*>(k + (size_t)h * dim_ld) = v;
+        }
+        return;
+    }
+    for (int j = blockIdx.z * 256 + threadIdx.x; j < n * a.ld_rank; j += 256 * hs) {
+        const int i = j / a.ld_rank, d = j - i * a.ld_rank;
+        c[(row0 + i) * a.ld_rank + d] = __float2bfloat16_rn(d < a.rank ? __half2float(pool[(size_t)i * a.ld + d]) : 0.f);
+    }
+    for (int j = threadIdx.x; j < n * tail; j += 256) {
+        const int i = j / tail, d = j - i * tail;
+        const __half v = d < a.rot_dim ? pool[(size_t)i * a.ld + a.rank + d] : __float2half_rn(0.f);
+        __half* k = keys + (row0 + i) * a.heads * dim_ld + a.dim + d;
+        for (int h = h0; h < a.heads; h += hs) k[(size_t)h * dim_ld] = v;
     }
 }
 
@@ -294,7 +321,8 @@ extern "C" int cmlb200_latent_query(const cmlb200_latent* a, const uint16_t* d_w
     if (rc) return rc;
     CMLB_REQUIRE(d_wukt && d_proj && d_row_pos && d_row_slot && rows > 0 && d_q_f16 && a->cache_dtype == CMLB200_DT_F16, "cmlb200_latent_query: bad argument");
     CMLB_REQUIRE(((uintptr_t)d_wukt & 15) == 0 && rows <= 65535 * LQ_ROWS, "cmlb200_latent_query: alignment or %d rows", rows);
-    const dim3 grid((a->rank + LQ_COLS - 1) / LQ_COLS, a->heads + 1, (rows + LQ_ROWS - 1) / LQ_ROWS);
+    const int gx = (a->rank + LQ_COLS - 1) / LQ_COLS, most = rows < LQ_ROWS ? rows : LQ_ROWS;
+    const dim3 grid(gx, a->heads + (most + gx - 1) / gx, (rows + LQ_ROWS - 1) / LQ_ROWS);
     const int nb = rows <= 8 ? 1 : (rows <= 16 ? 2 : 4);
     const size_t x = (size_t)nb * 8 * (((a->dim + 63) & ~63) + 8) * 2 + (size_t)nb * 8 * (LQ_COLS + 8) * 2, rot = (size_t)a->rot_dim * 4;
     const size_t smem = x > rot ? x : rot;
@@ -341,8 +369,12 @@ extern "C" int cmlb200_latent_gather(const cmlb200_latent* a, const int (*keys)[
         list.k[i] = make_int4(keys[i][0], keys[i][1], keys[i][2], keys[i][3]);
         if (keys[i][2] > most) most = keys[i][2];
     }
-    CMLB_CUDA(launch_chain(latent_gather_kernel, dim3((most + a->block_size - 1) / a->block_size, n), dim3(256), 0, 1, as_stream(stream), *a, list,
-                           (__nv_bfloat16*)d_c_bf16, (__half*)s->k_pool, s->dim_ld, const_cast<int*>(s->block_table), s->table_ld));
+    const dim3 grid((most + a->block_size - 1) / a->block_size, n, a->heads < 8 ? a->heads : 8);
+    const bool vec = a->rank % 8 == 0 && a->rot_dim % 8 == 0 && a->dim % 8 == 0 && s->dim_ld % 8 == 0 && (((uintptr_t)d_c_bf16 | (uintptr_t)s->k_pool | (uintptr_t)a->pool) & 15) == 0;
+#define LG_LAUNCH(V) CMLB_CUDA(launch_chain(latent_gather_kernel<V>, grid, dim3(256), 0, 1, as_stream(stream), *a, list, (__nv_bfloat16*)d_c_bf16, (__half*)s->k_pool, s->dim_ld, const_cast<int*>(s->block_table), s->table_ld))
+    if (vec) LG_LAUNCH(true);
+    else LG_LAUNCH(false);
+#undef LG_LAUNCH
     return CMLB200_OK;
 }
 

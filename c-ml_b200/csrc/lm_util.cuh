@@ -102,6 +102,17 @@ __device__ __forceinline__ float glu_act(int act, float g, float u, float limit 
     return (act == CMLB200_ACT_GELU_TANH ? gelu_tanh(g) : silu(g)) * u;
 }
 
+// The same for results that are rounded to bf16: hardware exponential and reciprocal without branches, so that
+// independent values overlap. The tanh form of gelu is z sigmoid(2 sqrt(2/pi) (z + 0.044715 z^3)).
+__device__ __forceinline__ float sigmoid_fast(float z) { return __fdividef(1.0f, 1.0f + __expf(-z)); }
+__device__ __forceinline__ float glu_act_fast(int act, float g, float u, float limit = 0.f) {
+    const bool clamped = act == CMLB200_ACT_CLAMPED;
+    g = clamped ? fminf(g, limit) : g;
+    u = clamped ? fminf(fmaxf(u, -limit), limit) + 1.0f : u;
+    const float gelu = 1.5957691216057308f * (g + 0.044715f * g * g * g);
+    return g * sigmoid_fast(clamped ? 1.702f * g : (act == CMLB200_ACT_GELU_TANH ? gelu : g)) * u;
+}
+
 // Pieces of the mma.sync kernels.
 constexpr float kLog2e = 1.4426950408889634f;
 __device__ __forceinline__ uint32_t smem_addr(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }

@@ -17,23 +17,20 @@ __device__ __forceinline__ void route_row(const cmlb200_moe& m, const float* __r
     sum = lane_sum(sum);
     for (int k = 0; k < m.top; k++) {
         float best = -INFINITY;
-        int at = 0x7fffffff;
-        for (int e = lane; e < m.experts; e += 32)
-            if (z[e] > best || at == 0x7fffffff) { best = z[e]; at = e; }
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) {
-            const float v = __shfl_xor_sync(0xffffffffu, best, o);
-            const int i = __shfl_xor_sync(0xffffffffu, at, o);
-            if (v > best || (v == best && i < at)) { best = v; at = i; }
+        int at = -1;
+        for (int e = lane; e < m.experts; e += 32) {
+            const float v = z[e];
+            if (v > best) { best = v; at = e; }
         }
-        at = min(at, m.experts - 1);
-        __syncwarp();
-        if (lane == (at & 31)) {
-            m.ids[r * m.top + k] = at;
-            m.weight[r * m.top + k] = expf(best - mx) / sum;
-            z[at] = -INFINITY;
+        // order-preserving bits; 0: nothing left on this lane
+        const unsigned b = __float_as_uint(best), key = at < 0 ? 0u : ((b & 0x80000000u) ? ~b : b | 0x80000000u);
+        const unsigned top = __reduce_max_sync(0xffffffffu, key);
+        const int win = (int)min(__reduce_min_sync(0xffffffffu, key == top && at >= 0 ? (unsigned)at : 0xffffffffu), (unsigned)m.experts - 1u);
+        if (lane == (win & 31)) {
+            m.ids[r * m.top + k] = win;
+            m.weight[r * m.top + k] = expf(z[win] - mx) / sum;
+            z[win] = -INFINITY;
         }
-        __syncwarp();
     }
 }
 
@@ -46,7 +43,7 @@ route_rows_kernel(const cmlb200_moe m, const float* __restrict__ logits, int ld,
     if (r < rows) route_row(m, logits + (size_t)r * ld, r, z + warp * m.experts);
 }
 
-// One CTA. logits given (up to 32 rows): routes the rows first. Then counts, first positions (multiples of `align`), the
+// One CTA, with a warp per row where it routes. logits given (up to 32 rows): routes the rows first. Then counts, first positions (multiples of `align`), the
 // lists of chosen experts and of row tiles, and a position for every pair.
 __global__ void __launch_bounds__(PLAN_THREADS)
 plan_kernel(const cmlb200_moe m, const float* __restrict__ logits, int ld, int rows, int align) {
@@ -59,9 +56,9 @@ plan_kernel(const cmlb200_moe m, const float* __restrict__ logits, int ld, int r
         if (warp < rows) route_row(m, logits + (size_t)warp * ld, warp, z + warp * m.experts);
         __syncthreads();                                                // also orders the choices' global writes for this block
     }
-    for (int e = threadIdx.x; e < m.experts; e += PLAN_THREADS) count[e] = 0;
+    for (int e = threadIdx.x; e < m.experts; e += blockDim.x) count[e] = 0;
     __syncthreads();
-    for (int p = threadIdx.x; p < pairs; p += PLAN_THREADS) atomicAdd(&count[m.ids[p]], 1);
+    for (int p = threadIdx.x; p < pairs; p += blockDim.x) atomicAdd(&count[m.ids[p]], 1);
     __syncthreads();
     if (warp == 0) {
         int pos = 0, act = 0, til = 0;                                  // positions, chosen experts, tiles so far
@@ -90,7 +87,7 @@ plan_kernel(const cmlb200_moe m, const float* __restrict__ logits, int ld, int r
         if (lane == 0) { *m.num_active = act; *m.num_tiles = til; }
     }
     __syncthreads();
-    for (int p = threadIdx.x; p < pairs; p += PLAN_THREADS) {
+    for (int p = threadIdx.x; p < pairs; p += blockDim.x) {
         const int e = m.ids[p], at = atomicAdd(&count[e], 1);
         m.pos[p] = at;
         m.src[at] = p / m.top;
@@ -144,7 +141,7 @@ extern "C" int cmlb200_moe_route(const cmlb200_moe* m, const float* d_logits, in
     if (!fused) CMLB_CUDA(launch_chain(route_rows_kernel, dim3((rows + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(ROUTE_WARPS * 32), ROUTE_WARPS * row, 1, st, *m, d_logits, ld, rows));
     const size_t smem = fused ? (size_t)rows * row : row;
     CMLB_CUDA(cmlb_ensure_smem(plan_kernel, smem, attr));
-    CMLB_CUDA(launch_chain(plan_kernel, dim3(1), dim3(PLAN_THREADS), smem, 1, st, *m, fused ? d_logits : (const float*)nullptr, ld, rows, align));
+    CMLB_CUDA(launch_chain(plan_kernel, dim3(1), dim3(rows <= 8 ? PLAN_THREADS / 4 : PLAN_THREADS), smem, 1, st, *m, fused ? d_logits : (const float*)nullptr, ld, rows, align));
     return CMLB200_OK;
 }
 

@@ -241,7 +241,7 @@ static int round_keys(int keys) {
 static int upload_rows(CMLLanguageModel* lm, const CMLLMEntry* entries, int n, int rows, CMLLMBatch* b, const int** d_want) {
     const int stride = rows <= SMALL_ROWS ? SMALL_ROWS : (lm->opt.max_step_rows + 3) & ~3;
     int *tok = lm->h_meta, *pos = tok + stride, *slot = pos + stride, *want = slot + stride, *tiles = want + stride;
-    int one = 0, one_keys = 0, w = 0, t = 0, short_rows = 0, short_tiles = 0, portions = 0;
+    int one = 0, one_keys = 0, w = 0, t = 0, short_rows = 0, short_tiles = 0, short_keys = 0, portions = 0;
     for (int i = 0; i < n; i++) {
         const int k = entries[i].num_tokens;
         one += k == 1;
@@ -264,6 +264,7 @@ static int upload_rows(CMLLanguageModel* lm, const CMLLMEntry* entries, int n, i
         }
         for (int k = 0; k < e->num_want; k++) want[w++] = r0 + e->want[k];
         if (len == 1) { if (first > one_keys) one_keys = first; continue; }
+        if (len <= TILE_ROWS && first + len > short_keys) short_keys = first + len;
         if (len > TILE_ROWS) { CMLLMPortion p = {r0, len, e->seq, first, t}; lm->portions[portions++] = p; }
         for (int k = 0; k < len; k += TILE_ROWS, ++*tile) {
             tiles[4 * *tile] = r0 + k;
@@ -279,6 +280,7 @@ static int upload_rows(CMLLanguageModel* lm, const CMLLMEntry* entries, int n, i
     b->tiles = t;
     b->short_rows = short_rows;
     b->short_tiles = short_tiles;
+    b->short_keys = short_keys;
     b->portions = lm->portions;
     b->num_portions = portions;
     b->max_keys = round_keys(one_keys);

@@ -17,7 +17,7 @@ typedef struct CMLLMPortion {
  * a tile each), then the longer ones. */
 typedef struct CMLLMBatch {
     int rows, one_rows, tiles;
-    int short_rows, short_tiles;
+    int short_rows, short_tiles, short_keys;         /* short_keys: most keys of such a tile, its own included */
     const CMLLMPortion* portions;   /* host: the longer ones */
     int num_portions;
     int max_keys;                   /* no single-token row has more cached keys than this */

@@ -683,14 +683,14 @@ static int feed_forward(const Layered* m, const Layer* l, const LayerWeights* w,
 }
 
 /* Rows first .. first + rows - 1 against the latents themselves: queries through Wuk^T, weighted latents through Wuv.
- * one: that many single tokens, then `tiles` tiles from the batch's tile `tile` on. */
+ * one: that many single tokens, then `tiles` tiles from the batch's tile `tile` on, with up to tile_keys keys. */
 static int attend_latents(const Layered* m, const cmlb200_latent* a, const Layer* l, const LayerWeights* w, const CMLLMBatch* b, int first, int rows, int one,
-                          int tile, int tiles, void* st) {
+                          int tile, int tiles, int tile_keys, void* st) {
     const float* proj = m->qkvg + (size_t)first * (size_t)m->ld_qkvg;
     uint16_t *q = (uint16_t*)m->q, *o = (uint16_t*)m->o;
     DEV(cmlb200_latent_query(a, (const uint16_t*)w->wukt, proj, m->ld_qkvg, b->d_pos + first, b->d_slot + first, rows, q, st));
     if (one) DEV(cmlb200_attention_latent(a, q, b->d_pos + first, b->d_slot + first, one, b->max_keys, NULL, 0, o, st));
-    if (tiles) DEV(cmlb200_attention_latent(a, q, NULL, NULL, first, 0, b->d_tiles + 4 * tile, tiles, o, st));
+    if (tiles) DEV(cmlb200_attention_latent(a, q, NULL, NULL, first, tile_keys, b->d_tiles + 4 * tile, tiles, o, st));
     DEV(cmlb200_latent_output(a, value_rows(l, w), o, proj, m->ld_qkvg, rows, (uint16_t*)m->att + (size_t)first * (size_t)m->ld_att, m->ld_att, st));
     return 0;
 }
@@ -743,7 +743,7 @@ static int attend_expanded(const Layered* m, const cmlb200_latent* a, const Laye
         const int at_once = m->q_rows / 64 * 64;
         for (int r = 0; r < p0->rows; r += at_once) {
             const int k = p0->rows - r < at_once ? p0->rows - r : at_once;
-            if (attend_latents(m, a, l, w, b, p0->row + r, k, 0, p0->tile + r / 64, (k + 63) / 64, st)) return -1;
+            if (attend_latents(m, a, l, w, b, p0->row + r, k, 0, p0->tile + r / 64, (k + 63) / 64, p0->pos + p0->rows, st)) return -1;
         }
         i++;
     }
@@ -780,7 +780,7 @@ static int attend_latent(const Layered* m, const Layer* l, const LayerWeights* w
         return 0;
     }
     const int near = b->one_rows + b->short_rows;
-    if (near && attend_latents(m, &a, l, w, b, 0, near, b->one_rows, 0, b->short_tiles, st)) return -1;
+    if (near && attend_latents(m, &a, l, w, b, 0, near, b->one_rows, 0, b->short_tiles, b->short_keys, st)) return -1;
     return b->num_portions ? attend_expanded(m, &a, l, w, b, st) : 0;
 }
 

@@ -520,7 +520,8 @@ int cmlb200_latent_append(const cmlb200_latent* a, float* d_proj, int ld, const 
 int cmlb200_latent_query(const cmlb200_latent* a, const uint16_t* d_wukt, const float* d_proj, int ld, const int* d_row_pos, const int* d_row_slot,
                          int rows, uint16_t* d_q_f16, void* stream);
 /* Weighted latents bf16 [rows][heads][ld_rank] of such query rows. d_tiles NULL: row r is one token (position and slot
- * from the row arrays); otherwise tiles as in cmlb200_attention_tiles, and `rows` is the row that d_q_f16 begins with. */
+ * from the row arrays); otherwise tiles as in cmlb200_attention_tiles, and `rows` is the row that d_q_f16 begins
+ * with. max_keys bounds the cached keys in front of any row or tile (it picks the launch shape). */
 int cmlb200_attention_latent(const cmlb200_latent* a, const uint16_t* d_q_f16, const int* d_row_pos, const int* d_row_slot, int rows, int max_keys,
                              const int* d_tiles, int tiles, uint16_t* d_o_bf16, void* stream);
 /* out[row][head * vdim + v] = Wuv o, times the sigmoid of the gate. Wuv per head: [vdim rounded up to 16][ld_rank]. */

@@ -136,7 +136,7 @@ class LatentLayer:
                         pkg.check(L.cmlb200_attention_latent(a, P(q), P(dp), P(ds), one, keys, None, 0, P(o), None))
                     if tiles[0]:
                         t = up(tiles[0], self.dev, np.int32)
-                        pkg.check(L.cmlb200_attention_latent(a, P(q), None, None, 0, 0, P(t), len(tiles[0]), P(o), None))
+                        pkg.check(L.cmlb200_attention_latent(a, P(q), None, None, 0, max(x[3] + x[1] for x in tiles[0]), P(t), len(tiles[0]), P(o), None))
                     pkg.check(L.cmlb200_latent_output(a, P(self.wuv), P(o), P(d), ld, near, P(out), old, None))
                 if long:
                     pkg.check(L.cmlb200_latent_append(a, P(d, near * ld * 4), ld, P(dp, near * 4), P(ds, near * 4), n - near, None))
