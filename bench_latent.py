@@ -76,7 +76,7 @@ def latent(pkg, torch, H, B, ctx, rows_of_table=None, D=128, P=64, V=128, R=512,
     ld, q = (R + P + 15) // 16 * 16, H * (D + P)
     keep["pool"] = torch.randn(B * per * 16, ld, device=dev).half()
     a = pkg.Latent(H, D, P, V, R, ld, (R + 63) // 64 * 64, (D + P) ** -0.5, 0, keep["norm"].data_ptr(), 1e-5, keep["freq"].data_ptr(), 1.0, q, -1, pkg.DT_F16,
-                   keep["pool"].data_ptr(), 16, keep["table"].data_ptr(), per)
+                   keep["pool"].data_ptr(), 16, keep["table"].data_ptr(), per, B * per)
     return a, keep, q + R + P
 
 
@@ -123,7 +123,7 @@ def attention(pkg, torch, T, add):
                 ls = [latent(pkg, torch, H, B, ctx) for _ in range(n)]
                 q, o = torch.randn(B, H, ls[0][0].ld, device=dev).half(), torch.zeros(B, H, R, device=dev).bfloat16()
                 pos, slot = torch.full((B,), ctx, device=dev, dtype=torch.int32), torch.arange(B, device=dev, dtype=torch.int32)
-                calls = [lambda s, a=l[0]: ck(lib.cmlb200_attention_latent(a, q.data_ptr(), pos.data_ptr(), slot.data_ptr(), B, ctx, None, 0, o.data_ptr(), s)) for l in ls]
+                calls = [lambda s, a=l[0]: ck(lib.cmlb200_attention_latent(a, q.data_ptr(), B, pos.data_ptr(), slot.data_ptr(), B, ctx, None, 0, o.data_ptr(), s)) for l in ls]
                 add("attention_latent", f"H={H} B={B} ctx={ctx}", T.us(calls, 8), 2.0 * B * ctx * (R + P) + 2.0 * B * H * (2 * R + P), 2.0 * B * H * ctx * (2 * R + P))
                 del ls
                 torch.cuda.empty_cache()
@@ -182,7 +182,7 @@ def attention(pkg, torch, T, add):
             tile = i32([0, rows, 0, ctx])
             pairs = rows * ctx + rows * (rows + 1) / 2
             add("attention_latent (portion)", f"H={H} rows={rows} ctx={ctx}",
-                T.us([lambda s: ck(lib.cmlb200_attention_latent(a, q.data_ptr(), None, None, 0, ctx + rows, tile.data_ptr(), 1, o.data_ptr(), s))], 10), 2.0 * ctx * (R + P), 2.0 * pairs * H * (2 * R + P))
+                T.us([lambda s: ck(lib.cmlb200_attention_latent(a, q.data_ptr(), rows, None, None, 0, ctx + rows, tile.data_ptr(), 1, o.data_ptr(), s))], 10), 2.0 * ctx * (R + P), 2.0 * pairs * H * (2 * R + P))
             per, kp = (ctx + rows) // 16 + 1, []
             tab = torch.arange(per, device=dev, dtype=torch.int32).view(1, -1).contiguous()
             kk, vv = torch.randn(per * 16, H, D, device=dev).half(), torch.randn(per * 16, H, D, device=dev).half()

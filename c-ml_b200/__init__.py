@@ -451,7 +451,7 @@ class Latent(C.Structure):
     """cmlb200_latent."""
     _fields_ = [("heads", ci), ("dim", ci), ("rot_dim", ci), ("vdim", ci), ("rank", ci), ("ld", ci), ("ld_rank", ci), ("scale", C.c_float), ("window", ci),
                 ("c_norm", vp), ("eps", C.c_float), ("freq", vp), ("rot_mul", C.c_float), ("kv_col", ci), ("gate_col", ci), ("cache_dtype", ci), ("pool", vp),
-                ("block_size", ci), ("block_table", vp), ("table_ld", ci)]
+                ("block_size", ci), ("block_table", vp), ("table_ld", ci), ("pool_blocks", ci)]
 
 
 class Moe(C.Structure):
@@ -486,7 +486,8 @@ _sig("cmlb200_poly_norm", ci, vp, ci, ci, ci, vp, _cf, vp, ci, ci, vp)
 _sig("cmlb200_latent_append", ci, _LAT, vp, ci, vp, vp, ci, vp)
 for _n in ("cmlb200_latent_query", "cmlb200_latent_query_f32"):
     _sig(_n, ci, _LAT, vp, vp, ci, vp, vp, ci, vp, vp)
-_sig("cmlb200_attention_latent", ci, _LAT, vp, vp, vp, ci, ci, vp, ci, vp, vp)
+_sig("cmlb200_attention_latent", ci, _LAT, vp, ci, vp, vp, ci, ci, vp, ci, vp, vp)
+_sig("cmlb200_attention_latent_status", ci, C.POINTER(ci), ci)
 for _n in ("cmlb200_latent_output", "cmlb200_latent_output_f32"):
     _sig(_n, ci, _LAT, vp, vp, vp, ci, ci, vp, ci, vp)
 _sig("cmlb200_latent_gather", ci, _LAT, vp, ci, vp, C.POINTER(Attn), vp)

@@ -1,4 +1,5 @@
-// Attention over latents: every head of a row attends the same keys, one vector [latent | rotated part] per token of a
+// Attention over latents, the mma.sync form for what attention_latent_tc.cu does not take, and the entry point of both:
+// every head of a row attends the same keys, one vector [latent | rotated part] per token of a
 // paged cache, and the weighted sum of the latents is what a head returns. Queries come transformed
 // (cmlb200_latent_query), in units of log2. One kernel serves decoded tokens and short prompt portions:
 // the (token, head) pairs of a portion are the rows of the matrix products, 16, 32 or 64 to a CTA.
@@ -278,17 +279,24 @@ attention_latent_kernel(const cmlb200_latent a, const __half* __restrict__ q, co
 
 }  // namespace
 
-extern "C" int cmlb200_attention_latent(const cmlb200_latent* a, const uint16_t* d_q_f16, const int* d_row_pos, const int* d_row_slot, int rows, int max_keys,
-                                        const int* d_tiles, int tiles, uint16_t* d_o_bf16, void* stream) {
+extern "C" int cmlb200_attention_latent_tc_fits_(const cmlb200_latent* a);
+extern "C" int cmlb200_attention_latent_tc_(const cmlb200_latent* a, const uint16_t* q, long q_rows, const int* row_pos, const int* row_slot, int max_keys,
+                                            const int* tiles, int items, int most, int first, uint16_t* o, cudaStream_t st);
+
+extern "C" int cmlb200_attention_latent(const cmlb200_latent* a, const uint16_t* d_q_f16, int q_rows, const int* d_row_pos, const int* d_row_slot, int rows,
+                                        int max_keys, const int* d_tiles, int tiles, uint16_t* d_o_bf16, void* stream) {
     static const char* who = "cmlb200_attention_latent";
-    CMLB_REQUIRE(a && d_q_f16 && d_o_bf16 && (d_tiles ? tiles > 0 && rows >= 0 : d_row_pos && d_row_slot && rows > 0) && max_keys >= 0, "%s: bad argument", who);
+    CMLB_REQUIRE(a && d_q_f16 && d_o_bf16 && (d_tiles ? tiles > 0 && rows >= 0 : d_row_pos && d_row_slot && rows > 0 && q_rows >= rows) && q_rows > 0 && max_keys >= 0, "%s: bad argument", who);
     CMLB_REQUIRE(a->heads > 0 && a->rank > 0 && a->ld >= a->rank && a->ld % 16 == 0 && a->ld_rank >= a->rank && a->ld_rank % 64 == 0 && a->rank <= 512,
                  "%s: rank %d (up to 512), strides %d / %d", who, a->rank, a->ld, a->ld_rank);
     CMLB_REQUIRE(a->pool && a->block_table && a->table_ld > 0 && a->cache_dtype == CMLB200_DT_F16, "%s: fp16 cache", who);
     CMLB_REQUIRE(a->block_size >= 16 && (a->block_size & (a->block_size - 1)) == 0, "%s: block size %d must be a power of two >= 16", who, a->block_size);
-    CMLB_REQUIRE((((uintptr_t)d_q_f16 | (uintptr_t)a->pool | (uintptr_t)d_tiles) & 15) == 0 && ((uintptr_t)d_o_bf16 & 3) == 0, "%s: alignment", who);
+    CMLB_REQUIRE((((uintptr_t)d_q_f16 | (uintptr_t)a->pool | (uintptr_t)d_tiles) & 15) == 0 && ((uintptr_t)d_o_bf16 & 15) == 0, "%s: alignment", who);
     const int items = d_tiles ? tiles : rows, most = d_tiles ? 64 * a->heads : a->heads, sms = cmlb_num_sms();
     CMLB_REQUIRE(items <= 65535, "%s: %d rows", who, items);
+    if (cmlb200_attention_latent_tc_fits_(a))
+        return cmlb200_attention_latent_tc_(a, d_q_f16, (long)q_rows * a->heads, d_row_pos, d_row_slot, max_keys, d_tiles, items, most, d_tiles ? rows : 0, d_o_bf16,
+                                            as_stream(stream));
     const int keys = (a->window > 0 && a->window < max_keys + 1) ? a->window : max_keys + 1, rank16 = (a->rank + 15) & ~15;
     auto blocks = [&](int m) { return (long)items * ((most + 16 * m - 1) / (16 * m)); };
     // rows per CTA and parts of the keys, by an estimate of the time in microseconds: wide tiles do more per key, narrow

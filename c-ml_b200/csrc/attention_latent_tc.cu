@@ -1,0 +1,362 @@
+// Attention over latents on the 5th-generation tensor cores: the same operation as attention_latent.cu, for latents
+// whose operands fit shared memory.
+//
+// A CTA holds up to 32 or 64 (token, head) rows of queries and walks key tiles of 64 tokens; a cluster of up to 8 CTAs
+// splits the tiles and merges through distributed shared memory. Latents of more than 256 values give two CTAs a half
+// of the output columns each (both compute the scores). Roles:
+//   warp 0     TMA: the queries once, then key tiles, 16 tokens to a copy (the block table says where), two stages;
+//              64-column slabs, 128-byte swizzle
+//   warp 1     owns tensor memory; one lane issues tcgen05.mma: S = Q K^T into two alternating accumulators, and
+//              O += P V, where V is the same tile read with its columns as the contiguous dimension
+//   warps 2-5  softmax, a thread per row (those whose quarter of tensor memory holds rows): S from tensor memory, mask,
+//              exponentials, P as fp16 into shared memory. The reference of the exponentials moves, and O is scaled,
+//              only when a row's maximum has grown by more than 8 (a factor of 256); sums are fp32
+// The scores of tile i + 1 are computed while the softmax of tile i runs. An MMA is 128 rows high: those past the CTA's
+// read whatever follows in shared memory and are never looked at. Keys past the sequence's last are zeroed in the tile,
+// so that nothing other requests left in a block can reach the sums.
+// Every wait is bounded; one that gives up leaves a code in a status word in host memory, and the CTA still drains its
+// copies, meets its cluster and frees its tensor memory.
+#include "tcgen05_util.cuh"
+
+namespace {
+
+constexpr int TC_THREADS = 192, TC_KEYS = 64, TC_SPLITS = 8, TC_SLAB = TC_KEYS * 128, TC_S_COL = 256, TC_TMEM = 512;
+
+__host__ __device__ inline size_t tc_operands(int mr, int slabs) { return (size_t)slabs * mr * 128 + (size_t)mr * 128 + 2 * (size_t)slabs * TC_SLAB; }
+__host__ __device__ inline size_t tc_smem(int mr, int slabs) { return tc_operands(mr, slabs) + 128 + 2 * 4 * (size_t)mr + 1024; }
+
+// grid = (splits, row blocks * halves, items), clusters of `splits` CTAs along x.
+template <int MR>
+__global__ void __launch_bounds__(TC_THREADS, 1)
+attention_latent_tc_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_constant__ CUtensorMap kmap, const cmlb200_latent a,
+                           const int* __restrict__ row_pos, const int* __restrict__ row_slot, const int4* __restrict__ tiles, int first,
+                           __nv_bfloat16* __restrict__ out, int halves, int* status) {
+    extern __shared__ uint8_t smem_raw[];
+    uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
+    const int slabs = (a.ld + 63) / 64, stage_bytes = slabs * TC_SLAB;
+    const uint32_t qs = smem_addr(smem), ps = qs + slabs * MR * 128, ks = ps + MR * 128;
+    uint8_t* tail = smem + tc_operands(MR, slabs);
+    const uint32_t bars = smem_addr(tail);
+    const uint32_t q_full = bars, p_full = bars + 8, pv_done = bars + 16;
+    auto k_full = [&](int s) { return bars + 24 + 8 * s; };
+    auto k_empty = [&](int s) { return bars + 40 + 8 * s; };
+    auto s_full = [&](int s) { return bars + 56 + 8 * s; };
+    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(tail + 80);
+    volatile int* abort_flag = reinterpret_cast<volatile int*>(tail + 88);
+    float* c_m = reinterpret_cast<float*>(tail + 128);
+    float* c_l = c_m + MR;
+    float* Os = reinterpret_cast<float*>(smem);                         // [MR][columns + 4], over the operands once they are done
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+
+    if (threadIdx.x == 0) {
+        mbar_init(q_full, 1);
+        mbar_init(p_full, MR / 32);
+        mbar_init(pv_done, 1);
+        for (int s = 0; s < 2; s++) { mbar_init(k_full(s), 1); mbar_init(k_empty(s), 1); mbar_init(s_full(s), 1); }
+        *abort_flag = 0;
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    if (warp == 1) {
+        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_addr(tmem_slot)), "r"((uint32_t)TC_TMEM) : "memory");
+        asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
+    }
+    tmem_fence_before();
+    __syncthreads();
+    tmem_fence_after();
+    const uint32_t tmem = *tmem_slot;
+    // a launch that allocates tensor memory too may start from here on: every CTA of this one has its own
+    dep_wait();
+    dep_trigger();
+
+    int4 tl = tiles ? tiles[blockIdx.z] : make_int4((int)blockIdx.z, 1, row_slot[blockIdx.z], row_pos[blockIdx.z]);
+    tl.x -= first;
+    const int total = tl.y * a.heads, half = blockIdx.y % halves, m0 = blockIdx.y / halves * MR;
+    const bool live = m0 < total;                                       // the same for a whole cluster
+    const int splits = gridDim.x, rank = blockIdx.x, shift = __ffs(a.block_size) - 1;
+    const int* table = a.block_table + (size_t)tl.z * a.table_ld;
+    const int window = a.window > 0 ? a.window : 0x7fffffff;
+    const int p_first = tl.w + m0 / a.heads, p_last = tl.w + (min(m0 + MR, total) - 1) / a.heads;
+    const int k_lo = (window > p_first ? 0 : p_first - window + 1) & ~15;
+    const int ntiles = live ? (p_last - k_lo) / TC_KEYS + 1 : 0;
+    const int n = rank < ntiles ? (ntiles - rank + splits - 1) / splits : 0;          // tiles of this CTA: rank, rank + splits, ..
+    const int nv = (a.rank + 63) / 64, per = (nv + halves - 1) / halves, v0 = half * per, cols = min(per, nv - v0) * 64;
+    const int row0 = tl.x * a.heads + m0;
+
+    if (warp == 0) {
+        bool ok = true;
+        int i = 0;
+        if (n > 0) {
+            if (lane == 0) mbar_expect_tx(q_full, (uint32_t)(slabs * MR * 128));
+            __syncwarp();
+            if (lane < slabs) tma_load_2d(qs + lane * MR * 128, &qmap, lane * 64, row0, q_full);
+        }
+        for (; i < n; i++) {
+            const int st = i & 1, kt = k_lo + (rank + i * splits) * TC_KEYS;
+            ok = __all_sync(0xffffffffu, mbar_wait(k_empty(st), ((i >> 1) & 1) ^ 1, abort_flag, 1, status));
+            if (!ok) break;
+            if (lane == 0) mbar_expect_tx(k_full(st), (uint32_t)stage_bytes);
+            __syncwarp();
+            for (int j = lane; j < 4 * slabs; j += 32) {
+                const int g = j & 3, s = j >> 2, key = min(kt + 16 * g, p_last & ~15);      // past the end: the last block again
+                const int slot = (table[key >> shift] << shift) + (key & (a.block_size - 1));
+                tma_load_2d(ks + st * stage_bytes + s * TC_SLAB + g * 2048, &kmap, s * 64, slot, k_full(st));
+            }
+        }
+        if (!ok && n > 0) {                                             // no copy outlives the CTA
+            mbar_wait(q_full, 0, abort_flag, 2, status);
+            for (int j = max(0, i - 2); j < i; j++) mbar_wait(k_full(j & 1), (j >> 1) & 1, abort_flag, 2, status);
+        }
+    } else if (warp == 1) {
+        if (lane == 0 && n > 0) {
+            // fp16 operands, fp32 accumulators, 128 rows; the second one takes V with its columns contiguous
+            const uint32_t is = (1u << 4) | ((uint32_t)(TC_KEYS >> 3) << 17) | ((uint32_t)(128 >> 4) << 24);
+            const uint32_t io = (1u << 4) | (1u << 16) | ((uint32_t)(cols >> 3) << 17) | ((uint32_t)(128 >> 4) << 24);
+            const int steps = a.ld / 16;
+            bool ok = mbar_wait(q_full, 0, abort_flag, 3, status);
+            auto scores = [&](int i) {
+                if (!mbar_wait(k_full(i & 1), (i >> 1) & 1, abort_flag, 4, status)) return false;
+                tmem_fence_after();
+                const uint32_t kst = ks + (i & 1) * stage_bytes;
+                for (int k = 0; k < steps; k++)
+                    umma(tmem + TC_S_COL + (i & 1) * TC_KEYS, make_desc(qs + (k >> 2) * MR * 128) + (uint64_t)(2 * (k & 3)),
+                         make_desc(kst + (k >> 2) * TC_SLAB) + (uint64_t)(2 * (k & 3)), is, k ? 1u : 0u);
+                umma_commit(s_full(i & 1));
+                return true;
+            };
+            ok = ok && scores(0);
+            for (int i = 0; i < n && ok; i++) {
+                if (i + 1 < n) ok = scores(i + 1);
+                ok = ok && mbar_wait(p_full, i & 1, abort_flag, 5, status);
+                if (!ok) break;
+                tmem_fence_after();
+                const uint32_t vst = ks + (i & 1) * stage_bytes + v0 * TC_SLAB;
+#pragma unroll
+                for (int k = 0; k < TC_KEYS / 16; k++)
+                    umma(tmem, make_desc(ps) + (uint64_t)(2 * k), make_desc_mn(vst + k * 2048, TC_SLAB), io, (i | k) ? 1u : 0u);
+                umma_commit(k_empty(i & 1));
+                umma_commit(pv_done);
+            }
+        }
+        __syncwarp();
+    } else if ((warp & 3) * 32 < MR && live) {
+        const int q = warp & 3, r = q * 32 + lane;                      // the quarter of tensor memory's lanes this warp may read
+        const uint32_t lanes = tmem + ((uint32_t)(q * 32) << 16);
+        const int p = m0 + r < total ? tl.w + (m0 + r) / a.heads : -1;
+        float m = -INFINITY, l = 0.f;
+        bool ok = true;
+        for (int i = 0; i < n; i++) {
+            const int kt = k_lo + (rank + i * splits) * TC_KEYS;
+            ok = __all_sync(0xffffffffu, mbar_wait(s_full(i & 1), (i >> 1) & 1, abort_flag, 6, status));
+            if (!ok) break;
+            tmem_fence_after();
+            uint32_t v[2][32];
+            tmem_ld32(lanes + TC_S_COL + (i & 1) * TC_KEYS, v[0]);
+            tmem_ld32(lanes + TC_S_COL + (i & 1) * TC_KEYS + 32, v[1]);
+            if (kt + TC_KEYS - 1 > p_first || kt <= p_last - window) {
+#pragma unroll
+                for (int j = 0; j < TC_KEYS; j++) {
+                    const int d = p - kt - j;
+                    if (d < 0 || d >= window) v[j >> 5][j & 31] = 0xff800000u;
+                }
+            }
+            float mx = -INFINITY;
+#pragma unroll
+            for (int j = 0; j < TC_KEYS; j++) mx = fmaxf(mx, __uint_as_float(v[j >> 5][j & 31]));
+            float c = 1.f;
+            const bool scale = __any_sync(0xffffffffu, mx > m + 8.f);  // -inf + 8 is -inf: a row's first keys count
+            if (scale) {
+                const float nm = fmaxf(m, mx);
+                c = nm == -INFINITY ? 1.f : ex2(m - nm);
+                m = nm;
+                l *= c;
+            }
+            const float u = m == -INFINITY ? 0.f : m;
+            uint32_t pk[TC_KEYS / 2];
+            float l2 = 0.f;
+#pragma unroll
+            for (int j = 0; j < TC_KEYS / 2; j++) {
+                const float e0 = ex2(__uint_as_float(v[j >> 4][(2 * j) & 31]) - u), e1 = ex2(__uint_as_float(v[j >> 4][(2 * j + 1) & 31]) - u);
+                l += e0;
+                l2 += e1;
+                const __half2 h = __floats2half2_rn(e0, e1);
+                pk[j] = *reinterpret_cast<const uint32_t*>(&h);
+            }
+            l += l2;
+            if (i > 0) {                                                // P and O are the last product's until it is done
+                ok = __all_sync(0xffffffffu, mbar_wait(pv_done, (i - 1) & 1, abort_flag, 7, status));
+                if (!ok) break;
+                tmem_fence_after();
+                if (scale) {
+                    for (int c0 = 0; c0 < cols; c0 += 32) {
+                        uint32_t o[32];
+                        tmem_ld32(lanes + c0, o);
+#pragma unroll
+                        for (int j = 0; j < 32; j++) o[j] = __float_as_uint(__uint_as_float(o[j]) * c);
+                        tmem_st32(lanes + c0, o);
+                    }
+                    tmem_st_wait();
+                }
+            }
+            uint8_t* prow = smem + (ps - qs) + r * 128;
+#pragma unroll
+            for (int j = 0; j < 8; j++) *reinterpret_cast<uint4*>(prow + ((j ^ (r & 7)) << 4)) = make_uint4(pk[4 * j], pk[4 * j + 1], pk[4 * j + 2], pk[4 * j + 3]);
+            const int valid = p_last - kt + 1;                          // keys of this tile that exist
+            if (valid < TC_KEYS) {
+                uint8_t* vst = smem + (ks - qs) + (i & 1) * stage_bytes + v0 * TC_SLAB;
+                const int chunks = (TC_KEYS - valid) * 8;
+                for (int j = r; j < chunks * (cols / 64); j += MR)
+                    *reinterpret_cast<uint4*>(vst + j / chunks * TC_SLAB + valid * 128 + j % chunks * 16) = make_uint4(0u, 0u, 0u, 0u);
+            }
+            asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+            tmem_fence_before();
+            __syncwarp();
+            if (lane == 0) mbar_arrive(p_full);
+        }
+        if (ok && n > 0) ok = __all_sync(0xffffffffu, mbar_wait(pv_done, (n - 1) & 1, abort_flag, 8, status));
+        tmem_fence_after();
+        if (!ok) { m = -INFINITY; l = 0.f; }
+        c_m[r] = m;
+        c_l[r] = l;
+        const float inv = l > 0.f ? 1.0f / l : 0.f;
+        for (int c0 = 0; c0 < cols && n > 0; c0 += 32) {
+            uint32_t o[32];
+            tmem_ld32(lanes + c0, o);
+            if (splits > 1) {
+                float4* d = reinterpret_cast<float4*>(Os + r * (cols + 4) + c0);
+#pragma unroll
+                for (int j = 0; j < 8; j++)
+                    d[j] = make_float4(__uint_as_float(o[4 * j]), __uint_as_float(o[4 * j + 1]), __uint_as_float(o[4 * j + 2]), __uint_as_float(o[4 * j + 3]));
+            } else if (m0 + r < total) {
+                uint32_t w[16];
+#pragma unroll
+                for (int j = 0; j < 16; j++) {
+                    const int col = v0 * 64 + c0 + 2 * j;
+                    const __nv_bfloat162 h = __floats2bfloat162_rn(col < a.rank ? __uint_as_float(o[2 * j]) * inv : 0.f, col + 1 < a.rank ? __uint_as_float(o[2 * j + 1]) * inv : 0.f);
+                    w[j] = *reinterpret_cast<const uint32_t*>(&h);
+                }
+                uint4* d = reinterpret_cast<uint4*>(out + (size_t)(row0 + r) * a.ld_rank + v0 * 64 + c0);
+#pragma unroll
+                for (int j = 0; j < 4; j++) d[j] = make_uint4(w[4 * j], w[4 * j + 1], w[4 * j + 2], w[4 * j + 3]);
+            }
+        }
+        tmem_fence_before();
+    }
+    __syncwarp();
+    if (splits > 1 && live) {
+        asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
+        asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
+        const int rows = min(MR, total - m0), quads = cols / 4;
+        for (int i = rank * TC_THREADS + threadIdx.x; i < rows * quads; i += splits * TC_THREADS) {
+            const int r = i / quads, c = (i - r * quads) * 4;
+            float ms[TC_SPLITS], ls[TC_SPLITS];
+            float4 xs[TC_SPLITS];
+#pragma unroll
+            for (int s = 0; s < TC_SPLITS; s++) {
+                ms[s] = -INFINITY; ls[s] = 0.f; xs[s] = make_float4(0.f, 0.f, 0.f, 0.f);
+                if (s < splits) {
+                    uint32_t am, al, ax;
+                    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(am) : "r"(smem_addr(c_m + r)), "r"(s));
+                    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(al) : "r"(smem_addr(c_l + r)), "r"(s));
+                    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(ax) : "r"(smem_addr(Os + r * (cols + 4) + c)), "r"(s));
+                    asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(ms[s]) : "r"(am) : "memory");
+                    asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(ls[s]) : "r"(al) : "memory");
+                    asm volatile("ld.shared::cluster.v4.f32 {%0,%1,%2,%3}, [%4];" : "=f"(xs[s].x), "=f"(xs[s].y), "=f"(xs[s].z), "=f"(xs[s].w) : "r"(ax) : "memory");
+                }
+            }
+            float mx = ms[0], sum = 0.f;
+            float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+            for (int s = 1; s < TC_SPLITS; s++) mx = fmaxf(mx, ms[s]);
+#pragma unroll
+            for (int s = 0; s < TC_SPLITS; s++) {
+                if (ms[s] == -INFINITY) continue;                       // saw nothing: its values may be anything
+                const float f = exp2f(ms[s] - mx);
+                sum = fmaf(ls[s], f, sum);
+                x.x = fmaf(xs[s].x, f, x.x); x.y = fmaf(xs[s].y, f, x.y); x.z = fmaf(xs[s].z, f, x.z); x.w = fmaf(xs[s].w, f, x.w);
+            }
+            const float inv = sum > 0.f ? 1.0f / sum : 0.f;
+            const int col = v0 * 64 + c;
+            const __nv_bfloat162 lo = __floats2bfloat162_rn(col < a.rank ? x.x * inv : 0.f, col + 1 < a.rank ? x.y * inv : 0.f);
+            const __nv_bfloat162 hi = __floats2bfloat162_rn(col + 2 < a.rank ? x.z * inv : 0.f, col + 3 < a.rank ? x.w * inv : 0.f);
+            *reinterpret_cast<uint2*>(out + (size_t)(row0 + r) * a.ld_rank + col) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+        }
+        asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");  // nobody leaves while others read its shared memory
+        asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
+    }
+    tmem_fence_before();
+    __syncthreads();
+    if (warp == 1) {
+        tmem_fence_after();
+        asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"((uint32_t)TC_TMEM) : "memory");
+    }
+}
+
+int* g_status[kMaxDevices] = {};
+
+int status_word(int** word) {
+    int dev = 0;
+    CMLB_CUDA(cudaGetDevice(&dev));
+    CMLB_REQUIRE(dev >= 0 && dev < kMaxDevices, "device %d", dev);
+    if (!g_status[dev]) {
+        void* p = nullptr;
+        CMLB_CUDA(cudaHostAlloc(&p, sizeof(int), cudaHostAllocDefault));
+        *static_cast<int*>(p) = 0;
+        g_status[dev] = static_cast<int*>(p);
+    }
+    *word = g_status[dev];
+    return CMLB200_OK;
+}
+
+}  // namespace
+
+// 1: these sizes run here. Operands must fit, and the pool's extent must be known for its tensor map.
+extern "C" int cmlb200_attention_latent_tc_fits_(const cmlb200_latent* a) {
+    return a->pool_blocks > 0 && a->rank <= 512 && a->ld <= 8192 && tc_smem(64, (a->ld + 63) / 64) <= 227 * 1024;
+}
+
+extern "C" int cmlb200_attention_latent_tc_(const cmlb200_latent* a, const uint16_t* q, long q_rows, const int* row_pos, const int* row_slot, int max_keys,
+                                            const int* tiles, int items, int most, int first, uint16_t* o, cudaStream_t st) {
+    const int sms = cmlb_num_sms(), mr = most <= 32 ? 32 : 64, slabs = (a->ld + 63) / 64, halves = a->rank > 256 ? 2 : 1;
+    const int keys = (a->window > 0 && a->window < max_keys + 1) ? a->window : max_keys + 1;
+    const long blocks = (long)((most + mr - 1) / mr) * halves;
+    CMLB_REQUIRE(blocks <= 65535, "cmlb200_attention_latent: %d heads", a->heads);
+    int splits = 1;
+    double best = 0.0;
+    for (int s = 1; s <= TC_SPLITS && (s == 1 || (s - 1) * TC_KEYS < keys); s *= 2) {          // microseconds, by estimate
+        const long ctas = blocks * items * s, waves = (ctas + sms - 1) / sms, each = ((keys + TC_KEYS - 1) / TC_KEYS + s - 1) / s;
+        const double t = (double)waves * (3.0 + (double)each) + (s > 1 ? 1.5 : 0.0);
+        if (s == 1 || t < best) { splits = s; best = t; }
+    }
+    int* status;
+    int rc = status_word(&status);
+    if (rc) return rc;
+    CUtensorMap qmap, kmap;
+    rc = encode_map(&qmap, CU_TENSOR_MAP_DATA_TYPE_FLOAT16, q, q_rows, a->ld, a->ld, 64, mr);
+    if (!rc) rc = encode_map(&kmap, CU_TENSOR_MAP_DATA_TYPE_FLOAT16, a->pool, (long)a->pool_blocks * a->block_size, a->ld, a->ld, 64, 16);
+    if (rc) return rc;
+    // one CTA to an SM: each needs all of the SM's tensor memory, and a cluster's CTAs wait for one another
+    const size_t need = tc_smem(mr, slabs), smem = need > 118 * 1024 ? need : 118 * 1024;
+    const dim3 grid(splits, (unsigned)blocks, items);
+    static size_t attr[2][kMaxDevices] = {};
+#define TC_LAUNCH(MR, slot)                                                                                                      \
+    do {                                                                                                                         \
+        auto kern = attention_latent_tc_kernel<MR>;                                                                              \
+        CMLB_CUDA(cmlb_ensure_smem(kern, smem, attr[slot]));                                                                     \
+        CMLB_CUDA(launch_chain(kern, grid, dim3(TC_THREADS), smem, splits, st, qmap, kmap, *a, row_pos, row_slot, (const int4*)tiles, first, (__nv_bfloat16*)o, \
+                               halves, status));                                                                                 \
+    } while (0)
+    if (mr == 32) TC_LAUNCH(32, 0);
+    else TC_LAUNCH(64, 1);
+#undef TC_LAUNCH
+    return CMLB200_OK;
+}
+
+extern "C" int cmlb200_attention_latent_status(int* status, int reset) {
+    CMLB_REQUIRE(status, "cmlb200_attention_latent_status: NULL argument");
+    int* word;
+    const int rc = status_word(&word);
+    if (rc) return rc;
+    *status = *static_cast<volatile int*>(word);
+    if (reset) *static_cast<volatile int*>(word) = 0;
+    return CMLB200_OK;
+}

@@ -614,6 +614,7 @@ static int layered_make_pools(void* model, int blocks, int block_size, int slots
             cmlb200_latent* a = &l->lat;
             a->cache_dtype = m->f32 ? CMLB200_DT_F32 : CMLB200_DT_F16;
             a->block_size = block_size;
+            a->pool_blocks = blocks;
             a->c_norm = w->c_norm;
             a->eps = m->eps;
             if (l->kv_from != i) a->pool = m->layers[l->kv_from].lat.pool;
@@ -689,8 +690,8 @@ static int attend_latents(const Layered* m, const cmlb200_latent* a, const Layer
     const float* proj = m->qkvg + (size_t)first * (size_t)m->ld_qkvg;
     uint16_t *q = (uint16_t*)m->q, *o = (uint16_t*)m->o;
     DEV(cmlb200_latent_query(a, (const uint16_t*)w->wukt, proj, m->ld_qkvg, b->d_pos + first, b->d_slot + first, rows, q, st));
-    if (one) DEV(cmlb200_attention_latent(a, q, b->d_pos + first, b->d_slot + first, one, b->max_keys, NULL, 0, o, st));
-    if (tiles) DEV(cmlb200_attention_latent(a, q, NULL, NULL, first, tile_keys, b->d_tiles + 4 * tile, tiles, o, st));
+    if (one) DEV(cmlb200_attention_latent(a, q, rows, b->d_pos + first, b->d_slot + first, one, b->max_keys, NULL, 0, o, st));
+    if (tiles) DEV(cmlb200_attention_latent(a, q, rows, NULL, NULL, first, tile_keys, b->d_tiles + 4 * tile, tiles, o, st));
     DEV(cmlb200_latent_output(a, value_rows(l, w), o, proj, m->ld_qkvg, rows, (uint16_t*)m->att + (size_t)first * (size_t)m->ld_att, m->ld_att, st));
     return 0;
 }
@@ -842,7 +843,10 @@ static int layered_head(void* model, const int* d_rows, int n, float* d_logits, 
 static int layered_check(void* model, const CMLLMBatch* b) {
     const Layered* m = (const Layered*)model;
     int status = 0;
-    if (m->f32 || b->rows <= SKINNY_ROWS) return 0;
+    if (m->f32) return 0;
+    if (m->q) DEV(cmlb200_attention_latent_status(&status, 1));
+    if (status) return -1;
+    if (b->rows <= SKINNY_ROWS) return 0;
     DEV(cmlb200_gemm_dense_status(&status, 1));
     return status ? -1 : 0;
 }

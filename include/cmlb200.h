@@ -455,10 +455,11 @@ typedef struct cmlb200_latent {
     int kv_col;                 /* column of the rank + rot_dim latent projections; -1: another layer fills the cache */
     int gate_col;               /* column of heads * vdim gate logits; -1: none */
     int cache_dtype;            /* CMLB200_DT_F32 or CMLB200_DT_F16 */
-    void* pool;                 /* [blocks][block_size][ld] */
+    void* pool;                 /* [pool_blocks][block_size][ld] */
     int block_size;             /* a power of two >= 16 */
     const int* block_table;
     int table_ld;
+    int pool_blocks;            /* 0: not known, which leaves cmlb200_attention_latent to its mma.sync form */
 } cmlb200_latent;
 
 /* Where a step's (row, expert) pairs go: `top` pairs per row, ordered by expert, each expert's first position a
@@ -519,11 +520,13 @@ int cmlb200_poly_norm(const float* d_z, int ld, int rows, int ff, const float* d
 int cmlb200_latent_append(const cmlb200_latent* a, float* d_proj, int ld, const int* d_row_pos, const int* d_row_slot, int rows, void* stream);
 int cmlb200_latent_query(const cmlb200_latent* a, const uint16_t* d_wukt, const float* d_proj, int ld, const int* d_row_pos, const int* d_row_slot,
                          int rows, uint16_t* d_q_f16, void* stream);
-/* Weighted latents bf16 [rows][heads][ld_rank] of such query rows. d_tiles NULL: row r is one token (position and slot
+/* Weighted latents bf16 [q_rows][heads][ld_rank] of such query rows, on tcgen05 where the sizes fit. d_tiles NULL: row r is one token (position and slot
  * from the row arrays); otherwise tiles as in cmlb200_attention_tiles, and `rows` is the row that d_q_f16 begins
  * with. max_keys bounds the cached keys in front of any row or tile (it picks the launch shape). */
-int cmlb200_attention_latent(const cmlb200_latent* a, const uint16_t* d_q_f16, const int* d_row_pos, const int* d_row_slot, int rows, int max_keys,
-                             const int* d_tiles, int tiles, uint16_t* d_o_bf16, void* stream);
+int cmlb200_attention_latent(const cmlb200_latent* a, const uint16_t* d_q_f16, int q_rows, const int* d_row_pos, const int* d_row_slot, int rows,
+                             int max_keys, const int* d_tiles, int tiles, uint16_t* d_o_bf16, void* stream);
+/* Not 0: a bounded wait of that kernel expired (valid once the stream has drained). */
+int cmlb200_attention_latent_status(int* status, int reset);
 /* out[row][head * vdim + v] = Wuv o, times the sigmoid of the gate. Wuv per head: [vdim rounded up to 16][ld_rank]. */
 int cmlb200_latent_output(const cmlb200_latent* a, const uint16_t* d_wuv, const uint16_t* d_o_bf16, const float* d_proj, int ld, int rows,
                           uint16_t* d_out_bf16, int out_ld, void* stream);

@@ -33,6 +33,8 @@ class LatentLayer:
     """Random projections of `lengths` tokens per sequence for a mixer, a shuffled block table and a device pool."""
 
     def __init__(self, pkg, synth, dev, mixer, lengths, f32, gated=True, seed=0):
+        """f32: False (fp16 cache, tcgen05 where it fits), "mma" (fp16 cache, the mma.sync form) or True (32-bit)."""
+        self.mma, f32 = f32 == "mma", f32 is True
         r = RNG(seed)
         exact = lambda *shape: synth.bf16_round(r.standard_normal(shape))[1]
         self.pkg, self.synth, self.dev, self.m, self.f32, self.gated = pkg, synth, dev, mixer, f32, gated
@@ -75,7 +77,7 @@ class LatentLayer:
         k = self.keep
         self.a = pkg.Latent(H, D, P, V, R, self.ld, self.ldr, m["scale"], (m.get("mask") or {}).get("size", 0), k[0].data_ptr(), self.eps, k[1].data_ptr(), mul,
                             self.qw, self.qw + self.kw if self.gated else -1, pkg.DT_F32 if self.f32 else pkg.DT_F16, self.pool.data_ptr(), BS, k[2].data_ptr(),
-                            self.table.shape[1])
+                            self.table.shape[1], 0 if self.mma else self.blocks)
 
     def want(self, s):
         m, x = self.m, self.rows[s].astype(np.float64)
@@ -133,10 +135,10 @@ class LatentLayer:
                     pkg.check(L.cmlb200_latent_query(a, P(self.wukt), P(d), ld, P(dp), P(ds), near, P(q), None))
                     if one:
                         keys = max(b for _, b, e in step if e - b == 1)
-                        pkg.check(L.cmlb200_attention_latent(a, P(q), P(dp), P(ds), one, keys, None, 0, P(o), None))
+                        pkg.check(L.cmlb200_attention_latent(a, P(q), near, P(dp), P(ds), one, keys, None, 0, P(o), None))
                     if tiles[0]:
                         t = up(tiles[0], self.dev, np.int32)
-                        pkg.check(L.cmlb200_attention_latent(a, P(q), None, None, 0, max(x[3] + x[1] for x in tiles[0]), P(t), len(tiles[0]), P(o), None))
+                        pkg.check(L.cmlb200_attention_latent(a, P(q), near, None, None, 0, max(x[3] + x[1] for x in tiles[0]), P(t), len(tiles[0]), P(o), None))
                     pkg.check(L.cmlb200_latent_output(a, P(self.wuv), P(o), P(d), ld, near, P(out), old, None))
                 if long:
                     pkg.check(L.cmlb200_latent_append(a, P(d, near * ld * 4), ld, P(dp, near * 4), P(ds, near * 4), n - near, None))
@@ -156,6 +158,9 @@ class LatentLayer:
                     t = up(tiles[1], self.dev, np.int32)
                     pkg.check(L.cmlb200_attention_tiles(s2, P(d), ld, P(t), len(tiles[1]), P(out), old, None))
             sync()
+            st = C.c_int(-1)
+            pkg.check(L.cmlb200_attention_latent_status(C.byref(st), 1))
+            assert st.value == 0
             res, at = out.float().cpu().numpy(), 0
             assert (res[:, ow:] == 0).all()
             for s, b, e in step:
@@ -175,7 +180,7 @@ def mixer(H, D, P, V, R, window=0, scaling=None, base=1000.0, scale=None):
 
 
 def tol(f32):
-    return 2e-5 if f32 else 1.5e-2
+    return 2e-5 if f32 is True else 1.5e-2
 
 
 def whole(lengths):
@@ -194,7 +199,7 @@ SHAPES = [(4, 32, 16, 48, 80, 23), (3, 13, 6, 7, 21, 1), (20, 72, 64, 136, 300, 
           (1, 200, 32, 200, 256, 1000), (5, 24, 24, 33, 16, 31), (17, 64, 32, 64, 128, 64)]
 
 
-@pytest.mark.parametrize("f32", [False, True])
+@pytest.mark.parametrize("f32", [False, "mma", True])
 @pytest.mark.parametrize("shape", SHAPES)
 def test_prompts_portions_and_tokens(pkg, synth, torch_dev, shape, f32):
     lengths = [130, 1, 65, 17]
@@ -205,7 +210,7 @@ def test_prompts_portions_and_tokens(pkg, synth, torch_dev, shape, f32):
             assert np.abs(w - g).max() < tol(f32) * max(1, np.abs(w).max())
 
 
-@pytest.mark.parametrize("f32", [False, True])
+@pytest.mark.parametrize("f32", [False, "mma", True])
 @pytest.mark.parametrize("scaling", [None, (4.0, 64, 8.0, 1.0), (1.0, 32, 4.0, 0.5), (40.0, 4096, 32.0, 1.0), (2.0, 4, 50.0, 40.0)])
 def test_rotation_without_a_gate(pkg, synth, torch_dev, scaling, f32):
     """The rotated part carries nearly the whole score."""
@@ -219,7 +224,7 @@ def test_rotation_without_a_gate(pkg, synth, torch_dev, scaling, f32):
             assert np.abs(w - g).max() < tol(f32) * 2
 
 
-@pytest.mark.parametrize("f32", [False, True])
+@pytest.mark.parametrize("f32", [False, "mma", True])
 def test_portions_beside_single_tokens(pkg, synth, torch_dev, f32):
     lengths = [200, 231, 40, 7]
     for seed in (5, 6):
@@ -262,7 +267,7 @@ def stand_out(L, pairs, rotated, strength=14.0):
         x[q, :L.qw] = bf(qq.ravel())
 
 
-@pytest.mark.parametrize("f32", [False, True])
+@pytest.mark.parametrize("f32", [False, "mma", True])
 @pytest.mark.parametrize("window", [16, 17, 31, 33, 64, 80, 129])
 def test_window_edges(pkg, synth, torch_dev, window, f32):
     """Keys exactly at the edge: distance window - 1 is seen and dominates, distance window is not and leaves no trace.
@@ -288,7 +293,7 @@ def test_window_edges(pkg, synth, torch_dev, window, f32):
         assert (np.abs(other - want)[[q for q, _ in pairs]].max(1) > 6 * tol(f32)).all()
 
 
-@pytest.mark.parametrize("f32", [False, True])
+@pytest.mark.parametrize("f32", [False, "mma", True])
 @pytest.mark.parametrize("rotated", [False, True])
 def test_far_key_among_hundreds(pkg, synth, torch_dev, rotated, f32):
     """No window: one key hundreds of tokens back takes the weight, wherever it lies in its block or tile."""
@@ -305,20 +310,22 @@ def test_far_key_among_hundreds(pkg, synth, torch_dev, rotated, f32):
     assert (np.abs(L.want(0) - want)[[q for q, _ in pairs]].max(1) > 20 * tol(f32)).all()
 
 
-def test_long_decode_splits_keys_over_a_cluster(pkg, synth, torch_dev):
+@pytest.mark.parametrize("form", [False, "mma"])
+def test_long_decode_splits_keys_over_a_cluster(pkg, synth, torch_dev, form):
     """Few rows and thousands of keys: up to eight CTAs share a row's keys; the split must not show."""
     n = 3000
     for shape in ((4, 32, 16, 24, 64, 0), (2, 128, 64, 64, 512, 2500), (40, 16, 8, 16, 136, 1500)):
-        L = LatentLayer(pkg, synth, torch_dev, mixer(*shape, base=1e5), [n], False)
+        L = LatentLayer(pkg, synth, torch_dev, mixer(*shape, base=1e5), [n], form)
         got = L.run([[(0, 0, n - 9)]] + [[(0, t, t + 1)] for t in range(n - 9, n)])[0]
         rows = slice(n - 40, n)
         assert np.abs(L.want(0) - got)[rows].max() < tol(False)
 
 
-def test_many_rows_decode_together(pkg, synth, torch_dev):
+@pytest.mark.parametrize("form", [False, "mma"])
+def test_many_rows_decode_together(pkg, synth, torch_dev, form):
     """Batches above one block of query rows, with histories from none to hundreds of keys."""
     lengths = [1 + (37 * i) % 300 for i in range(75)]
-    L = LatentLayer(pkg, synth, torch_dev, mixer(6, 24, 8, 24, 48, 0), lengths, False)
+    L = LatentLayer(pkg, synth, torch_dev, mixer(6, 24, 8, 24, 48, 0), lengths, form)
     prompts = [(s, 0, n - 1) for s, n in enumerate(lengths) if n > 1]
     steps = [prompts[i::6] for i in range(6)]                            # at most 16 sequences to an expansion
     got = L.run(steps + [[(s, n - 1, n) for s, n in enumerate(lengths)]])
@@ -338,7 +345,7 @@ def test_latent_kernels_refuse_bad_arguments(pkg, synth, torch_dev):
     for field, value in (("rank", 513), ("cache_dtype", pkg.DT_F32), ("block_size", 24), ("ld", 72)):
         a = pkg.Latent.from_buffer_copy(L.a)
         setattr(a, field, value)
-        assert lib.cmlb200_attention_latent(a, fake, fake, fake, 1, 1, None, 0, fake, None) == -1
+        assert lib.cmlb200_attention_latent(a, fake, 1, fake, fake, 1, 1, None, 0, fake, None) == -1
     assert lib.cmlb200_latent_append(L.a, fake, 100, fake, fake, 1, None) == -1
 
 
