@@ -279,7 +279,6 @@ attention_latent_kernel(const cmlb200_latent a, const __half* __restrict__ q, co
 
 }  // namespace
 
-extern "C" int cmlb200_attention_latent_tc_fits_(const cmlb200_latent* a);
 extern "C" int cmlb200_attention_latent_tc_(const cmlb200_latent* a, const uint16_t* q, long q_rows, const int* row_pos, const int* row_slot, int max_keys,
                                             const int* tiles, int items, int most, int first, uint16_t* o, cudaStream_t st);
 
@@ -294,7 +293,7 @@ extern "C" int cmlb200_attention_latent(const cmlb200_latent* a, const uint16_t*
     CMLB_REQUIRE((((uintptr_t)d_q_f16 | (uintptr_t)a->pool | (uintptr_t)d_tiles) & 15) == 0 && ((uintptr_t)d_o_bf16 & 15) == 0, "%s: alignment", who);
     const int items = d_tiles ? tiles : rows, most = d_tiles ? 64 * a->heads : a->heads, sms = cmlb_num_sms();
     CMLB_REQUIRE(items <= 65535, "%s: %d rows", who, items);
-    if (cmlb200_attention_latent_tc_fits_(a))
+    if (cmlb200_attention_latent_tc_fits(a))
         return cmlb200_attention_latent_tc_(a, d_q_f16, (long)q_rows * a->heads, d_row_pos, d_row_slot, max_keys, d_tiles, items, most, d_tiles ? rows : 0, d_o_bf16,
                                             as_stream(stream));
     const int keys = (a->window > 0 && a->window < max_keys + 1) ? a->window : max_keys + 1, rank16 = (a->rank + 15) & ~15;

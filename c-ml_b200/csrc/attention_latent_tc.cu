@@ -2,15 +2,17 @@
 // whose operands fit shared memory.
 //
 // A CTA holds up to 32 or 64 (token, head) rows of queries and walks key tiles of 64 tokens; a cluster of up to 8 CTAs
-// splits the tiles and merges through distributed shared memory. Latents of more than 256 values give two CTAs a half
+// (4 for 64 rows) splits the tiles and merges through distributed shared memory. Latents of more than 256 values give two CTAs a half
 // of the output columns each (both compute the scores). Roles:
-//   warp 0     TMA: the queries once, then key tiles, 16 tokens to a copy (the block table says where), two stages;
-//              64-column slabs, 128-byte swizzle
-//   warp 1     owns tensor memory; one lane issues tcgen05.mma: S = Q K^T into two alternating accumulators, and
-//              O += P V, where V is the same tile read with its columns as the contiguous dimension
-//   warps 2-5  softmax, a thread per row (those whose quarter of tensor memory holds rows): S from tensor memory, mask,
-//              exponentials, P as fp16 into shared memory. The reference of the exponentials moves, and O is scaled,
-//              only when a row's maximum has grown by more than 8 (a factor of 256); sums are fp32
+//   warps 0, 2, 3  TMA: the queries once, then key tiles, 16 tokens to a copy (the block table says where), in slabs of 64
+//              columns with 128-byte swizzle; the slabs are shared out, since issuing the many small copies takes long.
+//              Slabs that are values too stay until O has taken them and have two or three stages, the others are free
+//              after the scores and have two
+//   warp 1     owns tensor memory; issues tcgen05.mma: S = Q K^T into two alternating accumulators, and
+//              O += P V, where V is the same tile read with its columns as the contiguous dimension; whichever of the two
+//              has its operands goes first
+//   warps 4, 5 softmax, a thread per row (warp 5 for 64 rows): S from tensor memory, mask, exponentials, P as fp16
+//              into shared memory. The reference of the exponentials moves, and O is scaled, only when a row's maximum has grown by more than 8 (a factor of 256); sums are fp32
 // The scores of tile i + 1 are computed while the softmax of tile i runs. An MMA is 128 rows high: those past the CTA's
 // read whatever follows in shared memory and are never looked at. Keys past the sequence's last are zeroed in the tile,
 // so that nothing other requests left in a block can reach the sums.
@@ -20,31 +22,42 @@
 
 namespace {
 
-constexpr int TC_THREADS = 192, TC_KEYS = 64, TC_SPLITS = 8, TC_SLAB = TC_KEYS * 128, TC_S_COL = 256, TC_TMEM = 512;
+constexpr int TC_THREADS = 192, TC_LOADERS = 3, TC_KEYS = 64, TC_SLAB = TC_KEYS * 128, TC_S_COL = 256, TC_TMEM = 512;
 
-__host__ __device__ inline size_t tc_operands(int mr, int slabs) { return (size_t)slabs * mr * 128 + (size_t)mr * 128 + 2 * (size_t)slabs * TC_SLAB; }
-__host__ __device__ inline size_t tc_smem(int mr, int slabs) { return tc_operands(mr, slabs) + 128 + 2 * 4 * (size_t)mr + 1024; }
+// Slabs of a tile: `v` of them are values of this launch's CTAs too (`stages` copies), `k` are keys alone (two copies).
+struct TcSlabs {
+    int all, v, k, stages;
+};
+__host__ __device__ inline size_t tc_operands(int mr, const TcSlabs& t) { return (size_t)t.all * mr * 128 + (size_t)mr * 128 + (size_t)(t.stages * t.v + 2 * t.k) * TC_SLAB; }
+__host__ __device__ constexpr int tc_splits(int mr) { return mr == 32 ? 8 : 4; }
+__host__ __device__ inline size_t tc_smem(int mr, const TcSlabs& t) { return tc_operands(mr, t) + 256 + 2 * 4 * (size_t)tc_splits(mr) * mr; }
 
 // grid = (splits, row blocks * halves, items), clusters of `splits` CTAs along x.
 template <int MR>
 __global__ void __launch_bounds__(TC_THREADS, 1)
 attention_latent_tc_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_constant__ CUtensorMap kmap, const cmlb200_latent a,
                            const int* __restrict__ row_pos, const int* __restrict__ row_slot, const int4* __restrict__ tiles, int first,
-                           __nv_bfloat16* __restrict__ out, int halves, int* status) {
-    extern __shared__ uint8_t smem_raw[];
-    uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
-    const int slabs = (a.ld + 63) / 64, stage_bytes = slabs * TC_SLAB;
-    const uint32_t qs = smem_addr(smem), ps = qs + slabs * MR * 128, ks = ps + MR * 128;
-    uint8_t* tail = smem + tc_operands(MR, slabs);
+                           __nv_bfloat16* __restrict__ out, int halves, const TcSlabs sl, int* status) {
+    extern __shared__ __align__(1024) uint8_t smem[];
+    constexpr int TC_SPLITS = tc_splits(MR);
+    if (smem_addr(smem) & 1023) {                                       // the swizzle needs it; the declaration asks for it
+        if (threadIdx.x == 0) *(volatile int*)status = 9;
+        return;
+    }
+    const int v_bytes = sl.v * TC_SLAB, k_bytes = sl.k * TC_SLAB;
+    const uint32_t qs = smem_addr(smem), ps = qs + sl.all * MR * 128, vs = ps + MR * 128, ks = vs + sl.stages * v_bytes;
+    uint8_t* tail = smem + tc_operands(MR, sl);
     const uint32_t bars = smem_addr(tail);
     const uint32_t q_full = bars, p_full = bars + 8, pv_done = bars + 16;
-    auto k_full = [&](int s) { return bars + 24 + 8 * s; };
-    auto k_empty = [&](int s) { return bars + 40 + 8 * s; };
-    auto s_full = [&](int s) { return bars + 56 + 8 * s; };
-    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(tail + 80);
-    volatile int* abort_flag = reinterpret_cast<volatile int*>(tail + 88);
-    float* c_m = reinterpret_cast<float*>(tail + 128);
-    float* c_l = c_m + MR;
+    auto s_full = [&](int s) { return bars + 24 + 8 * s; };
+    auto k_full = [&](int s) { return bars + 40 + 8 * s; };
+    auto k_empty = [&](int s) { return bars + 56 + 8 * s; };
+    auto v_full = [&](int s) { return bars + 72 + 8 * s; };
+    auto v_empty = [&](int s) { return bars + 96 + 8 * s; };
+    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(tail + 128);
+    volatile int* abort_flag = reinterpret_cast<volatile int*>(tail + 136);
+    float* c_m = reinterpret_cast<float*>(tail + 256);
+    float* c_l = c_m + TC_SPLITS * MR;                                  // [TC_SPLITS][MR] maxima and sums of the whole cluster
     float* Os = reinterpret_cast<float*>(smem);                         // [MR][columns + 4], over the operands once they are done
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
 
@@ -52,7 +65,8 @@ attention_latent_tc_kernel(const __grid_constant__ CUtensorMap qmap, const __gri
         mbar_init(q_full, 1);
         mbar_init(p_full, MR / 32);
         mbar_init(pv_done, 1);
-        for (int s = 0; s < 2; s++) { mbar_init(k_full(s), 1); mbar_init(k_empty(s), 1); mbar_init(s_full(s), 1); }
+        for (int s = 0; s < 2; s++) { mbar_init(k_full(s), TC_LOADERS); mbar_init(k_empty(s), 1); mbar_init(s_full(s), 1); }
+        for (int s = 0; s < 3; s++) { mbar_init(v_full(s), TC_LOADERS); mbar_init(v_empty(s), 1); }
         *abort_flag = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
@@ -68,6 +82,8 @@ attention_latent_tc_kernel(const __grid_constant__ CUtensorMap qmap, const __gri
     dep_wait();
     dep_trigger();
 
+    // first phase of the cluster's barrier: nothing is stored into another CTA before that one runs
+    if (gridDim.x > 1) asm volatile("barrier.cluster.arrive.relaxed.aligned;" ::: "memory");
     int4 tl = tiles ? tiles[blockIdx.z] : make_int4((int)blockIdx.z, 1, row_slot[blockIdx.z], row_pos[blockIdx.z]);
     tl.x -= first;
     const int total = tl.y * a.heads, half = blockIdx.y % halves, m0 = blockIdx.y / halves * MR;
@@ -79,72 +95,137 @@ attention_latent_tc_kernel(const __grid_constant__ CUtensorMap qmap, const __gri
     const int k_lo = (window > p_first ? 0 : p_first - window + 1) & ~15;
     const int ntiles = live ? (p_last - k_lo) / TC_KEYS + 1 : 0;
     const int n = rank < ntiles ? (ntiles - rank + splits - 1) / splits : 0;          // tiles of this CTA: rank, rank + splits, ..
-    const int nv = (a.rank + 63) / 64, per = (nv + halves - 1) / halves, v0 = half * per, cols = min(per, nv - v0) * 64;
+    // slabs v0 .. v0 + sl.v - 1 are this half's values; of an odd number both halves take the middle one
+    const int nv = (a.rank + 63) / 64, v0 = half * (nv - sl.v), cols = sl.v * 64;
     const int row0 = tl.x * a.heads + m0;
 
-    if (warp == 0) {
+    if (warp == 0 || warp == 2 || warp == 3) {
+        const int w = warp ? warp - 1 : 0;                              // slabs w, w + 3, .. of either kind
         bool ok = true;
-        int i = 0;
-        if (n > 0) {
-            if (lane == 0) mbar_expect_tx(q_full, (uint32_t)(slabs * MR * 128));
-            __syncwarp();
-            if (lane < slabs) tma_load_2d(qs + lane * MR * 128, &qmap, lane * 64, row0, q_full);
-        }
-        for (; i < n; i++) {
-            const int st = i & 1, kt = k_lo + (rank + i * splits) * TC_KEYS;
-            ok = __all_sync(0xffffffffu, mbar_wait(k_empty(st), ((i >> 1) & 1) ^ 1, abort_flag, 1, status));
-            if (!ok) break;
-            if (lane == 0) mbar_expect_tx(k_full(st), (uint32_t)stage_bytes);
-            __syncwarp();
-            for (int j = lane; j < 4 * slabs; j += 32) {
-                const int g = j & 3, s = j >> 2, key = min(kt + 16 * g, p_last & ~15);      // past the end: the last block again
-                const int slot = (table[key >> shift] << shift) + (key & (a.block_size - 1));
-                tma_load_2d(ks + st * stage_bytes + s * TC_SLAB + g * 2048, &kmap, s * 64, slot, k_full(st));
+        int i = 0, vst = 0, vpar = 1;
+        if (n > 0 && w == 0) {
+            if (elect_one()) {
+                mbar_expect_tx(q_full, (uint32_t)(sl.all * MR * 128));
+                for (int s = 0; s < sl.all; s++) tma_load_2d(qs + s * MR * 128, &qmap, s * 64, row0, q_full);
             }
+            __syncwarp();
         }
-        if (!ok && n > 0) {                                             // no copy outlives the CTA
-            mbar_wait(q_full, 0, abort_flag, 2, status);
-            for (int j = max(0, i - 2); j < i; j++) mbar_wait(k_full(j & 1), (j >> 1) & 1, abort_flag, 2, status);
+        // this warp's share of `count` slabs, the tile's slabs from `from` on (`skip` of them left out behind `gap`)
+        auto load = [&](const int (&slot)[4], int count, int from, int gap, int skip, uint32_t dst, uint32_t bar) {
+            const int mine = (count - w + TC_LOADERS - 1) / TC_LOADERS;
+            if (elect_one()) {
+                mbar_expect_tx(bar, (uint32_t)(max(mine, 0) * TC_SLAB));
+                for (int c = w; c < count; c += TC_LOADERS) {
+                    const int x = (from + c + (c >= gap ? skip : 0)) * 64;
+#pragma unroll
+                    for (int g = 0; g < 4; g++) tma_load_2d(dst + c * TC_SLAB + g * 2048, &kmap, x, slot[g], bar);
+                }
+            }
+            __syncwarp();
+        };
+        for (; i < n; i++) {
+            const int kt = k_lo + (rank + i * splits) * TC_KEYS;
+            // where the four blocks of 16 tokens lie; past the end the last one again
+            const int key = min(kt + 16 * (lane & 3), p_last & ~15), at = (table[key >> shift] << shift) + (key & (a.block_size - 1));
+            const int slot[4] = {__shfl_sync(0xffffffffu, at, 0), __shfl_sync(0xffffffffu, at, 1), __shfl_sync(0xffffffffu, at, 2), __shfl_sync(0xffffffffu, at, 3)};
+            if (sl.k) {
+                ok = __all_sync(0xffffffffu, mbar_wait(k_empty(i & 1), ((i >> 1) & 1) ^ 1, abort_flag, 1, status));
+                if (!ok) break;
+                load(slot, sl.k, 0, v0, sl.v, ks + (i & 1) * k_bytes, k_full(i & 1));
+            }
+            ok = __all_sync(0xffffffffu, mbar_wait(v_empty(vst), vpar, abort_flag, 1, status));
+            if (!ok) break;
+            load(slot, sl.v, v0, sl.v, 0, vs + vst * v_bytes, v_full(vst));
+            if (++vst == sl.stages) { vst = 0; vpar ^= 1; }
+        }
+        if (!ok && n > 0) {                                             // no copy outlives the CTA: tiles 0 .. i - 1, and the keys of tile i
+            if (w == 0) mbar_wait(q_full, 0, abort_flag, 2, status);
+            for (int j = max(0, i - sl.stages); j < i; j++) mbar_wait(v_full(j % sl.stages), (j / sl.stages) & 1, abort_flag, 2, status);
+            for (int j = max(0, i - 1); j <= i && sl.k; j++)
+                for (uint32_t it = 0; it < 65536 && !mbar_test(k_full(j & 1), (j >> 1) & 1); it++) __nanosleep(32);
         }
     } else if (warp == 1) {
-        if (lane == 0 && n > 0) {
+        if (n > 0) {
             // fp16 operands, fp32 accumulators, 128 rows; the second one takes V with its columns contiguous
             const uint32_t is = (1u << 4) | ((uint32_t)(TC_KEYS >> 3) << 17) | ((uint32_t)(128 >> 4) << 24);
             const uint32_t io = (1u << 4) | (1u << 16) | ((uint32_t)(cols >> 3) << 17) | ((uint32_t)(128 >> 4) << 24);
-            const int steps = a.ld / 16;
-            bool ok = mbar_wait(q_full, 0, abort_flag, 3, status);
-            auto scores = [&](int i) {
-                if (!mbar_wait(k_full(i & 1), (i >> 1) & 1, abort_flag, 4, status)) return false;
-                tmem_fence_after();
-                const uint32_t kst = ks + (i & 1) * stage_bytes;
-                for (int k = 0; k < steps; k++)
-                    umma(tmem + TC_S_COL + (i & 1) * TC_KEYS, make_desc(qs + (k >> 2) * MR * 128) + (uint64_t)(2 * (k & 3)),
-                         make_desc(kst + (k >> 2) * TC_SLAB) + (uint64_t)(2 * (k & 3)), is, k ? 1u : 0u);
-                umma_commit(s_full(i & 1));
-                return true;
-            };
-            ok = ok && scores(0);
-            for (int i = 0; i < n && ok; i++) {
-                if (i + 1 < n) ok = scores(i + 1);
-                ok = ok && mbar_wait(p_full, i & 1, abort_flag, 5, status);
-                if (!ok) break;
-                tmem_fence_after();
-                const uint32_t vst = ks + (i & 1) * stage_bytes + v0 * TC_SLAB;
+            const uint32_t acc = __shfl_sync(0xffffffffu, tmem, 0);
+            const int last = (a.ld & 63) >> 4;                          // steps of 16 columns in the last slab, 0: all four
+            bool ok = __all_sync(0xffffffffu, mbar_wait(q_full, 0, abort_flag, 3, status));
+            int i_s = 0, i_o = 0, s_st = 0, s_par = 0, o_st = 0;        // next tile of either product, value stages
+            uint32_t spins = 0;
+            while (ok && i_o < n) {
+                bool did = false;
+                // at most one tile ahead: the scores of the one before last have been read
+                if (i_s < n && i_s <= i_o + 1 && __all_sync(0xffffffffu, mbar_test(v_full(s_st), s_par) && (!sl.k || mbar_test(k_full(i_s & 1), (i_s >> 1) & 1)))) {
+                    tmem_fence_after();
+                    const uint32_t d = acc + TC_S_COL + (i_s & 1) * TC_KEYS, vst = vs + s_st * v_bytes, kst = ks + (i_s & 1) * k_bytes;
+                    // slabs s .. end - 1, which lie one behind the other from `at` on
+                    auto run = [&](int s, int end, uint32_t at) {
+                        const int whole = end == sl.all && last ? end - 1 : end;
+                        uint64_t ad = make_desc(qs + s * MR * 128), bd = make_desc(at);
+                        for (; s < whole; s++, ad += (uint64_t)(MR * 128 >> 4), bd += (uint64_t)(TC_SLAB >> 4)) {
+                            if (elect_one()) {
 #pragma unroll
-                for (int k = 0; k < TC_KEYS / 16; k++)
-                    umma(tmem, make_desc(ps) + (uint64_t)(2 * k), make_desc_mn(vst + k * 2048, TC_SLAB), io, (i | k) ? 1u : 0u);
-                umma_commit(k_empty(i & 1));
-                umma_commit(pv_done);
+                                for (int k = 0; k < 4; k++) umma(d, ad + (uint64_t)(2 * k), bd + (uint64_t)(2 * k), is, (s | k) ? 1u : 0u);
+                            }
+                            __syncwarp();
+                        }
+                        if (s < end && elect_one()) {
+#pragma unroll
+                            for (int k = 0; k < 3; k++)
+                                if (k < last) umma(d, ad + (uint64_t)(2 * k), bd + (uint64_t)(2 * k), is, (s | k) ? 1u : 0u);
+                        }
+                        __syncwarp();
+                    };
+                    run(0, v0, kst);
+                    run(v0, v0 + sl.v, vst);
+                    run(v0 + sl.v, sl.all, kst + v0 * TC_SLAB);
+                    if (elect_one()) {
+                        if (sl.k) umma_commit(k_empty(i_s & 1));
+                        umma_commit(s_full(i_s & 1));
+                    }
+                    __syncwarp();
+                    if (++s_st == sl.stages) { s_st = 0; s_par ^= 1; }
+                    i_s++;
+                    did = true;
+                }
+                if (i_o < i_s && __all_sync(0xffffffffu, mbar_test(p_full, i_o & 1))) {
+                    tmem_fence_after();
+                    const uint64_t pd = make_desc(ps), vd = make_desc_mn(vs + o_st * v_bytes, TC_SLAB);
+                    if (elect_one()) {
+#pragma unroll
+                        for (int k = 0; k < TC_KEYS / 16; k++) umma(acc, pd + (uint64_t)(2 * k), vd + (uint64_t)(k * (2048 >> 4)), io, (i_o | k) ? 1u : 0u);
+                        umma_commit(v_empty(o_st));
+                        umma_commit(pv_done);
+                    }
+                    __syncwarp();
+                    if (++o_st == sl.stages) o_st = 0;
+                    i_o++;
+                    did = true;
+                }
+                if (did) {
+                    spins = 0;
+                } else if (++spins > 1024) {
+                    ok = !__any_sync(0xffffffffu, *abort_flag != 0);
+                    __nanosleep(32);
+                    if (ok && spins > SPIN_LIMIT) {
+                        ok = false;
+                        *abort_flag = 4;
+                        if (*(volatile int*)status == 0) *(volatile int*)status = 4;
+                    }
+                }
             }
         }
         __syncwarp();
-    } else if ((warp & 3) * 32 < MR && live) {
+    } else if (warp >= 4 && (warp & 3) * 32 < MR && live) {
         const int q = warp & 3, r = q * 32 + lane;                      // the quarter of tensor memory's lanes this warp may read
         const uint32_t lanes = tmem + ((uint32_t)(q * 32) << 16);
         const int p = m0 + r < total ? tl.w + (m0 + r) / a.heads : -1;
         float m = -INFINITY, l = 0.f;
         bool ok = true;
-        for (int i = 0; i < n; i++) {
+        int vst = 0;
+        for (int i = 0; i < n; i++, vst = vst + 1 == sl.stages ? 0 : vst + 1) {
             const int kt = k_lo + (rank + i * splits) * TC_KEYS;
             ok = __all_sync(0xffffffffu, mbar_wait(s_full(i & 1), (i >> 1) & 1, abort_flag, 6, status));
             if (!ok) break;
@@ -202,10 +283,10 @@ attention_latent_tc_kernel(const __grid_constant__ CUtensorMap qmap, const __gri
             for (int j = 0; j < 8; j++) *reinterpret_cast<uint4*>(prow + ((j ^ (r & 7)) << 4)) = make_uint4(pk[4 * j], pk[4 * j + 1], pk[4 * j + 2], pk[4 * j + 3]);
             const int valid = p_last - kt + 1;                          // keys of this tile that exist
             if (valid < TC_KEYS) {
-                uint8_t* vst = smem + (ks - qs) + (i & 1) * stage_bytes + v0 * TC_SLAB;
+                uint8_t* v = smem + (vs - qs) + vst * v_bytes;
                 const int chunks = (TC_KEYS - valid) * 8;
-                for (int j = r; j < chunks * (cols / 64); j += MR)
-                    *reinterpret_cast<uint4*>(vst + j / chunks * TC_SLAB + valid * 128 + j % chunks * 16) = make_uint4(0u, 0u, 0u, 0u);
+                for (int j = r; j < chunks * sl.v; j += MR)
+                    *reinterpret_cast<uint4*>(v + j / chunks * TC_SLAB + valid * 128 + j % chunks * 16) = make_uint4(0u, 0u, 0u, 0u);
             }
             asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
             tmem_fence_before();
@@ -215,8 +296,20 @@ attention_latent_tc_kernel(const __grid_constant__ CUtensorMap qmap, const __gri
         if (ok && n > 0) ok = __all_sync(0xffffffffu, mbar_wait(pv_done, (n - 1) & 1, abort_flag, 8, status));
         tmem_fence_after();
         if (!ok) { m = -INFINITY; l = 0.f; }
-        c_m[r] = m;
-        c_l[r] = l;
+        __syncwarp();
+        if (splits > 1) {
+            asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
+#pragma unroll
+            for (int s = 0; s < TC_SPLITS; s++) {
+                if (s < splits) {
+                    uint32_t am, al;
+                    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(am) : "r"(smem_addr(c_m + rank * MR + r)), "r"(s));
+                    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(al) : "r"(smem_addr(c_l + rank * MR + r)), "r"(s));
+                    asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(am), "f"(m) : "memory");
+                    asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(al), "f"(l) : "memory");
+                }
+            }
+        }
         const float inv = l > 0.f ? 1.0f / l : 0.f;
         for (int c0 = 0; c0 < cols && n > 0; c0 += 32) {
             uint32_t o[32];
@@ -242,36 +335,32 @@ attention_latent_tc_kernel(const __grid_constant__ CUtensorMap qmap, const __gri
         tmem_fence_before();
     }
     __syncwarp();
+    if (splits > 1 && !(warp >= 4 && (warp & 3) * 32 < MR && live)) asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
     if (splits > 1 && live) {
         asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
         asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
         const int rows = min(MR, total - m0), quads = cols / 4;
         for (int i = rank * TC_THREADS + threadIdx.x; i < rows * quads; i += splits * TC_THREADS) {
             const int r = i / quads, c = (i - r * quads) * 4;
-            float ms[TC_SPLITS], ls[TC_SPLITS];
             float4 xs[TC_SPLITS];
 #pragma unroll
             for (int s = 0; s < TC_SPLITS; s++) {
-                ms[s] = -INFINITY; ls[s] = 0.f; xs[s] = make_float4(0.f, 0.f, 0.f, 0.f);
+                xs[s] = make_float4(0.f, 0.f, 0.f, 0.f);
                 if (s < splits) {
-                    uint32_t am, al, ax;
-                    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(am) : "r"(smem_addr(c_m + r)), "r"(s));
-                    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(al) : "r"(smem_addr(c_l + r)), "r"(s));
+                    uint32_t ax;
                     asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(ax) : "r"(smem_addr(Os + r * (cols + 4) + c)), "r"(s));
-                    asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(ms[s]) : "r"(am) : "memory");
-                    asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(ls[s]) : "r"(al) : "memory");
                     asm volatile("ld.shared::cluster.v4.f32 {%0,%1,%2,%3}, [%4];" : "=f"(xs[s].x), "=f"(xs[s].y), "=f"(xs[s].z), "=f"(xs[s].w) : "r"(ax) : "memory");
                 }
             }
-            float mx = ms[0], sum = 0.f;
+            float mx = -INFINITY, sum = 0.f;
             float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-            for (int s = 1; s < TC_SPLITS; s++) mx = fmaxf(mx, ms[s]);
+            for (int s = 0; s < TC_SPLITS; s++) mx = fmaxf(mx, s < splits ? c_m[s * MR + r] : -INFINITY);
 #pragma unroll
             for (int s = 0; s < TC_SPLITS; s++) {
-                if (ms[s] == -INFINITY) continue;                       // saw nothing: its values may be anything
-                const float f = exp2f(ms[s] - mx);
-                sum = fmaf(ls[s], f, sum);
+                if (s >= splits || c_m[s * MR + r] == -INFINITY) continue;      // saw nothing: its values may be anything
+                const float f = exp2f(c_m[s * MR + r] - mx);
+                sum = fmaf(c_l[s * MR + r], f, sum);
                 x.x = fmaf(xs[s].x, f, x.x); x.y = fmaf(xs[s].y, f, x.y); x.z = fmaf(xs[s].z, f, x.z); x.w = fmaf(xs[s].w, f, x.w);
             }
             const float inv = sum > 0.f ? 1.0f / sum : 0.f;
@@ -309,22 +398,31 @@ int status_word(int** word) {
 
 }  // namespace
 
-// 1: these sizes run here. Operands must fit, and the pool's extent must be known for its tensor map.
-extern "C" int cmlb200_attention_latent_tc_fits_(const cmlb200_latent* a) {
-    return a->pool_blocks > 0 && a->rank <= 512 && a->ld <= 8192 && tc_smem(64, (a->ld + 63) / 64) <= 227 * 1024;
+// Slabs and stages for CTAs of mr rows; stages 0: the operands do not fit.
+static TcSlabs tc_plan(const cmlb200_latent* a, int mr) {
+    TcSlabs t;
+    t.all = (a->ld + 63) / 64;
+    t.v = a->rank > 256 ? (a->rank + 127) / 128 : (a->rank + 63) / 64;
+    t.k = t.all - t.v;
+    for (t.stages = 3; t.stages > 1 && tc_smem(mr, t) > 227 * 1024; t.stages--) {}
+    if (t.stages == 1) t.stages = 0;
+    return t;
 }
+
+// 1: these sizes run here. Operands must fit, and the pool's extent must be known for its tensor map.
+extern "C" int cmlb200_attention_latent_tc_fits(const cmlb200_latent* a) { return a && a->pool_blocks > 0 && a->rank > 0 && a->rank <= 512 && a->ld <= 2048 && tc_plan(a, 64).stages > 0; }
 
 extern "C" int cmlb200_attention_latent_tc_(const cmlb200_latent* a, const uint16_t* q, long q_rows, const int* row_pos, const int* row_slot, int max_keys,
                                             const int* tiles, int items, int most, int first, uint16_t* o, cudaStream_t st) {
-    const int sms = cmlb_num_sms(), mr = most <= 32 ? 32 : 64, slabs = (a->ld + 63) / 64, halves = a->rank > 256 ? 2 : 1;
+    const int sms = cmlb_num_sms(), mr = most <= 32 ? 32 : 64, halves = a->rank > 256 ? 2 : 1;
     const int keys = (a->window > 0 && a->window < max_keys + 1) ? a->window : max_keys + 1;
     const long blocks = (long)((most + mr - 1) / mr) * halves;
     CMLB_REQUIRE(blocks <= 65535, "cmlb200_attention_latent: %d heads", a->heads);
     int splits = 1;
     double best = 0.0;
-    for (int s = 1; s <= TC_SPLITS && (s == 1 || (s - 1) * TC_KEYS < keys); s *= 2) {          // microseconds, by estimate
+    for (int s = 1; s <= tc_splits(mr) && (s == 1 || (s - 1) * TC_KEYS < keys); s *= 2) {          // microseconds, by estimate
         const long ctas = blocks * items * s, waves = (ctas + sms - 1) / sms, each = ((keys + TC_KEYS - 1) / TC_KEYS + s - 1) / s;
-        const double t = (double)waves * (3.0 + (double)each) + (s > 1 ? 1.5 : 0.0);
+        const double t = (double)waves * (5.0 + 1.6 * (double)each) + (s > 1 ? 2.0 : 0.0);
         if (s == 1 || t < best) { splits = s; best = t; }
     }
     int* status;
@@ -335,7 +433,8 @@ extern "C" int cmlb200_attention_latent_tc_(const cmlb200_latent* a, const uint1
     if (!rc) rc = encode_map(&kmap, CU_TENSOR_MAP_DATA_TYPE_FLOAT16, a->pool, (long)a->pool_blocks * a->block_size, a->ld, a->ld, 64, 16);
     if (rc) return rc;
     // one CTA to an SM: each needs all of the SM's tensor memory, and a cluster's CTAs wait for one another
-    const size_t need = tc_smem(mr, slabs), smem = need > 118 * 1024 ? need : 118 * 1024;
+    const TcSlabs sl = tc_plan(a, mr);
+    const size_t need = tc_smem(mr, sl), smem = need > 118 * 1024 ? need : 118 * 1024;
     const dim3 grid(splits, (unsigned)blocks, items);
     static size_t attr[2][kMaxDevices] = {};
 #define TC_LAUNCH(MR, slot)                                                                                                      \
@@ -343,7 +442,7 @@ extern "C" int cmlb200_attention_latent_tc_(const cmlb200_latent* a, const uint1
         auto kern = attention_latent_tc_kernel<MR>;                                                                              \
         CMLB_CUDA(cmlb_ensure_smem(kern, smem, attr[slot]));                                                                     \
         CMLB_CUDA(launch_chain(kern, grid, dim3(TC_THREADS), smem, splits, st, qmap, kmap, *a, row_pos, row_slot, (const int4*)tiles, first, (__nv_bfloat16*)o, \
-                               halves, status));                                                                                 \
+                               halves, sl, status));                                                                                 \
     } while (0)
     if (mr == 32) TC_LAUNCH(32, 0);
     else TC_LAUNCH(64, 1);

@@ -6,8 +6,6 @@
 
 namespace {
 
-template <typename T> __device__ __forceinline__ T to_query(float v) { return narrow<T>(v); }
-
 // Where the rotated queries of a row go: base + head * head_ld + off + i, times mul; entries up to off + fill are zeroed.
 template <typename TQ>
 struct QueryOut {
@@ -16,9 +14,17 @@ struct QueryOut {
     float mul;
 };
 
-// A block's work on one projection row. cs: rot_dim floats, red: 32.
+__device__ __forceinline__ void store2(float* d, float x, float y) { *reinterpret_cast<float2*>(d) = make_float2(x, y); }
+__device__ __forceinline__ void store2(__half* d, float x, float y) {
+    const __half v[2] = {narrow<__half>(x), narrow<__half>(y)};
+    *reinterpret_cast<uint32_t*>(d) = *reinterpret_cast<const uint32_t*>(v);
+}
+
+// A block's work on one projection row, or part `part` of it (the first one fills the cache). cs: rot_dim floats, red: 32.
 template <typename KV, typename TQ>
-__device__ __forceinline__ void latent_row(const cmlb200_latent& a, const float* row, int p, int slot, const QueryOut<TQ>& q, float* cs, float* red) {
+__device__ __forceinline__ void latent_row(const cmlb200_latent& a, const float* row, int p, int slot, const QueryOut<TQ>& q, int part, int parts, float* cs,
+                                           float* red) {
+    const bool fill = a.kv_col >= 0 && part == 0;
     const int half = a.rot_dim / 2, nt = blockDim.x;
     for (int i = threadIdx.x; i < half; i += nt) {
         float s, c;
@@ -28,14 +34,14 @@ __device__ __forceinline__ void latent_row(const cmlb200_latent& a, const float*
     }
     float inv = 0.f;
     const float* kv = row + a.kv_col;
-    if (a.kv_col >= 0) {
+    if (fill) {
         const float ss = block_sum(square_share(kv, a.rank), red);
         inv = 1.0f / sqrtf(ss / (float)a.rank + a.eps);
     } else {
         __syncthreads();
     }
     __syncthreads();
-    if (a.kv_col >= 0) {
+    if (fill) {
         const size_t at = (size_t)a.block_table[(size_t)slot * a.table_ld + p / a.block_size] * a.block_size + p % a.block_size;
         KV* d = static_cast<KV*>(a.pool) + at * a.ld;
 #pragma unroll 4
@@ -47,20 +53,34 @@ __device__ __forceinline__ void latent_row(const cmlb200_latent& a, const float*
         }
         for (int i = a.rank + a.rot_dim + threadIdx.x; i < a.ld; i += nt) d[i] = narrow<KV>(0.f);
     }
-    const int hd = a.dim + a.rot_dim;
+    const int hd = a.dim + a.rot_dim, first = part * nt + threadIdx.x, step = parts * nt;
+    // two neighbouring pairs at a time where everything is aligned for it
+    if ((half & 1) == 0 && ((a.dim | hd | q.head_ld | q.off) & 1) == 0 && (((uintptr_t)row | ((uintptr_t)q.base * (8 / (2 * sizeof(TQ))))) & 7) == 0) {
+        const int h2 = half >> 1;
 #pragma unroll 4
-    for (int j = threadIdx.x; j < a.heads * half; j += nt) {
-        const int h = j / half, i = j - h * half;
-        const float* s = row + h * hd + a.dim;
-        const float u = s[i], v = s[half + i];
-        TQ* d = q.base + (size_t)h * q.head_ld + q.off;
-        d[i] = to_query<TQ>((u * cs[i] - v * cs[half + i]) * q.mul);
-        d[half + i] = to_query<TQ>((v * cs[i] + u * cs[half + i]) * q.mul);
+        for (int j = first; j < a.heads * h2; j += step) {
+            const int h = j / h2, i = (j - h * h2) * 2;
+            const float* s = row + h * hd + a.dim;
+            const float2 u = *reinterpret_cast<const float2*>(s + i), v = *reinterpret_cast<const float2*>(s + half + i);
+            const float2 c = *reinterpret_cast<const float2*>(cs + i), n = *reinterpret_cast<const float2*>(cs + half + i);
+            TQ* d = q.base + (size_t)h * q.head_ld + q.off;
+            store2(d + i, (u.x * c.x - v.x * n.x) * q.mul, (u.y * c.y - v.y * n.y) * q.mul);
+            store2(d + half + i, (v.x * c.x + u.x * n.x) * q.mul, (v.y * c.y + u.y * n.y) * q.mul);
+        }
+    } else {
+        for (int j = first; j < a.heads * half; j += step) {
+            const int h = j / half, i = j - h * half;
+            const float* s = row + h * hd + a.dim;
+            const float u = s[i], v = s[half + i];
+            TQ* d = q.base + (size_t)h * q.head_ld + q.off;
+            d[i] = narrow<TQ>((u * cs[i] - v * cs[half + i]) * q.mul);
+            d[half + i] = narrow<TQ>((v * cs[i] + u * cs[half + i]) * q.mul);
+        }
     }
     const int pad = q.fill - a.rot_dim;
-    for (int j = threadIdx.x; j < a.heads * pad; j += nt) {
+    for (int j = first; j < a.heads * pad; j += step) {
         const int h = j / pad;
-        q.base[(size_t)h * q.head_ld + q.off + a.rot_dim + j - h * pad] = to_query<TQ>(0.f);
+        q.base[(size_t)h * q.head_ld + q.off + a.rot_dim + j - h * pad] = narrow<TQ>(0.f);
     }
 }
 
@@ -76,13 +96,15 @@ latent_append_kernel(const cmlb200_latent a, float* proj, int ld, const int* __r
     const int r = blockIdx.x;
     float* row = proj + (size_t)r * ld;
     const QueryOut<float> q = {q_out ? q_out + (size_t)r * q_ld : row, head_ld, off, a.rot_dim, 1.0f};
-    latent_row<KV, float>(a, row, row_pos[r], row_slot[r], q, cs, red);
+    latent_row<KV, float>(a, row, row_pos[r], row_slot[r], q, 0, 1, cs, red);
 }
 
 constexpr int LQ_WARPS = 4, LQ_THREADS = LQ_WARPS * 32, LQ_COLS = LQ_WARPS * 16, LQ_ROWS = 32;
 
+__host__ __device__ inline int row_parts(int rows) { return rows <= 8 ? 4 : 1; }      // blocks that share a row's rotation
+
 // grid = (rank / 64, heads + extra, rows / 32). Blocks y < heads: q16[row][y][n] = scale log2 e sum_d q[row][y][d] Wuk[y][d][n],
-// a warp per 16 outputs n, up to 32 rows. The blocks behind them: latent_row of the same rows, one each.
+// a warp per 16 outputs n, up to 32 rows. The blocks behind them: latent_row of the same rows.
 template <int NB>
 __global__ void __launch_bounds__(LQ_THREADS)
 latent_query_kernel(const cmlb200_latent a, const __nv_bfloat16* __restrict__ wukt, const float* __restrict__ proj, int ld, const int* __restrict__ row_pos,
@@ -94,10 +116,10 @@ latent_query_kernel(const cmlb200_latent a, const __nv_bfloat16* __restrict__ wu
     if ((int)blockIdx.y >= a.heads) {
         dep_wait();
         dep_trigger();
-        const int r = r0 + (blockIdx.y - a.heads) * gridDim.x + blockIdx.x;
+        const int job = (blockIdx.y - a.heads) * gridDim.x + blockIdx.x, parts = row_parts(rows), r = r0 + job / parts;
         if (r >= r0 + n) return;
         const QueryOut<__half> q = {q16 + (size_t)r * a.heads * a.ld, a.ld, a.rank, a.ld - a.rank, mul};
-        latent_row<__half, __half>(a, proj + (size_t)r * ld, row_pos[r], row_slot[r], q, reinterpret_cast<float*>(sm), red);
+        latent_row<__half, __half>(a, proj + (size_t)r * ld, row_pos[r], row_slot[r], q, job % parts, parts, reinterpret_cast<float*>(sm), red);
         return;
     }
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, t = lane & 3, h = blockIdx.y;
@@ -322,7 +344,8 @@ extern "C" int cmlb200_latent_query(const cmlb200_latent* a, const uint16_t* d_w
     CMLB_REQUIRE(d_wukt && d_proj && d_row_pos && d_row_slot && rows > 0 && d_q_f16 && a->cache_dtype == CMLB200_DT_F16, "cmlb200_latent_query: bad argument");
     CMLB_REQUIRE(((uintptr_t)d_wukt & 15) == 0 && rows <= 65535 * LQ_ROWS, "cmlb200_latent_query: alignment or %d rows", rows);
     const int gx = (a->rank + LQ_COLS - 1) / LQ_COLS, most = rows < LQ_ROWS ? rows : LQ_ROWS;
-    const dim3 grid(gx, a->heads + (most + gx - 1) / gx, (rows + LQ_ROWS - 1) / LQ_ROWS);
+    const int jobs = most * row_parts(rows);
+    const dim3 grid(gx, a->heads + (jobs + gx - 1) / gx, (rows + LQ_ROWS - 1) / LQ_ROWS);
     const int nb = rows <= 8 ? 1 : (rows <= 16 ? 2 : 4);
     const size_t x = (size_t)nb * 8 * (((a->dim + 63) & ~63) + 8) * 2 + (size_t)nb * 8 * (LQ_COLS + 8) * 2, rot = (size_t)a->rot_dim * 4;
     const size_t smem = x > rot ? x : rot;

@@ -525,6 +525,7 @@ int cmlb200_latent_query(const cmlb200_latent* a, const uint16_t* d_wukt, const 
  * with. max_keys bounds the cached keys in front of any row or tile (it picks the launch shape). */
 int cmlb200_attention_latent(const cmlb200_latent* a, const uint16_t* d_q_f16, int q_rows, const int* d_row_pos, const int* d_row_slot, int rows,
                              int max_keys, const int* d_tiles, int tiles, uint16_t* d_o_bf16, void* stream);
+int cmlb200_attention_latent_tc_fits(const cmlb200_latent* a);
 /* Not 0: a bounded wait of that kernel expired (valid once the stream has drained). */
 int cmlb200_attention_latent_status(int* status, int reset);
 /* out[row][head * vdim + v] = Wuv o, times the sigmoid of the gate. Wuv per head: [vdim rounded up to 16][ld_rank]. */

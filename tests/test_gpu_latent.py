@@ -196,7 +196,7 @@ def near_only(lengths, k=40):
 
 
 SHAPES = [(4, 32, 16, 48, 80, 23), (3, 13, 6, 7, 21, 1), (20, 72, 64, 136, 300, 100), (40, 16, 2, 24, 129, 0), (2, 128, 64, 128, 512, 0), (70, 8, 8, 8, 40, 65),
-          (1, 200, 32, 200, 256, 1000), (5, 24, 24, 33, 16, 31), (17, 64, 32, 64, 128, 64)]
+          (1, 200, 32, 200, 256, 1000), (5, 24, 24, 33, 16, 31), (17, 64, 32, 64, 128, 64), (6, 32, 96, 24, 500, 70), (33, 64, 64, 40, 512, 129)]
 
 
 @pytest.mark.parametrize("f32", [False, "mma", True])

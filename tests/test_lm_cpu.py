@@ -251,6 +251,17 @@ def test_tensor_file_refusals(pkg, synth, tmp_path):
         assert not _load(pkg, folder)
 
 
+def test_which_latents_run_on_the_tensor_cores(pkg):
+    """Usual sizes do; a pool of unknown extent and what exceeds shared memory go to the other form."""
+    def fits(rank, rot, pool_blocks=8):
+        a = pkg.Latent(heads=16, dim=64, rot_dim=rot, vdim=64, rank=rank, ld=(rank + rot + 15) // 16 * 16, ld_rank=(rank + 63) // 64 * 64, pool_blocks=pool_blocks)
+        return pkg.lib.cmlb200_attention_latent_tc_fits(a)
+    for rank, rot in ((512, 64), (512, 32), (256, 64), (300, 64), (128, 128), (16, 2), (72, 24)):
+        assert fits(rank, rot) == 1
+    assert fits(512, 64, 0) == 0 and fits(512, 128) == 0 and fits(513, 16) == 0
+    assert pkg.lib.cmlb200_attention_latent_tc_fits(None) == 0
+
+
 def test_null_arguments(pkg):
     lib = pkg.lib
     lib.cml_lm_free(None)
