@@ -487,6 +487,7 @@ _sig("cmlb200_latent_append", ci, _LAT, vp, ci, vp, vp, ci, vp)
 for _n in ("cmlb200_latent_query", "cmlb200_latent_query_f32"):
     _sig(_n, ci, _LAT, vp, vp, ci, vp, vp, ci, vp, vp)
 _sig("cmlb200_attention_latent", ci, _LAT, vp, ci, vp, vp, ci, ci, vp, ci, vp, vp)
+_sig("cmlb200_set_attention_latent_form", ci, ci)
 _sig("cmlb200_attention_latent_tc_fits", ci, _LAT)
 _sig("cmlb200_attention_latent_status", ci, C.POINTER(ci), ci)
 for _n in ("cmlb200_latent_output", "cmlb200_latent_output_f32"):

@@ -1,5 +1,5 @@
-// Attention over latents, the mma.sync form for what attention_latent_tc.cu does not take, and the entry point of both:
-// every head of a row attends the same keys, one vector [latent | rotated part] per token of a
+// Attention over latents, the mma.sync form for few rows and for what attention_latent_tc.cu does not take, and the entry
+// point of both: every head of a row attends the same keys, one vector [latent | rotated part] per token of a
 // paged cache, and the weighted sum of the latents is what a head returns. Queries come transformed
 // (cmlb200_latent_query), in units of log2. One kernel serves decoded tokens and short prompt portions:
 // the (token, head) pairs of a portion are the rows of the matrix products, 16, 32 or 64 to a CTA.
@@ -279,7 +279,15 @@ attention_latent_kernel(const cmlb200_latent a, const __half* __restrict__ q, co
 
 }  // namespace
 
-extern "C" int cmlb200_attention_latent_tc_(const cmlb200_latent* a, const uint16_t* q, long q_rows, const int* row_pos, const int* row_slot, int max_keys,
+static int g_form = 0;
+extern "C" int cmlb200_set_attention_latent_form(int form) {
+    CMLB_REQUIRE(form >= 0 && form <= 2, "cmlb200_set_attention_latent_form: form %d", form);
+    g_form = form;
+    return CMLB200_OK;
+}
+
+extern "C" double cmlb200_attention_latent_tc_estimate_(const cmlb200_latent* a, int items, int most, int keys, int* splits);
+extern "C" int cmlb200_attention_latent_tc_(const cmlb200_latent* a, const uint16_t* q, long q_rows, const int* row_pos, const int* row_slot, int splits,
                                             const int* tiles, int items, int most, int first, uint16_t* o, cudaStream_t st);
 
 extern "C" int cmlb200_attention_latent(const cmlb200_latent* a, const uint16_t* d_q_f16, int q_rows, const int* d_row_pos, const int* d_row_slot, int rows,
@@ -293,9 +301,6 @@ extern "C" int cmlb200_attention_latent(const cmlb200_latent* a, const uint16_t*
     CMLB_REQUIRE((((uintptr_t)d_q_f16 | (uintptr_t)a->pool | (uintptr_t)d_tiles) & 15) == 0 && ((uintptr_t)d_o_bf16 & 15) == 0, "%s: alignment", who);
     const int items = d_tiles ? tiles : rows, most = d_tiles ? 64 * a->heads : a->heads, sms = cmlb_num_sms();
     CMLB_REQUIRE(items <= 65535, "%s: %d rows", who, items);
-    if (cmlb200_attention_latent_tc_fits(a))
-        return cmlb200_attention_latent_tc_(a, d_q_f16, (long)q_rows * a->heads, d_row_pos, d_row_slot, max_keys, d_tiles, items, most, d_tiles ? rows : 0, d_o_bf16,
-                                            as_stream(stream));
     const int keys = (a->window > 0 && a->window < max_keys + 1) ? a->window : max_keys + 1, rank16 = (a->rank + 15) & ~15;
     auto blocks = [&](int m) { return (long)items * ((most + 16 * m - 1) / (16 * m)); };
     // rows per CTA and parts of the keys, by an estimate of the time in microseconds: wide tiles do more per key, narrow
@@ -305,13 +310,20 @@ extern "C" int cmlb200_attention_latent(const cmlb200_latent* a, const uint16_t*
     for (int m = 1; m <= 4; m *= 2) {
         const size_t bytes = latent_smem(16 * m, a->ld, rank16 + 4);
         if (bytes > 227 * 1024 || (m > 1 && most <= 8 * m)) continue;
-        const double tile = m == 1 ? 1.2 : (m == 2 ? 1.6 : 2.8);
         const long room = (long)sms * (m == 1 && 2 * bytes + 2048 <= 228 * 1024 ? 2 : 1);
         for (int s = 1; s <= (m == 1 ? LT_SPLITS : LT_SPLITS / 2) && (s == 1 || (s - 1) * LT_KEYS < keys); s *= 2) {
             const long ctas = blocks(m) * s, waves = (ctas + room - 1) / room, tiles_each = ((keys + LT_KEYS - 1) / LT_KEYS + s - 1) / s;
-            const double t = (double)waves * (3.0 + tile * (double)tiles_each) + (s > 1 ? 1.0 : 0.0);
+            const double tile = m == 1 ? (ctas > sms ? 3.6 : 2.2) : (m == 2 ? 3.6 : 5.2);
+            const double t = (double)waves * (6.0 + tile * (double)tiles_each) + (s > 1 ? 1.0 : 0.0);
             if (!mt || t < best) { mt = m; splits = s; best = t; }
         }
+    }
+    if (g_form != 1 && cmlb200_attention_latent_tc_fits(a)) {
+        int s = 1;
+        const double t = cmlb200_attention_latent_tc_estimate_(a, items, most, keys, &s);
+        if (!mt || t < best || g_form == 2)
+            return cmlb200_attention_latent_tc_(a, d_q_f16, (long)q_rows * a->heads, d_row_pos, d_row_slot, s, d_tiles, items, most, d_tiles ? rows : 0, d_o_bf16,
+                                                as_stream(stream));
     }
     CMLB_REQUIRE(mt > 0, "%s: rank %d and %d elements per token do not fit shared memory", who, a->rank, a->ld);
     const size_t smem = latent_smem(16 * mt, a->ld, rank16 + 4);

@@ -409,22 +409,61 @@ static TcSlabs tc_plan(const cmlb200_latent* a, int mr) {
     return t;
 }
 
+// One CTA to an SM: each needs all of the SM's tensor memory, and a cluster's CTAs wait for one another.
+static size_t tc_bytes(int mr, const TcSlabs& sl) {
+    const size_t need = tc_smem(mr, sl);
+    return need > 118 * 1024 ? need : 118 * 1024;
+}
+
 // 1: these sizes run here. Operands must fit, and the pool's extent must be known for its tensor map.
 extern "C" int cmlb200_attention_latent_tc_fits(const cmlb200_latent* a) { return a && a->pool_blocks > 0 && a->rank > 0 && a->rank <= 512 && a->ld <= 2048 && tc_plan(a, 64).stages > 0; }
 
-extern "C" int cmlb200_attention_latent_tc_(const cmlb200_latent* a, const uint16_t* q, long q_rows, const int* row_pos, const int* row_slot, int max_keys,
+// CTAs that run at a time when clusters of `splits` share the device: one to an SM, and a cluster stays within a group of
+// SMs whose size it may not divide.
+static long tc_room(int mr, int splits, size_t smem) {
+    static int active[2][4][kMaxDevices] = {};
+    if (splits == 1) return cmlb_num_sms();
+    int* n = &active[mr == 64][splits == 2 ? 1 : (splits == 4 ? 2 : 3)][cmlb_device_index()];
+    if (!*n) {
+        cudaLaunchAttribute attr;
+        attr.id = cudaLaunchAttributeClusterDimension;
+        attr.val.clusterDim.x = (unsigned)splits;
+        attr.val.clusterDim.y = attr.val.clusterDim.z = 1;
+        cudaLaunchConfig_t cfg = {};
+        cfg.gridDim = dim3(splits);
+        cfg.blockDim = dim3(TC_THREADS);
+        cfg.dynamicSmemBytes = smem;
+        cfg.attrs = &attr;
+        cfg.numAttrs = 1;
+        const void* kern = mr == 32 ? (const void*)attention_latent_tc_kernel<32> : (const void*)attention_latent_tc_kernel<64>;
+        if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess ||
+            cudaOccupancyMaxActiveClusters(n, kern, &cfg) != cudaSuccess || *n < 1) {
+            cudaGetLastError();
+            *n = cmlb_num_sms() / splits * 3 / 4;
+        }
+    }
+    return (long)*n * splits;
+}
+
+// Microseconds, by estimate, of the best split of the keys.
+extern "C" double cmlb200_attention_latent_tc_estimate_(const cmlb200_latent* a, int items, int most, int keys, int* splits) {
+    const int mr = most <= 32 ? 32 : 64;
+    const size_t smem = tc_bytes(mr, tc_plan(a, mr));
+    const long blocks = (long)items * ((most + mr - 1) / mr) * (a->rank > 256 ? 2 : 1);
+    double best = 0.0;
+    for (int s = 1; s <= tc_splits(mr) && (s == 1 || (s - 1) * TC_KEYS < keys); s *= 2) {
+        const long ctas = blocks * s, room = tc_room(mr, s, smem), waves = (ctas + room - 1) / room, each = ((keys + TC_KEYS - 1) / TC_KEYS + s - 1) / s;
+        const double t = (double)waves * (9.0 + 1.7 * (double)each) + (s > 1 ? 2.0 : 0.0);
+        if (s == 1 || t < best) { *splits = s; best = t; }
+    }
+    return best;
+}
+
+extern "C" int cmlb200_attention_latent_tc_(const cmlb200_latent* a, const uint16_t* q, long q_rows, const int* row_pos, const int* row_slot, int splits,
                                             const int* tiles, int items, int most, int first, uint16_t* o, cudaStream_t st) {
-    const int sms = cmlb_num_sms(), mr = most <= 32 ? 32 : 64, halves = a->rank > 256 ? 2 : 1;
-    const int keys = (a->window > 0 && a->window < max_keys + 1) ? a->window : max_keys + 1;
+    const int mr = most <= 32 ? 32 : 64, halves = a->rank > 256 ? 2 : 1;
     const long blocks = (long)((most + mr - 1) / mr) * halves;
     CMLB_REQUIRE(blocks <= 65535, "cmlb200_attention_latent: %d heads", a->heads);
-    int splits = 1;
-    double best = 0.0;
-    for (int s = 1; s <= tc_splits(mr) && (s == 1 || (s - 1) * TC_KEYS < keys); s *= 2) {          // microseconds, by estimate
-        const long ctas = blocks * items * s, waves = (ctas + sms - 1) / sms, each = ((keys + TC_KEYS - 1) / TC_KEYS + s - 1) / s;
-        const double t = (double)waves * (5.0 + 1.6 * (double)each) + (s > 1 ? 2.0 : 0.0);
-        if (s == 1 || t < best) { splits = s; best = t; }
-    }
     int* status;
     int rc = status_word(&status);
     if (rc) return rc;
@@ -432,9 +471,8 @@ extern "C" int cmlb200_attention_latent_tc_(const cmlb200_latent* a, const uint1
     rc = encode_map(&qmap, CU_TENSOR_MAP_DATA_TYPE_FLOAT16, q, q_rows, a->ld, a->ld, 64, mr);
     if (!rc) rc = encode_map(&kmap, CU_TENSOR_MAP_DATA_TYPE_FLOAT16, a->pool, (long)a->pool_blocks * a->block_size, a->ld, a->ld, 64, 16);
     if (rc) return rc;
-    // one CTA to an SM: each needs all of the SM's tensor memory, and a cluster's CTAs wait for one another
     const TcSlabs sl = tc_plan(a, mr);
-    const size_t need = tc_smem(mr, sl), smem = need > 118 * 1024 ? need : 118 * 1024;
+    const size_t smem = tc_bytes(mr, sl);
     const dim3 grid(splits, (unsigned)blocks, items);
     static size_t attr[2][kMaxDevices] = {};
 #define TC_LAUNCH(MR, slot)                                                                                                      \

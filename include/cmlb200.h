@@ -520,12 +520,15 @@ int cmlb200_poly_norm(const float* d_z, int ld, int rows, int ff, const float* d
 int cmlb200_latent_append(const cmlb200_latent* a, float* d_proj, int ld, const int* d_row_pos, const int* d_row_slot, int rows, void* stream);
 int cmlb200_latent_query(const cmlb200_latent* a, const uint16_t* d_wukt, const float* d_proj, int ld, const int* d_row_pos, const int* d_row_slot,
                          int rows, uint16_t* d_q_f16, void* stream);
-/* Weighted latents bf16 [q_rows][heads][ld_rank] of such query rows, on tcgen05 where the sizes fit. d_tiles NULL: row r is one token (position and slot
+/* Weighted latents bf16 [q_rows][heads][ld_rank] of such query rows. d_tiles NULL: row r is one token (position and slot
  * from the row arrays); otherwise tiles as in cmlb200_attention_tiles, and `rows` is the row that d_q_f16 begins
  * with. max_keys bounds the cached keys in front of any row or tile (it picks the launch shape). */
 int cmlb200_attention_latent(const cmlb200_latent* a, const uint16_t* d_q_f16, int q_rows, const int* d_row_pos, const int* d_row_slot, int rows,
                              int max_keys, const int* d_tiles, int tiles, uint16_t* d_o_bf16, void* stream);
 int cmlb200_attention_latent_tc_fits(const cmlb200_latent* a);
+/* 0: the form that is estimated to be faster (the default), 1: mma.sync, 2: tcgen05 where it fits. For launches made after
+ * the call. */
+int cmlb200_set_attention_latent_form(int form);
 /* Not 0: a bounded wait of that kernel expired (valid once the stream has drained). */
 int cmlb200_attention_latent_status(int* status, int reset);
 /* out[row][head * vdim + v] = Wuv o, times the sigmoid of the gate. Wuv per head: [vdim rounded up to 16][ld_rank]. */

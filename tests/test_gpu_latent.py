@@ -93,8 +93,15 @@ class LatentLayer:
     def run(self, portions):
         """portions: steps, each a list of (sequence, first, end). Ranges of one token and of up to 64 go over the latents,
         longer ones through the expansion (or everything through the 32-bit kernels)."""
-        import torch
         self.upload()
+        self.pkg.check(self.pkg.lib.cmlb200_set_attention_latent_form(1 if self.mma else 2))
+        try:
+            return self._run(portions)
+        finally:
+            self.pkg.check(self.pkg.lib.cmlb200_set_attention_latent_form(0))
+
+    def _run(self, portions):
+        import torch
         pkg, L, a, m = self.pkg, self.pkg.lib, self.a, self.m
         H, V, ow = m["heads"], m["vdim"], m["heads"] * m["vdim"]
         got = [np.full((len(x), ow), np.nan) for x in self.rows]

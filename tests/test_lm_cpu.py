@@ -260,6 +260,7 @@ def test_which_latents_run_on_the_tensor_cores(pkg):
         assert fits(rank, rot) == 1
     assert fits(512, 64, 0) == 0 and fits(512, 128) == 0 and fits(513, 16) == 0
     assert pkg.lib.cmlb200_attention_latent_tc_fits(None) == 0
+    assert pkg.lib.cmlb200_set_attention_latent_form(3) == -1 and pkg.lib.cmlb200_set_attention_latent_form(0) == 0
 
 
 def test_null_arguments(pkg):
