@@ -245,13 +245,14 @@ attention_latent_kernel(const cmlb200_latent a, const __half* __restrict__ q, co
         }
     asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
     asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
-    const int live = min(MR, total - m0);
-    for (int i = rank * LT_THREADS + threadIdx.x; i < live * a.rank; i += splits * LT_THREADS) {
-        const int r = i / a.rank, d = i - r * a.rank;
-        float ms[LT_SPLITS], ls[LT_SPLITS], xs[LT_SPLITS];
+    const int live = min(MR, total - m0), quads = rank16 / 4;
+    for (int i = rank * LT_THREADS + threadIdx.x; i < live * quads; i += splits * LT_THREADS) {
+        const int r = i / quads, d = (i - r * quads) * 4;
+        float ms[LT_SPLITS], ls[LT_SPLITS];
+        float4 xs[LT_SPLITS];
 #pragma unroll
         for (int s = 0; s < LT_SPLITS; s++) {
-            ms[s] = -INFINITY; ls[s] = 0.f; xs[s] = 0.f;
+            ms[s] = -INFINITY; ls[s] = 0.f; xs[s] = make_float4(0.f, 0.f, 0.f, 0.f);
             if (s < splits) {
                 uint32_t am, al, ax;
                 asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(am) : "r"(smem_addr(c_m + r)), "r"(s));
@@ -259,19 +260,25 @@ attention_latent_kernel(const cmlb200_latent a, const __half* __restrict__ q, co
                 asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(ax) : "r"(smem_addr(Os + r * LDO + d)), "r"(s));
                 asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(ms[s]) : "r"(am) : "memory");
                 asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(ls[s]) : "r"(al) : "memory");
-                asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(xs[s]) : "r"(ax) : "memory");
+                asm volatile("ld.shared::cluster.v4.f32 {%0,%1,%2,%3}, [%4];" : "=f"(xs[s].x), "=f"(xs[s].y), "=f"(xs[s].z), "=f"(xs[s].w) : "r"(ax) : "memory");
             }
         }
-        float mx = ms[0], x = 0.f, sum = 0.f;
+        float mx = ms[0], sum = 0.f;
+        float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
         for (int s = 1; s < LT_SPLITS; s++) mx = fmaxf(mx, ms[s]);
 #pragma unroll
         for (int s = 0; s < LT_SPLITS; s++) {
             const float c = ms[s] == -INFINITY ? 0.f : exp2f(ms[s] - mx);
-            x = fmaf(xs[s], c, x);
             sum = fmaf(ls[s], c, sum);
+            x.x = fmaf(xs[s].x, c, x.x); x.y = fmaf(xs[s].y, c, x.y); x.z = fmaf(xs[s].z, c, x.z); x.w = fmaf(xs[s].w, c, x.w);
         }
-        out[(out0 + r) * a.ld_rank + d] = __float2bfloat16_rn(x / sum);
+        // columns rank .. ld_rank meet zero weights
+        const float inv = 1.0f / sum;
+        const __nv_bfloat162 lo = __floats2bfloat162_rn(x.x * inv, d + 1 < a.rank ? x.y * inv : 0.f);
+        const __nv_bfloat162 hi = __floats2bfloat162_rn(d + 2 < a.rank ? x.z * inv : 0.f, d + 3 < a.rank ? x.w * inv : 0.f);
+        if (d < a.rank)
+            *reinterpret_cast<uint2*>(out + (out0 + r) * a.ld_rank + d) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
     }
     asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");      // nobody leaves while others read its shared memory
     asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");

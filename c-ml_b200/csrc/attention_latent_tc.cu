@@ -436,7 +436,7 @@ static long tc_room(int mr, int splits, size_t smem) {
         cfg.attrs = &attr;
         cfg.numAttrs = 1;
         const void* kern = mr == 32 ? (const void*)attention_latent_tc_kernel<32> : (const void*)attention_latent_tc_kernel<64>;
-        if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess ||
+        if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess ||
             cudaOccupancyMaxActiveClusters(n, kern, &cfg) != cudaSuccess || *n < 1) {
             cudaGetLastError();
             *n = cmlb_num_sms() / splits * 3 / 4;
