@@ -319,9 +319,9 @@ extern "C" int cmlb200_attention_latent(const cmlb200_latent* a, const uint16_t*
         if (bytes > 227 * 1024 || (m > 1 && most <= 8 * m)) continue;
         const long room = (long)sms * (m == 1 && 2 * bytes + 2048 <= 228 * 1024 ? 2 : 1);
         for (int s = 1; s <= (m == 1 ? LT_SPLITS : LT_SPLITS / 2) && (s == 1 || (s - 1) * LT_KEYS < keys); s *= 2) {
-            const long ctas = blocks(m) * s, waves = (ctas + room - 1) / room, tiles_each = ((keys + LT_KEYS - 1) / LT_KEYS + s - 1) / s;
-            const double tile = m == 1 ? (ctas > sms ? 3.6 : 2.2) : (m == 2 ? 3.6 : 5.2);
-            const double t = (double)waves * (6.0 + tile * (double)tiles_each) + (s > 1 ? 1.0 : 0.0);
+            const long ctas = blocks(m) * s, fit = s == LT_SPLITS ? sms : room, waves = (ctas + fit - 1) / fit, tiles_each = ((keys + LT_KEYS - 1) / LT_KEYS + s - 1) / s;
+            const double tile = m == 1 ? (ctas > sms ? 2.65 : 1.9) : (m == 2 ? 3.6 : 5.2);
+            const double t = (double)waves * (5.0 + tile * (double)tiles_each) + (s > 1 ? 1.0 : 0.0);
             if (!mt || t < best) { mt = m; splits = s; best = t; }
         }
     }

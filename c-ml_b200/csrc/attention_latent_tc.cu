@@ -453,7 +453,7 @@ extern "C" double cmlb200_attention_latent_tc_estimate_(const cmlb200_latent* a,
     double best = 0.0;
     for (int s = 1; s <= tc_splits(mr) && (s == 1 || (s - 1) * TC_KEYS < keys); s *= 2) {
         const long ctas = blocks * s, room = tc_room(mr, s, smem), waves = (ctas + room - 1) / room, each = ((keys + TC_KEYS - 1) / TC_KEYS + s - 1) / s;
-        const double t = (double)waves * (9.0 + 1.7 * (double)each) + (s > 1 ? 2.0 : 0.0);
+        const double t = (double)waves * (9.0 + 1.8 * (double)each) + (s > 1 ? 2.0 : 0.0);
         if (s == 1 || t < best) { *splits = s; best = t; }
     }
     return best;
