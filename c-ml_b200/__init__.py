@@ -436,7 +436,7 @@ DTYPE_FLOAT32, DTYPE_BFLOAT16 = 0, 6
 
 class Dense(C.Structure):
     """cmlb200_dense."""
-    _fields_ = [("dtype", ci), ("rows", ci), ("cols", ci), ("ld", ci), ("w", vp)]
+    _fields_ = [("dtype", ci), ("rows", ci), ("cols", ci), ("ld", ci), ("w", vp), ("bias", vp), ("cap", C.c_float)]
 
 
 class Attn(C.Structure):
@@ -444,7 +444,8 @@ class Attn(C.Structure):
     _fields_ = [("heads", ci), ("kv_heads", ci), ("dim", ci), ("vdim", ci), ("dim_ld", ci), ("vdim_ld", ci), ("scale", C.c_float),
                 ("window", ci), ("slopes", vp), ("sink", ci), ("q_norm", vp), ("k_norm", vp), ("eps", C.c_float), ("temp_coef", C.c_float),
                 ("temp_every", C.c_float), ("gate_col", ci), ("cache_dtype", ci), ("k_pool", vp), ("v_pool", vp), ("block_size", ci),
-                ("block_table", vp), ("table_ld", ci), ("gate_wide", ci)]
+                ("block_table", vp), ("table_ld", ci), ("gate_wide", ci), ("keep", ci), ("chunk", ci), ("sinks", vp), ("head_norm", ci), ("keys_as_values", ci),
+                ("out_scale", C.c_float)]
 
 
 class Latent(C.Structure):
@@ -457,7 +458,24 @@ class Latent(C.Structure):
 class Moe(C.Structure):
     """cmlb200_moe."""
     _fields_ = [("experts", ci), ("top", ci)] + [(n, vp) for n in ("ids", "weight", "pos", "src", "expert", "start", "count", "active", "num_active", "tiles",
-                                                                     "num_tiles")]
+                                                                     "num_tiles")] + \
+               [("identity", ci), ("groups", ci), ("keep", ci), ("correction", vp), ("normalize", ci), ("scale", C.c_float), ("self", vp)]
+
+
+class Streams(C.Structure):
+    """cmlb200_streams."""
+    _fields_ = [("streams", ci), ("mix", vp), ("out", vp), ("read", vp)]
+
+
+class Join(C.Structure):
+    """cmlb200_join."""
+    _fields_ = [("parts", C.POINTER(Moe)), ("h", vp), ("add", vp), ("ld_add", ci)]
+
+
+class Delta(C.Structure):
+    """cmlb200_delta."""
+    _fields_ = [("heads", ci), ("kv_heads", ci), ("dim", ci), ("vdim", ci), ("taps", ci), ("vdim_ld", ci), ("col", ci), ("conv", vp), ("rate", vp),
+                ("dt_bias", vp), ("norm", vp), ("eps", C.c_float), ("out_scale", C.c_float), ("state", vp), ("ring", vp)]
 
 
 class LMOptions(C.Structure):
@@ -483,6 +501,12 @@ _sig("cmlb200_glu_rows_f32", ci, vp, ci, ci, ci, ci, vp, ci, vp)
 _LAT, _MOE, _DENSE, _cf = C.POINTER(Latent), C.POINTER(Moe), C.POINTER(Dense), C.c_float
 _sig("cmlb200_residual_add", ci, vp, vp, ci, _MOE, vp, _cf, ci, ci, vp, ci, ci, vp)
 _sig("cmlb200_poly_norm", ci, vp, ci, ci, ci, vp, _cf, vp, ci, ci, vp)
+_sig("cmlb200_embed_streams", ci, vp, ci, vp, _cf, ci, ci, ci, ci, vp, vp)
+_sig("cmlb200_stream_join", ci, C.POINTER(Streams), vp, vp, ci, C.POINTER(Join), vp, _cf, ci, ci, vp, vp, ci, ci, vp)
+_sig("cmlb200_delta_one", ci, C.POINTER(Delta), vp, ci, vp, ci, vp, ci, vp, vp, ci, vp, ci, ci, vp)
+_sig("cmlb200_delta_rows", ci, C.POINTER(Delta), vp, ci, vp, ci, vp, ci, vp, vp, ci, ci, vp, ci, vp, vp, ci, ci, vp)
+_sig("cmlb200_delta_work_floats", ci, C.POINTER(Delta))
+_sig("cmlb200_pack_columns", ci, vp, ci, ci, ci, ci, vp, ci, vp)
 _sig("cmlb200_latent_append", ci, _LAT, vp, ci, vp, vp, ci, vp)
 for _n in ("cmlb200_latent_query", "cmlb200_latent_query_f32"):
     _sig(_n, ci, _LAT, vp, vp, ci, vp, vp, ci, vp, vp)
@@ -521,6 +545,7 @@ _sig("cml_paged_kv_cache_create_device", C.POINTER(PagedKVCache), ci, ci, ci)
 _sig("cml_paged_cache_blocks_for", ci, C.POINTER(PagedKVCache), ci, ci)
 _sig("cml_paged_cache_extend", ci, C.POINTER(PagedKVCache), ci, ci)
 _sig("cml_paged_cache_release_before", None, C.POINTER(PagedKVCache), ci, ci)
+_sig("cml_paged_cache_release_between", None, C.POINTER(PagedKVCache), ci, ci, ci)
 
 
 class LanguageModel:

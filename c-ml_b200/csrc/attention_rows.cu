@@ -1,7 +1,9 @@
 // Attention of a step's rows over paged caches, for layers described by a cmlb200_attn: grouped heads
-// with separate query/key and value sizes, a sliding window, a per-head linear distance bias, a sink
-// (one added to the softmax denominator), a per-head output gate. Rows of different sequences share a
-// launch; every row finds its keys through its sequence's block table.
+// with separate query/key and value sizes, a sliding window or chunks (with or without the sequence's first
+// tokens kept in sight), a per-head linear distance bias, a sink (one, or a learned exponential per head, added
+// to the softmax denominator), norms over all heads or per head, values that are the keys before their norm, a
+// per-head output gate. Rows of different sequences share a launch; every row finds its keys through its
+// sequence's block table.
 //
 //   attention_tiles_kernel   prompt portions: 64 consecutive query rows of one sequence and one head per
 //                            CTA, key tiles of 64 (only those some row's window reaches) double-buffered
@@ -14,7 +16,7 @@
 //   attention_rows_f32_kernel  fp32 caches, one CTA per (row, head), everything in fp32
 //
 // Scores are kept in units of log2 in the first two kernels (the scale carries log2 e). A sink starts
-// the running maximum at 0, so its weight exp(0 - m) joins the denominator exactly once.
+// the running maximum at its score, so its weight joins the denominator exactly once.
 #include "lm_util.cuh"
 
 namespace {
@@ -24,6 +26,14 @@ __device__ __forceinline__ uint32_t pack_h2(float lo, float hi) {
     return *reinterpret_cast<const uint32_t*>(&v);
 }
 constexpr int QT = 64, KT = 64, TILE_THREADS = 128;
+
+// The first key that the row at position p sees, the kept ones (0 .. keep - 1) aside.
+__device__ __forceinline__ int first_key(const cmlb200_attn& a, int p) {
+    if (a.chunk > 0) return p / a.chunk * a.chunk;
+    return (a.window > 0 && a.window <= p) ? p - a.window + 1 : 0;
+}
+__device__ __forceinline__ float sink_score(const cmlb200_attn& a, int h) { return a.sinks ? a.sinks[h] : 0.f; }
+__device__ __forceinline__ float out_scale(const cmlb200_attn& a) { return a.out_scale == 0.f ? 1.f : a.out_scale; }
 
 // grid = (tiles, heads). tiles[i] = {first row, rows (1..64), sequence slot, position of the first row}.
 // DV: room for value columns. DK: 0, or the padded key size, and then DV is the padded value size.
@@ -43,16 +53,18 @@ attention_tiles_kernel(const cmlb200_attn a, const float* __restrict__ qkv, int 
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, t = lane & 3;
     const int shift = __ffs(a.block_size) - 1;
     const int* table = a.block_table + (size_t)tl.z * a.table_ld;
-    const int window = a.window > 0 ? a.window : 0x7fffffff;
     const int p_last = p0 + n - 1;
-    const int k_lo = (window > p0 ? 0 : p0 - window + 1) & ~15;
-    const int ntiles = (p_last - k_lo) / KT + 1;
+    // key tiles: those of the kept tokens, then from k_lo on (one run from 0 where they meet)
+    int k_lo = first_key(a, p0) & ~15, kept_tiles = (min(a.keep, k_lo) + KT - 1) / KT;
+    if (kept_tiles * KT >= k_lo) { k_lo = 0; kept_tiles = 0; }
+    const int ntiles = kept_tiles + (p_last - k_lo) / KT + 1;
+    auto tile_start = [&](int it) { return it < kept_tiles ? it * KT : k_lo + (it - kept_tiles) * KT; };
     const __half* kp = static_cast<const __half*>(a.k_pool) + (size_t)kh * dk;
     const __half* vp = static_cast<const __half*>(a.v_pool) + (size_t)kh * dv;
     const int kstride = a.kv_heads * dk, vstride = a.kv_heads * dv;
 
     auto load = [&](int it) {
-        const int kt = k_lo + it * KT, st = it & 1;
+        const int kt = tile_start(it), st = it & 1;
         const int kc = dk >> 3, vc = dv >> 3;
         for (int row = threadIdx.x >> 3; row < KT; row += TILE_THREADS / 8) {
             const int key = min(kt + row, p_last);     // rows past the end repeat the last key (masked below)
@@ -75,10 +87,12 @@ attention_tiles_kernel(const cmlb200_attn a, const float* __restrict__ qkv, int 
     const int r0 = warp * 16 + g, r1 = r0 + 8;
     const int q0 = r0 < n ? p0 + r0 : -1, q1 = r1 < n ? p0 + r1 : -1;         // -1: sees nothing
     const int w_first = p0 + warp * 16, w_last = min(p0 + warp * 16 + 15, p_last);
+    const int lo0 = first_key(a, max(q0, 0)), lo1 = first_key(a, max(q1, 0)), w_lo = first_key(a, w_first), w_lo_last = first_key(a, max(w_last, 0));
+    const float sink = a.sink ? sink_score(a, h) * kLog2e : -INFINITY;
     float o[DV / 8][4];
 #pragma unroll
     for (int i = 0; i < DV / 8; i++) { o[i][0] = 0.f; o[i][1] = 0.f; o[i][2] = 0.f; o[i][3] = 0.f; }
-    float m0 = a.sink ? 0.f : -INFINITY, m1 = m0, l0 = 0.f, l1 = 0.f;
+    float m0 = sink, m1 = m0, l0 = 0.f, l1 = 0.f;
     // score of key kt + c from position q: dot - slope (q - kt - c). The part that depends on the column alone
     // is what the accumulators start from; the rest is one constant per row and tile.
     float bias[KT / 8][2];
@@ -94,9 +108,9 @@ attention_tiles_kernel(const cmlb200_attn a, const float* __restrict__ qkv, int 
             asm volatile("cp.async.wait_group 0;" ::: "memory");
         }
         __syncthreads();
-        const int kt = k_lo + it * KT, st = it & 1;
-        // nothing of this tile is in reach of this warp's rows: below every window, or past the last row
-        const bool active = w_first <= w_last && kt <= w_last && (window > w_first || kt + KT - 1 > w_first - window);
+        const int kt = tile_start(it), st = it & 1;
+        // nothing of this tile is in reach of this warp's rows: before all they see, or past the last row
+        const bool active = w_first <= w_last && kt <= w_last && (kt + KT - 1 >= w_lo || kt < a.keep);
         if (active) {
             float s[KT / 8][4];
 #pragma unroll
@@ -115,14 +129,15 @@ attention_tiles_kernel(const cmlb200_attn a, const float* __restrict__ qkv, int 
                 }
             }
             // unless every row of the warp sees every key of the tile
-            if (!(kt + KT - 1 <= w_first && (window > w_last - kt)) || w_last - w_first < 15) {
+            if (!(kt + KT - 1 <= w_first && kt >= w_lo_last) || w_last - w_first < 15) {
 #pragma unroll
                 for (int i = 0; i < KT / 8; i++) {
 #pragma unroll
                     for (int e = 0; e < 2; e++) {
-                        const int key = kt + i * 8 + 2 * t + e, d0 = q0 - key, d1 = q1 - key;
-                        if (d0 < 0 || d0 >= window) s[i][e] = -INFINITY;
-                        if (d1 < 0 || d1 >= window) s[i][2 + e] = -INFINITY;
+                        const int key = kt + i * 8 + 2 * t + e;
+                        const bool kept_key = key < a.keep;
+                        if (key > q0 || (key < lo0 && !kept_key)) s[i][e] = -INFINITY;
+                        if (key > q1 || (key < lo1 && !kept_key)) s[i][2 + e] = -INFINITY;
                     }
                 }
             }
@@ -172,8 +187,8 @@ attention_tiles_kernel(const cmlb200_attn a, const float* __restrict__ qkv, int 
     }
     l0 += __shfl_xor_sync(0xffffffffu, l0, 1); l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
     l1 += __shfl_xor_sync(0xffffffffu, l1, 1); l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
-    if (a.sink) { l0 += exp2f(-m0); l1 += exp2f(-m1); }
-    float i0 = l0 > 0.f ? 1.0f / l0 : 0.f, i1 = l1 > 0.f ? 1.0f / l1 : 0.f;
+    if (a.sink) { l0 += exp2f(sink - m0); l1 += exp2f(sink - m1); }
+    float i0 = l0 > 0.f ? out_scale(a) / l0 : 0.f, i1 = l1 > 0.f ? out_scale(a) / l1 : 0.f;
     if (a.gate_col >= 0 && !a.gate_wide) {
         if (r0 < n) i0 *= sigmoidf(qkv[(size_t)(tl.x + r0) * ld + a.gate_col + h]);
         if (r1 < n) i1 *= sigmoidf(qkv[(size_t)(tl.x + r1) * ld + a.gate_col + h]);
@@ -238,7 +253,17 @@ attention_one_kernel(const cmlb200_attn a, const float* __restrict__ qkv, int ld
     const int* table = a.block_table + (size_t)row_slot[r] * a.table_ld;
 
     float iq = 1.0f, ik = 1.0f;
-    if (a.q_norm || a.k_norm) {
+    __shared__ float head_inv[RM + 1];                 // per-head norms: of this CTA's query heads, then of its key
+    if (a.head_norm) {
+        for (int j = warp; j <= nh; j += ONE_WARPS) {
+            const float* v = j < nh ? row + (h0 + j) * a.dim : row + qw + kh * a.dim;
+            float ss = 0.f;
+            for (int d = lane; d < a.dim; d += 32) ss = fmaf(v[d], v[d], ss);
+            ss = lane_sum(ss);
+            if (lane == 0) head_inv[j < nh ? j : RM] = (j < nh ? a.q_norm : a.k_norm) ? 1.0f / sqrtf(ss / (float)a.dim + a.eps) : 1.0f;
+        }
+        __syncthreads();
+    } else if (a.q_norm || a.k_norm) {
         const float2 ss = block_sum2(a.q_norm ? square_share(row, qw) : 0.f, a.k_norm && rank == 0 ? square_share(row + qw, kw) : 0.f, red);
         if (a.q_norm) iq = 1.0f / sqrtf(ss.x / (float)qw + a.eps);
         if (a.k_norm) ik = 1.0f / sqrtf(ss.y / (float)kw + a.eps);      // used where the row's own key is made: rank 0
@@ -248,7 +273,7 @@ attention_one_kernel(const cmlb200_attn a, const float* __restrict__ qkv, int ld
     for (int i = threadIdx.x; i < RM * dk; i += ONE_THREADS) {
         const int j = i / dk, d = i - j * dk;
         const int c = (h0 + j) * a.dim + d;
-        q_s[i] = (j < nh && d < a.dim) ? row[c] * iq * (a.q_norm ? a.q_norm[c] : 1.0f) * temp * qs : 0.f;
+        q_s[i] = (j < nh && d < a.dim) ? row[c] * (a.head_norm ? head_inv[j] : iq) * (a.q_norm ? a.q_norm[a.head_norm ? d : c] : 1.0f) * temp * qs : 0.f;
     }
     if (rank == 0) {
         const size_t slot = ((size_t)table[p >> shift] << shift) + (p & (a.block_size - 1));
@@ -256,12 +281,12 @@ attention_one_kernel(const cmlb200_attn a, const float* __restrict__ qkv, int ld
         __half* vd = static_cast<__half*>(a.v_pool) + (slot * a.kv_heads + kh) * dv;
         for (int d = threadIdx.x; d < dk; d += ONE_THREADS) {
             const int c = kh * a.dim + d;
-            const __half v = narrow<__half>(d < a.dim ? row[qw + c] * ik * (a.k_norm ? a.k_norm[c] : 1.0f) : 0.f);
+            const __half v = narrow<__half>(d < a.dim ? row[qw + c] * (a.head_norm ? head_inv[RM] : ik) * (a.k_norm ? a.k_norm[a.head_norm ? d : c] : 1.0f) : 0.f);
             k_new[d] = __half2float(v);
             if (pass == 0) kd[d] = v;
         }
         for (int d = threadIdx.x; d < dv; d += ONE_THREADS) {
-            const __half v = narrow<__half>(d < a.vdim ? row[qw + kw + kh * a.vdim + d] : 0.f);
+            const __half v = narrow<__half>(d < a.vdim ? row[qw + (a.keys_as_values ? 0 : kw) + kh * a.vdim + d] : 0.f);
             v_new[d] = __half2float(v);
             if (pass == 0) vd[d] = v;
         }
@@ -277,7 +302,8 @@ attention_one_kernel(const cmlb200_attn a, const float* __restrict__ qkv, int ld
 #pragma unroll
         for (int e = 0; e < 2 * VP; e++) acc[j][e] = 0.f;
     }
-    const int k_lo = (a.window > 0 && a.window <= p) ? p - a.window + 1 : 0;
+    // the keys in sight, numbered from 0: the kept ones, then those from k_lo on
+    const int k_lo = first_key(a, p), kept = min(a.keep, k_lo), skip = k_lo - kept, seen = p - skip;
     const __half* kp = static_cast<const __half*>(a.k_pool) + (size_t)kh * dk;
     const __half* vp = static_cast<const __half*>(a.v_pool) + (size_t)kh * dv;
     const int kstride = a.kv_heads * dk, vstride = a.kv_heads * dv;
@@ -297,10 +323,10 @@ attention_one_kernel(const cmlb200_attn a, const float* __restrict__ qkv, int ld
             else u[k][0] = *reinterpret_cast<const uint32_t*>(src);
         }
     };
-    // cached keys k_lo .. p - 1, 32 per warp and step; a lane scores one key
-    for (int kt = k_lo + (rank * ONE_WARPS + warp) * 32; kt < p; kt += splits * ONE_WARPS * 32) {
-        const int key = kt + lane, count = min(32, p - kt);
-        const int kc = min(key, p - 1);
+    // cached keys, 32 per warp and step; a lane scores one key
+    for (int kt = (rank * ONE_WARPS + warp) * 32; kt < seen; kt += splits * ONE_WARPS * 32) {
+        const int count = min(32, seen - kt), nth = min(kt + lane, seen - 1);
+        const int key = nth + (nth < kept ? 0 : skip), kc = key;
         const int slot = (table[kc >> shift] << shift) + (kc & (a.block_size - 1));
         float s[RM];
 #pragma unroll
@@ -426,12 +452,12 @@ attention_one_kernel(const cmlb200_attn a, const float* __restrict__ qkv, int ld
             } else {
                 x = w_acc[i]; sum = c_l[j]; mx = c_m[j];
             }
-            if (a.sink) {                              // its score is 0 and it carries no value
-                const float mt = fmaxf(mx, 0.f), c = exp2f(mx - mt);
+            if (a.sink) {                              // it carries no value
+                const float sk = sink_score(a, h0 + j) * kLog2e, mt = fmaxf(mx, sk), c = exp2f(mx - mt);
                 x *= c;
-                sum = sum * c + exp2f(-mt);
+                sum = sum * c + exp2f(sk - mt);
             }
-            float v = x / sum;
+            float v = x / sum * out_scale(a);
             if (a.gate_col >= 0) v *= sigmoidf(row[a.gate_col + h0 + j]);
             if (d < a.vdim) out[(size_t)r * out_ld + (h0 + j) * a.vdim + d] = __float2bfloat16_rn(v);
         }
@@ -465,13 +491,14 @@ attention_rows_f32_kernel(const cmlb200_attn a, const float* __restrict__ qkv, i
     const float slope = a.slopes ? a.slopes[h] : 0.f;
     for (int d = threadIdx.x; d < a.dim; d += ROW_THREADS) q_s[d] = row[h * a.dim + d];
     for (int d = threadIdx.x; d < a.vdim; d += ROW_THREADS) acc[d] = 0.f;
-    float m = a.sink ? 0.f : -INFINITY, l = a.sink ? 1.f : 0.f;
-    const int k_lo = (a.window > 0 && a.window <= p) ? p - a.window + 1 : 0;
-    for (int kt = k_lo; kt <= p; kt += ROW_THREADS) {
-        const int n = min(ROW_THREADS, p - kt + 1);
+    float m = a.sink ? sink_score(a, h) : -INFINITY, l = a.sink ? 1.f : 0.f;
+    const int k_lo = first_key(a, p), kept = min(a.keep, k_lo), skip = k_lo - kept, seen = p + 1 - skip;
+    auto key_of = [&](int nth) { return nth + (nth < kept ? 0 : skip); };
+    for (int kt = 0; kt < seen; kt += ROW_THREADS) {
+        const int n = min(ROW_THREADS, seen - kt);
         __syncthreads();                               // the previous chunk's weights are consumed (and q_s is there)
         if ((int)threadIdx.x < n) {
-            const int key = kt + threadIdx.x;
+            const int key = key_of(kt + threadIdx.x);
             slots[threadIdx.x] = table[key / a.block_size] * a.block_size + key % a.block_size;
         }
         __syncthreads();
@@ -480,7 +507,7 @@ attention_rows_f32_kernel(const cmlb200_attn a, const float* __restrict__ qkv, i
             float s = 0.f;
             for (int d = lane; d < a.dim; d += 32) s = fmaf(q_s[d], kr[d], s);
             s = lane_sum(s);
-            if (lane == 0) sc[k] = s * a.scale - slope * (float)(p - kt - k);
+            if (lane == 0) sc[k] = s * a.scale - slope * (float)(p - key_of(kt + k));
         }
         __syncthreads();
         float mx = m;
@@ -497,7 +524,7 @@ attention_rows_f32_kernel(const cmlb200_attn a, const float* __restrict__ qkv, i
             acc[d] = x;
         }
     }
-    const float inv = (a.gate_col >= 0 ? sigmoidf(row[a.gate_col + h]) : 1.0f) / l;
+    const float inv = (a.gate_col >= 0 ? sigmoidf(row[a.gate_col + h]) : 1.0f) * out_scale(a) / l;
     for (int d = threadIdx.x; d < a.vdim; d += ROW_THREADS) out[(size_t)r * out_ld + h * a.vdim + d] = acc[d] * inv;
 }
 
@@ -510,6 +537,8 @@ extern "C" int cmlb200_attn_check_(const cmlb200_attn* a, const char* who) {
                  "%s: head sizes %d (stride %d) / %d (stride %d)", who, a->dim, a->dim_ld, a->vdim, a->vdim_ld);
     CMLB_REQUIRE(a->cache_dtype == CMLB200_DT_F32 || a->cache_dtype == CMLB200_DT_F16, "%s: cache dtype %d", who, a->cache_dtype);
     CMLB_REQUIRE(!a->gate_wide || a->gate_col >= 0, "%s: gate_wide without a gate column", who);
+    CMLB_REQUIRE(a->keep >= 0 && a->chunk >= 0 && (!a->keys_as_values || a->dim == a->vdim), "%s: kept tokens %d, chunk %d, values as keys of %d / %d", who, a->keep,
+                 a->chunk, a->dim, a->vdim);
     CMLB_REQUIRE(a->k_pool && a->v_pool && a->block_table && a->table_ld > 0, "%s: no cache", who);
     CMLB_REQUIRE(a->block_size > 0 && (a->block_size & (a->block_size - 1)) == 0 && a->block_size % 16 == 0, "%s: block size %d must be a power of two >= 16", who, a->block_size);
     CMLB_REQUIRE((((uintptr_t)a->k_pool | (uintptr_t)a->v_pool) & 15) == 0, "%s: pools must be 16-byte aligned", who);
@@ -554,7 +583,8 @@ extern "C" int cmlb200_attention_one(const cmlb200_attn* a, const float* d_qkv, 
     // few rows: fewer heads per CTA, so that more CTAs share the work (the keys are read again from L2)
     const int group = a->heads / a->kv_heads, rm = group == 1 ? 1 : (group <= 4 || rows * a->kv_heads * 8 < cmlb_num_sms() ? 4 : 8), passes = (group + rm - 1) / rm;
     CMLB_REQUIRE((long long)a->kv_heads * passes <= 65535, "cmlb200_attention_one: too many heads");
-    const int keys = (a->window > 0 && a->window < max_keys) ? a->window : max_keys;
+    const int reach = a->chunk > 0 ? a->chunk : a->window;
+    const int keys = (reach > 0 && reach < max_keys - a->keep) ? reach + a->keep : max_keys;
     const long long base = (long long)rows * a->kv_heads * passes;
     int splits = 1;
     while (splits < 8 && base * splits < 2 * cmlb_num_sms() && keys > splits * ONE_WARPS * 32) splits *= 2;

@@ -54,6 +54,8 @@ struct GemmOut {
     float limit;
     void* y;
     int ldy, n_out;
+    const float* bias;                                 // OUT_F32
+    float cap;
     // OUT_HEADS: columns below key_cols are heads of `dim` in key rows, those behind them heads of `vdim` in y's rows
     __half* keys;
     int key_cols, dim, dim_ld, vdim, vdim_ld, ldk;
@@ -183,9 +185,14 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constant
                     __syncwarp();
                     const int col = n0 + c0 + lane;
                     if (out.form == OUT_F32) {
+                        float bias = out.bias && col < out.n_out ? out.bias[col] : 0.f;
+                        if (out.cap > 0.f) {
+                            for (int j = 0; j < 32; j++) buf[j * 33 + lane] = soft_cap(buf[j * 33 + lane] + bias, out.cap);
+                            bias = 0.f;
+                        }
 #pragma unroll 8
                         for (int j = 0; j < 32; j++)
-                            if (m0 + j < m_end && col < out.n_out) static_cast<float*>(out.y)[(size_t)(m0 + j) * out.ldy + col] = buf[j * 33 + lane];
+                            if (m0 + j < m_end && col < out.n_out) static_cast<float*>(out.y)[(size_t)(m0 + j) * out.ldy + col] = buf[j * 33 + lane] + bias;
                     } else {
                         const bool key = col < out.key_cols;
                         const int c = key ? col : col - out.key_cols, per = key ? out.dim : out.vdim, ldo = key ? out.ldk : out.ldy;
@@ -258,7 +265,7 @@ int gemm_experts(const cmlb200_moe* m, const cmlb200_dense* W, const uint16_t* x
 extern "C" int cmlb200_gemm_dense(const cmlb200_dense* W, const uint16_t* d_x, int ldx, int M, float* d_y, int ldy, void* stream) {
     CMLB_REQUIRE(W && ldy >= W->rows, "cmlb200_gemm_dense: output stride %d", ldy);
     GemmOut out = {};
-    out.form = OUT_F32; out.y = d_y; out.ldy = ldy; out.n_out = W->rows;
+    out.form = OUT_F32; out.y = d_y; out.ldy = ldy; out.n_out = W->rows; out.bias = W->bias; out.cap = W->cap;
     return gemm_entry(W, d_x, ldx, M, M, W->rows, out, GemmExperts{}, "cmlb200_gemm_dense", stream);
 }
 

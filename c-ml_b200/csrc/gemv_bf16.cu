@@ -26,7 +26,7 @@ struct GemvExperts {
 template <int RT, int NB, bool GLU, bool EXPERT>
 __global__ void __launch_bounds__(GV_WARPS * 32)
 gemv_bf16_kernel(const __nv_bfloat16* __restrict__ W, int ldw, const __nv_bfloat16* __restrict__ x, int ldx, int M, int N, int K, int act,
-                 float limit, void* __restrict__ y, int ldy, const GemvExperts ex) {
+                 float limit, const float* __restrict__ bias, float cap, void* __restrict__ y, int ldy, const GemvExperts ex) {
     __shared__ float part[GV_WARPS][RT * 16][NB * 8 + 1];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, t = lane & 3;
     const int n0 = blockIdx.x * RT * 16;
@@ -120,6 +120,8 @@ gemv_bf16_kernel(const __nv_bfloat16* __restrict__ W, int ldw, const __nv_bfloat
             const int c = blockIdx.x * 16 + n;
             if (c < N) static_cast<__nv_bfloat16*>(y)[(size_t)(first + m) * ldy + c] = __float2bfloat16_rn(glu_act_fast(act, s, s2, limit));
         } else if (n0 + n < N) {
+            if (!EXPERT && bias) s += bias[n0 + n];
+            if (!EXPERT && cap > 0.f) s = soft_cap(s, cap);
             static_cast<float*>(y)[(size_t)(first + m) * ldy + n0 + n] = s;
         }
     }
@@ -130,7 +132,7 @@ int launch_gemv(const cmlb200_dense* W, const uint16_t* x, int ldx, int M, int a
     const dim3 grid((unsigned)((W->rows + RT * 16 - 1) / (RT * 16)));
     const __nv_bfloat16* w = static_cast<const __nv_bfloat16*>(W->w);
     const __nv_bfloat16* xb = reinterpret_cast<const __nv_bfloat16*>(x);
-#define GV_LAUNCH(NB) CMLB_CUDA(launch_chain(gemv_bf16_kernel<RT, NB, GLU, false>, grid, dim3(GV_WARPS * 32), 0, 1, st, w, W->ld, xb, ldx, M, n_out, W->cols, act, 0.f, y, ldy, GemvExperts{}))
+#define GV_LAUNCH(NB) CMLB_CUDA(launch_chain(gemv_bf16_kernel<RT, NB, GLU, false>, grid, dim3(GV_WARPS * 32), 0, 1, st, w, W->ld, xb, ldx, M, n_out, W->cols, act, 0.f, W->bias, W->cap, y, ldy, GemvExperts{}))
     if (M <= 8) GV_LAUNCH(1);
     else if (M <= 16) GV_LAUNCH(2);
     else GV_LAUNCH(4);
@@ -146,7 +148,7 @@ int launch_gemv_experts(const cmlb200_moe* m, const cmlb200_dense* W, const uint
     const __nv_bfloat16* w = static_cast<const __nv_bfloat16*>(W->w);
     const __nv_bfloat16* xb = reinterpret_cast<const __nv_bfloat16*>(x);
     const GemvExperts ex = {*m, per, gather};
-#define GE_LAUNCH(NB) CMLB_CUDA(launch_chain(gemv_bf16_kernel<RT, NB, GLU, true>, grid, dim3(GV_WARPS * 32), 0, 1, st, w, W->ld, xb, ldx, rows, n_out, W->cols, act, limit, y, ldy, ex))
+#define GE_LAUNCH(NB) CMLB_CUDA(launch_chain(gemv_bf16_kernel<RT, NB, GLU, true>, grid, dim3(GV_WARPS * 32), 0, 1, st, w, W->ld, xb, ldx, rows, n_out, W->cols, act, limit, (const float*)nullptr, 0.f, y, ldy, ex))
     if (rows <= 8) GE_LAUNCH(1);
     else if (rows <= 16) GE_LAUNCH(2);
     else GE_LAUNCH(4);

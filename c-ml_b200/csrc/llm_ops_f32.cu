@@ -92,10 +92,10 @@ __global__ void rope_general_kernel(float* __restrict__ x, size_t nvec, int last
     p[1] = x0 * s + x1 * c;
 }
 
-// y[m][n] = sum_k x[m][k] * w[n][k] (+ b[n]); one warp per output element. Row strides ldx, ldw, ldy.
+// y[m][n] = sum_k x[m][k] * w[n][k] (+ b[n]), capped where cap > 0; one warp per output element. Row strides ldx, ldw, ldy.
 __global__ void __launch_bounds__(256)
 linear_f32_kernel(const float* __restrict__ x, int ldx, const float* __restrict__ w, int ldw, const float* __restrict__ bias, int N, int K,
-                  float* __restrict__ y, int ldy) {
+                  float cap, float* __restrict__ y, int ldy) {
     const int n = blockIdx.x * 8 + (threadIdx.x >> 5), m = blockIdx.y, lane = threadIdx.x & 31;
     if (n >= N) return;
     const float* xr = x + (size_t)m * ldx;
@@ -104,7 +104,9 @@ linear_f32_kernel(const float* __restrict__ x, int ldx, const float* __restrict_
     for (int kk = lane; kk < K; kk += 32) acc = fmaf(xr[kk], wr[kk], acc);
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
-    if (lane == 0) y[(size_t)m * ldy + n] = acc + (bias ? bias[n] : 0.f);
+    if (lane != 0) return;
+    acc += bias ? bias[n] : 0.f;
+    y[(size_t)m * ldy + n] = cap > 0.f ? cap * tanhf(acc / cap) : acc;
 }
 
 }  // namespace
@@ -146,7 +148,7 @@ extern "C" int cmlb200_rope_f32(float* d_x, size_t nvec, int last_dim, int dim, 
 // y[M, N] = x[M, K] . w[N, K]^T (+ bias[N]), all fp32.
 extern "C" int cmlb200_linear_f32(const float* d_x, const float* d_w, const float* d_bias, int M, int N, int K, float* d_y, void* stream) {
     CMLB_REQUIRE(d_x && d_w && d_y && M > 0 && N > 0 && K > 0 && M <= 65535, "cmlb200_linear_f32: bad argument");
-    linear_f32_kernel<<<dim3((N + 7) / 8, M), 256, 0, as_stream(stream)>>>(d_x, K, d_w, K, d_bias, N, K, d_y, N);
+    linear_f32_kernel<<<dim3((N + 7) / 8, M), 256, 0, as_stream(stream)>>>(d_x, K, d_w, K, d_bias, N, K, 0.f, d_y, N);
     CMLB_LAUNCH_CHECK();
     return CMLB200_OK;
 }
@@ -156,7 +158,7 @@ extern "C" int cmlb200_linear_dense_f32(const cmlb200_dense* W, const float* d_x
     CMLB_REQUIRE(W && W->w && d_x && d_y && M > 0 && M <= 65535, "cmlb200_linear_dense_f32: bad argument");
     CMLB_REQUIRE(W->dtype == CMLB200_DT_F32 && W->rows > 0 && W->cols > 0 && W->ld >= W->cols && ldx >= W->cols && ldy >= W->rows,
                  "cmlb200_linear_dense_f32: weight [%d, %d], strides %d / %d / %d", W->rows, W->cols, W->ld, ldx, ldy);
-    linear_f32_kernel<<<dim3((W->rows + 7) / 8, M), 256, 0, as_stream(stream)>>>(d_x, ldx, (const float*)W->w, W->ld, nullptr, W->rows, W->cols, d_y, ldy);
+    linear_f32_kernel<<<dim3((W->rows + 7) / 8, M), 256, 0, as_stream(stream)>>>(d_x, ldx, (const float*)W->w, W->ld, W->bias, W->rows, W->cols, W->cap, d_y, ldy);
     CMLB_LAUNCH_CHECK();
     return CMLB200_OK;
 }

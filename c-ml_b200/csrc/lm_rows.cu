@@ -1,11 +1,151 @@
-// Row-wise kernels of the layered models: embedding with a sinusoidal position vector, the fused
-// "norm a sublayer's output, add it to the residual, norm the sum for the next sublayer" step, the
+// Row-wise kernels of the layered models: embedding with a sinusoidal position vector or into residual streams, the
+// fused "norm a sublayer's output, add it to the residual, norm the sum for the next sublayer" step and its like over
+// streams, the
 // query/key norm with query temperature and paged cache append, and the gated activation of the
 // 32-bit path. The residual and every norm are fp32; the operand handed to the next matrix product
 // is bf16 or fp32.
 #include "lm_util.cuh"
 
 namespace {
+
+// x[r][s] = scale * table[token[r]] for every stream s
+template <typename T>
+__global__ void __launch_bounds__(256)
+embed_streams_kernel(const T* __restrict__ table, const int* __restrict__ tokens, float scale, int streams, int width, int vocab, float* __restrict__ x) {
+    dep_wait();
+    dep_trigger();
+    const int r = blockIdx.x;
+    int t = tokens[r];
+    if (t < 0 || t >= vocab) t = 0;
+    const T* src = table + (size_t)t * width;
+    float* dst = x + (size_t)r * streams * width;
+    for (int i = blockIdx.y * 256 + threadIdx.x; i < width; i += gridDim.y * 256) {
+        const float v = widen(src[i]) * scale;
+        for (int s = 0; s < streams; s++) dst[(size_t)s * width + i] = v;
+    }
+}
+
+// One CTA per output row of residual streams. y: the sublayer's output y[r], or the weighted sum of the rows its pairs point
+// at, plus the row itself times self_w (identity experts), plus a further row. With y: x_t <- sum_s mix[s][t] x_s + out[t] y.
+// With w_next: out = norm(sum_s in[s] x_s) * w_next, whose row waits in shared memory between the passes. W: 4 or 1 columns
+// at a time; a thread meets the same columns in every pass, so `out` may be the rows h that identity experts return.
+template <typename TO, int S, int W>
+__global__ void __launch_bounds__(S <= 2 ? 1024 : 512)
+stream_join_kernel(const cmlb200_streams hc, float* __restrict__ x, const float* __restrict__ y, int ldy, int parts, const int* __restrict__ part_pos,
+                   const float* __restrict__ part_w, const float* __restrict__ self_w, const TO* h, const float* __restrict__ add, int ld_add,
+                   const float* __restrict__ w_next, float eps, int width, const int* __restrict__ idx, TO* out, int ldo) {
+    extern __shared__ __align__(16) float row[];
+    __shared__ float red[32];
+    float mix[S][S], to[S], from[S];
+#pragma unroll
+    for (int s = 0; s < S; s++) {
+        const bool have = s < hc.streams;
+        from[s] = have ? (hc.in ? hc.in[s] : 1.f) : 0.f;
+        to[s] = y && have ? hc.out[s] : 0.f;
+#pragma unroll
+        for (int t = 0; t < S; t++) mix[s][t] = y && have && t < hc.streams ? hc.mix[s * hc.streams + t] : 0.f;
+    }
+    dep_wait();
+    dep_trigger();
+    const int r = blockIdx.x;
+    float* xr = x + (size_t)(idx ? idx[r] : r) * hc.streams * width;
+    const float own = self_w ? self_w[r] : 0.f;
+    auto load = [](const float* p, float (&v)[W]) {
+        if constexpr (W == 4) { const float4 q = *reinterpret_cast<const float4*>(p); v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w; }
+        else v[0] = *p;
+    };
+    auto store = [](float* p, const float (&v)[W]) {
+        if constexpr (W == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+        else *p = v[0];
+    };
+    float ss = 0.f;
+    for (int i = threadIdx.x * W; i < width; i += blockDim.x * W) {
+        float v[S][W], u[W];
+#pragma unroll
+        for (int s = 0; s < S; s++)
+            if (s < hc.streams) load(xr + (size_t)s * width + i, v[s]);
+            else
+#pragma unroll
+                for (int e = 0; e < W; e++) v[s][e] = 0.f;
+#pragma unroll
+        for (int e = 0; e < W; e++) u[e] = 0.f;
+        if (y) {
+            float z[W], p[W];
+#pragma unroll
+            for (int e = 0; e < W; e++) z[e] = 0.f;
+            if (parts > 0) {
+#pragma unroll 4
+                for (int k = 0; k < parts; k++) {
+                    const int at = part_pos[r * parts + k];
+                    if (at < 0) continue;
+                    const float w = part_w[r * parts + k];
+                    load(y + (size_t)at * ldy + i, p);
+#pragma unroll
+                    for (int e = 0; e < W; e++) z[e] = fmaf(w, p[e], z[e]);
+                }
+            } else {
+                load(y + (size_t)r * ldy + i, z);
+            }
+            if (own != 0.f)
+#pragma unroll
+                for (int e = 0; e < W; e++) z[e] = fmaf(own, widen(h[(size_t)r * ldo + i + e]), z[e]);
+            if (add) {
+                load(add + (size_t)r * ld_add + i, p);
+#pragma unroll
+                for (int e = 0; e < W; e++) z[e] += p[e];
+            }
+#pragma unroll
+            for (int t = 0; t < S; t++) {
+                if (t >= hc.streams) continue;
+                float n[W];
+#pragma unroll
+                for (int e = 0; e < W; e++) {
+                    n[e] = to[t] * z[e];
+#pragma unroll
+                    for (int s = 0; s < S; s++) n[e] = fmaf(mix[s][t], v[s][e], n[e]);
+                    u[e] = fmaf(from[t], n[e], u[e]);
+                }
+                store(xr + (size_t)t * width + i, n);
+            }
+        } else {
+#pragma unroll
+            for (int s = 0; s < S; s++)
+#pragma unroll
+                for (int e = 0; e < W; e++) u[e] = fmaf(from[s], v[s][e], u[e]);
+        }
+        store(row + i, u);
+#pragma unroll
+        for (int e = 0; e < W; e++) ss = fmaf(u[e], u[e], ss);
+    }
+    if (!w_next) return;
+    const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)width + eps);
+    TO* o = out + (size_t)r * ldo;
+    for (int i = threadIdx.x * W; i < width; i += blockDim.x * W) {
+        float v[W], w[W];
+        load(row + i, v);
+        load(w_next + i, w);
+        TO n[W];
+#pragma unroll
+        for (int e = 0; e < W; e++) n[e] = narrow<TO>(v[e] * inv * w[e]);
+        if constexpr (W == 4 && sizeof(TO) == 2) {
+            uint2 b;
+            memcpy(&b, n, sizeof b);
+            *reinterpret_cast<uint2*>(o + i) = b;
+        } else if constexpr (W == 4) {
+            store(reinterpret_cast<float*>(o + i), reinterpret_cast<const float(&)[W]>(n));
+        } else {
+            o[i] = n[0];
+        }
+    }
+}
+
+__global__ void __launch_bounds__(256)
+pack_columns_kernel(const float* __restrict__ x, int ld, int col, int n, __nv_bfloat16* __restrict__ out, int ldo) {
+    dep_wait();
+    dep_trigger();
+    const float* src = x + (size_t)blockIdx.x * ld + col;
+    for (int i = threadIdx.x; i < n; i += 256) out[(size_t)blockIdx.x * ldo + i] = __float2bfloat16_rn(src[i]);
+}
 
 // x[r] = table[token[r]] (+ the position vector: entry 2i = sin(p f_i), entry 2i + 1 = cos(p f_i),
 // f_i = freq[i], angle and sine in fp32). freq == NULL: no position vector.
@@ -181,13 +321,27 @@ __global__ void __launch_bounds__(256)
 qk_norm_append_kernel(float* __restrict__ qkv, int ld, const int* __restrict__ row_pos, const int* __restrict__ row_slot,
                       const cmlb200_attn a, KV* __restrict__ kpool, KV* __restrict__ vpool) {
     __shared__ float2 red[32];
+    extern __shared__ float inv[];                     // head_norm: of every query head, then of every key head
     dep_wait();
     dep_trigger();
-    const int r = blockIdx.x, qw = a.heads * a.dim, kw = a.kv_heads * a.dim;
+    const int r = blockIdx.x, qw = a.heads * a.dim, kw = a.kv_heads * a.dim, vcol = qw + (a.keys_as_values ? 0 : kw);
     float* row = qkv + (size_t)r * ld;
     const int p = row_pos[r];
     const size_t slot = (size_t)a.block_table[(size_t)row_slot[r] * a.table_ld + p / a.block_size] * a.block_size + p % a.block_size;
-    const float2 ss = block_sum2(square_share(row, qw), square_share(row + qw, kw), red);
+    float2 ss = make_float2(0.f, 0.f);
+    if (a.head_norm) {
+        const int lane = threadIdx.x & 31;
+        for (int j = threadIdx.x >> 5; j < a.heads + a.kv_heads; j += 8) {
+            const float* v = row + (size_t)j * a.dim;
+            float s = 0.f;
+            for (int d = lane; d < a.dim; d += 32) s = fmaf(v[d], v[d], s);
+            s = lane_sum(s);
+            if (lane == 0) inv[j] = (j < a.heads ? a.q_norm : a.k_norm) ? 1.0f / sqrtf(s / (float)a.dim + a.eps) : 1.0f;
+        }
+        __syncthreads();
+    } else {
+        ss = block_sum2(square_share(row, qw), square_share(row + qw, kw), red);
+    }
     const float temp = a.temp_every > 0.f ? 1.0f + a.temp_coef * logf(floorf((float)(p + 1) / a.temp_every) + 1.0f) : 1.0f;
     const float iq = a.q_norm ? 1.0f / sqrtf(ss.x / (float)qw + a.eps) : 1.0f, ik = a.k_norm ? 1.0f / sqrtf(ss.y / (float)kw + a.eps) : 1.0f;
     KV* kd = kpool + slot * a.kv_heads * a.dim_ld;
@@ -196,8 +350,10 @@ qk_norm_append_kernel(float* __restrict__ qkv, int ld, const int* __restrict__ r
 #pragma unroll 4
         for (int i = threadIdx.x * 4; i < qw; i += 1024) {
             float4 v = *reinterpret_cast<const float4*>(row + i);
-            const float4 w = a.q_norm ? *reinterpret_cast<const float4*>(a.q_norm + i) : make_float4(1.f, 1.f, 1.f, 1.f);
-            v.x = v.x * iq * w.x * temp; v.y = v.y * iq * w.y * temp; v.z = v.z * iq * w.z * temp; v.w = v.w * iq * w.w * temp;
+            const int j = a.head_norm ? i / a.dim : 0;
+            const float f = a.head_norm ? inv[j] : iq;
+            const float4 w = a.q_norm ? *reinterpret_cast<const float4*>(a.q_norm + i - j * a.dim) : make_float4(1.f, 1.f, 1.f, 1.f);
+            v.x = v.x * f * w.x * temp; v.y = v.y * f * w.y * temp; v.z = v.z * f * w.z * temp; v.w = v.w * f * w.w * temp;
             *reinterpret_cast<float4*>(row + i) = v;
         }
 #pragma unroll 4
@@ -206,26 +362,30 @@ qk_norm_append_kernel(float* __restrict__ qkv, int ld, const int* __restrict__ r
             float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
             if (d < a.dim) {
                 v = *reinterpret_cast<const float4*>(row + qw + c);
-                const float4 w = a.k_norm ? *reinterpret_cast<const float4*>(a.k_norm + c) : make_float4(1.f, 1.f, 1.f, 1.f);
-                v.x *= ik * w.x; v.y *= ik * w.y; v.z *= ik * w.z; v.w *= ik * w.w;
+                const float4 w = a.k_norm ? *reinterpret_cast<const float4*>(a.k_norm + (a.head_norm ? d : c)) : make_float4(1.f, 1.f, 1.f, 1.f);
+                const float f = a.head_norm ? inv[a.heads + g] : ik;
+                v.x *= f * w.x; v.y *= f * w.y; v.z *= f * w.z; v.w *= f * w.w;
             }
             store4(kd + i, v);
         }
 #pragma unroll 4
         for (int i = threadIdx.x * 4; i < a.kv_heads * a.vdim_ld; i += 1024) {
             const int g = i / a.vdim_ld, d = i - g * a.vdim_ld;
-            store4(vd + i, d < a.vdim ? *reinterpret_cast<const float4*>(row + qw + kw + g * a.vdim + d) : make_float4(0.f, 0.f, 0.f, 0.f));
+            store4(vd + i, d < a.vdim ? *reinterpret_cast<const float4*>(row + vcol + g * a.vdim + d) : make_float4(0.f, 0.f, 0.f, 0.f));
         }
         return;
     }
-    for (int i = threadIdx.x; i < qw; i += 256) row[i] = row[i] * iq * (a.q_norm ? a.q_norm[i] : 1.0f) * temp;
+    for (int i = threadIdx.x; i < qw; i += 256) {
+        const int j = a.head_norm ? i / a.dim : 0;
+        row[i] = row[i] * (a.head_norm ? inv[j] : iq) * (a.q_norm ? a.q_norm[i - j * a.dim] : 1.0f) * temp;
+    }
     for (int i = threadIdx.x; i < a.kv_heads * a.dim_ld; i += 256) {
         const int g = i / a.dim_ld, d = i - g * a.dim_ld, c = g * a.dim + d;
-        kd[i] = narrow<KV>(d < a.dim ? row[qw + c] * ik * (a.k_norm ? a.k_norm[c] : 1.0f) : 0.f);
+        kd[i] = narrow<KV>(d < a.dim ? row[qw + c] * (a.head_norm ? inv[a.heads + g] : ik) * (a.k_norm ? a.k_norm[a.head_norm ? d : c] : 1.0f) : 0.f);
     }
     for (int i = threadIdx.x; i < a.kv_heads * a.vdim_ld; i += 256) {
         const int g = i / a.vdim_ld, d = i - g * a.vdim_ld;
-        vd[i] = narrow<KV>(d < a.vdim ? row[qw + kw + g * a.vdim + d] : 0.f);
+        vd[i] = narrow<KV>(d < a.vdim ? row[vcol + g * a.vdim + d] : 0.f);
     }
 }
 
@@ -312,6 +472,57 @@ extern "C" int cmlb200_residual_add(float* d_x, const float* d_y, int ldy, const
     return launch_residual(d_x, d_y, ldy, parts, d_w_post, nullptr, eps, rows, dim, nullptr, d_out, out_dtype, ldo, 1, as_stream(stream));
 }
 
+extern "C" int cmlb200_embed_streams(const void* d_table, int dtype, const int* d_tokens, float scale, int streams, int rows, int width, int vocab,
+                                     float* d_x, void* stream) {
+    CMLB_REQUIRE(d_table && d_tokens && d_x && streams > 0 && rows > 0 && width > 0 && vocab > 0, "cmlb200_embed_streams: bad argument");
+    CMLB_REQUIRE(dtype == CMLB200_DT_F32 || dtype == CMLB200_DT_BF16, "cmlb200_embed_streams: dtype %d", dtype);
+    const dim3 grid(rows, rows < 64 ? (width + 511) / 512 : 1);
+#define ES_LAUNCH(T) CMLB_CUDA(launch_chain(embed_streams_kernel<T>, grid, dim3(256), 0, 1, as_stream(stream), (const T*)d_table, d_tokens, scale, streams, width, vocab, d_x))
+    if (dtype == CMLB200_DT_BF16) ES_LAUNCH(__nv_bfloat16);
+    else ES_LAUNCH(float);
+#undef ES_LAUNCH
+    return CMLB200_OK;
+}
+
+extern "C" int cmlb200_stream_join(const cmlb200_streams* hc, float* d_x, const float* d_y, int ldy, const cmlb200_join* j, const float* d_w_next, float eps,
+                                   int rows, int width, const int* d_row_idx, void* d_out, int out_dtype, int ldo, void* stream) {
+    CMLB_REQUIRE(hc && d_x && rows > 0 && width > 0 && (d_y || d_w_next), "cmlb200_stream_join: bad argument");
+    CMLB_REQUIRE(hc->streams > 0 && hc->streams <= 8 && (!d_y || (hc->mix && hc->out)), "cmlb200_stream_join: %d streams", hc->streams);
+    CMLB_REQUIRE(!d_w_next || (d_out && ldo >= width), "cmlb200_stream_join: no output for the normed rows");
+    CMLB_REQUIRE(!(d_y && d_row_idx) && (!d_y || ldy >= width) && (!j || d_y), "cmlb200_stream_join: a row list goes with the norm-only form");
+    CMLB_REQUIRE(out_dtype == CMLB200_DT_F32 || out_dtype == CMLB200_DT_BF16, "cmlb200_stream_join: dtype %d", out_dtype);
+    const cmlb200_moe* parts = j ? j->parts : nullptr;
+    const bool self = parts && parts->identity > 0;
+    CMLB_REQUIRE(!parts || (parts->top > 0 && parts->pos && parts->weight), "cmlb200_stream_join: parts without rows");
+    CMLB_REQUIRE(!self || (j->h && parts->self && ldo >= width), "cmlb200_stream_join: identity experts without their rows");
+    CMLB_REQUIRE(!j || !j->add || j->ld_add >= width, "cmlb200_stream_join: stride %d", j->ld_add);
+    const size_t smem = (size_t)((width + 3) / 4) * 16;
+    CMLB_REQUIRE(smem <= 200 * 1024, "cmlb200_stream_join: rows of %d elements do not fit shared memory", width);
+    const void *h = self ? j->h : nullptr, *add = j ? j->add : nullptr;
+    const int ld_add = j ? j->ld_add : 0;
+    const bool vec = width % 4 == 0 && (!d_y || ldy % 4 == 0) && (!d_w_next || ldo % 4 == 0) && ld_add % 4 == 0 &&
+                     (((uintptr_t)d_x | (uintptr_t)d_y | (uintptr_t)d_w_next | (uintptr_t)d_out | (uintptr_t)add) & 15) == 0;
+    int threads = 256;
+    if (rows <= 2 * cmlb_num_sms()) while (threads < 1024 && threads * 4 < width) threads *= 2;
+    if (hc->streams > 2 && threads > 512) threads = 512;               // registers
+    static size_t attr[12][kMaxDevices] = {};
+#define SJ_LAUNCH(TO, S, W, slot)                                                                                                        do {                                                                                                                                    auto kern = stream_join_kernel<TO, S, W>;                                                                                           CMLB_CUDA(cmlb_ensure_smem(kern, smem, attr[slot]));                                                                                CMLB_CUDA(launch_chain(kern, dim3(rows), dim3(threads), smem, 1, as_stream(stream), *hc, d_x, d_y, ldy, parts ? parts->top : 0,                                (const int*)(parts ? parts->pos : nullptr), (const float*)(parts ? parts->weight : nullptr),                                         (const float*)(self ? parts->self : nullptr), (const TO*)h, (const float*)add, ld_add, d_w_next, eps, width, d_row_idx,                                (TO*)d_out, ldo));                                                                                       } while (0)
+#define SJ_WIDTH(TO, S, slot) do { if (vec) SJ_LAUNCH(TO, S, 4, slot); else SJ_LAUNCH(TO, S, 1, slot + 1); } while (0)
+#define SJ_STREAMS(TO, slot) do { if (hc->streams <= 2) SJ_WIDTH(TO, 2, slot); else if (hc->streams <= 4) SJ_WIDTH(TO, 4, slot + 2); else SJ_WIDTH(TO, 8, slot + 4); } while (0)
+    if (out_dtype == CMLB200_DT_BF16) SJ_STREAMS(__nv_bfloat16, 0);
+    else SJ_STREAMS(float, 6);
+#undef SJ_STREAMS
+#undef SJ_WIDTH
+#undef SJ_LAUNCH
+    return CMLB200_OK;
+}
+
+extern "C" int cmlb200_pack_columns(const float* d_x, int ld, int col, int n, int rows, uint16_t* d_out_bf16, int ldo, void* stream) {
+    CMLB_REQUIRE(d_x && d_out_bf16 && col >= 0 && n > 0 && rows > 0 && ld >= col + n && ldo >= n, "cmlb200_pack_columns: bad argument");
+    CMLB_CUDA(launch_chain(pack_columns_kernel, dim3(rows), dim3(256), 0, 1, as_stream(stream), d_x, ld, col, n, (__nv_bfloat16*)d_out_bf16, ldo));
+    return CMLB200_OK;
+}
+
 extern "C" int cmlb200_poly_norm(const float* d_z, int ld, int rows, int ff, const float* d_coef, float eps, void* d_f, int out_dtype, int ldf, void* stream) {
     CMLB_REQUIRE(d_z && d_coef && d_f && rows > 0 && ff > 0 && ld >= ff && ldf >= ff, "cmlb200_poly_norm: bad argument");
     CMLB_REQUIRE(out_dtype == CMLB200_DT_F32 || out_dtype == CMLB200_DT_BF16, "cmlb200_poly_norm: dtype %d", out_dtype);
@@ -338,10 +549,12 @@ extern "C" int cmlb200_qk_norm_append(const cmlb200_attn* a, float* d_qkv, int l
     CMLB_REQUIRE(a && d_qkv && d_row_pos && d_row_slot && rows > 0, "cmlb200_qk_norm_append: bad argument");
     const int rc = cmlb200_attn_check_(a, "cmlb200_qk_norm_append");
     if (rc) return rc;
-    CMLB_REQUIRE(ld >= a->heads * a->dim + a->kv_heads * (a->dim + a->vdim), "cmlb200_qk_norm_append: row stride %d", ld);
+    CMLB_REQUIRE(ld >= a->heads * a->dim + a->kv_heads * (a->dim + (a->keys_as_values ? 0 : a->vdim)), "cmlb200_qk_norm_append: row stride %d", ld);
+    const size_t smem = a->head_norm ? (size_t)(a->heads + a->kv_heads) * 4 : 0;
+    CMLB_REQUIRE(smem <= 40 * 1024, "cmlb200_qk_norm_append: %d heads", a->heads);
     cudaStream_t st = as_stream(stream);
     const bool vec = a->dim % 4 == 0 && a->vdim % 4 == 0 && ld % 4 == 0 && (((uintptr_t)d_qkv | (uintptr_t)a->q_norm | (uintptr_t)a->k_norm) & 15) == 0;
-#define QK_LAUNCH(KV, V) CMLB_CUDA(launch_chain(qk_norm_append_kernel<KV, V>, dim3(rows), dim3(256), 0, 1, st, d_qkv, ld, d_row_pos, d_row_slot, *a, (KV*)a->k_pool, (KV*)a->v_pool))
+#define QK_LAUNCH(KV, V) CMLB_CUDA(launch_chain(qk_norm_append_kernel<KV, V>, dim3(rows), dim3(256), smem, 1, st, d_qkv, ld, d_row_pos, d_row_slot, *a, (KV*)a->k_pool, (KV*)a->v_pool))
     if (a->cache_dtype == CMLB200_DT_F32) { if (vec) QK_LAUNCH(float, true); else QK_LAUNCH(float, false); }
     else { if (vec) QK_LAUNCH(__half, true); else QK_LAUNCH(__half, false); }
 #undef QK_LAUNCH

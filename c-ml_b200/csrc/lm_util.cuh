@@ -113,6 +113,8 @@ __device__ __forceinline__ float glu_act_fast(int act, float g, float u, float l
     return g * sigmoid_fast(clamped ? 1.702f * g : (act == CMLB200_ACT_GELU_TANH ? gelu : g)) * u;
 }
 
+__device__ __forceinline__ float soft_cap(float v, float cap) { return cap * tanhf(v / cap); }
+
 // Pieces of the mma.sync kernels.
 constexpr float kLog2e = 1.4426950408889634f;
 __device__ __forceinline__ uint32_t smem_addr(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }

@@ -6,32 +6,78 @@ namespace {
 
 constexpr int ROUTE_WARPS = 8, PLAN_THREADS = 1024;
 
-// One warp, one row: softmax over all experts, then `top` times the largest that is left (the lower index wins a tie).
+// The largest of n values above minus infinity (the lower index wins a tie); one warp, the same answer on every lane.
+__device__ __forceinline__ int warp_arg_max(const float* v, int n) {
+    float best = -INFINITY;
+    int at = -1;
+    for (int e = threadIdx.x & 31; e < n; e += 32)
+        if (v[e] > best) { best = v[e]; at = e; }
+    // order-preserving bits; 0: nothing left on this lane
+    const unsigned b = __float_as_uint(best), key = at < 0 ? 0u : ((b & 0x80000000u) ? ~b : b | 0x80000000u);
+    const unsigned top = __reduce_max_sync(0xffffffffu, key);
+    return (int)min(__reduce_min_sync(0xffffffffu, key == top && at >= 0 ? (unsigned)at : 0xffffffffu), (unsigned)n - 1u);
+}
+
+// Floats of shared memory a row's choice takes: what is chosen by, the scores, the groups' largest and which are open.
+__host__ __device__ inline int route_floats(const cmlb200_moe& m) {
+    const int n = m.experts + m.identity;
+    return n + (m.correction ? n : 0) + 2 * m.groups;
+}
+
+// One warp, one row: softmax over all outputs, then `top` times the largest that is left. With a correction the choice
+// is by score + correction, otherwise by the logits themselves, which have the scores' order.
 __device__ __forceinline__ void route_row(const cmlb200_moe& m, const float* __restrict__ logits, int r, float* z) {
-    const int lane = threadIdx.x & 31;
+    const int lane = threadIdx.x & 31, n = m.experts + m.identity;
+    float* score = m.correction ? z + n : z;                            // without a correction: still logits
     float mx = -INFINITY;
-    for (int e = lane; e < m.experts; e += 32) { const float v = logits[e]; z[e] = v; mx = fmaxf(mx, v); }
+    for (int e = lane; e < n; e += 32) { const float v = logits[e]; z[e] = v; mx = fmaxf(mx, v); }
     mx = lane_max(mx);
     float sum = 0.f;
-    for (int e = lane; e < m.experts; e += 32) sum += expf(z[e] - mx);
+    for (int e = lane; e < n; e += 32) sum += expf(z[e] - mx);
     sum = lane_sum(sum);
-    for (int k = 0; k < m.top; k++) {
-        float best = -INFINITY;
-        int at = -1;
-        for (int e = lane; e < m.experts; e += 32) {
-            const float v = z[e];
-            if (v > best) { best = v; at = e; }
-        }
-        // order-preserving bits; 0: nothing left on this lane
-        const unsigned b = __float_as_uint(best), key = at < 0 ? 0u : ((b & 0x80000000u) ? ~b : b | 0x80000000u);
-        const unsigned top = __reduce_max_sync(0xffffffffu, key);
-        const int win = (int)min(__reduce_min_sync(0xffffffffu, key == top && at >= 0 ? (unsigned)at : 0xffffffffu), (unsigned)m.experts - 1u);
-        if (lane == (win & 31)) {
-            m.ids[r * m.top + k] = win;
-            m.weight[r * m.top + k] = expf(z[win] - mx) / sum;
-            z[win] = -INFINITY;
+    if (m.correction) {
+        for (int e = lane; e < n; e += 32) {
+            score[e] = expf(z[e] - mx) / sum;
+            z[e] = score[e] + m.correction[e];
         }
     }
+    if (m.groups > 0) {
+        float *best = score + n, *open = best + m.groups;
+        const int per = n / m.groups;
+        __syncwarp();
+        for (int g = lane; g < m.groups; g += 32) {
+            best[g] = -INFINITY;
+            open[g] = 0.f;
+            for (int e = g * per; e < (g + 1) * per; e++) best[g] = fmaxf(best[g], z[e]);
+        }
+        for (int k = 0; k < m.keep; k++) {
+            const int win = warp_arg_max(best, m.groups);
+            if (lane == (win & 31)) { best[win] = -INFINITY; open[win] = 1.f; }
+        }
+        __syncwarp();
+        for (int e = lane; e < n; e += 32)
+            if (open[e / per] == 0.f) z[e] = -INFINITY;
+    }
+    float total = 0.f, self = 0.f;
+    for (int k = 0; k < m.top; k++) {
+        const int win = warp_arg_max(z, n);
+        float w = 0.f;
+        if (lane == (win & 31)) {
+            w = m.correction ? score[win] : expf(z[win] - mx) / sum;
+            m.ids[r * m.top + k] = win;
+            m.weight[r * m.top + k] = w;
+            z[win] = -INFINITY;
+        }
+        w = __shfl_sync(0xffffffffu, w, win & 31);
+        total += w;
+        if (win >= m.experts) self += w;
+    }
+    const float f = m.normalize ? m.scale / (total + 1e-20f) : 1.f;
+    if (m.normalize) {
+        __syncwarp();                                                   // other lanes wrote the weights
+        for (int k = lane; k < m.top; k += 32) m.weight[r * m.top + k] *= f;
+    }
+    if (m.identity > 0 && lane == 0) m.self[r] = self * f;
 }
 
 __global__ void __launch_bounds__(ROUTE_WARPS * 32)
@@ -40,7 +86,7 @@ route_rows_kernel(const cmlb200_moe m, const float* __restrict__ logits, int ld,
     dep_wait();
     dep_trigger();
     const int warp = threadIdx.x >> 5, r = blockIdx.x * ROUTE_WARPS + warp;
-    if (r < rows) route_row(m, logits + (size_t)r * ld, r, z + warp * m.experts);
+    if (r < rows) route_row(m, logits + (size_t)r * ld, r, z + warp * route_floats(m));
 }
 
 // One CTA, with a warp per row where it routes. logits given (up to 32 rows): routes the rows first. Then counts, first positions (multiples of `align`), the
@@ -53,12 +99,13 @@ plan_kernel(const cmlb200_moe m, const float* __restrict__ logits, int ld, int r
     dep_trigger();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, pairs = rows * m.top;
     if (logits) {
-        if (warp < rows) route_row(m, logits + (size_t)warp * ld, warp, z + warp * m.experts);
+        if (warp < rows) route_row(m, logits + (size_t)warp * ld, warp, z + warp * route_floats(m));
         __syncthreads();                                                // also orders the choices' global writes for this block
     }
     for (int e = threadIdx.x; e < m.experts; e += blockDim.x) count[e] = 0;
     __syncthreads();
-    for (int p = threadIdx.x; p < pairs; p += blockDim.x) atomicAdd(&count[m.ids[p]], 1);
+    for (int p = threadIdx.x; p < pairs; p += blockDim.x)
+        if (m.ids[p] < m.experts) atomicAdd(&count[m.ids[p]], 1);
     __syncthreads();
     if (warp == 0) {
         int pos = 0, act = 0, til = 0;                                  // positions, chosen experts, tiles so far
@@ -88,7 +135,9 @@ plan_kernel(const cmlb200_moe m, const float* __restrict__ logits, int ld, int r
     }
     __syncthreads();
     for (int p = threadIdx.x; p < pairs; p += blockDim.x) {
-        const int e = m.ids[p], at = atomicAdd(&count[e], 1);
+        const int e = m.ids[p];
+        if (e >= m.experts) { m.pos[p] = -1; continue; }
+        const int at = atomicAdd(&count[e], 1);
         m.pos[p] = at;
         m.src[at] = p / m.top;
         m.expert[at] = e;
@@ -103,7 +152,10 @@ gather_rows_kernel(const cmlb200_moe m, const uint4* __restrict__ x, int ldx, in
     const uint4* s = x + (size_t)blockIdx.x * ldx;
     for (int i = threadIdx.x; i < width; i += 256) {
         const uint4 v = s[i];
-        for (int k = 0; k < m.top; k++) xp[(size_t)m.pos[blockIdx.x * m.top + k] * ldxp + i] = v;
+        for (int k = 0; k < m.top; k++) {
+            const int p = m.pos[blockIdx.x * m.top + k];
+            if (p >= 0) xp[(size_t)p * ldxp + i] = v;
+        }
     }
 }
 
@@ -114,7 +166,7 @@ moe_linear_f32_kernel(const cmlb200_moe m, const float* __restrict__ W, int ldw,
     dep_wait();
     dep_trigger();
     const int p = m.pos[blockIdx.y], n = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-    if (n >= n_out) return;
+    if (n >= n_out || p < 0) return;
     const float* w = W + ((size_t)m.expert[p] * w_rows + n) * ldw;
     const float* xr = x + (size_t)(gather ? (int)blockIdx.y / m.top : p) * ldx;
     float s = 0.f;
@@ -131,15 +183,23 @@ extern "C" long cmlb200_moe_positions(int rows, int top, int experts, int align)
 }
 
 extern "C" int cmlb200_moe_route(const cmlb200_moe* m, const float* d_logits, int ld, int rows, int align, void* stream) {
-    CMLB_REQUIRE(m && d_logits && rows > 0 && align > 0 && m->experts > 0 && m->top > 0 && m->top <= m->experts && ld >= m->experts, "cmlb200_moe_route: bad argument");
+    CMLB_REQUIRE(m && d_logits && rows > 0 && align > 0 && m->experts > 0 && m->top > 0 && m->identity >= 0, "cmlb200_moe_route: bad argument");
+    const int outputs = m->experts + m->identity;
+    CMLB_REQUIRE(m->top <= outputs && ld >= outputs && (m->identity == 0 || m->self), "cmlb200_moe_route: %d of %d outputs, stride %d", m->top, outputs, ld);
+    CMLB_REQUIRE(m->groups == 0 || (m->groups > 0 && outputs % m->groups == 0 && m->keep > 0 && m->keep <= m->groups && m->keep * (outputs / m->groups) >= m->top),
+                 "cmlb200_moe_route: %d of %d groups of %d outputs for %d", m->keep, m->groups, outputs, m->top);
     CMLB_REQUIRE(m->ids && m->weight && m->pos && m->src && m->expert && m->start && m->count && m->active && m->num_active && m->num_tiles, "cmlb200_moe_route: a plan without arrays");
-    CMLB_REQUIRE(m->experts <= 1536 && (long)rows * m->top < (1l << 30), "cmlb200_moe_route: %d experts", m->experts);
+    CMLB_REQUIRE(outputs <= 1536 && (long)rows * m->top < (1l << 30), "cmlb200_moe_route: %d experts", m->experts);
     cudaStream_t st = as_stream(stream);
     static size_t attr[kMaxDevices] = {};
-    const bool fused = rows <= 32;
-    const size_t row = (size_t)m->experts * 4;
-    if (!fused) CMLB_CUDA(launch_chain(route_rows_kernel, dim3((rows + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(ROUTE_WARPS * 32), ROUTE_WARPS * row, 1, st, *m, d_logits, ld, rows));
-    const size_t smem = fused ? (size_t)rows * row : row;
+    static size_t route_attr[kMaxDevices] = {};
+    const size_t row = (size_t)route_floats(*m) * 4, counts = (size_t)m->experts * 4;
+    const bool fused = rows <= 32 && (size_t)rows * row <= 200 * 1024;
+    if (!fused) {
+        CMLB_CUDA(cmlb_ensure_smem(route_rows_kernel, ROUTE_WARPS * row, route_attr));
+        CMLB_CUDA(launch_chain(route_rows_kernel, dim3((rows + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(ROUTE_WARPS * 32), ROUTE_WARPS * row, 1, st, *m, d_logits, ld, rows));
+    }
+    const size_t smem = fused && (size_t)rows * row > counts ? (size_t)rows * row : counts;
     CMLB_CUDA(cmlb_ensure_smem(plan_kernel, smem, attr));
     CMLB_CUDA(launch_chain(plan_kernel, dim3(1), dim3(rows <= 8 ? PLAN_THREADS / 4 : PLAN_THREADS), smem, 1, st, *m, fused ? d_logits : (const float*)nullptr, ld, rows, align));
     return CMLB200_OK;

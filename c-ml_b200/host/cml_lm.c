@@ -75,7 +75,7 @@ static int make_buffers(CMLLanguageModel* lm) {
     if (!lm->cache) return -1;
     /* blocks that every window has passed go back to the pool, so a sequence may outgrow it */
     lm->table_ld = lm->info.window > 0 ? 4 * blocks : blocks;
-    lm->meta_cap = 4 * (R > SMALL_ROWS ? R : SMALL_ROWS) + 4 * (R / 2 + R / TILE_ROWS + SMALL_ROWS + (size_t)lm->opt.max_sequences);
+    lm->meta_cap = 4 * (R > SMALL_ROWS ? R : SMALL_ROWS) + 4 * (R / 2 + R / TILE_ROWS + SMALL_ROWS + 2 * (size_t)lm->opt.max_sequences);
     const size_t table = (size_t)lm->opt.max_sequences * (size_t)lm->table_ld * sizeof(int);
     DEV(cmlb200_stream_create(&lm->stream));
     DEV(cmlb200_host_alloc_pinned((void**)&lm->h_meta, lm->meta_cap * sizeof(int)));
@@ -190,9 +190,9 @@ static int grow_sequence(CMLLanguageModel* lm, int seq, int n) {
     return 0;
 }
 
-/* Blocks that every layer's window has passed go back to the pool. */
+/* Blocks that every layer's window has passed go back to the pool, those of first tokens that stay in sight aside. */
 static void release_passed(CMLLanguageModel* lm, int seq) {
-    if (lm->info.window > 0) cml_paged_cache_release_before(lm->cache, seq, lm->cache->sequences[seq].seq_len - lm->info.window + 1);
+    if (lm->info.window > 0) cml_paged_cache_release_between(lm->cache, seq, lm->info.keep_first, lm->cache->sequences[seq].seq_len - lm->info.window + 1);
 }
 
 /* ---- steps ------------------------------------------------------------------------------------------- */
@@ -240,7 +240,8 @@ static int round_keys(int keys) {
 /* Fills the packed row array from the entries (whose sequences have grown already) and uploads it. */
 static int upload_rows(CMLLanguageModel* lm, const CMLLMEntry* entries, int n, int rows, CMLLMBatch* b, const int** d_want) {
     const int stride = rows <= SMALL_ROWS ? SMALL_ROWS : (lm->opt.max_step_rows + 3) & ~3;
-    int *tok = lm->h_meta, *pos = tok + stride, *slot = pos + stride, *want = slot + stride, *tiles = want + stride;
+    int *tok = lm->h_meta, *pos = tok + stride, *slot = pos + stride, *want = slot + stride, *runs = want + stride;
+    int *tiles = runs + 4 * lm->opt.max_sequences, num_runs = 0;
     int one = 0, one_keys = 0, w = 0, t = 0, short_rows = 0, short_tiles = 0, short_keys = 0, portions = 0;
     for (int i = 0; i < n; i++) {
         const int k = entries[i].num_tokens;
@@ -264,6 +265,7 @@ static int upload_rows(CMLLanguageModel* lm, const CMLLMEntry* entries, int n, i
         }
         for (int k = 0; k < e->num_want; k++) want[w++] = r0 + e->want[k];
         if (len == 1) { if (first > one_keys) one_keys = first; continue; }
+        num_runs++;
         if (len <= TILE_ROWS && first + len > short_keys) short_keys = first + len;
         if (len > TILE_ROWS) { CMLLMPortion p = {r0, len, e->seq, first, t}; lm->portions[portions++] = p; }
         for (int k = 0; k < len; k += TILE_ROWS, ++*tile) {
@@ -273,7 +275,16 @@ static int upload_rows(CMLLanguageModel* lm, const CMLLMEntry* entries, int n, i
             tiles[4 * *tile + 3] = first + k;
         }
     }
-    DEV(cmlb200_memcpy_h2d(lm->d_meta, lm->h_meta, (4 * (size_t)stride + 4 * (size_t)t) * sizeof(int), lm->stream));
+    for (int i = 0, at = 0; i < 2; i++)                    /* portions of one tile, then the longer ones, as their rows lie */
+        for (int k = 0; k < n; k++) {
+            const CMLLMEntry* e = &entries[k];
+            if (e->num_tokens == 1 || (e->num_tokens > TILE_ROWS) != i) continue;
+            const int r[4] = {one + at, e->num_tokens, e->seq, lm->cache->sequences[e->seq].seq_len - e->num_tokens};
+            memcpy(runs, r, sizeof r);
+            runs += 4;
+            at += e->num_tokens;
+        }
+    DEV(cmlb200_memcpy_h2d(lm->d_meta, lm->h_meta, (4 * (size_t)stride + 4 * (size_t)lm->opt.max_sequences + 4 * (size_t)t) * sizeof(int), lm->stream));
     memset(b, 0, sizeof *b);
     b->rows = rows;
     b->one_rows = one;
@@ -288,7 +299,9 @@ static int upload_rows(CMLLanguageModel* lm, const CMLLMEntry* entries, int n, i
     b->d_pos = lm->d_meta + stride;
     b->d_slot = lm->d_meta + 2 * stride;
     *d_want = lm->d_meta + 3 * stride;
-    b->d_tiles = lm->d_meta + 4 * stride;
+    b->d_runs = lm->d_meta + 4 * stride;
+    b->num_runs = num_runs;
+    b->d_tiles = b->d_runs + 4 * lm->opt.max_sequences;
     b->d_table = lm->d_table;
     b->table_ld = lm->table_ld;
     return 0;
@@ -464,7 +477,8 @@ static int blocks_of(const CMLLanguageModel* lm, const CMLSequenceRequest* r) {
     long tokens = (long)r->num_prompt_tokens + r->max_new_tokens;
     if (lm->info.window > 0) {
         const long portion = r->num_prompt_tokens < lm->opt.max_step_rows ? r->num_prompt_tokens : lm->opt.max_step_rows;
-        if (lm->info.window + portion + bs < tokens) tokens = lm->info.window + portion + bs;
+        const long reach = lm->info.window + portion + bs + (lm->info.keep_first ? lm->info.keep_first + bs : 0);
+        if (reach < tokens) tokens = reach;
     }
     return (int)((tokens + bs - 1) / bs);
 }

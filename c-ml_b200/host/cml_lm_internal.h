@@ -23,6 +23,8 @@ typedef struct CMLLMBatch {
     int max_keys;                   /* no single-token row has more cached keys than this */
     const int *d_tokens, *d_pos, *d_slot;
     const int* d_tiles;             /* {first row, rows, slot, position of the first row} each */
+    const int* d_runs;              /* whole portions, the same way, in the order of their rows */
+    int num_runs;
     const int* d_table;             /* [slots][table_ld] block ids */
     int table_ld;
 } CMLLMBatch;
@@ -30,6 +32,7 @@ typedef struct CMLLMBatch {
 typedef struct CMLLMInfo {
     int vocab;
     int window;                     /* no layer looks further back than this many tokens (itself included); 0: no bound */
+    int keep_first;                 /* except at a sequence's first tokens, up to this many */
     CMLTokenizer* tokenizer;
 } CMLLMInfo;
 

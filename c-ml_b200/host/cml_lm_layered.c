@@ -1,19 +1,25 @@
 /* Decoder-only models described layer by layer in config.json and stored as safetensors. A design is a row
- * of switches (LayeredDesign below); sizes, windows, scales and the order of layers come from the file.
+ * of switches (LayeredDesign); sizes, windows, scales and the order of layers come from the file.
  *
- *   config.json     architecture, vocab, width, norm.eps, layers: [{type, mixer, mlp, weights_of?}]
- *   mixer           grouped heads: heads, kv_heads, dim, vdim, scale, mask.size, q_temp {coef, every}
+ *   config.json     architecture, vocab, width, norm.eps, layers: [{type, mixer, mlp, weights_of?}]; designs with streams also
+ *                   streams, embedding.scale and logit_softcap
+ *   mixer           grouped heads: heads, kv_heads, dim, vdim, scale, mask {size, keep_first}, q_temp {coef, every}
  *                   latents: heads, dim, rot_dim, vdim, kv_rank, scale, mask.size, rot {base, dims, scaling {factor,
  *                   original, fast, slow}}, kv_from (the layer whose cache this one reads)
- *   mlp             {kind: "dense", ff}, {kind: "moe", expert {ff, limit}, router {experts, top}} or null
+ *                   parallel: left (grouped heads), right (gated delta rule, cml_lm_delta.c), left_scale, right_scale
+ *   mlp             {kind: "dense", ff}, {kind: "moe", expert {ff, limit}, router {experts, top, identity, groups {count, keep},
+ *                   scale}, shared {ff}} or null
  *   weights_of      index of the layer whose tensors this one uses; its cache is its own
  *   tensors         embed, final.norm, head, l<i>.norm1 / norm1b / norm2 / norm2b (as the design has them),
- *                   l<i>.mix.q / k / v / g / o / q.norm / k.norm, or q / dkv / dkv.norm / uk / uv / g / o,
- *                   l<i>.mlp.gate / up / down, up / down / act, or router and e<j>.gate / up / down; linear weights [out, in]
+ *                   l<i>.mix.q / k / v / g / o / q.norm / k.norm / sink and biases .b, the same under mix.left and mix.right, or
+ *                   q / dkv / dkv.norm / uk / uv / g / o, l<i>.mlp.gate / up / down, up / down / act, or router, correction,
+ *                   e<j>.gate / up / down and shared.gate / up / down, l<i>.hc1 / hc2 .in / out / mix; linear weights [out, in]
  *
- * On the device a layer's q, k, v and gate rows are one matrix, and the feed-forward's gate and up rows one
- * matrix interleaved in groups of 16 (the epilogues of both products pair them). Between two sublayers runs
- * one kernel: norm of the finished sublayer's output, residual add, norm for the next one. The residual, norms,
+ * On the device all of a layer's projections of its input are one matrix, and the feed-forward's gate and up rows one
+ * matrix interleaved in groups of 16 (the epilogues of both products pair them). Two mixers side by side leave their
+ * outputs, scaled, in neighbouring columns, which one output matrix takes. Between two sublayers runs
+ * one kernel: norm of the finished sublayer's output, residual add, norm for the next one; with streams, the join into
+ * all of them, what the next sublayer reads, and its norm. The residual, norms,
  * scores and weights are fp32; in the bfloat16 form matrix operands are bf16 and cached keys, values and latents
  * fp16. Up to 32 rows a step streams its weights through the decode product, above that tcgen05 tiles.
  *
@@ -25,96 +31,31 @@
 #include <stdlib.h>
 #include <string.h>
 
-#include "cml_lm_internal.h"
-#include "cml_safetensors.h"
+#include "cml_lm_layered.h"
 
-#define SKINNY_ROWS 32
 #define MAX_LAYERS 4096
-#define EXPERT_ROWS 128            /* row tile of the experts' tensor-core product */
 #define EXPAND_KEYS 65536          /* keys the scratch cache of long portions holds at most (CMLB200_EXPAND_KEYS: another number) */
-#define DEV(call) do { if (CML_DEV_FAIL((call), __func__)) return -1; } while (0)
-
-typedef struct MixerKind {
-    const char* type;
-    int latent;                  /* latent attention; 0: grouped heads */
-    int wide_gate;               /* latent: sigmoid gate on every element of the heads' output */
-} MixerKind;
-
-typedef enum { FF_GATED, FF_POLY_NORM } DenseForm;
-
-typedef struct LayeredDesign {
-    const char* architecture;
-    MixerKind mixers[2];
-    double position_base;        /* > 0: sinusoidal position vector with that base added to the embedding */
-    int input_norms;             /* each sublayer reads a normed residual; 0: the residual itself */
-    const char* output_norms[2]; /* tensors of the norm on each sublayer's output before it joins the residual; NULL: none */
-    int wide_qk_norm;            /* RMS norm of the whole q and k projections */
-    int linear_bias;             /* scores lose slope_h * distance, slope_h = 2^(-8 (h + 1) / heads) */
-    int sink;                    /* one added to the softmax denominator */
-    int head_gate;               /* sigmoid gate per head */
-    DenseForm dense;             /* of a dense feed-forward */
-    int act;                     /* of a gated feed-forward, or of the experts */
-    int experts;                 /* feed-forwards of experts are known */
-} LayeredDesign;
 
 static const LayeredDesign kDesigns[] = {
-    {"Rarolorn", {{"attention", 0, 0}}, 10000.0, 1, {"norm1b", "norm2b"}, 1, 1, 1, 1, FF_GATED, CMLB200_ACT_GELU_TANH, 0},
-    {"Situlorn", {{"latent_attention", 1, 0}, {"latent_attention_2", 1, 1}}, 0.0, 0, {"norm1", "norm2"}, 0, 0, 0, 0, FF_POLY_NORM, CMLB200_ACT_CLAMPED, 1},
+    {.architecture = "Rarolorn",
+     .mixers = {{"attention", MIXER_GROUPED, 0, {.norm = NORM_WIDE, .sink = SINK_ONE, .linear_bias = 1, .head_gate = 1}}},
+     .position_base = 10000.0, .input_norms = 1, .output_norms = {"norm1b", "norm2b"}, .dense = FF_GATED, .act = CMLB200_ACT_GELU_TANH},
+    {.architecture = "Situlorn",
+     .mixers = {{.type = "latent_attention", .form = MIXER_LATENT}, {.type = "latent_attention_2", .form = MIXER_LATENT, .wide_gate = 1}},
+     .output_norms = {"norm1", "norm2"}, .dense = FF_POLY_NORM, .act = CMLB200_ACT_CLAMPED, .experts = EXPERTS_PLAIN},
+    {.architecture = "Lenedra",
+     .mixers = {{"attention", MIXER_GROUPED, 0, {.norm = NORM_HEAD, .linear_bias = 1, .in_bias = 1, .out_bias = 1, .keys_as_values = 1}},
+                {"parallel", MIXER_PARALLEL, 0, {.sink = SINK_LEARNED, .chunked = 1, .in_bias = 1}}},
+     .input_norms = 1, .norm_offset = 1.f, .streams = 1, .dense = FF_GATED, .act = CMLB200_ACT_SILU, .experts = EXPERTS_GROUPED},
 };
-
-typedef struct LayerWeights {    /* device tensors of a layer that owns some */
-    cmlb200_dense wqkvg, wo, wgu, wd;        /* latent layers: q, dkv and g rows; wgu without a gate: the up rows alone */
-    float *norm1, *norm1b, *norm2, *norm2b, *q_norm, *k_norm, *slopes;
-    float *c_norm, *coef;
-    void* wukt;                  /* per head, transposed */
-    cmlb200_dense wukv;          /* all Wuk rows, then all Wuv rows (per head padded to 16); in the 32-bit form Wuv alone */
-    cmlb200_dense router, experts_gu, experts_down;
-} LayerWeights;
-
-typedef struct Layer {
-    int source;                  /* the layer whose weights it uses */
-    int ff;                      /* 0: no feed-forward */
-    int experts, top;            /* 0: a dense feed-forward; ff is an expert's */
-    float limit;
-    const MixerKind* kind;
-    cmlb200_attn attn;
-    cmlb200_latent lat;
-    int kv_from;                 /* the layer whose latents it reads: itself, as a rule */
-    double rot_base, rot_scaling[4];         /* scaling[0]: factor, 0 without */
-    float* freq;
-    LayerWeights w;
-} Layer;
-
-typedef struct Layered {
-    const LayeredDesign* design;
-    int f32, vocab, width, num_layers;
-    float eps;
-    Layer* layers;
-    void* embed;
-    float *freq, *final_norm;
-    cmlb200_dense head;
-    int max_rows, max_sequences, ld_h, ld_qkvg, ld_att, ld_y, ld_f, ld_gu;
-    float *x, *qkvg, *y, *gu;
-    void *h, *att, *f;           /* operands of the matrix products: bf16, or fp32 in the 32-bit form */
-    /* latent layers */
-    int q_rows;                  /* rows whose queries are transformed at a time */
-    void *q, *o;                 /* transformed queries (fp16 or fp32) and weighted latents (bf16 or fp32) */
-    int expand_keys, *expand_table;
-    void *expand_k, *expand_v, *expand_c;
-    int slots, table_ld;
-    /* experts */
-    cmlb200_moe plan;
-    void* xp;
-    float* router;
-    int ld_router;
-} Layered;
-
-static int round_up(int v, int to) { return (v + to - 1) / to * to; }
 
 /* ---- configuration ---------------------------------------------------------------------------------- */
 static int is_object(const CMLJson* j) { return j && j->type == CML_JSON_OBJECT; }
 
-static int read_grouped(const CMLJson* mixer, Layer* l, int index, const LayeredDesign* design) {
+static int grouped_columns(const cmlb200_attn* a) { return a->heads * a->dim + a->kv_heads * (a->dim + (a->keys_as_values ? 0 : a->vdim)); }
+
+static int read_grouped(const CMLJson* mixer, Layer* l, int index) {
+    const GroupedForm* form = &l->kind->grouped;
     const CMLJson *mask = cml_json_get(mixer, "mask"), *temp = cml_json_get(mixer, "q_temp");
     cmlb200_attn* a = &l->attn;
     double scale = 0.0, coef = 0.0, every = 0.0;
@@ -124,15 +65,20 @@ static int read_grouped(const CMLJson* mixer, Layer* l, int index, const Layered
         LOG_ERROR("layer %d: heads, kv_heads, dim, vdim (up to 256) or scale are missing or do not fit", index);
         return -1;
     }
-    if (is_object(mask) && (cml_json_int(mask, "size", &a->window) || a->window <= 0)) { LOG_ERROR("layer %d: mask.size", index); return -1; }
+    int* size = form->chunked ? &a->chunk : &a->window;
+    if (is_object(mask) && (cml_json_int(mask, "size", size) || *size <= 0)) { LOG_ERROR("layer %d: mask.size", index); return -1; }
+    if (!cml_json_int(mask, "keep_first", &a->keep) && a->keep < 0) { LOG_ERROR("layer %d: mask.keep_first", index); return -1; }
+    if (form->keys_as_values && a->dim != a->vdim) { LOG_ERROR("layer %d: values are keys, but vdim %d is not dim %d", index, a->vdim, a->dim); return -1; }
     if (is_object(temp) && (cml_json_double(temp, "coef", &coef) || cml_json_double(temp, "every", &every) || every <= 0.0)) { LOG_ERROR("layer %d: q_temp", index); return -1; }
     a->scale = (float)scale;
     a->temp_coef = (float)coef;
     a->temp_every = (float)every;
-    a->dim_ld = round_up(a->dim, 16);
-    a->vdim_ld = round_up(a->vdim, 16);
-    a->sink = design->sink;
-    a->gate_col = design->head_gate ? a->heads * a->dim + a->kv_heads * (a->dim + a->vdim) : -1;
+    a->dim_ld = lml_round_up(a->dim, 16);
+    a->vdim_ld = lml_round_up(a->vdim, 16);
+    a->sink = form->sink != SINK_NONE;
+    a->keys_as_values = form->keys_as_values;
+    a->head_norm = form->norm == NORM_HEAD;
+    a->gate_col = form->head_gate ? grouped_columns(a) : -1;
     return 0;
 }
 
@@ -161,26 +107,52 @@ static int read_latent(const CMLJson* mixer, Layer* l, int index) {
     if (from && from->type != CML_JSON_NULL && cml_json_int(mixer, "kv_from", &l->kv_from)) { LOG_ERROR("layer %d: kv_from", index); return -1; }
     const int q = a->heads * (a->dim + a->rot_dim), kv = a->rank + a->rot_dim;
     a->scale = (float)scale;
-    a->ld = round_up(kv, 16);
-    a->ld_rank = round_up(a->rank, 64);
+    a->ld = lml_round_up(kv, 16);
+    a->ld_rank = lml_round_up(a->rank, 64);
     a->kv_col = l->kv_from == index ? q : -1;
     a->gate_col = l->kind->wide_gate ? q + (l->kv_from == index ? kv : 0) : -1;
+    return 0;
+}
+
+static int read_parallel(const CMLJson* mixer, Layer* l, int index) {
+    double left = 0.0, right = 0.0;
+    if (cml_json_double(mixer, "left_scale", &left) || cml_json_double(mixer, "right_scale", &right) || left == 0.0 || right == 0.0) {
+        LOG_ERROR("layer %d: left_scale or right_scale is missing or 0", index);
+        return -1;
+    }
+    if (read_grouped(cml_json_get(mixer, "left"), l, index) || cml_delta_read(cml_json_get(mixer, "right"), l, index, grouped_columns(&l->attn))) return -1;
+    l->attn.out_scale = (float)left;
+    l->delta.out_scale = (float)right;
     return 0;
 }
 
 static int read_feed_forward(const CMLJson* mlp, Layer* l, int index, const LayeredDesign* design) {
     const char* kind = cml_json_string(mlp, "kind");
     if (kind && !strcmp(kind, "dense") && !cml_json_int(mlp, "ff", &l->ff) && l->ff > 0) return 0;
-    const CMLJson *expert = cml_json_get(mlp, "expert"), *router = cml_json_get(mlp, "router");
-    double limit = 0.0;
-    if (design->experts && kind && !strcmp(kind, "moe") && !cml_json_int(expert, "ff", &l->ff) && l->ff > 0 && !cml_json_double(expert, "limit", &limit) &&
-        !cml_json_int(router, "experts", &l->experts) && !cml_json_int(router, "top", &l->top) && l->experts > 0 && l->experts <= 1024 && l->top > 0 &&
-        l->top <= l->experts) {
-        l->limit = (float)limit;
-        return 0;
+    const CMLJson *expert = cml_json_get(mlp, "expert"), *router = cml_json_get(mlp, "router"), *groups = cml_json_get(router, "groups");
+    const CMLJson* shared = cml_json_get(mlp, "shared");
+    double limit = 0.0, scale = 1.0;
+    if (design->experts == EXPERTS_NONE || !kind || strcmp(kind, "moe") || cml_json_int(expert, "ff", &l->ff) || l->ff <= 0 ||
+        (design->act == CMLB200_ACT_CLAMPED && cml_json_double(expert, "limit", &limit)) || cml_json_int(router, "experts", &l->experts) ||
+        cml_json_int(router, "top", &l->top) || l->experts <= 0 || l->experts > 1024 || l->top <= 0) {
+        LOG_ERROR("layer %d: feed-forward of kind '%s' is not known or incomplete", index, kind ? kind : "(none)");
+        return -1;
     }
-    LOG_ERROR("layer %d: feed-forward of kind '%s' is not known or incomplete", index, kind ? kind : "(none)");
-    return -1;
+    l->limit = (float)limit;
+    if (design->experts == EXPERTS_GROUPED) {
+        cml_json_int(router, "identity", &l->identity);
+        cml_json_double(router, "scale", &scale);
+        l->router_scale = (float)scale;
+        const int all = l->experts + l->identity;
+        if (l->identity < 0 || l->identity > 1024 || (is_object(groups) && (cml_json_int(groups, "count", &l->groups) || cml_json_int(groups, "keep", &l->keep) || l->groups <= 0 ||
+            all % l->groups || l->keep <= 0 || l->keep > l->groups || (long)l->keep * (all / l->groups) < l->top)) ||
+            (is_object(shared) && (cml_json_int(shared, "ff", &l->shared_ff) || l->shared_ff <= 0))) {
+            LOG_ERROR("layer %d: router.identity, router.groups or shared.ff does not fit", index);
+            return -1;
+        }
+    }
+    if (l->top > l->experts + l->identity) { LOG_ERROR("layer %d: %d of %d experts", index, l->top, l->experts + l->identity); return -1; }
+    return 0;
 }
 
 static int read_layer(const CMLJson* j, Layer* l, int index, const LayeredDesign* design) {
@@ -190,7 +162,8 @@ static int read_layer(const CMLJson* j, Layer* l, int index, const LayeredDesign
         if (type && design->mixers[k].type && !strcmp(type, design->mixers[k].type)) l->kind = &design->mixers[k];
     if (!l->kind) { LOG_ERROR("layer %d: mixer type '%s' is not known to %s", index, type ? type : "(none)", design->architecture); return -1; }
     l->kv_from = index;
-    if (l->kind->latent ? read_latent(mixer, l, index) : read_grouped(mixer, l, index, design)) return -1;
+    if (l->kind->form == MIXER_LATENT ? read_latent(mixer, l, index) : (l->kind->form == MIXER_PARALLEL ? read_parallel(mixer, l, index) : read_grouped(mixer, l, index)))
+        return -1;
     if (is_object(mlp) && read_feed_forward(mlp, l, index, design)) return -1;
     l->source = index;
     int of;
@@ -198,11 +171,18 @@ static int read_layer(const CMLJson* j, Layer* l, int index, const LayeredDesign
     return 0;
 }
 
-static int window_of(const Layer* l) { return l->kind->latent ? l->lat.window : l->attn.window; }
+/* No token sees further back than this, kept first tokens aside; 0: no bound. */
+static int window_of(const Layer* l) {
+    if (l->kind->form == MIXER_LATENT) return l->lat.window;
+    return l->kind->grouped.chunked ? l->attn.chunk : l->attn.window;
+}
 
 static int same_shape(const Layer* a, const Layer* b) {
-    if (a->kind != b->kind || a->ff != b->ff || a->experts != b->experts) return 0;
-    if (a->kind->latent)
+    if (a->kind != b->kind || a->ff != b->ff || a->experts != b->experts || a->identity != b->identity || a->shared_ff != b->shared_ff) return 0;
+    if (a->kind->form == MIXER_PARALLEL && (a->delta.heads != b->delta.heads || a->delta.kv_heads != b->delta.kv_heads || a->delta.dim != b->delta.dim ||
+                                            a->delta.vdim != b->delta.vdim || a->delta.taps != b->delta.taps))
+        return 0;
+    if (a->kind->form == MIXER_LATENT)
         return a->lat.heads == b->lat.heads && a->lat.dim == b->lat.dim && a->lat.rot_dim == b->lat.rot_dim && a->lat.vdim == b->lat.vdim &&
                a->lat.rank == b->lat.rank && (a->lat.kv_col < 0) == (b->lat.kv_col < 0);
     return a->attn.heads == b->attn.heads && a->attn.kv_heads == b->attn.kv_heads && a->attn.dim == b->attn.dim && a->attn.vdim == b->attn.vdim;
@@ -211,9 +191,9 @@ static int same_shape(const Layer* a, const Layer* b) {
 /* A layer that reads another one's cache: an earlier one, which fills its own, with the same latents and rotation. */
 static int check_kv_from(const Layered* m, int i) {
     const Layer* l = &m->layers[i];
-    if (!l->kind->latent || l->kv_from == i) return 0;
+    if (l->kind->form != MIXER_LATENT || l->kv_from == i) return 0;
     const Layer* f = l->kv_from >= 0 && l->kv_from < i ? &m->layers[l->kv_from] : NULL;
-    if (f && f->kind->latent && f->kv_from == l->kv_from && f->lat.rank == l->lat.rank && f->lat.rot_dim == l->lat.rot_dim && f->rot_base == l->rot_base &&
+    if (f && f->kind->form == MIXER_LATENT && f->kv_from == l->kv_from && f->lat.rank == l->lat.rank && f->lat.rot_dim == l->lat.rot_dim && f->rot_base == l->rot_base &&
         !memcmp(f->rot_scaling, l->rot_scaling, sizeof l->rot_scaling))
         return 0;
     LOG_ERROR("layer %d: kv_from does not name an earlier layer with the same latents", i);
@@ -229,6 +209,14 @@ static int read_config(const CMLJson* c, Layered* m) {
         return -1;
     }
     m->eps = (float)eps;
+    if (m->design->streams) {
+        double scale = 1.0, cap = 0.0;
+        if (cml_json_int(c, "streams", &m->streams) || m->streams < 1 || m->streams > 8) { LOG_ERROR("config.json: streams is missing or not 1 .. 8"); return -1; }
+        cml_json_double(cml_json_get(c, "embedding"), "scale", &scale);
+        cml_json_double(c, "logit_softcap", &cap);
+        m->embed_scale = (float)scale;
+        m->cap = (float)cap;
+    }
     m->num_layers = layers->count;
     m->layers = (Layer*)calloc((size_t)m->num_layers, sizeof(Layer));
     if (!m->layers) return -1;
@@ -251,7 +239,7 @@ static float bits_f32(uint32_t u) {
     memcpy(&f, &u, sizeof f);
     return f;
 }
-static float element(const CMLSafetensor* t, size_t i) {
+float lml_element(const CMLSafetensor* t, size_t i) {
     uint16_t h;
     float f;
     if (t->dtype == DTYPE_FLOAT32) { memcpy(&f, (const uint8_t*)t->data + 4 * i, 4); return f; }
@@ -265,18 +253,18 @@ static uint16_t to_bf16(float f) {
     return (uint16_t)((u + 0x7FFFu + ((u >> 16) & 1)) >> 16);
 }
 
-static int find(const CMLSafetensors* st, const char* prefix, const char* name, int rows, int cols, CMLSafetensor* t) {
+int lml_find(const CMLSafetensors* st, const char* prefix, const char* name, int rows, int cols, CMLSafetensor* t) {
     char full[160];
     snprintf(full, sizeof full, "%s%s", prefix, name);
     if (cml_safetensors_find(st, full, t)) { LOG_ERROR("tensor '%s' is missing", full); return -1; }
-    if (t->dtype == DTYPE_INT32 || t->ndim != (cols ? 2 : 1) || t->shape[0] != rows || (cols && t->shape[1] != cols)) {
+    if (t->dtype == DTYPE_INT32 || t->ndim != (cols ? 2 : 1) || (rows < 0 ? t->shape[0] < 1 || t->shape[0] > 65536 : t->shape[0] != rows) || (cols && t->shape[1] != cols)) {
         LOG_ERROR("tensor '%s' has another shape or type than config.json says ([%d, %d] expected)", full, rows, cols);
         return -1;
     }
     return 0;
 }
 
-static int upload(void** dst, const void* src, size_t bytes) {
+int lml_upload(void** dst, const void* src, size_t bytes) {
     if (CML_DEV_FAIL(cmlb200_malloc(dst, bytes), "upload") || CML_DEV_FAIL(cmlb200_memcpy_h2d(*dst, src, bytes, NULL), "upload") ||
         CML_DEV_FAIL(cmlb200_stream_sync(NULL), "upload"))
         return -1;
@@ -303,19 +291,19 @@ static int make_rotation(Layer* l) {
         f[i] = (float)(ramp > 0.0 ? plain / s[0] * ramp + plain * (1.0 - ramp) : plain);
     }
     a->rot_mul = s[0] > 0.0 ? (float)(0.1 * log(s[0]) + 1.0) : 1.0f;
-    const int rc = upload((void**)&l->freq, f, (size_t)(a->rot_dim / 2) * sizeof(float));
+    const int rc = lml_upload((void**)&l->freq, f, (size_t)(a->rot_dim / 2) * sizeof(float));
     free(f);
     a->freq = l->freq;
     return rc;
 }
 
-static int load_vector(const CMLSafetensors* st, const char* prefix, const char* name, int n, float** dst) {
+int lml_load_vector(const CMLSafetensors* st, const char* prefix, const char* name, int n, float offset, float** dst) {
     CMLSafetensor t;
-    if (find(st, prefix, name, n, 0, &t)) return -1;
+    if (lml_find(st, prefix, name, n, 0, &t)) return -1;
     float* v = (float*)malloc((size_t)n * sizeof(float));
     if (!v) return -1;
-    for (int i = 0; i < n; i++) v[i] = element(&t, (size_t)i);
-    const int rc = upload((void**)dst, v, (size_t)n * sizeof(float));
+    for (int i = 0; i < n; i++) v[i] = lml_element(&t, (size_t)i) + offset;
+    const int rc = lml_upload((void**)dst, v, (size_t)n * sizeof(float));
     free(v);
     return rc;
 }
@@ -323,20 +311,19 @@ static int load_vector(const CMLSafetensors* st, const char* prefix, const char*
 static void put_row(const Layered* m, uint8_t* dst, const CMLSafetensor* t, int row, int cols) {
     const size_t at = (size_t)row * (size_t)cols;
     if (!m->f32 && t->dtype == DTYPE_BFLOAT16) memcpy(dst, (const uint8_t*)t->data + 2 * at, (size_t)cols * 2);
-    else if (m->f32) for (int c = 0; c < cols; c++) ((float*)(void*)dst)[c] = element(t, at + (size_t)c);
-    else for (int c = 0; c < cols; c++) ((uint16_t*)(void*)dst)[c] = to_bf16(element(t, at + (size_t)c));
+    else if (m->f32) for (int c = 0; c < cols; c++) ((float*)(void*)dst)[c] = lml_element(t, at + (size_t)c);
+    else for (int c = 0; c < cols; c++) ((uint16_t*)(void*)dst)[c] = to_bf16(lml_element(t, at + (size_t)c));
 }
 
-/* Stacks up to four [rows, cols] tensors; interleave: two of them in turns of 16 rows, each padded to whole groups. */
-static int load_matrix(const Layered* m, const CMLSafetensors* st, const char* prefix, const char* const* names, const int* rows, int parts, int cols,
+int lml_load_matrix(const Layered* m, const CMLSafetensors* st, const char* prefix, const char* const* names, const int* rows, int parts, int cols,
                        int interleave, cmlb200_dense* out) {
     int total = 0;
-    CMLSafetensor t[4];
+    CMLSafetensor t[MAX_PARTS];
     for (int p = 0; p < parts; p++) {
-        if (find(st, prefix, names[p], rows[p], cols, &t[p])) return -1;
-        total += interleave ? round_up(rows[p], 16) : rows[p];
+        if (lml_find(st, prefix, names[p], rows[p], cols, &t[p])) return -1;
+        total += interleave ? lml_round_up(rows[p], 16) : rows[p];
     }
-    const size_t es = m->f32 ? 4 : 2, ld = (size_t)round_up(cols, 64), bytes = (size_t)round_up(total, 16) * ld * es;
+    const size_t es = m->f32 ? 4 : 2, ld = (size_t)lml_round_up(cols, 64), bytes = (size_t)lml_round_up(total, 16) * ld * es;
     uint8_t* host = (uint8_t*)calloc(bytes, 1);
     if (!host) { LOG_ERROR("out of memory for '%s%s'", prefix, names[0]); return -1; }
     int at = 0;
@@ -351,7 +338,7 @@ static int load_matrix(const Layered* m, const CMLSafetensors* st, const char* p
     out->rows = total;
     out->cols = cols;
     out->ld = (int)ld;
-    const int rc = upload(&out->w, host, bytes);
+    const int rc = lml_upload(&out->w, host, bytes);
     free(host);
     return rc;
 }
@@ -360,13 +347,13 @@ static int alloc_matrix(const Layered* m, int rows, int cols, cmlb200_dense* out
     out->dtype = m->f32 ? CMLB200_DT_F32 : CMLB200_DT_BF16;
     out->rows = rows;
     out->cols = cols;
-    out->ld = round_up(cols, 64);
-    *host = (uint8_t*)calloc((size_t)round_up(rows, 16) * (size_t)out->ld, m->f32 ? 4 : 2);
+    out->ld = lml_round_up(cols, 64);
+    *host = (uint8_t*)calloc((size_t)lml_round_up(rows, 16) * (size_t)out->ld, m->f32 ? 4 : 2);
     if (!*host) LOG_ERROR("out of memory for a [%d, %d] weight", rows, cols);
     return *host ? 0 : -1;
 }
 static int upload_matrix(const Layered* m, cmlb200_dense* w, uint8_t* host) {
-    const int rc = upload(&w->w, host, (size_t)round_up(w->rows, 16) * (size_t)w->ld * (m->f32 ? 4 : 2));
+    const int rc = lml_upload(&w->w, host, (size_t)lml_round_up(w->rows, 16) * (size_t)w->ld * (m->f32 ? 4 : 2));
     free(host);
     return rc;
 }
@@ -374,11 +361,12 @@ static int upload_matrix(const Layered* m, cmlb200_dense* w, uint8_t* host) {
 /* The experts' gate and up rows (interleaved as in load_matrix) and their down rows, one expert behind the other. */
 static int load_experts(Layered* m, const CMLSafetensors* st, const char* prefix, Layer* l) {
     LayerWeights* w = &l->w;
-    const int gu = 2 * round_up(l->ff, 16), down = round_up(m->width, 16);
+    const int gu = 2 * lml_round_up(l->ff, 16), down = lml_round_up(m->width, 16);
     const size_t es = m->f32 ? 4 : 2;
     const char* router[1] = {"mlp.router"};
     uint8_t *hg, *hd;
-    if (load_matrix(m, st, prefix, router, &l->experts, 1, m->width, 0, &w->router) || alloc_matrix(m, l->experts * gu, m->width, &w->experts_gu, &hg)) return -1;
+    const int outputs = l->experts + l->identity;
+    if (lml_load_matrix(m, st, prefix, router, &outputs, 1, m->width, 0, &w->router) || alloc_matrix(m, l->experts * gu, m->width, &w->experts_gu, &hg)) return -1;
     if (alloc_matrix(m, l->experts * down, l->ff, &w->experts_down, &hd)) { free(hg); return -1; }
     int rc = 0;
     for (int e = 0; e < l->experts && !rc; e++) {
@@ -387,7 +375,7 @@ static int load_experts(Layered* m, const CMLSafetensors* st, const char* prefix
         snprintf(name[0], sizeof name[0], "mlp.e%d.gate", e);
         snprintf(name[1], sizeof name[1], "mlp.e%d.up", e);
         snprintf(name[2], sizeof name[2], "mlp.e%d.down", e);
-        rc = find(st, prefix, name[0], l->ff, m->width, &t[0]) || find(st, prefix, name[1], l->ff, m->width, &t[1]) || find(st, prefix, name[2], m->width, l->ff, &t[2]);
+        rc = lml_find(st, prefix, name[0], l->ff, m->width, &t[0]) || lml_find(st, prefix, name[1], l->ff, m->width, &t[1]) || lml_find(st, prefix, name[2], m->width, l->ff, &t[2]);
         for (int p = 0; p < 2 && !rc; p++)
             for (int r = 0; r < l->ff; r++)
                 put_row(m, hg + ((size_t)e * gu + (size_t)(r / 16) * 32 + (size_t)(p * 16 + r % 16)) * (size_t)w->experts_gu.ld * es, &t[p], r, m->width);
@@ -395,7 +383,13 @@ static int load_experts(Layered* m, const CMLSafetensors* st, const char* prefix
     }
     if (rc) { free(hg); free(hd); return -1; }
     rc = upload_matrix(m, &w->experts_gu, hg);
-    return upload_matrix(m, &w->experts_down, hd) || rc ? -1 : 0;
+    if (upload_matrix(m, &w->experts_down, hd) || rc) return -1;
+    if (m->design->experts != EXPERTS_GROUPED) return 0;
+    const char *gate_up[2] = {"mlp.shared.gate", "mlp.shared.up"}, *shared_down[1] = {"mlp.shared.down"};
+    const int rows[2] = {l->shared_ff, l->shared_ff};
+    return lml_load_vector(st, prefix, "mlp.correction", outputs, 0.f, &w->correction) ||
+           (l->shared_ff && (lml_load_matrix(m, st, prefix, gate_up, rows, 2, m->width, 1, &w->shared_gu) ||
+                             lml_load_matrix(m, st, prefix, shared_down, &m->width, 1, l->shared_ff, 0, &w->shared_down))) ? -1 : 0;
 }
 
 /* Wuk and Wuv in the forms of the two ways a latent layer attends, or of the 32-bit one. */
@@ -404,8 +398,8 @@ static int load_latent_heads(const Layered* m, const CMLSafetensors* st, const c
     LayerWeights* w = &l->w;
     CMLSafetensor uk, uv;
     const int H = a->heads, D = a->dim, V = a->vdim, R = a->rank;
-    if (find(st, prefix, "mix.uk", H * D, R, &uk) || find(st, prefix, "mix.uv", H * V, R, &uv)) return -1;
-    const int rp = m->f32 ? R : round_up(R, 16), dp = m->f32 ? D : round_up(D, 64);
+    if (lml_find(st, prefix, "mix.uk", H * D, R, &uk) || lml_find(st, prefix, "mix.uv", H * V, R, &uv)) return -1;
+    const int rp = m->f32 ? R : lml_round_up(R, 16), dp = m->f32 ? D : lml_round_up(D, 64);
     const size_t es = m->f32 ? 4 : 2, bytes = (size_t)H * (size_t)rp * (size_t)dp * es;
     uint8_t* t = (uint8_t*)calloc(bytes, 1);
     if (!t) { LOG_ERROR("out of memory for '%smix.uk'", prefix); return -1; }
@@ -413,22 +407,22 @@ static int load_latent_heads(const Layered* m, const CMLSafetensors* st, const c
         for (int d = 0; d < D; d++)
             for (int r = 0; r < R; r++) {
                 const size_t to = ((size_t)h * (size_t)rp + (size_t)r) * (size_t)dp + (size_t)d;
-                const float v = element(&uk, (size_t)(h * D + d) * (size_t)R + (size_t)r);
+                const float v = lml_element(&uk, (size_t)(h * D + d) * (size_t)R + (size_t)r);
                 if (m->f32) ((float*)(void*)t)[to] = v;
                 else ((uint16_t*)(void*)t)[to] = to_bf16(v);
             }
-    int rc = upload(&w->wukt, t, bytes);
+    int rc = lml_upload(&w->wukt, t, bytes);
     free(t);
     if (rc) return -1;
     if (m->f32) {
         float* v = (float*)malloc((size_t)H * (size_t)V * (size_t)R * sizeof(float));
         if (!v) return -1;
         for (int r = 0; r < H * V; r++) put_row(m, (uint8_t*)(v + (size_t)r * (size_t)R), &uv, r, R);
-        rc = upload(&w->wukv.w, v, (size_t)H * (size_t)V * (size_t)R * sizeof(float));
+        rc = lml_upload(&w->wukv.w, v, (size_t)H * (size_t)V * (size_t)R * sizeof(float));
         free(v);
         return rc;
     }
-    const int vp = round_up(V, 16);
+    const int vp = lml_round_up(V, 16);
     uint8_t* host;
     if (alloc_matrix(m, H * (D + vp), R, &w->wukv, &host)) return -1;
     const size_t row = (size_t)w->wukv.ld * es;
@@ -441,35 +435,119 @@ static const uint16_t* value_rows(const Layer* l, const LayerWeights* w) {
     return (const uint16_t*)w->wukv.w + (size_t)(l->lat.heads * l->lat.dim) * (size_t)w->wukv.ld;
 }
 
+/* A bias of the stacked projections: the tensors' where they have one, else zero. */
+static int load_bias(const CMLSafetensors* st, const char* prefix, const char* const* names, const int* rows, int with_bias, cmlb200_dense* w) {
+    float* v = (float*)calloc((size_t)w->rows, sizeof(float));
+    int rc = v ? 0 : -1;
+    for (int p = 0, at = 0; p < with_bias && !rc; at += rows[p++]) {
+        char name[64];
+        CMLSafetensor t;
+        snprintf(name, sizeof name, "%s.b", names[p]);
+        rc = lml_find(st, prefix, name, rows[p], 0, &t);
+        for (int i = 0; i < rows[p] && !rc; i++) v[at + i] = lml_element(&t, (size_t)i);
+    }
+    rc = rc || lml_upload((void**)&w->bias, v, (size_t)w->rows * sizeof(float));
+    free(v);
+    return rc ? -1 : 0;
+}
+
+/* Output matrices of two mixers side by side: [width, left | right]. */
+static int load_outputs(const Layered* m, const CMLSafetensors* st, const char* prefix, int left, int right, cmlb200_dense* out) {
+    CMLSafetensor l, r;
+    uint8_t* host;
+    if (lml_find(st, prefix, "mix.left.o", m->width, left, &l) || lml_find(st, prefix, "mix.right.o", m->width, right, &r) ||
+        alloc_matrix(m, m->width, left + right, out, &host))
+        return -1;
+    const size_t es = m->f32 ? 4 : 2;
+    for (int i = 0; i < m->width; i++) {
+        uint8_t* row = host + (size_t)i * (size_t)out->ld * es;
+        put_row(m, row, &l, i, left);
+        put_row(m, row + (size_t)left * es, &r, i, right);
+    }
+    return upload_matrix(m, out, host);
+}
+
+/* Grouped heads, alone or with the delta rule beside them. */
+static int load_grouped(Layered* m, const CMLSafetensors* st, const char* prefix, Layer* l) {
+    const GroupedForm* form = &l->kind->grouped;
+    const cmlb200_attn* a = &l->attn;
+    const cmlb200_delta* d = &l->delta;
+    LayerWeights* w = &l->w;
+    const int both = l->kind->form == MIXER_PARALLEL;
+    const char* at = both ? "mix.left." : "mix.";
+    char names[MAX_PARTS][32], group[64];
+    const char* parts[MAX_PARTS];
+    int rows[MAX_PARTS], n = 0;
+#define PART(where, name, count) do { snprintf(names[n], sizeof names[n], "%s%s", (where), (name)); parts[n] = names[n]; rows[n++] = (count); } while (0)
+    PART(at, "q", a->heads * a->dim);
+    PART(at, "k", a->kv_heads * a->dim);
+    if (!form->keys_as_values) PART(at, "v", a->kv_heads * a->vdim);
+    const int with_bias = form->in_bias ? n : 0;
+    if (form->head_gate) PART(at, "g", a->heads);
+    if (both) {
+        if (cml_delta_ranks(st, prefix, l, m->width)) return -1;
+        PART("mix.right.", "q", d->kv_heads * d->dim);
+        PART("mix.right.", "k", d->kv_heads * d->dim);
+        PART("mix.right.", "v", d->heads * d->vdim);
+        PART("mix.right.", "b", d->heads);
+        PART("mix.right.", "a1", l->a_rank);
+        PART("mix.right.", "g1", l->g_rank);
+    }
+#undef PART
+    snprintf(group, sizeof group, "%s%s", prefix, at);
+    const int norm_q = form->norm == NORM_HEAD ? a->dim : rows[0], norm_k = form->norm == NORM_HEAD ? a->dim : rows[1];
+    const char* out[1] = {"o"};
+    if ((form->norm != NORM_NONE && (lml_load_vector(st, group, "q.norm", norm_q, 0.f, &w->q_norm) || lml_load_vector(st, group, "k.norm", norm_k, 0.f, &w->k_norm))) ||
+        (form->sink == SINK_LEARNED && lml_load_vector(st, group, "sink", a->heads, 0.f, &w->sinks)) ||
+        lml_load_matrix(m, st, prefix, parts, rows, n, m->width, 0, &w->wqkvg) || (with_bias && load_bias(st, prefix, parts, rows, with_bias, &w->wqkvg)) ||
+        (both ? load_outputs(m, st, prefix, a->heads * a->vdim, d->heads * d->vdim, &w->wo)
+              : lml_load_matrix(m, st, group, out, &m->width, 1, a->heads * a->vdim, 0, &w->wo)) ||
+        (form->out_bias && load_bias(st, group, out, &m->width, 1, &w->wo)) || (both && cml_delta_load(m, st, prefix, l)))
+        return -1;
+    if (!form->linear_bias) return 0;
+    float* s = (float*)malloc((size_t)a->heads * sizeof(float));
+    if (!s) return -1;
+    for (int h = 0; h < a->heads; h++) s[h] = (float)exp2(-8.0 * (h + 1) / a->heads);
+    const int rc = lml_upload((void**)&w->slopes, s, (size_t)a->heads * sizeof(float));
+    free(s);
+    return rc;
+}
+
 static int load_mixer(Layered* m, const CMLSafetensors* st, const char* prefix, Layer* l) {
     LayerWeights* w = &l->w;
     const char* out[1] = {"mix.o"};
     const int out_rows[1] = {m->width};
-    if (l->kind->latent) {
+    if (l->kind->form == MIXER_LATENT) {
         const cmlb200_latent* a = &l->lat;
         const char* proj[3] = {"mix.q"};
         int rows[3] = {a->heads * (a->dim + a->rot_dim)}, parts = 1;
         if (a->kv_col >= 0) { proj[parts] = "mix.dkv"; rows[parts++] = a->rank + a->rot_dim; }
         if (a->gate_col >= 0) { proj[parts] = "mix.g"; rows[parts++] = a->heads * a->vdim; }
-        return (a->kv_col >= 0 && load_vector(st, prefix, "mix.dkv.norm", a->rank, &w->c_norm)) || load_matrix(m, st, prefix, proj, rows, parts, m->width, 0, &w->wqkvg) ||
-               load_latent_heads(m, st, prefix, l) || load_matrix(m, st, prefix, out, out_rows, 1, a->heads * a->vdim, 0, &w->wo) ? -1 : 0;
+        return (a->kv_col >= 0 && lml_load_vector(st, prefix, "mix.dkv.norm", a->rank, 0.f, &w->c_norm)) || lml_load_matrix(m, st, prefix, proj, rows, parts, m->width, 0, &w->wqkvg) ||
+               load_latent_heads(m, st, prefix, l) || lml_load_matrix(m, st, prefix, out, out_rows, 1, a->heads * a->vdim, 0, &w->wo) ? -1 : 0;
     }
-    const cmlb200_attn* a = &l->attn;
-    const char* proj[4] = {"mix.q", "mix.k", "mix.v", "mix.g"};
-    const int proj_rows[4] = {a->heads * a->dim, a->kv_heads * a->dim, a->kv_heads * a->vdim, a->heads};
-    if ((m->design->wide_qk_norm && (load_vector(st, prefix, "mix.q.norm", proj_rows[0], &w->q_norm) || load_vector(st, prefix, "mix.k.norm", proj_rows[1], &w->k_norm))) ||
-        load_matrix(m, st, prefix, proj, proj_rows, m->design->head_gate ? 4 : 3, m->width, 0, &w->wqkvg) ||
-        load_matrix(m, st, prefix, out, out_rows, 1, a->heads * a->vdim, 0, &w->wo))
+    return load_grouped(m, st, prefix, l);
+}
+
+static int load_sublayer(const Layered* m, const CMLSafetensors* st, const char* prefix, int which, LayerWeights* w) {
+    const LayeredDesign* d = m->design;
+    Sublayer* s = &w->sub[which];
+    char name[4][16];
+    snprintf(name[0], sizeof name[0], "norm%d", which + 1);
+    snprintf(name[1], sizeof name[1], "hc%d.in", which + 1);
+    snprintf(name[2], sizeof name[2], "hc%d.out", which + 1);
+    snprintf(name[3], sizeof name[3], "hc%d.mix", which + 1);
+    if ((d->input_norms && lml_load_vector(st, prefix, name[0], m->width, d->norm_offset, &s->norm)) ||
+        (d->output_norms[which] && lml_load_vector(st, prefix, d->output_norms[which], m->width, d->norm_offset, &s->post)))
         return -1;
-    if (m->design->linear_bias) {
-        float* s = (float*)malloc((size_t)a->heads * sizeof(float));
-        if (!s) return -1;
-        for (int h = 0; h < a->heads; h++) s[h] = (float)exp2(-8.0 * (h + 1) / a->heads);
-        const int rc = upload((void**)&w->slopes, s, (size_t)a->heads * sizeof(float));
-        free(s);
-        return rc;
-    }
-    return 0;
+    if (!m->streams) return 0;
+    CMLSafetensor t;
+    if (lml_load_vector(st, prefix, name[1], m->streams, 0.f, &s->in) || lml_load_vector(st, prefix, name[2], m->streams, 0.f, &s->out) ||
+        lml_find(st, prefix, name[3], m->streams, m->streams, &t))
+        return -1;
+    float mix[64];
+    for (int i = 0; i < m->streams * m->streams; i++) mix[i] = lml_element(&t, (size_t)i);
+    return lml_upload((void**)&s->mix, mix, (size_t)(m->streams * m->streams) * sizeof(float));
 }
 
 static int load_layer(Layered* m, const CMLSafetensors* st, int index) {
@@ -479,106 +557,107 @@ static int load_layer(Layered* m, const CMLSafetensors* st, int index) {
     char prefix[32];
     snprintf(prefix, sizeof prefix, "l%d.", index);
     const char *gu[2] = {"mlp.gate", "mlp.up"}, *up[1] = {"mlp.up"}, *down[1] = {"mlp.down"};
-    const int out_rows[1] = {m->width}, ff_rows[2] = {l->ff, l->ff};
-    if ((d->input_norms && load_vector(st, prefix, "norm1", m->width, &w->norm1)) ||
-        (d->output_norms[0] && load_vector(st, prefix, d->output_norms[0], m->width, &w->norm1b)) || load_mixer(m, st, prefix, l))
-        return -1;
+    const int ff_rows[2] = {l->ff, l->ff};
+    if (load_sublayer(m, st, prefix, 0, w) || load_mixer(m, st, prefix, l)) return -1;
     if (!l->ff) return 0;
-    if ((d->input_norms && load_vector(st, prefix, "norm2", m->width, &w->norm2)) ||
-        (d->output_norms[1] && load_vector(st, prefix, d->output_norms[1], m->width, &w->norm2b)))
-        return -1;
+    if (load_sublayer(m, st, prefix, 1, w)) return -1;
     if (l->experts) return load_experts(m, st, prefix, l);
-    if (d->dense == FF_POLY_NORM ? load_matrix(m, st, prefix, up, ff_rows, 1, m->width, 0, &w->wgu) || load_vector(st, prefix, "mlp.act", 4, &w->coef)
-                                 : load_matrix(m, st, prefix, gu, ff_rows, 2, m->width, 1, &w->wgu))
+    if (d->dense == FF_POLY_NORM ? lml_load_matrix(m, st, prefix, up, ff_rows, 1, m->width, 0, &w->wgu) || lml_load_vector(st, prefix, "mlp.act", 4, 0.f, &w->coef)
+                                 : lml_load_matrix(m, st, prefix, gu, ff_rows, 2, m->width, 1, &w->wgu))
         return -1;
-    return load_matrix(m, st, prefix, down, out_rows, 1, l->ff, 0, &w->wd);
+    return lml_load_matrix(m, st, prefix, down, &m->width, 1, l->ff, 0, &w->wd);
 }
 
 static int load_shared(Layered* m, const CMLSafetensors* st) {
     CMLSafetensor t;
     const char* head[1] = {"head"};
     const int head_rows[1] = {m->vocab};
-    if (find(st, "", "embed", m->vocab, m->width, &t)) return -1;
+    if (lml_find(st, "", "embed", m->vocab, m->width, &t)) return -1;
     const size_t row = (size_t)m->width * (m->f32 ? 4 : 2);
     uint8_t* e = (uint8_t*)malloc((size_t)m->vocab * row);
     float* fr = (float*)malloc((size_t)(m->width / 2 + 1) * sizeof(float));
     int rc = e && fr ? 0 : -1;
     for (int i = 0; i < m->vocab && !rc; i++) put_row(m, e + (size_t)i * row, &t, i, m->width);
-    rc = rc || upload(&m->embed, e, (size_t)m->vocab * row);
+    rc = rc || lml_upload(&m->embed, e, (size_t)m->vocab * row);
     if (!rc && m->design->position_base > 0.0) {
         for (int i = 0; i <= m->width / 2; i++) fr[i] = (float)pow(m->design->position_base, -2.0 * i / m->width);
-        rc = upload((void**)&m->freq, fr, (size_t)(m->width / 2 + 1) * sizeof(float));
+        rc = lml_upload((void**)&m->freq, fr, (size_t)(m->width / 2 + 1) * sizeof(float));
     }
     free(e);
     free(fr);
-    return rc || load_vector(st, "", "final.norm", m->width, &m->final_norm) || load_matrix(m, st, "", head, head_rows, 1, m->width, 0, &m->head) ? -1 : 0;
+    rc = rc || lml_load_vector(st, "", "final.norm", m->width, m->design->norm_offset, &m->final_norm) || lml_load_matrix(m, st, "", head, head_rows, 1, m->width, 0, &m->head);
+    m->head.cap = m->cap;
+    return rc ? -1 : 0;
 }
 
 /* ---- activations and caches --------------------------------------------------------------------------- */
-static int zeroed(void** dst, size_t bytes) {
+int lml_zeroed(void** dst, size_t bytes) {
     DEV(cmlb200_malloc(dst, bytes));
     DEV(cmlb200_memset(*dst, 0, bytes, NULL));
     return 0;
 }
 
-static int most(int a, int b) { return a > b ? a : b; }
-
 /* Operand buffers have strides that are multiples of 64 and start out zero: the decode product reads up
  * to the padded width, where its weights are zero. */
 static int make_activations(Layered* m, int rows) {
-    int q = 0, att = 0, ff = 0, z = 0, latent_q = 0, latent_o = 0, experts = 0, top = 0;
+    int q = 0, att = 0, ff = 0, z = 0, latent_q = 0, latent_o = 0, experts = 0, outputs = 0, top = 0, shared = 0;
     long positions = 0, tiles = 0;
     for (int i = 0; i < m->num_layers; i++) {
         const Layer* l = &m->layers[i];
-        q = most(q, m->layers[l->source].w.wqkvg.rows);
-        ff = most(ff, l->ff);
-        if (l->kind->latent) {
+        q = lml_most(q, m->layers[l->source].w.wqkvg.rows);
+        ff = lml_most(ff, l->ff);
+        if (l->kind->form == MIXER_LATENT) {
             const cmlb200_latent* a = &l->lat;
-            att = most(att, a->heads * a->vdim);
-            latent_q = most(latent_q, a->heads * (m->f32 ? a->rank + a->rot_dim : a->ld));
-            latent_o = most(latent_o, a->heads * (m->f32 ? a->rank : a->ld_rank));
+            att = lml_most(att, a->heads * a->vdim);
+            latent_q = lml_most(latent_q, a->heads * (m->f32 ? a->rank + a->rot_dim : a->ld));
+            latent_o = lml_most(latent_o, a->heads * (m->f32 ? a->rank : a->ld_rank));
         } else {
-            att = most(att, l->attn.heads * l->attn.vdim);
+            att = lml_most(att, l->attn.heads * l->attn.vdim + (l->kind->form == MIXER_PARALLEL ? l->delta.heads * l->delta.vdim : 0));
         }
         if (l->experts) {
             const long p = cmlb200_moe_positions(rows, l->top, l->experts, EXPERT_ROWS);
             if (p > positions) positions = p;
             if (p / EXPERT_ROWS + l->experts + 1 > tiles) tiles = p / EXPERT_ROWS + l->experts + 1;
-            experts = most(experts, l->experts);
-            top = most(top, l->top);
+            experts = lml_most(experts, l->experts);
+            outputs = lml_most(outputs, l->experts + l->identity);
+            shared = lml_most(shared, l->shared_ff);
+            top = lml_most(top, l->top);
         } else if (l->ff) {
-            z = most(z, m->design->dense == FF_POLY_NORM ? l->ff : (m->f32 ? 2 * round_up(l->ff, 16) : 0));
+            z = lml_most(z, m->design->dense == FF_POLY_NORM ? l->ff : (m->f32 ? 2 * lml_round_up(l->ff, 16) : 0));
         }
-        if (l->experts && m->f32) z = most(z, 2 * round_up(l->ff, 16));
+        if (l->experts && m->f32) z = lml_most(z, 2 * lml_round_up(lml_most(l->ff, l->shared_ff), 16));
     }
+    ff = lml_most(ff, shared);
     m->max_rows = rows;
-    m->ld_h = round_up(m->width, 64);
-    m->ld_qkvg = round_up(q, 16);
-    m->ld_att = round_up(att, 64);
-    m->ld_y = round_up(m->width, 16);
-    m->ld_f = round_up(ff ? ff : 1, 64);
-    m->ld_gu = round_up(z, 16);
-    m->ld_router = round_up(experts, 16);
+    m->ld_h = lml_round_up(m->width, 64);
+    m->ld_qkvg = lml_round_up(q, 16);
+    m->ld_att = lml_round_up(att, 64);
+    m->ld_y = lml_round_up(m->width, 16);
+    m->ld_f = lml_round_up(ff ? ff : 1, 64);
+    m->ld_gu = lml_round_up(z, 16);
+    m->ld_router = lml_round_up(outputs, 16);
     const size_t R = (size_t)rows, P = (size_t)(positions > rows ? positions : rows), es = m->f32 ? 4 : 2;
     const size_t head = R > 256 ? R : 256;                 /* the head normalises up to 256 rows at once into h */
-    if (zeroed((void**)&m->x, R * (size_t)m->width * 4) || zeroed(&m->h, head * (size_t)m->ld_h * es) || zeroed((void**)&m->qkvg, R * (size_t)m->ld_qkvg * 4) ||
-        zeroed(&m->att, R * (size_t)m->ld_att * es) || zeroed((void**)&m->y, P * (size_t)m->ld_y * 4) || zeroed(&m->f, P * (size_t)m->ld_f * es) ||
-        (z && zeroed((void**)&m->gu, (m->f32 ? P : R) * (size_t)m->ld_gu * 4)))
+    if (lml_zeroed((void**)&m->x, R * (size_t)m->width * (size_t)lml_most(m->streams, 1) * 4) || lml_zeroed(&m->h, head * (size_t)m->ld_h * es) || lml_zeroed((void**)&m->qkvg, R * (size_t)m->ld_qkvg * 4) ||
+        lml_zeroed(&m->att, R * (size_t)m->ld_att * es) || lml_zeroed((void**)&m->y, P * (size_t)m->ld_y * 4) || lml_zeroed(&m->f, P * (size_t)m->ld_f * es) ||
+        (z && lml_zeroed((void**)&m->gu, (m->f32 ? P : R) * (size_t)m->ld_gu * 4)))
         return -1;
     if (latent_q) {
         const long q_rows = (long)m->max_sequences * 64;
         m->q_rows = q_rows < rows ? (int)q_rows : rows;
-        if (zeroed(&m->q, (size_t)m->q_rows * (size_t)latent_q * es) || zeroed(&m->o, (size_t)m->q_rows * (size_t)latent_o * es)) return -1;
+        if (lml_zeroed(&m->q, (size_t)m->q_rows * (size_t)latent_q * es) || lml_zeroed(&m->o, (size_t)m->q_rows * (size_t)latent_o * es)) return -1;
     }
     if (experts) {
         cmlb200_moe* p = &m->plan;
         const size_t pairs = R * (size_t)top * 4, pos = P * 4, per = (size_t)experts * 4;
-        if (zeroed((void**)&m->router, R * (size_t)m->ld_router * 4) || (!m->f32 && zeroed(&m->xp, P * (size_t)m->ld_h * es)) || zeroed((void**)&p->ids, pairs) ||
-            zeroed((void**)&p->weight, pairs) || zeroed((void**)&p->pos, pairs) || zeroed((void**)&p->src, pos) || zeroed((void**)&p->expert, pos) ||
-            zeroed((void**)&p->start, per) || zeroed((void**)&p->count, per) || zeroed((void**)&p->active, per) || zeroed((void**)&p->num_active, 4) ||
-            zeroed((void**)&p->tiles, (size_t)tiles * 16) || zeroed((void**)&p->num_tiles, 4))
+        if (lml_zeroed((void**)&m->router, R * (size_t)m->ld_router * 4) || (!m->f32 && lml_zeroed(&m->xp, P * (size_t)m->ld_h * es)) || lml_zeroed((void**)&p->ids, pairs) ||
+            lml_zeroed((void**)&p->weight, pairs) || lml_zeroed((void**)&p->pos, pairs) || lml_zeroed((void**)&p->src, pos) || lml_zeroed((void**)&p->expert, pos) ||
+            lml_zeroed((void**)&p->start, per) || lml_zeroed((void**)&p->count, per) || lml_zeroed((void**)&p->active, per) || lml_zeroed((void**)&p->num_active, 4) ||
+            lml_zeroed((void**)&p->tiles, (size_t)tiles * 16) || lml_zeroed((void**)&p->num_tiles, 4) || (outputs > experts && lml_zeroed((void**)&p->self, R * 4)) ||
+            (shared && lml_zeroed((void**)&m->y_shared, R * (size_t)m->ld_y * 4)))
             return -1;
     }
+    if (cml_delta_activations(m, rows)) return -1;
     return CML_DEV_FAIL(cmlb200_stream_sync(NULL), "make_activations") ? -1 : 0;
 }
 
@@ -587,21 +666,21 @@ static int make_expansion(Layered* m, int blocks, int block_size, int slots, int
     int k = 0, v = 0, c = 0;
     for (int i = 0; i < m->num_layers; i++) {
         const cmlb200_latent* a = &m->layers[i].lat;
-        if (!m->layers[i].kind->latent) continue;
-        k = most(k, a->heads * round_up(a->dim + a->rot_dim, 16));
-        v = most(v, a->heads * round_up(a->vdim, 16));
-        c = most(c, a->ld_rank);
+        if (m->layers[i].kind->form != MIXER_LATENT) continue;
+        k = lml_most(k, a->heads * lml_round_up(a->dim + a->rot_dim, 16));
+        v = lml_most(v, a->heads * lml_round_up(a->vdim, 16));
+        c = lml_most(c, a->ld_rank);
     }
     if (!k || m->f32) return 0;
     m->slots = slots;
     m->table_ld = table_ld;
     const char* env = getenv("CMLB200_EXPAND_KEYS");
-    int keys = env && atoi(env) > 0 && atoi(env) < (1 << 28) ? round_up(atoi(env), block_size) : EXPAND_KEYS;
+    int keys = env && atoi(env) > 0 && atoi(env) < (1 << 28) ? lml_round_up(atoi(env), block_size) : EXPAND_KEYS;
     if ((long)blocks * block_size < keys) keys = blocks * block_size;
     m->expand_keys = keys;
     const size_t n = (size_t)m->expand_keys;
-    return zeroed(&m->expand_k, n * (size_t)k * 2) || zeroed(&m->expand_v, n * (size_t)v * 2) || zeroed(&m->expand_c, n * (size_t)c * 2) ||
-           zeroed((void**)&m->expand_table, (size_t)slots * (size_t)table_ld * sizeof(int)) ? -1 : 0;
+    return lml_zeroed(&m->expand_k, n * (size_t)k * 2) || lml_zeroed(&m->expand_v, n * (size_t)v * 2) || lml_zeroed(&m->expand_c, n * (size_t)c * 2) ||
+           lml_zeroed((void**)&m->expand_table, (size_t)slots * (size_t)table_ld * sizeof(int)) ? -1 : 0;
 }
 
 static int layered_make_pools(void* model, int blocks, int block_size, int slots, int table_ld) {
@@ -610,7 +689,7 @@ static int layered_make_pools(void* model, int blocks, int block_size, int slots
     for (int i = 0; i < m->num_layers; i++) {
         Layer* l = &m->layers[i];
         const LayerWeights* w = &m->layers[l->source].w;
-        if (l->kind->latent) {
+        if (l->kind->form == MIXER_LATENT) {
             cmlb200_latent* a = &l->lat;
             a->cache_dtype = m->f32 ? CMLB200_DT_F32 : CMLB200_DT_F16;
             a->block_size = block_size;
@@ -618,7 +697,7 @@ static int layered_make_pools(void* model, int blocks, int block_size, int slots
             a->c_norm = w->c_norm;
             a->eps = m->eps;
             if (l->kv_from != i) a->pool = m->layers[l->kv_from].lat.pool;
-            else if (zeroed(&a->pool, tokens * (size_t)a->ld * es)) return -1;
+            else if (lml_zeroed(&a->pool, tokens * (size_t)a->ld * es)) return -1;
             continue;
         }
         cmlb200_attn* a = &l->attn;
@@ -629,7 +708,9 @@ static int layered_make_pools(void* model, int blocks, int block_size, int slots
         a->k_norm = w->k_norm;
         a->eps = m->eps;
         a->slopes = w->slopes;
-        if (zeroed(&a->k_pool, heads * (size_t)a->dim_ld * es) || zeroed(&a->v_pool, heads * (size_t)a->vdim_ld * es)) return -1;
+        a->sinks = w->sinks;
+        if (l->kind->form == MIXER_PARALLEL && cml_delta_make_state(m, l, w, slots)) return -1;
+        if (lml_zeroed(&a->k_pool, heads * (size_t)a->dim_ld * es) || lml_zeroed(&a->v_pool, heads * (size_t)a->vdim_ld * es)) return -1;
     }
     if (make_expansion(m, blocks, block_size, slots, table_ld)) return -1;
     DEV(cmlb200_stream_sync(NULL));
@@ -637,23 +718,46 @@ static int layered_make_pools(void* model, int blocks, int block_size, int slots
 }
 
 /* ---- a step ------------------------------------------------------------------------------------------- */
-static int product(const Layered* m, const cmlb200_dense* w, const void* x, int ldx, int rows, float* y, int ldy, void* st) {
+int lml_product(const Layered* m, const cmlb200_dense* w, const void* x, int ldx, int rows, float* y, int ldy, void* st) {
     if (m->f32) DEV(cmlb200_linear_dense_f32(w, (const float*)x, ldx, rows, y, ldy, st));
     else if (rows <= SKINNY_ROWS) DEV(cmlb200_gemv_dense(w, (const uint16_t*)x, ldx, rows, y, ldy, st));
     else DEV(cmlb200_gemm_dense(w, (const uint16_t*)x, ldx, rows, y, ldy, st));
     return 0;
 }
 
-/* Router, plan, the chosen experts' products; y then holds a row per (row, expert) pair. */
+/* y = Wd (act(gate) * up) of the rows in h */
+static int gated_product(const Layered* m, const cmlb200_dense* gu, const cmlb200_dense* down, int ff, int rows, float* y, void* st) {
+    const int act = m->design->act;
+    if (m->f32) {
+        DEV(cmlb200_linear_dense_f32(gu, (const float*)m->h, m->ld_h, rows, m->gu, m->ld_gu, st));
+        DEV(cmlb200_glu_rows_f32(m->gu, m->ld_gu, rows, ff, act, (float*)m->f, m->ld_f, st));
+    } else if (rows <= SKINNY_ROWS) {
+        DEV(cmlb200_gemv_dense_glu(gu, (const uint16_t*)m->h, m->ld_h, rows, ff, act, (uint16_t*)m->f, m->ld_f, st));
+    } else {
+        DEV(cmlb200_gemm_dense_glu(gu, (const uint16_t*)m->h, m->ld_h, rows, ff, act, (uint16_t*)m->f, m->ld_f, st));
+    }
+    return lml_product(m, down, m->f, m->ld_f, rows, y, m->ld_y, st);
+}
+
+/* Router, plan, the chosen experts' products (and a shared expert's); y then holds a row per (row, expert) pair. */
 static int expert_layer(const Layered* m, const Layer* l, const LayerWeights* w, int rows, cmlb200_moe* plan, void* st) {
     const int act = m->design->act;
     *plan = m->plan;
     plan->experts = l->experts;
     plan->top = l->top;
-    if (product(m, &w->router, m->h, m->ld_h, rows, m->router, m->ld_router, st)) return -1;
+    if (m->design->experts == EXPERTS_GROUPED) {
+        plan->identity = l->identity;
+        plan->groups = l->groups;
+        plan->keep = l->keep;
+        plan->correction = w->correction;
+        plan->normalize = 1;
+        plan->scale = l->router_scale;
+        if (l->shared_ff && gated_product(m, &w->shared_gu, &w->shared_down, l->shared_ff, rows, m->y_shared, st)) return -1;
+    }
+    if (lml_product(m, &w->router, m->h, m->ld_h, rows, m->router, m->ld_router, st)) return -1;
     DEV(cmlb200_moe_route(plan, m->router, m->ld_router, rows, m->f32 || rows <= SKINNY_ROWS ? 1 : EXPERT_ROWS, st));
     if (m->f32) {
-        DEV(cmlb200_moe_linear_f32(plan, &w->experts_gu, (const float*)m->h, m->ld_h, 1, rows, 2 * round_up(l->ff, 16), m->gu, m->ld_gu, st));
+        DEV(cmlb200_moe_linear_f32(plan, &w->experts_gu, (const float*)m->h, m->ld_h, 1, rows, 2 * lml_round_up(l->ff, 16), m->gu, m->ld_gu, st));
         DEV(cmlb200_moe_glu_rows_f32(m->gu, m->ld_gu, rows * l->top, l->ff, act, l->limit, (float*)m->f, m->ld_f, st));
         DEV(cmlb200_moe_linear_f32(plan, &w->experts_down, (const float*)m->f, m->ld_f, 0, rows, m->width, m->y, m->ld_y, st));
     } else if (rows <= SKINNY_ROWS) {
@@ -668,19 +772,10 @@ static int expert_layer(const Layered* m, const Layer* l, const LayerWeights* w,
 }
 
 static int feed_forward(const Layered* m, const Layer* l, const LayerWeights* w, int rows, void* st) {
-    const int act = m->design->act;
-    if (m->design->dense == FF_POLY_NORM) {
-        if (product(m, &w->wgu, m->h, m->ld_h, rows, m->gu, m->ld_gu, st)) return -1;
-        DEV(cmlb200_poly_norm(m->gu, m->ld_gu, rows, l->ff, w->coef, m->eps, m->f, m->f32 ? CMLB200_DT_F32 : CMLB200_DT_BF16, m->ld_f, st));
-    } else if (m->f32) {
-        DEV(cmlb200_linear_dense_f32(&w->wgu, (const float*)m->h, m->ld_h, rows, m->gu, m->ld_gu, st));
-        DEV(cmlb200_glu_rows_f32(m->gu, m->ld_gu, rows, l->ff, act, (float*)m->f, m->ld_f, st));
-    } else if (rows <= SKINNY_ROWS) {
-        DEV(cmlb200_gemv_dense_glu(&w->wgu, (const uint16_t*)m->h, m->ld_h, rows, l->ff, act, (uint16_t*)m->f, m->ld_f, st));
-    } else {
-        DEV(cmlb200_gemm_dense_glu(&w->wgu, (const uint16_t*)m->h, m->ld_h, rows, l->ff, act, (uint16_t*)m->f, m->ld_f, st));
-    }
-    return product(m, &w->wd, m->f, m->ld_f, rows, m->y, m->ld_y, st);
+    if (m->design->dense != FF_POLY_NORM) return gated_product(m, &w->wgu, &w->wd, l->ff, rows, m->y, st);
+    if (lml_product(m, &w->wgu, m->h, m->ld_h, rows, m->gu, m->ld_gu, st)) return -1;
+    DEV(cmlb200_poly_norm(m->gu, m->ld_gu, rows, l->ff, w->coef, m->eps, m->f, m->f32 ? CMLB200_DT_F32 : CMLB200_DT_BF16, m->ld_f, st));
+    return lml_product(m, &w->wd, m->f, m->ld_f, rows, m->y, m->ld_y, st);
 }
 
 /* Rows first .. first + rows - 1 against the latents themselves: queries through Wuk^T, weighted latents through Wuv.
@@ -704,8 +799,8 @@ static int attend_expanded(const Layered* m, const cmlb200_latent* a, const Laye
     s.heads = s.kv_heads = a->heads;
     s.dim = a->dim + a->rot_dim;
     s.vdim = a->vdim;
-    s.dim_ld = round_up(s.dim, 16);
-    s.vdim_ld = round_up(s.vdim, 16);
+    s.dim_ld = lml_round_up(s.dim, 16);
+    s.vdim_ld = lml_round_up(s.vdim, 16);
     s.scale = a->scale;
     s.window = a->window;
     s.gate_col = a->gate_col;
@@ -729,7 +824,7 @@ static int attend_expanded(const Layered* m, const cmlb200_latent* a, const Laye
             list[n][1] = lo;
             list[n][2] = k;
             list[n][3] = keys;
-            keys += round_up(k, a->block_size);
+            keys += lml_round_up(k, a->block_size);
             rows += p->rows;
             tiles += (p->rows + 63) / 64;
         }
@@ -786,7 +881,8 @@ static int attend_latent(const Layered* m, const Layer* l, const LayerWeights* w
 }
 
 static int attend(const Layered* m, const Layer* l, const LayerWeights* w, const CMLLMBatch* b, void* st) {
-    if (l->kind->latent) return attend_latent(m, l, w, b, st);
+    if (l->kind->form == MIXER_PARALLEL && cml_delta_run(m, l, w, b, l->attn.heads * l->attn.vdim, st)) return -1;
+    if (l->kind->form == MIXER_LATENT) return attend_latent(m, l, w, b, st);
     cmlb200_attn a = l->attn;
     a.block_table = b->d_table;
     a.table_ld = b->table_ld;
@@ -804,11 +900,21 @@ static int attend(const Layered* m, const Layer* l, const LayerWeights* w, const
     return 0;
 }
 
-/* A sublayer's output joins the residual; `next`: the norm in front of what reads it next (designs with input norms). */
-static int join(const Layered* m, const float* post, const float* next, const cmlb200_moe* parts, int rows, void* st) {
+/* A sublayer's output joins the residual; `next`: the sublayer that reads it then (NULL: none). parts: y holds a row per pair of that
+ * plan. done NULL: the embedding is all there is. */
+static int join(const Layered* m, const Sublayer* done, const Sublayer* next, const cmlb200_moe* parts, const float* add, int rows, void* st) {
     const int out = m->f32 ? CMLB200_DT_F32 : CMLB200_DT_BF16;
-    if (m->design->input_norms) DEV(cmlb200_residual_norm(m->x, m->y, m->ld_y, post, next, m->eps, rows, m->width, NULL, m->h, out, m->ld_h, st));
-    else DEV(cmlb200_residual_add(m->x, m->y, m->ld_y, parts, post, m->eps, rows, m->width, m->h, out, m->ld_h, st));
+    const float* y = done ? m->y : NULL;
+    const float *post = done ? done->post : NULL, *norm = next ? next->norm : NULL;
+    if (m->streams) {
+        const cmlb200_streams hc = {m->streams, done ? done->mix : NULL, done ? done->out : NULL, next ? next->in : NULL};
+        const cmlb200_join j = {parts, m->h, add, m->ld_y};
+        DEV(cmlb200_stream_join(&hc, m->x, y, m->ld_y, done ? &j : NULL, norm, m->eps, rows, m->width, NULL, m->h, out, m->ld_h, st));
+    } else if (m->design->input_norms) {
+        DEV(cmlb200_residual_norm(m->x, y, m->ld_y, post, norm, m->eps, rows, m->width, NULL, m->h, out, m->ld_h, st));
+    } else {
+        DEV(cmlb200_residual_add(m->x, y, m->ld_y, parts, post, m->eps, rows, m->width, m->h, out, m->ld_h, st));
+    }
     return 0;
 }
 
@@ -816,28 +922,34 @@ static int layered_forward(void* model, const CMLLMBatch* b, void* st) {
     const Layered* m = (const Layered*)model;
     const int rows = b->rows, out = m->f32 ? CMLB200_DT_F32 : CMLB200_DT_BF16;
     if (rows > m->max_rows) { LOG_ERROR("layered_forward: %d rows of %d", rows, m->max_rows); return -1; }
-    DEV(cmlb200_embed_rows(m->embed, out, b->d_tokens, b->d_pos, m->freq, rows, m->width, m->vocab, m->x, st));
-    if (m->design->input_norms) DEV(cmlb200_residual_norm(m->x, NULL, 0, NULL, m->layers[m->layers[0].source].w.norm1, m->eps, rows, m->width, NULL, m->h, out, m->ld_h, st));
-    else DEV(cmlb200_residual_add(m->x, NULL, 0, NULL, NULL, m->eps, rows, m->width, m->h, out, m->ld_h, st));
+    if (m->streams) DEV(cmlb200_embed_streams(m->embed, out, b->d_tokens, m->embed_scale, m->streams, rows, m->width, m->vocab, m->x, st));
+    else DEV(cmlb200_embed_rows(m->embed, out, b->d_tokens, b->d_pos, m->freq, rows, m->width, m->vocab, m->x, st));
+    if (join(m, NULL, &m->layers[m->layers[0].source].w.sub[0], NULL, NULL, rows, st)) return -1;
     for (int i = 0; i < m->num_layers; i++) {
         const Layer* l = &m->layers[i];
         const LayerWeights* w = &m->layers[l->source].w;
-        const float* next = i + 1 < m->num_layers ? m->layers[m->layers[i + 1].source].w.norm1 : NULL;
+        const Sublayer* next = i + 1 < m->num_layers ? &m->layers[m->layers[i + 1].source].w.sub[0] : NULL;
         cmlb200_moe plan;
-        if (product(m, &w->wqkvg, m->h, m->ld_h, rows, m->qkvg, m->ld_qkvg, st) || attend(m, l, w, b, st) ||
-            product(m, &w->wo, m->att, m->ld_att, rows, m->y, m->ld_y, st) || join(m, w->norm1b, l->ff ? w->norm2 : next, NULL, rows, st))
+        if (lml_product(m, &w->wqkvg, m->h, m->ld_h, rows, m->qkvg, m->ld_qkvg, st) || attend(m, l, w, b, st) ||
+            lml_product(m, &w->wo, m->att, m->ld_att, rows, m->y, m->ld_y, st) || join(m, &w->sub[0], l->ff ? &w->sub[1] : next, NULL, NULL, rows, st))
             return -1;
         if (!l->ff) continue;
         if (l->experts ? expert_layer(m, l, w, rows, &plan, st) : feed_forward(m, l, w, rows, st)) return -1;
-        if (join(m, w->norm2b, next, l->experts ? &plan : NULL, rows, st)) return -1;
+        if (join(m, &w->sub[1], next, l->experts ? &plan : NULL, l->shared_ff ? m->y_shared : NULL, rows, st)) return -1;
     }
     return 0;
 }
 
 static int layered_head(void* model, const int* d_rows, int n, float* d_logits, void* st) {
     const Layered* m = (const Layered*)model;
-    DEV(cmlb200_residual_norm(m->x, NULL, 0, NULL, m->final_norm, m->eps, n, m->width, d_rows, m->h, m->f32 ? CMLB200_DT_F32 : CMLB200_DT_BF16, m->ld_h, st));
-    return product(m, &m->head, m->h, m->ld_h, n, d_logits, m->vocab, st);
+    const int out = m->f32 ? CMLB200_DT_F32 : CMLB200_DT_BF16;
+    if (m->streams) {
+        const cmlb200_streams sum = {m->streams, NULL, NULL, NULL};
+        DEV(cmlb200_stream_join(&sum, m->x, NULL, 0, NULL, m->final_norm, m->eps, n, m->width, d_rows, m->h, out, m->ld_h, st));
+    } else {
+        DEV(cmlb200_residual_norm(m->x, NULL, 0, NULL, m->final_norm, m->eps, n, m->width, d_rows, m->h, out, m->ld_h, st));
+    }
+    return lml_product(m, &m->head, m->h, m->ld_h, n, d_logits, m->vocab, st);
 }
 
 static int layered_check(void* model, const CMLLMBatch* b) {
@@ -858,15 +970,17 @@ static void layered_free(void* model) {
     for (int i = 0; m->layers && i < m->num_layers; i++) {
         Layer* l = &m->layers[i];
         LayerWeights* w = &l->w;
-        void* bufs[] = {w->wqkvg.w, w->wo.w, w->wgu.w, w->wd.w, w->norm1, w->norm1b, w->norm2, w->norm2b, w->q_norm, w->k_norm, w->slopes, w->c_norm, w->coef,
-                        w->wukt, w->wukv.w, w->router.w, w->experts_gu.w, w->experts_down.w, l->freq, l->attn.k_pool, l->attn.v_pool,
-                        l->kv_from == i ? l->lat.pool : NULL};
+        const Sublayer *a = &w->sub[0], *b = &w->sub[1];
+        void* bufs[] = {w->wqkvg.w, w->wo.w, w->wgu.w, w->wd.w, a->norm, a->post, a->in, a->out, a->mix, b->norm, b->post, b->in, b->out, b->mix, w->q_norm, w->k_norm,
+                        w->slopes, w->sinks, w->c_norm, w->coef, (void*)w->wqkvg.bias, (void*)w->wo.bias, w->wukt, w->wukv.w, w->router.w, w->experts_gu.w,
+                        w->experts_down.w, w->shared_gu.w, w->shared_down.w, w->correction, w->conv, w->rate, w->dt_bias, w->o_norm, w->wa.w, w->wg.w, l->freq,
+                        l->attn.k_pool, l->attn.v_pool, l->delta.state, l->delta.ring, l->kv_from == i ? l->lat.pool : NULL};
         for (size_t k = 0; k < sizeof bufs / sizeof bufs[0]; k++) cmlb200_free(bufs[k]);
     }
     const cmlb200_moe* p = &m->plan;
     void* bufs[] = {m->embed, m->freq, m->final_norm, m->head.w, m->x, m->qkvg, m->y, m->gu, m->h, m->att, m->f, m->q, m->o, m->expand_table, m->expand_k,
                     m->expand_v, m->expand_c, m->xp, m->router, p->ids, p->weight, p->pos, p->src, p->expert, p->start, p->count, p->active, p->num_active,
-                    p->tiles, p->num_tiles};
+                    p->tiles, p->num_tiles, p->self, m->y_shared, m->dec, m->gate, m->low, m->delta_work};
     for (size_t k = 0; k < sizeof bufs / sizeof bufs[0]; k++) cmlb200_free(bufs[k]);
     free(m->layers);
     free(m);
@@ -887,7 +1001,7 @@ static void* layered_load(const char* path, const CMLJson* config, const CMLLMOp
     int rc = read_config(config, m) || !(st = cml_safetensors_open(file)) || load_shared(m, st);
     for (int i = 0; i < m->num_layers && !rc; i++) {
         if (m->layers[i].source == i) rc = load_layer(m, st, i);
-        if (!rc && m->layers[i].kind->latent) rc = make_rotation(&m->layers[i]);
+        if (!rc && m->layers[i].kind->form == MIXER_LATENT) rc = make_rotation(&m->layers[i]);
     }
     cml_safetensors_close(st);
     if (rc || make_activations(m, options->max_step_rows)) { layered_free(m); return NULL; }
@@ -896,13 +1010,14 @@ static void* layered_load(const char* path, const CMLJson* config, const CMLLMOp
         const int window = window_of(&m->layers[i]);
         if (window <= 0) { info->window = 0; break; }
         if (window > info->window) info->window = window;
+        info->keep_first = lml_most(info->keep_first, m->layers[i].attn.keep);
     }
     return m;
 }
 
 #define LAYERED_CLASS(name) {.architecture = name, .load = layered_load, .free = layered_free, .make_pools = layered_make_pools, .forward = layered_forward, \
                              .head = layered_head, .check = layered_check}
-static const CMLLMClass kLayeredClasses[] = {LAYERED_CLASS("Rarolorn"), LAYERED_CLASS("Situlorn")};
+static const CMLLMClass kLayeredClasses[] = {LAYERED_CLASS("Rarolorn"), LAYERED_CLASS("Situlorn"), LAYERED_CLASS("Lenedra")};
 
 __attribute__((constructor)) static void register_layered(void) {
     for (size_t i = 0; i < sizeof kLayeredClasses / sizeof kLayeredClasses[0]; i++) cml_lm_register(&kLayeredClasses[i]);

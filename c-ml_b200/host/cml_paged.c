@@ -12,7 +12,7 @@
  * cml_paged_kv_cache_create_device makes a cache of bookkeeping alone, for models whose kernels write and
  * read device pools of their own through the block tables (cml_lm.c): blocks are taken with
  * cml_paged_cache_extend and those that every layer's window has passed go back with
- * cml_paged_cache_release_before. */
+ * cml_paged_cache_release_before / _between. */
 #include <math.h>
 #include <pthread.h>
 #include <stdlib.h>
@@ -217,12 +217,15 @@ int cml_paged_cache_extend(CMLPagedKVCache* cache, int seq_id, int num_tokens) {
     return 0;
 }
 
-void cml_paged_cache_release_before(CMLPagedKVCache* cache, int seq_id, int position) {
+void cml_paged_cache_release_before(CMLPagedKVCache* cache, int seq_id, int position) { cml_paged_cache_release_between(cache, seq_id, 0, position); }
+
+void cml_paged_cache_release_between(CMLPagedKVCache* cache, int seq_id, int from, int position) {
     CMLBlockTable* bt = live_sequence(cache, seq_id);
     if (!bt) return;
+    const int first = from > 0 ? (from + cache->block_size - 1) / cache->block_size : 0;
     int last = position / cache->block_size - 1;           /* the last block that ends at or before `position` */
     if (last >= bt->num_blocks) last = bt->num_blocks - 1;
-    for (int i = last; i >= 0 && bt->block_ids[i] >= 0; i--) {
+    for (int i = last; i >= first && bt->block_ids[i] >= 0; i--) {
         cml_paged_cache_free_block(cache, bt->block_ids[i]);
         bt->block_ids[i] = -1;
     }

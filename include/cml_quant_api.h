@@ -323,11 +323,12 @@ int cml_paged_cache_append(CMLPagedKVCache* cache, int seq_id, const float* key,
  * that a model's kernels own (key_data / value_data are NULL; append and cml_paged_gqa_forward refuse it).
  * blocks_for: blocks the next num_tokens tokens of a sequence take; extend: takes them, all or none;
  * release_before: gives back the blocks that lie wholly before `position` (their block_ids become -1),
- * for models in which no layer looks further back. */
+ * for models in which no layer looks further back; release_between: the same, but keeps the blocks that hold tokens before `from`. */
 CMLPagedKVCache* cml_paged_kv_cache_create_device(int max_blocks, int max_sequences, int block_size);
 int cml_paged_cache_blocks_for(CMLPagedKVCache* cache, int seq_id, int num_tokens);
 int cml_paged_cache_extend(CMLPagedKVCache* cache, int seq_id, int num_tokens);
 void cml_paged_cache_release_before(CMLPagedKVCache* cache, int seq_id, int position);
+void cml_paged_cache_release_between(CMLPagedKVCache* cache, int seq_id, int from, int position);
 /* Q [1, seq_q, num_heads*head_dim]; query row i sits at position seq_len - seq_q + i of the
  * sequence. Returns a new [1, seq_q, num_heads*head_dim] tensor, NULL on error. */
 Tensor* cml_paged_gqa_forward(CMLPagedKVCache* cache, int seq_id, Tensor* Q, const CMLGQAConfig* config);

@@ -411,11 +411,14 @@ int cmlb200_ipc_close(void* d_ptr);
 #define CMLB200_ACT_CLAMPED 2     /* g = min(gate, limit), u = clamp(up, -limit, limit): g sigmoid(1.702 g) (u + 1) */
 
 /* A dense [rows, cols] weight (rows = out features), row stride `ld` elements. Allocated with rows rounded
- * up to 16 and ld a multiple of 64, the padding zero. dtype CMLB200_DT_F32 or CMLB200_DT_BF16. */
+ * up to 16 and ld a multiple of 64, the padding zero. dtype CMLB200_DT_F32 or CMLB200_DT_BF16. bias and cap belong to the
+ * products with fp32 results (not to the _glu forms and not to the experts'). */
 typedef struct cmlb200_dense {
     int dtype;
     int rows, cols, ld;
     void* w;
+    const float* bias;          /* device, one per row, added to the product; NULL: none */
+    float cap;                  /* > 0: y = cap tanh(y / cap) */
 } cmlb200_dense;
 
 /* An attention layer over a paged cache, as the kernels below see it. Projection rows hold
@@ -426,8 +429,8 @@ typedef struct cmlb200_attn {
     float scale;                /* score = q.k * scale - slopes[h] * (i - j) */
     int window;                 /* row at position i sees i - window + 1 .. i; <= 0: everything before it */
     const float* slopes;        /* device, one per query head; NULL: no distance bias */
-    int sink;                   /* 1: the softmax denominator starts at exp(0) */
-    const float *q_norm, *k_norm; /* device, RMS norm weights over the whole q / k projection; NULL: none */
+    int sink;                   /* 1: the softmax denominator starts at exp(0), or at exp(sinks[h]) */
+    const float *q_norm, *k_norm; /* device, RMS norm weights over the whole q / k projection (see head_norm); NULL: none */
     float eps;
     float temp_coef, temp_every;  /* q *= 1 + coef ln(floor((i + 1) / every) + 1); every <= 0: none */
     int gate_col;               /* column of the first of `heads` gate logits in a projection row; -1: none */
@@ -437,6 +440,12 @@ typedef struct cmlb200_attn {
     const int* block_table;     /* device, [slots][table_ld] block ids */
     int table_ld;
     int gate_wide;              /* 1: heads * vdim gate logits, one for every element of the output (_tiles only) */
+    int keep;                   /* the sequence's first `keep` tokens stay visible behind the window or chunk */
+    int chunk;                  /* > 0: row at position i sees keys from floor(i / chunk) * chunk on (window is then not looked at) */
+    const float* sinks;         /* device, one per query head; NULL: 0 */
+    int head_norm;              /* 1: the norms are per head, q_norm and k_norm hold `dim` weights that all heads share */
+    int keys_as_values;         /* 1: no v columns; a value is the projected key before its norm (vdim == dim) */
+    float out_scale;            /* factor on the output; 0: 1 */
 } cmlb200_attn;
 
 /* Latent attention over a paged cache of one vector per token: a normed latent of `rank` values and a rotated key
@@ -474,7 +483,48 @@ typedef struct cmlb200_moe {
     int *start, *count;         /* [experts] */
     int *active, *num_active;   /* [experts] experts that were chosen at all */
     int *tiles, *num_tiles;     /* {first position, expert, rows, 0} per 128 positions of an expert */
+    /* how the choice is made; all zero: the `top` largest of a softmax over the experts, weighted by it */
+    int identity;               /* router outputs behind the experts' whose choice returns the row itself: such a pair has position -1 */
+    int groups, keep;           /* > 0: outputs in that many groups of neighbours; only those of the `keep` groups with the largest member */
+    const float* correction;    /* device, [experts + identity], added to the scores for the choice alone */
+    int normalize;              /* 1: weights are divided by their sum (+ 1e-20) and multiplied by `scale` */
+    float scale;
+    float* self;                /* [rows] sum of a row's identity weights; needed with identity > 0 */
 } cmlb200_moe;
+
+/* Residual streams: `streams` rows of `width` per token in place of one residual. A sublayer reads sum_s in[s] x_s; its
+ * output y joins by x_t <- sum_s mix[s][t] x_s + out[t] y, all from the old rows. fp32, device. */
+typedef struct cmlb200_streams {
+    int streams;                /* 1 .. 8 */
+    const float *mix, *out;     /* [streams][streams] (from, to), [streams] */
+    const float* in;            /* of the sublayer that reads next; NULL: ones */
+} cmlb200_streams;
+
+/* What a feed-forward of experts leaves for the join besides y: the row of the pairs, the identity part, another row. */
+typedef struct cmlb200_join {
+    const cmlb200_moe* parts;   /* host pointer; NULL: y has one row per row */
+    const void* h;              /* the rows the experts read (parts->identity > 0), dtype and stride of the output */
+    const float* add;           /* a further fp32 row per row (a shared expert's output); NULL: none */
+    int ld_add;
+} cmlb200_join;
+
+/* Gated delta rule: per head a state S [dim][vdim] in fp32 that a token changes by S <- g S, u = beta (v - S^T k),
+ * S <- S + k u^T, and reads by o = S^T q. g is a factor per key channel, q and k are unit vectors (q / sqrt(dim)), and
+ * q, k, v come out of a causal convolution over `taps` tokens per channel, and silu. The output is divided by its root
+ * mean square per head, weighted and gated. Projection rows hold, from column `col` on, [q (kv_heads * dim) |
+ * k (kv_heads * dim) | v (heads * vdim) | beta logits (heads)]; `channels` = q, k and v columns together. */
+typedef struct cmlb200_delta {
+    int heads, kv_heads, dim, vdim, taps;
+    int vdim_ld;                /* row stride of a state: vdim rounded up to 4, zeros behind vdim */
+    int col;
+    const float* conv;          /* device, [taps][channels], the last row meets the current token */
+    const float* rate;          /* [heads]: decay factor exp(-rate softplus(a + dt_bias)) */
+    const float* dt_bias;       /* [heads * dim] */
+    const float* norm;          /* [vdim] */
+    float eps, out_scale;       /* out_scale 0: 1 */
+    float* state;               /* [slots][heads][dim][vdim_ld]; a token at position 0 finds it as zeros */
+    float* ring;                /* [slots][taps][channels] projections of the latest tokens, position p in entry p mod taps */
+} cmlb200_delta;
 
 /* x[r] = table[token[r]] (+ a sinusoidal vector of position pos[r]: sin, cos of pos * freq[i] in entries
  * 2i, 2i + 1; d_freq NULL: none). fp32 rows of `width`. */
@@ -514,6 +564,28 @@ int cmlb200_residual_add(float* d_x, const float* d_y, int ldy, const cmlb200_mo
 /* f = a N(z) + b N(z^2) + c N(z^3) + e per element, N dividing a row by its root mean square; d_coef = {a, b, c, e}. */
 int cmlb200_poly_norm(const float* d_z, int ld, int rows, int ff, const float* d_coef, float eps, void* d_f, int out_dtype, int ldf, void* stream);
 
+/* Embedding rows times `scale` into `streams` equal rows each (x [rows][streams][width]). */
+int cmlb200_embed_streams(const void* d_table, int dtype, const int* d_tokens, float scale, int streams, int rows, int width, int vocab, float* d_x,
+                          void* stream);
+/* The join of a sublayer's output into the streams (y NULL: none, x unchanged), then out = rms_norm of what the next sublayer
+ * reads * w_next (w_next NULL: no output). Without y, d_row_idx (optional) picks the rows. j (optional): y is the sum of parts. */
+int cmlb200_stream_join(const cmlb200_streams* hc, float* d_x, const float* d_y, int ldy, const cmlb200_join* j, const float* d_w_next, float eps, int rows,
+                        int width, const int* d_row_idx, void* d_out, int out_dtype, int ldo, void* stream);
+
+/* Gated delta rule over a step's rows. d_decay: [rows][heads * dim] inputs a of the decay, d_gate: [rows][heads * vdim] gate
+ * logits, fp32 with their strides. out: fp32 or bf16.
+ * _one: single tokens, at most one row per sequence, everything in one launch.
+ * _rows: portions whose rows are first .. first + rows - 1 of the step, runs[i] = {first row, rows, slot, position} (device):
+ * convolutions, norms and decays, the recurrence, output norm and gate. work: [rows][cmlb200_delta_work_floats] fp32, row 0 is the step's row `first`; d_decay is overwritten with the decays. All row arrays begin at the step's row 0. */
+int cmlb200_delta_one(const cmlb200_delta* a, const float* d_proj, int ld, const float* d_decay, int ld_decay, const float* d_gate, int ld_gate,
+                      const int* d_row_pos, const int* d_row_slot, int rows, void* d_out, int out_dtype, int out_ld, void* stream);
+int cmlb200_delta_rows(const cmlb200_delta* a, const float* d_proj, int ld, float* d_decay, int ld_decay, const float* d_gate, int ld_gate,
+                       const int* d_row_pos, const int* d_row_slot, int first, int rows, const int* d_runs, int runs, float* d_work, void* d_out,
+                       int out_dtype, int out_ld, void* stream);
+int cmlb200_delta_work_floats(const cmlb200_delta* a);
+/* bf16 rows of columns col .. col + n - 1 of fp32 rows; columns n .. ldo - 1 are left alone. */
+int cmlb200_pack_columns(const float* d_x, int ld, int col, int n, int rows, uint16_t* d_out_bf16, int ldo, void* stream);
+
 /* Latent attention. _append: rotates the query columns in place and fills the cache (any rows). _query: the same for
  * rows whose attention runs over the latents themselves, into fp16 rows [heads][ld] = [Wuk^T q | rotated q] times
  * scale log2 e. Wuk^T is stored per head as [rank rounded up to 16][dim rounded up to 64]. */
@@ -547,8 +619,8 @@ int cmlb200_latent_query_f32(const cmlb200_latent* a, const float* d_wukt, const
 int cmlb200_latent_output_f32(const cmlb200_latent* a, const float* d_wuv, const float* d_o, const float* d_proj, int ld, int rows, float* d_out,
                               int out_ld, void* stream);
 
-/* Experts. _route: softmax over all experts of fp32 router logits, the `top` largest scores (ties: lower index), and
- * the plan. The products take a weight whose experts are stacked, each `rows / experts` rows (a multiple of 16);
+/* Experts. _route: softmax over all router outputs (fp32 logits), the `top` largest scores (ties: lower index) under the
+ * plan's rules, and the plan. The products take a weight whose experts are stacked, each `rows / experts` rows (a multiple of 16);
  * gather: x has one row per step row, otherwise one per position. y has one row per position. _gemv: up to 32 rows. */
 long cmlb200_moe_positions(int rows, int top, int experts, int align);
 int cmlb200_moe_route(const cmlb200_moe* m, const float* d_logits, int ld, int rows, int align, void* stream);
