@@ -392,6 +392,9 @@ def main():
     ap.add_argument("--cpu-leg", default=None, choices=["gemv", "llama"], help=argparse.SUPPRESS)
     ap.add_argument("--calls", type=int, default=3, help=argparse.SUPPRESS)
     ap.add_argument("--llama-steps", type=int, default=4, help=argparse.SUPPRESS)
+    ap.add_argument("--streams", nargs="?", const="all", default=None, choices=["all", "kernels", "models"],
+                    help="instead of the default workload: models with residual streams, chunked attention beside a gated delta rule and grouped routing, "
+                         "beside the layered models of equal sizes, and their kernels")
     args = ap.parse_args()
 
     if args.cpu_leg:                                   # child process of run_cpu_leg
@@ -425,6 +428,9 @@ def main():
     if args.layered:
         import bench_layered
         return bench_layered.run(pkg, synth, torch, peaks, ClockSampler(local), args.layered == "kernels", args.layered == "models")
+    if args.streams:
+        import bench_streams
+        return bench_streams.run(pkg, synth, torch, peaks, ClockSampler(local), args.streams == "kernels", args.streams == "models")
     if args.latent:
         import bench_latent
         return bench_latent.run(pkg, synth, torch, peaks, ClockSampler(local), args.latent == "kernels", args.latent == "models")

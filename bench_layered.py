@@ -29,15 +29,17 @@ def layered_leg(pkg, synth, torch, c, peaks):
     return model_leg(pkg, synth, torch, cfg, c, peaks, body, lambda B: total, lambda: 4 * c["layers"] * c["kv_heads"] * c["dim"])
 
 
-def model_leg(pkg, synth, torch, cfg, c, peaks, body, weights, cache_bytes):
+def model_leg(pkg, synth, torch, cfg, c, peaks, body, weights, cache_bytes, row_bytes=0, weight=None):
     """Prefill and decode of a configuration with random weights. body: multiplications per token of a prompt. weights(B): those a
-    decode step of B rows reads. cache_bytes(): read per row and cached token, all layers together (c["window"] of them)."""
+    decode step of B rows reads. cache_bytes(): read per row and cached token, all layers together (c["window"] of them).
+    row_bytes: further bytes per row of a decode step (states). weight: (rng, name, shape) -> a tensor; the default suits designs
+    whose norms are stored as they are."""
     rng = np.random.default_rng(5)
     out = {"weight_bytes": 2 * weights(max(c["batches"]))}
     with tempfile.TemporaryDirectory() as tmp:
         gen = lambda name, shape: (1 + 0.1 * rng.standard_normal(shape, dtype=np.float32)) if len(shape) == 1 else \
             rng.standard_normal(shape, dtype=np.float32) * np.float32(1.0 if name == "embed" else shape[1] ** -0.5)
-        synth.write_layered(Path(tmp) / "m", cfg, gen, alias_layers=True)
+        synth.write_layered(Path(tmp) / "m", cfg, (lambda name, shape: weight(rng, name, shape)) if weight else gen, alias_layers=True)
         nb = max(c["batches"])
         m = pkg.LanguageModel(Path(tmp) / "m", max_tokens=max(max(PROMPTS), nb * (c["window"] + NEW + 16)) + 64, max_sequences=nb, max_step_rows=4096)
     for n in PROMPTS:
@@ -64,7 +66,7 @@ def model_leg(pkg, synth, torch, cfg, c, peaks, body, weights, cache_bytes):
         for s in seqs:
             m.end(s)
         step = ms / NEW
-        nbytes = 2 * weights(B) + B * c["window"] * cache_bytes()
+        nbytes = 2 * weights(B) + B * (c["window"] * cache_bytes() + row_bytes)
         out[f"decode_b{B}"] = {"tok_s": B / (step * 1e-3), "ms_per_step": step, "gbs": nbytes / (step * 1e-3) / 1e9,
                                "frac_of_hbm": nbytes / (step * 1e-3) / 1e9 / peaks["hbm_gbs"]}
     m.close()

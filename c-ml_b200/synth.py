@@ -288,10 +288,105 @@ def latent_layer_shapes(layer, W, p):
     return out
 
 
+def routed_mlp(experts, identity, top, groups, keep, ff, shared, scale=1.5):
+    return {"kind": "moe", "expert": {"ff": ff}, "shared": {"ff": shared},
+            "router": {"experts": experts, "identity": identity, "top": top, "groups": {"count": groups, "keep": keep}, "scale": scale}}
+
+
+def kept_layer(heads, kv_heads, dim, window, keep, mlp, scale=None):
+    """mlp: a dense layer's size, routed_mlp(..), or None."""
+    return {"type": "attention", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": scale or dim ** -0.5,
+                                           "mask": {"size": window, "keep_first": keep}},
+            "mlp": {"kind": "dense", "ff": mlp} if isinstance(mlp, int) else mlp}
+
+
+def parallel_layer(left, right, ranks, mlp, scales=(0.8, 1.3)):
+    """left: (heads, kv_heads, dim, vdim, chunk), right: (heads, kv_heads, dim, vdim, taps), ranks: of the decay's and the gate's projections
+    (these only shape tensors)."""
+    lm = dict(zip(("heads", "kv_heads", "dim", "vdim"), left), scale=left[2] ** -0.5, mask={"size": left[4]})
+    return {"type": "parallel", "mixer": {"left": lm, "left_scale": scales[0], "right": dict(zip(("heads", "kv_heads", "dim", "vdim", "conv"), right)), "right_scale": scales[1]},
+            "mlp": {"kind": "dense", "ff": mlp} if isinstance(mlp, int) else mlp, "ranks": list(ranks)}
+
+
+def streams_config(vocab, width, streams, layers, eps=1e-5, scale=2.0, cap=6.0):
+    return {"architecture": "Lenedra", "vocab": vocab, "width": width, "streams": streams, "norm": {"eps": eps}, "embedding": {"scale": scale},
+            "logit_softcap": cap, "layers": layers}
+
+
+def streams_layer_shapes(layer, W, streams, p):
+    m, f, out = layer["mixer"], layer["mlp"], {}
+
+    def sublayer(n):
+        out.update({p + f"norm{n}": (W,), p + f"hc{n}.in": (streams,), p + f"hc{n}.out": (streams,), p + f"hc{n}.mix": (streams, streams)})
+
+    def projections(q, pairs):
+        for name, rows in pairs:
+            out.update({q + name: (rows, W), q + name + ".b": (rows,)})
+    sublayer(1)
+    if layer["type"] == "attention":
+        H, G, D, q = m["heads"], m["kv_heads"], m["dim"], p + "mix."
+        projections(q, (("q", H * D), ("k", G * D)))
+        out.update({q + "q.norm": (D,), q + "k.norm": (D,), q + "o": (W, H * D), q + "o.b": (W,)})
+    else:
+        a, r, q = m["left"], m["right"], p + "mix.left."
+        projections(q, (("q", a["heads"] * a["dim"]), ("k", a["kv_heads"] * a["dim"]), ("v", a["kv_heads"] * a["vdim"])))
+        out.update({q + "sink": (a["heads"],), q + "o": (W, a["heads"] * a["vdim"])})
+        H, qk, v, q = r["heads"], r["kv_heads"] * r["dim"], r["heads"] * r["vdim"], p + "mix.right."
+        for name, rows in (("q", qk), ("k", qk), ("v", v)):
+            out.update({q + name: (rows, W), q + name + ".conv": (rows, r["conv"])})
+        ra, rg = layer["ranks"]
+        out.update({q + "b": (H, W), q + "A_log": (H,), q + "dt_bias": (H * r["dim"],), q + "norm": (r["vdim"],), q + "a1": (ra, W), q + "a2": (H * r["dim"], ra),
+                    q + "g1": (rg, W), q + "g2": (v, rg), q + "o": (W, v)})
+    if not f:
+        return out
+    sublayer(2)
+
+    def gated(q, n):
+        out.update({q + "gate": (n, W), q + "up": (n, W), q + "down": (W, n)})
+    if f["kind"] == "dense":
+        gated(p + "mlp.", f["ff"])
+        return out
+    n = f["router"]["experts"] + f["router"]["identity"]
+    out.update({p + "mlp.router": (n, W), p + "mlp.correction": (n,)})
+    for e in range(f["router"]["experts"]):
+        gated(p + f"mlp.e{e}.", f["expert"]["ff"])
+    gated(p + "mlp.shared.", f["shared"]["ff"])
+    return out
+
+
+def streams_weight(rng, name, shape):
+    """A random tensor of a design with streams: decays between nearly none and nearly all, sinks that take a visible share,
+    streams that mix, corrections in widely separated steps."""
+    a = rng.standard_normal(shape).astype(np.float32)
+    leaf = name.split(".", 1)[1] if name[0] == "l" and name[1].isdigit() else name
+    if leaf.startswith("norm") or leaf == "final.norm":
+        a *= 0.2
+    elif leaf.endswith(".norm"):
+        a = 1 + 0.2 * a
+    elif leaf.endswith((".q.b", ".k.b", ".v.b", ".o.b")):
+        a *= 0.3
+    elif leaf.endswith(".sink"):
+        a += 1
+    elif leaf.endswith(".A_log"):
+        a = rng.uniform(-4, 1, shape)
+    elif leaf.endswith(".dt_bias"):
+        a -= 1
+    elif leaf.endswith(".correction"):
+        a = rng.choice([0.75, -1.5, -3.75], shape)
+    elif leaf.startswith("hc"):
+        a = 0.15 * a + (np.eye(shape[0]) if len(shape) == 2 else 0.7)
+    elif leaf != "embed":
+        a /= np.sqrt(shape[-1])
+    return bf16_round(np.asarray(a, np.float32))[1]
+
+
 def layered_shapes(cfg):
     """Tensor name -> shape of every tensor a configuration asks for."""
     W, out = cfg["width"], {"embed": (cfg["vocab"], cfg["width"])}
     for i, layer in enumerate(cfg["layers"]):
+        if "streams" in cfg:
+            out.update(streams_layer_shapes(layer, W, cfg["streams"], f"l{i}."))
+            continue
         if layer.get("weights_of") is not None:
             continue
         if layer["type"].startswith("latent"):
@@ -312,6 +407,9 @@ def layered_weights(rng, cfg):
     """Random bf16-exact fp32 weights: products of unit inputs have unit size, norms lie around 1."""
     w = {}
     for name, shape in layered_shapes(cfg).items():
+        if "streams" in cfg:
+            w[name] = streams_weight(rng, name, shape)
+            continue
         a = rng.standard_normal(shape, dtype=np.float32)
         if name.endswith("mlp.act"):
             w[name] = bf16_round(0.6 * a)[1]

@@ -2,12 +2,14 @@
 import numpy as np
 
 import latent_oracle
+import lenedra_oracle
 import lm_oracle
 
 
 def variants(synth):
     """name -> configuration. Sizes are chosen so that no two of them coincide by accident."""
     L, A = synth.layered_layer, synth.latent_layer
+    K, P, R = synth.kept_layer, synth.parallel_layer, synth.routed_mlp
     return {
         # grouped heads, two windows, a layer without feed-forward, shared weights with another layer between
         "mixed": synth.layered_config(211, 144, [L(6, 3, 24, 40, 19, 200, coef=0.4, every=7), L(4, 1, 32, 16, 70, None, coef=0.1, every=33),
@@ -31,21 +33,40 @@ def variants(synth):
         "latent_wide": synth.latent_config(130, 192, [A(20, 72, 64, 136, 300, 320, base=1e6), A(12, 104, 32, 72, 200, (40, 3, 48, 1.0), 90, True, 1e4, (8.0, 40, 16.0, 2.0))]),
         # sizes with tiles of their own, more than 64 (token, head) pairs per token
         "latent_full": synth.latent_config(64, 128, [A(4, 128, 64, 128, 512, 96, base=1e5), A(70, 8, 8, 8, 128, (9, 4, 24, 1.5), 40, True)]),
+        # streams: every mechanism, key heads shared on both sides, value sizes of their own, a layer without feed-forward, windows and
+        # chunks of different sizes, identity experts, one of them with all groups open
+        "streams": synth.streams_config(211, 144, 3, [K(6, 3, 24, 19, 5, 200), P((6, 2, 24, 40, 37), (4, 2, 24, 32, 3), (12, 20), R(7, 3, 3, 5, 2, 40, 56)),
+                                                       K(4, 1, 32, 70, 33, None), P((3, 3, 16, 8, 64), (5, 5, 40, 16, 5), (9, 33), R(4, 0, 2, 1, 1, 33, 17)),
+                                                       K(5, 5, 16, 30, 1, R(6, 2, 5, 4, 4, 24, 72, 0.7))], eps=1e-3, scale=0.75),
+        # odd sizes everywhere, a window of one token with more kept than it, a chunk of one, a convolution of one tap, one stream
+        "streams_odd": synth.streams_config(97, 75, 1, [P((3, 1, 13, 7, 23), (3, 1, 11, 9, 2), (5, 3), 51, (-0.7, 0.4)), K(3, 3, 7, 1, 9, R(3, 4, 3, 7, 4, 17, 33, 2.5)),
+                                                        P((5, 5, 9, 21, 1), (6, 3, 5, 3, 1), (1, 2), None), K(9, 3, 13, 50, 0, 33)], eps=2e-2, scale=0.7, cap=3.0),
+        # wide heads, many heads, many streams, a window and a chunk longer than the prompts
+        "streams_wide": synth.streams_config(130, 192, 6, [K(12, 4, 136, 400, 16, 96), P((20, 2, 72, 136, 500), (9, 3, 136, 200, 4), (24, 130), R(40, 8, 6, 12, 5, 48, 320, 1.0))],
+                                             cap=12.0),
+        # sizes with tiles of their own; chunks and windows that end where blocks and tiles do
+        "streams_full": synth.streams_config(64, 128, 4, [P((4, 2, 64, 64, 64), (2, 1, 128, 128, 4), (16, 16), R(9, 3, 4, 3, 2, 24, 24)), K(2, 1, 128, 64, 16, 96),
+                                                          P((4, 4, 128, 128, 16), (4, 4, 64, 64, 4), (64, 64), 64)]),
         "plain": synth.layered_config(64, 64, [L(2, 1, 32, 32, 16, 64, coef=0.0, every=1), L(2, 2, 32, 32, 17, 64, coef=1.0, every=1)], eps=1e-6),
     }
 
 
 def steady_routes(synth, rng, cfg, w):
     """Makes the experts' choice independent of rounding: the routers read only the last columns of the residual, which
-    hold well separated levels in an order of each token's own and which no sublayer adds to."""
+    hold well separated levels in an order of each token's own and which no sublayer adds to (identity experts and the
+    mixing of streams only scale them)."""
     moe = [i for i, l in enumerate(cfg["layers"]) if (l["mlp"] or {}).get("kind") == "moe"]
     if not moe:
         return
-    n = max(cfg["layers"][i]["mlp"]["router"]["experts"] for i in moe)
+    n = max(len(w[f"l{i}.mlp.router"]) for i in moe)
     level = (np.arange(n) - n / 2) * min(0.5, 4.0 / n)
     w["embed"][:, -n:] = synth.bf16_round(np.stack([rng.permutation(level) for _ in range(cfg["vocab"])]))[1]
     for name in w:
-        if name.endswith((".norm1", ".norm2")):
+        if "streams" in cfg and name.endswith((".norm1", ".norm2", "mix.o.b")):
+            w[name][-n:] = 0.0
+        elif "streams" in cfg and name[0] == "l" and name.endswith((".o", ".down")):
+            w[name][-n:] = 0.0
+        elif name.endswith((".norm1", ".norm2")):
             w[name][-n:] = 0.0
             w[name] *= 0.5                             # rounding errors then grow little from layer to layer
     for i in moe:
@@ -77,7 +98,7 @@ TOL = {6: 0.02, 0: 2e-5}            # by dtype of the device model: bfloat16, fl
 
 def model(cfg, w):
     """The plain restatement of a configuration's design."""
-    return (latent_oracle if cfg["architecture"] == "Situlorn" else lm_oracle).Model(cfg, w)
+    return {"Rarolorn": lm_oracle, "Situlorn": latent_oracle, "Lenedra": lenedra_oracle}[cfg["architecture"]].Model(cfg, w)
 
 
 def reference(cfg, w, tokens):

@@ -14,7 +14,8 @@ from lm_util import TOL, cut, error
 pytestmark = pytest.mark.gpu
 ROOT = Path(__file__).resolve().parents[1]
 LATENT = ["latent", "latent_odd", "latent_wide", "latent_full"]
-NAMES = ["mixed", "odd", "wide", "plain"] + LATENT
+STREAMS = ["streams", "streams_odd", "streams_wide", "streams_full"]
+NAMES = ["mixed", "odd", "wide", "plain"] + LATENT + STREAMS
 DTYPES = [6, 0]                      # bfloat16, float32
 
 
@@ -72,7 +73,7 @@ def test_first_tokens(synth, tmp_path, load, name, dtype):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("name", ["mixed", "odd", "latent", "latent_odd", "latent_wide"])
+@pytest.mark.parametrize("name", ["mixed", "odd", "latent", "latent_odd", "latent_wide", "streams", "streams_odd", "streams_full"])
 def test_unequal_requests_in_one_batch_with_blocks_used_again(pkg, synth, tmp_path, load, name, dtype):
     """Random schedules over a pool that is too small for all requests together: requests come and go, pause,
     take portions beside single tokens, and sit on blocks and slots that others have used."""
@@ -109,7 +110,7 @@ def test_unequal_requests_in_one_batch_with_blocks_used_again(pkg, synth, tmp_pa
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("name", ["wide", "latent", "latent_wide"])
+@pytest.mark.parametrize("name", ["wide", "latent", "latent_wide", "streams", "streams_wide"])
 def test_batch_does_not_change_a_request(synth, tmp_path, load, name, dtype):
     cfg, w, folder = lm_util.build(synth, tmp_path, name)
     m = load(folder, dtype, max_sequences=8)
@@ -129,18 +130,18 @@ def test_batch_does_not_change_a_request(synth, tmp_path, load, name, dtype):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("name", ["mixed", "latent_odd"])
+@pytest.mark.parametrize("name", ["mixed", "latent_odd", "streams", "streams_odd"])
 def test_long_decoding(pkg, synth, tmp_path, load, name, dtype):
     """Hundreds of decoded tokens, over many blocks; windows let blocks go on the way, so the sequence outgrows what
     the pool could hold of it at once."""
     cfg, w, folder = lm_util.build(synth, tmp_path, name)
     t = prompt(cfg, 420)
-    m = load(folder, dtype, max_tokens=128, max_sequences=2)
+    m = load(folder, dtype, max_tokens=160, max_sequences=2)
     s = m.open()
     got = feed(m, s, t, [20] + [1] * 400)
     assert error(got, lm_util.reference(cfg, w, t)) < TOL[dtype]
     lib = pkg.lib
-    assert lib.cml_lm_sequence_length(m.h, s) == 420 and lib.cml_lm_blocks_total(m.h) - lib.cml_lm_blocks_free(m.h) <= 6      # the longest window is 70
+    assert lib.cml_lm_sequence_length(m.h, s) == 420 and lib.cml_lm_blocks_total(m.h) - lib.cml_lm_blocks_free(m.h) <= 9      # the longest window is 70, and up to 33 first tokens are kept
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
@@ -224,7 +225,7 @@ def serve(pkg, m, prompts, lengths, batch, gen=None):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("name", ["wide", "latent"])
+@pytest.mark.parametrize("name", ["wide", "latent", "streams"])
 def test_scheduler_serves_more_requests_than_fit(pkg, synth, tmp_path, load, name, dtype):
     cfg, w, folder = lm_util.build(synth, tmp_path, name)
     m = load(folder, dtype, max_tokens=256, max_sequences=3, max_step_rows=48)       # prompts are cut, requests wait
@@ -237,11 +238,12 @@ def test_scheduler_serves_more_requests_than_fit(pkg, synth, tmp_path, load, nam
         assert same_until_a_tie(g, want, gap)
     assert pkg.lib.cml_lm_blocks_free(m.h) == pkg.lib.cml_lm_blocks_total(m.h)
     # a request the pool can never hold, and one with an unknown token, end with an error; the others run
-    _, got, status = serve(pkg, m, [prompts[0], prompt(cfg, 250), [1, cfg["vocab"]], prompts[1]], [4, 50, 3, 5], 2)
+    never = prompt(cfg, 1000 if name == "streams" else 250)                          # windows in every layer: only its block table bounds a sequence
+    _, got, status = serve(pkg, m, [prompts[0], never, [1, cfg["vocab"]], prompts[1]], [4, 50, 3, 5], 2)
     assert [len(g) for g in got] == [4, 0, 0, 5] and status[1] == status[2] == 4
 
 
-@pytest.mark.parametrize("name", ["plain", "latent"])
+@pytest.mark.parametrize("name", ["plain", "latent", "streams"])
 def test_generation_and_sampling(pkg, synth, tmp_path, load, name):
     cfg, w, folder = lm_util.build(synth, tmp_path, name)
     m, lib = load(folder, 0), pkg.lib
@@ -288,7 +290,7 @@ def test_step_refusals_change_nothing(pkg, synth, tmp_path, load):
     assert error(np.concatenate(parts), lm_util.reference(cfg, w, t)) < TOL[0]
 
 
-@pytest.mark.parametrize("name", ["odd", "latent_odd"])
+@pytest.mark.parametrize("name", ["odd", "latent_odd", "streams_odd"])
 def test_wanted_places_only_and_many_of_them(synth, tmp_path, load, name):
     cfg, w, folder = lm_util.build(synth, tmp_path, name)
     m = load(folder, 6, max_tokens=1024)
@@ -332,7 +334,7 @@ def test_llama_behind_the_same_interface(pkg, tmp_path, load):
     assert [len(g) for g in got] == [5, 8] and got[0][0] == int(want[6].argmax())
 
 
-@pytest.mark.parametrize("name", ["mixed", "latent"])
+@pytest.mark.parametrize("name", ["mixed", "latent", "streams"])
 def test_trace_run_replays(synth, tmp_path, torch_dev, name):
     cfg, w, folder = lm_util.build(synth, tmp_path, name)
     t = {"a": prompt(cfg, 90, 1), "b": prompt(cfg, 50, 2), "c": prompt(cfg, 30, 3)}
@@ -364,7 +366,7 @@ def test_trace_run_replays(synth, tmp_path, torch_dev, name):
                 assert error(got, np.array(mine)) < TOL[code]
 
 
-@pytest.mark.parametrize("name", ["plain", "latent_odd"])
+@pytest.mark.parametrize("name", ["plain", "latent_odd", "streams_odd"])
 def test_cml_generate_program(pkg, synth, tmp_path, load, name):
     cfg, w, folder = lm_util.build(synth, tmp_path, name)
     prompts = [prompt(cfg, 9, 1).tolist(), prompt(cfg, 30, 2).tolist()]

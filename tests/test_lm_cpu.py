@@ -8,6 +8,7 @@ import numpy as np
 import pytest
 
 import latent_oracle as la
+import lenedra_oracle as le
 import lm_oracle as lo
 import lm_util
 
@@ -47,7 +48,8 @@ def test_norm_and_activation():
     assert np.allclose(lo.gelu_tanh(np.array([0.0, 1.0, -1.0])), [0.0, 0.841192, -0.158808], atol=1e-6)
 
 
-@pytest.mark.parametrize("name", ["mixed", "odd", "wide", "plain", "latent", "latent_odd", "latent_wide", "latent_full"])
+@pytest.mark.parametrize("name", ["mixed", "odd", "wide", "plain", "latent", "latent_odd", "latent_wide", "latent_full", "streams", "streams_odd", "streams_wide",
+                                  "streams_full"])
 def test_portions_change_nothing(synth, tmp_path, name):
     cfg, w, _ = lm_util.build(synth, tmp_path, name)
     m = lm_util.model(cfg, w)
@@ -149,9 +151,88 @@ def test_a_layer_reads_the_named_cache(synth, tmp_path):
     assert st["caches"][2] == {} and len(st["caches"][0]["c"]) == 3 and "l2.mix.dkv" not in w
 
 
+# ---- the restatement of streams, kept windows, chunks, the delta rule and grouped routing ----------------
+def test_kept_window_and_chunks_by_hand():
+    seen = le.window_with_kept([6], range(9), 2, 3)[0]
+    assert seen.tolist() == [True] * 3 + [False] * 2 + [True] * 2 + [False] * 2
+    assert le.window_with_kept([1], range(4), 1, 3)[0].tolist() == [True, True, False, False]          # kept, but not before its time
+    assert le.same_chunk([3, 4, 7], range(8), 4).tolist() == [[True] * 4 + [False] * 4, [False] * 4 + [True] + [False] * 3, [False] * 4 + [True] * 4]
+
+
+def test_learned_sink_by_hand():
+    p = le.weights_over(np.array([[0.0, np.log(2.0), 9.0]]), np.array([[True, True, False]]), np.log(5.0))
+    assert np.allclose(p, [[1 / 8, 2 / 8, 0]])
+    assert np.allclose(le.weights_over(np.array([[-900.0]]), np.array([[True]]), -900.0), [[0.5]])
+
+
+def test_delta_rule_by_hand():
+    S = np.array([[2.0], [4.0]])
+    o = le.delta_rule(np.array([[1.0, 2.0]]), np.array([[0.6, 0.8]]), np.array([[5.0]]), np.array([[0.5, 0.25]]), np.array([0.5]), S)
+    u = 0.5 * (5 - (0.6 * 1 + 0.8 * 1))                                       # the decayed state is (1, 1)
+    assert np.allclose(S, [[1 + 0.6 * u], [1 + 0.8 * u]]) and np.allclose(o, [[S[0, 0] + 2 * S[1, 0]]])       # the read sees the write
+
+
+def test_causal_convolution_by_hand():
+    x, taps = np.array([[1.0], [2.0], [3.0]]), np.array([[10.0, 1.0]])
+    y, past = le.causal_conv(x, taps, np.zeros((1, 1)))
+    assert np.allclose(y, le.silu(np.array([[1.0], [12.0], [23.0]]))) and past.tolist() == [[3.0]]
+    y, past = le.causal_conv(x, taps[:, 1:], np.zeros((0, 1)))
+    assert np.allclose(y, le.silu(x)) and past.shape == (0, 1)
+
+
+def test_grouped_choice_by_hand():
+    z = np.log(np.array([[0.4, 0.1, 0.2, 0.3]]))
+    w = {"router": np.eye(4), "correction": np.array([-1.0, -1.0, -2.0, -1.05])}
+    r = {"groups": {"count": 2, "keep": 1}, "top": 2, "scale": 3.0}
+    ids, p = le.route(z, w, r)                                                # choice: -0.6 -0.9 | -1.8 -0.75
+    assert ids.tolist() == [[0, 1]] and np.allclose(p, [[3 * 0.8, 3 * 0.2]])
+    ids, _ = le.route(z, w, {**r, "groups": {"count": 2, "keep": 2}})
+    assert ids.tolist() == [[0, 3]]
+
+
+def test_streams_by_hand():
+    x = np.array([[[1.0]], [[10.0]]])
+    assert le.read_streams(x, np.array([2.0, 3.0])).tolist() == [[32.0]]
+    y = le.write_streams(x, np.array([[1.0, 2.0], [3.0, 4.0]]), np.array([5.0, 6.0]), np.array([[100.0]]))
+    assert y.tolist() == [[[1 + 30 + 500]], [[2 + 40 + 600]]]                  # mix is [from, to]
+
+
+def test_every_setting_of_a_design_with_streams_shows(synth, tmp_path):
+    cfg, w, _ = lm_util.build(synth, tmp_path, "streams")
+    t = np.random.default_rng(3).integers(0, cfg["vocab"], 90)
+    want = lm_util.reference(cfg, w, t)
+
+    def moved(change, w2=None):
+        other = json.loads(json.dumps(cfg))
+        change(other, other["layers"])
+        assert lm_util.error(lm_util.reference(other, w2 or w, t), want) > 100 * lm_util.TOL[0]
+    moved(lambda c, l: l[0]["mixer"]["mask"].update(size=18))
+    moved(lambda c, l: l[0]["mixer"]["mask"].update(keep_first=4))
+    moved(lambda c, l: l[0]["mixer"].update(scale=0.3))
+    moved(lambda c, l: l[1]["mixer"]["left"]["mask"].update(size=38))
+    moved(lambda c, l: l[1]["mixer"]["left"].update(scale=0.3))
+    moved(lambda c, l: l[1]["mixer"].update(left_scale=0.9))
+    moved(lambda c, l: l[3]["mixer"].update(right_scale=1.1))
+    moved(lambda c, l: l[1]["mlp"]["router"].update(top=2))
+    moved(lambda c, l: l[1]["mlp"]["router"].update(scale=1.2))
+    moved(lambda c, l: l[1]["mlp"]["router"]["groups"].update(keep=1))
+    moved(lambda c, l: l[1]["mlp"]["router"].update(experts=6, identity=4))    # the last expert becomes an identity
+    moved(lambda c, l: c["embedding"].update(scale=2.5))
+    moved(lambda c, l: c.update(logit_softcap=5.0))
+    for name in ("l0.mix.q.b", "l0.mix.k.b", "l0.mix.o.b", "l0.mix.q.norm", "l0.mix.k.norm", "l1.mix.left.sink", "l1.mix.left.v.b", "l1.mix.right.q.conv", "l1.mix.right.v.conv",
+                 "l1.mix.right.A_log", "l1.mix.right.dt_bias", "l1.mix.right.b", "l1.mix.right.norm", "l3.mix.right.a2", "l3.mix.right.g1", "l1.mlp.correction", "l1.mlp.shared.up",
+                 "l1.hc1.in", "l1.hc2.out", "l3.norm1", "final.norm"):
+        w2 = dict(w)
+        w2[name] = np.roll(w[name][::-1], 1, 0) if len(w[name]) == 3 else w[name][::-1]
+        moved(lambda c, l: None, w2)
+    w2 = dict(w)
+    w2["l1.hc1.mix"] = w["l1.hc1.mix"].T
+    moved(lambda c, l: None, w2)
+
+
 # ---- registry and readers ------------------------------------------------------------------------------
 def test_registry_knows_its_classes(pkg):
-    assert pkg.lib.cml_lm_known(b"Situlorn") == 1
+    assert pkg.lib.cml_lm_known(b"Situlorn") == 1 and pkg.lib.cml_lm_known(b"Lenedra") == 1
     assert pkg.lib.cml_lm_known(b"Rarolorn") == 1 and pkg.lib.cml_lm_known(b"llama") == 1
     assert pkg.lib.cml_lm_known(b"nothing") == 0 and pkg.lib.cml_lm_known(None) == 0
     o = pkg.lib.cml_lm_default_options()
@@ -227,6 +308,40 @@ def test_latent_load_refusals(pkg, synth, tmp_path):
     with_config(lambda c: c["layers"][0]["mlp"].update(ff=-1))
 
 
+def test_streams_load_refusals(pkg, synth, tmp_path):
+    cfg, w, folder = lm_util.build(synth, tmp_path, "streams")
+    mixer = lambda c, i: c["layers"][i]["mixer"]
+
+    def with_config(change):
+        c = json.loads(json.dumps(cfg))
+        change(c)
+        (folder / "config.json").write_text(json.dumps(c))
+        assert not _load(pkg, folder)
+
+    with_config(lambda c: c.pop("streams"))
+    with_config(lambda c: c.update(streams=0))
+    with_config(lambda c: c.update(streams=9))
+    with_config(lambda c: c["layers"][0].update(type="latent_attention"))
+    with_config(lambda c: mixer(c, 0)["mask"].update(keep_first=-1))
+    with_config(lambda c: mixer(c, 0).update(vdim=25))                           # values are keys
+    for side in ("left", "right"):
+        for key in ("heads", "kv_heads", "dim", "vdim"):
+            with_config(lambda c: mixer(c, 1)[side].pop(key))
+        with_config(lambda c: mixer(c, 1).pop(side))
+        with_config(lambda c: mixer(c, 1).pop(side + "_scale"))
+    with_config(lambda c: mixer(c, 1)["left"]["mask"].update(size=0))
+    with_config(lambda c: mixer(c, 1)["right"].update(conv=0))
+    with_config(lambda c: mixer(c, 1)["right"].update(kv_heads=3))
+    with_config(lambda c: mixer(c, 1)["right"].update(dim=257))
+    router = lambda c: c["layers"][1]["mlp"]["router"]
+    with_config(lambda c: router(c).update(identity=-1))
+    with_config(lambda c: router(c).update(top=11))
+    with_config(lambda c: router(c)["groups"].update(count=3))                   # does not divide the outputs
+    with_config(lambda c: router(c)["groups"].update(keep=6))
+    with_config(lambda c: router(c).update(top=5))                               # more than the kept groups hold
+    with_config(lambda c: c["layers"][1]["mlp"]["shared"].update(ff=0))
+
+
 def test_tensor_file_refusals(pkg, synth, tmp_path):
     cfg, w, folder = lm_util.build(synth, tmp_path, "plain")
     path = folder / "model.safetensors"
@@ -291,6 +406,16 @@ def test_blocks_are_taken_released_and_used_again(pkg):
     assert {c.contents.sequences[b].block_ids[i] for i in (3, 4)} == set(first[:2])
     lib.cml_paged_cache_free_sequence(c, a)
     lib.cml_paged_cache_free_sequence(c, b)
+    assert c.contents.free_count == 6
+    s = lib.cml_paged_cache_init_sequence(c)
+    assert lib.cml_paged_cache_extend(c, s, 90) == 0 and c.contents.free_count == 0
+    lib.cml_paged_cache_release_between(c, s, 17, 70)                  # blocks 0 and 1 hold the first 17 tokens, block 4 position 70
+    kept = [c.contents.sequences[s].block_ids[i] >= 0 for i in range(6)]
+    assert kept == [True, True, False, False, True, True] and c.contents.free_count == 2
+    lib.cml_paged_cache_release_between(c, s, 17, 80)
+    lib.cml_paged_cache_release_between(c, s, 17, 200)
+    assert c.contents.free_count == 4
+    lib.cml_paged_cache_free_sequence(c, s)
     assert c.contents.free_count == 6
     one = np.zeros(4, np.float32)
     s = lib.cml_paged_cache_init_sequence(c)
