@@ -159,7 +159,7 @@ def delta(pkg, torch, T, add):
             proj, dec0, gate = torch.randn(rows, ld, device=dev), torch.randn(rows, H * D, device=dev), torch.randn(rows, H * D, device=dev)
             pos, slot = torch.arange(n, device=dev, dtype=torch.int32).repeat(seqs), torch.arange(seqs, device=dev, dtype=torch.int32).repeat_interleave(n)
             runs = torch.tensor([[i * n, n, i, 0] for i in range(seqs)], device=dev, dtype=torch.int32)
-            w, o = torch.empty(rows, lib.cmlb200_delta_work_floats(a), device=dev), torch.empty(rows, H * D, device=dev, dtype=torch.bfloat16)
+            w, o = torch.empty(lib.cmlb200_delta_work_floats(a, rows, seqs), device=dev), torch.empty(rows, H * D, device=dev, dtype=torch.bfloat16)
             us = T.us([lambda s: ck(lib.cmlb200_delta_rows(a, P(proj), ld, P(dec0), H * D, P(gate), H * D, P(pos), P(slot), 0, rows, P(runs), seqs, P(w), P(o), pkg.DT_BF16, H * D, s))], 10)
             # bytes: projections, decays and gates in, outputs out, the state once. Operations: decay, two sums, one update per element of the state
             add("delta_rows (3 launches)", f"H={H} G={G} {seqs} x {n} rows", us, rows * (4.0 * ch + 8.0 * H * D + 2 * H * D) + 8.0 * seqs * H * D * D, flops32=7.0 * rows * H * D * D)

@@ -5,10 +5,20 @@
 //
 //   delta_one_kernel      decoded tokens, one row per sequence: convolution, unit norms, decay, state, output norm and gate
 //                         in one launch. A head's columns may be split over a cluster, which shares the output's square sum
-//   delta_prepare_kernel  portions: convolutions, unit norms, decays, steps and k . q of all rows, a warp per head
-//   delta_scan_kernel     portions: the recurrence. A CTA keeps 32 columns of a head's state in registers and walks the
-//                         run's tokens, which arrive through a ring of shared memory; 8 lanes share a column
+//   delta_prepare_kernel  portions, cut into chunks of eight tokens: everything of a chunk that does not depend on the state, a
+//                         warp per chunk and head
+//   delta_scan_kernel     portions: the recurrence, a chunk at a time, on the tensor cores. A CTA keeps 16 columns of a
+//                         head's state as accumulators, its warps a share of the key channels each
 //   delta_output_kernel   portions: output norm and gate, a warp per (row, head)
+//
+// A chunk of eight tokens, G_i the product of the decays up to token i, G_ij of those after j up to i (all products of
+// factors below one, nothing is ever divided by a decay): the sums over the state before the chunk are R_i = (k_i G_i)^T S
+// and (q_i G_i)^T S, and with A_ij = (k_i G_ij) . k_j, B_ij = (q_i G_ij) . k_j (B_ii = q_i . k_i)
+//   u_i = beta_i (v_i - R_i - sum_j<i A_ij u_j)  =  M (v - R),   M = (1 + beta A)^-1 beta,
+//   o_i = (q_i G_i)^T S + sum_j<=i B_ij u_j,   S <- G_8 S + sum_j (k_j G_8j) u_j^T.
+// Every product of matrices is fp32 to rounding: operands are split into two tf32 parts, and three products of the parts
+// are added in fp32. Accumulators of one product have the layout of the next one's left operand when the columns of
+// both operands are taken in the order 0 2 4 6 1 3 5 7, so nothing moves between lanes.
 //
 // A sequence's latest projections lie in a ring of `taps` entries, position p in entry p mod taps: a token reads the
 // entries before its own and writes its own, so the heads that share a key may do both in any order.
@@ -19,29 +29,52 @@ namespace {
 constexpr float kUnitEps = 1e-6f;
 
 __device__ __forceinline__ int delta_channels(const cmlb200_delta& a) { return 2 * a.kv_heads * a.dim + a.heads * a.vdim; }
-__device__ __forceinline__ float softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
-__device__ __forceinline__ float decay(const cmlb200_delta& a, int h, int i, float z) { return expf(-a.rate[h] * softplus(z + a.dt_bias[i])); }
+__device__ __forceinline__ float silu_fast(float z) { return __fdividef(z, 1.0f + __expf(-z)); }
+// log(1 + e^z) = max(z, 0) + 2 artanh(e / (2 + e)) with e = e^-|z|: the argument of the series is at most 1/3, and nothing
+// cancels where e is small.
+__device__ __forceinline__ float softplus(float z) {
+    const float e = __expf(-fabsf(z)), s = __fdividef(e, 2.0f + e), w = s * s;
+    float p = 1.0f / 15.0f;
+    p = fmaf(p, w, 1.0f / 13.0f);
+    p = fmaf(p, w, 1.0f / 11.0f);
+    p = fmaf(p, w, 1.0f / 9.0f);
+    p = fmaf(p, w, 1.0f / 7.0f);
+    p = fmaf(p, w, 1.0f / 5.0f);
+    p = fmaf(p, w, 1.0f / 3.0f);
+    p = fmaf(p, w, 1.0f);
+    return fmaf(2.0f * s, p, fmaxf(z, 0.f));
+}
+__device__ __forceinline__ float decay(float rate, float z) { return expf(-rate * softplus(z)); }
 __device__ __forceinline__ float delta_scale(const cmlb200_delta& a) { return a.out_scale == 0.f ? 1.f : a.out_scale; }
 
-// Channel c at a row: the row's own projection and those of the tokens before it, from the rows in front (`back` of them belong to the
-// same sequence's portion) or from the ring.
-__device__ __forceinline__ float convolve(const cmlb200_delta& a, const float* __restrict__ proj, int ld, const float* __restrict__ ring, int channels, int c, int p,
-                                          int back) {
-    const float* x = proj + a.col + c;
-    float y = a.conv[(size_t)(a.taps - 1) * channels + c] * x[0];
-    for (int t = 1; t < a.taps && t <= p; t++) {
-        const float v = t <= back ? x[-(ptrdiff_t)t * ld] : ring[(size_t)((p - t) % a.taps) * channels + c];
-        y = fmaf(a.conv[(size_t)(a.taps - 1 - t) * channels + c], v, y);
+// Channel c at a decoded token's row: its own projection and those of the tokens before it, from the ring. T: the number of taps
+// where it is known (all loads are then under way together), 0: any.
+template <int T>
+__device__ __forceinline__ float convolve(const cmlb200_delta& a, const float* __restrict__ proj, const float* __restrict__ ring, int channels, int c, int p) {
+    const float now = proj[a.col + c];
+    if constexpr (T > 0) {
+        float w[T], x[T];
+#pragma unroll
+        for (int t = 0; t < T; t++) {
+            w[t] = a.conv[(size_t)(T - 1 - t) * channels + c];
+            x[t] = t == 0 ? now : (t <= p ? ring[(size_t)((p - t) % T) * channels + c] : 0.f);
+        }
+        float y = 0.f;
+#pragma unroll
+        for (int t = 0; t < T; t++) y = fmaf(w[t], x[t], y);
+        return silu_fast(y);
     }
-    return silu(y);
+    float y = a.conv[(size_t)(a.taps - 1) * channels + c] * now;
+    for (int t = 1; t < a.taps && t <= p; t++) y = fmaf(a.conv[(size_t)(a.taps - 1 - t) * channels + c], ring[(size_t)((p - t) % a.taps) * channels + c], y);
+    return silu_fast(y);
 }
 
 constexpr int ONE_THREADS = 256, ONE_WARPS = ONE_THREADS / 32;
 
 // grid = (splits, heads, rows), clusters of `splits` CTAs along x. Thread (rg, c): four columns 4c of every `groups`-th row
 // from rg on; RPT: room for those rows. lanes: threads across the columns of a CTA, a power of two.
-template <typename TO, int RPT>
-__global__ void __launch_bounds__(ONE_THREADS)
+template <typename TO, int RPT, int T>
+__global__ void __launch_bounds__(ONE_THREADS, RPT <= 4 ? 4 : (RPT <= 8 ? 3 : (RPT <= 16 ? 2 : 1)))
 delta_one_kernel(const cmlb200_delta a, const float* __restrict__ proj, int ld, const float* __restrict__ dec, int ld_dec, const float* __restrict__ gate, int ld_gate,
                  const int* __restrict__ row_pos, const int* __restrict__ row_slot, int cols, int lanes, TO* __restrict__ out, int out_ld) {
     extern __shared__ __align__(16) float sm[];
@@ -53,11 +86,8 @@ delta_one_kernel(const cmlb200_delta a, const float* __restrict__ proj, int ld, 
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int channels = delta_channels(a), group = a.heads / a.kv_heads, kh = h / group;
     const int c = tid & (lanes - 1), rg = tid / lanes, groups = ONE_THREADS / lanes, c0 = rank * cols + 4 * c;
-    dep_wait();
-    dep_trigger();
+    // positions, slots and states do not come from the launch in front, so the states are under way while that one ends
     const int p = row_pos[r], slot = row_slot[r];
-    const float* row = proj + (size_t)r * ld;
-    float* ring = a.ring + (size_t)slot * a.taps * channels;
     float4* state = reinterpret_cast<float4*>(a.state + ((size_t)slot * a.heads + h) * a.dim * a.vdim_ld + c0);
     const bool mine = 4 * c < cols && c0 < a.vdim_ld;
     float4 S[RPT];
@@ -66,26 +96,23 @@ delta_one_kernel(const cmlb200_delta a, const float* __restrict__ proj, int ld, 
         const int d = rg + i * groups;
         S[i] = mine && p > 0 && d < a.dim ? state[(size_t)d * (a.vdim_ld >> 2)] : make_float4(0.f, 0.f, 0.f, 0.f);
     }
+    dep_wait();
+    dep_trigger();
+    const float* row = proj + (size_t)r * ld;
+    float* ring = a.ring + (size_t)slot * a.taps * channels;
     float sq = 0.f, sk = 0.f;
     const bool keeps = rank == 0 && h == kh * group;
-    for (int d = tid; d < a.dim; d += ONE_THREADS) {
-        const int cq = kh * a.dim + d, ck = a.kv_heads * a.dim + cq;
-        const float q = convolve(a, row, ld, ring, channels, cq, p, 0), k = convolve(a, row, ld, ring, channels, ck, p, 0);
-        q_s[d] = q;
-        k_s[d] = k;
-        g_s[d] = decay(a, h, h * a.dim + d, dec[(size_t)r * ld_dec + h * a.dim + d]);
-        sq = fmaf(q, q, sq);
-        sk = fmaf(k, k, sk);
-        if (keeps) {
-            ring[(size_t)(p % a.taps) * channels + cq] = row[a.col + cq];
-            ring[(size_t)(p % a.taps) * channels + ck] = row[a.col + ck];
-        }
+    for (int i = tid; i < 2 * a.dim + cols; i += ONE_THREADS) {        // q, k and this CTA's values
+        const int which = i < a.dim ? 0 : (i < 2 * a.dim ? 1 : 2), d = i - which * a.dim, col = rank * cols + d;
+        const int ch = which == 2 ? 2 * a.kv_heads * a.dim + h * a.vdim + col : (which * a.kv_heads + kh) * a.dim + d;
+        const bool have = which < 2 || col < a.vdim;
+        const float y = have ? convolve<T>(a, row, ring, channels, ch, p) : 0.f;
+        (which == 0 ? q_s : (which == 1 ? k_s : v_s))[d] = y;
+        sq += which == 0 ? y * y : 0.f;
+        sk += which == 1 ? y * y : 0.f;
+        if (have && (keeps || which == 2)) ring[(size_t)(p % a.taps) * channels + ch] = row[a.col + ch];
     }
-    for (int j = tid; j < cols; j += ONE_THREADS) {
-        const int d = rank * cols + j, cv = 2 * a.kv_heads * a.dim + h * a.vdim + d;
-        v_s[j] = d < a.vdim ? convolve(a, row, ld, ring, channels, cv, p, 0) : 0.f;
-        if (d < a.vdim) ring[(size_t)(p % a.taps) * channels + cv] = row[a.col + cv];
-    }
+    for (int d = tid; d < a.dim; d += ONE_THREADS) g_s[d] = decay(a.rate[h], dec[(size_t)r * ld_dec + h * a.dim + d] + a.dt_bias[h * a.dim + d]);
     const float2 ss = block_sum2(sq, sk, red2);        // the barriers inside also publish q_s .. v_s
     const float iq = 1.0f / sqrtf(ss.x + kUnitEps) / sqrtf((float)a.dim), ik = 1.0f / sqrtf(ss.y + kUnitEps);
     const float beta = sigmoidf(row[a.col + channels + h]);
@@ -169,243 +196,404 @@ delta_one_kernel(const cmlb200_delta a, const float* __restrict__ proj, int ld, 
     }
 }
 
-// A work row of a portion's token: [q (kv_heads dim) | k (kv_heads dim) | v, later o (heads vdim) | beta (heads) | k . q (kv_heads)].
-__host__ __device__ inline int work_ld(const cmlb200_delta& a) { return (2 * a.kv_heads * a.dim + a.heads * a.vdim + a.heads + a.kv_heads + 3) & ~3; }
+// What the scan needs of a chunk and head: per 8 key channels (a tile) k G and q G as [token][k k q q, four times], k G_8 as
+// [channel][token], G_8; then M and B as [token][token], and the factors that make k and q unit vectors, which none of the
+// first three carry. tiles: 8-channel tiles, a size the scan is built for.
+constexpr int CHUNK = 8;
+__host__ __device__ inline int scan_tiles(const cmlb200_delta& a) { return a.dim <= 32 ? 4 : (a.dim <= 64 ? 8 : (a.dim <= 128 ? 16 : 32)); }
+__host__ __device__ inline int packet_floats(int tiles) { return tiles * 200 + 144; }
+__host__ __device__ inline int value_ld(const cmlb200_delta& a) { return (a.heads * a.vdim + 3) & ~3; }
+// A run's first packet: runs do not overlap, and each has one packet more than its rows' share at most.
+__device__ __forceinline__ int first_packet(const int4 run, int i, int first) { return (run.x - first) / CHUNK + i; }
 
-// grid = (rows, units / 8): a warp makes a key head's q and k, or a head's v, decays and step.
-__global__ void __launch_bounds__(256)
-delta_prepare_kernel(const cmlb200_delta a, const float* __restrict__ proj, int ld, float* __restrict__ dec, int ld_dec, const int* __restrict__ row_pos,
-                     const int* __restrict__ row_slot, int first, float* __restrict__ work) {
+// The sum over the warp of v[l] ends up on lane l.
+__device__ __forceinline__ float scatter_sums(float (&v)[32]) {
+    const int lane = threadIdx.x & 31;
+#pragma unroll
+    for (int n = 16; n > 0; n >>= 1) {
+        const bool upper = lane & n;
+#pragma unroll
+        for (int i = 0; i < n; i++) {
+            const float mine = upper ? v[n + i] : v[i], other = upper ? v[i] : v[n + i];
+            v[i] = mine + __shfl_xor_sync(0xffffffffu, other, n);
+        }
+    }
+    return v[0];
+}
+
+// grid = (packets, heads / 4). T: taps if known (all loads of a channel are then under way together), 0: any.
+template <int T>
+__global__ void __launch_bounds__(128, 3)
+delta_prepare_kernel(const cmlb200_delta a, const float* __restrict__ proj, int ld, const float* __restrict__ dec, int ld_dec, const int* __restrict__ row_pos,
+                     const int4* __restrict__ runs, int num_runs, int first, float* __restrict__ values, float* __restrict__ packets) {
+    __shared__ float sums[4][96], betas[4][CHUNK];
     dep_wait();
     dep_trigger();
-    const int r = first + blockIdx.x, unit = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-    if (unit >= a.kv_heads + a.heads) return;
-    const int channels = delta_channels(a), p = row_pos[r], slot = row_slot[r], kd = a.kv_heads * a.dim;
-    int back = 0;                                      // rows right in front that belong to the same portion: a step has one per sequence
-    while (back < a.taps - 1 && r - back - 1 >= first && row_slot[r - back - 1] == slot) back++;
-    const float* row = proj + (size_t)r * ld;
-    const float* ring = a.ring + (size_t)slot * a.taps * channels;
-    float* w = work + (size_t)blockIdx.x * work_ld(a);
-    if (unit < a.kv_heads) {
-        float sq = 0.f, sk = 0.f, kq = 0.f, q[8], k[8];
-#pragma unroll
-        for (int i = 0; i < 8; i++) {                  // dim up to 256
-            const int d = lane + 32 * i, c = unit * a.dim + d;
-            q[i] = 0.f; k[i] = 0.f;
-            if (d >= a.dim) continue;
-            q[i] = convolve(a, row, ld, ring, channels, c, p, back);
-            k[i] = convolve(a, row, ld, ring, channels, kd + c, p, back);
-            sq = fmaf(q[i], q[i], sq);
-            sk = fmaf(k[i], k[i], sk);
-        }
-        const float iq = 1.0f / sqrtf(lane_sum(sq) + kUnitEps) / sqrtf((float)a.dim), ik = 1.0f / sqrtf(lane_sum(sk) + kUnitEps);
-#pragma unroll
-        for (int i = 0; i < 8; i++) {
-            const int d = lane + 32 * i;
-            if (d >= a.dim) continue;
-            q[i] *= iq;
-            k[i] *= ik;
-            kq = fmaf(k[i], q[i], kq);
-            w[unit * a.dim + d] = q[i];
-            w[kd + unit * a.dim + d] = k[i];
-        }
-        kq = lane_sum(kq);
-        if (lane == 0) w[channels + a.heads + unit] = kq;
-        return;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, h = blockIdx.y * 4 + warp;
+    int at = -1, c0 = 0;                               // the run this packet belongs to, and the chunk's first token in it
+    for (int i0 = 0; i0 < num_runs && at < 0; i0 += 32) {
+        const int i = i0 + lane, c = i < num_runs ? (int)blockIdx.x - first_packet(runs[i], i, first) : -1;
+        const unsigned hit = __ballot_sync(0xffffffffu, c >= 0 && c * CHUNK < (i < num_runs ? runs[i].y : 0));
+        if (hit) { at = i0 + __ffs(hit) - 1; c0 = __shfl_sync(0xffffffffu, c, __ffs(hit) - 1) * CHUNK; }
     }
-    const int h = unit - a.kv_heads;
-    for (int d = lane; d < a.vdim; d += 32) {
-        const int c = 2 * kd + h * a.vdim + d;
-        w[c] = convolve(a, row, ld, ring, channels, c, p, back);
+    if (at < 0 || h >= a.heads) return;
+    const int4 run = runs[at];
+    const int n = run.y, count = min(CHUNK, n - c0), p0 = row_pos[run.x], tiles = scan_tiles(a), channels = delta_channels(a);
+    const int kh = h / (a.heads / a.kv_heads), kd = a.kv_heads * a.dim;
+    const float* ring = a.ring + (size_t)run.z * a.taps * channels;
+    const float* rows = proj + (size_t)run.x * ld + a.col;
+    constexpr int PAST = T > 0 ? T - 1 : 0;
+    static_assert(PAST <= CHUNK, "a chunk's history is the chunk before it or the ring");
+    int off[CHUNK], past[PAST + 1];                    // of the rows that a chunk's convolutions read (past the end: the last), and of the tokens before it
+    bool seen[PAST + 1];
+#pragma unroll
+    for (int j = 0; j < CHUNK; j++) off[j] = min(c0 + j, n - 1) * ld;
+    const float* before = c0 > 0 ? rows : ring;
+#pragma unroll
+    for (int j = 0; j < PAST; j++) {
+        const int t = c0 + j - PAST;
+        seen[j] = p0 + t >= 0;
+        past[j] = c0 > 0 ? t * ld : max(p0 + t, 0) % T * channels;
     }
-    float* g = dec + (size_t)r * ld_dec + h * a.dim;
-    for (int d = lane; d < a.dim; d += 32) g[d] = decay(a, h, h * a.dim + d, g[d]);
-    if (lane == 0) w[channels + h] = sigmoidf(row[a.col + channels + h]);
-}
-
-__device__ __forceinline__ uint64_t pack2(float x, float y) {
-    uint64_t v;
-    asm("mov.b64 %0, {%1, %2};" : "=l"(v) : "f"(x), "f"(y));
-    return v;
-}
-__device__ __forceinline__ float sum2(uint64_t v) {
-    float x, y;
-    asm("mov.b64 {%0, %1}, %2;" : "=f"(x), "=f"(y) : "l"(v));
-    return x + y;
-}
-__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
-    uint64_t v;
-    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(v) : "l"(a), "l"(b), "l"(c));
-    return v;
-}
-__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
-    uint64_t v;
-    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(v) : "l"(a), "l"(b));
-    return v;
-}
-template <int N> __device__ __forceinline__ void copy_async(float* dst, const float* src) {
-    if (N == 4) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_addr(dst)), "l"(src) : "memory");
-    else asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_addr(dst)), "l"(src) : "memory");
-}
-
-constexpr int SCAN_THREADS = 128, SCAN_COLS = 32;
-
-// grid = (column slices, heads, runs). Lane (rg, cl) of a warp: rows 32 i + 4 rg .. + 3 of two columns; pairs of neighbouring
-// rows share a register pair. RPL: rows per lane, a multiple of 4. N: floats per copy.
-template <int RPL, int N>
-__global__ void __launch_bounds__(SCAN_THREADS)
-delta_scan_kernel(const cmlb200_delta a, const float* __restrict__ proj, int ld, const float* __restrict__ dec, int ld_dec, const int* __restrict__ row_pos,
-                  const int4* __restrict__ runs, int first, float* __restrict__ work) {
-    constexpr int DIM = RPL * 8, SCAN_TOKENS = RPL > 16 ? 4 : 8;       // tokens per stage
-    __shared__ __align__(16) float ks[2][SCAN_TOKENS][DIM], qs[2][SCAN_TOKENS][DIM], gs[2][SCAN_TOKENS][DIM], vs[2][SCAN_TOKENS][SCAN_COLS];
-    __shared__ float bs[2][SCAN_TOKENS], kqs[2][SCAN_TOKENS];
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, rg = lane >> 2, cl = lane & 3;
-    const int h = blockIdx.y, group = a.heads / a.kv_heads, kh = h / group, channels = delta_channels(a), wld = work_ld(a);
-    const int col0 = blockIdx.x * SCAN_COLS, mycol = col0 + warp * 8 + cl * 2;
-    for (int i = tid; i < 2 * SCAN_TOKENS * DIM; i += SCAN_THREADS) { (&ks[0][0][0])[i] = 0.f; (&qs[0][0][0])[i] = 0.f; (&gs[0][0][0])[i] = 0.f; }
-    for (int i = tid; i < 2 * SCAN_TOKENS * SCAN_COLS; i += SCAN_THREADS) (&vs[0][0][0])[i] = 0.f;
-    dep_wait();
-    dep_trigger();
-    const int4 run = runs[blockIdx.z];
-    const int r0 = run.x, n = run.y, slot = run.z, p0 = row_pos[r0];
-    float* o = work + (size_t)(r0 - first) * wld + 2 * a.kv_heads * a.dim + h * a.vdim;
-    __syncthreads();                                   // the zeros behind dim and vdim are in place
-    auto fetch = [&](int b) {
-        const int t0 = b * SCAN_TOKENS, st = b & 1, kd = a.dim / N, kv = min(SCAN_COLS, a.vdim - col0) / N;
-        for (int i = tid; i < SCAN_TOKENS * kd; i += SCAN_THREADS) {
-            const int t = i / kd, d = (i - t * kd) * N;
-            if (t0 + t >= n) break;
-            const float* w = work + (size_t)(r0 - first + t0 + t) * wld + kh * a.dim + d;
-            copy_async<N>(&qs[st][t][d], w);
-            copy_async<N>(&ks[st][t][d], w + a.kv_heads * a.dim);
-            copy_async<N>(&gs[st][t][d], dec + (size_t)(r0 + t0 + t) * ld_dec + h * a.dim + d);
-        }
-        for (int i = tid; i < SCAN_TOKENS * kv; i += SCAN_THREADS) {
-            const int t = i / kv, d = (i - t * kv) * N;
-            if (t0 + t >= n) break;
-            copy_async<N>(&vs[st][t][d], o + (size_t)(t0 + t) * wld + col0 + d);
-        }
-        if (tid < 2 * SCAN_TOKENS) {
-            const int t = tid >> 1;
-            if (t0 + t < n) {
-                const float* w = work + (size_t)(r0 - first + t0 + t) * wld + channels;
-                if (tid & 1) copy_async<1>(&kqs[st][t], w + a.heads + kh);
-                else copy_async<1>(&bs[st][t], w + h);
+    auto convolve_chunk = [&](int c, float (&y)[CHUNK]) {
+#pragma unroll
+        for (int j = 0; j < CHUNK; j++) y[j] = 0.f;
+        if constexpr (T > 0) {
+            float x[PAST + CHUNK];
+#pragma unroll
+            for (int j = 0; j < PAST; j++) x[j] = seen[j] ? before[past[j] + c] : 0.f;
+#pragma unroll
+            for (int j = 0; j < CHUNK; j++) x[PAST + j] = rows[off[j] + c];
+#pragma unroll
+            for (int t = 0; t < T; t++) {
+                const float w = a.conv[(T - 1 - t) * channels + c];
+#pragma unroll
+                for (int j = 0; j < CHUNK; j++) y[j] = fmaf(w, x[j + T - 1 - t], y[j]);
             }
+        } else {
+            for (int t = 0; t < a.taps; t++) {
+                const float w = a.conv[(a.taps - 1 - t) * channels + c];
+#pragma unroll
+                for (int j = 0; j < CHUNK; j++) {
+                    const int at = c0 + j - t;         // a token of the run, or before it
+                    const float x = at >= 0 ? rows[min(at, n - 1) * ld + c] : (p0 + at >= 0 ? ring[(p0 + at) % a.taps * channels + c] : 0.f);
+                    y[j] = fmaf(w, x, y[j]);
+                }
+            }
+        }
+#pragma unroll
+        for (int j = 0; j < CHUNK; j++) y[j] = j < count ? silu_fast(y[j]) : 0.f;
+    };
+    float* packet = packets + ((size_t)blockIdx.x * a.heads + h) * packet_floats(tiles);
+    float *kq = packet, *kt = kq + tiles * 128, *gt = kt + tiles * 64, *mat = gt + tiles * 8;
+    float acc[96];                                     // A_ij, j < i, then B_ij, j <= i, then the square sums of q and of k
+#pragma unroll
+    for (int i = 0; i < 96; i++) acc[i] = 0.f;
+    const float rate = a.rate[h];
+    for (int d = lane; d < tiles * 8; d += 32) {
+        float q[CHUNK], k[CHUNK], g[CHUNK], kg[CHUNK], qg[CHUNK], tail[CHUNK], run_g = 1.f;
+        const bool have = d < a.dim;
+        const int c = kh * a.dim + (have ? d : 0), gc = h * a.dim + (have ? d : 0);
+        const float bias = a.dt_bias[gc];
+#pragma unroll
+        for (int j = 0; j < CHUNK; j++) g[j] = dec[(size_t)(run.x + min(c0 + j, n - 1)) * ld_dec + gc];
+        convolve_chunk(c, q);
+        convolve_chunk(kd + c, k);
+#pragma unroll
+        for (int j = 0; j < CHUNK; j++) {
+            g[j] = j < count ? decay(rate, g[j] + bias) : 1.f;
+            if (!have) { q[j] = 0.f; k[j] = 0.f; }
+            run_g *= g[j];
+            kg[j] = k[j] * run_g;
+            qg[j] = q[j] * run_g;
+            acc[64 + j] = fmaf(q[j], q[j], acc[64 + j]);
+            acc[72 + j] = fmaf(k[j], k[j], acc[72 + j]);
+        }
+#pragma unroll
+        for (int j = 0; j < CHUNK; j++) {
+            float t = k[j];
+            acc[28 + j * (j + 1) / 2 + j] = fmaf(q[j], t, acc[28 + j * (j + 1) / 2 + j]);
+#pragma unroll
+            for (int i = j + 1; i < CHUNK; i++) {
+                t *= g[i];
+                acc[i * (i - 1) / 2 + j] = fmaf(k[i], t, acc[i * (i - 1) / 2 + j]);
+                acc[28 + i * (i + 1) / 2 + j] = fmaf(q[i], t, acc[28 + i * (i + 1) / 2 + j]);
+            }
+            tail[j] = t;
+        }
+        float* to = kq + (size_t)(d >> 3) * 128 + ((d & 7) >> 1) * 4 + (d & 1);
+#pragma unroll
+        for (int j = 0; j < CHUNK; j++) { to[j * 16] = kg[j]; to[j * 16 + 2] = qg[j]; }
+        gt[d] = run_g;
+        float4* end = reinterpret_cast<float4*>(kt + (size_t)d * CHUNK);
+        end[0] = make_float4(tail[0], tail[1], tail[2], tail[3]);
+        end[1] = make_float4(tail[4], tail[5], tail[6], tail[7]);
+    }
+#pragma unroll
+    for (int b = 0; b < 3; b++) {
+        float v[32];
+#pragma unroll
+        for (int i = 0; i < 32; i++) v[i] = acc[b * 32 + i];
+        sums[warp][b * 32 + lane] = scatter_sums(v);
+    }
+    if (lane < CHUNK) betas[warp][lane] = lane < count ? sigmoidf(rows[(size_t)(c0 + lane) * ld + channels + h]) : 0.f;
+    __syncwarp();
+    float* sum = sums[warp];
+    if (lane < CHUNK) {                                // from here on factors instead of square sums
+        sum[64 + lane] = 1.0f / sqrtf(sum[64 + lane] + kUnitEps) / sqrtf((float)a.dim);
+        sum[72 + lane] = 1.0f / sqrtf(sum[72 + lane] + kUnitEps);
+        mat[136 + lane] = sum[64 + lane];
+        mat[128 + lane] = sum[72 + lane];
+    }
+    __syncwarp();
+    const float *iq = sum + 64, *ik = sum + 72;
+    if (lane < CHUNK) {                                // a column of M by substitution
+        float x[CHUNK];
+#pragma unroll
+        for (int i = 0; i < CHUNK; i++) {
+            float s = 0.f;
+#pragma unroll
+            for (int j = 0; j < i; j++) s = fmaf(sum[i * (i - 1) / 2 + j] * ik[j], x[j], s);
+            x[i] = i < lane ? 0.f : betas[warp][i] * ((i == lane ? 1.f : 0.f) - ik[i] * s);
+            mat[i * CHUNK + lane] = x[i];
+        }
+    }
+    for (int e = lane; e < 64; e += 32) {
+        const int i = e >> 3, j = e & 7;
+        mat[64 + e] = j <= i ? sum[28 + i * (i + 1) / 2 + j] * iq[i] * ik[j] : 0.f;
+    }
+    for (int d = lane; d < a.vdim; d += 32) {
+        float v[CHUNK];
+        convolve_chunk(2 * kd + h * a.vdim + d, v);
+#pragma unroll
+        for (int j = 0; j < CHUNK; j++)
+            if (j < count) values[(size_t)(run.x - first + c0 + j) * value_ld(a) + h * a.vdim + d] = v[j];
+    }
+}
+
+// A number as two tf32 parts (10 bits behind the leading one), the first rounded to nearest; of the second the product drops what is below
+// its own 10 bits.
+__device__ __forceinline__ void split_tf32(float v, uint32_t& hi, uint32_t& lo) {
+    hi = (__float_as_uint(v) + 0x1000u) & 0xffffe000u;
+    lo = __float_as_uint(v - __uint_as_float(hi));
+}
+__device__ __forceinline__ void mma_tf32(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm("mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+// Accumulators as a left operand
+__device__ __forceinline__ void split_rows(const float (&c)[4], uint32_t (&hi)[4], uint32_t (&lo)[4]) {
+    split_tf32(c[0], hi[0], lo[0]);
+    split_tf32(c[2], hi[1], lo[1]);
+    split_tf32(c[1], hi[2], lo[2]);
+    split_tf32(c[3], hi[3], lo[3]);
+}
+
+constexpr int SCAN_COLS = 16, SCAN_WARPS = 4;          // columns of a CTA; warps that share the key channels
+
+// grid = (column slices, heads, runs); SCAN_STAGES: packets under way. A CTA keeps 16 columns of a state, each warp TILES tiles of 8 key channels of them. Lane (g, t):
+// columns g and g + 8, channels 2t and 2t + 1 of every tile, tokens 2t and 2t + 1 of a chunk.
+template <int TILES, int SCAN_STAGES>
+__global__ void __launch_bounds__(SCAN_WARPS * 32)
+delta_scan_kernel(const cmlb200_delta a, const float* __restrict__ proj, int ld, const int* __restrict__ row_pos, const int4* __restrict__ runs, int first,
+                  float* __restrict__ values, const float* __restrict__ packets) {
+    extern __shared__ __align__(16) float stage[];
+    constexpr int ALL = TILES * SCAN_WARPS, FLOATS = ALL * 200 + 144, AHEAD = 3;            // AHEAD: chunks whose values are under way
+    __shared__ __align__(16) float4 part[2][SCAN_WARPS][2][32];        // the warps' shares of both sums, by turns
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
+    const int h = blockIdx.y, group = a.heads / a.kv_heads, kh = h / group, vld = value_ld(a);
+    const int col = blockIdx.x * SCAN_COLS + g, d0 = warp * TILES * 8;
+    dep_wait();
+    const int4 run = runs[blockIdx.z];
+    const int n = run.y, slot = run.z, p0 = row_pos[run.x], chunks = (n + CHUNK - 1) / CHUNK;
+    const float* src = packets + ((size_t)first_packet(run, blockIdx.z, first) * a.heads + h) * FLOATS;
+    float* vrow = values + (size_t)(run.x - first) * vld + h * a.vdim;
+    auto fetch = [&](int c) {
+        if (c < chunks) {
+            const float* from = src + (size_t)c * a.heads * FLOATS;
+            float* to = stage + (c % SCAN_STAGES) * FLOATS;
+#pragma unroll 8
+            for (int i = tid * 4; i < FLOATS; i += SCAN_WARPS * 32 * 4) cp16(smem_addr(to + i), from + i);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
-    fetch(0);
-    uint64_t S[2][RPL / 2];
+    auto fetch_values = [&](int c, float (&v)[4]) {
+#pragma unroll
+        for (int e = 0; e < 4; e++) {
+            const int tok = c * CHUNK + 2 * t + (e & 1), cc = col + (e >> 1) * 8;
+            v[e] = tok < n && cc < a.vdim ? vrow[(size_t)tok * vld + cc] : 0.f;
+        }
+    };
+    for (int c = 0; c < SCAN_STAGES - 1; c++) fetch(c);
+    float v_next[AHEAD][4];
+#pragma unroll
+    for (int k = 0; k < AHEAD; k++) fetch_values(k, v_next[k]);
+    float S[TILES][4];
     float* state = a.state + ((size_t)slot * a.heads + h) * a.dim * a.vdim_ld;
 #pragma unroll
-    for (int i = 0; i < RPL / 4; i++)
+    for (int i = 0; i < TILES; i++)
 #pragma unroll
-        for (int j = 0; j < 4; j += 2) {
-            const int d = i * 32 + rg * 4 + j;
-            const bool c_ok = mycol < a.vdim_ld && p0 > 0;              // vdim_ld is a multiple of 4 and mycol is even
-            const float2 z = make_float2(0.f, 0.f);
-            const float2 x = c_ok && d < a.dim ? *reinterpret_cast<const float2*>(state + (size_t)d * a.vdim_ld + mycol) : z;
-            const float2 y = c_ok && d + 1 < a.dim ? *reinterpret_cast<const float2*>(state + (size_t)(d + 1) * a.vdim_ld + mycol) : z;
-            S[0][i * 2 + j / 2] = pack2(x.x, y.x);
-            S[1][i * 2 + j / 2] = pack2(x.y, y.y);
+        for (int e = 0; e < 4; e++) {
+            const int d = d0 + i * 8 + 2 * t + (e & 1), cc = col + (e >> 1) * 8;
+            S[i][e] = p0 > 0 && d < a.dim && cc < a.vdim ? state[(size_t)d * a.vdim_ld + cc] : 0.f;
         }
     if (blockIdx.x == 0) {                             // the latest projections; nobody reads the ring in this launch
-        const int keep = min(n, a.taps - 1), kd = a.kv_heads * a.dim;
-        for (int t = n - keep; t < n; t++) {
-            float* ring = a.ring + ((size_t)slot * a.taps + (p0 + t) % a.taps) * channels;
-            const float* row = proj + (size_t)(r0 + t) * ld + a.col;
+        const int keep = min(n, a.taps - 1), kd = a.kv_heads * a.dim, channels = delta_channels(a);
+        for (int k = n - keep; k < n; k++) {
+            float* ring = a.ring + ((size_t)slot * a.taps + (p0 + k) % a.taps) * channels;
+            const float* row = proj + (size_t)(run.x + k) * ld + a.col;
             if (h == kh * group)
-                for (int d = tid; d < a.dim; d += SCAN_THREADS) {
+                for (int d = tid; d < a.dim; d += blockDim.x) {
                     ring[kh * a.dim + d] = row[kh * a.dim + d];
                     ring[kd + kh * a.dim + d] = row[kd + kh * a.dim + d];
                 }
-            for (int d = tid; d < a.vdim; d += SCAN_THREADS) ring[2 * kd + h * a.vdim + d] = row[2 * kd + h * a.vdim + d];
+            for (int d = tid; d < a.vdim; d += blockDim.x) ring[2 * kd + h * a.vdim + d] = row[2 * kd + h * a.vdim + d];
         }
     }
-    const int blocks = (n + SCAN_TOKENS - 1) / SCAN_TOKENS;
-    for (int b = 0; b < blocks; b++) {
-        if (b + 1 < blocks) {
-            fetch(b + 1);
-            asm volatile("cp.async.wait_group 1;" ::: "memory");
-        } else {
-            asm volatile("cp.async.wait_group 0;" ::: "memory");
+    for (int c = 0; c < chunks; c++) {
+        asm volatile("cp.async.wait_group %0;" ::"n"(SCAN_STAGES - 2) : "memory");
+        __syncthreads();                               // this chunk is there, and the one before it is read
+        const float* st = stage + (c % SCAN_STAGES) * FLOATS;
+        const float *kq = st + warp * TILES * 128, *kt = st + ALL * 128 + warp * TILES * 64, *gt = st + ALL * 192 + d0, *mat = st + ALL * 200;
+        float rk[3][4] = {}, rq[3][4] = {};
+#pragma unroll
+        for (int i = 0; i < TILES; i++) {
+            const float4 x = *reinterpret_cast<const float4*>(kq + i * 128 + g * 16 + t * 4);
+            uint32_t hi[4], lo[4], k0, k1, l0, l1, q0, q1, m0, m1;
+            split_rows(S[i], hi, lo);
+            split_tf32(x.x, k0, l0);
+            split_tf32(x.y, k1, l1);
+            split_tf32(x.z, q0, m0);
+            split_tf32(x.w, q1, m1);
+            mma_tf32(rk[0], hi, k0, k1);
+            mma_tf32(rq[0], hi, q0, q1);
+            mma_tf32(rk[1], hi, l0, l1);
+            mma_tf32(rq[1], hi, m0, m1);
+            mma_tf32(rk[2], lo, k0, k1);
+            mma_tf32(rq[2], lo, q0, q1);
         }
+        float v[4];
+#pragma unroll
+        for (int e = 0; e < 4; e++) {
+            v[e] = v_next[0][e];
+#pragma unroll
+            for (int k = 1; k < AHEAD; k++) v_next[k - 1][e] = v_next[k][e];
+            rk[0][e] += rk[1][e] + rk[2][e];
+            rq[0][e] += rq[1][e] + rq[2][e];
+        }
+        part[c & 1][warp][0][lane] = make_float4(rk[0][0], rk[0][1], rk[0][2], rk[0][3]);
+        part[c & 1][warp][1][lane] = make_float4(rq[0][0], rq[0][1], rq[0][2], rq[0][3]);
+        fetch(c + SCAN_STAGES - 1);                    // into the stage that the barrier above released
+        fetch_values(c + AHEAD, v_next[AHEAD - 1]);
         __syncthreads();
-        const int st = b & 1, tokens = min(SCAN_TOKENS, n - b * SCAN_TOKENS);
-        for (int t = 0; t < tokens; t++) {
-            const ulonglong2 *k4 = reinterpret_cast<const ulonglong2*>(ks[st][t]), *q4 = reinterpret_cast<const ulonglong2*>(qs[st][t]), *g4 = reinterpret_cast<const ulonglong2*>(gs[st][t]);
-            uint64_t k[RPL / 2], ak[2][2] = {}, aq[2][2] = {};
+        const float2 ik = *reinterpret_cast<const float2*>(mat + 128 + 2 * t), iq = *reinterpret_cast<const float2*>(mat + 136 + 2 * t);
+        float4 k = part[c & 1][0][0][lane], q = part[c & 1][0][1][lane];
 #pragma unroll
-            for (int i = 0; i < RPL / 4; i++) {
-                const ulonglong2 g = g4[i * 8 + rg], kk = k4[i * 8 + rg], qq = q4[i * 8 + rg];
-                k[2 * i] = kk.x;
-                k[2 * i + 1] = kk.y;
+        for (int w = 1; w < SCAN_WARPS; w++) {
+            const float4 x = part[c & 1][w][0][lane], y = part[c & 1][w][1][lane];
+            k.x += x.x; k.y += x.y; k.z += x.z; k.w += x.w;
+            q.x += y.x; q.y += y.y; q.z += y.z; q.w += y.w;
+        }
+        const float x[4] = {fmaf(-ik.x, k.x, v[0]), fmaf(-ik.y, k.y, v[1]), fmaf(-ik.x, k.z, v[2]), fmaf(-ik.y, k.w, v[3])};
+        uint32_t hi[4], lo[4], b0, b1, c0, c1;
+        float u[4] = {}, u1[4] = {}, u2[4] = {};
+        float2 m = *reinterpret_cast<const float2*>(mat + g * 8 + 2 * t);
+        split_rows(x, hi, lo);
+        split_tf32(m.x, b0, c0);
+        split_tf32(m.y, b1, c1);
+        mma_tf32(u, hi, b0, b1);
+        mma_tf32(u1, hi, c0, c1);
+        mma_tf32(u2, lo, b0, b1);
 #pragma unroll
-                for (int c = 0; c < 2; c++) {
-                    S[c][2 * i] = mul2(S[c][2 * i], g.x);
-                    S[c][2 * i + 1] = mul2(S[c][2 * i + 1], g.y);
-                    ak[c][0] = fma2(S[c][2 * i], kk.x, ak[c][0]);
-                    ak[c][1] = fma2(S[c][2 * i + 1], kk.y, ak[c][1]);
-                    aq[c][0] = fma2(S[c][2 * i], qq.x, aq[c][0]);
-                    aq[c][1] = fma2(S[c][2 * i + 1], qq.y, aq[c][1]);
-                }
-            }
-            float sk[2], sq[2];
+        for (int e = 0; e < 4; e++) u[e] += u1[e] + u2[e];
+        if (warp == (c & (SCAN_WARPS - 1))) {          // the output, a chunk each in turn
+            float o[4] = {iq.x * q.x, iq.y * q.y, iq.x * q.z, iq.y * q.w}, o1[4] = {}, o2[4] = {};
+            m = *reinterpret_cast<const float2*>(mat + 64 + g * 8 + 2 * t);
+            split_rows(u, hi, lo);
+            split_tf32(m.x, b0, c0);
+            split_tf32(m.y, b1, c1);
+            mma_tf32(o, hi, b0, b1);
+            mma_tf32(o1, hi, c0, c1);
+            mma_tf32(o2, lo, b0, b1);
 #pragma unroll
-            for (int c = 0; c < 2; c++) { sk[c] = sum2(ak[c][0]) + sum2(ak[c][1]); sq[c] = sum2(aq[c][0]) + sum2(aq[c][1]); }
-#pragma unroll
-            for (int x = 4; x < 32; x <<= 1) {
-#pragma unroll
-                for (int c = 0; c < 2; c++) { sk[c] += __shfl_xor_sync(0xffffffffu, sk[c], x); sq[c] += __shfl_xor_sync(0xffffffffu, sq[c], x); }
-            }
-            const float2 v = *reinterpret_cast<const float2*>(&vs[st][t][warp * 8 + cl * 2]);
-            const float beta = bs[st][t], kq = kqs[st][t], u0 = beta * (v.x - sk[0]), u1 = beta * (v.y - sk[1]);
-            const uint64_t uu0 = pack2(u0, u0), uu1 = pack2(u1, u1);
-#pragma unroll
-            for (int i = 0; i < RPL / 2; i++) { S[0][i] = fma2(k[i], uu0, S[0][i]); S[1][i] = fma2(k[i], uu1, S[1][i]); }
-            if (rg == 0) {
-                float* dst = o + (size_t)(b * SCAN_TOKENS + t) * wld + mycol;
-                if (mycol < a.vdim) dst[0] = fmaf(kq, u0, sq[0]);
-                if (mycol + 1 < a.vdim) dst[1] = fmaf(kq, u1, sq[1]);
+            for (int e = 0; e < 4; e++) {
+                const int tok = c * CHUNK + 2 * t + (e & 1), cc = col + (e >> 1) * 8;
+                if (tok < n && cc < a.vdim) vrow[(size_t)tok * vld + cc] = o[e] + (o1[e] + o2[e]);
             }
         }
-        __syncthreads();                               // this stage may be refilled
+        u[0] *= ik.x; u[1] *= ik.y; u[2] *= ik.x; u[3] *= ik.y;
+        split_rows(u, hi, lo);
+        constexpr int AT_ONCE = TILES < 4 ? TILES : 4; // a tile's three products wait for one another
+#pragma unroll
+        for (int i = 0; i < TILES; i += AT_ONCE) {
+            uint32_t k0[AT_ONCE], k1[AT_ONCE], l0[AT_ONCE], l1[AT_ONCE];
+#pragma unroll
+            for (int j = 0; j < AT_ONCE; j++) {
+                const float2 y = *reinterpret_cast<const float2*>(kt + (i + j) * 64 + g * 8 + 2 * t), f = *reinterpret_cast<const float2*>(gt + (i + j) * 8 + 2 * t);
+                split_tf32(y.x, k0[j], l0[j]);
+                split_tf32(y.y, k1[j], l1[j]);
+                S[i + j][0] *= f.x; S[i + j][1] *= f.y; S[i + j][2] *= f.x; S[i + j][3] *= f.y;
+            }
+#pragma unroll
+            for (int j = 0; j < AT_ONCE; j++) mma_tf32(S[i + j], hi, k0[j], k1[j]);
+#pragma unroll
+            for (int j = 0; j < AT_ONCE; j++) mma_tf32(S[i + j], hi, l0[j], l1[j]);
+#pragma unroll
+            for (int j = 0; j < AT_ONCE; j++) mma_tf32(S[i + j], lo, k0[j], k1[j]);
+        }
     }
+    dep_trigger();
 #pragma unroll
-    for (int i = 0; i < RPL / 4; i++)
+    for (int i = 0; i < TILES; i++)
 #pragma unroll
-        for (int j = 0; j < 4; j += 2) {
-            const int d = i * 32 + rg * 4 + j;
-            float x0, x1, y0, y1;
-            asm("mov.b64 {%0, %1}, %2;" : "=f"(x0), "=f"(y0) : "l"(S[0][i * 2 + j / 2]));
-            asm("mov.b64 {%0, %1}, %2;" : "=f"(x1), "=f"(y1) : "l"(S[1][i * 2 + j / 2]));
-            if (mycol < a.vdim_ld && d < a.dim) *reinterpret_cast<float2*>(state + (size_t)d * a.vdim_ld + mycol) = make_float2(x0, x1);
-            if (mycol < a.vdim_ld && d + 1 < a.dim) *reinterpret_cast<float2*>(state + (size_t)(d + 1) * a.vdim_ld + mycol) = make_float2(y0, y1);
+        for (int e = 0; e < 4; e++) {
+            const int d = d0 + i * 8 + 2 * t + (e & 1), cc = col + (e >> 1) * 8;
+            if (d < a.dim && cc < a.vdim) state[(size_t)d * a.vdim_ld + cc] = S[i][e];
         }
 }
 
-template <typename TO>
+// W: 4 where value rows, gates and outputs allow four columns at a time, else 1
+template <typename TO, int W>
 __global__ void __launch_bounds__(256)
-delta_output_kernel(const cmlb200_delta a, const float* __restrict__ work, const float* __restrict__ gate, int ld_gate, int first, TO* __restrict__ out, int out_ld) {
+delta_output_kernel(const cmlb200_delta a, const float* __restrict__ values, const float* __restrict__ gate, int ld_gate, int first, TO* __restrict__ out, int out_ld) {
+    constexpr int N = 8 / W;                           // vdim up to 256
     dep_wait();
     dep_trigger();
     const int h = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31, r = first + blockIdx.x;
     if (h >= a.heads) return;
-    const float* o = work + (size_t)blockIdx.x * work_ld(a) + 2 * a.kv_heads * a.dim + h * a.vdim;
+    const float* o = values + (size_t)blockIdx.x * value_ld(a) + h * a.vdim;
     const float* g = gate + (size_t)r * ld_gate + h * a.vdim;
-    float v[8], ss = 0.f;
+    TO* dst = out + (size_t)r * out_ld + h * a.vdim;
+    float v[N][W], z[N][W], ss = 0.f;
 #pragma unroll
-    for (int i = 0; i < 8; i++) {                      // vdim up to 256
-        const int d = lane + 32 * i;
-        v[i] = d < a.vdim ? o[d] : 0.f;
-        ss = fmaf(v[i], v[i], ss);
+    for (int i = 0; i < N; i++) {
+        const int d = (lane + 32 * i) * W;
+        const bool have = d < a.vdim;
+        if constexpr (W == 4) {
+            const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f), x = have ? *reinterpret_cast<const float4*>(o + d) : zero, y = have ? *reinterpret_cast<const float4*>(g + d) : zero;
+            v[i][0] = x.x; v[i][1] = x.y; v[i][2] = x.z; v[i][3] = x.w;
+            z[i][0] = y.x; z[i][1] = y.y; z[i][2] = y.z; z[i][3] = y.w;
+        } else {
+            v[i][0] = have ? o[d] : 0.f;
+            z[i][0] = have ? g[d] : 0.f;
+        }
+#pragma unroll
+        for (int e = 0; e < W; e++) ss = fmaf(v[i][e], v[i][e], ss);
     }
     const float inv = delta_scale(a) / sqrtf(lane_sum(ss) / (float)a.vdim + a.eps);
 #pragma unroll
-    for (int i = 0; i < 8; i++) {
-        const int d = lane + 32 * i;
-        if (d < a.vdim) out[(size_t)r * out_ld + h * a.vdim + d] = narrow<TO>(v[i] * inv * a.norm[d] * sigmoidf(g[d]));
+    for (int i = 0; i < N; i++) {
+        const int d = (lane + 32 * i) * W;
+        if (d >= a.vdim) continue;
+        TO n[W];
+#pragma unroll
+        for (int e = 0; e < W; e++) n[e] = narrow<TO>(v[i][e] * inv * a.norm[d + e] * sigmoid_fast(z[i][e]));
+        if constexpr (W == 4) {
+            if constexpr (sizeof(TO) == 2) *reinterpret_cast<uint2*>(dst + d) = *reinterpret_cast<const uint2*>(n);
+            else *reinterpret_cast<float4*>(dst + d) = *reinterpret_cast<const float4*>(n);
+        } else {
+            dst[d] = n[0];
+        }
     }
 }
 
@@ -436,46 +624,65 @@ extern "C" int cmlb200_delta_one(const cmlb200_delta* a, const float* d_proj, in
         return (a->dim + ONE_THREADS / lanes - 1) / (ONE_THREADS / lanes);
     };
     int splits = 1, cols, lanes, rpt = shape(1, cols, lanes);
-    while (splits < 8 && cols > 16 && (rpt > 16 || (long long)rows * a->heads * splits < 2 * cmlb_num_sms())) rpt = shape(splits *= 2, cols, lanes);
+    while (splits < 8 && cols > 16 && (rpt > 8 || (long long)rows * a->heads * splits < 2 * cmlb_num_sms())) rpt = shape(splits *= 2, cols, lanes);
     CMLB_REQUIRE(rpt <= 32, "cmlb200_delta_one: states of %d x %d", a->dim, a->vdim);
     const size_t smem = sizeof(float) * ((size_t)3 * ((a->dim + 3) & ~3) + cols + (size_t)8 * lanes * 8 + 8);
     const dim3 grid(splits, a->heads, rows);
-#define DO_LAUNCH(TO, RPT) CMLB_CUDA(launch_chain(delta_one_kernel<TO, RPT>, grid, dim3(ONE_THREADS), smem, splits, as_stream(stream), *a, d_proj, ld, d_decay, ld_decay, \
-                                                  d_gate, ld_gate, d_row_pos, d_row_slot, cols, lanes, (TO*)d_out, out_ld))
-#define DO_ROWS(TO) do { if (rpt <= 4) DO_LAUNCH(TO, 4); else if (rpt <= 8) DO_LAUNCH(TO, 8); else if (rpt <= 16) DO_LAUNCH(TO, 16); else DO_LAUNCH(TO, 32); } while (0)
+#define DO_LAUNCH(TO, RPT, T) CMLB_CUDA(launch_chain(delta_one_kernel<TO, RPT, T>, grid, dim3(ONE_THREADS), smem, splits, as_stream(stream), *a, d_proj, ld, d_decay, \
+                                                     ld_decay, d_gate, ld_gate, d_row_pos, d_row_slot, cols, lanes, (TO*)d_out, out_ld))
+#define DO_TAPS(TO, RPT) do { if (a->taps == 4) DO_LAUNCH(TO, RPT, 4); else DO_LAUNCH(TO, RPT, 0); } while (0)
+#define DO_ROWS(TO) do { if (rpt <= 4) DO_TAPS(TO, 4); else if (rpt <= 8) DO_TAPS(TO, 8); else if (rpt <= 16) DO_TAPS(TO, 16); else DO_TAPS(TO, 32); } while (0)
     if (out_dtype == CMLB200_DT_BF16) DO_ROWS(__nv_bfloat16);
     else DO_ROWS(float);
 #undef DO_ROWS
+#undef DO_TAPS
 #undef DO_LAUNCH
     return CMLB200_OK;
 }
 
-extern "C" int cmlb200_delta_work_floats(const cmlb200_delta* a) { return a ? work_ld(*a) : 0; }
+extern "C" long cmlb200_delta_work_floats(const cmlb200_delta* a, int rows, int runs) {
+    return a ? (long)rows * value_ld(*a) + (long)(rows / CHUNK + runs) * a->heads * packet_floats(scan_tiles(*a)) : 0;
+}
 
-extern "C" int cmlb200_delta_rows(const cmlb200_delta* a, const float* d_proj, int ld, float* d_decay, int ld_decay, const float* d_gate, int ld_gate,
+extern "C" int cmlb200_delta_rows(const cmlb200_delta* a, const float* d_proj, int ld, const float* d_decay, int ld_decay, const float* d_gate, int ld_gate,
                                   const int* d_row_pos, const int* d_row_slot, int first, int rows, const int* d_runs, int runs, float* d_work, void* d_out,
                                   int out_dtype, int out_ld, void* stream) {
     const int rc = delta_check(a, d_proj, ld, d_decay, ld_decay, d_gate, ld_gate, d_row_pos, d_row_slot, 1, d_out, out_dtype, out_ld, "cmlb200_delta_rows");
     if (rc) return rc;
+    CMLB_REQUIRE((long long)rows * ld < (1ll << 31), "cmlb200_delta_rows: %d rows of %d", rows, ld);
     CMLB_REQUIRE(d_runs && runs > 0 && runs <= 65535 && rows > 0 && first >= 0 && d_work && (((uintptr_t)d_runs | (uintptr_t)d_work) & 15) == 0, "cmlb200_delta_rows: bad argument");
     cudaStream_t st = as_stream(stream);
-    CMLB_CUDA(launch_chain(delta_prepare_kernel, dim3(rows, (a->kv_heads + a->heads + 7) / 8), dim3(256), 0, 1, st, *a, d_proj, ld, d_decay, ld_decay, d_row_pos, d_row_slot,
-                           first, d_work));
-    const bool vec = a->dim % 4 == 0 && a->vdim % 4 == 0 && ld_decay % 4 == 0 && ((uintptr_t)d_decay & 15) == 0;
-    const dim3 grid((a->vdim + SCAN_COLS - 1) / SCAN_COLS, a->heads, runs);
-#define DS_LAUNCH(RPL, N) CMLB_CUDA(launch_chain(delta_scan_kernel<RPL, N>, grid, dim3(SCAN_THREADS), 0, 1, st, *a, d_proj, ld, (const float*)d_decay, ld_decay, d_row_pos, \
-                                                 (const int4*)d_runs, first, d_work))
-#define DS_COPY(RPL) do { if (vec) DS_LAUNCH(RPL, 4); else DS_LAUNCH(RPL, 1); } while (0)
-    if (a->dim <= 32) DS_COPY(4);
-    else if (a->dim <= 64) DS_COPY(8);
-    else if (a->dim <= 128) DS_COPY(16);
-    else DS_COPY(32);
-#undef DS_COPY
+    const int tiles = scan_tiles(*a);
+    float* packets = d_work + (size_t)rows * value_ld(*a);
+    const dim3 grid(rows / CHUNK + runs, (a->heads + 3) / 4);
+#define DP_LAUNCH(T) CMLB_CUDA(launch_chain(delta_prepare_kernel<T>, grid, dim3(128), 0, 1, st, *a, d_proj, ld, d_decay, ld_decay, d_row_pos, (const int4*)d_runs, runs, first, \
+                                            d_work, packets))
+    if (a->taps == 4) DP_LAUNCH(4);
+    else DP_LAUNCH(0);
+#undef DP_LAUNCH
+    const dim3 grid_scan((a->vdim + SCAN_COLS - 1) / SCAN_COLS, a->heads, runs);
+    // few CTAs: each has to cover the latency of its packets alone; many: more of them fit an SM
+    const bool deep = (long long)grid_scan.x * grid_scan.y * grid_scan.z <= 2 * cmlb_num_sms();
+    static size_t attr[8][kMaxDevices] = {};
+#define DS_LAUNCH(N, STAGES, slot)                                                                                                  \
+    do {                                                                                                                            \
+        auto kern = delta_scan_kernel<N, STAGES>;                                                                                   \
+        const size_t smem = (size_t)STAGES * packet_floats(tiles) * sizeof(float);                                                  \
+        CMLB_CUDA(cmlb_ensure_smem(kern, smem, attr[slot]));                                                                        \
+        CMLB_CUDA(launch_chain(kern, grid_scan, dim3(SCAN_WARPS * 32), smem, 1, st, *a, d_proj, ld, d_row_pos, (const int4*)d_runs, first, d_work, (const float*)packets)); \
+    } while (0)
+#define DS_DEPTH(N, slot) do { if (deep) DS_LAUNCH(N, (N > 4 ? 4 : 6), slot); else DS_LAUNCH(N, 3, slot + 1); } while (0)
+    if (tiles == 4) DS_DEPTH(1, 0);
+    else if (tiles == 8) DS_DEPTH(2, 2);
+    else if (tiles == 16) DS_DEPTH(4, 4);
+    else DS_DEPTH(8, 6);
+#undef DS_DEPTH
 #undef DS_LAUNCH
     const dim3 grid_out(rows, (a->heads + 7) / 8);
-    if (out_dtype == CMLB200_DT_BF16)
-        CMLB_CUDA(launch_chain(delta_output_kernel<__nv_bfloat16>, grid_out, dim3(256), 0, 1, st, *a, (const float*)d_work, d_gate, ld_gate, first, (__nv_bfloat16*)d_out, out_ld));
-    else
-        CMLB_CUDA(launch_chain(delta_output_kernel<float>, grid_out, dim3(256), 0, 1, st, *a, (const float*)d_work, d_gate, ld_gate, first, (float*)d_out, out_ld));
+    const bool vec = a->vdim % 4 == 0 && ld_gate % 4 == 0 && out_ld % 4 == 0 && (((uintptr_t)d_gate | (uintptr_t)d_out) & 15) == 0;
+#define DU_LAUNCH(TO, W) CMLB_CUDA(launch_chain(delta_output_kernel<TO, W>, grid_out, dim3(256), 0, 1, st, *a, (const float*)d_work, d_gate, ld_gate, first, (TO*)d_out, out_ld))
+    if (out_dtype == CMLB200_DT_BF16) { if (vec) DU_LAUNCH(__nv_bfloat16, 4); else DU_LAUNCH(__nv_bfloat16, 1); }
+    else { if (vec) DU_LAUNCH(float, 4); else DU_LAUNCH(float, 1); }
+#undef DU_LAUNCH
     return CMLB200_OK;
 }

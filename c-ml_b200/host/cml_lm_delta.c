@@ -77,14 +77,16 @@ int cml_delta_load(Layered* m, const CMLSafetensors* st, const char* prefix, Lay
 }
 
 int cml_delta_activations(Layered* m, int rows) {
-    int dec = 0, gate = 0, low = 0, work = 0;
+    int dec = 0, gate = 0, low = 0;
+    long work = 0;
     for (int i = 0; i < m->num_layers; i++) {
         const Layer *l = &m->layers[i], *s = &m->layers[l->source];
         if (l->kind->form != MIXER_PARALLEL) continue;
         dec = lml_most(dec, l->delta.heads * l->delta.dim);
         gate = lml_most(gate, l->delta.heads * l->delta.vdim);
         low = lml_most(low, lml_most(s->a_rank, s->g_rank));
-        work = lml_most(work, cmlb200_delta_work_floats(&l->delta));
+        const long floats = cmlb200_delta_work_floats(&l->delta, rows, m->max_sequences);
+        if (floats > work) work = floats;
     }
     if (!dec) return 0;
     m->ld_dec = lml_round_up(dec, 16);
@@ -92,7 +94,7 @@ int cml_delta_activations(Layered* m, int rows) {
     m->ld_low = lml_round_up(low, 64);
     const size_t R = (size_t)rows;
     return lml_zeroed((void**)&m->dec, R * (size_t)m->ld_dec * 4) || lml_zeroed((void**)&m->gate, R * (size_t)m->ld_gate * 4) ||
-           lml_zeroed((void**)&m->delta_work, R * (size_t)work * 4) || (!m->f32 && lml_zeroed(&m->low, R * (size_t)m->ld_low * 2)) ? -1 : 0;
+           lml_zeroed((void**)&m->delta_work, (size_t)work * 4) || (!m->f32 && lml_zeroed(&m->low, R * (size_t)m->ld_low * 2)) ? -1 : 0;
 }
 
 int cml_delta_make_state(Layered* m, Layer* l, const LayerWeights* w, int slots) {

@@ -574,15 +574,17 @@ int cmlb200_stream_join(const cmlb200_streams* hc, float* d_x, const float* d_y,
 
 /* Gated delta rule over a step's rows. d_decay: [rows][heads * dim] inputs a of the decay, d_gate: [rows][heads * vdim] gate
  * logits, fp32 with their strides. out: fp32 or bf16.
- * _one: single tokens, at most one row per sequence, everything in one launch.
+ * _one: single tokens, at most one row per sequence, everything in one launch. Positions, slots and the rows' states must
+ * be older than the launch directly in front of it in the stream.
  * _rows: portions whose rows are first .. first + rows - 1 of the step, runs[i] = {first row, rows, slot, position} (device):
- * convolutions, norms and decays, the recurrence, output norm and gate. work: [rows][cmlb200_delta_work_floats] fp32, row 0 is the step's row `first`; d_decay is overwritten with the decays. All row arrays begin at the step's row 0. */
+ * what does not depend on the state, chunk by chunk; the recurrence; output norm and gate. work: cmlb200_delta_work_floats(a,
+ * rows, runs) floats. The row arrays begin at the step's row 0. */
 int cmlb200_delta_one(const cmlb200_delta* a, const float* d_proj, int ld, const float* d_decay, int ld_decay, const float* d_gate, int ld_gate,
                       const int* d_row_pos, const int* d_row_slot, int rows, void* d_out, int out_dtype, int out_ld, void* stream);
-int cmlb200_delta_rows(const cmlb200_delta* a, const float* d_proj, int ld, float* d_decay, int ld_decay, const float* d_gate, int ld_gate,
+int cmlb200_delta_rows(const cmlb200_delta* a, const float* d_proj, int ld, const float* d_decay, int ld_decay, const float* d_gate, int ld_gate,
                        const int* d_row_pos, const int* d_row_slot, int first, int rows, const int* d_runs, int runs, float* d_work, void* d_out,
                        int out_dtype, int out_ld, void* stream);
-int cmlb200_delta_work_floats(const cmlb200_delta* a);
+long cmlb200_delta_work_floats(const cmlb200_delta* a, int rows, int runs);
 /* bf16 rows of columns col .. col + n - 1 of fp32 rows; columns n .. ldo - 1 are left alone. */
 int cmlb200_pack_columns(const float* d_x, int ld, int col, int n, int rows, uint16_t* d_out_bf16, int ldo, void* stream);
 

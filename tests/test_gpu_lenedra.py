@@ -332,7 +332,7 @@ class DeltaLayer:
             out = torch.zeros((n, ow + 3), device=self.dev, dtype=torch.float32 if self.f32 else torch.bfloat16)
             t, P = pkg.DT_F32 if self.f32 else pkg.DT_BF16, lambda x: x.data_ptr()
             if n > one:
-                w = torch.full((n - one, L.cmlb200_delta_work_floats(a)), float("nan"), device=self.dev)
+                w = torch.full((L.cmlb200_delta_work_floats(a, n - one, len(runs)),), float("nan"), device=self.dev)
                 dr = up(runs, self.dev, np.int32)
                 pkg.check(L.cmlb200_delta_rows(a, P(d), ld, P(dec), ldd, P(gate), ldg, P(dp), P(ds), one, n - one, P(dr), len(runs), P(w), P(out), t, ow + 3, None))
             if one:
