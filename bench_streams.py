@@ -234,8 +234,8 @@ def products(pkg, torch, T, add):
         del ws
         torch.cuda.empty_cache()
     for rows in (1, 32, 2048):
-        x, o = torch.randn(rows, 10512, device=dev), torch.empty(rows, 128, device=dev, dtype=torch.bfloat16)
-        add("pack_columns", f"{rows}x128", T.us([lambda s: ck(lib.cmlb200_pack_columns(P(x), 10512, 9232, 128, rows, P(o), 128, s))], 10), rows * 128 * 6.0)
+        x, o = torch.randn(rows, 10512, device=dev), torch.empty(rows, 256, device=dev, dtype=torch.bfloat16)
+        add("pack_columns", f"{rows}x256", T.us([lambda s: ck(lib.cmlb200_pack_columns(P(x), 10512, 9232, 128, 128, 128, rows, P(o), 256, s))], 10), rows * 256 * 6.0)
 
 
 def run(pkg, synth, torch, peaks, sampler, kernels_only=False, models_only=False):

@@ -506,7 +506,7 @@ _sig("cmlb200_stream_join", ci, C.POINTER(Streams), vp, vp, ci, C.POINTER(Join),
 _sig("cmlb200_delta_one", ci, C.POINTER(Delta), vp, ci, vp, ci, vp, ci, vp, vp, ci, vp, ci, ci, vp)
 _sig("cmlb200_delta_rows", ci, C.POINTER(Delta), vp, ci, vp, ci, vp, ci, vp, vp, ci, ci, vp, ci, vp, vp, ci, ci, vp)
 _sig("cmlb200_delta_work_floats", C.c_long, C.POINTER(Delta), ci, ci)
-_sig("cmlb200_pack_columns", ci, vp, ci, ci, ci, ci, vp, ci, vp)
+_sig("cmlb200_pack_columns", ci, vp, ci, ci, ci, ci, ci, ci, vp, ci, vp)
 _sig("cmlb200_latent_append", ci, _LAT, vp, ci, vp, vp, ci, vp)
 for _n in ("cmlb200_latent_query", "cmlb200_latent_query_f32"):
     _sig(_n, ci, _LAT, vp, vp, ci, vp, vp, ci, vp, vp)

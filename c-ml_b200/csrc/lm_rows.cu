@@ -8,8 +8,8 @@
 
 namespace {
 
-// x[r][s] = scale * table[token[r]] for every stream s
-template <typename T>
+// x[r][s] = scale * table[token[r]] for every stream s. W: 4 or 1 columns at a time.
+template <typename T, int W>
 __global__ void __launch_bounds__(256)
 embed_streams_kernel(const T* __restrict__ table, const int* __restrict__ tokens, float scale, int streams, int width, int vocab, float* __restrict__ x) {
     dep_wait();
@@ -19,9 +19,20 @@ embed_streams_kernel(const T* __restrict__ table, const int* __restrict__ tokens
     if (t < 0 || t >= vocab) t = 0;
     const T* src = table + (size_t)t * width;
     float* dst = x + (size_t)r * streams * width;
-    for (int i = blockIdx.y * 256 + threadIdx.x; i < width; i += gridDim.y * 256) {
-        const float v = widen(src[i]) * scale;
-        for (int s = 0; s < streams; s++) dst[(size_t)s * width + i] = v;
+    for (int i = (blockIdx.y * 256 + threadIdx.x) * W; i < width; i += gridDim.y * 256 * W) {
+        if constexpr (W == 4) {
+            float4 v;
+            if constexpr (sizeof(T) == 4) v = *reinterpret_cast<const float4*>(src + i);
+            else {
+                const uint2 b = *reinterpret_cast<const uint2*>(src + i);
+                v = make_float4(__uint_as_float(b.x << 16), __uint_as_float(b.x & 0xffff0000u), __uint_as_float(b.y << 16), __uint_as_float(b.y & 0xffff0000u));
+            }
+            v.x *= scale; v.y *= scale; v.z *= scale; v.w *= scale;
+            for (int s = 0; s < streams; s++) *reinterpret_cast<float4*>(dst + (size_t)s * width + i) = v;
+        } else {
+            const float v = widen(src[i]) * scale;
+            for (int s = 0; s < streams; s++) dst[(size_t)s * width + i] = v;
+        }
     }
 }
 
@@ -140,11 +151,11 @@ stream_join_kernel(const cmlb200_streams hc, float* __restrict__ x, const float*
 }
 
 __global__ void __launch_bounds__(256)
-pack_columns_kernel(const float* __restrict__ x, int ld, int col, int n, __nv_bfloat16* __restrict__ out, int ldo) {
+pack_columns_kernel(const float* __restrict__ x, int ld, int col, int n, int more, int at, __nv_bfloat16* __restrict__ out, int ldo) {
     dep_wait();
     dep_trigger();
     const float* src = x + (size_t)blockIdx.x * ld + col;
-    for (int i = threadIdx.x; i < n; i += 256) out[(size_t)blockIdx.x * ldo + i] = __float2bfloat16_rn(src[i]);
+    for (int i = threadIdx.x; i < n + more; i += 256) out[(size_t)blockIdx.x * ldo + (i < n ? i : at + i - n)] = __float2bfloat16_rn(src[i]);
 }
 
 // x[r] = table[token[r]] (+ the position vector: entry 2i = sin(p f_i), entry 2i + 1 = cos(p f_i),
@@ -331,10 +342,18 @@ qk_norm_append_kernel(float* __restrict__ qkv, int ld, const int* __restrict__ r
     float2 ss = make_float2(0.f, 0.f);
     if (a.head_norm) {
         const int lane = threadIdx.x & 31;
+#pragma unroll 4
         for (int j = threadIdx.x >> 5; j < a.heads + a.kv_heads; j += 8) {
             const float* v = row + (size_t)j * a.dim;
             float s = 0.f;
-            for (int d = lane; d < a.dim; d += 32) s = fmaf(v[d], v[d], s);
+            if (VEC) {
+                for (int d = lane * 4; d < a.dim; d += 128) {
+                    const float4 x = *reinterpret_cast<const float4*>(v + d);
+                    s = fmaf(x.x, x.x, fmaf(x.y, x.y, fmaf(x.z, x.z, fmaf(x.w, x.w, s))));
+                }
+            } else {
+                for (int d = lane; d < a.dim; d += 32) s = fmaf(v[d], v[d], s);
+            }
             s = lane_sum(s);
             if (lane == 0) inv[j] = (j < a.heads ? a.q_norm : a.k_norm) ? 1.0f / sqrtf(s / (float)a.dim + a.eps) : 1.0f;
         }
@@ -476,10 +495,11 @@ extern "C" int cmlb200_embed_streams(const void* d_table, int dtype, const int* 
                                      float* d_x, void* stream) {
     CMLB_REQUIRE(d_table && d_tokens && d_x && streams > 0 && rows > 0 && width > 0 && vocab > 0, "cmlb200_embed_streams: bad argument");
     CMLB_REQUIRE(dtype == CMLB200_DT_F32 || dtype == CMLB200_DT_BF16, "cmlb200_embed_streams: dtype %d", dtype);
-    const dim3 grid(rows, rows < 64 ? (width + 511) / 512 : 1);
-#define ES_LAUNCH(T) CMLB_CUDA(launch_chain(embed_streams_kernel<T>, grid, dim3(256), 0, 1, as_stream(stream), (const T*)d_table, d_tokens, scale, streams, width, vocab, d_x))
-    if (dtype == CMLB200_DT_BF16) ES_LAUNCH(__nv_bfloat16);
-    else ES_LAUNCH(float);
+    const bool vec = width % 4 == 0 && (((uintptr_t)d_table | (uintptr_t)d_x) & 15) == 0;
+    const dim3 grid(rows, rows < 64 ? (width + 1023) / 1024 : 1);
+#define ES_LAUNCH(T, W) CMLB_CUDA(launch_chain(embed_streams_kernel<T, W>, grid, dim3(256), 0, 1, as_stream(stream), (const T*)d_table, d_tokens, scale, streams, width, vocab, d_x))
+    if (dtype == CMLB200_DT_BF16) { if (vec) ES_LAUNCH(__nv_bfloat16, 4); else ES_LAUNCH(__nv_bfloat16, 1); }
+    else { if (vec) ES_LAUNCH(float, 4); else ES_LAUNCH(float, 1); }
 #undef ES_LAUNCH
     return CMLB200_OK;
 }
@@ -517,9 +537,10 @@ extern "C" int cmlb200_stream_join(const cmlb200_streams* hc, float* d_x, const 
     return CMLB200_OK;
 }
 
-extern "C" int cmlb200_pack_columns(const float* d_x, int ld, int col, int n, int rows, uint16_t* d_out_bf16, int ldo, void* stream) {
-    CMLB_REQUIRE(d_x && d_out_bf16 && col >= 0 && n > 0 && rows > 0 && ld >= col + n && ldo >= n, "cmlb200_pack_columns: bad argument");
-    CMLB_CUDA(launch_chain(pack_columns_kernel, dim3(rows), dim3(256), 0, 1, as_stream(stream), d_x, ld, col, n, (__nv_bfloat16*)d_out_bf16, ldo));
+extern "C" int cmlb200_pack_columns(const float* d_x, int ld, int col, int n, int more, int at, int rows, uint16_t* d_out_bf16, int ldo, void* stream) {
+    CMLB_REQUIRE(d_x && d_out_bf16 && col >= 0 && n > 0 && more >= 0 && rows > 0 && ld >= col + n + more && ldo >= n && (!more || (at >= n && ldo >= at + more)),
+                 "cmlb200_pack_columns: bad argument");
+    CMLB_CUDA(launch_chain(pack_columns_kernel, dim3(rows), dim3(256), 0, 1, as_stream(stream), d_x, ld, col, n, more, at, (__nv_bfloat16*)d_out_bf16, ldo));
     return CMLB200_OK;
 }
 

@@ -84,14 +84,14 @@ int cml_delta_activations(Layered* m, int rows) {
         if (l->kind->form != MIXER_PARALLEL) continue;
         dec = lml_most(dec, l->delta.heads * l->delta.dim);
         gate = lml_most(gate, l->delta.heads * l->delta.vdim);
-        low = lml_most(low, lml_most(s->a_rank, s->g_rank));
+        low = lml_most(low, lml_round_up(s->a_rank, 64) + lml_round_up(s->g_rank, 64));
         const long floats = cmlb200_delta_work_floats(&l->delta, rows, m->max_sequences);
         if (floats > work) work = floats;
     }
     if (!dec) return 0;
     m->ld_dec = lml_round_up(dec, 16);
     m->ld_gate = lml_round_up(gate, 16);
-    m->ld_low = lml_round_up(low, 64);
+    m->ld_low = low;
     const size_t R = (size_t)rows;
     return lml_zeroed((void**)&m->dec, R * (size_t)m->ld_dec * 4) || lml_zeroed((void**)&m->gate, R * (size_t)m->ld_gate * 4) ||
            lml_zeroed((void**)&m->delta_work, (size_t)work * 4) || (!m->f32 && lml_zeroed(&m->low, R * (size_t)m->ld_low * 2)) ? -1 : 0;
@@ -108,11 +108,15 @@ int cml_delta_make_state(Layered* m, Layer* l, const LayerWeights* w, int slots)
            lml_zeroed((void**)&a->ring, (size_t)slots * (size_t)a->taps * (size_t)channels_of(a) * 4) ? -1 : 0;
 }
 
-/* y = W2 (rank columns of the projection from `col` on) */
-static int second_factor(const Layered* m, const cmlb200_dense* w, int col, int rank, int rows, float* y, int ldy, void* st) {
-    if (m->f32) return lml_product(m, w, m->qkvg + col, m->ld_qkvg, rows, y, ldy, st);
-    DEV(cmlb200_pack_columns(m->qkvg, m->ld_qkvg, col, rank, rows, (uint16_t*)m->low, m->ld_low, st));
-    return lml_product(m, w, m->low, m->ld_low, rows, y, ldy, st);
+/* Inputs of the decays and gate logits: second factors on the columns of the first ones, which lie side by side. */
+static int second_factors(const Layered* m, const Layer* s, const LayerWeights* w, int col, int rows, void* st) {
+    const int g = lml_round_up(s->a_rank, 64);
+    if (m->f32)
+        return lml_product(m, &w->wa, m->qkvg + col, m->ld_qkvg, rows, m->dec, m->ld_dec, st) ||
+               lml_product(m, &w->wg, m->qkvg + col + s->a_rank, m->ld_qkvg, rows, m->gate, m->ld_gate, st) ? -1 : 0;
+    uint16_t* low = (uint16_t*)m->low;
+    DEV(cmlb200_pack_columns(m->qkvg, m->ld_qkvg, col, s->a_rank, s->g_rank, g, rows, low, m->ld_low, st));
+    return lml_product(m, &w->wa, low, m->ld_low, rows, m->dec, m->ld_dec, st) || lml_product(m, &w->wg, low + g, m->ld_low, rows, m->gate, m->ld_gate, st) ? -1 : 0;
 }
 
 int cml_delta_run(const Layered* m, const Layer* l, const LayerWeights* w, const CMLLMBatch* b, int col, void* st) {
@@ -120,9 +124,7 @@ int cml_delta_run(const Layered* m, const Layer* l, const LayerWeights* w, const
     const Layer* s = &m->layers[l->source];
     const int low = a->col + channels_of(a) + a->heads, type = m->f32 ? CMLB200_DT_F32 : CMLB200_DT_BF16;
     uint8_t* out = (uint8_t*)m->att + (size_t)col * (m->f32 ? 4 : 2);
-    if (second_factor(m, &w->wa, low, s->a_rank, b->rows, m->dec, m->ld_dec, st) ||
-        second_factor(m, &w->wg, low + s->a_rank, s->g_rank, b->rows, m->gate, m->ld_gate, st))
-        return -1;
+    if (second_factors(m, s, w, low, b->rows, st)) return -1;
     if (b->rows > b->one_rows)
         DEV(cmlb200_delta_rows(a, m->qkvg, m->ld_qkvg, m->dec, m->ld_dec, m->gate, m->ld_gate, b->d_pos, b->d_slot, b->one_rows, b->rows - b->one_rows, b->d_runs,
                                b->num_runs, m->delta_work, out, type, m->ld_att, st));

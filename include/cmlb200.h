@@ -585,8 +585,9 @@ int cmlb200_delta_rows(const cmlb200_delta* a, const float* d_proj, int ld, cons
                        const int* d_row_pos, const int* d_row_slot, int first, int rows, const int* d_runs, int runs, float* d_work, void* d_out,
                        int out_dtype, int out_ld, void* stream);
 long cmlb200_delta_work_floats(const cmlb200_delta* a, int rows, int runs);
-/* bf16 rows of columns col .. col + n - 1 of fp32 rows; columns n .. ldo - 1 are left alone. */
-int cmlb200_pack_columns(const float* d_x, int ld, int col, int n, int rows, uint16_t* d_out_bf16, int ldo, void* stream);
+/* bf16 rows of columns col .. col + n - 1 of fp32 rows, and of the `more` columns behind those from output column `at` on; other
+ * output columns are left alone. */
+int cmlb200_pack_columns(const float* d_x, int ld, int col, int n, int more, int at, int rows, uint16_t* d_out_bf16, int ldo, void* stream);
 
 /* Latent attention. _append: rotates the query columns in place and fills the cache (any rows). _query: the same for
  * rows whose attention runs over the latents themselves, into fp16 rows [heads][ld] = [Wuk^T q | rotated q] times

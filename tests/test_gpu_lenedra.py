@@ -481,9 +481,10 @@ def test_packed_columns(pkg, torch_dev):
     import torch
     x = RNG(1).standard_normal((9, 301)).astype(np.float32)
     out, d = torch.full((9, 128), 7.0, device=torch_dev).bfloat16(), up(x, torch_dev)
-    pkg.check(pkg.lib.cmlb200_pack_columns(d.data_ptr(), 301, 17, 99, 9, out.data_ptr(), 128, None))
+    pkg.check(pkg.lib.cmlb200_pack_columns(d.data_ptr(), 301, 17, 49, 13, 64, 9, out.data_ptr(), 128, None))
     sync()
-    assert torch.equal(out[:, :99], d[:, 17:116].bfloat16()) and (out[:, 99:] == 7).all()
+    assert torch.equal(out[:, :49], d[:, 17:66].bfloat16()) and torch.equal(out[:, 64:77], d[:, 66:79].bfloat16()) and (out[:, 49:64] == 7).all() and (out[:, 77:] == 7).all()
+    assert pkg.lib.cmlb200_pack_columns(d.data_ptr(), 301, 17, 49, 13, 40, 9, out.data_ptr(), 128, None) != 0 and pkg.lib.cmlb200_pack_columns(d.data_ptr(), 60, 17, 49, 0, 0, 9, out.data_ptr(), 128, None) != 0
 
 
 # ---- routing -------------------------------------------------------------------------------------------------
