@@ -339,35 +339,66 @@ qk_norm_append_kernel(float* __restrict__ qkv, int ld, const int* __restrict__ r
     float* row = qkv + (size_t)r * ld;
     const int p = row_pos[r];
     const size_t slot = (size_t)a.block_table[(size_t)row_slot[r] * a.table_ld + p / a.block_size] * a.block_size + p % a.block_size;
+    const float temp = a.temp_every > 0.f ? 1.0f + a.temp_coef * logf(floorf((float)(p + 1) / a.temp_every) + 1.0f) : 1.0f;
+    KV* kd = kpool + slot * a.kv_heads * a.dim_ld;
+    KV* vd = vpool + slot * a.kv_heads * a.vdim_ld;
     float2 ss = make_float2(0.f, 0.f);
+    if (VEC && a.head_norm && a.dim <= 256) {          // a warp per head, which it holds in registers
+        const int lane = threadIdx.x & 31;
+        const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f), ones = make_float4(1.f, 1.f, 1.f, 1.f);
+#pragma unroll 4
+        for (int j = threadIdx.x >> 5; j < a.heads + a.kv_heads; j += 8) {
+            const bool query = j < a.heads;
+            const float* norm = query ? a.q_norm : a.k_norm;
+            float* v = row + (size_t)j * a.dim;
+            float4 x[2];
+            float s = 0.f;
+#pragma unroll
+            for (int i = 0; i < 2; i++) {
+                const int d = lane * 4 + 128 * i;
+                x[i] = d < a.dim ? *reinterpret_cast<const float4*>(v + d) : zero;
+                s = fmaf(x[i].x, x[i].x, fmaf(x[i].y, x[i].y, fmaf(x[i].z, x[i].z, fmaf(x[i].w, x[i].w, s))));
+            }
+            s = lane_sum(s);
+            const float f = (norm ? 1.0f / sqrtf(s / (float)a.dim + a.eps) : 1.0f) * (query ? temp : 1.0f);
+#pragma unroll
+            for (int i = 0; i < 2; i++) {
+                const int d = lane * 4 + 128 * i;
+                const float4 w = norm && d < a.dim ? *reinterpret_cast<const float4*>(norm + d) : ones;
+                const float4 y = make_float4(x[i].x * f * w.x, x[i].y * f * w.y, x[i].z * f * w.z, x[i].w * f * w.w);
+                if (query) {
+                    if (d < a.dim) *reinterpret_cast<float4*>(v + d) = y;
+                } else if (d < a.dim_ld) {             // zeros behind dim
+                    store4(kd + (size_t)(j - a.heads) * a.dim_ld + d, y);
+                    if (a.keys_as_values) store4(vd + (size_t)(j - a.heads) * a.vdim_ld + d, x[i]);
+                }
+            }
+        }
+        if (!a.keys_as_values)
+            for (int i = threadIdx.x * 4; i < a.kv_heads * a.vdim_ld; i += 1024) {
+                const int g = i / a.vdim_ld, d = i - g * a.vdim_ld;
+                store4(vd + i, d < a.vdim ? *reinterpret_cast<const float4*>(row + vcol + g * a.vdim + d) : zero);
+            }
+        return;
+    }
     if (a.head_norm) {
         const int lane = threadIdx.x & 31;
-#pragma unroll 4
         for (int j = threadIdx.x >> 5; j < a.heads + a.kv_heads; j += 8) {
             const float* v = row + (size_t)j * a.dim;
             float s = 0.f;
-            if (VEC) {
-                for (int d = lane * 4; d < a.dim; d += 128) {
-                    const float4 x = *reinterpret_cast<const float4*>(v + d);
-                    s = fmaf(x.x, x.x, fmaf(x.y, x.y, fmaf(x.z, x.z, fmaf(x.w, x.w, s))));
-                }
-            } else {
-                for (int d = lane; d < a.dim; d += 32) s = fmaf(v[d], v[d], s);
-            }
+            for (int d = lane; d < a.dim; d += 32) s = fmaf(v[d], v[d], s);
             s = lane_sum(s);
             if (lane == 0) inv[j] = (j < a.heads ? a.q_norm : a.k_norm) ? 1.0f / sqrtf(s / (float)a.dim + a.eps) : 1.0f;
         }
         __syncthreads();
-    } else {
+    } else if (a.q_norm || a.k_norm) {
         ss = block_sum2(square_share(row, qw), square_share(row + qw, kw), red);
     }
-    const float temp = a.temp_every > 0.f ? 1.0f + a.temp_coef * logf(floorf((float)(p + 1) / a.temp_every) + 1.0f) : 1.0f;
+    const bool same_q = !a.q_norm && a.temp_every <= 0.f;                // q stays as it is
     const float iq = a.q_norm ? 1.0f / sqrtf(ss.x / (float)qw + a.eps) : 1.0f, ik = a.k_norm ? 1.0f / sqrtf(ss.y / (float)kw + a.eps) : 1.0f;
-    KV* kd = kpool + slot * a.kv_heads * a.dim_ld;
-    KV* vd = vpool + slot * a.kv_heads * a.vdim_ld;
     if (VEC) {
 #pragma unroll 4
-        for (int i = threadIdx.x * 4; i < qw; i += 1024) {
+        for (int i = same_q ? qw : threadIdx.x * 4; i < qw; i += 1024) {
             float4 v = *reinterpret_cast<const float4*>(row + i);
             const int j = a.head_norm ? i / a.dim : 0;
             const float f = a.head_norm ? inv[j] : iq;
@@ -394,7 +425,7 @@ qk_norm_append_kernel(float* __restrict__ qkv, int ld, const int* __restrict__ r
         }
         return;
     }
-    for (int i = threadIdx.x; i < qw; i += 256) {
+    for (int i = same_q ? qw : threadIdx.x; i < qw; i += 256) {
         const int j = a.head_norm ? i / a.dim : 0;
         row[i] = row[i] * (a.head_norm ? inv[j] : iq) * (a.q_norm ? a.q_norm[i - j * a.dim] : 1.0f) * temp;
     }
