@@ -600,7 +600,7 @@ int lml_zeroed(void** dst, size_t bytes) {
 /* Operand buffers have strides that are multiples of 64 and start out zero: the decode product reads up
  * to the padded width, where its weights are zero. */
 static int make_activations(Layered* m, int rows) {
-    int q = 0, att = 0, ff = 0, z = 0, latent_q = 0, latent_o = 0, experts = 0, outputs = 0, top = 0, shared = 0;
+    int q = 0, att = 0, ff = 0, z = 0, latent_q = 0, latent_o = 0, experts = 0, identity = 0, outputs = 0, top = 0, shared = 0;
     long positions = 0, tiles = 0;
     for (int i = 0; i < m->num_layers; i++) {
         const Layer* l = &m->layers[i];
@@ -619,6 +619,7 @@ static int make_activations(Layered* m, int rows) {
             if (p > positions) positions = p;
             if (p / EXPERT_ROWS + l->experts + 1 > tiles) tiles = p / EXPERT_ROWS + l->experts + 1;
             experts = lml_most(experts, l->experts);
+            identity = lml_most(identity, l->identity);
             outputs = lml_most(outputs, l->experts + l->identity);
             shared = lml_most(shared, l->shared_ff);
             top = lml_most(top, l->top);
@@ -653,7 +654,7 @@ static int make_activations(Layered* m, int rows) {
         if (lml_zeroed((void**)&m->router, R * (size_t)m->ld_router * 4) || (!m->f32 && lml_zeroed(&m->xp, P * (size_t)m->ld_h * es)) || lml_zeroed((void**)&p->ids, pairs) ||
             lml_zeroed((void**)&p->weight, pairs) || lml_zeroed((void**)&p->pos, pairs) || lml_zeroed((void**)&p->src, pos) || lml_zeroed((void**)&p->expert, pos) ||
             lml_zeroed((void**)&p->start, per) || lml_zeroed((void**)&p->count, per) || lml_zeroed((void**)&p->active, per) || lml_zeroed((void**)&p->num_active, 4) ||
-            lml_zeroed((void**)&p->tiles, (size_t)tiles * 16) || lml_zeroed((void**)&p->num_tiles, 4) || (outputs > experts && lml_zeroed((void**)&p->self, R * 4)) ||
+            lml_zeroed((void**)&p->tiles, (size_t)tiles * 16) || lml_zeroed((void**)&p->num_tiles, 4) || (identity && lml_zeroed((void**)&p->self, R * 4)) ||
             (shared && lml_zeroed((void**)&m->y_shared, R * (size_t)m->ld_y * 4)))
             return -1;
     }

@@ -8,7 +8,7 @@
 
 #define SKINNY_ROWS 32
 #define EXPERT_ROWS 128            /* row tile of the experts' tensor-core product */
-#define MAX_PARTS 9                /* tensors stacked into one matrix at most */
+#define MAX_PARTS 12               /* tensors stacked into one matrix at most */
 #define DEV(call) do { if (CML_DEV_FAIL((call), __func__)) return -1; } while (0)
 
 /* grouped heads; latent attention; chunked grouped heads beside a gated delta rule, their outputs scaled and added */

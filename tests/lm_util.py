@@ -42,8 +42,8 @@ def variants(synth):
         "streams_odd": synth.streams_config(97, 75, 1, [P((3, 1, 13, 7, 23), (3, 1, 11, 9, 2), (5, 3), 51, (-0.7, 0.4)), K(3, 3, 7, 1, 9, R(3, 4, 3, 7, 4, 17, 33, 2.5)),
                                                         P((5, 5, 9, 21, 1), (6, 3, 5, 3, 1), (1, 2), None), K(9, 3, 13, 50, 0, 33)], eps=2e-2, scale=0.7, cap=3.0),
         # wide heads, many heads, many streams, a window and a chunk longer than the prompts
-        "streams_wide": synth.streams_config(130, 192, 6, [K(12, 4, 136, 400, 16, 96), P((20, 2, 72, 136, 500), (9, 3, 136, 200, 4), (24, 130), R(40, 8, 6, 12, 5, 48, 320, 1.0))],
-                                             cap=12.0),
+        "streams_wide": synth.streams_config(130, 192, 6, [K(12, 4, 136, 400, 16, 96), P((20, 2, 72, 136, 500), (9, 3, 136, 200, 4), (24, 130), R(40, 8, 6, 12, 5, 48, 320, 1.0)),
+                                                            K(3, 3, 40, 90, 2, R(5, 3, 3, 2, 1, 24, 33)), K(2, 1, 16, 25, 7, R(60, 0, 4, 6, 3, 17, 40))], cap=12.0),
         # sizes with tiles of their own; chunks and windows that end where blocks and tiles do
         "streams_full": synth.streams_config(64, 128, 4, [P((4, 2, 64, 64, 64), (2, 1, 128, 128, 4), (16, 16), R(9, 3, 4, 3, 2, 24, 24)), K(2, 1, 128, 64, 16, 96),
                                                           P((4, 4, 128, 128, 16), (4, 4, 64, 64, 4), (64, 64), 64)]),
