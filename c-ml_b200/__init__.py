@@ -430,7 +430,7 @@ REFERENCE_QUIRKS, KV_FP32, ALL_LOGITS_FP32 = 1, 2, 4
 
 # ---- layered models (include/cml_lm.h and the kernels behind it) ---------------------------------
 DT_F32, DT_BF16, DT_F16 = 0, 1, 2
-ACT_SILU, ACT_GELU_TANH, ACT_CLAMPED = 0, 1, 2
+ACT_SILU, ACT_GELU_TANH, ACT_CLAMPED, ACT_GELU_ERF = 0, 1, 2, 3
 DTYPE_FLOAT32, DTYPE_BFLOAT16 = 0, 6
 
 
@@ -445,21 +445,22 @@ class Attn(C.Structure):
                 ("window", ci), ("slopes", vp), ("sink", ci), ("q_norm", vp), ("k_norm", vp), ("eps", C.c_float), ("temp_coef", C.c_float),
                 ("temp_every", C.c_float), ("gate_col", ci), ("cache_dtype", ci), ("k_pool", vp), ("v_pool", vp), ("block_size", ci),
                 ("block_table", vp), ("table_ld", ci), ("gate_wide", ci), ("keep", ci), ("chunk", ci), ("sinks", vp), ("head_norm", ci), ("keys_as_values", ci),
-                ("out_scale", C.c_float)]
+                ("out_scale", C.c_float), ("freq", vp), ("rot_dims", ci), ("taps", ci), ("conv", vp), ("ring", vp), ("cap", C.c_float), ("talk", vp),
+                ("scores", vp), ("scores_ld", ci)]
 
 
 class Latent(C.Structure):
     """cmlb200_latent."""
     _fields_ = [("heads", ci), ("dim", ci), ("rot_dim", ci), ("vdim", ci), ("rank", ci), ("ld", ci), ("ld_rank", ci), ("scale", C.c_float), ("window", ci),
                 ("c_norm", vp), ("eps", C.c_float), ("freq", vp), ("rot_mul", C.c_float), ("kv_col", ci), ("gate_col", ci), ("cache_dtype", ci), ("pool", vp),
-                ("block_size", ci), ("block_table", vp), ("table_ld", ci), ("pool_blocks", ci)]
+                ("block_size", ci), ("block_table", vp), ("table_ld", ci), ("pool_blocks", ci), ("gate_heads", ci), ("sinks", vp)]
 
 
 class Moe(C.Structure):
     """cmlb200_moe."""
     _fields_ = [("experts", ci), ("top", ci)] + [(n, vp) for n in ("ids", "weight", "pos", "src", "expert", "start", "count", "active", "num_active", "tiles",
                                                                      "num_tiles")] + \
-               [("identity", ci), ("groups", ci), ("keep", ci), ("correction", vp), ("normalize", ci), ("scale", C.c_float), ("self", vp)]
+               [("sigmoid", ci), ("group_best", ci), ("identity", ci), ("groups", ci), ("keep", ci), ("correction", vp), ("normalize", ci), ("scale", C.c_float), ("self", vp)]
 
 
 class Streams(C.Structure):
@@ -476,6 +477,17 @@ class Delta(C.Structure):
     """cmlb200_delta."""
     _fields_ = [("heads", ci), ("kv_heads", ci), ("dim", ci), ("vdim", ci), ("taps", ci), ("vdim_ld", ci), ("col", ci), ("conv", vp), ("rate", vp),
                 ("dt_bias", vp), ("norm", vp), ("eps", C.c_float), ("out_scale", C.c_float), ("state", vp), ("ring", vp)]
+
+
+class Gru(C.Structure):
+    """cmlb200_gru."""
+    _fields_ = [("width", ci), ("col", ci), ("state", vp)]
+
+
+class GatedJoin(C.Structure):
+    """cmlb200_gated_join."""
+    _fields_ = [("a", vp), ("b", vp), ("ldm", ci), ("a_norm", vp), ("b_norm", vp), ("f", vp), ("ldf", ci), ("parts", C.POINTER(Moe)), ("ga", vp), ("gf", vp), ("ldg", ci),
+                ("table", vp), ("table_dtype", ci), ("vocab", ci), ("tokens", vp)]
 
 
 class LMOptions(C.Structure):
@@ -506,6 +518,18 @@ _sig("cmlb200_stream_join", ci, C.POINTER(Streams), vp, vp, ci, C.POINTER(Join),
 _sig("cmlb200_delta_one", ci, C.POINTER(Delta), vp, ci, vp, ci, vp, ci, vp, vp, ci, vp, ci, ci, vp)
 _sig("cmlb200_delta_rows", ci, C.POINTER(Delta), vp, ci, vp, ci, vp, ci, vp, vp, ci, ci, vp, ci, vp, vp, ci, ci, vp)
 _sig("cmlb200_delta_work_floats", C.c_long, C.POINTER(Delta), ci, ci)
+_sig("cmlb200_gru_one", ci, C.POINTER(Gru), vp, ci, vp, vp, ci, vp, ci, ci, vp)
+_sig("cmlb200_gru_rows", ci, C.POINTER(Gru), vp, ci, vp, ci, vp, ci, ci, vp)
+_sig("cmlb200_rotate_append", ci, C.POINTER(Attn), vp, ci, vp, vp, ci, ci, ci, vp, vp)
+_sig("cmlb200_ring_rows", ci, C.POINTER(Attn), vp, ci, vp, ci, vp)
+_sig("cmlb200_talk_scores_tiles", ci, C.POINTER(Attn), vp, vp, ci, ci, vp, ci, vp)
+_sig("cmlb200_talk_scores_rows", ci, C.POINTER(Attn), vp, vp, vp, ci, ci, vp, ci, vp)
+_sig("cmlb200_talk_scores_heads", ci)
+_sig("cmlb200_gated_join_rows", ci, C.POINTER(GatedJoin), vp, vp, _cf, ci, ci, vp, ci, ci, vp)
+_sig("cmlb200_norm_columns", ci, vp, ci, ci, ci, vp, _cf, ci, vp, ci, ci, vp)
+_sig("cmlb200_moe_gemv_act", ci, _MOE, _DENSE, vp, ci, ci, ci, ci, ci, vp, ci, vp)
+_sig("cmlb200_moe_gemm_act", ci, _MOE, _DENSE, vp, ci, ci, ci, ci, vp, ci, vp)
+_sig("cmlb200_act_rows_f32", ci, vp, ci, ci, ci, ci, vp, ci, vp)
 _sig("cmlb200_pack_columns", ci, vp, ci, ci, ci, ci, ci, ci, vp, ci, vp)
 _sig("cmlb200_latent_append", ci, _LAT, vp, ci, vp, vp, ci, vp)
 for _n in ("cmlb200_latent_query", "cmlb200_latent_query_f32"):

@@ -83,9 +83,9 @@ def _version_script() -> Path:
 
 # Sources of the programs besides their own; None: everything the library holds.
 PROGRAMS = {
-    "trace_run": ["host/cml_json.c", "host/cml_safetensors.c", "host/cml_lm.c", "host/cml_lm_layered.c", "host/cml_lm_delta.c", "host/cml_paged.c", "host/cml_serving.c",
+    "trace_run": ["host/cml_json.c", "host/cml_safetensors.c", "host/cml_lm.c", "host/cml_lm_layered.c", "host/cml_lm_delta.c", "host/cml_lm_gru.c", "host/cml_lm_talk.c", "host/cml_paged.c", "host/cml_serving.c",
                   "host/cml_sampling.c", "host/cml_tensor.c", "host/cml_tokenizer.c", "csrc/shim.cu", "csrc/argmax.cu",
-                  "csrc/lm_rows.cu", "csrc/attention_rows.cu", "csrc/latent_rows.cu", "csrc/attention_latent.cu", "csrc/attention_latent_tc.cu", "csrc/moe_rows.cu", "csrc/delta_rule.cu", "csrc/gemv_bf16.cu", "csrc/gemm_bf16.cu", "csrc/llm_ops_f32.cu", "csrc/paged_attention.cu"],
+                  "csrc/lm_rows.cu", "csrc/attention_rows.cu", "csrc/latent_rows.cu", "csrc/attention_latent.cu", "csrc/attention_latent_tc.cu", "csrc/moe_rows.cu", "csrc/delta_rule.cu", "csrc/gru_rows.cu", "csrc/rotate_rows.cu", "csrc/talk_scores.cu", "csrc/gemv_bf16.cu", "csrc/gemm_bf16.cu", "csrc/llm_ops_f32.cu", "csrc/paged_attention.cu"],
     "cml_generate": None,
 }
 LINK_LIBS = ["-lcudart_static", "-ldl", "-lpthread", "-lrt", "-lm"]

@@ -205,7 +205,8 @@ attention_latent_kernel(const cmlb200_latent a, const __half* __restrict__ q, co
     if (sk == 0) {
         c_m[sr] = m;
         c_l[sr] = l;
-        corr[sr] = l > 0.f ? 1.0f / l : 0.f;
+        const float all = l > 0.f && a.sinks ? l + exp2f(a.sinks[(m0 + sr) % a.heads] * kLog2e - m) : l;      // a sink carries no value
+        corr[sr] = all > 0.f ? 1.0f / all : 0.f;
     }
     const size_t out0 = (size_t)tl.x * a.heads + m0;
     if (splits == 1) {
@@ -273,6 +274,7 @@ attention_latent_kernel(const cmlb200_latent a, const __half* __restrict__ q, co
             sum = fmaf(ls[s], c, sum);
             x.x = fmaf(xs[s].x, c, x.x); x.y = fmaf(xs[s].y, c, x.y); x.z = fmaf(xs[s].z, c, x.z); x.w = fmaf(xs[s].w, c, x.w);
         }
+        if (a.sinks) sum += exp2f(a.sinks[(m0 + r) % a.heads] * kLog2e - mx);
         // columns rank .. ld_rank meet zero weights
         const float inv = 1.0f / sum;
         const __nv_bfloat162 lo = __floats2bfloat162_rn(x.x * inv, d + 1 < a.rank ? x.y * inv : 0.f);

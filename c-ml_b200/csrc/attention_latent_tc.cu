@@ -310,7 +310,9 @@ attention_latent_tc_kernel(const __grid_constant__ CUtensorMap qmap, const __gri
                 }
             }
         }
-        const float inv = l > 0.f ? 1.0f / l : 0.f;
+        // a sink carries no value; with several splits it joins below
+        const float all = l > 0.f && a.sinks && splits == 1 ? l + exp2f(a.sinks[(m0 + r) % a.heads] * kLog2e - m) : l;
+        const float inv = all > 0.f ? 1.0f / all : 0.f;
         for (int c0 = 0; c0 < cols && n > 0; c0 += 32) {
             uint32_t o[32];
             tmem_ld32(lanes + c0, o);
@@ -363,6 +365,7 @@ attention_latent_tc_kernel(const __grid_constant__ CUtensorMap qmap, const __gri
                 sum = fmaf(c_l[s * MR + r], f, sum);
                 x.x = fmaf(xs[s].x, f, x.x); x.y = fmaf(xs[s].y, f, x.y); x.z = fmaf(xs[s].z, f, x.z); x.w = fmaf(xs[s].w, f, x.w);
             }
+            if (a.sinks && sum > 0.f) sum += exp2f(a.sinks[(m0 + r) % a.heads] * kLog2e - mx);
             const float inv = sum > 0.f ? 1.0f / sum : 0.f;
             const int col = v0 * 64 + c;
             const __nv_bfloat162 lo = __floats2bfloat162_rn(col < a.rank ? x.x * inv : 0.f, col + 1 < a.rank ? x.y * inv : 0.f);

@@ -1,8 +1,8 @@
 // Attention of a step's rows over paged caches, for layers described by a cmlb200_attn: grouped heads
 // with separate query/key and value sizes, a sliding window or chunks (with or without the sequence's first
 // tokens kept in sight), a per-head linear distance bias, a sink (one, or a learned exponential per head, added
-// to the softmax denominator), norms over all heads or per head, values that are the keys before their norm, a
-// per-head output gate. Rows of different sequences share a launch; every row finds its keys through its
+// to the softmax denominator), norms over all heads or per head, rotated queries and keys, values that are the keys before their
+// norm, scores that another kernel has made (talk_scores.cu), a per-head output gate. Rows of different sequences share a launch; every row finds its keys through its
 // sequence's block table.
 //
 //   attention_tiles_kernel   prompt portions: 64 consecutive query rows of one sequence and one head per
@@ -36,16 +36,17 @@ __device__ __forceinline__ float sink_score(const cmlb200_attn& a, int h) { retu
 __device__ __forceinline__ float out_scale(const cmlb200_attn& a) { return a.out_scale == 0.f ? 1.f : a.out_scale; }
 
 // grid = (tiles, heads). tiles[i] = {first row, rows (1..64), sequence slot, position of the first row}.
-// DV: room for value columns. DK: 0, or the padded key size, and then DV is the padded value size.
-template <int DV, int DK>
+// DV: room for value columns. DK: 0, or the padded key size, and then DV is the padded value size. SCORED: scores come from
+// a.scores, so there are neither queries nor keys.
+template <int DV, int DK, bool SCORED>
 __global__ void __launch_bounds__(TILE_THREADS)
 attention_tiles_kernel(const cmlb200_attn a, const float* __restrict__ qkv, int ld, const int4* __restrict__ tiles, __nv_bfloat16* __restrict__ out,
                        int out_ld) {
     extern __shared__ __align__(16) __half sm[];
     const int dk = DK ? DK : a.dim_ld, dv = DK ? DV : a.vdim_ld, LK = dk + 8, LV = dv + 8;
     __half* Qs = sm;
-    __half* Ks = Qs + QT * LK;                         // two stages each
-    __half* Vs = Ks + 2 * KT * LK;
+    __half* Ks = Qs + (SCORED ? 0 : QT * LK);          // two stages each
+    __half* Vs = Ks + (SCORED ? 0 : 2 * KT * LK);
     dep_wait();
     dep_trigger();
     const int4 tl = tiles[blockIdx.x];
@@ -69,13 +70,14 @@ attention_tiles_kernel(const cmlb200_attn a, const float* __restrict__ qkv, int 
         for (int row = threadIdx.x >> 3; row < KT; row += TILE_THREADS / 8) {
             const int key = min(kt + row, p_last);     // rows past the end repeat the last key (masked below)
             const size_t slot = ((size_t)table[key >> shift] << shift) + (key & (a.block_size - 1));
-            for (int c = threadIdx.x & 7; c < kc; c += 8) cp16(smem_addr(Ks + (st * KT + row) * LK + c * 8), kp + slot * kstride + c * 8);
+            if (!SCORED)
+                for (int c = threadIdx.x & 7; c < kc; c += 8) cp16(smem_addr(Ks + (st * KT + row) * LK + c * 8), kp + slot * kstride + c * 8);
             for (int c = threadIdx.x & 7; c < vc; c += 8) cp16(smem_addr(Vs + (st * KT + row) * LV + c * 8), vp + slot * vstride + c * 8);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     load(0);
-    {
+    if (!SCORED) {
         const float qs = a.scale * kLog2e;
         for (int r = warp; r < QT; r += TILE_THREADS / 32) {
             const float* src = qkv + (size_t)(tl.x + min(r, n - 1)) * ld + h * a.dim;
@@ -99,6 +101,7 @@ attention_tiles_kernel(const cmlb200_attn a, const float* __restrict__ qkv, int 
 #pragma unroll
     for (int i = 0; i < KT / 8; i++) { bias[i][0] = slope * (float)(i * 8 + 2 * t); bias[i][1] = slope * (float)(i * 8 + 2 * t + 1); }
     const uint32_t q_base = smem_addr(Qs + (warp * 16 + (lane & 15)) * LK + (lane >> 4) * 8);
+    const float* scores = SCORED ? a.scores + (((size_t)blockIdx.x * a.heads + h) * QT + r0) * a.scores_ld : nullptr;
 
     for (int it = 0; it < ntiles; it++) {
         if (it + 1 < ntiles) {
@@ -115,17 +118,26 @@ attention_tiles_kernel(const cmlb200_attn a, const float* __restrict__ qkv, int 
             float s[KT / 8][4];
 #pragma unroll
             for (int i = 0; i < KT / 8; i++) { s[i][0] = bias[i][0]; s[i][1] = bias[i][1]; s[i][2] = bias[i][0]; s[i][3] = bias[i][1]; }
-            const uint32_t k_base = smem_addr(Ks + (st * KT + (lane & 7) + ((lane >> 4) & 1) * 8) * LK + ((lane >> 3) & 1) * 8);
-#pragma unroll (DK ? DK / 16 : 1)
-            for (int kk = 0; kk < dk; kk += 16) {
-                uint32_t qa[4];
-                ldsm4(q_base + kk * 2, qa);
+            if constexpr (SCORED) {
+                const float* src = scores + kt - k_lo + 2 * t;
 #pragma unroll
-                for (int j = 0; j < KT / 16; j++) {
-                    uint32_t b[4];
-                    ldsm4(k_base + (j * 16 * LK + kk) * 2, b);
-                    mma_f16(s[2 * j], qa, b[0], b[1]);
-                    mma_f16(s[2 * j + 1], qa, b[2], b[3]);
+                for (int i = 0; i < KT / 8; i++) {
+                    const float2 x = *reinterpret_cast<const float2*>(src + i * 8), y = *reinterpret_cast<const float2*>(src + (size_t)8 * a.scores_ld + i * 8);
+                    s[i][0] += x.x; s[i][1] += x.y; s[i][2] += y.x; s[i][3] += y.y;
+                }
+            } else {
+                const uint32_t k_base = smem_addr(Ks + (st * KT + (lane & 7) + ((lane >> 4) & 1) * 8) * LK + ((lane >> 3) & 1) * 8);
+#pragma unroll (DK ? DK / 16 : 1)
+                for (int kk = 0; kk < dk; kk += 16) {
+                    uint32_t qa[4];
+                    ldsm4(q_base + kk * 2, qa);
+#pragma unroll
+                    for (int j = 0; j < KT / 16; j++) {
+                        uint32_t b[4];
+                        ldsm4(k_base + (j * 16 * LK + kk) * 2, b);
+                        mma_f16(s[2 * j], qa, b[0], b[1]);
+                        mma_f16(s[2 * j + 1], qa, b[2], b[3]);
+                    }
                 }
             }
             // unless every row of the warp sees every key of the tile
@@ -226,17 +238,19 @@ attention_tiles_kernel(const cmlb200_attn a, const float* __restrict__ qkv, int 
 constexpr int ONE_THREADS = 128, ONE_WARPS = ONE_THREADS / 32;
 
 // grid = (splits, kv_heads * passes, rows), clusters of `splits` CTAs along x. Pass b of a key/value
-// head serves its query heads b * RM .. b * RM + RM - 1. A lane owns VP * 2 consecutive value columns.
-template <int RM, int VP>
+// head serves its query heads b * RM .. b * RM + RM - 1. A lane owns VP * 2 consecutive value columns. SCORED: scores come from
+// a.scores, the row's own among them, and the cache holds the row's value already.
+template <int RM, int VP, bool SCORED>
 __global__ void __launch_bounds__(ONE_THREADS)
 attention_one_kernel(const cmlb200_attn a, const float* __restrict__ qkv, int ld, const int* __restrict__ row_pos, const int* __restrict__ row_slot,
                      __nv_bfloat16* __restrict__ out, int out_ld) {
     extern __shared__ __align__(16) float fs[];
     const int dk = a.dim_ld, dv = a.vdim_ld, group = a.heads / a.kv_heads, passes = (group + RM - 1) / RM;
-    float* q_s = fs;                                   // [RM][dk], normed and scaled
-    float* k_new = q_s + RM * dk;                      // [dk] and [dv] as the cache holds them
-    float* v_new = k_new + dk;
-    float* w_m = v_new + dv;                           // [ONE_WARPS][RM] maxima and sums
+    float* q_s = fs;                                   // [RM][dk], normed, rotated and scaled
+    float* k_new = q_s + (SCORED ? 0 : RM * dk);       // [dk] and [dv] as the cache holds them
+    float* v_new = k_new + (SCORED ? 0 : dk);
+    float* turn = v_new + (SCORED ? 0 : dv);           // [rot_dims]: cosines, then sines
+    float* w_m = turn + (SCORED || !a.freq ? 0 : a.rot_dims);                         // [ONE_WARPS][RM] maxima and sums
     float* w_l = w_m + ONE_WARPS * RM;
     float* c_m = w_l + ONE_WARPS * RM;                 // [RM] this CTA's
     float* c_l = c_m + RM;
@@ -252,46 +266,63 @@ attention_one_kernel(const cmlb200_attn a, const float* __restrict__ qkv, int ld
     const int shift = __ffs(a.block_size) - 1;
     const int* table = a.block_table + (size_t)row_slot[r] * a.table_ld;
 
-    float iq = 1.0f, ik = 1.0f;
-    __shared__ float head_inv[RM + 1];                 // per-head norms: of this CTA's query heads, then of its key
-    if (a.head_norm) {
-        for (int j = warp; j <= nh; j += ONE_WARPS) {
-            const float* v = j < nh ? row + (h0 + j) * a.dim : row + qw + kh * a.dim;
-            float ss = 0.f;
-            for (int d = lane; d < a.dim; d += 32) ss = fmaf(v[d], v[d], ss);
-            ss = lane_sum(ss);
-            if (lane == 0) head_inv[j < nh ? j : RM] = (j < nh ? a.q_norm : a.k_norm) ? 1.0f / sqrtf(ss / (float)a.dim + a.eps) : 1.0f;
+    if constexpr (!SCORED) {
+        float iq = 1.0f, ik = 1.0f;
+        __shared__ float head_inv[RM + 1];             // per-head norms: of this CTA's query heads, then of its key
+        if (a.freq) {
+            const int half = a.rot_dims / 2;
+            for (int i = threadIdx.x; i < half; i += ONE_THREADS) sincosf((float)p * a.freq[i], &turn[half + i], &turn[i]);
+            __syncthreads();
+        }
+        if (a.head_norm) {
+            for (int j = warp; j <= nh; j += ONE_WARPS) {
+                const float* v = j < nh ? row + (h0 + j) * a.dim : row + qw + kh * a.dim;
+                float ss = 0.f;
+                for (int d = lane; d < a.dim; d += 32) ss = fmaf(v[d], v[d], ss);
+                ss = lane_sum(ss);
+                if (lane == 0) head_inv[j < nh ? j : RM] = (j < nh ? a.q_norm : a.k_norm) ? 1.0f / sqrtf(ss / (float)a.dim + a.eps) : 1.0f;
+            }
+            __syncthreads();
+        } else if (a.q_norm || a.k_norm) {
+            const float2 ss = block_sum2(a.q_norm ? square_share(row, qw) : 0.f, a.k_norm && rank == 0 ? square_share(row + qw, kw) : 0.f, red);
+            if (a.q_norm) iq = 1.0f / sqrtf(ss.x / (float)qw + a.eps);
+            if (a.k_norm) ik = 1.0f / sqrtf(ss.y / (float)kw + a.eps);  // used where the row's own key is made: rank 0
+        }
+        const float temp = a.temp_every > 0.f ? 1.0f + a.temp_coef * logf(floorf((float)(p + 1) / a.temp_every) + 1.0f) : 1.0f;
+        const float qs = a.scale * kLog2e;
+        // entry d of a head's vector v, turned with the one beside it
+        auto turned = [&](int d, auto v) {
+            if (!a.freq || d >= a.rot_dims) return v(d);
+            const float c = turn[d >> 1], n = turn[(a.rot_dims + d) >> 1];
+            return (d & 1) ? v(d) * c + v(d - 1) * n : v(d) * c - v(d + 1) * n;
+        };
+        for (int i = threadIdx.x; i < RM * dk; i += ONE_THREADS) {
+            const int j = i / dk, d0 = i - j * dk;
+            q_s[i] = (j < nh && d0 < a.dim) ? turned(d0, [&](int d) {
+                const int c = (h0 + j) * a.dim + d;
+                return row[c] * (a.head_norm ? head_inv[j] : iq) * (a.q_norm ? a.q_norm[a.head_norm ? d : c] : 1.0f) * temp * qs;
+            }) : 0.f;
+        }
+        if (rank == 0) {
+            const size_t slot = ((size_t)table[p >> shift] << shift) + (p & (a.block_size - 1));
+            __half* kd = static_cast<__half*>(a.k_pool) + (slot * a.kv_heads + kh) * dk;
+            __half* vd = static_cast<__half*>(a.v_pool) + (slot * a.kv_heads + kh) * dv;
+            for (int d0 = threadIdx.x; d0 < dk; d0 += ONE_THREADS) {
+                const __half v = narrow<__half>(d0 < a.dim ? turned(d0, [&](int d) {
+                    const int c = kh * a.dim + d;
+                    return row[qw + c] * (a.head_norm ? head_inv[RM] : ik) * (a.k_norm ? a.k_norm[a.head_norm ? d : c] : 1.0f);
+                }) : 0.f);
+                k_new[d0] = __half2float(v);
+                if (pass == 0) kd[d0] = v;
+            }
+            for (int d = threadIdx.x; d < dv; d += ONE_THREADS) {
+                const __half v = narrow<__half>(d < a.vdim ? row[qw + (a.keys_as_values ? 0 : kw) + kh * a.vdim + d] : 0.f);
+                v_new[d] = __half2float(v);
+                if (pass == 0) vd[d] = v;
+            }
         }
         __syncthreads();
-    } else if (a.q_norm || a.k_norm) {
-        const float2 ss = block_sum2(a.q_norm ? square_share(row, qw) : 0.f, a.k_norm && rank == 0 ? square_share(row + qw, kw) : 0.f, red);
-        if (a.q_norm) iq = 1.0f / sqrtf(ss.x / (float)qw + a.eps);
-        if (a.k_norm) ik = 1.0f / sqrtf(ss.y / (float)kw + a.eps);      // used where the row's own key is made: rank 0
     }
-    const float temp = a.temp_every > 0.f ? 1.0f + a.temp_coef * logf(floorf((float)(p + 1) / a.temp_every) + 1.0f) : 1.0f;
-    const float qs = a.scale * kLog2e;
-    for (int i = threadIdx.x; i < RM * dk; i += ONE_THREADS) {
-        const int j = i / dk, d = i - j * dk;
-        const int c = (h0 + j) * a.dim + d;
-        q_s[i] = (j < nh && d < a.dim) ? row[c] * (a.head_norm ? head_inv[j] : iq) * (a.q_norm ? a.q_norm[a.head_norm ? d : c] : 1.0f) * temp * qs : 0.f;
-    }
-    if (rank == 0) {
-        const size_t slot = ((size_t)table[p >> shift] << shift) + (p & (a.block_size - 1));
-        __half* kd = static_cast<__half*>(a.k_pool) + (slot * a.kv_heads + kh) * dk;
-        __half* vd = static_cast<__half*>(a.v_pool) + (slot * a.kv_heads + kh) * dv;
-        for (int d = threadIdx.x; d < dk; d += ONE_THREADS) {
-            const int c = kh * a.dim + d;
-            const __half v = narrow<__half>(d < a.dim ? row[qw + c] * (a.head_norm ? head_inv[RM] : ik) * (a.k_norm ? a.k_norm[a.head_norm ? d : c] : 1.0f) : 0.f);
-            k_new[d] = __half2float(v);
-            if (pass == 0) kd[d] = v;
-        }
-        for (int d = threadIdx.x; d < dv; d += ONE_THREADS) {
-            const __half v = narrow<__half>(d < a.vdim ? row[qw + (a.keys_as_values ? 0 : kw) + kh * a.vdim + d] : 0.f);
-            v_new[d] = __half2float(v);
-            if (pass == 0) vd[d] = v;
-        }
-    }
-    __syncthreads();
 
     float m[RM], l[RM], acc[RM][2 * VP], slope[RM];
 #pragma unroll
@@ -303,7 +334,7 @@ attention_one_kernel(const cmlb200_attn a, const float* __restrict__ qkv, int ld
         for (int e = 0; e < 2 * VP; e++) acc[j][e] = 0.f;
     }
     // the keys in sight, numbered from 0: the kept ones, then those from k_lo on
-    const int k_lo = first_key(a, p), kept = min(a.keep, k_lo), skip = k_lo - kept, seen = p - skip;
+    const int k_lo = first_key(a, p), kept = min(a.keep, k_lo), skip = k_lo - kept, seen = p - skip + (SCORED ? 1 : 0);
     const __half* kp = static_cast<const __half*>(a.k_pool) + (size_t)kh * dk;
     const __half* vp = static_cast<const __half*>(a.v_pool) + (size_t)kh * dv;
     const int kstride = a.kv_heads * dk, vstride = a.kv_heads * dv;
@@ -335,8 +366,12 @@ attention_one_kernel(const cmlb200_attn a, const float* __restrict__ qkv, int ld
         uint32_t u[PRE][VP];
         load_values(u, slot, 0);
         const uint4* kr = reinterpret_cast<const uint4*>(kp + (size_t)slot * kstride);
+        if constexpr (SCORED) {
+#pragma unroll
+            for (int j = 0; j < RM; j++) s[j] = a.scores[((size_t)r * a.heads + h0 + min(j, nh - 1)) * a.scores_ld + nth];
+        }
 #pragma unroll 8
-        for (int c = 0; c < (dk >> 3); c++) {
+        for (int c = 0; c < (SCORED ? 0 : dk >> 3); c++) {
             const uint4 w = kr[c];
             const float2 k01 = __half22float2(*reinterpret_cast<const __half2*>(&w.x)), k23 = __half22float2(*reinterpret_cast<const __half2*>(&w.y));
             const float2 k45 = __half22float2(*reinterpret_cast<const __half2*>(&w.z)), k67 = __half22float2(*reinterpret_cast<const __half2*>(&w.w));
@@ -377,7 +412,7 @@ attention_one_kernel(const cmlb200_attn a, const float* __restrict__ qkv, int ld
     }
 #pragma unroll
     for (int j = 0; j < RM; j++) l[j] = lane_sum(l[j]);
-    if (rank == 0 && warp == 0) {                      // the row's own key and value, distance 0
+    if (!SCORED && rank == 0 && warp == 0) {           // the row's own key and value, distance 0
 #pragma unroll
         for (int j = 0; j < RM; j++) {
             float s = 0.f;
@@ -489,7 +524,8 @@ attention_rows_f32_kernel(const cmlb200_attn a, const float* __restrict__ qkv, i
     const float* kp = static_cast<const float*>(a.k_pool) + (size_t)kh * a.dim_ld;
     const float* vp = static_cast<const float*>(a.v_pool) + (size_t)kh * a.vdim_ld;
     const float slope = a.slopes ? a.slopes[h] : 0.f;
-    for (int d = threadIdx.x; d < a.dim; d += ROW_THREADS) q_s[d] = row[h * a.dim + d];
+    const float* given = a.scores ? a.scores + ((size_t)r * a.heads + h) * a.scores_ld : nullptr;
+    for (int d = threadIdx.x; d < a.dim && !given; d += ROW_THREADS) q_s[d] = row[h * a.dim + d];
     for (int d = threadIdx.x; d < a.vdim; d += ROW_THREADS) acc[d] = 0.f;
     float m = a.sink ? sink_score(a, h) : -INFINITY, l = a.sink ? 1.f : 0.f;
     const int k_lo = first_key(a, p), kept = min(a.keep, k_lo), skip = k_lo - kept, seen = p + 1 - skip;
@@ -502,7 +538,8 @@ attention_rows_f32_kernel(const cmlb200_attn a, const float* __restrict__ qkv, i
             slots[threadIdx.x] = table[key / a.block_size] * a.block_size + key % a.block_size;
         }
         __syncthreads();
-        for (int k = warp; k < n; k += ROW_THREADS / 32) {
+        if (given && (int)threadIdx.x < n) sc[threadIdx.x] = given[kt + threadIdx.x];
+        for (int k = warp; k < n && !given; k += ROW_THREADS / 32) {
             const float* kr = kp + (size_t)slots[k] * a.kv_heads * a.dim_ld;
             float s = 0.f;
             for (int d = lane; d < a.dim; d += 32) s = fmaf(q_s[d], kr[d], s);
@@ -540,6 +577,8 @@ extern "C" int cmlb200_attn_check_(const cmlb200_attn* a, const char* who) {
     CMLB_REQUIRE(a->keep >= 0 && a->chunk >= 0 && (!a->keys_as_values || a->dim == a->vdim), "%s: kept tokens %d, chunk %d, values as keys of %d / %d", who, a->keep,
                  a->chunk, a->dim, a->vdim);
     CMLB_REQUIRE(a->k_pool && a->v_pool && a->block_table && a->table_ld > 0, "%s: no cache", who);
+    CMLB_REQUIRE(!a->scores || (a->scores_ld > 0 && !a->slopes && a->chunk == 0 && a->keep == 0), "%s: given scores go with windows alone, stride %d", who, a->scores_ld);
+    CMLB_REQUIRE(!a->freq || (a->rot_dims > 0 && a->rot_dims % 2 == 0 && a->rot_dims <= a->dim), "%s: %d of %d dimensions rotated", who, a->rot_dims, a->dim);
     CMLB_REQUIRE(a->block_size > 0 && (a->block_size & (a->block_size - 1)) == 0 && a->block_size % 16 == 0, "%s: block size %d must be a power of two >= 16", who, a->block_size);
     CMLB_REQUIRE((((uintptr_t)a->k_pool | (uintptr_t)a->v_pool) & 15) == 0, "%s: pools must be 16-byte aligned", who);
     return CMLB200_OK;
@@ -552,23 +591,30 @@ extern "C" int cmlb200_attention_tiles(const cmlb200_attn* a, const float* d_qkv
     if (rc) return rc;
     CMLB_REQUIRE(a->cache_dtype == CMLB200_DT_F16 && a->vdim_ld <= 256 && a->heads <= 65535, "cmlb200_attention_tiles: fp16 cache and value heads up to 256");
     CMLB_REQUIRE(((uintptr_t)d_tiles & 15) == 0, "cmlb200_attention_tiles: the tile list must be 16-byte aligned");
-    const size_t smem = 2 * ((size_t)(QT + 2 * KT) * (a->dim_ld + 8) + (size_t)2 * KT * (a->vdim_ld + 8));
+    const bool scored = a->scores != nullptr;
+    CMLB_REQUIRE(!scored || (a->scores_ld % 64 == 0 && ((uintptr_t)a->scores & 15) == 0), "cmlb200_attention_tiles: score stride %d", a->scores_ld);
+    const size_t smem = 2 * ((scored ? 0 : (size_t)(QT + 2 * KT) * (a->dim_ld + 8)) + (size_t)2 * KT * (a->vdim_ld + 8));
     CMLB_REQUIRE(smem <= 227 * 1024, "cmlb200_attention_tiles: head sizes %d / %d do not fit shared memory", a->dim, a->vdim);
     cudaStream_t st = as_stream(stream);
     const dim3 grid(tiles, a->heads);
-    static size_t attr[6][kMaxDevices] = {};
-#define AT_LAUNCH(DV, DK, slot)                                                                                                   \
+    static size_t attr[9][kMaxDevices] = {};
+#define AT_LAUNCH(DV, DK, S, slot)                                                                                                   \
     do {                                                                                                                        \
-        auto kern = attention_tiles_kernel<DV, DK>;                                                                               \
+        auto kern = attention_tiles_kernel<DV, DK, S>;                                                                               \
         CMLB_CUDA(cmlb_ensure_smem(kern, smem, attr[slot]));                                                                    \
         CMLB_CUDA(launch_chain(kern, grid, dim3(TILE_THREADS), smem, 1, st, *a, d_qkv, ld, (const int4*)d_tiles, (__nv_bfloat16*)d_out_bf16, out_ld)); \
     } while (0)
-    if (a->vdim_ld == 64 && a->dim_ld == 64) AT_LAUNCH(64, 64, 3);
-    else if (a->vdim_ld == 128 && a->dim_ld == 128) AT_LAUNCH(128, 128, 4);
-    else if (a->vdim_ld == 128 && a->dim_ld == 192) AT_LAUNCH(128, 192, 5);
-    else if (a->vdim_ld <= 64) AT_LAUNCH(64, 0, 0);
-    else if (a->vdim_ld <= 128) AT_LAUNCH(128, 0, 1);
-    else AT_LAUNCH(256, 0, 2);
+    if (scored) {
+        if (a->vdim_ld <= 64) AT_LAUNCH(64, 0, true, 6);
+        else if (a->vdim_ld <= 128) AT_LAUNCH(128, 0, true, 7);
+        else AT_LAUNCH(256, 0, true, 8);
+    }
+    else if (a->vdim_ld == 64 && a->dim_ld == 64) AT_LAUNCH(64, 64, false, 3);
+    else if (a->vdim_ld == 128 && a->dim_ld == 128) AT_LAUNCH(128, 128, false, 4);
+    else if (a->vdim_ld == 128 && a->dim_ld == 192) AT_LAUNCH(128, 192, false, 5);
+    else if (a->vdim_ld <= 64) AT_LAUNCH(64, 0, false, 0);
+    else if (a->vdim_ld <= 128) AT_LAUNCH(128, 0, false, 1);
+    else AT_LAUNCH(256, 0, false, 2);
 #undef AT_LAUNCH
     return CMLB200_OK;
 }
@@ -588,27 +634,36 @@ extern "C" int cmlb200_attention_one(const cmlb200_attn* a, const float* d_qkv, 
     const long long base = (long long)rows * a->kv_heads * passes;
     int splits = 1;
     while (splits < 8 && base * splits < 2 * cmlb_num_sms() && keys > splits * ONE_WARPS * 32) splits *= 2;
-    const size_t smem = sizeof(float) * ((size_t)rm * a->dim_ld + a->dim_ld + a->vdim_ld + 2 * ONE_WARPS * rm + 2 * rm + (size_t)ONE_WARPS * rm * a->vdim_ld);
+    const bool scored = a->scores != nullptr;
+    CMLB_REQUIRE(!scored || a->scores_ld >= keys, "cmlb200_attention_one: score stride %d for %d keys", a->scores_ld, keys);
+    const size_t operands = scored ? 0 : (size_t)rm * a->dim_ld + a->dim_ld + a->vdim_ld + (a->freq ? a->rot_dims : 0);
+    const size_t smem = sizeof(float) * (operands + 2 * ONE_WARPS * rm + 2 * rm + (size_t)ONE_WARPS * rm * a->vdim_ld);
     CMLB_REQUIRE(smem <= 200 * 1024, "cmlb200_attention_one: head sizes %d / %d do not fit shared memory", a->dim, a->vdim);
     cudaStream_t st = as_stream(stream);
     const dim3 grid(splits, a->kv_heads * passes, rows);
     const int vp = a->vdim_ld <= 64 ? 1 : (a->vdim_ld <= 128 ? 2 : 4);
-    static size_t attr[9][kMaxDevices] = {};
-#define AO_LAUNCH(RM, VP, slot)                                                                                                  \
+    static size_t attr[18][kMaxDevices] = {};
+#define AO_LAUNCH(RM, VP, S, slot)                                                                                                  \
     do {                                                                                                                         \
-        auto kern = attention_one_kernel<RM, VP>;                                                                                \
+        auto kern = attention_one_kernel<RM, VP, S>;                                                                                \
         CMLB_CUDA(cmlb_ensure_smem(kern, smem, attr[slot]));                                                                     \
         CMLB_CUDA(launch_chain(kern, grid, dim3(ONE_THREADS), smem, splits, st, *a, d_qkv, ld, d_row_pos, d_row_slot, (__nv_bfloat16*)d_out_bf16, out_ld)); \
     } while (0)
-#define AO_ROWS(RM, slot)                                \
-    do {                                                 \
-        if (vp == 1) AO_LAUNCH(RM, 1, slot);             \
-        else if (vp == 2) AO_LAUNCH(RM, 2, slot + 1);    \
-        else AO_LAUNCH(RM, 4, slot + 2);                 \
+#define AO_ROWS(RM, S, slot)                                \
+    do {                                                    \
+        if (vp == 1) AO_LAUNCH(RM, 1, S, slot);             \
+        else if (vp == 2) AO_LAUNCH(RM, 2, S, slot + 1);    \
+        else AO_LAUNCH(RM, 4, S, slot + 2);                 \
     } while (0)
-    if (rm == 1) AO_ROWS(1, 0);
-    else if (rm == 4) AO_ROWS(4, 3);
-    else AO_ROWS(8, 6);
+#define AO_FORM(S, slot)                                    \
+    do {                                                    \
+        if (rm == 1) AO_ROWS(1, S, slot);                   \
+        else if (rm == 4) AO_ROWS(4, S, slot + 3);          \
+        else AO_ROWS(8, S, slot + 6);                       \
+    } while (0)
+    if (scored) AO_FORM(true, 9);
+    else AO_FORM(false, 0);
+#undef AO_FORM
 #undef AO_ROWS
 #undef AO_LAUNCH
     return CMLB200_OK;

@@ -11,7 +11,7 @@
 // Two accumulators alternate in tensor memory, so the epilogue of a tile overlaps the next tile's MMAs.
 // Output forms: fp32; or the gated activation of weights stored as pairs of 16-row groups (16 gate
 // rows, 16 up rows, ...): both halves of a pair sit in one lane's columns, and bf16 act(gate) * up is
-// all that leaves the SM; or per-head keys and values as fp16 cache rows. Rows and columns past the edges arrive as
+// all that leaves the SM; or bf16 act(y); or per-head keys and values as fp16 cache rows. Rows and columns past the edges arrive as
 // zeros and are not stored. With a plan of experts the row tiles come from the plan: each has a first row, a number of
 // rows and an expert, whose weight rows follow those of the expert before it.
 // No cluster multicast. Every mbarrier wait is bounded; on expiry the CTA raises a status word
@@ -48,7 +48,7 @@ __device__ __forceinline__ void tile_at(int i, int tm, int tn, int& m, int& n) {
     n = in / rows;
 }
 
-enum { OUT_F32, OUT_GLU, OUT_HEADS };
+enum { OUT_F32, OUT_GLU, OUT_ACT, OUT_HEADS };
 struct GemmOut {
     int form, act;
     float limit;
@@ -193,6 +193,11 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constant
 #pragma unroll 8
                         for (int j = 0; j < 32; j++)
                             if (m0 + j < m_end && col < out.n_out) static_cast<float*>(out.y)[(size_t)(m0 + j) * out.ldy + col] = buf[j * 33 + lane] + bias;
+                    } else if (out.form == OUT_ACT) {
+#pragma unroll 8
+                        for (int j = 0; j < 32; j++)
+                            if (m0 + j < m_end && col < out.n_out)
+                                static_cast<__nv_bfloat16*>(out.y)[(size_t)(m0 + j) * out.ldy + col] = __float2bfloat16_rn(unary_act_fast(out.act, buf[j * 33 + lane]));
                     } else {
                         const bool key = col < out.key_cols;
                         const int c = key ? col : col - out.key_cols, per = key ? out.dim : out.vdim, ldo = key ? out.ldk : out.ldy;
@@ -290,6 +295,15 @@ extern "C" int cmlb200_moe_gemm_glu(const cmlb200_moe* m, const cmlb200_dense* W
     GemmOut out = {};
     out.form = OUT_GLU; out.act = act; out.limit = limit; out.y = d_f; out.ldy = ldf; out.n_out = ff;
     return gemm_experts(m, W, d_x, ldx, rows, out, "cmlb200_moe_gemm_glu", stream);
+}
+
+extern "C" int cmlb200_moe_gemm_act(const cmlb200_moe* m, const cmlb200_dense* W, const uint16_t* d_x, int ldx, int rows, int ff, int act, uint16_t* d_f, int ldf,
+                                    void* stream) {
+    CMLB_REQUIRE(m && W && ff > 0 && W->rows == m->experts * ((ff + 15) & ~15) && ldf >= ff, "cmlb200_moe_gemm_act: weight rows do not fit %d outputs", ff);
+    CMLB_REQUIRE(act == CMLB200_ACT_SILU || act == CMLB200_ACT_GELU_TANH || act == CMLB200_ACT_GELU_ERF, "cmlb200_moe_gemm_act: activation %d", act);
+    GemmOut out = {};
+    out.form = OUT_ACT; out.act = act; out.y = d_f; out.ldy = ldf; out.n_out = ff;
+    return gemm_experts(m, W, d_x, ldx, rows, out, "cmlb200_moe_gemm_act", stream);
 }
 
 extern "C" int cmlb200_latent_expand(const cmlb200_latent* a, const cmlb200_dense* W, const uint16_t* d_c_bf16, int rows, const cmlb200_attn* s, void* stream) {

@@ -18,7 +18,8 @@ constexpr int GV_WARPS = 8;
 // RT tiles of 16 weight rows per CTA, NB groups of 8 rows of x. GLU: tile 0 = 16 gate rows, tile 1 = the
 // 16 up rows that go with them; the output is bf16 act(gate) * up.
 // EXPERT: blockIdx.y counts the chosen experts; an expert's w_rows weight rows follow those of the one before it, its
-// rows of x are those that chose it (m.src, or the positions themselves), and y has a row per position.
+// rows of x are those that chose it (m.src, or the positions themselves), and y has a row per position. Without a gate its
+// output is fp32, or bf16 act(y) where act is not negative.
 struct GemvExperts {
     cmlb200_moe m;
     int w_rows, gather;
@@ -122,7 +123,8 @@ gemv_bf16_kernel(const __nv_bfloat16* __restrict__ W, int ldw, const __nv_bfloat
         } else if (n0 + n < N) {
             if (!EXPERT && bias) s += bias[n0 + n];
             if (!EXPERT && cap > 0.f) s = soft_cap(s, cap);
-            static_cast<float*>(y)[(size_t)(first + m) * ldy + n0 + n] = s;
+            if (EXPERT && act >= 0) static_cast<__nv_bfloat16*>(y)[(size_t)(first + m) * ldy + n0 + n] = __float2bfloat16_rn(unary_act_fast(act, s));
+            else static_cast<float*>(y)[(size_t)(first + m) * ldy + n0 + n] = s;
         }
     }
 }
@@ -186,7 +188,7 @@ extern "C" int cmlb200_moe_gemv(const cmlb200_moe* m, const cmlb200_dense* W, co
     if (rc) return rc;
     CMLB_REQUIRE(m && m->experts > 0 && m->experts <= 65535 && W->rows % (16 * m->experts) == 0 && n_out > 0 && n_out <= W->rows / m->experts && ldy >= n_out,
                  "cmlb200_moe_gemv: %d weight rows, %d outputs, stride %d", W->rows, n_out, ldy);
-    return launch_gemv_experts<1, false>(m, W, d_x, ldx, gather, rows, 0, 0.f, d_y, ldy, n_out, as_stream(stream));
+    return launch_gemv_experts<1, false>(m, W, d_x, ldx, gather, rows, -1, 0.f, d_y, ldy, n_out, as_stream(stream));
 }
 
 extern "C" int cmlb200_moe_gemv_glu(const cmlb200_moe* m, const cmlb200_dense* W, const uint16_t* d_x, int ldx, int gather, int rows, int ff, int act,
@@ -196,4 +198,14 @@ extern "C" int cmlb200_moe_gemv_glu(const cmlb200_moe* m, const cmlb200_dense* W
     CMLB_REQUIRE(m && m->experts > 0 && m->experts <= 65535 && ff > 0 && W->rows == m->experts * 2 * ((ff + 15) & ~15) && ldf >= ff,
                  "cmlb200_moe_gemv_glu: %d weight rows for %d outputs", W->rows, ff);
     return launch_gemv_experts<2, true>(m, W, d_x, ldx, gather, rows, act, limit, d_f, ldf, ff, as_stream(stream));
+}
+
+extern "C" int cmlb200_moe_gemv_act(const cmlb200_moe* m, const cmlb200_dense* W, const uint16_t* d_x, int ldx, int gather, int rows, int ff, int act, uint16_t* d_f,
+                                    int ldf, void* stream) {
+    const int rc = check_gemv(W, d_x, ldx, rows, d_f, "cmlb200_moe_gemv_act");
+    if (rc) return rc;
+    CMLB_REQUIRE(m && m->experts > 0 && m->experts <= 65535 && ff > 0 && W->rows == m->experts * ((ff + 15) & ~15) && ldf >= ff,
+                 "cmlb200_moe_gemv_act: %d weight rows for %d outputs", W->rows, ff);
+    CMLB_REQUIRE(act == CMLB200_ACT_SILU || act == CMLB200_ACT_GELU_TANH || act == CMLB200_ACT_GELU_ERF, "cmlb200_moe_gemv_act: activation %d", act);
+    return launch_gemv_experts<1, false>(m, W, d_x, ldx, gather, rows, act, 0.f, d_f, ldf, ff, as_stream(stream));
 }

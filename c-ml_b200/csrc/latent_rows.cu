@@ -1,6 +1,6 @@
 // Row-wise pieces of latent attention (cmlb200_latent): the cache append (norm of the latent, rotation of the shared
 // key part) with the rotation of the queries; the two per-head products around attention over latents
-// (q -> Wuk^T q in front, o -> Wuv o with the element-wise gate behind); and the gathering of a long portion's latents
+// (q -> Wuk^T q in front, o -> Wuv o with the gate, per element or per head, behind); and the gathering of a long portion's latents
 // for the expansion into per-head keys and values. Norms, angles and rotations are fp32.
 #include "lm_util.cuh"
 
@@ -231,16 +231,16 @@ latent_output_kernel(const cmlb200_latent a, const __nv_bfloat16* __restrict__ w
         float s = 0.f;
 #pragma unroll
         for (int k = 0; k < LO_WARPS; k++) s += part[k][v][m];
-        if (a.gate_col >= 0) s *= sigmoidf(proj[(size_t)(r0 + m) * ld + a.gate_col + col]);
+        if (a.gate_col >= 0) s *= sigmoidf(proj[(size_t)(r0 + m) * ld + a.gate_col + (a.gate_heads ? h : col)]);
         out[(size_t)(r0 + m) * out_ld + col] = __float2bfloat16_rn(s);
     }
 }
 
 // 32-bit per-head product, a warp per output: y[r][h * y_ld + n] = sum_k x[r][h * x_ld + k] W[h][n][k], times the
-// sigmoid of gate[r][h * N + n]. grid = (N / 8, heads, rows).
+// sigmoid of gate[r][h * N + n], or of gate[r][h]. grid = (N / 8, heads, rows).
 __global__ void __launch_bounds__(256)
 heads_linear_f32_kernel(const float* __restrict__ W, int N, int K, const float* __restrict__ x, size_t x_row, int x_ld, const float* __restrict__ gate,
-                        size_t gate_row, float* __restrict__ y, size_t y_row, int y_ld) {
+                        size_t gate_row, int gate_heads, float* __restrict__ y, size_t y_row, int y_ld) {
     dep_wait();
     dep_trigger();
     const int n = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31, h = blockIdx.y;
@@ -250,7 +250,7 @@ heads_linear_f32_kernel(const float* __restrict__ W, int N, int K, const float* 
     float s = 0.f;
     for (int k = lane; k < K; k += 32) s = fmaf(w[k], xr[k], s);
     s = lane_sum(s);
-    if (gate) s *= sigmoidf(gate[blockIdx.z * gate_row + (size_t)h * N + n]);
+    if (gate) s *= sigmoidf(gate[blockIdx.z * gate_row + (gate_heads ? (size_t)h : (size_t)h * N + n)]);
     if (lane == 0) y[blockIdx.z * y_row + (size_t)h * y_ld + n] = s;
 }
 
@@ -317,7 +317,7 @@ int check_latent(const cmlb200_latent* a, int ld, const char* who) {
     CMLB_REQUIRE(a->block_size >= 16 && (a->block_size & (a->block_size - 1)) == 0, "%s: block size %d must be a power of two >= 16", who, a->block_size);
     CMLB_REQUIRE(a->kv_col < 0 || a->c_norm, "%s: no norm weights", who);
     CMLB_REQUIRE(ld >= a->heads * (a->dim + a->rot_dim) && (a->kv_col < 0 || ld >= a->kv_col + a->rank + a->rot_dim) &&
-                 (a->gate_col < 0 || ld >= a->gate_col + a->heads * a->vdim), "%s: row stride %d", who, ld);
+                 (a->gate_col < 0 || ld >= a->gate_col + a->heads * (a->gate_heads ? 1 : a->vdim)), "%s: row stride %d", who, ld);
     CMLB_REQUIRE(a->rot_dim <= 8192, "%s: rotated size %d", who, a->rot_dim);
     return CMLB200_OK;
 }
@@ -411,7 +411,7 @@ extern "C" int cmlb200_latent_query_f32(const cmlb200_latent* a, const float* d_
     CMLB_CUDA(launch_chain(latent_append_kernel<float>, dim3(rows), dim3(256), (size_t)a->rot_dim * 4, 1, st, *a, const_cast<float*>(d_proj), ld, d_row_pos, d_row_slot,
                            d_q, (size_t)a->heads * kd, kd, a->rank));
     CMLB_CUDA(launch_chain(heads_linear_f32_kernel, dim3((a->rank + 7) / 8, a->heads, rows), dim3(256), 0, 1, st, d_wukt, a->rank, a->dim, d_proj, (size_t)ld,
-                           a->dim + a->rot_dim, (const float*)nullptr, (size_t)0, d_q, (size_t)a->heads * kd, kd));
+                           a->dim + a->rot_dim, (const float*)nullptr, (size_t)0, 0, d_q, (size_t)a->heads * kd, kd));
     return CMLB200_OK;
 }
 
@@ -421,6 +421,6 @@ extern "C" int cmlb200_latent_output_f32(const cmlb200_latent* a, const float* d
     if (rc) return rc;
     CMLB_REQUIRE(d_wuv && d_o && d_proj && d_out && rows > 0 && rows <= 65535 && out_ld >= a->heads * a->vdim, "cmlb200_latent_output_f32: bad argument");
     CMLB_CUDA(launch_chain(heads_linear_f32_kernel, dim3((a->vdim + 7) / 8, a->heads, rows), dim3(256), 0, 1, as_stream(stream), d_wuv, a->vdim, a->rank, d_o,
-                           (size_t)a->heads * a->rank, a->rank, a->gate_col >= 0 ? d_proj + a->gate_col : (const float*)nullptr, (size_t)ld, d_out, (size_t)out_ld, a->vdim));
+                           (size_t)a->heads * a->rank, a->rank, a->gate_col >= 0 ? d_proj + a->gate_col : (const float*)nullptr, (size_t)ld, a->gate_heads, d_out, (size_t)out_ld, a->vdim));
     return CMLB200_OK;
 }

@@ -1,6 +1,6 @@
 // Row-wise kernels of the layered models: embedding with a sinusoidal position vector or into residual streams, the
-// fused "norm a sublayer's output, add it to the residual, norm the sum for the next sublayer" step and its like over
-// streams, the
+// fused "norm a sublayer's output, add it to the residual, norm the sum for the next sublayer" step and its likes over
+// streams and for two sublayers that join together through gates, the
 // query/key norm with query temperature and paged cache append, and the gated activation of the
 // 32-bit path. The residual and every norm are fp32; the operand handed to the next matrix product
 // is bf16 or fp32.
@@ -148,6 +148,124 @@ stream_join_kernel(const cmlb200_streams hc, float* __restrict__ x, const float*
             o[i] = n[0];
         }
     }
+}
+
+// One CTA per row. m: j.a, or half the sum of the norms of j.a and j.b; f: a row, or the weighted sum of the rows its pairs point at.
+// x += sigmoid(ga) m + sigmoid(gf) f (+ table[token]); with w_next: out = norm(x) * w_next, whose row waits in shared memory.
+// W: 4 or 1 columns at a time.
+template <typename TO, typename TE, int W>
+__global__ void __launch_bounds__(1024)
+gated_join_kernel(const cmlb200_gated_join j, int parts, const int* __restrict__ part_pos, const float* __restrict__ part_w, float* __restrict__ x,
+                  const float* __restrict__ w_next, float eps, int width, TO* __restrict__ out, int ldo) {
+    extern __shared__ __align__(16) float row[];
+    __shared__ float red[32];
+    __shared__ float2 red2[32];
+    dep_wait();
+    dep_trigger();
+    const int r = blockIdx.x;
+    const float *a = j.a + (size_t)r * j.ldm, *b = j.b ? j.b + (size_t)r * j.ldm : nullptr;
+    const float *ga = j.ga + (size_t)r * j.ldg, *gf = j.f ? j.gf + (size_t)r * j.ldg : nullptr;
+    float* xr = x + (size_t)r * width;
+    const TE* again = nullptr;
+    if (j.table) {
+        const int t = j.tokens[r];
+        again = static_cast<const TE*>(j.table) + (size_t)(t < 0 || t >= j.vocab ? 0 : t) * width;
+    }
+    auto load = [](const float* p, float (&v)[W]) {
+        if constexpr (W == 4) { const float4 q = *reinterpret_cast<const float4*>(p); v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w; }
+        else v[0] = *p;
+    };
+    auto store = [](float* p, const float (&v)[W]) {
+        if constexpr (W == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+        else *p = v[0];
+    };
+    float ia = 1.f, ib = 1.f;
+    if (b) {
+        const float2 ss = block_sum2(square_share(a, width), square_share(b, width), red2);
+        ia = 0.5f / sqrtf(ss.x / (float)width + eps);
+        ib = 0.5f / sqrtf(ss.y / (float)width + eps);
+    }
+    float ss = 0.f;
+    for (int i = threadIdx.x * W; i < width; i += blockDim.x * W) {
+        float v[W], m[W], g[W], p[W];
+        load(xr + i, v);
+        load(a + i, m);
+        load(ga + i, g);
+        if (b) {
+            float wa[W], wb[W];
+            load(b + i, p);
+            load(j.a_norm + i, wa);
+            load(j.b_norm + i, wb);
+#pragma unroll
+            for (int e = 0; e < W; e++) m[e] = m[e] * ia * wa[e] + p[e] * ib * wb[e];
+        }
+#pragma unroll
+        for (int e = 0; e < W; e++) v[e] = fmaf(sigmoidf(g[e]), m[e], v[e]);
+        if (j.f) {
+            if (parts > 0) {
+#pragma unroll
+                for (int e = 0; e < W; e++) m[e] = 0.f;
+#pragma unroll 4
+                for (int k = 0; k < parts; k++) {
+                    const float w = part_w[r * parts + k];
+                    load(j.f + (size_t)part_pos[r * parts + k] * j.ldf + i, p);
+#pragma unroll
+                    for (int e = 0; e < W; e++) m[e] = fmaf(w, p[e], m[e]);
+                }
+            } else {
+                load(j.f + (size_t)r * j.ldf + i, m);
+            }
+            load(gf + i, g);
+#pragma unroll
+            for (int e = 0; e < W; e++) v[e] = fmaf(sigmoidf(g[e]), m[e], v[e]);
+        }
+        if (again)
+#pragma unroll
+            for (int e = 0; e < W; e++) v[e] += widen(again[i + e]);
+        store(xr + i, v);
+        store(row + i, v);
+#pragma unroll
+        for (int e = 0; e < W; e++) ss = fmaf(v[e], v[e], ss);
+    }
+    if (!w_next) return;
+    const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)width + eps);
+    TO* o = out + (size_t)r * ldo;
+    for (int i = threadIdx.x * W; i < width; i += blockDim.x * W) {
+        float v[W], w[W];
+        load(row + i, v);
+        load(w_next + i, w);
+        TO n[W];
+#pragma unroll
+        for (int e = 0; e < W; e++) n[e] = narrow<TO>(v[e] * inv * w[e]);
+        if constexpr (W == 4 && sizeof(TO) == 2) {
+            uint2 q;
+            memcpy(&q, n, sizeof q);
+            *reinterpret_cast<uint2*>(o + i) = q;
+        } else if constexpr (W == 4) {
+            store(reinterpret_cast<float*>(o + i), reinterpret_cast<const float(&)[W]>(n));
+        } else {
+            o[i] = n[0];
+        }
+    }
+}
+
+// out[r] = norm of columns col .. col + n - 1 of row r, times w
+template <typename TO>
+__global__ void __launch_bounds__(256)
+norm_columns_kernel(const float* __restrict__ x, int ld, int col, int n, const float* __restrict__ w, float eps, TO* __restrict__ out, int ldo) {
+    __shared__ float red[32];
+    dep_wait();
+    dep_trigger();
+    const float* src = x + (size_t)blockIdx.x * ld + col;
+    const float inv = 1.0f / sqrtf(block_sum(square_share(src, n), red) / (float)n + eps);
+    for (int i = threadIdx.x; i < n; i += 256) out[(size_t)blockIdx.x * ldo + i] = narrow<TO>(src[i] * inv * w[i]);
+}
+
+__global__ void __launch_bounds__(256)
+act_rows_f32_kernel(const float* __restrict__ z, int ld, int ff, int act, float* __restrict__ f, int ldf) {
+    dep_wait();
+    dep_trigger();
+    for (int c = blockIdx.y * 256 + threadIdx.x; c < ff; c += gridDim.y * 256) f[(size_t)blockIdx.x * ldf + c] = unary_act(act, z[(size_t)blockIdx.x * ld + c]);
 }
 
 __global__ void __launch_bounds__(256)
@@ -565,6 +683,57 @@ extern "C" int cmlb200_stream_join(const cmlb200_streams* hc, float* d_x, const 
 #undef SJ_STREAMS
 #undef SJ_WIDTH
 #undef SJ_LAUNCH
+    return CMLB200_OK;
+}
+
+extern "C" int cmlb200_gated_join_rows(const cmlb200_gated_join* j, float* d_x, const float* d_w_next, float norm_eps, int rows, int width, void* d_out, int out_dtype, int ldo,
+                                       void* stream) {
+    static const char* who = "cmlb200_gated_join_rows";
+    CMLB_REQUIRE(j && d_x && rows > 0 && width > 0 && j->a && j->ga && j->ldm >= width && j->ldg >= width, "%s: bad argument", who);
+    CMLB_REQUIRE((!j->b || (j->a_norm && j->b_norm)) && (!j->f || (j->gf && j->ldf >= width)), "%s: norms or gates are missing", who);
+    CMLB_REQUIRE(!j->parts || (j->f && j->parts->top > 0 && j->parts->identity == 0 && j->parts->pos && j->parts->weight), "%s: parts without rows", who);
+    CMLB_REQUIRE(!j->table || (j->tokens && j->vocab > 0 && (j->table_dtype == CMLB200_DT_F32 || j->table_dtype == CMLB200_DT_BF16)), "%s: table without tokens", who);
+    CMLB_REQUIRE((out_dtype == CMLB200_DT_F32 || out_dtype == CMLB200_DT_BF16) && (!d_w_next || (d_out && ldo >= width)), "%s: no output for the normed rows", who);
+    const size_t smem = (size_t)((width + 3) / 4) * 16;
+    CMLB_REQUIRE(smem <= 200 * 1024, "%s: rows of %d elements do not fit shared memory", who, width);
+    const bool vec = width % 4 == 0 && j->ldm % 4 == 0 && j->ldg % 4 == 0 && (!j->f || j->ldf % 4 == 0) && (!d_w_next || ldo % 4 == 0) &&
+                     (((uintptr_t)d_x | (uintptr_t)d_w_next | (uintptr_t)d_out | (uintptr_t)j->a | (uintptr_t)j->b | (uintptr_t)j->a_norm | (uintptr_t)j->b_norm | (uintptr_t)j->f |
+                       (uintptr_t)j->ga | (uintptr_t)j->gf) & 15) == 0;
+    int threads = 256;
+    if (rows <= 2 * cmlb_num_sms()) while (threads < 1024 && threads * 4 < width) threads *= 2;
+    const cmlb200_moe* parts = j->parts;
+    static size_t attr[8][kMaxDevices] = {};
+#define GJ_LAUNCH(TO, TE, W, slot)                                                                                                    \
+    do {                                                                                                                              \
+        auto kern = gated_join_kernel<TO, TE, W>;                                                                                     \
+        CMLB_CUDA(cmlb_ensure_smem(kern, smem, attr[slot]));                                                                          \
+        CMLB_CUDA(launch_chain(kern, dim3(rows), dim3(threads), smem, 1, as_stream(stream), *j, parts ? parts->top : 0,               \
+                               (const int*)(parts ? parts->pos : nullptr), (const float*)(parts ? parts->weight : nullptr), d_x, d_w_next, norm_eps, width, (TO*)d_out, ldo)); \
+    } while (0)
+#define GJ_WIDTH(TO, TE, slot) do { if (vec) GJ_LAUNCH(TO, TE, 4, slot); else GJ_LAUNCH(TO, TE, 1, slot + 1); } while (0)
+#define GJ_TABLE(TO, slot) do { if (j->table && j->table_dtype == CMLB200_DT_F32) GJ_WIDTH(TO, float, slot); else GJ_WIDTH(TO, __nv_bfloat16, slot + 2); } while (0)
+    if (out_dtype == CMLB200_DT_BF16) GJ_TABLE(__nv_bfloat16, 0);
+    else GJ_TABLE(float, 4);
+#undef GJ_TABLE
+#undef GJ_WIDTH
+#undef GJ_LAUNCH
+    return CMLB200_OK;
+}
+
+extern "C" int cmlb200_norm_columns(const float* d_x, int ld, int col, int n, const float* d_w, float eps, int rows, void* d_out, int out_dtype, int ldo, void* stream) {
+    CMLB_REQUIRE(d_x && d_w && d_out && col >= 0 && n > 0 && rows > 0 && ld >= col + n && ldo >= n, "cmlb200_norm_columns: bad argument");
+    CMLB_REQUIRE(out_dtype == CMLB200_DT_F32 || out_dtype == CMLB200_DT_BF16, "cmlb200_norm_columns: dtype %d", out_dtype);
+#define NC_LAUNCH(TO) CMLB_CUDA(launch_chain(norm_columns_kernel<TO>, dim3(rows), dim3(256), 0, 1, as_stream(stream), d_x, ld, col, n, d_w, eps, (TO*)d_out, ldo))
+    if (out_dtype == CMLB200_DT_BF16) NC_LAUNCH(__nv_bfloat16);
+    else NC_LAUNCH(float);
+#undef NC_LAUNCH
+    return CMLB200_OK;
+}
+
+extern "C" int cmlb200_act_rows_f32(const float* d_z, int ld, int rows, int ff, int act, float* d_f, int ldf, void* stream) {
+    CMLB_REQUIRE(d_z && d_f && rows > 0 && ff > 0 && ld >= ff && ldf >= ff, "cmlb200_act_rows_f32: bad argument");
+    CMLB_REQUIRE(act == CMLB200_ACT_SILU || act == CMLB200_ACT_GELU_TANH || act == CMLB200_ACT_GELU_ERF, "cmlb200_act_rows_f32: activation %d", act);
+    CMLB_CUDA(launch_chain(act_rows_f32_kernel, dim3(rows, (ff + 1023) / 1024), dim3(256), 0, 1, as_stream(stream), d_z, ld, ff, act, d_f, ldf));
     return CMLB200_OK;
 }
 

@@ -94,12 +94,15 @@ __device__ __forceinline__ float gelu_tanh(float z) {
 }
 __device__ __forceinline__ float silu(float z) { return z / (1.0f + expf(-z)); }
 __device__ __forceinline__ float sigmoidf(float z) { return 1.0f / (1.0f + expf(-z)); }
+// 0.5 z (1 + erf(z / sqrt(2)))
+__device__ __forceinline__ float gelu_erf(float z) { return 0.5f * z * (1.0f + erff(0.7071067811865476f * z)); }
+__device__ __forceinline__ float unary_act(int act, float z) { return act == CMLB200_ACT_GELU_ERF ? gelu_erf(z) : (act == CMLB200_ACT_GELU_TANH ? gelu_tanh(z) : silu(z)); }
 __device__ __forceinline__ float glu_act(int act, float g, float u, float limit = 0.f) {
     if (act == CMLB200_ACT_CLAMPED) {
         g = fminf(g, limit);
         return g * sigmoidf(1.702f * g) * (fminf(fmaxf(u, -limit), limit) + 1.0f);
     }
-    return (act == CMLB200_ACT_GELU_TANH ? gelu_tanh(g) : silu(g)) * u;
+    return unary_act(act, g) * u;
 }
 
 // The same for results that are rounded to bf16: hardware exponential and reciprocal without branches, so that
@@ -111,6 +114,12 @@ __device__ __forceinline__ float glu_act_fast(int act, float g, float u, float l
     u = clamped ? fminf(fmaxf(u, -limit), limit) + 1.0f : u;
     const float gelu = 1.5957691216057308f * (g + 0.044715f * g * g * g);
     return g * sigmoid_fast(clamped ? 1.702f * g : (act == CMLB200_ACT_GELU_TANH ? gelu : g)) * u;
+}
+
+// act: CMLB200_ACT_SILU, _GELU_TANH or _GELU_ERF
+__device__ __forceinline__ float unary_act_fast(int act, float z) {
+    if (act == CMLB200_ACT_GELU_ERF) return gelu_erf(z);
+    return z * sigmoid_fast(act == CMLB200_ACT_GELU_TANH ? 1.5957691216057308f * (z + 0.044715f * z * z * z) : z);
 }
 
 __device__ __forceinline__ float soft_cap(float v, float cap) { return cap * tanhf(v / cap); }

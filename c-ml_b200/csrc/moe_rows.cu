@@ -24,20 +24,23 @@ __host__ __device__ inline int route_floats(const cmlb200_moe& m) {
     return n + (m.correction ? n : 0) + 2 * m.groups;
 }
 
-// One warp, one row: softmax over all outputs, then `top` times the largest that is left. With a correction the choice
-// is by score + correction, otherwise by the logits themselves, which have the scores' order.
+// One warp, one row: softmax over all outputs, or their sigmoids, then `top` times the largest that is left. With a correction the choice
+// is by score + correction, otherwise by the sigmoids or by the logits themselves, which have the softmax's order.
 __device__ __forceinline__ void route_row(const cmlb200_moe& m, const float* __restrict__ logits, int r, float* z) {
     const int lane = threadIdx.x & 31, n = m.experts + m.identity;
-    float* score = m.correction ? z + n : z;                            // without a correction: still logits
-    float mx = -INFINITY;
-    for (int e = lane; e < n; e += 32) { const float v = logits[e]; z[e] = v; mx = fmaxf(mx, v); }
-    mx = lane_max(mx);
-    float sum = 0.f;
-    for (int e = lane; e < n; e += 32) sum += expf(z[e] - mx);
-    sum = lane_sum(sum);
+    float* score = m.correction ? z + n : z;                            // without a correction: sigmoids, or still logits
+    float mx = -INFINITY, sum = 0.f;
+    if (m.sigmoid) {
+        for (int e = lane; e < n; e += 32) z[e] = sigmoidf(logits[e]);
+    } else {
+        for (int e = lane; e < n; e += 32) { const float v = logits[e]; z[e] = v; mx = fmaxf(mx, v); }
+        mx = lane_max(mx);
+        for (int e = lane; e < n; e += 32) sum += expf(z[e] - mx);
+        sum = lane_sum(sum);
+    }
     if (m.correction) {
         for (int e = lane; e < n; e += 32) {
-            score[e] = expf(z[e] - mx) / sum;
+            score[e] = m.sigmoid ? z[e] : expf(z[e] - mx) / sum;
             z[e] = score[e] + m.correction[e];
         }
     }
@@ -46,9 +49,13 @@ __device__ __forceinline__ void route_row(const cmlb200_moe& m, const float* __r
         const int per = n / m.groups;
         __syncwarp();
         for (int g = lane; g < m.groups; g += 32) {
-            best[g] = -INFINITY;
+            float one = -INFINITY, two = -INFINITY;
+            for (int e = g * per; e < (g + 1) * per; e++) {
+                two = fmaxf(two, fminf(one, z[e]));
+                one = fmaxf(one, z[e]);
+            }
+            best[g] = m.group_best == 2 && per > 1 ? one + two : one;
             open[g] = 0.f;
-            for (int e = g * per; e < (g + 1) * per; e++) best[g] = fmaxf(best[g], z[e]);
         }
         for (int k = 0; k < m.keep; k++) {
             const int win = warp_arg_max(best, m.groups);
@@ -63,7 +70,7 @@ __device__ __forceinline__ void route_row(const cmlb200_moe& m, const float* __r
         const int win = warp_arg_max(z, n);
         float w = 0.f;
         if (lane == (win & 31)) {
-            w = m.correction ? score[win] : expf(z[win] - mx) / sum;
+            w = m.correction || m.sigmoid ? score[win] : expf(z[win] - mx) / sum;
             m.ids[r * m.top + k] = win;
             m.weight[r * m.top + k] = w;
             z[win] = -INFINITY;
@@ -188,6 +195,7 @@ extern "C" int cmlb200_moe_route(const cmlb200_moe* m, const float* d_logits, in
     CMLB_REQUIRE(m->top <= outputs && ld >= outputs && (m->identity == 0 || m->self), "cmlb200_moe_route: %d of %d outputs, stride %d", m->top, outputs, ld);
     CMLB_REQUIRE(m->groups == 0 || (m->groups > 0 && outputs % m->groups == 0 && m->keep > 0 && m->keep <= m->groups && m->keep * (outputs / m->groups) >= m->top),
                  "cmlb200_moe_route: %d of %d groups of %d outputs for %d", m->keep, m->groups, outputs, m->top);
+    CMLB_REQUIRE(m->group_best >= 0 && m->group_best <= 2, "cmlb200_moe_route: groups by their %d largest", m->group_best);
     CMLB_REQUIRE(m->ids && m->weight && m->pos && m->src && m->expert && m->start && m->count && m->active && m->num_active && m->num_tiles, "cmlb200_moe_route: a plan without arrays");
     CMLB_REQUIRE(outputs <= 1536 && (long)rows * m->top < (1l << 30), "cmlb200_moe_route: %d experts", m->experts);
     cudaStream_t st = as_stream(stream);

@@ -37,24 +37,6 @@ int cml_delta_ranks(const CMLSafetensors* st, const char* prefix, Layer* l, int 
     return 0;
 }
 
-/* [taps][channels] from three tensors [channels, taps] */
-static int load_taps(const CMLSafetensors* st, const char* prefix, const cmlb200_delta* a, float** dst) {
-    static const char* const names[3] = {"mix.right.q.conv", "mix.right.k.conv", "mix.right.v.conv"};
-    const int n[3] = {a->kv_heads * a->dim, a->kv_heads * a->dim, a->heads * a->vdim}, channels = channels_of(a);
-    float* v = (float*)malloc((size_t)channels * (size_t)a->taps * sizeof(float));
-    if (!v) return -1;
-    int at = 0, rc = 0;
-    for (int p = 0; p < 3 && !rc; at += n[p++]) {
-        CMLSafetensor t;
-        rc = lml_find(st, prefix, names[p], n[p], a->taps, &t);
-        for (int c = 0; c < n[p] && !rc; c++)
-            for (int k = 0; k < a->taps; k++) v[(size_t)k * (size_t)channels + (size_t)(at + c)] = lml_element(&t, (size_t)c * (size_t)a->taps + (size_t)k);
-    }
-    rc = rc || lml_upload((void**)dst, v, (size_t)channels * (size_t)a->taps * sizeof(float));
-    free(v);
-    return rc ? -1 : 0;
-}
-
 static int load_rates(const CMLSafetensors* st, const char* prefix, int heads, float** dst) {
     CMLSafetensor t;
     if (lml_find(st, prefix, "mix.right.A_log", heads, 0, &t)) return -1;
@@ -70,8 +52,9 @@ int cml_delta_load(Layered* m, const CMLSafetensors* st, const char* prefix, Lay
     const cmlb200_delta* a = &l->delta;
     LayerWeights* w = &l->w;
     const char *a2[1] = {"mix.right.a2"}, *g2[1] = {"mix.right.g2"};
-    const int decays[1] = {a->heads * a->dim}, gates[1] = {a->heads * a->vdim};
-    return load_taps(st, prefix, a, &w->conv) || load_rates(st, prefix, a->heads, &w->rate) ||
+    static const char* const taps[3] = {"mix.right.q.conv", "mix.right.k.conv", "mix.right.v.conv"};
+    const int decays[1] = {a->heads * a->dim}, gates[1] = {a->heads * a->vdim}, channels[3] = {a->kv_heads * a->dim, a->kv_heads * a->dim, a->heads * a->vdim};
+    return lml_load_taps(st, prefix, taps, channels, 3, a->taps, &w->conv) || load_rates(st, prefix, a->heads, &w->rate) ||
            lml_load_vector(st, prefix, "mix.right.dt_bias", decays[0], 0.f, &w->dt_bias) || lml_load_vector(st, prefix, "mix.right.norm", a->vdim, 0.f, &w->o_norm) ||
            lml_load_matrix(m, st, prefix, a2, decays, 1, l->a_rank, 0, &w->wa) || lml_load_matrix(m, st, prefix, g2, gates, 1, l->g_rank, 0, &w->wg) ? -1 : 0;
 }
@@ -81,7 +64,7 @@ int cml_delta_activations(Layered* m, int rows) {
     long work = 0;
     for (int i = 0; i < m->num_layers; i++) {
         const Layer *l = &m->layers[i], *s = &m->layers[l->source];
-        if (l->kind->form != MIXER_PARALLEL) continue;
+        if (l->kind->form != MIXER_PARALLEL || l->kind->beside != BESIDE_DELTA) continue;
         dec = lml_most(dec, l->delta.heads * l->delta.dim);
         gate = lml_most(gate, l->delta.heads * l->delta.vdim);
         low = lml_most(low, lml_round_up(s->a_rank, 64) + lml_round_up(s->g_rank, 64));

@@ -2,24 +2,29 @@
  * of switches (LayeredDesign); sizes, windows, scales and the order of layers come from the file.
  *
  *   config.json     architecture, vocab, width, norm.eps, layers: [{type, mixer, mlp, weights_of?}]; designs with streams also
- *                   streams, embedding.scale and logit_softcap
- *   mixer           grouped heads: heads, kv_heads, dim, vdim, scale, mask {size, keep_first}, q_temp {coef, every}
- *                   latents: heads, dim, rot_dim, vdim, kv_rank, scale, mask.size, rot {base, dims, scaling {factor,
+ *                   streams, embedding.scale and logit_softcap; designs with loops also loop {start, stop, times}
+ *   mixer           grouped heads: heads, kv_heads, dim, vdim, scale, mask {size, keep_first}, q_temp {coef, every}, rot {base, dims,
+ *                   scaling {factor}, or {factor, low, high, original}}, and what cml_lm_talk.c says
+ *                   latents: heads, dim, rot_dim, vdim, q_rank, kv_rank, scale, mask.size, rot {base, dims, scaling {factor,
  *                   original, fast, slow}}, kv_from (the layer whose cache this one reads)
- *                   parallel: left (grouped heads), right (gated delta rule, cml_lm_delta.c), left_scale, right_scale
+ *                   parallel: left (grouped heads), right (gated delta rule, cml_lm_delta.c, with left_scale and right_scale; or
+ *                   minimal gated recurrence, cml_lm_gru.c)
  *   mlp             {kind: "dense", ff}, {kind: "moe", expert {ff, limit}, router {experts, top, identity, groups {count, keep},
  *                   scale}, shared {ff}} or null
  *   weights_of      index of the layer whose tensors this one uses; its cache is its own
  *   tensors         embed, final.norm, head, l<i>.norm1 / norm1b / norm2 / norm2b (as the design has them),
  *                   l<i>.mix.q / k / v / g / o / q.norm / k.norm / sink and biases .b, the same under mix.left and mix.right, or
- *                   q / dkv / dkv.norm / uk / uv / g / o, l<i>.mlp.gate / up / down, up / down / act, or router, correction,
- *                   e<j>.gate / up / down and shared.gate / up / down, l<i>.hc1 / hc2 .in / out / mix; linear weights [out, in]
+ *                   q (or dq / dq.norm / uq) / dkv / dkv.norm / uk / uv / sink / g / o, l<i>.mlp.gate / up / down, up / down / act, or
+ *                   router, correction, e<j>.gate / up / down and shared.gate / up / down, l<i>.hc1 / hc2 .in / out / mix, l<i>.rg1 /
+ *                   rg2 and biases; linear weights [out, in]
  *
  * On the device all of a layer's projections of its input are one matrix, and the feed-forward's gate and up rows one
  * matrix interleaved in groups of 16 (the epilogues of both products pair them). Two mixers side by side leave their
- * outputs, scaled, in neighbouring columns, which one output matrix takes. Between two sublayers runs
- * one kernel: norm of the finished sublayer's output, residual add, norm for the next one; with streams, the join into
- * all of them, what the next sublayer reads, and its norm. The residual, norms,
+ * outputs, scaled, in neighbouring columns, which one output matrix takes, unless their outputs are normed one by one. Between two
+ * sublayers runs one kernel: norm of the finished sublayer's output, residual add, norm for the next one; with streams, the
+ * join into all of them, what the next sublayer reads, and its norm. Where both sublayers read the same row, the gates' and
+ * the router's rows belong to the layer's one projection too, and one kernel joins both. A layer that runs several times
+ * has an entry for every pass, with a cache of its own and the first pass's weights. The residual, norms,
  * scores and weights are fp32; in the bfloat16 form matrix operands are bf16 and cached keys, values and latents
  * fp16. Up to 32 rows a step streams its weights through the decode product, above that tcgen05 tiles.
  *
@@ -38,21 +43,40 @@
 
 static const LayeredDesign kDesigns[] = {
     {.architecture = "Rarolorn",
-     .mixers = {{"attention", MIXER_GROUPED, 0, {.norm = NORM_WIDE, .sink = SINK_ONE, .linear_bias = 1, .head_gate = 1}}},
+     .mixers = {{.type = "attention", .form = MIXER_GROUPED, .grouped = {.norm = NORM_WIDE, .sink = SINK_ONE, .linear_bias = 1, .head_gate = 1}}},
      .position_base = 10000.0, .input_norms = 1, .output_norms = {"norm1b", "norm2b"}, .dense = FF_GATED, .act = CMLB200_ACT_GELU_TANH},
     {.architecture = "Situlorn",
-     .mixers = {{.type = "latent_attention", .form = MIXER_LATENT}, {.type = "latent_attention_2", .form = MIXER_LATENT, .wide_gate = 1}},
+     .mixers = {{.type = "latent_attention", .form = MIXER_LATENT}, {.type = "latent_attention_2", .form = MIXER_LATENT, .gate = GATE_WIDE}},
      .output_norms = {"norm1", "norm2"}, .dense = FF_POLY_NORM, .act = CMLB200_ACT_CLAMPED, .experts = EXPERTS_PLAIN},
     {.architecture = "Lenedra",
-     .mixers = {{"attention", MIXER_GROUPED, 0, {.norm = NORM_HEAD, .linear_bias = 1, .in_bias = 1, .out_bias = 1, .keys_as_values = 1}},
-                {"parallel", MIXER_PARALLEL, 0, {.sink = SINK_LEARNED, .chunked = 1, .in_bias = 1}}},
+     .mixers = {{.type = "attention", .form = MIXER_GROUPED,
+                 .grouped = {.norm = NORM_HEAD, .linear_bias = 1, .in_bias = 1, .out_bias = 1, .keys_as_values = 1}},
+                {.type = "parallel", .form = MIXER_PARALLEL, .beside = BESIDE_DELTA, .grouped = {.sink = SINK_LEARNED, .chunked = 1, .in_bias = 1}}},
      .input_norms = 1, .norm_offset = 1.f, .streams = 1, .dense = FF_GATED, .act = CMLB200_ACT_SILU, .experts = EXPERTS_GROUPED},
+    {.architecture = "Zevilorn",
+     .mixers = {{.type = "attention", .form = MIXER_GROUPED,
+                 .grouped = {.sink = SINK_ONE, .in_bias = 1, .out_bias = 1, .rotate = ROTATE_BANDS, .conv = 1, .talk = 1}},
+                {.type = "latent_attention", .form = MIXER_LATENT, .gate = GATE_HEAD, .q_latent = 1, .sink = SINK_LEARNED},
+                {.type = "parallel", .form = MIXER_PARALLEL, .beside = BESIDE_GRU, .grouped = {.head_gate = 1, .rotate = ROTATE_LINEAR}}},
+     .input_norms = 1, .side_by_side = 1, .loops = 1, .act = CMLB200_ACT_GELU_ERF, .experts = EXPERTS_SIGMOID},
 };
 
 /* ---- configuration ---------------------------------------------------------------------------------- */
 static int is_object(const CMLJson* j) { return j && j->type == CML_JSON_OBJECT; }
 
 static int grouped_columns(const cmlb200_attn* a) { return a->heads * a->dim + a->kv_heads * (a->dim + (a->keys_as_values ? 0 : a->vdim)); }
+
+/* Rotated dimensions and what scales their frequencies: the constants' names in `keys` (the first is a factor). */
+static int read_rotation(const CMLJson* mixer, Layer* l, const char* const* keys, int count, int* dims, int index) {
+    const CMLJson *rot = cml_json_get(mixer, "rot"), *scaling = cml_json_get(rot, "scaling");
+    if (cml_json_double(rot, "base", &l->rot_base) || cml_json_int(rot, "dims", dims) || *dims <= 0 || *dims % 2 || l->rot_base <= 0.0 || l->rot_base == 1.0) {
+        LOG_ERROR("layer %d: rot.base or rot.dims is missing or does not fit", index);
+        return -1;
+    }
+    for (int k = 0; is_object(scaling) && k < count; k++)
+        if (cml_json_double(scaling, keys[k], &l->rot_scaling[k]) || l->rot_scaling[k] <= 0.0) { LOG_ERROR("layer %d: rot.scaling.%s", index, keys[k]); return -1; }
+    return 0;
+}
 
 static int read_grouped(const CMLJson* mixer, Layer* l, int index) {
     const GroupedForm* form = &l->kind->grouped;
@@ -79,11 +103,16 @@ static int read_grouped(const CMLJson* mixer, Layer* l, int index) {
     a->keys_as_values = form->keys_as_values;
     a->head_norm = form->norm == NORM_HEAD;
     a->gate_col = form->head_gate ? grouped_columns(a) : -1;
-    return 0;
+    if (form->rotate != ROTATE_NONE) {
+        static const char* const keys[4] = {"factor", "original", "low", "high"};
+        if (read_rotation(mixer, l, keys, form->rotate == ROTATE_BANDS ? 4 : 1, &a->rot_dims, index)) return -1;
+        if (a->rot_dims > a->dim || (l->rot_scaling[3] > 0.0 && l->rot_scaling[3] <= l->rot_scaling[2])) { LOG_ERROR("layer %d: rot.dims or rot.scaling.high", index); return -1; }
+    }
+    return form->conv || form->talk ? cml_talk_read(mixer, l, index) : 0;
 }
 
 static int read_latent(const CMLJson* mixer, Layer* l, int index) {
-    const CMLJson *mask = cml_json_get(mixer, "mask"), *rot = cml_json_get(mixer, "rot"), *scaling = cml_json_get(rot, "scaling");
+    const CMLJson* mask = cml_json_get(mixer, "mask");
     static const char* const keys[4] = {"factor", "original", "fast", "slow"};
     cmlb200_latent* a = &l->lat;
     double scale = 0.0;
@@ -96,25 +125,26 @@ static int read_latent(const CMLJson* mixer, Layer* l, int index) {
         return -1;
     }
     if (is_object(mask) && (cml_json_int(mask, "size", &a->window) || a->window <= 0)) { LOG_ERROR("layer %d: mask.size", index); return -1; }
-    if (cml_json_double(rot, "base", &l->rot_base) || cml_json_int(rot, "dims", &dims) || dims != a->rot_dim || l->rot_base <= 0.0 || l->rot_base == 1.0) {
-        LOG_ERROR("layer %d: rot.base is missing or rot.dims is not rot_dim", index);
-        return -1;
-    }
-    if (is_object(scaling))
-        for (int k = 0; k < 4; k++)
-            if (cml_json_double(scaling, keys[k], &l->rot_scaling[k]) || l->rot_scaling[k] <= 0.0) { LOG_ERROR("layer %d: rot.scaling.%s", index, keys[k]); return -1; }
+    if (read_rotation(mixer, l, keys, 4, &dims, index)) return -1;
+    if (dims != a->rot_dim) { LOG_ERROR("layer %d: rot.dims is not rot_dim", index); return -1; }
+    if (l->kind->q_latent && (cml_json_int(mixer, "q_rank", &l->q_rank) || l->q_rank <= 0)) { LOG_ERROR("layer %d: q_rank", index); return -1; }
     const CMLJson* from = cml_json_get(mixer, "kv_from");
     if (from && from->type != CML_JSON_NULL && cml_json_int(mixer, "kv_from", &l->kv_from)) { LOG_ERROR("layer %d: kv_from", index); return -1; }
-    const int q = a->heads * (a->dim + a->rot_dim), kv = a->rank + a->rot_dim;
+    /* queries out of a latent of their own land in front of the projection, which then begins with that latent */
+    l->proj_col = l->kind->q_latent ? lml_round_up(a->heads * (a->dim + a->rot_dim), 16) : 0;
+    const int q = l->kind->q_latent ? l->proj_col + l->q_rank : a->heads * (a->dim + a->rot_dim), kv = a->rank + a->rot_dim;
     a->scale = (float)scale;
     a->ld = lml_round_up(kv, 16);
     a->ld_rank = lml_round_up(a->rank, 64);
     a->kv_col = l->kv_from == index ? q : -1;
-    a->gate_col = l->kind->wide_gate ? q + (l->kv_from == index ? kv : 0) : -1;
+    a->gate_col = l->kind->gate != GATE_NONE ? q + (l->kv_from == index ? kv : 0) : -1;
+    a->gate_heads = l->kind->gate == GATE_HEAD;
     return 0;
 }
 
 static int read_parallel(const CMLJson* mixer, Layer* l, int index) {
+    if (l->kind->beside == BESIDE_GRU)
+        return read_grouped(cml_json_get(mixer, "left"), l, index) || cml_gru_read(cml_json_get(mixer, "right"), l, index) ? -1 : 0;
     double left = 0.0, right = 0.0;
     if (cml_json_double(mixer, "left_scale", &left) || cml_json_double(mixer, "right_scale", &right) || left == 0.0 || right == 0.0) {
         LOG_ERROR("layer %d: left_scale or right_scale is missing or 0", index);
@@ -128,7 +158,7 @@ static int read_parallel(const CMLJson* mixer, Layer* l, int index) {
 
 static int read_feed_forward(const CMLJson* mlp, Layer* l, int index, const LayeredDesign* design) {
     const char* kind = cml_json_string(mlp, "kind");
-    if (kind && !strcmp(kind, "dense") && !cml_json_int(mlp, "ff", &l->ff) && l->ff > 0) return 0;
+    if (kind && !strcmp(kind, "dense") && !design->side_by_side && !cml_json_int(mlp, "ff", &l->ff) && l->ff > 0) return 0;
     const CMLJson *expert = cml_json_get(mlp, "expert"), *router = cml_json_get(mlp, "router"), *groups = cml_json_get(router, "groups");
     const CMLJson* shared = cml_json_get(mlp, "shared");
     double limit = 0.0, scale = 1.0;
@@ -139,14 +169,16 @@ static int read_feed_forward(const CMLJson* mlp, Layer* l, int index, const Laye
         return -1;
     }
     l->limit = (float)limit;
-    if (design->experts == EXPERTS_GROUPED) {
-        cml_json_int(router, "identity", &l->identity);
-        cml_json_double(router, "scale", &scale);
+    if (design->experts >= EXPERTS_GROUPED) {
+        if (design->experts == EXPERTS_GROUPED) {
+            cml_json_int(router, "identity", &l->identity);
+            cml_json_double(router, "scale", &scale);
+        }
         l->router_scale = (float)scale;
         const int all = l->experts + l->identity;
         if (l->identity < 0 || l->identity > 1024 || (is_object(groups) && (cml_json_int(groups, "count", &l->groups) || cml_json_int(groups, "keep", &l->keep) || l->groups <= 0 ||
             all % l->groups || l->keep <= 0 || l->keep > l->groups || (long)l->keep * (all / l->groups) < l->top)) ||
-            (is_object(shared) && (cml_json_int(shared, "ff", &l->shared_ff) || l->shared_ff <= 0))) {
+            (design->experts == EXPERTS_GROUPED && is_object(shared) && (cml_json_int(shared, "ff", &l->shared_ff) || l->shared_ff <= 0))) {
             LOG_ERROR("layer %d: router.identity, router.groups or shared.ff does not fit", index);
             return -1;
         }
@@ -155,16 +187,36 @@ static int read_feed_forward(const CMLJson* mlp, Layer* l, int index, const Laye
     return 0;
 }
 
-static int read_layer(const CMLJson* j, Layer* l, int index, const LayeredDesign* design) {
+/* Columns of a side-by-side layer's projection behind its mixer's own: the sublayers' gates (which the join reads four columns at a
+ * time), the gates of heads, the router's logits. */
+static void place_gates(Layer* l, int width) {
+    const int latent = l->kind->form == MIXER_LATENT;
+    int col = !latent ? grouped_columns(&l->attn) : (l->lat.kv_col >= 0 ? l->lat.kv_col + l->lat.rank + l->lat.rot_dim : l->proj_col + l->q_rank);
+    if (l->kind->form == MIXER_PARALLEL) {
+        l->gru.col = col;
+        col += 3 * l->gru.width;
+    }
+    l->gate_cols = col;
+    col += (l->ff ? 2 : 1) * width;
+    int* heads = latent ? &l->lat.gate_col : &l->attn.gate_col;
+    if (*heads >= 0) {
+        *heads = col;
+        col += latent ? l->lat.heads : l->attn.heads;
+    }
+    l->router_col = col;
+}
+
+static int read_layer(const CMLJson* j, Layer* l, int index, int width, const LayeredDesign* design) {
     const CMLJson *mixer = cml_json_get(j, "mixer"), *mlp = cml_json_get(j, "mlp");
     const char* type = cml_json_string(j, "type");
     for (size_t k = 0; k < sizeof design->mixers / sizeof design->mixers[0]; k++)
         if (type && design->mixers[k].type && !strcmp(type, design->mixers[k].type)) l->kind = &design->mixers[k];
     if (!l->kind) { LOG_ERROR("layer %d: mixer type '%s' is not known to %s", index, type ? type : "(none)", design->architecture); return -1; }
-    l->kv_from = index;
+    l->index = l->kv_from = index;
     if (l->kind->form == MIXER_LATENT ? read_latent(mixer, l, index) : (l->kind->form == MIXER_PARALLEL ? read_parallel(mixer, l, index) : read_grouped(mixer, l, index)))
         return -1;
     if (is_object(mlp) && read_feed_forward(mlp, l, index, design)) return -1;
+    if (design->side_by_side) place_gates(l, width);
     l->source = index;
     int of;
     if (!cml_json_int(j, "weights_of", &of)) l->source = of;
@@ -179,6 +231,7 @@ static int window_of(const Layer* l) {
 
 static int same_shape(const Layer* a, const Layer* b) {
     if (a->kind != b->kind || a->ff != b->ff || a->experts != b->experts || a->identity != b->identity || a->shared_ff != b->shared_ff) return 0;
+    if (a->q_rank != b->q_rank || a->gru.width != b->gru.width || a->attn.taps != b->attn.taps) return 0;
     if (a->kind->form == MIXER_PARALLEL && (a->delta.heads != b->delta.heads || a->delta.kv_heads != b->delta.kv_heads || a->delta.dim != b->delta.dim ||
                                             a->delta.vdim != b->delta.vdim || a->delta.taps != b->delta.taps))
         return 0;
@@ -217,12 +270,31 @@ static int read_config(const CMLJson* c, Layered* m) {
         m->embed_scale = (float)scale;
         m->cap = (float)cap;
     }
-    m->num_layers = layers->count;
+    int start = 0, stop = 0, times = 1;
+    const CMLJson* loop = m->design->loops ? cml_json_get(c, "loop") : NULL;
+    if (is_object(loop) && (cml_json_int(loop, "start", &start) || cml_json_int(loop, "stop", &stop) || cml_json_int(loop, "times", &times) || start < 0 || stop < start ||
+                            stop > layers->count || times < 1 || (long)times * (stop - start) > MAX_LAYERS)) {
+        LOG_ERROR("config.json: loop does not fit %d layers", layers->count);
+        return -1;
+    }
+    const int span = stop - start, more = (times - 1) * span;
+    m->num_layers = layers->count + more;
     m->layers = (Layer*)calloc((size_t)m->num_layers, sizeof(Layer));
     if (!m->layers) return -1;
     int i = 0;
-    for (const CMLJson* j = layers->child; j; j = j->next, i++)
-        if (read_layer(j, &m->layers[i], i, m->design)) return -1;
+    for (const CMLJson* j = layers->child; j; j = j->next, i++) {
+        Layer* l = &m->layers[i < stop ? i : i + more];
+        if (read_layer(j, l, i, m->width, m->design)) return -1;
+        /* from the places in config.json to the first passes over them */
+        if (l->source >= stop) l->source += more;
+        if (l->kv_from >= stop) l->kv_from += more;
+    }
+    for (i = stop; i < stop + more; i++) {                 /* further passes */
+        m->layers[i] = m->layers[i - span];
+        m->layers[i].again = m->layers[i].index == start;
+        m->layers[i].source = start + (i - start) % span;
+        if (m->layers[i].kv_from == i - span) m->layers[i].kv_from = i;
+    }
     for (i = 0; i < m->num_layers; i++) {                  /* follow chains of weights_of to the layer that has tensors */
         int s = m->layers[i].source, hops = 0;
         while (s >= 0 && s < m->num_layers && m->layers[s].source != s && hops++ < m->num_layers) s = m->layers[s].source;
@@ -271,29 +343,40 @@ int lml_upload(void** dst, const void* src, size_t bytes) {
     return 0;
 }
 
-/* Frequencies of the rotated pairs and the factor on sine and cosine. With scaling, the pairs that turn fewer than `slow`
- * times within `original` positions are slowed down by the factor, those that turn more than `fast` times are not, and a
- * ramp over the pairs lies between. */
+/* Frequencies of the rotated pairs of grouped heads: all divided by a factor, or by where 2 pi / f lies between two shares of
+ * `original`: short wavelengths stay, long ones are stretched by the factor, a ramp in original / wavelength lies between. */
+static double grouped_frequency(const Layer* l, double f) {
+    const double *s = l->rot_scaling, turns = s[1] * f / 6.283185307179586476925;
+    if (s[0] <= 0.0) return f;
+    if (l->kind->grouped.rotate == ROTATE_LINEAR) return f / s[0];
+    const double keep = fmin(fmax((turns - s[2]) / (s[3] - s[2]), 0.0), 1.0);
+    return keep < 1.0 ? (1.0 - keep) * f / s[0] + keep * f : f;
+}
+
+/* Frequencies of the rotated pairs, for latents with the factor on sine and cosine. With scaling, the pairs of a latent layer
+ * that turn fewer than `slow` times within `original` positions are slowed down by the factor, those that turn more than
+ * `fast` times are not, and a ramp over the pairs lies between. */
 static int make_rotation(Layer* l) {
-    cmlb200_latent* a = &l->lat;
-    const double n = a->rot_dim, *s = l->rot_scaling;
-    float* f = (float*)malloc((size_t)(a->rot_dim / 2) * sizeof(float));
+    const int latent = l->kind->form == MIXER_LATENT, dims = latent ? l->lat.rot_dim : l->attn.rot_dims;
+    if (!dims) return 0;
+    const double n = dims, *s = l->rot_scaling;
+    float* f = (float*)malloc((size_t)(dims / 2) * sizeof(float));
     if (!f) return -1;
     double lo = 0.0, hi = 0.0;
-    if (s[0] > 0.0) {
+    if (latent && s[0] > 0.0) {
         const double two_pi = 6.283185307179586476925;
         lo = fmax(floor(n * log(s[1] / (two_pi * s[2])) / (2.0 * log(l->rot_base))), 0.0);
         hi = fmin(ceil(n * log(s[1] / (two_pi * s[3])) / (2.0 * log(l->rot_base))), n - 1.0);
     }
-    for (int i = 0; i < a->rot_dim / 2; i++) {
+    for (int i = 0; i < dims / 2; i++) {
         const double plain = pow(l->rot_base, -2.0 * i / n);
-        const double ramp = s[0] > 0.0 ? fmin(fmax((i - lo) / fmax(hi - lo, 0.001), 0.0), 1.0) : 0.0;
-        f[i] = (float)(ramp > 0.0 ? plain / s[0] * ramp + plain * (1.0 - ramp) : plain);
+        const double ramp = latent && s[0] > 0.0 ? fmin(fmax((i - lo) / fmax(hi - lo, 0.001), 0.0), 1.0) : 0.0;
+        f[i] = (float)(latent ? (ramp > 0.0 ? plain / s[0] * ramp + plain * (1.0 - ramp) : plain) : grouped_frequency(l, plain));
     }
-    a->rot_mul = s[0] > 0.0 ? (float)(0.1 * log(s[0]) + 1.0) : 1.0f;
-    const int rc = lml_upload((void**)&l->freq, f, (size_t)(a->rot_dim / 2) * sizeof(float));
+    const int rc = lml_upload((void**)&l->freq, f, (size_t)(dims / 2) * sizeof(float));
     free(f);
-    a->freq = l->freq;
+    l->attn.freq = l->lat.freq = l->freq;
+    l->lat.rot_mul = latent && s[0] > 0.0 ? (float)(0.1 * log(s[0]) + 1.0) : 1.0f;
     return rc;
 }
 
@@ -306,6 +389,22 @@ int lml_load_vector(const CMLSafetensors* st, const char* prefix, const char* na
     const int rc = lml_upload((void**)dst, v, (size_t)n * sizeof(float));
     free(v);
     return rc;
+}
+
+int lml_load_taps(const CMLSafetensors* st, const char* prefix, const char* const* names, const int* channels, int parts, int taps, float** dst) {
+    int all = 0, at = 0, rc = 0;
+    for (int p = 0; p < parts; p++) all += channels[p];
+    float* v = (float*)malloc((size_t)all * (size_t)taps * sizeof(float));
+    if (!v) return -1;
+    for (int p = 0; p < parts && !rc; at += channels[p++]) {
+        CMLSafetensor t;
+        rc = lml_find(st, prefix, names[p], channels[p], taps, &t);
+        for (int c = 0; c < channels[p] && !rc; c++)
+            for (int k = 0; k < taps; k++) v[(size_t)k * (size_t)all + (size_t)(at + c)] = lml_element(&t, (size_t)c * (size_t)taps + (size_t)k);
+    }
+    rc = rc || lml_upload((void**)dst, v, (size_t)all * (size_t)taps * sizeof(float));
+    free(v);
+    return rc ? -1 : 0;
 }
 
 static void put_row(const Layered* m, uint8_t* dst, const CMLSafetensor* t, int row, int cols) {
@@ -358,15 +457,16 @@ static int upload_matrix(const Layered* m, cmlb200_dense* w, uint8_t* host) {
     return rc;
 }
 
-/* The experts' gate and up rows (interleaved as in load_matrix) and their down rows, one expert behind the other. */
+/* The experts' gate and up rows (interleaved as in load_matrix), or their up rows alone, and their down rows, one expert behind
+ * the other. */
 static int load_experts(Layered* m, const CMLSafetensors* st, const char* prefix, Layer* l) {
     LayerWeights* w = &l->w;
-    const int gu = 2 * lml_round_up(l->ff, 16), down = lml_round_up(m->width, 16);
+    const int gated = m->design->experts != EXPERTS_SIGMOID, gu = (gated ? 2 : 1) * lml_round_up(l->ff, 16), down = lml_round_up(m->width, 16);
     const size_t es = m->f32 ? 4 : 2;
     const char* router[1] = {"mlp.router"};
     uint8_t *hg, *hd;
     const int outputs = l->experts + l->identity;
-    if (lml_load_matrix(m, st, prefix, router, &outputs, 1, m->width, 0, &w->router) || alloc_matrix(m, l->experts * gu, m->width, &w->experts_gu, &hg)) return -1;
+    if ((!m->design->side_by_side && lml_load_matrix(m, st, prefix, router, &outputs, 1, m->width, 0, &w->router)) || alloc_matrix(m, l->experts * gu, m->width, &w->experts_gu, &hg)) return -1;
     if (alloc_matrix(m, l->experts * down, l->ff, &w->experts_down, &hd)) { free(hg); return -1; }
     int rc = 0;
     for (int e = 0; e < l->experts && !rc; e++) {
@@ -375,10 +475,12 @@ static int load_experts(Layered* m, const CMLSafetensors* st, const char* prefix
         snprintf(name[0], sizeof name[0], "mlp.e%d.gate", e);
         snprintf(name[1], sizeof name[1], "mlp.e%d.up", e);
         snprintf(name[2], sizeof name[2], "mlp.e%d.down", e);
-        rc = lml_find(st, prefix, name[0], l->ff, m->width, &t[0]) || lml_find(st, prefix, name[1], l->ff, m->width, &t[1]) || lml_find(st, prefix, name[2], m->width, l->ff, &t[2]);
-        for (int p = 0; p < 2 && !rc; p++)
-            for (int r = 0; r < l->ff; r++)
-                put_row(m, hg + ((size_t)e * gu + (size_t)(r / 16) * 32 + (size_t)(p * 16 + r % 16)) * (size_t)w->experts_gu.ld * es, &t[p], r, m->width);
+        rc = (gated && lml_find(st, prefix, name[0], l->ff, m->width, &t[0])) || lml_find(st, prefix, name[1], l->ff, m->width, &t[1]) || lml_find(st, prefix, name[2], m->width, l->ff, &t[2]);
+        for (int p = gated ? 0 : 1; p < 2 && !rc; p++)
+            for (int r = 0; r < l->ff; r++) {
+                const size_t at = gated ? (size_t)(r / 16) * 32 + (size_t)(p * 16 + r % 16) : (size_t)r;
+                put_row(m, hg + ((size_t)e * gu + at) * (size_t)w->experts_gu.ld * es, &t[p], r, m->width);
+            }
         for (int r = 0; r < m->width && !rc; r++) put_row(m, hd + ((size_t)e * down + (size_t)r) * (size_t)w->experts_down.ld * es, &t[2], r, l->ff);
     }
     if (rc) { free(hg); free(hd); return -1; }
@@ -435,13 +537,15 @@ static const uint16_t* value_rows(const Layer* l, const LayerWeights* w) {
     return (const uint16_t*)w->wukv.w + (size_t)(l->lat.heads * l->lat.dim) * (size_t)w->wukv.ld;
 }
 
-/* A bias of the stacked projections: the tensors' where they have one, else zero. */
-static int load_bias(const CMLSafetensors* st, const char* prefix, const char* const* names, const int* rows, int with_bias, cmlb200_dense* w) {
+/* A bias of the stacked projections: the tensors' where they have one (bit p of with_bias), else zero. */
+static int load_bias(const CMLSafetensors* st, const char* prefix, const char* const* names, const int* rows, int parts, unsigned with_bias, cmlb200_dense* w) {
+    if (!with_bias) return 0;
     float* v = (float*)calloc((size_t)w->rows, sizeof(float));
     int rc = v ? 0 : -1;
-    for (int p = 0, at = 0; p < with_bias && !rc; at += rows[p++]) {
+    for (int p = 0, at = 0; p < parts && !rc; at += rows[p++]) {
         char name[64];
         CMLSafetensor t;
+        if (!(with_bias >> p & 1)) continue;
         snprintf(name, sizeof name, "%s.b", names[p]);
         rc = lml_find(st, prefix, name, rows[p], 0, &t);
         for (int i = 0; i < rows[p] && !rc; i++) v[at + i] = lml_element(&t, (size_t)i);
@@ -449,6 +553,34 @@ static int load_bias(const CMLSafetensors* st, const char* prefix, const char* c
     rc = rc || lml_upload((void**)&w->bias, v, (size_t)w->rows * sizeof(float));
     free(v);
     return rc ? -1 : 0;
+}
+
+/* Tensors whose rows make one matrix, with their names' room. */
+typedef struct Parts {
+    char names[MAX_PARTS][32];
+    const char* list[MAX_PARTS];
+    int rows[MAX_PARTS], count, total;
+    unsigned with_bias;
+} Parts;
+
+static void add_part(Parts* p, const char* where, const char* name, int rows, int bias) {
+    snprintf(p->names[p->count], sizeof p->names[p->count], "%s%s", where, name);
+    p->list[p->count] = p->names[p->count];
+    p->with_bias |= (unsigned)(bias != 0) << p->count;
+    p->rows[p->count++] = rows;
+    p->total += rows;
+}
+
+/* The rest of a layer's projection, and the matrix: gates of sublayers side by side and the router read the same row. */
+static int load_projection(const Layered* m, const CMLSafetensors* st, const char* prefix, Layer* l, Parts* p) {
+    const int latent = l->kind->form == MIXER_LATENT;
+    if (m->design->side_by_side) {                         /* in the order of place_gates */
+        add_part(p, "", "rg1", m->width, 1);
+        if (l->ff) add_part(p, "", "rg2", m->width, 1);
+        if ((latent ? l->lat.gate_col : l->attn.gate_col) >= 0) add_part(p, l->kind->form == MIXER_PARALLEL ? "mix.left." : "mix.", "g", latent ? l->lat.heads : l->attn.heads, 0);
+        if (l->ff) add_part(p, "mlp.", "router", l->experts, 0);
+    }
+    return lml_load_matrix(m, st, prefix, p->list, p->rows, p->count, m->width, 0, &l->w.wqkvg) || load_bias(st, prefix, p->list, p->rows, p->count, p->with_bias, &l->w.wqkvg) ? -1 : 0;
 }
 
 /* Output matrices of two mixers side by side: [width, left | right]. */
@@ -467,42 +599,45 @@ static int load_outputs(const Layered* m, const CMLSafetensors* st, const char* 
     return upload_matrix(m, out, host);
 }
 
-/* Grouped heads, alone or with the delta rule beside them. */
+/* Grouped heads, alone or with a recurrence beside them. */
 static int load_grouped(Layered* m, const CMLSafetensors* st, const char* prefix, Layer* l) {
     const GroupedForm* form = &l->kind->grouped;
     const cmlb200_attn* a = &l->attn;
     const cmlb200_delta* d = &l->delta;
     LayerWeights* w = &l->w;
-    const int both = l->kind->form == MIXER_PARALLEL;
+    const int both = l->kind->form == MIXER_PARALLEL, delta = both && l->kind->beside == BESIDE_DELTA, gru = both && !delta;
     const char* at = both ? "mix.left." : "mix.";
-    char names[MAX_PARTS][32], group[64];
-    const char* parts[MAX_PARTS];
-    int rows[MAX_PARTS], n = 0;
-#define PART(where, name, count) do { snprintf(names[n], sizeof names[n], "%s%s", (where), (name)); parts[n] = names[n]; rows[n++] = (count); } while (0)
-    PART(at, "q", a->heads * a->dim);
-    PART(at, "k", a->kv_heads * a->dim);
-    if (!form->keys_as_values) PART(at, "v", a->kv_heads * a->vdim);
-    const int with_bias = form->in_bias ? n : 0;
-    if (form->head_gate) PART(at, "g", a->heads);
-    if (both) {
+    char group[64];
+    Parts p = {.count = 0};
+    add_part(&p, at, "q", a->heads * a->dim, form->in_bias);
+    add_part(&p, at, "k", a->kv_heads * a->dim, form->in_bias);
+    if (!form->keys_as_values) add_part(&p, at, "v", a->kv_heads * a->vdim, form->in_bias);
+    if (form->head_gate && !m->design->side_by_side) add_part(&p, at, "g", a->heads, 0);
+    if (delta) {
         if (cml_delta_ranks(st, prefix, l, m->width)) return -1;
-        PART("mix.right.", "q", d->kv_heads * d->dim);
-        PART("mix.right.", "k", d->kv_heads * d->dim);
-        PART("mix.right.", "v", d->heads * d->vdim);
-        PART("mix.right.", "b", d->heads);
-        PART("mix.right.", "a1", l->a_rank);
-        PART("mix.right.", "g1", l->g_rank);
+        add_part(&p, "mix.right.", "q", d->kv_heads * d->dim, 0);
+        add_part(&p, "mix.right.", "k", d->kv_heads * d->dim, 0);
+        add_part(&p, "mix.right.", "v", d->heads * d->vdim, 0);
+        add_part(&p, "mix.right.", "b", d->heads, 0);
+        add_part(&p, "mix.right.", "a1", l->a_rank, 0);
+        add_part(&p, "mix.right.", "g1", l->g_rank, 0);
     }
-#undef PART
+    if (gru) {
+        add_part(&p, "mix.right.", "z", l->gru.width, 1);
+        add_part(&p, "mix.right.", "x", l->gru.width, 1);
+        add_part(&p, "mix.right.", "g", l->gru.width, 0);
+    }
     snprintf(group, sizeof group, "%s%s", prefix, at);
-    const int norm_q = form->norm == NORM_HEAD ? a->dim : rows[0], norm_k = form->norm == NORM_HEAD ? a->dim : rows[1];
-    const char* out[1] = {"o"};
+    const int norm_q = form->norm == NORM_HEAD ? a->dim : p.rows[0], norm_k = form->norm == NORM_HEAD ? a->dim : p.rows[1];
+    const char *out[1] = {"o"}, *right[1] = {"mix.right.o"};
     if ((form->norm != NORM_NONE && (lml_load_vector(st, group, "q.norm", norm_q, 0.f, &w->q_norm) || lml_load_vector(st, group, "k.norm", norm_k, 0.f, &w->k_norm))) ||
-        (form->sink == SINK_LEARNED && lml_load_vector(st, group, "sink", a->heads, 0.f, &w->sinks)) ||
-        lml_load_matrix(m, st, prefix, parts, rows, n, m->width, 0, &w->wqkvg) || (with_bias && load_bias(st, prefix, parts, rows, with_bias, &w->wqkvg)) ||
-        (both ? load_outputs(m, st, prefix, a->heads * a->vdim, d->heads * d->vdim, &w->wo)
-              : lml_load_matrix(m, st, group, out, &m->width, 1, a->heads * a->vdim, 0, &w->wo)) ||
-        (form->out_bias && load_bias(st, group, out, &m->width, 1, &w->wo)) || (both && cml_delta_load(m, st, prefix, l)))
+        (form->sink == SINK_LEARNED && lml_load_vector(st, group, "sink", a->heads, 0.f, &w->sinks)) || load_projection(m, st, prefix, l, &p) ||
+        (delta ? load_outputs(m, st, prefix, a->heads * a->vdim, d->heads * d->vdim, &w->wo)
+               : lml_load_matrix(m, st, group, out, &m->width, 1, a->heads * a->vdim, 0, &w->wo)) ||
+        (form->out_bias && load_bias(st, group, out, &m->width, 1, 1, &w->wo)) || (delta && cml_delta_load(m, st, prefix, l)) ||
+        (gru && (lml_load_matrix(m, st, prefix, right, &m->width, 1, l->gru.width, 0, &w->wo2) || lml_load_vector(st, prefix, "mix.left.out", m->width, 0.f, &w->left_out) ||
+                 lml_load_vector(st, prefix, "mix.right.out", m->width, 0.f, &w->right_out))) ||
+        ((form->conv || form->talk) && cml_talk_load(st, group, l)))
         return -1;
     if (!form->linear_bias) return 0;
     float* s = (float*)malloc((size_t)a->heads * sizeof(float));
@@ -519,12 +654,18 @@ static int load_mixer(Layered* m, const CMLSafetensors* st, const char* prefix, 
     const int out_rows[1] = {m->width};
     if (l->kind->form == MIXER_LATENT) {
         const cmlb200_latent* a = &l->lat;
-        const char* proj[3] = {"mix.q"};
-        int rows[3] = {a->heads * (a->dim + a->rot_dim)}, parts = 1;
-        if (a->kv_col >= 0) { proj[parts] = "mix.dkv"; rows[parts++] = a->rank + a->rot_dim; }
-        if (a->gate_col >= 0) { proj[parts] = "mix.g"; rows[parts++] = a->heads * a->vdim; }
-        return (a->kv_col >= 0 && lml_load_vector(st, prefix, "mix.dkv.norm", a->rank, 0.f, &w->c_norm)) || lml_load_matrix(m, st, prefix, proj, rows, parts, m->width, 0, &w->wqkvg) ||
-               load_latent_heads(m, st, prefix, l) || lml_load_matrix(m, st, prefix, out, out_rows, 1, a->heads * a->vdim, 0, &w->wo) ? -1 : 0;
+        const int q[1] = {a->heads * (a->dim + a->rot_dim)};
+        const char* uq[1] = {"mix.uq"};
+        Parts p = {.count = 0};
+        if (l->kind->q_latent) add_part(&p, "mix.", "dq", l->q_rank, 0);
+        else add_part(&p, "mix.", "q", q[0], 0);
+        if (a->kv_col >= 0) add_part(&p, "mix.", "dkv", a->rank + a->rot_dim, 0);
+        if (a->gate_col >= 0 && !m->design->side_by_side) add_part(&p, "mix.", "g", a->heads * (a->gate_heads ? 1 : a->vdim), 0);
+        if (l->kind->q_latent && (lml_load_vector(st, prefix, "mix.dq.norm", l->q_rank, 0.f, &w->dq_norm) || lml_load_matrix(m, st, prefix, uq, q, 1, l->q_rank, 0, &w->wuq)))
+            return -1;
+        return (a->kv_col >= 0 && lml_load_vector(st, prefix, "mix.dkv.norm", a->rank, 0.f, &w->c_norm)) || load_projection(m, st, prefix, l, &p) ||
+               (l->kind->sink == SINK_LEARNED && lml_load_vector(st, prefix, "mix.sink", a->heads, 0.f, &w->sinks)) || load_latent_heads(m, st, prefix, l) ||
+               lml_load_matrix(m, st, prefix, out, out_rows, 1, a->heads * a->vdim, 0, &w->wo) ? -1 : 0;
     }
     return load_grouped(m, st, prefix, l);
 }
@@ -550,17 +691,17 @@ static int load_sublayer(const Layered* m, const CMLSafetensors* st, const char*
     return lml_upload((void**)&s->mix, mix, (size_t)(m->streams * m->streams) * sizeof(float));
 }
 
-static int load_layer(Layered* m, const CMLSafetensors* st, int index) {
-    Layer* l = &m->layers[index];
+static int load_layer(Layered* m, const CMLSafetensors* st, int run) {
+    Layer* l = &m->layers[run];
     LayerWeights* w = &l->w;
     const LayeredDesign* d = m->design;
     char prefix[32];
-    snprintf(prefix, sizeof prefix, "l%d.", index);
+    snprintf(prefix, sizeof prefix, "l%d.", l->index);
     const char *gu[2] = {"mlp.gate", "mlp.up"}, *up[1] = {"mlp.up"}, *down[1] = {"mlp.down"};
     const int ff_rows[2] = {l->ff, l->ff};
     if (load_sublayer(m, st, prefix, 0, w) || load_mixer(m, st, prefix, l)) return -1;
     if (!l->ff) return 0;
-    if (load_sublayer(m, st, prefix, 1, w)) return -1;
+    if (!d->side_by_side && load_sublayer(m, st, prefix, 1, w)) return -1;
     if (l->experts) return load_experts(m, st, prefix, l);
     if (d->dense == FF_POLY_NORM ? lml_load_matrix(m, st, prefix, up, ff_rows, 1, m->width, 0, &w->wgu) || lml_load_vector(st, prefix, "mlp.act", 4, 0.f, &w->coef)
                                  : lml_load_matrix(m, st, prefix, gu, ff_rows, 2, m->width, 1, &w->wgu))
@@ -597,20 +738,27 @@ int lml_zeroed(void** dst, size_t bytes) {
     return 0;
 }
 
+/* Where a second mixer with an output product of its own leaves its operand: a product reads whole groups of 64 columns. */
+static int beside_col(const Layer* l) { return lml_round_up(l->attn.heads * l->attn.vdim, 64); }
+
 /* Operand buffers have strides that are multiples of 64 and start out zero: the decode product reads up
  * to the padded width, where its weights are zero. */
 static int make_activations(Layered* m, int rows) {
-    int q = 0, att = 0, ff = 0, z = 0, latent_q = 0, latent_o = 0, experts = 0, identity = 0, outputs = 0, top = 0, shared = 0;
+    int q = 0, att = 0, ff = 0, z = 0, latent_q = 0, latent_o = 0, cq = 0, two = 0, experts = 0, identity = 0, outputs = 0, top = 0, shared = 0;
     long positions = 0, tiles = 0;
     for (int i = 0; i < m->num_layers; i++) {
         const Layer* l = &m->layers[i];
-        q = lml_most(q, m->layers[l->source].w.wqkvg.rows);
+        q = lml_most(q, l->proj_col + m->layers[l->source].w.wqkvg.rows);
+        cq = lml_most(cq, l->q_rank);
         ff = lml_most(ff, l->ff);
         if (l->kind->form == MIXER_LATENT) {
             const cmlb200_latent* a = &l->lat;
             att = lml_most(att, a->heads * a->vdim);
             latent_q = lml_most(latent_q, a->heads * (m->f32 ? a->rank + a->rot_dim : a->ld));
             latent_o = lml_most(latent_o, a->heads * (m->f32 ? a->rank : a->ld_rank));
+        } else if (l->kind->form == MIXER_PARALLEL && l->kind->beside == BESIDE_GRU) {
+            att = lml_most(att, beside_col(l) + l->gru.width);
+            two = 1;
         } else {
             att = lml_most(att, l->attn.heads * l->attn.vdim + (l->kind->form == MIXER_PARALLEL ? l->delta.heads * l->delta.vdim : 0));
         }
@@ -658,6 +806,11 @@ static int make_activations(Layered* m, int rows) {
             (shared && lml_zeroed((void**)&m->y_shared, R * (size_t)m->ld_y * 4)))
             return -1;
     }
+    if (cq) {
+        m->ld_cq = lml_round_up(cq, 64);
+        if (lml_zeroed(&m->cq, R * (size_t)m->ld_cq * es)) return -1;
+    }
+    if (m->design->side_by_side && (lml_zeroed((void**)&m->y_mix, R * (size_t)m->ld_y * 4) || (two && lml_zeroed((void**)&m->y_mix2, R * (size_t)m->ld_y * 4)))) return -1;
     if (cml_delta_activations(m, rows)) return -1;
     return CML_DEV_FAIL(cmlb200_stream_sync(NULL), "make_activations") ? -1 : 0;
 }
@@ -696,6 +849,7 @@ static int layered_make_pools(void* model, int blocks, int block_size, int slots
             a->block_size = block_size;
             a->pool_blocks = blocks;
             a->c_norm = w->c_norm;
+            a->sinks = w->sinks;
             a->eps = m->eps;
             if (l->kv_from != i) a->pool = m->layers[l->kv_from].lat.pool;
             else if (lml_zeroed(&a->pool, tokens * (size_t)a->ld * es)) return -1;
@@ -710,10 +864,11 @@ static int layered_make_pools(void* model, int blocks, int block_size, int slots
         a->eps = m->eps;
         a->slopes = w->slopes;
         a->sinks = w->sinks;
-        if (l->kind->form == MIXER_PARALLEL && cml_delta_make_state(m, l, w, slots)) return -1;
+        if (l->kind->form == MIXER_PARALLEL && (l->kind->beside == BESIDE_GRU ? cml_gru_make_state(l, slots) : cml_delta_make_state(m, l, w, slots))) return -1;
+        if ((l->kind->grouped.conv || l->kind->grouped.talk) && cml_talk_make_state(l, w, slots)) return -1;
         if (lml_zeroed(&a->k_pool, heads * (size_t)a->dim_ld * es) || lml_zeroed(&a->v_pool, heads * (size_t)a->vdim_ld * es)) return -1;
     }
-    if (make_expansion(m, blocks, block_size, slots, table_ld)) return -1;
+    if (make_expansion(m, blocks, block_size, slots, table_ld) || cml_talk_make_scores(m, slots, table_ld, block_size)) return -1;
     DEV(cmlb200_stream_sync(NULL));
     return 0;
 }
@@ -755,8 +910,31 @@ static int expert_layer(const Layered* m, const Layer* l, const LayerWeights* w,
         plan->scale = l->router_scale;
         if (l->shared_ff && gated_product(m, &w->shared_gu, &w->shared_down, l->shared_ff, rows, m->y_shared, st)) return -1;
     }
-    if (lml_product(m, &w->router, m->h, m->ld_h, rows, m->router, m->ld_router, st)) return -1;
-    DEV(cmlb200_moe_route(plan, m->router, m->ld_router, rows, m->f32 || rows <= SKINNY_ROWS ? 1 : EXPERT_ROWS, st));
+    const int side = m->design->side_by_side, ld_router = side ? m->ld_qkvg : m->ld_router;
+    const float* router = side ? m->qkvg + l->router_col : m->router;
+    if (!side && lml_product(m, &w->router, m->h, m->ld_h, rows, m->router, m->ld_router, st)) return -1;
+    if (m->design->experts == EXPERTS_SIGMOID) {
+        plan->sigmoid = 1;
+        plan->group_best = 2;
+        plan->groups = l->groups;
+        plan->keep = l->keep;
+    }
+    DEV(cmlb200_moe_route(plan, router, ld_router, rows, m->f32 || rows <= SKINNY_ROWS ? 1 : EXPERT_ROWS, st));
+    if (m->design->experts == EXPERTS_SIGMOID) {           /* no gate */
+        if (m->f32) {
+            DEV(cmlb200_moe_linear_f32(plan, &w->experts_gu, (const float*)m->h, m->ld_h, 1, rows, l->ff, m->gu, m->ld_gu, st));
+            DEV(cmlb200_act_rows_f32(m->gu, m->ld_gu, rows * l->top, l->ff, act, (float*)m->f, m->ld_f, st));
+            DEV(cmlb200_moe_linear_f32(plan, &w->experts_down, (const float*)m->f, m->ld_f, 0, rows, m->width, m->y, m->ld_y, st));
+        } else if (rows <= SKINNY_ROWS) {
+            DEV(cmlb200_moe_gemv_act(plan, &w->experts_gu, (const uint16_t*)m->h, m->ld_h, 1, rows, l->ff, act, (uint16_t*)m->f, m->ld_f, st));
+            DEV(cmlb200_moe_gemv(plan, &w->experts_down, (const uint16_t*)m->f, m->ld_f, 0, rows, m->width, m->y, m->ld_y, st));
+        } else {
+            DEV(cmlb200_moe_gather(plan, (const uint16_t*)m->h, m->ld_h, rows, m->width, (uint16_t*)m->xp, m->ld_h, st));
+            DEV(cmlb200_moe_gemm_act(plan, &w->experts_gu, (const uint16_t*)m->xp, m->ld_h, rows, l->ff, act, (uint16_t*)m->f, m->ld_f, st));
+            DEV(cmlb200_moe_gemm(plan, &w->experts_down, (const uint16_t*)m->f, m->ld_f, rows, m->width, m->y, m->ld_y, st));
+        }
+        return 0;
+    }
     if (m->f32) {
         DEV(cmlb200_moe_linear_f32(plan, &w->experts_gu, (const float*)m->h, m->ld_h, 1, rows, 2 * lml_round_up(l->ff, 16), m->gu, m->ld_gu, st));
         DEV(cmlb200_moe_glu_rows_f32(m->gu, m->ld_gu, rows * l->top, l->ff, act, l->limit, (float*)m->f, m->ld_f, st));
@@ -805,7 +983,9 @@ static int attend_expanded(const Layered* m, const cmlb200_latent* a, const Laye
     s.scale = a->scale;
     s.window = a->window;
     s.gate_col = a->gate_col;
-    s.gate_wide = a->gate_col >= 0;
+    s.gate_wide = a->gate_col >= 0 && !a->gate_heads;
+    s.sink = a->sinks != NULL;
+    s.sinks = a->sinks;
     s.cache_dtype = CMLB200_DT_F16;
     s.k_pool = m->expand_k;
     s.v_pool = m->expand_v;
@@ -862,6 +1042,8 @@ static int attend_latent(const Layered* m, const Layer* l, const LayerWeights* w
         s.scale = a.scale;
         s.window = a.window;
         s.gate_col = -1;
+        s.sink = a.sinks != NULL;
+        s.sinks = a.sinks;
         s.cache_dtype = CMLB200_DT_F32;
         s.k_pool = s.v_pool = a.pool;
         s.block_size = a.block_size;
@@ -882,19 +1064,24 @@ static int attend_latent(const Layered* m, const Layer* l, const LayerWeights* w
 }
 
 static int attend(const Layered* m, const Layer* l, const LayerWeights* w, const CMLLMBatch* b, void* st) {
-    if (l->kind->form == MIXER_PARALLEL && cml_delta_run(m, l, w, b, l->attn.heads * l->attn.vdim, st)) return -1;
+    if (l->kind->form == MIXER_PARALLEL &&
+        (l->kind->beside == BESIDE_GRU ? cml_gru_run(m, l, b, beside_col(l), st) : cml_delta_run(m, l, w, b, l->attn.heads * l->attn.vdim, st)))
+        return -1;
     if (l->kind->form == MIXER_LATENT) return attend_latent(m, l, w, b, st);
     cmlb200_attn a = l->attn;
     a.block_table = b->d_table;
     a.table_ld = b->table_ld;
+    if (l->kind->grouped.conv || l->kind->grouped.talk) return cml_talk_run(m, &a, b, st);
     if (m->f32) {
-        DEV(cmlb200_qk_norm_append(&a, m->qkvg, m->ld_qkvg, b->d_pos, b->d_slot, b->rows, st));
+        if (a.freq) DEV(cmlb200_rotate_append(&a, m->qkvg, m->ld_qkvg, b->d_pos, b->d_slot, 0, b->rows, 0, NULL, st));
+        else DEV(cmlb200_qk_norm_append(&a, m->qkvg, m->ld_qkvg, b->d_pos, b->d_slot, b->rows, st));
         DEV(cmlb200_attention_rows_f32(&a, m->qkvg, m->ld_qkvg, b->d_pos, b->d_slot, b->rows, (float*)m->att, m->ld_att, st));
         return 0;
     }
     const int one = b->one_rows, more = b->rows - one;
     if (more) {
-        DEV(cmlb200_qk_norm_append(&a, m->qkvg + (size_t)one * m->ld_qkvg, m->ld_qkvg, b->d_pos + one, b->d_slot + one, more, st));
+        if (a.freq) DEV(cmlb200_rotate_append(&a, m->qkvg, m->ld_qkvg, b->d_pos, b->d_slot, one, more, one, NULL, st));
+        else DEV(cmlb200_qk_norm_append(&a, m->qkvg + (size_t)one * m->ld_qkvg, m->ld_qkvg, b->d_pos + one, b->d_slot + one, more, st));
         DEV(cmlb200_attention_tiles(&a, m->qkvg, m->ld_qkvg, b->d_tiles, b->tiles, (uint16_t*)m->att, m->ld_att, st));
     }
     if (one) DEV(cmlb200_attention_one(&a, m->qkvg, m->ld_qkvg, b->d_pos, b->d_slot, one, b->max_keys, (uint16_t*)m->att, m->ld_att, st));
@@ -919,6 +1106,47 @@ static int join(const Layered* m, const Sublayer* done, const Sublayer* next, co
     return 0;
 }
 
+/* A layer whose sublayers read the same row: h holds its norm, and is the next layer's behind it. */
+static int forward_side_by_side(const Layered* m, int run, const CMLLMBatch* b, void* st) {
+    const Layer *l = &m->layers[run], *next = run + 1 < m->num_layers ? &m->layers[run + 1] : NULL;
+    const LayerWeights* w = &m->layers[l->source].w;
+    const int rows = b->rows, type = m->f32 ? CMLB200_DT_F32 : CMLB200_DT_BF16;
+    cmlb200_moe plan;
+    cmlb200_gated_join j;
+    memset(&j, 0, sizeof j);
+    if (lml_product(m, &w->wqkvg, m->h, m->ld_h, rows, m->qkvg + l->proj_col, m->ld_qkvg, st)) return -1;
+    if (w->wuq.w) {
+        DEV(cmlb200_norm_columns(m->qkvg, m->ld_qkvg, l->proj_col, l->q_rank, w->dq_norm, m->eps, rows, m->cq, type, m->ld_cq, st));
+        if (lml_product(m, &w->wuq, m->cq, m->ld_cq, rows, m->qkvg, m->ld_qkvg, st)) return -1;
+    }
+    if (attend(m, l, w, b, st) || lml_product(m, &w->wo, m->att, m->ld_att, rows, m->y_mix, m->ld_y, st)) return -1;
+    if (w->wo2.w) {
+        const void* operand = (const uint8_t*)m->att + (size_t)beside_col(l) * (m->f32 ? 4 : 2);
+        if (lml_product(m, &w->wo2, operand, m->ld_att, rows, m->y_mix2, m->ld_y, st)) return -1;
+        j.b = m->y_mix2;
+        j.a_norm = w->left_out;
+        j.b_norm = w->right_out;
+    }
+    j.a = m->y_mix;
+    j.ldm = j.ldf = m->ld_y;
+    j.ga = m->qkvg + l->gate_cols;
+    j.ldg = m->ld_qkvg;
+    if (l->ff) {
+        if (expert_layer(m, l, w, rows, &plan, st)) return -1;
+        j.f = m->y;
+        j.gf = j.ga + m->width;
+        j.parts = &plan;
+    }
+    if (next && next->again) {
+        j.table = m->embed;
+        j.table_dtype = type;
+        j.vocab = m->vocab;
+        j.tokens = b->d_tokens;
+    }
+    DEV(cmlb200_gated_join_rows(&j, m->x, next ? m->layers[next->source].w.sub[0].norm : NULL, m->eps, rows, m->width, m->h, type, m->ld_h, st));
+    return 0;
+}
+
 static int layered_forward(void* model, const CMLLMBatch* b, void* st) {
     const Layered* m = (const Layered*)model;
     const int rows = b->rows, out = m->f32 ? CMLB200_DT_F32 : CMLB200_DT_BF16;
@@ -931,6 +1159,10 @@ static int layered_forward(void* model, const CMLLMBatch* b, void* st) {
         const LayerWeights* w = &m->layers[l->source].w;
         const Sublayer* next = i + 1 < m->num_layers ? &m->layers[m->layers[i + 1].source].w.sub[0] : NULL;
         cmlb200_moe plan;
+        if (m->design->side_by_side) {
+            if (forward_side_by_side(m, i, b, st)) return -1;
+            continue;
+        }
         if (lml_product(m, &w->wqkvg, m->h, m->ld_h, rows, m->qkvg, m->ld_qkvg, st) || attend(m, l, w, b, st) ||
             lml_product(m, &w->wo, m->att, m->ld_att, rows, m->y, m->ld_y, st) || join(m, &w->sub[0], l->ff ? &w->sub[1] : next, NULL, NULL, rows, st))
             return -1;
@@ -974,14 +1206,14 @@ static void layered_free(void* model) {
         const Sublayer *a = &w->sub[0], *b = &w->sub[1];
         void* bufs[] = {w->wqkvg.w, w->wo.w, w->wgu.w, w->wd.w, a->norm, a->post, a->in, a->out, a->mix, b->norm, b->post, b->in, b->out, b->mix, w->q_norm, w->k_norm,
                         w->slopes, w->sinks, w->c_norm, w->coef, (void*)w->wqkvg.bias, (void*)w->wo.bias, w->wukt, w->wukv.w, w->router.w, w->experts_gu.w,
-                        w->experts_down.w, w->shared_gu.w, w->shared_down.w, w->correction, w->conv, w->rate, w->dt_bias, w->o_norm, w->wa.w, w->wg.w, l->freq,
+                        w->experts_down.w, w->shared_gu.w, w->shared_down.w, w->correction, w->conv, w->rate, w->dt_bias, w->o_norm, w->wa.w, w->wg.w, w->wuq.w, w->wo2.w, w->dq_norm, w->talk, w->left_out, w->right_out, l->attn.ring, l->gru.state, l->freq,
                         l->attn.k_pool, l->attn.v_pool, l->delta.state, l->delta.ring, l->kv_from == i ? l->lat.pool : NULL};
         for (size_t k = 0; k < sizeof bufs / sizeof bufs[0]; k++) cmlb200_free(bufs[k]);
     }
     const cmlb200_moe* p = &m->plan;
     void* bufs[] = {m->embed, m->freq, m->final_norm, m->head.w, m->x, m->qkvg, m->y, m->gu, m->h, m->att, m->f, m->q, m->o, m->expand_table, m->expand_k,
                     m->expand_v, m->expand_c, m->xp, m->router, p->ids, p->weight, p->pos, p->src, p->expert, p->start, p->count, p->active, p->num_active,
-                    p->tiles, p->num_tiles, p->self, m->y_shared, m->dec, m->gate, m->low, m->delta_work};
+                    p->tiles, p->num_tiles, p->self, m->y_shared, m->dec, m->gate, m->low, m->delta_work, m->y_mix, m->y_mix2, m->cq, m->q_rows_out, m->scores};
     for (size_t k = 0; k < sizeof bufs / sizeof bufs[0]; k++) cmlb200_free(bufs[k]);
     free(m->layers);
     free(m);
@@ -1002,7 +1234,7 @@ static void* layered_load(const char* path, const CMLJson* config, const CMLLMOp
     int rc = read_config(config, m) || !(st = cml_safetensors_open(file)) || load_shared(m, st);
     for (int i = 0; i < m->num_layers && !rc; i++) {
         if (m->layers[i].source == i) rc = load_layer(m, st, i);
-        if (!rc && m->layers[i].kind->form == MIXER_LATENT) rc = make_rotation(&m->layers[i]);
+        if (!rc) rc = make_rotation(&m->layers[i]);
     }
     cml_safetensors_close(st);
     if (rc || make_activations(m, options->max_step_rows)) { layered_free(m); return NULL; }
@@ -1018,7 +1250,7 @@ static void* layered_load(const char* path, const CMLJson* config, const CMLLMOp
 
 #define LAYERED_CLASS(name) {.architecture = name, .load = layered_load, .free = layered_free, .make_pools = layered_make_pools, .forward = layered_forward, \
                              .head = layered_head, .check = layered_check}
-static const CMLLMClass kLayeredClasses[] = {LAYERED_CLASS("Rarolorn"), LAYERED_CLASS("Situlorn"), LAYERED_CLASS("Lenedra")};
+static const CMLLMClass kLayeredClasses[] = {LAYERED_CLASS("Rarolorn"), LAYERED_CLASS("Situlorn"), LAYERED_CLASS("Lenedra"), LAYERED_CLASS("Zevilorn")};
 
 __attribute__((constructor)) static void register_layered(void) {
     for (size_t i = 0; i < sizeof kLayeredClasses / sizeof kLayeredClasses[0]; i++) cml_lm_register(&kLayeredClasses[i]);

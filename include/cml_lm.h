@@ -5,7 +5,8 @@
  * (cml_quant_api.h). No C-ML counterpart: C-ML's forward is one LLaMA, one sequence.
  *
  * A model is either a folder with config.json ("architecture" names the class) and model.safetensors, or
- * a GGUF file (class "llama"). Built-in classes: "Rarolorn", "Situlorn" and "Lenedra" (folders), "llama" (GGUF).
+ * a GGUF file (class "llama"). Built-in classes: "Rarolorn", "Situlorn", "Lenedra" and
+ * "Zevilorn" (folders), "llama" (GGUF).
  *
  * Errors as in cml_quant_api.h: NULL or -1, with a line through cml_log_message.
  */

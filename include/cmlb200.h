@@ -409,6 +409,7 @@ int cmlb200_ipc_close(void* d_ptr);
 #define CMLB200_ACT_SILU 0
 #define CMLB200_ACT_GELU_TANH 1
 #define CMLB200_ACT_CLAMPED 2     /* g = min(gate, limit), u = clamp(up, -limit, limit): g sigmoid(1.702 g) (u + 1) */
+#define CMLB200_ACT_GELU_ERF 3
 
 /* A dense [rows, cols] weight (rows = out features), row stride `ld` elements. Allocated with rows rounded
  * up to 16 and ld a multiple of 64, the padding zero. dtype CMLB200_DT_F32 or CMLB200_DT_BF16. bias and cap belong to the
@@ -446,6 +447,15 @@ typedef struct cmlb200_attn {
     int head_norm;              /* 1: the norms are per head, q_norm and k_norm hold `dim` weights that all heads share */
     int keys_as_values;         /* 1: no v columns; a value is the projected key before its norm (vdim == dim) */
     float out_scale;            /* factor on the output; 0: 1 */
+    const float* freq;          /* device, rot_dims / 2: entries 2i and 2i + 1 of a query or key head turn by pos * freq[i]; NULL: none */
+    int rot_dims;               /* the first rot_dims entries of a head turn */
+    int taps;                   /* > 0: q, k and v are convolved over time before anything else (cmlb200_rotate_append) */
+    const float* conv;          /* device, [taps][q, k and v columns], the last row meets the current token */
+    float* ring;                /* [slots][taps][q, k and v columns] projections of the latest tokens, position p in entry p mod taps */
+    float cap;                  /* > 0: score = cap tanh(q.k scale / cap) (cmlb200_talk_scores_*) */
+    const float* talk;          /* device, [heads][heads]: a head's score is that combination of all heads' scores (the same); NULL: its own */
+    const float* scores;        /* device: scores made by cmlb200_talk_scores_*, which q . k is then not computed for; NULL: none */
+    int scores_ld;
 } cmlb200_attn;
 
 /* Latent attention over a paged cache of one vector per token: a normed latent of `rank` values and a rotated key
@@ -469,6 +479,8 @@ typedef struct cmlb200_latent {
     const int* block_table;
     int table_ld;
     int pool_blocks;            /* 0: not known, which leaves cmlb200_attention_latent to its mma.sync form */
+    int gate_heads;             /* 1: `heads` gate logits, one for all of a head's output */
+    const float* sinks;         /* device, one per head: exp(sinks[h]) joins the softmax denominator; NULL: none */
 } cmlb200_latent;
 
 /* Where a step's (row, expert) pairs go: `top` pairs per row, ordered by expert, each expert's first position a
@@ -484,8 +496,10 @@ typedef struct cmlb200_moe {
     int *active, *num_active;   /* [experts] experts that were chosen at all */
     int *tiles, *num_tiles;     /* {first position, expert, rows, 0} per 128 positions of an expert */
     /* how the choice is made; all zero: the `top` largest of a softmax over the experts, weighted by it */
+    int sigmoid;                /* 1: scores are sigmoids of the logits; 0: a softmax over all outputs */
+    int group_best;             /* a group counts by the sum of that many of its largest members, 1 or 2; 0: 1 */
     int identity;               /* router outputs behind the experts' whose choice returns the row itself: such a pair has position -1 */
-    int groups, keep;           /* > 0: outputs in that many groups of neighbours; only those of the `keep` groups with the largest member */
+    int groups, keep;           /* > 0: outputs in that many groups of neighbours; only those of the `keep` best groups */
     const float* correction;    /* device, [experts + identity], added to the scores for the choice alone */
     int normalize;              /* 1: weights are divided by their sum (+ 1e-20) and multiplied by `scale` */
     float scale;
@@ -525,6 +539,30 @@ typedef struct cmlb200_delta {
     float* state;               /* [slots][heads][dim][vdim_ld]; a token at position 0 finds it as zeros */
     float* ring;                /* [slots][taps][channels] projections of the latest tokens, position p in entry p mod taps */
 } cmlb200_delta;
+
+/* Minimal gated recurrence: per channel a state S in fp32 that a token changes by S <- (1 - z) S + z c, z = sigmoid of its first
+ * projection, c = u + 1/2 where its second projection u is not negative and sigmoid(u) elsewhere; the output is S silu(g).
+ * Projection rows hold, from column `col` on, [z | u | g] of `width` each. */
+typedef struct cmlb200_gru {
+    int width, col;
+    float* state;               /* [slots][width]; a token at position 0 finds it as zeros */
+} cmlb200_gru;
+
+/* Two sublayers that read the same row and join the residual together, each times sigmoids of logits of the row's width:
+ * x += sigmoid(ga) m + sigmoid(gf) f. fp32 rows, device. */
+typedef struct cmlb200_gated_join {
+    const float *a, *b;         /* m is a, or half the sum of a and b, each normed with its weights (b not NULL) */
+    int ldm;
+    const float *a_norm, *b_norm;
+    const float* f;             /* NULL: no second sublayer */
+    int ldf;
+    const cmlb200_moe* parts;   /* host pointer; f is then the weighted sum of the rows of a row's pairs */
+    const float *ga, *gf;
+    int ldg;
+    const void* table;          /* not NULL: table[token] (table_dtype, of `vocab` rows) is added as well */
+    int table_dtype, vocab;
+    const int* tokens;
+} cmlb200_gated_join;
 
 /* x[r] = table[token[r]] (+ a sinusoidal vector of position pos[r]: sin, cos of pos * freq[i] in entries
  * 2i, 2i + 1; d_freq NULL: none). fp32 rows of `width`. */
@@ -585,6 +623,33 @@ int cmlb200_delta_rows(const cmlb200_delta* a, const float* d_proj, int ld, cons
                        const int* d_row_pos, const int* d_row_slot, int first, int rows, const int* d_runs, int runs, float* d_work, void* d_out,
                        int out_dtype, int out_ld, void* stream);
 long cmlb200_delta_work_floats(const cmlb200_delta* a, int rows, int runs);
+/* Minimal gated recurrence. _one: single tokens, at most one row per sequence; positions, slots and the rows' states must be
+ * older than the launch directly in front of it in the stream. _rows: portions runs[i] = {first row, rows, slot, position}
+ * (device) of the step whose row 0 d_proj and d_out begin with. out: fp32 or bf16. */
+int cmlb200_gru_one(const cmlb200_gru* a, const float* d_proj, int ld, const int* d_row_pos, const int* d_row_slot, int rows, void* d_out, int out_dtype,
+                    int out_ld, void* stream);
+int cmlb200_gru_rows(const cmlb200_gru* a, const float* d_proj, int ld, const int* d_runs, int runs, void* d_out, int out_dtype, int out_ld, void* stream);
+/* Convolution over time and rotation of projection rows first .. first + rows - 1 of a step (the row arrays begin at its row 0),
+ * keys and values into the cache. Queries stay in place, or go to d_q_out [step row][heads][dim_ld] in the cache's number
+ * format (always when they are convolved). The step's first `singles` rows are single tokens, whose projections enter the ring
+ * here; those of portions enter by cmlb200_ring_rows, which follows. */
+int cmlb200_rotate_append(const cmlb200_attn* a, float* d_qkv, int ld, const int* d_row_pos, const int* d_row_slot, int first, int rows, int singles,
+                          void* d_q_out, void* stream);
+int cmlb200_ring_rows(const cmlb200_attn* a, const float* d_qkv, int ld, const int* d_runs, int runs, void* stream);
+/* Scores with cap and talking heads, for cmlb200_attn's `scores`; queries as cmlb200_rotate_append leaves them.
+ * _tiles (fp16 cache): [tile][heads][64][ld] in units of log2, keys from the tile's first visible one rounded down to 16 on, tiles as in
+ * cmlb200_attention_tiles, ld a multiple of 64. _rows: [row][heads][ld], keys from the row's first visible one on; natural
+ * units over an fp32 cache, log2 over fp16. max_keys bounds the keys of any row or tile, its own included. _heads: the most
+ * heads that _tiles takes. */
+int cmlb200_talk_scores_tiles(const cmlb200_attn* a, const uint16_t* d_q_f16, const int* d_tiles, int tiles, int max_keys, float* d_scores, int ld, void* stream);
+int cmlb200_talk_scores_rows(const cmlb200_attn* a, const void* d_q, const int* d_row_pos, const int* d_row_slot, int rows, int max_keys, float* d_scores, int ld,
+                             void* stream);
+int cmlb200_talk_scores_heads(void);
+/* x takes what `j` describes, then out = rms_norm(x) * w_next (w_next NULL: no output). norm_eps: of a, b and the next norm. */
+int cmlb200_gated_join_rows(const cmlb200_gated_join* j, float* d_x, const float* d_w_next, float norm_eps, int rows, int width, void* d_out, int out_dtype, int ldo,
+                            void* stream);
+/* out = rms_norm of columns col .. col + n - 1 * w; fp32 or bf16. */
+int cmlb200_norm_columns(const float* d_x, int ld, int col, int n, const float* d_w, float eps, int rows, void* d_out, int out_dtype, int ldo, void* stream);
 /* bf16 rows of columns col .. col + n - 1 of fp32 rows, and of the `more` columns behind those from output column `at` on; other
  * output columns are left alone. */
 int cmlb200_pack_columns(const float* d_x, int ld, int col, int n, int more, int at, int rows, uint16_t* d_out_bf16, int ldo, void* stream);
@@ -637,6 +702,11 @@ int cmlb200_moe_gemm_glu(const cmlb200_moe* m, const cmlb200_dense* W, const uin
                          int ldf, void* stream);
 int cmlb200_moe_linear_f32(const cmlb200_moe* m, const cmlb200_dense* W, const float* d_x, int ldx, int gather, int rows, int n_out, float* d_y, int ldy,
                            void* stream);
+/* Experts without a gate: act(W x) as bf16 (W's experts: `ff` rows rounded up to 16), and of fp32 rows. */
+int cmlb200_moe_gemv_act(const cmlb200_moe* m, const cmlb200_dense* W, const uint16_t* d_x, int ldx, int gather, int rows, int ff, int act, uint16_t* d_f, int ldf,
+                         void* stream);
+int cmlb200_moe_gemm_act(const cmlb200_moe* m, const cmlb200_dense* W, const uint16_t* d_x, int ldx, int rows, int ff, int act, uint16_t* d_f, int ldf, void* stream);
+int cmlb200_act_rows_f32(const float* d_z, int ld, int rows, int ff, int act, float* d_f, int ldf, void* stream);
 int cmlb200_moe_glu_rows_f32(const float* d_gu, int ld, int rows, int ff, int act, float limit, float* d_f, int ldf, void* stream);
 /* tokens[i] = picked[i], pos[i] += 1, hist[step * rows + i] = picked[i], step += 1 */
 int cmlb200_advance_tokens(const int* d_picked, int rows, int* d_tokens, int* d_pos, int* d_hist, int* d_step, void* stream);
