@@ -380,12 +380,98 @@ def streams_weight(rng, name, shape):
     return bf16_round(np.asarray(a, np.float32))[1]
 
 
+def sigmoid_mlp(experts, top, ff, groups=None):
+    """Experts without a gate; groups: (count, keep)."""
+    router = {"experts": experts, "top": top}
+    if groups:
+        router["groups"] = dict(zip(("count", "keep"), groups))
+    return {"kind": "moe", "expert": {"ff": ff}, "router": router}
+
+
+def _rotation(dims, base, keys, scaling):
+    rot = {"dims": dims, "base": base}
+    if scaling:
+        rot["scaling"] = dict(zip(keys, scaling))
+    return rot
+
+
+def talking_layer(heads, kv_heads, dim, vdim, window, taps, cap, mlp, rot, scaling=None, scale=None):
+    """rot: (dims, base), scaling: (factor, low, high, original)."""
+    return {"type": "attention", "mlp": mlp, "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "mask": {"size": window}, "conv": taps, "softcap": cap,
+                                                       "scale": scale or dim ** -0.5, "rot": _rotation(*rot, ("factor", "low", "high", "original"), scaling)}}
+
+
+def queried_layer(heads, dim, rot_dim, vdim, q_rank, kv_rank, mlp, base=10000.0, scale=None):
+    return {"type": "latent_attention", "mlp": mlp, "mixer": {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "q_rank": q_rank, "kv_rank": kv_rank,
+                                                              "scale": scale or (dim + rot_dim) ** -0.5, "rot": {"dims": rot_dim, "base": base}}}
+
+
+def recurrent_layer(left, rot, width, mlp, factor=None, scale=None):
+    """left: (heads, kv_heads, dim, vdim, window), rot: (dims, base)."""
+    m = dict(zip(("heads", "kv_heads", "dim", "vdim"), left), mask={"size": left[4]}, scale=scale or left[2] ** -0.5, rot=_rotation(*rot, ("factor",), factor and (factor,)))
+    return {"type": "parallel", "mlp": mlp, "mixer": {"left": m, "right": {"width": width}}}
+
+
+def looped_config(vocab, width, layers, loop=None, eps=1e-5):
+    """loop: (start, stop, times)."""
+    cfg = {"architecture": "Zevilorn", "vocab": vocab, "width": width, "norm": {"eps": eps}, "layers": layers}
+    if loop:
+        cfg["loop"] = dict(zip(("start", "stop", "times"), loop))
+    return cfg
+
+
+def gated_layer_shapes(layer, W, p):
+    m, f, q = layer["mixer"], layer["mlp"], p + "mix."
+    out = {p + "norm1": (W,), p + "rg1": (W, W), p + "rg1.b": (W,)}
+    if layer["type"] == "attention":
+        H, G, D, V, n = m["heads"], m["kv_heads"], m["dim"], m["vdim"], m["conv"]
+        for name, rows in (("q", H * D), ("k", G * D), ("v", G * V)):
+            out.update({q + name: (rows, W), q + name + ".b": (rows,), q + name + ".conv": (rows, n)})
+        out.update({q + "talk": (H, H), q + "o": (W, H * V), q + "o.b": (W,)})
+    elif layer["type"] == "latent_attention":
+        H, R = m["heads"], m["kv_rank"]
+        out.update({q + "dq": (m["q_rank"], W), q + "dq.norm": (m["q_rank"],), q + "uq": (H * (m["dim"] + m["rot_dim"]), m["q_rank"]), q + "dkv": (R + m["rot_dim"], W),
+                    q + "dkv.norm": (R,), q + "uk": (H * m["dim"], R), q + "uv": (H * m["vdim"], R), q + "sink": (H,), q + "g": (H, W), q + "o": (W, H * m["vdim"])})
+    else:
+        a, C = m["left"], m["right"]["width"]
+        H, G, D, V = a["heads"], a["kv_heads"], a["dim"], a["vdim"]
+        out.update({q + "left.q": (H * D, W), q + "left.k": (G * D, W), q + "left.v": (G * V, W), q + "left.g": (H, W), q + "left.o": (W, H * V), q + "right.z": (C, W),
+                    q + "right.z.b": (C,), q + "right.x": (C, W), q + "right.x.b": (C,), q + "right.g": (C, W), q + "right.o": (W, C), q + "left.out": (W,), q + "right.out": (W,)})
+    if f:
+        n = f["expert"]["ff"]
+        out.update({p + "rg2": (W, W), p + "rg2.b": (W,), p + "mlp.router": (f["router"]["experts"], W)})
+        for e in range(f["router"]["experts"]):
+            out.update({p + f"mlp.e{e}.up": (n, W), p + f"mlp.e{e}.down": (W, n)})
+    return out
+
+
+def gated_weight(rng, name, shape):
+    """A random tensor of a design whose sublayers join through gates: heads that mostly keep their own score, taps of one size, sinks that take
+    a visible share."""
+    a = rng.standard_normal(shape).astype(np.float32)
+    leaf = name.split(".", 1)[1] if name[0] == "l" and name[1].isdigit() else name
+    if leaf.endswith((".norm", "norm1", ".out")):
+        a = 1 + 0.2 * a
+    elif leaf.endswith(".talk"):
+        a = 0.6 * np.eye(shape[0]) + a / np.sqrt(shape[0])
+    elif leaf.endswith(".sink"):
+        a += 1
+    elif leaf.endswith(".b"):
+        a *= 0.4
+    elif leaf != "embed":
+        a /= np.sqrt(shape[-1])
+    return bf16_round(np.asarray(a, np.float32))[1]
+
+
 def layered_shapes(cfg):
     """Tensor name -> shape of every tensor a configuration asks for."""
     W, out = cfg["width"], {"embed": (cfg["vocab"], cfg["width"])}
     for i, layer in enumerate(cfg["layers"]):
         if "streams" in cfg:
             out.update(streams_layer_shapes(layer, W, cfg["streams"], f"l{i}."))
+            continue
+        if cfg["architecture"] == "Zevilorn":
+            out.update(gated_layer_shapes(layer, W, f"l{i}."))
             continue
         if layer.get("weights_of") is not None:
             continue
@@ -409,6 +495,9 @@ def layered_weights(rng, cfg):
     for name, shape in layered_shapes(cfg).items():
         if "streams" in cfg:
             w[name] = streams_weight(rng, name, shape)
+            continue
+        if cfg["architecture"] == "Zevilorn":
+            w[name] = gated_weight(rng, name, shape)
             continue
         a = rng.standard_normal(shape, dtype=np.float32)
         if name.endswith("mlp.act"):

@@ -4,12 +4,14 @@ import numpy as np
 import latent_oracle
 import lenedra_oracle
 import lm_oracle
+import zevilorn_oracle
 
 
 def variants(synth):
     """name -> configuration. Sizes are chosen so that no two of them coincide by accident."""
     L, A = synth.layered_layer, synth.latent_layer
     K, P, R = synth.kept_layer, synth.parallel_layer, synth.routed_mlp
+    T, Q, G, S = synth.talking_layer, synth.queried_layer, synth.recurrent_layer, synth.sigmoid_mlp
     return {
         # grouped heads, two windows, a layer without feed-forward, shared weights with another layer between
         "mixed": synth.layered_config(211, 144, [L(6, 3, 24, 40, 19, 200, coef=0.4, every=7), L(4, 1, 32, 16, 70, None, coef=0.1, every=33),
@@ -47,8 +49,36 @@ def variants(synth):
         # sizes with tiles of their own; chunks and windows that end where blocks and tiles do
         "streams_full": synth.streams_config(64, 128, 4, [P((4, 2, 64, 64, 64), (2, 1, 128, 128, 4), (16, 16), R(9, 3, 4, 3, 2, 24, 24)), K(2, 1, 128, 64, 16, 96),
                                                           P((4, 4, 128, 128, 16), (4, 4, 64, 64, 4), (64, 64), 64)]),
+        # sublayers side by side: every mixer, a loop over some of them, key heads shared, part of a head rotated, both ways to scale
+        # frequencies and neither, a layer without feed-forward, groups and none
+        "loops": synth.looped_config(211, 144, [T(6, 3, 24, 40, 37, 3, 4.0, S(8, 2, 40, (4, 2)), (16, 500.0), (3.0, 1.0, 4.0, 100)), Q(5, 24, 8, 40, 56, 40, S(6, 3, 33)),
+                                                G((4, 2, 32, 24, 23), (8, 2000.0), 56, None, 2.5), T(4, 1, 16, 24, 70, 4, 2.5, S(9, 1, 24, (3, 1)), (16, 300.0)),
+                                                G((3, 3, 24, 40, 90), (24, 900.0), 130, S(7, 7, 17))], (1, 4, 3), eps=1e-3),
+        # odd sizes everywhere, one pair rotated, one tap and many, windows of one token, a loop from the first layer to the last
+        "loops_odd": synth.looped_config(97, 75, [G((3, 1, 13, 7, 1), (2, 50.0), 37, S(5, 2, 51, (5, 2))), T(9, 3, 11, 5, 50, 1, 1.5, S(3, 1, 17), (6, 60.0), (2.0, 0.5, 3.0, 40)),
+                                                  Q(3, 13, 6, 7, 21, 33, None, 100.0), T(1, 1, 7, 9, 1, 7, 3.0, None, (2, 10.0)), Q(1, 5, 2, 9, 3, 17, S(4, 2, 33, (2, 1)))], (0, 5, 2), eps=2e-2),
+        # many heads, wide heads and latents, windows longer than the prompts, no loop
+        "loops_wide": synth.looped_config(130, 192, [T(40, 8, 40, 72, 400, 4, 6.0, S(40, 5, 48, (8, 3)), (40, 1e4), (8.0, 1.0, 4.0, 64)), Q(20, 72, 64, 136, 200, 300, S(5, 2, 96)),
+                                                     G((12, 4, 136, 200, 300), (64, 1e4), 320, S(12, 3, 40, (2, 2)), 4.0), T(100, 4, 8, 8, 65, 2, 2.0, None, (8, 100.0))]),
+        # sizes with tiles of their own; windows that end where blocks and tiles do; a loop of one pass in front of a layer
+        "loops_full": synth.looped_config(64, 128, [Q(4, 128, 64, 128, 64, 512, S(9, 4, 24, (3, 2))), G((4, 2, 64, 64, 64), (64, 1e4), 64, S(4, 2, 64, (4, 3))),
+                                                    T(8, 4, 64, 128, 16, 3, 5.0, S(16, 2, 16, (2, 1)), (32, 1e3)), G((2, 1, 128, 128, 128), (32, 1e4), 128, None)], (1, 2, 1)),
+        # windows in every layer, so that blocks are let go
+        "loops_windows": synth.looped_config(90, 80, [T(4, 2, 24, 16, 33, 3, 3.0, S(4, 2, 24, (2, 1)), (12, 200.0)), G((2, 1, 16, 24, 70), (16, 500.0), 40, S(3, 2, 20))], (0, 1, 2), eps=1e-3),
         "plain": synth.layered_config(64, 64, [L(2, 1, 32, 32, 16, 64, coef=0.0, every=1), L(2, 2, 32, 32, 17, 64, coef=1.0, every=1)], eps=1e-6),
     }
+
+
+def clear_groups(z, groups):
+    """Whether the groups picked by the sum of their two best sigmoids lead by more than rounding, whatever the row's norm."""
+    if not groups or groups["keep"] == groups["count"]:
+        return True
+    for scale in (0.1, 0.2, 0.4, 0.8, 1.5):
+        two = np.sort(zevilorn_oracle.sigmoid(z * scale).reshape(groups["count"], -1), -1)[:, -2:].sum(-1)
+        order = np.sort(two)[::-1]
+        if order[groups["keep"] - 1] - order[groups["keep"]] < 0.02 * scale:
+            return False
+    return True
 
 
 def steady_routes(synth, rng, cfg, w):
@@ -60,8 +90,23 @@ def steady_routes(synth, rng, cfg, w):
         return
     n = max(len(w[f"l{i}.mlp.router"]) for i in moe)
     level = (np.arange(n) - n / 2) * min(0.5, 4.0 / n)
-    w["embed"][:, -n:] = synth.bf16_round(np.stack([rng.permutation(level) for _ in range(cfg["vocab"])]))[1]
+    orders = {i: rng.permutation(n)[:len(w[f"l{i}.mlp.router"])] for i in moe}
+    side = cfg["architecture"] == "Zevilorn"
+    if side:
+        level = level * 2
+    rows = []
+    while len(rows) < cfg["vocab"]:
+        row = rng.permutation(level)
+        if not side or all(clear_groups(row[o], cfg["layers"][i]["mlp"]["router"].get("groups")) for i, o in orders.items()):
+            rows.append(row)
+    w["embed"][:, -n:] = synth.bf16_round(np.stack(rows))[1]
     for name in w:
+        if side:
+            if name.endswith(".norm1"):
+                w[name][-n:] = 1.0
+            elif name.endswith((".o", ".o.b", ".down", ".out")):
+                w[name][-n:] = 0.0
+            continue
         if "streams" in cfg and name.endswith((".norm1", ".norm2", "mix.o.b")):
             w[name][-n:] = 0.0
         elif "streams" in cfg and name[0] == "l" and name.endswith((".o", ".down")):
@@ -72,7 +117,7 @@ def steady_routes(synth, rng, cfg, w):
     for i in moe:
         r = w[f"l{i}.mlp.router"]
         r[:] = 0.0
-        r[np.arange(len(r)), cfg["width"] - n + rng.permutation(n)[:len(r)]] = 1.0
+        r[np.arange(len(r)), cfg["width"] - n + orders[i]] = 1.0
 
 
 def build(synth, tmp_path, name, seed=0):
@@ -98,7 +143,7 @@ TOL = {6: 0.02, 0: 2e-5}            # by dtype of the device model: bfloat16, fl
 
 def model(cfg, w):
     """The plain restatement of a configuration's design."""
-    return {"Rarolorn": lm_oracle, "Situlorn": latent_oracle, "Lenedra": lenedra_oracle}[cfg["architecture"]].Model(cfg, w)
+    return {"Rarolorn": lm_oracle, "Situlorn": latent_oracle, "Lenedra": lenedra_oracle, "Zevilorn": zevilorn_oracle}[cfg["architecture"]].Model(cfg, w)
 
 
 def reference(cfg, w, tokens):

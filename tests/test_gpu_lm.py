@@ -15,7 +15,8 @@ pytestmark = pytest.mark.gpu
 ROOT = Path(__file__).resolve().parents[1]
 LATENT = ["latent", "latent_odd", "latent_wide", "latent_full"]
 STREAMS = ["streams", "streams_odd", "streams_wide", "streams_full"]
-NAMES = ["mixed", "odd", "wide", "plain"] + LATENT + STREAMS
+LOOPS = ["loops", "loops_odd", "loops_wide", "loops_full"]
+NAMES = ["mixed", "odd", "wide", "plain"] + LATENT + STREAMS + LOOPS
 DTYPES = [6, 0]                      # bfloat16, float32
 
 
@@ -73,7 +74,7 @@ def test_first_tokens(synth, tmp_path, load, name, dtype):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("name", ["mixed", "odd", "latent", "latent_odd", "latent_wide", "streams", "streams_odd", "streams_full"])
+@pytest.mark.parametrize("name", ["mixed", "odd", "latent", "latent_odd", "latent_wide", "streams", "streams_odd", "streams_full", *LOOPS])
 def test_unequal_requests_in_one_batch_with_blocks_used_again(pkg, synth, tmp_path, load, name, dtype):
     """Random schedules over a pool that is too small for all requests together: requests come and go, pause,
     take portions beside single tokens, and sit on blocks and slots that others have used."""
@@ -110,7 +111,7 @@ def test_unequal_requests_in_one_batch_with_blocks_used_again(pkg, synth, tmp_pa
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("name", ["wide", "latent", "latent_wide", "streams", "streams_wide"])
+@pytest.mark.parametrize("name", ["wide", "latent", "latent_wide", "streams", "streams_wide", "loops", "loops_wide"])
 def test_batch_does_not_change_a_request(synth, tmp_path, load, name, dtype):
     cfg, w, folder = lm_util.build(synth, tmp_path, name)
     m = load(folder, dtype, max_sequences=8)
@@ -130,7 +131,7 @@ def test_batch_does_not_change_a_request(synth, tmp_path, load, name, dtype):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("name", ["mixed", "latent_odd", "streams", "streams_odd"])
+@pytest.mark.parametrize("name", ["mixed", "latent_odd", "streams", "streams_odd", "loops_windows"])
 def test_long_decoding(pkg, synth, tmp_path, load, name, dtype):
     """Hundreds of decoded tokens, over many blocks; windows let blocks go on the way, so the sequence outgrows what
     the pool could hold of it at once."""
@@ -142,6 +143,27 @@ def test_long_decoding(pkg, synth, tmp_path, load, name, dtype):
     assert error(got, lm_util.reference(cfg, w, t)) < TOL[dtype]
     lib = pkg.lib
     assert lib.cml_lm_sequence_length(m.h, s) == 420 and lib.cml_lm_blocks_total(m.h) - lib.cml_lm_blocks_free(m.h) <= 9      # the longest window is 70, and up to 33 first tokens are kept
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", ["latent", "loops", "loops_full"])
+def test_long_decoding_with_everything_in_sight(synth, tmp_path, load, name, dtype):
+    cfg, w, folder = lm_util.build(synth, tmp_path, name)
+    t = prompt(cfg, 420)
+    m = load(folder, dtype, max_tokens=432, max_sequences=2)
+    assert error(feed(m, m.open(), t, [23] + [1] * 397), lm_util.reference(cfg, w, t)) < TOL[dtype]
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_slots_of_closed_sequences_start_over(synth, tmp_path, load, dtype):
+    """A sequence in a slot that another one left in the middle of things finds no trace of it: states, rings, blocks."""
+    cfg, w, folder = lm_util.build(synth, tmp_path, "loops")
+    m = load(folder, dtype, max_tokens=128, max_sequences=1)
+    for n, sizes in ((90, [90]), (1, [1]), (70, [1]), (2, [2]), (33, [2]), (3, [1, 2]), (128, [64])):
+        t = prompt(cfg, n, seed=n)
+        s = m.open()
+        assert error(feed(m, s, t, sizes), lm_util.reference(cfg, w, t)) < TOL[dtype]
+        m.end(s)
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
@@ -225,7 +247,7 @@ def serve(pkg, m, prompts, lengths, batch, gen=None):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("name", ["wide", "latent", "streams"])
+@pytest.mark.parametrize("name", ["wide", "latent", "streams", "loops"])
 def test_scheduler_serves_more_requests_than_fit(pkg, synth, tmp_path, load, name, dtype):
     cfg, w, folder = lm_util.build(synth, tmp_path, name)
     m = load(folder, dtype, max_tokens=256, max_sequences=3, max_step_rows=48)       # prompts are cut, requests wait
@@ -243,7 +265,7 @@ def test_scheduler_serves_more_requests_than_fit(pkg, synth, tmp_path, load, nam
     assert [len(g) for g in got] == [4, 0, 0, 5] and status[1] == status[2] == 4
 
 
-@pytest.mark.parametrize("name", ["plain", "latent", "streams"])
+@pytest.mark.parametrize("name", ["plain", "latent", "streams", "loops"])
 def test_generation_and_sampling(pkg, synth, tmp_path, load, name):
     cfg, w, folder = lm_util.build(synth, tmp_path, name)
     m, lib = load(folder, 0), pkg.lib
@@ -290,10 +312,10 @@ def test_step_refusals_change_nothing(pkg, synth, tmp_path, load):
     assert error(np.concatenate(parts), lm_util.reference(cfg, w, t)) < TOL[0]
 
 
-@pytest.mark.parametrize("name", ["odd", "latent_odd", "streams_odd"])
+@pytest.mark.parametrize("name", ["odd", "latent_odd", "streams_odd", "loops_odd"])
 def test_wanted_places_only_and_many_of_them(synth, tmp_path, load, name):
     cfg, w, folder = lm_util.build(synth, tmp_path, name)
-    m = load(folder, 6, max_tokens=1024)
+    m = load(folder, 6, max_tokens=2048 if name == "loops_odd" else 1024)    # one of its layers sees everything, so no block is let go
     t = prompt(cfg, 600)
     want = lm_util.reference(cfg, w, t)
     s, u = m.open(), m.open()
@@ -334,7 +356,7 @@ def test_llama_behind_the_same_interface(pkg, tmp_path, load):
     assert [len(g) for g in got] == [5, 8] and got[0][0] == int(want[6].argmax())
 
 
-@pytest.mark.parametrize("name", ["mixed", "latent", "streams"])
+@pytest.mark.parametrize("name", ["mixed", "latent", "streams", "loops"])
 def test_trace_run_replays(synth, tmp_path, torch_dev, name):
     cfg, w, folder = lm_util.build(synth, tmp_path, name)
     t = {"a": prompt(cfg, 90, 1), "b": prompt(cfg, 50, 2), "c": prompt(cfg, 30, 3)}
@@ -366,7 +388,7 @@ def test_trace_run_replays(synth, tmp_path, torch_dev, name):
                 assert error(got, np.array(mine)) < TOL[code]
 
 
-@pytest.mark.parametrize("name", ["plain", "latent_odd", "streams_odd"])
+@pytest.mark.parametrize("name", ["plain", "latent_odd", "streams_odd", "loops_odd"])
 def test_cml_generate_program(pkg, synth, tmp_path, load, name):
     cfg, w, folder = lm_util.build(synth, tmp_path, name)
     prompts = [prompt(cfg, 9, 1).tolist(), prompt(cfg, 30, 2).tolist()]

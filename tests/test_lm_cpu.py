@@ -11,6 +11,7 @@ import latent_oracle as la
 import lenedra_oracle as le
 import lm_oracle as lo
 import lm_util
+import zevilorn_oracle as ze
 
 ROOT = Path(__file__).resolve().parents[1]
 
@@ -49,7 +50,7 @@ def test_norm_and_activation():
 
 
 @pytest.mark.parametrize("name", ["mixed", "odd", "wide", "plain", "latent", "latent_odd", "latent_wide", "latent_full", "streams", "streams_odd", "streams_wide",
-                                  "streams_full"])
+                                  "streams_full", "loops", "loops_odd", "loops_wide", "loops_full", "loops_windows"])
 def test_portions_change_nothing(synth, tmp_path, name):
     cfg, w, _ = lm_util.build(synth, tmp_path, name)
     m = lm_util.model(cfg, w)
@@ -230,9 +231,107 @@ def test_every_setting_of_a_design_with_streams_shows(synth, tmp_path):
     moved(lambda c, l: None, w2)
 
 
+# ---- the restatement of looped layers, gates, talking heads, the minimal recurrence and sigmoid routing ------
+def test_rotation_of_neighbours_and_halves_by_hand():
+    f = ze.frequencies({"dims": 4, "base": 100.0})
+    assert np.allclose(f, [1.0, 0.1])
+    x = np.array([[[1.0, 2.0, 3.0, 4.0, 9.0]]] * 2)
+    c, s = np.cos([5.0, 0.5]), np.sin([5.0, 0.5])
+    y = ze.rotate_neighbours(x, [0, 5], f)
+    assert np.allclose(y[0], x[0]) and np.allclose(y[1, 0], [c[0] - 2 * s[0], 2 * c[0] + s[0], 3 * c[1] - 4 * s[1], 4 * c[1] + 3 * s[1], 9])
+    y = ze.rotate_halves(x, [0, 5], f)
+    assert np.allclose(y[1, 0], [c[0] - 3 * s[0], 2 * c[1] - 4 * s[1], 3 * c[0] + s[0], 4 * c[1] + 2 * s[1], 9])
+
+
+def test_frequency_scalings_by_hand():
+    tau = 2 * np.pi
+    # turns within 100 positions: 8 (stays), 2 (a third of the way from 1 to 4), 0.5 (stretched)
+    f = np.array([8, 2, 0.5]) * tau / 100
+    s = {"factor": 5.0, "low": 1.0, "high": 4.0, "original": 100}
+    assert np.allclose(ze.scale_banded(f, s), f * [1, (2 / 3) / 5 + 1 / 3, 1 / 5])
+    assert np.allclose(ze.scale_linear(f, {"factor": 4.0}), f / 4)
+
+
+def test_cap_and_mixed_heads_by_hand():
+    assert np.allclose(ze.soft_cap(np.array([1.0, -50.0]), 2.0), [2 * np.tanh(0.5), -2])
+    s = np.array([[[1.0, 2.0]], [[10.0, 20.0]]])                              # [head, query, key]
+    assert np.allclose(ze.mix_heads(s, np.array([[1.0, 3.0], [0.0, -1.0]])), [[[31, 62]], [[-10, -20]]])
+    p = ze.weights_over(np.log(np.array([[[1.0, 3.0, 9.0]]])), ze.window([5], [4, 5, 6], 2), [0.0])
+    assert np.allclose(p, [[[1 / 5, 3 / 5, 0]]])
+    assert ze.window([5], range(8), 3)[0].tolist() == [False] * 3 + [True] * 3 + [False] * 2
+
+
+def test_convolution_without_activation_by_hand():
+    y, past = ze.causal_conv(np.array([[1.0], [2.0], [3.0]]), np.array([[100.0, 10.0, 1.0]]), np.zeros((2, 1)))
+    assert y.ravel().tolist() == [1, 12, 123] and past.ravel().tolist() == [2, 3]
+
+
+def test_minimal_recurrence_by_hand():
+    assert np.allclose(ze.candidate(np.array([0.0, 2.0, -1.0])), [0.5, 2.5, ze.sigmoid(-1.0)])
+    S = ze.gated_scan(np.array([[0.25], [1.0], [0.5]]), np.array([[4.0], [3.0], [1.0]]), np.array([8.0]))
+    assert S.ravel().tolist() == [7.0, 3.0, 2.0]
+
+
+def test_groups_by_their_two_best_by_hand():
+    z = np.log(np.array([[0.9, 0.1, 0.1, 0.5, 0.55, 0.1]]) / (1 - np.array([[0.9, 0.1, 0.1, 0.5, 0.55, 0.1]])))
+    r = {"groups": {"count": 2, "keep": 1}, "top": 2}
+    ids, p = ze.route(z, {"router": np.eye(6)}, r)                             # 0.9 + 0.1 against 0.55 + 0.5
+    assert ids.tolist() == [[4, 3]] and np.allclose(p, [[0.55, 0.5]])
+    ids, p = ze.route(z, {"router": np.eye(6)}, {"top": 2})
+    assert ids.tolist() == [[0, 4]] and np.allclose(p, [[0.9, 0.55]])
+    assert np.allclose(ze.gelu_erf(np.array([0.0, 1.0, -1.0])), [0, 0.8413447, -0.1586553])
+
+
+def test_loop_order_by_hand():
+    cfg = {"layers": [0] * 4, "loop": {"start": 1, "stop": 3, "times": 3}}
+    assert ze.runs(cfg) == [(0, False), (1, False), (2, False), (1, True), (2, False), (1, True), (2, False), (3, False)]
+    assert ze.runs({"layers": [0] * 2}) == [(0, False), (1, False)]
+
+
+def test_every_setting_of_a_design_with_loops_shows(synth, tmp_path):
+    cfg, w, _ = lm_util.build(synth, tmp_path, "loops")
+    t = np.random.default_rng(3).integers(0, cfg["vocab"], 110)
+    want = lm_util.reference(cfg, w, t)
+
+    def moved(change, w2=None):
+        other = json.loads(json.dumps(cfg))
+        change(other, other["layers"])
+        assert lm_util.error(lm_util.reference(other, w2 or w, t), want) > 100 * lm_util.TOL[0]
+    mixer = lambda l, i: l[i]["mixer"]
+    moved(lambda c, l: mixer(l, 0)["mask"].update(size=36))
+    moved(lambda c, l: mixer(l, 3)["mask"].update(size=71))
+    moved(lambda c, l: mixer(l, 2)["left"]["mask"].update(size=22))
+    moved(lambda c, l: mixer(l, 0).update(softcap=5.0))
+    for k in (0, 1):
+        moved(lambda c, l: mixer(l, k).update(scale=0.3))
+    moved(lambda c, l: mixer(l, 2)["left"].update(scale=0.3))
+    moved(lambda c, l: mixer(l, 0)["rot"].update(base=450.0))
+    moved(lambda c, l: mixer(l, 0)["rot"].update(dims=18))
+    moved(lambda c, l: mixer(l, 1)["rot"].update(base=9000.0))
+    moved(lambda c, l: mixer(l, 2)["left"]["rot"].update(dims=10))
+    for k, v in (("factor", 2.0), ("low", 0.5), ("high", 8.0), ("original", 50)):
+        moved(lambda c, l: mixer(l, 0)["rot"]["scaling"].update({k: v}))
+    moved(lambda c, l: mixer(l, 2)["left"]["rot"]["scaling"].update(factor=2.0))
+    moved(lambda c, l: mixer(l, 2)["left"]["rot"].pop("scaling"))
+    moved(lambda c, l: l[0]["mlp"]["router"].update(top=1))
+    moved(lambda c, l: l[0]["mlp"]["router"]["groups"].update(keep=4))
+    moved(lambda c, l: l[3]["mlp"]["router"].pop("groups"))
+    for loop in ((1, 4, 2), (0, 4, 3), (1, 3, 3), (2, 4, 3)):
+        moved(lambda c, l: c.update(loop=dict(zip(("start", "stop", "times"), loop))))
+    for name in ("l0.mix.q.b", "l0.mix.v.b", "l0.mix.o.b", "l0.mix.k.conv", "l0.mix.v.conv", "l0.mix.talk", "l1.mix.dq.norm", "l1.mix.dkv.norm", "l1.mix.uk", "l1.mix.uv",
+                 "l1.mix.sink", "l1.mix.g", "l2.mix.left.g", "l2.mix.left.out", "l2.mix.right.z", "l2.mix.right.z.b", "l2.mix.right.x.b", "l2.mix.right.g", "l2.mix.right.out",
+                 "l0.rg1", "l0.rg2.b", "l1.mlp.e2.up", "l3.norm1", "final.norm"):
+        w2 = dict(w)
+        w2[name] = w[name][::-1]
+        moved(lambda c, l: None, w2)
+    w2 = dict(w)
+    w2["l0.mix.talk"] = w["l0.mix.talk"].T
+    moved(lambda c, l: None, w2)
+
+
 # ---- registry and readers ------------------------------------------------------------------------------
 def test_registry_knows_its_classes(pkg):
-    assert pkg.lib.cml_lm_known(b"Situlorn") == 1 and pkg.lib.cml_lm_known(b"Lenedra") == 1
+    assert pkg.lib.cml_lm_known(b"Situlorn") == 1 and pkg.lib.cml_lm_known(b"Lenedra") == 1 and pkg.lib.cml_lm_known(b"Zevilorn") == 1
     assert pkg.lib.cml_lm_known(b"Rarolorn") == 1 and pkg.lib.cml_lm_known(b"llama") == 1
     assert pkg.lib.cml_lm_known(b"nothing") == 0 and pkg.lib.cml_lm_known(None) == 0
     o = pkg.lib.cml_lm_default_options()
@@ -340,6 +439,48 @@ def test_streams_load_refusals(pkg, synth, tmp_path):
     with_config(lambda c: router(c)["groups"].update(keep=6))
     with_config(lambda c: router(c).update(top=5))                               # more than the kept groups hold
     with_config(lambda c: c["layers"][1]["mlp"]["shared"].update(ff=0))
+
+
+def test_loops_load_refusals(pkg, synth, tmp_path):
+    cfg, w, folder = lm_util.build(synth, tmp_path, "loops")
+    mixer = lambda c, i: c["layers"][i]["mixer"]
+
+    def with_config(change):
+        c = json.loads(json.dumps(cfg))
+        change(c)
+        (folder / "config.json").write_text(json.dumps(c))
+        assert not _load(pkg, folder)
+
+    for loop in ({"start": 1, "stop": 6, "times": 2}, {"start": -1, "stop": 2, "times": 2}, {"start": 3, "stop": 2, "times": 2}, {"start": 0, "stop": 2, "times": 0}, {"start": 0, "stop": 2},
+                 {"start": 0, "stop": 5, "times": 100000}):
+        with_config(lambda c: c.update(loop=loop))
+    for key in ("heads", "kv_heads", "dim", "vdim", "scale", "conv", "rot"):
+        with_config(lambda c: mixer(c, 0).pop(key))
+    with_config(lambda c: mixer(c, 0).update(conv=0))
+    with_config(lambda c: mixer(c, 0).update(conv=65))
+    with_config(lambda c: mixer(c, 0).update(softcap=-1.0))
+    with_config(lambda c: mixer(c, 0).update(heads=999, kv_heads=1))              # more than can mix their scores
+    with_config(lambda c: mixer(c, 0)["mask"].update(size=0))
+    for dims in (0, 7, 26, -2):
+        with_config(lambda c: mixer(c, 0)["rot"].update(dims=dims))
+    for key in ("factor", "low", "high", "original"):
+        with_config(lambda c: mixer(c, 0)["rot"]["scaling"].pop(key))
+    with_config(lambda c: mixer(c, 0)["rot"]["scaling"].update(high=1.0))
+    with_config(lambda c: mixer(c, 2)["left"]["rot"]["scaling"].update(factor=0))
+    for key in ("q_rank", "kv_rank", "rot_dim", "vdim"):
+        with_config(lambda c: mixer(c, 1).pop(key))
+    with_config(lambda c: mixer(c, 1).update(q_rank=0))
+    with_config(lambda c: mixer(c, 2).pop("right"))
+    with_config(lambda c: mixer(c, 2).pop("left"))
+    with_config(lambda c: mixer(c, 2)["right"].update(width=0))
+    with_config(lambda c: c["layers"][0].update(type="latent_attention_2"))
+    with_config(lambda c: c["layers"][0].update(mlp={"kind": "dense", "ff": 8}))
+    with_config(lambda c: c["layers"][0]["mlp"]["router"]["groups"].update(count=3))
+    with_config(lambda c: c["layers"][0]["mlp"]["router"].update(top=5))           # more than the kept groups hold
+
+
+def test_heads_that_may_mix_their_scores(pkg):
+    assert 128 <= pkg.lib.cmlb200_talk_scores_heads() < 1000
 
 
 def test_tensor_file_refusals(pkg, synth, tmp_path):
