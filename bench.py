@@ -395,6 +395,9 @@ def main():
     ap.add_argument("--streams", nargs="?", const="all", default=None, choices=["all", "kernels", "models"],
                     help="instead of the default workload: models with residual streams, chunked attention beside a gated delta rule and grouped routing, "
                          "beside the layered models of equal sizes, and their kernels")
+    ap.add_argument("--loops", nargs="?", const="all", default=None, choices=["all", "kernels", "models"],
+                    help="instead of the default workload: models with looped layers, gated sublayers side by side, talking heads and a minimal recurrence, "
+                         "beside the layered models of equal sizes, and their kernels")
     args = ap.parse_args()
 
     if args.cpu_leg:                                   # child process of run_cpu_leg
@@ -428,6 +431,9 @@ def main():
     if args.layered:
         import bench_layered
         return bench_layered.run(pkg, synth, torch, peaks, ClockSampler(local), args.layered == "kernels", args.layered == "models")
+    if args.loops:
+        import bench_loops
+        return bench_loops.run(pkg, synth, torch, peaks, ClockSampler(local), args.loops == "kernels", args.loops == "models")
     if args.streams:
         import bench_streams
         return bench_streams.run(pkg, synth, torch, peaks, ClockSampler(local), args.streams == "kernels", args.streams == "models")
