@@ -179,6 +179,25 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constant
                         if (m0 + rr < m_end && col < out.n_out)
                             static_cast<__nv_bfloat16*>(out.y)[(size_t)(m0 + rr) * out.ldy + col] = __float2bfloat16_rn(buf[rr * 33 + (lane & 15)]);
                     }
+                } else if (out.form == OUT_ACT) {
+                    if (out.act == CMLB200_ACT_GELU_ERF) {      // decided outside, so that the values' chains overlap
+#pragma unroll
+                        for (int j = 0; j < 32; j++) buf[lane * 33 + j] = gelu_erf_fast(__uint_as_float(v[j]));
+                    } else {
+#pragma unroll
+                        for (int j = 0; j < 32; j++) buf[lane * 33 + j] = unary_act_fast(out.act, __uint_as_float(v[j]));
+                    }
+                    __syncwarp();
+                    const int col = n0 + c0 + 2 * (lane & 15);
+#pragma unroll 4
+                    for (int j = 0; j < 32; j += 2) {
+                        const int rr = j + (lane >> 4);
+                        if (m0 + rr >= m_end || col >= out.n_out) continue;
+                        const float* s = buf + rr * 33 + 2 * (lane & 15);
+                        __nv_bfloat16* d = static_cast<__nv_bfloat16*>(out.y) + (size_t)(m0 + rr) * out.ldy + col;
+                        if (col + 1 < out.n_out) *reinterpret_cast<__nv_bfloat162*>(d) = __floats2bfloat162_rn(s[0], s[1]);
+                        else *d = __float2bfloat16_rn(s[0]);
+                    }
                 } else {
 #pragma unroll
                     for (int j = 0; j < 32; j++) buf[lane * 33 + j] = __uint_as_float(v[j]);
@@ -193,11 +212,6 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constant
 #pragma unroll 8
                         for (int j = 0; j < 32; j++)
                             if (m0 + j < m_end && col < out.n_out) static_cast<float*>(out.y)[(size_t)(m0 + j) * out.ldy + col] = buf[j * 33 + lane] + bias;
-                    } else if (out.form == OUT_ACT) {
-#pragma unroll 8
-                        for (int j = 0; j < 32; j++)
-                            if (m0 + j < m_end && col < out.n_out)
-                                static_cast<__nv_bfloat16*>(out.y)[(size_t)(m0 + j) * out.ldy + col] = __float2bfloat16_rn(unary_act_fast(out.act, buf[j * 33 + lane]));
                     } else {
                         const bool key = col < out.key_cols;
                         const int c = key ? col : col - out.key_cols, per = key ? out.dim : out.vdim, ldo = key ? out.ldk : out.ldy;
@@ -301,6 +315,7 @@ extern "C" int cmlb200_moe_gemm_act(const cmlb200_moe* m, const cmlb200_dense* W
                                     void* stream) {
     CMLB_REQUIRE(m && W && ff > 0 && W->rows == m->experts * ((ff + 15) & ~15) && ldf >= ff, "cmlb200_moe_gemm_act: weight rows do not fit %d outputs", ff);
     CMLB_REQUIRE(act == CMLB200_ACT_SILU || act == CMLB200_ACT_GELU_TANH || act == CMLB200_ACT_GELU_ERF, "cmlb200_moe_gemm_act: activation %d", act);
+    CMLB_REQUIRE(ldf % 2 == 0 && ((uintptr_t)d_f & 3) == 0, "cmlb200_moe_gemm_act: output stride %d", ldf);
     GemmOut out = {};
     out.form = OUT_ACT; out.act = act; out.y = d_f; out.ldy = ldf; out.n_out = ff;
     return gemm_experts(m, W, d_x, ldx, rows, out, "cmlb200_moe_gemm_act", stream);

@@ -16,74 +16,126 @@ namespace {
 
 __device__ __forceinline__ int attn_channels(const cmlb200_attn& a) { return (a.heads + a.kv_heads) * a.dim + a.kv_heads * a.vdim; }
 
-__device__ __forceinline__ void store_pair(float* d, float2 v) { *reinterpret_cast<float2*>(d) = v; }
-__device__ __forceinline__ void store_pair(__half* d, float2 v) {
-    const __half h[2] = {narrow<__half>(v.x), narrow<__half>(v.y)};
-    *reinterpret_cast<uint32_t*>(d) = *reinterpret_cast<const uint32_t*>(h);
+template <int W> struct Cols { float v[W]; };
+template <int W, bool VEC> __device__ __forceinline__ Cols<W> load_cols(const float* s, int have) {
+    Cols<W> x;
+    if constexpr (VEC && W == 4) { const float4 q = *reinterpret_cast<const float4*>(s); x.v[0] = q.x; x.v[1] = q.y; x.v[2] = q.z; x.v[3] = q.w; }
+    else
+#pragma unroll
+        for (int e = 0; e < W; e++) x.v[e] = e < have ? s[e] : 0.f;
+    return x;
+}
+template <int W, bool VEC> __device__ __forceinline__ void store_cols(float* d, const Cols<W>& x, int have) {
+    if constexpr (VEC && W == 4) *reinterpret_cast<float4*>(d) = make_float4(x.v[0], x.v[1], x.v[2], x.v[3]);
+    else
+#pragma unroll
+        for (int e = 0; e < W; e++)
+            if (e < have) d[e] = x.v[e];
+}
+// whole padded heads: every store is aligned
+template <int W> __device__ __forceinline__ void store_padded(float* d, const Cols<W>& x) {
+    if constexpr (W == 4) *reinterpret_cast<float4*>(d) = make_float4(x.v[0], x.v[1], x.v[2], x.v[3]);
+    else *reinterpret_cast<float2*>(d) = make_float2(x.v[0], x.v[1]);
+}
+template <int W> __device__ __forceinline__ void store_padded(__half* d, const Cols<W>& x) {
+    __half h[W];
+#pragma unroll
+    for (int e = 0; e < W; e++) h[e] = narrow<__half>(x.v[e]);
+    if constexpr (W == 4) { uint2 u; memcpy(&u, h, sizeof u); *reinterpret_cast<uint2*>(d) = u; }
+    else { uint32_t u; memcpy(&u, h, sizeof u); *reinterpret_cast<uint32_t*>(d) = u; }
 }
 
-// grid = (rows, parts). Work is counted in pairs of neighbouring entries of a padded head: queries, keys, values. T: taps where
-// they are known (all loads of a pair are then under way together), 0: any number. VEC: heads start at even columns.
-template <typename KV, int T, bool VEC>
+// grid = (groups of R rows, parts). A thread owns W neighbouring entries of a padded head (queries, keys, values in turn) and takes them
+// through the group's rows, whose taps it loads once and whose latest projections it keeps. T: taps where they are known, 0: any
+// number. VEC: heads and rows start at multiples of four columns.
+template <typename KV, int T, bool VEC, int R>
 __global__ void __launch_bounds__(256)
-rotate_append_kernel(const cmlb200_attn a, float* __restrict__ qkv, int ld, const int* __restrict__ row_pos, const int* __restrict__ row_slot, int first, int singles,
-                     KV* __restrict__ q_out) {
-    extern __shared__ float cs[];                      // cosines, then sines, of the row's position
+rotate_append_kernel(const cmlb200_attn a, float* __restrict__ qkv, int ld, const int* __restrict__ row_pos, const int* __restrict__ row_slot, int first, int rows,
+                     int singles, KV* __restrict__ q_out) {
+    constexpr int W = VEC ? 4 : 2;
+    extern __shared__ float cs[];                      // per row cosines, then sines, of its position
+    __shared__ int s_pos[R], s_slot[R], s_near[R], s_at[R];
     dep_wait();
     dep_trigger();
-    const int r = first + blockIdx.x, p = row_pos[r], slot = row_slot[r], half = a.rot_dims / 2, taps = T ? T : a.taps;
-    for (int i = threadIdx.x; i < half; i += 256) sincosf((float)p * a.freq[i], &cs[half + i], &cs[i]);
-    int near = 0;                                      // rows directly in front that belong to the same portion
-    if (r >= singles)
-        while (near < taps - 1 && near < p && r - near - 1 >= singles && row_slot[r - near - 1] == slot) near++;
+    const int r0 = first + blockIdx.x * R, nr = min(R, first + rows - r0), half = a.rot_dims / 2, taps = T ? T : a.taps;
+    for (int i = threadIdx.x; i < nr * half; i += 256) {
+        const int k = i / half, j = i - k * half;
+        sincosf((float)row_pos[r0 + k] * a.freq[j], &cs[k * a.rot_dims + half + j], &cs[k * a.rot_dims + j]);
+    }
+    if ((int)threadIdx.x < nr) {
+        const int r = r0 + threadIdx.x, p = row_pos[r], slot = row_slot[r];
+        int near = 0;                                  // rows directly in front that belong to the same portion
+        if (r >= singles)
+            while (near < taps - 1 && near < p && r - near - 1 >= singles && row_slot[r - near - 1] == slot) near++;
+        s_pos[threadIdx.x] = p;
+        s_slot[threadIdx.x] = slot;
+        s_near[threadIdx.x] = near;
+        s_at[threadIdx.x] = a.block_table[(size_t)slot * a.table_ld + p / a.block_size] * a.block_size + p % a.block_size;
+    }
     __syncthreads();
-    const int channels = attn_channels(a), qp = a.heads * (a.dim_ld / 2), kp = a.kv_heads * (a.dim_ld / 2), vp = a.kv_heads * (a.vdim_ld / 2);
-    float* row = qkv + (size_t)r * ld;
-    float* ring = a.ring + (taps > 0 ? (size_t)slot * taps * channels : 0);
-    const size_t at = (size_t)a.block_table[(size_t)slot * a.table_ld + p / a.block_size] * a.block_size + p % a.block_size;
-    KV* kd = static_cast<KV*>(a.k_pool) + at * a.kv_heads * a.dim_ld;
-    KV* vd = static_cast<KV*>(a.v_pool) + at * a.kv_heads * a.vdim_ld;
-    auto load2 = [&](const float* s, int c, bool two) {
-        if (VEC) return *reinterpret_cast<const float2*>(s + c);
-        return make_float2(s[c], two ? s[c + 1] : 0.f);
-    };
-    auto convolved = [&](int c, bool two) {
-        const float2 now = load2(row, c, two);
-        if (taps <= 0) return now;
-        float2 y = load2(a.conv + (size_t)(taps - 1) * channels, c, two);
-        y.x *= now.x; y.y *= now.y;
-#pragma unroll (T ? T : 1)
-        for (int t = 1; t < taps; t++) {
-            if (t > p) break;
-            const float2 w = load2(a.conv + (size_t)(taps - 1 - t) * channels, c, two);
-            const float2 x = load2(t <= near ? row - (size_t)t * ld : ring + (size_t)((p - t) % taps) * channels, c, two);
-            y.x = fmaf(w.x, x.x, y.x);
-            y.y = fmaf(w.y, x.y, y.y);
+    const int channels = attn_channels(a), qu = a.heads * (a.dim_ld / W), ku = a.kv_heads * (a.dim_ld / W), vu = a.kv_heads * (a.vdim_ld / W);
+    for (int i = blockIdx.y * 256 + threadIdx.x; i < qu + ku + vu; i += gridDim.y * 256) {
+        const bool value = i >= qu + ku, query = i < qu;
+        const int j = value ? i - qu - ku : (query ? i : i - qu), per = (value ? a.vdim_ld : a.dim_ld) / W, h = j / per, d = W * (j - h * per);
+        const int dim = value ? a.vdim : a.dim, c = (value ? (a.heads + a.kv_heads) * a.dim : (query ? 0 : a.heads * a.dim)) + h * dim + d, have = min(W, dim - d);
+        constexpr int TT = T ? T : 1;
+        Cols<W> w[TT];                                 // weight of the token t back
+        if (T && have > 0)
+#pragma unroll
+            for (int t = 0; t < TT; t++) w[t] = load_cols<W, VEC>(a.conv + (size_t)(taps - 1 - t) * channels + c, have);
+        Cols<W> rows_now[R];                           // all under way together
+        if (have > 0)
+#pragma unroll
+            for (int k = 0; k < R; k++)
+                if (k < nr) rows_now[k] = load_cols<W, VEC>(qkv + (size_t)(r0 + k) * ld + c, have);
+#pragma unroll
+        for (int k = 0; k < R; k++) {
+            if (k >= nr) break;
+            const int p = s_pos[k], near = s_near[k], r = r0 + k;
+            float* row = qkv + (size_t)r * ld;
+            float* ring = a.ring + (taps > 0 ? (size_t)s_slot[k] * taps * channels : 0);
+            Cols<W> y;
+#pragma unroll
+            for (int e = 0; e < W; e++) y.v[e] = 0.f;
+            if (have > 0) {
+                const Cols<W> now = rows_now[k];
+                auto before = [&](int t) { return load_cols<W, VEC>(t <= near ? row - (size_t)t * ld + c : ring + (size_t)((p - t) % taps) * channels + c, have); };
+                auto weigh = [&](const Cols<W>& f, const Cols<W>& x) {
+#pragma unroll
+                    for (int e = 0; e < W; e++) y.v[e] = fmaf(f.v[e], x.v[e], y.v[e]);
+                };
+                if constexpr (T > 0) {
+                    weigh(w[0], now);
+#pragma unroll
+                    for (int t = 1; t < T; t++) {
+                        if (t <= near && t <= k) weigh(w[t], rows_now[k >= t ? k - t : 0]);
+                        else if (t <= p) weigh(w[t], before(t));
+                    }
+                } else if (taps > 0) {
+                    weigh(load_cols<W, VEC>(a.conv + (size_t)(taps - 1) * channels + c, have), now);
+                    for (int t = 1; t < taps && t <= p; t++) weigh(load_cols<W, VEC>(a.conv + (size_t)(taps - 1 - t) * channels + c, have), before(t));
+                } else {
+                    y = now;
+                }
+                if (taps > 0 && r < singles) store_cols<W, VEC>(ring + (size_t)(p % taps) * channels + c, now, have);
+            }
+            if (!value) {
+                const float* turn = cs + k * a.rot_dims;
+#pragma unroll
+                for (int e = 0; e < W; e += 2) {
+                    if (d + e >= a.rot_dims) continue;
+                    const float co = turn[(d + e) / 2], si = turn[half + (d + e) / 2], u = y.v[e], v = y.v[e + 1];
+                    y.v[e] = u * co - v * si;
+                    y.v[e + 1] = v * co + u * si;
+                }
+            }
+            if (query && !q_out) {
+                if (have > 0) store_cols<W, VEC>(row + c, y, have);      // nothing lies between the heads there
+                continue;
+            }
+            store_padded<W>(value ? static_cast<KV*>(a.v_pool) + ((size_t)s_at[k] * a.kv_heads + h) * a.vdim_ld + d
+                                  : (query ? q_out + ((size_t)r * a.heads + h) * a.dim_ld + d : static_cast<KV*>(a.k_pool) + ((size_t)s_at[k] * a.kv_heads + h) * a.dim_ld + d), y);
         }
-        if (r < singles) {
-            float* d = ring + (size_t)(p % taps) * channels + c;
-            d[0] = now.x;
-            if (two) d[1] = now.y;
-        }
-        return y;
-    };
-    for (int i = blockIdx.y * 256 + threadIdx.x; i < qp + kp + vp; i += gridDim.y * 256) {
-        const bool value = i >= qp + kp, query = i < qp;
-        const int j = value ? i - qp - kp : (query ? i : i - qp), per = (value ? a.vdim_ld : a.dim_ld) / 2, h = j / per, d = 2 * (j - h * per);
-        const int dim = value ? a.vdim : a.dim, c = (value ? (a.heads + a.kv_heads) * a.dim : (query ? 0 : a.heads * a.dim)) + h * dim + d;
-        float2 y = make_float2(0.f, 0.f);
-        if (d < dim) y = convolved(c, d + 1 < dim);
-        if (!value && d < a.rot_dims) {
-            const float co = cs[d / 2], si = cs[half + d / 2];
-            y = make_float2(y.x * co - y.y * si, y.y * co + y.x * si);
-        }
-        if (query && !q_out) {
-            if (d < dim) row[c] = y.x;
-            if (d + 1 < dim) row[c + 1] = y.y;
-            continue;
-        }
-        KV* o = (value ? vd : (query ? q_out + (size_t)r * a.heads * a.dim_ld : kd)) + (size_t)h * 2 * per + d;
-        store_pair(o, y);
     }
 }
 
@@ -119,18 +171,21 @@ extern "C" int cmlb200_rotate_append(const cmlb200_attn* a, float* d_qkv, int ld
     const int rc = check_rotated(a, ld, who);
     if (rc) return rc;
     CMLB_REQUIRE(a->taps == 0 || d_q_out, "%s: convolved queries go to rows of their own", who);
-    const int pairs = a->heads * (a->dim_ld / 2) + a->kv_heads * (a->dim_ld / 2 + a->vdim_ld / 2), most = (pairs + 255) / 256;
+    const bool vec = a->dim % 4 == 0 && a->vdim % 4 == 0 && ld % 4 == 0 && (((uintptr_t)d_qkv | (uintptr_t)a->conv | (uintptr_t)a->ring | (uintptr_t)d_q_out) & 15) == 0;
+    const int units = (a->heads + a->kv_heads) * (a->dim_ld / (vec ? 4 : 2)) + a->kv_heads * (a->vdim_ld / (vec ? 4 : 2)), most = (units + 255) / 256;
+    const int group = rows >= 64 ? 8 : 1, groups = (rows + group - 1) / group;
     int parts = 1;
-    while (parts < most && parts * rows < 2 * cmlb_num_sms()) parts++;
-    const bool vec = a->dim % 2 == 0 && a->vdim % 2 == 0 && ld % 2 == 0 && (((uintptr_t)d_qkv | (uintptr_t)a->conv | (uintptr_t)a->ring) & 7) == 0;
-    const size_t smem = (size_t)a->rot_dims * 4;
-#define RA_LAUNCH(KV, T, V) CMLB_CUDA(launch_chain(rotate_append_kernel<KV, T, V>, dim3(rows, parts), dim3(256), smem, 1, as_stream(stream), *a, d_qkv, ld, d_row_pos, d_row_slot, first, singles, (KV*)d_q_out))
-#define RA_VEC(KV, T) do { if (vec) RA_LAUNCH(KV, T, true); else RA_LAUNCH(KV, T, false); } while (0)
+    while (parts < most && parts * groups < 4 * cmlb_num_sms()) parts++;
+    const size_t smem = (size_t)group * a->rot_dims * 4;
+#define RA_LAUNCH(KV, T, V, R) CMLB_CUDA(launch_chain(rotate_append_kernel<KV, T, V, R>, dim3(groups, parts), dim3(256), smem, 1, as_stream(stream), *a, d_qkv, ld, d_row_pos, d_row_slot, first, rows, singles, (KV*)d_q_out))
+#define RA_ROWS(KV, T, V) do { if (group == 8) RA_LAUNCH(KV, T, V, 8); else RA_LAUNCH(KV, T, V, 1); } while (0)
+#define RA_VEC(KV, T) do { if (vec) RA_ROWS(KV, T, true); else RA_ROWS(KV, T, false); } while (0)
 #define RA_TAPS(KV) do { if (a->taps == 3) RA_VEC(KV, 3); else if (a->taps == 4) RA_VEC(KV, 4); else RA_VEC(KV, 0); } while (0)
     if (a->cache_dtype == CMLB200_DT_F32) RA_TAPS(float);
     else RA_TAPS(__half);
 #undef RA_TAPS
 #undef RA_VEC
+#undef RA_ROWS
 #undef RA_LAUNCH
     return CMLB200_OK;
 }

@@ -178,7 +178,7 @@ def schedules(lengths, seed=3):
 
 
 TALKING = [(4, 2, 32, 24, 23, 3, 3.0, 16), (3, 3, 13, 7, 1, 4, 1.5, 6), (20, 2, 72, 136, 100, 1, 5.0, 72), (8, 1, 64, 64, 64, 2, 4.0, 32), (2, 2, 128, 128, 65, 3, 6.0, 2),
-           (6, 3, 200, 17, 40, 5, 2.0, 100), (1, 1, 256, 40, 17, 9, 2.0, 30), (64, 8, 16, 24, 70, 4, 3.0, 8), (120, 5, 8, 9, 33, 3, 2.0, 8), (5, 5, 16, 256, 1000, 3, 8.0, 16)]
+           (6, 3, 200, 17, 40, 5, 2.0, 100), (1, 1, 256, 40, 17, 9, 2.0, 30), (64, 8, 16, 24, 70, 4, 3.0, 8), (110, 5, 8, 9, 33, 3, 2.0, 8), (5, 5, 16, 256, 1000, 3, 8.0, 16)]
 WINDOWED = [(4, 2, 32, 24, 23, 0, 0, 16), (3, 3, 13, 7, 1, 0, 0, 6), (20, 2, 72, 136, 100, 0, 0, 72), (8, 1, 64, 64, 64, 0, 0, 32), (2, 2, 128, 128, 65, 0, 0, 2), (6, 3, 200, 256, 40, 0, 0, 100),
             (5, 5, 16, 80, 1000, 0, 0, 16)]
 
