@@ -73,7 +73,7 @@ def clear_groups(z, groups):
     """Whether the groups picked by the sum of their two best sigmoids lead by more than rounding, whatever the row's norm."""
     if not groups or groups["keep"] == groups["count"]:
         return True
-    for scale in (0.1, 0.2, 0.4, 0.8, 1.5):
+    for scale in np.geomspace(0.05, 2.0, 20):
         two = np.sort(zevilorn_oracle.sigmoid(z * scale).reshape(groups["count"], -1), -1)[:, -2:].sum(-1)
         order = np.sort(two)[::-1]
         if order[groups["keep"] - 1] - order[groups["keep"]] < 0.02 * scale:
