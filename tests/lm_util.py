@@ -94,9 +94,10 @@ def steady_routes(synth, rng, cfg, w):
     side = cfg["architecture"] == "Zevilorn"
     if side:
         level = level * 2
-    rows = []
+    rows, tries = [], 0
     while len(rows) < cfg["vocab"]:
-        row = rng.permutation(level)
+        row, tries = rng.permutation(level), tries + 1
+        assert tries < 200 * cfg["vocab"], "no order of levels separates the groups of every layer"
         if not side or all(clear_groups(row[o], cfg["layers"][i]["mlp"]["router"].get("groups")) for i, o in orders.items()):
             rows.append(row)
     w["embed"][:, -n:] = synth.bf16_round(np.stack(rows))[1]
