@@ -36,7 +36,7 @@ __device__ __forceinline__ float2 halves_of(uint64_t y) {
 // grid = (key blocks, 64 / QN, tiles). scores: [tile][heads][64][ld], keys from that of the tile's first row rounded down to 16.
 // WHOLE: dim_ld is a multiple of 32.
 template <int QN, int KN, bool WHOLE>
-__global__ void __launch_bounds__(TT_THREADS)
+__global__ void __launch_bounds__(TT_THREADS, 1)
 talk_tiles_kernel(const cmlb200_attn a, const __half* __restrict__ q, const int4* __restrict__ tiles, float* __restrict__ scores, int ld) {
     extern __shared__ __align__(16) float sc[];        // [heads][QN * KN], then talk transposed and twice over [heads][heads rounded up to 8][2]
     constexpr int QM = QN / 16, KM = KN / 8, PAIRS = QN * KN;
